@@ -51,6 +51,7 @@ typedef struct pi_ctx pi_ctx;
 typedef struct pi_linear pi_linear;
 typedef struct pi_kv_pool pi_kv_pool;
 typedef struct pi_model pi_model;
+typedef struct pi_state_pool pi_state_pool;
 
 /* ---- context --------------------------------------------------------------- */
 
@@ -114,7 +115,7 @@ void pi_ctx_reset_kernel_launches(pi_ctx* ctx);
  * per class, the summed device time in milliseconds and the number of launches.
  * Classes: */
 enum { PI_PROF_GEMV = 0, PI_PROF_GEMM_TC = 1, PI_PROF_ATTENTION = 2, PI_PROF_ROPE_KV = 3, PI_PROF_OTHER = 4,
-       PI_PROF_COLLECTIVE = 5, PI_PROF_CLASSES = 6 };
+       PI_PROF_COLLECTIVE = 5, PI_PROF_RECURRENCE = 6, PI_PROF_CLASSES = 7 };
 pi_status pi_ctx_profile_begin(pi_ctx* ctx);
 pi_status pi_ctx_profile_end(pi_ctx* ctx, double* ms_out /*[PI_PROF_CLASSES]*/, uint64_t* launches_out /*[PI_PROF_CLASSES]*/);
 /* Tuning knobs (the 0/1 ones default on). */
@@ -354,6 +355,88 @@ pi_status pi_model_decode_multi(pi_ctx* ctx, pi_model* model, pi_kv_pool* pool,
 /* Fill the whole pool with N(0, std) values (synthetic KV for benchmarks).
  * No counterpart in the reference. */
 pi_status pi_kv_fill_normal(pi_ctx* ctx, pi_kv_pool* pool, uint64_t seed, float std);
+
+/* ---- layered designs --------------------------------------------------------------
+ * Models whose layers each name a token mixer with sizes of its own.  A pi_model made here is stepped with
+ * pi_model_step like every other model; what its mixers carry from token to token lives in a KV pool (attention) and
+ * in a state pool (recurrences).  No counterpart in the reference. */
+
+enum { PI_MIXER_ATTENTION = 0, PI_MIXER_GLA = 1, PI_MIXER_MLSTM = 2 };
+
+typedef struct {
+  int32_t mixer;
+  int32_t heads, kv_heads; /* kv_heads: attention */
+  int32_t dim, vdim;       /* channels of a query/key and of a value, per head (and per map) */
+  int32_t maps;            /* attention: softmax maps per head, 1 or 2 (differential) */
+  int32_t window;          /* attention: a position sees itself and the window - 1 before it; <= 0: all before it */
+  int32_t rot_dims;        /* attention: leading channels that carry rotary positions (interleaved pairs) */
+  float rot_base, scale, diff;
+  float tau;               /* GLA: log decay = log_sigmoid(z) / tau */
+  float gate_cap;          /* mLSTM: soft cap of both gates */
+  int32_t ff;              /* feed-forward size, 0: the layer has none */
+} pi_layer_config;
+
+typedef struct {
+  int32_t width, vocab_size, num_layers;
+  float norm_eps;
+  int32_t compute;         /* PI_BF16: bf16 projections and KV, f32 accumulation; PI_F32: f32 throughout */
+  int32_t max_rows;        /* tokens one step can take */
+  const pi_layer_config* layers;
+} pi_layered_config;
+
+typedef struct {
+  const char* name;
+  int32_t kind;            /* PI_BF16 or PI_F32 */
+  int64_t rows, cols;      /* vectors: rows = length, cols = 1; scalars 1 x 1 */
+  const void* data;        /* host */
+} pi_named_tensor;
+
+/* Layers pre- and post-normalised by Dynamic Tanh, gelu-gated feed-forward, tied embedding.  Tensors are looked up by
+ * their checkpoint names; matrices are bf16. */
+pi_status pi_model_create_layered(pi_ctx* ctx, const pi_layered_config* cfg, const pi_named_tensor* tensors, int n_tensors, pi_model** out);
+/* Random matrices N(0, std) generated on the device; gla_rank = rank of the GLA decay's low-rank input. */
+pi_status pi_model_create_layered_synthetic(pi_ctx* ctx, const pi_layered_config* cfg, int gla_rank, uint64_t seed, float std, pi_model** out);
+int pi_model_vocab_size(const pi_model* model);
+/* Bytes of recurrent state per sequence; 0: the model has none and needs no state pool. */
+size_t pi_model_state_bytes(const pi_model* model);
+/* Blocks of the KV pool hold block_size tokens of every attention layer, whatever the layers' geometry. */
+pi_status pi_kv_pool_create_for_model(pi_ctx* ctx, const pi_model* model, int num_blocks, int block_size, pi_kv_pool** out);
+
+/* One slot of f32 state per live sequence.  A slot needs no clearing: a sequence that starts at position 0 starts from
+ * the zero state. */
+pi_status pi_state_pool_create(pi_ctx* ctx, const pi_model* model, int num_slots, pi_state_pool** out);
+void pi_state_pool_destroy(pi_state_pool* pool);
+size_t pi_state_pool_bytes(const pi_state_pool* pool);
+/* Duplicate a sequence's state (a forked sequence). */
+pi_status pi_state_copy_slot(pi_ctx* ctx, pi_state_pool* pool, int32_t src, int32_t dst);
+
+/* A ragged batch: sequence i brings n_tokens[i] >= 1 consecutive tokens from position start_pos[i] on, portions of
+ * prompts beside single decoded tokens.  Rows are numbered through in this order. */
+typedef struct {
+  int32_t n_seqs;
+  const uint32_t* tokens;        /* all portions, one after the other */
+  const int32_t* n_tokens;       /* [n_seqs] */
+  const int32_t* start_pos;      /* [n_seqs] */
+  const int32_t* block_tables;   /* [n_seqs][max_blocks] */
+  int32_t max_blocks;
+  const int32_t* table_lens;     /* [n_seqs] */
+  const int32_t* state_slots;    /* [n_seqs], NULL for a model without state */
+  int32_t n_out;                 /* rows whose result is wanted */
+  const int32_t* out_rows;       /* [n_out], rows in increasing order */
+} pi_step_batch;
+
+/* Run one step for any model of this library.  logits_host_or_null: [n_out][vocab]; argmax_host_or_null: [n_out]
+ * greedy ids.  The logits of a row depend on its own sequence only. */
+pi_status pi_model_step(pi_ctx* ctx, pi_model* model, pi_kv_pool* pool, pi_state_pool* state_or_null, const pi_step_batch* batch,
+                        float* logits_host_or_null, uint32_t* argmax_host_or_null);
+/* n_steps greedy steps of sequences that bring one token each, without returning to the host in between (as
+ * pi_model_decode_multi): out_tokens_host receives [n_steps][n_seqs].  The tables must map every position written. */
+pi_status pi_model_step_multi(pi_ctx* ctx, pi_model* model, pi_kv_pool* pool, pi_state_pool* state_or_null, const pi_step_batch* batch,
+                              int n_steps, uint32_t* out_tokens_host);
+/* The residual stream behind layer `layer` of the last pi_model_step of a layered model ([rows][width] f32), for
+ * numerical tests: ask for it with pi_model_trace_layers(model, 1) before the step. */
+pi_status pi_model_trace_layers(pi_ctx* ctx, pi_model* model, int on);
+pi_status pi_model_read_layer(pi_ctx* ctx, const pi_model* model, int layer, int rows, float* x_host_out);
 
 #ifdef __cplusplus
 }

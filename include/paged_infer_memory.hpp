@@ -71,6 +71,32 @@ class BlockAllocator {
   std::vector<uint32_t> refs_;
 };
 
+// Fixed set of equal slots, one per live sequence, for what a recurrent model carries from token to token.
+class SlotAllocator {
+ public:
+  explicit SlotAllocator(size_t total = 0) : used_(total, false) {
+    for (size_t i = 0; i < total; ++i) free_.push_back((int32_t)i);
+  }
+  std::optional<int32_t> take() {   // first in, first out, like the blocks
+    if (free_.empty()) return std::nullopt;
+    const int32_t s = free_.front();
+    free_.pop_front();
+    used_[s] = true;
+    return s;
+  }
+  void give_back(int32_t s) {
+    if (s < 0 || (size_t)s >= used_.size() || !used_[s]) throw std::logic_error("state slot " + std::to_string(s) + " is not in use");
+    used_[s] = false;
+    free_.push_back(s);
+  }
+  size_t available() const { return free_.size(); }
+  size_t total() const { return used_.size(); }
+
+ private:
+  std::deque<int32_t> free_;
+  std::vector<bool> used_;
+};
+
 // One logical block of a sequence: the physical block, the hash of the whole prefix up to and including it
 // (complete prompt blocks only) and whether its KV came out of the prefix cache.
 struct BlockSlot {
@@ -211,6 +237,19 @@ class KvCacheManager {
     cache_enabled_ = enabled;
     return *this;
   }
+  // Models that carry recurrent state: every sequence also holds one of n state slots.  A cached block has the keys and
+  // values of its tokens but not the state behind them, so prompts then never resume from the prefix cache.
+  KvCacheManager& with_state_slots(size_t n) {
+    slots_ = SlotAllocator(n);
+    return *this;
+  }
+  std::optional<int32_t> state_slot(size_t seq_id) const {
+    auto it = seqs_.find(seq_id);
+    return it == seqs_.end() || it->second.slot < 0 ? std::nullopt : std::optional<int32_t>(it->second.slot);
+  }
+  size_t total_state_slots() const { return slots_.total(); }
+  size_t free_state_slots() const { return slots_.available(); }
+  bool can_hold_another() const { return slots_.total() == 0 || slots_.available() > 0; }
   size_t block_size() const { return alloc_.block_size; }
   size_t available_blocks() const { return alloc_.available_blocks(); }
   size_t total_blocks() const { return alloc_.total_blocks(); }
@@ -230,7 +269,9 @@ class KvCacheManager {
 
   // Map blocks for a prompt, reusing cached KV for its longest known prefix; nullopt when the prompt cannot be
   // housed even after evicting cold cache entries (the rejected admission leaves no references behind).
-  std::optional<Admission> admit(size_t seq_id, const std::vector<uint32_t>& tokens, uint64_t now_tick) {
+  // `reuse` false: every token is to be run, so nothing is taken from the cache.
+  std::optional<Admission> admit(size_t seq_id, const std::vector<uint32_t>& tokens, uint64_t now_tick, bool reuse = true) {
+    if (!can_hold_another()) return std::nullopt;
     const size_t bs = alloc_.block_size;
     const size_t total = std::max<size_t>((tokens.size() + bs - 1) / bs, 1);
     const size_t full = tokens.size() / bs;          // a trailing partial block has no stable identity yet
@@ -242,7 +283,7 @@ class KvCacheManager {
     }
     Admission adm;
     size_t reused = 0;
-    if (cache_enabled_)
+    if (cache_enabled_ && reuse && slots_.total() == 0)
       for (uint64_t h : hashes) {                      // stop at the first miss: later blocks have another history
         const auto hit = cache_.lookup(h);
         if (!hit) break;
@@ -264,14 +305,14 @@ class KvCacheManager {
     adm.reused_blocks = reused;
     adm.allocated_blocks = to_allocate;
     cache_.record_tokens_saved(adm.cached_tokens);
-    seqs_[seq_id] = SequenceAlloc{adm.block_table.physical_blocks(), now_tick};
+    seqs_[seq_id] = SequenceAlloc{adm.block_table.physical_blocks(), now_tick, take_slot()};
     return adm;
   }
 
   // Publish the prompt blocks this sequence computed (hash known, not themselves cache hits); returns how many
   // entries were added.
   size_t publish_prompt_blocks(const BlockTable& table) {
-    if (!cache_enabled_) return 0;
+    if (!cache_enabled_ || slots_.total() > 0) return 0;
     size_t published = 0;
     for (const auto& s : table.slots())
       if (s.hash && !s.cached) {
@@ -290,19 +331,21 @@ class KvCacheManager {
     if (!b) return false;
     table.append_block(*b);
     auto it = seqs_.find(seq_id);
-    if (it == seqs_.end()) it = seqs_.emplace(seq_id, SequenceAlloc{{}, now_tick}).first;
+    if (it == seqs_.end()) it = seqs_.emplace(seq_id, SequenceAlloc{{}, now_tick, -1}).first;
     it->second.blocks.push_back(*b);
     return true;
   }
 
-  // The child maps every one of the parent's blocks; no data moves.
+  // The child maps every one of the parent's blocks; no data moves.  (Its state slot, if there are any, is a new one that
+  // the caller fills from the parent's.)
   BlockTable fork(const BlockTable& parent, size_t child_seq, uint64_t now_tick) {
+    if (!can_hold_another()) throw std::logic_error("no state slot left for a forked sequence");
     BlockTable child;
     for (const auto& s : parent.slots()) {
       alloc_.incref(s.block);
       child.append_slot(s);
     }
-    seqs_[child_seq] = SequenceAlloc{child.physical_blocks(), now_tick};
+    seqs_[child_seq] = SequenceAlloc{child.physical_blocks(), now_tick, take_slot()};
     return child;
   }
 
@@ -337,6 +380,7 @@ class KvCacheManager {
     auto it = seqs_.find(seq_id);
     if (it == seqs_.end()) return;
     for (PhysicalBlock b : it->second.blocks) alloc_.free(b);
+    if (it->second.slot >= 0) slots_.give_back(it->second.slot);
     seqs_.erase(it);
   }
 
@@ -368,14 +412,20 @@ class KvCacheManager {
   struct SequenceAlloc {
     std::vector<PhysicalBlock> blocks;
     uint64_t last_used_tick;
+    int32_t slot = -1;
   };
+  int32_t take_slot() {   // -1 for a model without state; callers have checked can_hold_another()
+    const auto s = slots_.take();
+    return s ? *s : -1;
+  }
   bool record(size_t seq_id, PhysicalBlock b, uint64_t now_tick) {
     auto it = seqs_.find(seq_id);
-    if (it == seqs_.end()) it = seqs_.emplace(seq_id, SequenceAlloc{{}, now_tick}).first;
+    if (it == seqs_.end()) it = seqs_.emplace(seq_id, SequenceAlloc{{}, now_tick, -1}).first;
     it->second.blocks.push_back(b);
     return true;
   }
   BlockAllocator alloc_;
+  SlotAllocator slots_;
   std::map<size_t, SequenceAlloc> seqs_;
   PrefixCache cache_;
   bool cache_enabled_ = true;

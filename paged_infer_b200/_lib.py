@@ -22,7 +22,7 @@ PI_ERR_UNSUPPORTED = -6
 
 PI_SPLIT_NONE, PI_SPLIT_COLUMN, PI_SPLIT_ROW = 0, 1, 2
 PI_F32, PI_INT8, PI_BF16 = 0, 1, 2
-PROF_CLASSES = ("gemv", "gemm_tc", "attention", "rope_kv", "other", "collective")
+PROF_CLASSES = ("gemv", "gemm_tc", "attention", "rope_kv", "other", "collective", "recurrence")
 PI_OPT_TENSOR_GEMM, PI_OPT_CUDA_GRAPH, PI_OPT_PDL, PI_OPT_GEMV_MAX_M, PI_OPT_ATTN_TMA, PI_OPT_FUSE_PLANES, PI_OPT_ATTN_SHARED = 1, 2, 3, 4, 5, 6, 7
 PI_OPT_PEER_SPIN_LIMIT = 8
 PI_OPT_TP_PUSH = 9
@@ -58,6 +58,25 @@ class ModelWeightsC(C.Structure):
     _fields_ = [("token_embeddings_bf16", C.c_void_p), ("final_norm", C.c_void_p),
                 ("attention_norm", C.POINTER(C.c_void_p)), ("ffn_norm", C.POINTER(C.c_void_p)),
                 ("projections", C.POINTER(TensorC)), ("lm_head", TensorC)]
+
+
+class LayerConfigC(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "maps", "window", "rot_dims")] + \
+               [(n, C.c_float) for n in ("rot_base", "scale", "diff", "tau", "gate_cap")] + [("ff", C.c_int32)]
+
+
+class LayeredConfigC(C.Structure):
+    _fields_ = [("width", C.c_int32), ("vocab_size", C.c_int32), ("num_layers", C.c_int32), ("norm_eps", C.c_float), ("compute", C.c_int32),
+                ("max_rows", C.c_int32), ("layers", C.POINTER(LayerConfigC))]
+
+
+class NamedTensorC(C.Structure):
+    _fields_ = [("name", C.c_char_p), ("kind", C.c_int32), ("rows", C.c_int64), ("cols", C.c_int64), ("data", C.c_void_p)]
+
+
+class StepBatchC(C.Structure):
+    _fields_ = [("n_seqs", C.c_int32), ("tokens", C.c_void_p), ("n_tokens", C.c_void_p), ("start_pos", C.c_void_p), ("block_tables", C.c_void_p),
+                ("max_blocks", C.c_int32), ("table_lens", C.c_void_p), ("state_slots", C.c_void_p), ("n_out", C.c_int32), ("out_rows", C.c_void_p)]
 
 
 _P = C.c_void_p
@@ -123,6 +142,19 @@ SIGNATURES = {
     "pi_model_prefill": (_I, [_P, _P, _P, _P, _I, _I, _P, _I, _I, _P, _P]),
     "pi_model_decode_multi": (_I, [_P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _P]),
     "pi_kv_fill_normal": (_I, [_P, _P, C.c_uint64, C.c_float]),
+    "pi_model_create_layered": (_I, [_P, C.POINTER(LayeredConfigC), C.POINTER(NamedTensorC), _I, _PP]),
+    "pi_model_create_layered_synthetic": (_I, [_P, C.POINTER(LayeredConfigC), _I, C.c_uint64, C.c_float, _PP]),
+    "pi_model_vocab_size": (_I, [_P]),
+    "pi_model_state_bytes": (_SZ, [_P]),
+    "pi_kv_pool_create_for_model": (_I, [_P, _P, _I, _I, _PP]),
+    "pi_state_pool_create": (_I, [_P, _P, _I, _PP]),
+    "pi_state_pool_destroy": (None, [_P]),
+    "pi_state_pool_bytes": (_SZ, [_P]),
+    "pi_state_copy_slot": (_I, [_P, _P, C.c_int32, C.c_int32]),
+    "pi_model_step": (_I, [_P, _P, _P, _P, C.POINTER(StepBatchC), _P, _P]),
+    "pi_model_step_multi": (_I, [_P, _P, _P, _P, C.POINTER(StepBatchC), _I, _P]),
+    "pi_model_trace_layers": (_I, [_P, _P, _I]),
+    "pi_model_read_layer": (_I, [_P, _P, _I, _I, _P]),
 }
 
 _lib = None

@@ -16,7 +16,7 @@ import numpy as np
 
 from . import _lib
 from ._lib import PI_BF16, PI_F32, PI_INT8, PI_SPLIT_COLUMN, PI_SPLIT_NONE, PI_SPLIT_ROW, PiError, check
-from .loader import QUANT_F32, QUANT_INT8, HostWeights, LlamaConfig
+from .loader import QUANT_F32, QUANT_INT8, HostWeights, LayeredConfig, LlamaConfig
 
 
 def _f32(a) -> np.ndarray:
@@ -501,9 +501,153 @@ class PagedAttention:
         return out
 
 
+# ---- ragged steps, for every model ------------------------------------------------------------------
+
+class StatePool:
+    """One slot of recurrent state per live sequence (``pi_state_pool``)."""
+
+    def __init__(self, ctx: Context, model, num_slots: int):
+        self.ctx, self.num_slots = ctx, num_slots
+        h = C.c_void_p()
+        check(_lib.lib().pi_state_pool_create(ctx.handle, model.handle, num_slots, C.byref(h)), ctx.handle)
+        self.handle = h
+
+    def close(self):
+        if getattr(self, "handle", None) and _lib is not None:
+            _lib.lib().pi_state_pool_destroy(self.handle)
+            self.handle = None
+
+    __del__ = close
+
+    def bytes(self) -> int:
+        return int(_lib.lib().pi_state_pool_bytes(self.handle))
+
+    def copy_slot(self, src: int, dst: int):
+        check(_lib.lib().pi_state_copy_slot(self.ctx.handle, self.handle, src, dst), self.ctx.handle)
+
+
+class _Steps:
+    """What every model offers beside its own calls: pools of its geometry and ragged steps (``pi_model_step``)."""
+
+    def vocab_size(self) -> int:
+        return int(_lib.lib().pi_model_vocab_size(self.handle))
+
+    def state_bytes(self) -> int:
+        return int(_lib.lib().pi_model_state_bytes(self.handle))
+
+    def kv_pool(self, num_blocks: int, block_size: int) -> "KvCache":
+        """A KV pool for this model, whatever the geometry of its attention layers."""
+        pool = KvCache.__new__(KvCache)
+        pool.ctx, pool.layout = self.ctx, None
+        h = C.c_void_p()
+        check(_lib.lib().pi_kv_pool_create_for_model(self.ctx.handle, self.handle, num_blocks, block_size, C.byref(h)), self.ctx.handle)
+        pool.handle = h
+        return pool
+
+    def state_pool(self, num_slots: int) -> StatePool:
+        return StatePool(self.ctx, self, num_slots)
+
+    @staticmethod
+    def _batch(portions, starts, block_tables, slots, out_rows):
+        keep = [np.ascontiguousarray(np.concatenate([np.asarray(p, np.uint32).reshape(-1) for p in portions])),
+                _i32([len(p) for p in portions]), _i32(starts)]
+        mat, lens, mb = pack_block_tables(block_tables)
+        keep += [mat, _i32(lens), _i32(slots) if slots is not None else None, _i32(out_rows)]
+        b = _lib.StepBatchC(len(portions), _ptr(keep[0]), _ptr(keep[1]), _ptr(keep[2]), _ptr(mat), mat.shape[1] if mb else 0, _ptr(keep[4]),
+                            _ptr(keep[5]) if slots is not None else None, keep[6].size, _ptr(keep[6]) if keep[6].size else None)
+        return b, keep
+
+    def step(self, portions, starts, block_tables, kv_cache: "KvCache", state: StatePool | None = None, slots=None, out_rows=None,
+             want_logits: bool = True, want_argmax: bool = False):
+        """One batch of portions (lists of token ids) that begin at ``starts``; results of ``out_rows`` (default: the last token of
+        every portion), rows numbered through."""
+        if out_rows is None:
+            out_rows = np.cumsum([len(p) for p in portions]) - 1
+        b, keep = self._batch(portions, starts, block_tables, slots, out_rows)
+        n = b.n_out
+        logits = np.empty((n, self.vocab_size()), np.float32) if want_logits else None
+        ids = np.empty(n, np.uint32) if want_argmax else None
+        check(_lib.lib().pi_model_step(self.ctx.handle, self.handle, kv_cache.handle, state.handle if state else None, C.byref(b),
+                                       _ptr(logits) if want_logits else None, _ptr(ids) if want_argmax else None), self.ctx.handle)
+        if want_logits and want_argmax:
+            return logits, ids
+        return logits if want_logits else ids
+
+    def step_multi(self, tokens, positions, block_tables, kv_cache: "KvCache", n_steps: int, state: StatePool | None = None, slots=None) -> np.ndarray:
+        """``n_steps`` greedy steps of single tokens without host round trips; token ids [n_steps, B]."""
+        b, keep = self._batch([[t] for t in tokens], positions, block_tables, slots, [])
+        out = np.empty((n_steps, len(tokens)), np.uint32)
+        check(_lib.lib().pi_model_step_multi(self.ctx.handle, self.handle, kv_cache.handle, state.handle if state else None, C.byref(b), n_steps,
+                                             _ptr(out)), self.ctx.handle)
+        return out
+
+
+class LayeredModel(_Steps):
+    """A layered design on the device (``pi_model_create_layered``).  ``tensors``: checkpoint name -> array (bf16 bits or f32);
+    ``compute``: "bfloat16" or "float32"; ``max_rows``: tokens one step can take."""
+
+    COMPUTE = {"bfloat16": PI_BF16, "float32": PI_F32}
+
+    def __init__(self, ctx: Context, config: LayeredConfig, tensors: dict, compute: str = "bfloat16", max_rows: int = 64):
+        self.ctx, self.config, self.max_batch = ctx, config, max_rows
+        cfg = self._config(config, compute, max_rows)
+        keep, named = [], (_lib.NamedTensorC * len(tensors))()
+        n = 0
+        for name, t in tensors.items():
+            a = np.ascontiguousarray(t)
+            if a.dtype not in (np.uint16, np.float32):
+                continue   # integer tables: none in the designs built here
+            rows, cols = a.shape if a.ndim == 2 else (a.size, 1)
+            keep.append(a)
+            named[n] = _lib.NamedTensorC(name.encode(), PI_BF16 if a.dtype == np.uint16 else PI_F32, rows, cols, _ptr(a))
+            n += 1
+        h = C.c_void_p()
+        check(_lib.lib().pi_model_create_layered(ctx.handle, C.byref(cfg), named, n, C.byref(h)), ctx.handle)
+        self.handle = h
+
+    @classmethod
+    def _config(cls, config: LayeredConfig, compute: str, max_rows: int) -> _lib.LayeredConfigC:
+        layers = (_lib.LayerConfigC * len(config.layers))(*[
+            _lib.LayerConfigC(l.mixer, l.heads, l.kv_heads, l.dim, l.vdim, l.maps, 0 if l.window is None else l.window, l.rot_dims, l.rot_base,
+                              l.scale, l.diff, l.tau, l.gate_cap, l.ff) for l in config.layers])
+        cfg = _lib.LayeredConfigC(config.width, config.vocab_size, len(config.layers), config.norm_eps, cls.COMPUTE[compute], max_rows, layers)
+        cfg._layers = layers
+        return cfg
+
+    @classmethod
+    def synthetic(cls, ctx: Context, config: LayeredConfig, seed: int, std: float = 0.02, compute: str = "bfloat16", max_rows: int = 64,
+                  gla_rank: int = 16) -> "LayeredModel":
+        self = cls.__new__(cls)
+        self.ctx, self.config, self.max_batch = ctx, config, max_rows
+        cfg = cls._config(config, compute, max_rows)
+        h = C.c_void_p()
+        check(_lib.lib().pi_model_create_layered_synthetic(ctx.handle, C.byref(cfg), gla_rank, seed, std, C.byref(h)), ctx.handle)
+        self.handle = h
+        return self
+
+    def close(self):
+        if getattr(self, "handle", None) and _lib is not None:
+            _lib.lib().pi_model_destroy(self.handle)
+            self.handle = None
+
+    __del__ = close
+
+    def weight_bytes(self) -> int:
+        return int(_lib.lib().pi_model_weight_bytes(self.handle))
+
+    def trace_layers(self, on: bool = True):
+        check(_lib.lib().pi_model_trace_layers(self.ctx.handle, self.handle, int(on)), self.ctx.handle)
+
+    def read_layer(self, layer: int, rows: int) -> np.ndarray:
+        """Residual stream behind a layer in the last step, [rows, width]."""
+        out = np.empty((rows, self.config.width), np.float32)
+        check(_lib.lib().pi_model_read_layer(self.ctx.handle, self.handle, layer, rows, _ptr(out)), self.ctx.handle)
+        return out
+
+
 # ---- model.rs: forward ---------------------------------------------------------------------------
 
-class LlamaWeights:
+class LlamaWeights(_Steps):
     """``LlamaWeights`` + its forward entry points (src/model.rs:380-386, :585-1255) on the device.
 
     ``quantization`` follows the reference loader: ``"int8"`` quantises the seven

@@ -21,6 +21,8 @@ OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libpaged_infer_cuda.so")
 HOST_SRC = os.path.join(HERE, "host", "pi_host_shim.cpp")
 HOST_LIB = os.path.join(HERE, "libpaged_infer_host.so")
+ENGINE_SRC = os.path.join(HERE, "host", "pi_engine_shim.cpp")
+ENGINE_LIB = os.path.join(HERE, "libpaged_infer_engine.so")
 INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 
 NVCC_FLAGS = [
@@ -80,20 +82,30 @@ def build(verbose: bool = False, force: bool = False, ptxas_info: bool = False) 
             sys.stderr.write(r.stdout + r.stderr)
             raise RuntimeError("linking libpaged_infer_cuda.so failed")
     build_host()
+    build_engine()
     return LIB
+
+
+def _gxx(src: str, lib: str, deps, link=()) -> str:
+    if _newer(lib, deps):
+        gxx = "/usr/bin/g++" if os.path.exists("/usr/bin/g++") else (shutil.which("g++") or "g++")
+        r = subprocess.run([gxx, "-std=c++17", "-O2", "-Wall", "-Wextra", "-fPIC", "-shared", src, "-o", lib, *link],
+                           capture_output=True, text=True)
+        if r.returncode != 0:
+            sys.stderr.write(r.stdout + r.stderr)
+            raise RuntimeError(f"building {os.path.basename(lib)} failed")
+    return lib
 
 
 def build_host() -> str:
     """``libpaged_infer_host.so``: the C ABI over the host-side block bookkeeping (g++ only, no CUDA)."""
-    deps = [HOST_SRC, os.path.join(INCLUDE, "paged_infer_memory.hpp")]
-    if _newer(HOST_LIB, deps):
-        gxx = "/usr/bin/g++" if os.path.exists("/usr/bin/g++") else (shutil.which("g++") or "g++")
-        r = subprocess.run([gxx, "-std=c++17", "-O2", "-Wall", "-Wextra", "-fPIC", "-shared", HOST_SRC, "-o", HOST_LIB],
-                           capture_output=True, text=True)
-        if r.returncode != 0:
-            sys.stderr.write(r.stdout + r.stderr)
-            raise RuntimeError("building libpaged_infer_host.so failed")
-    return HOST_LIB
+    return _gxx(HOST_SRC, HOST_LIB, [HOST_SRC, os.path.join(INCLUDE, "paged_infer_memory.hpp")])
+
+
+def build_engine() -> str:
+    """``libpaged_infer_engine.so``: the C ABI over the engine loop; calls ``libpaged_infer_cuda.so`` beside it."""
+    deps = [ENGINE_SRC] + [os.path.join(INCLUDE, n) for n in ("paged_infer_memory.hpp", "paged_infer_engine.hpp", "paged_infer_cuda.h")]
+    return _gxx(ENGINE_SRC, ENGINE_LIB, deps, ["-L" + HERE, "-lpaged_infer_cuda", "-Wl,-rpath,$ORIGIN"])
 
 
 if __name__ == "__main__":

@@ -6,7 +6,7 @@
 #include <algorithm>
 #include <new>
 
-#include "pi_common.cuh"
+#include "pi_layered.cuh"
 
 namespace {
 thread_local std::string g_create_error;
@@ -504,6 +504,27 @@ void pi_kv_pool_destroy(pi_kv_pool* pool) {
   delete pool;
 }
 
+pi_status pi_kv_pool_create_for_model(pi_ctx* ctx, const pi_model* model, int num_blocks, int block_size, pi_kv_pool** out) {
+  PI_ENTER(ctx);
+  PI_REQUIRE(ctx, model && out, "null pointer");
+  *out = nullptr;
+  PI_REQUIRE(ctx, num_blocks > 0 && block_size > 0, "KV layout fields must be positive");
+  pi_kv_layout L;
+  const pi_layered* layered = pi_model_layered(model, &L);
+  L.num_blocks = num_blocks;
+  L.block_size = block_size;
+  if (!layered) return pi_kv_pool_create(ctx, &L, out);
+  pi_kv_pool* pool = new (std::nothrow) pi_kv_pool();
+  if (!pool) return pi_fail(ctx, PI_ERR_OOM, "host allocation failed");
+  const pi_status s = pi_layered_kv_regions(ctx, layered, num_blocks, block_size, pool);
+  if (s != PI_OK) {
+    pi_kv_pool_destroy(pool);
+    return s;
+  }
+  *out = pool;
+  return PI_OK;
+}
+
 size_t pi_kv_pool_bytes(const pi_kv_pool* pool) { return pool ? pool->floats * sizeof(float) : 0; }
 
 pi_status pi_kv_copy_block(pi_ctx* ctx, pi_kv_pool* pool, int32_t src, int32_t dst) {
@@ -518,6 +539,7 @@ pi_status pi_kv_copy_block(pi_ctx* ctx, pi_kv_pool* pool, int32_t src, int32_t d
 pi_status pi_kv_fill_normal(pi_ctx* ctx, pi_kv_pool* pool, uint64_t seed, float std) {
   PI_ENTER(ctx);
   PI_REQUIRE(ctx, pool, "null pool");
+  PI_REQUIRE(ctx, pool->regions.empty(), "this call is for pools of one uniform layout");
   PI_TRY(pi_launch_fill_normal(ctx, pool->data, pool->floats, seed, 0xCAC4Eull, 0, std));
   PI_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
   return PI_OK;
@@ -526,6 +548,7 @@ pi_status pi_kv_fill_normal(pi_ctx* ctx, pi_kv_pool* pool, uint64_t seed, float 
 pi_status pi_kv_upload(pi_ctx* ctx, pi_kv_pool* pool, const float* cache_host) {
   PI_ENTER(ctx);
   PI_REQUIRE(ctx, pool && cache_host, "null pointer");
+  PI_REQUIRE(ctx, pool->regions.empty(), "this call is for pools of one uniform layout");
   PI_TRY(pi_reserve(ctx, &ctx->staging_in, pool->floats * sizeof(float)));
   PI_CUDA(ctx, cudaMemcpyAsync(ctx->staging_in.ptr, cache_host, pool->floats * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
   PI_TRY(pi_launch_kv_relayout(ctx, pool, static_cast<float*>(ctx->staging_in.ptr), false));
@@ -536,6 +559,7 @@ pi_status pi_kv_upload(pi_ctx* ctx, pi_kv_pool* pool, const float* cache_host) {
 pi_status pi_kv_download(pi_ctx* ctx, const pi_kv_pool* pool, float* cache_host_out) {
   PI_ENTER(ctx);
   PI_REQUIRE(ctx, pool && cache_host_out, "null pointer");
+  PI_REQUIRE(ctx, pool->regions.empty(), "this call is for pools of one uniform layout");
   PI_TRY(pi_reserve(ctx, &ctx->staging_out, pool->floats * sizeof(float)));
   PI_TRY(pi_launch_kv_relayout(ctx, pool, static_cast<float*>(ctx->staging_out.ptr), true));
   PI_CUDA(ctx, cudaMemcpyAsync(cache_host_out, ctx->staging_out.ptr, pool->floats * sizeof(float), cudaMemcpyDeviceToHost, ctx->stream));
@@ -546,6 +570,7 @@ pi_status pi_kv_download(pi_ctx* ctx, const pi_kv_pool* pool, float* cache_host_
 static pi_status kv_token_io(pi_ctx* ctx, const pi_kv_pool* pool, int layer, int32_t block, int tok, float* k, float* v,
                              bool write) {
   PI_REQUIRE(ctx, pool && k && v, "null pointer");
+  PI_REQUIRE(ctx, pool->regions.empty(), "this call is for pools of one uniform layout");
   const pi_kv_layout& L = pool->L;
   PI_REQUIRE(ctx, layer >= 0 && layer < L.num_layers && block >= 0 && block < L.num_blocks && tok >= 0 && tok < L.block_size,
              "KV address (layer %d, block %d, token %d) out of range", layer, block, tok);
@@ -595,6 +620,7 @@ pi_status pi_paged_attention(pi_ctx* ctx, const pi_kv_pool* pool, int layer, int
                              const int32_t* start_host, int B) {
   PI_ENTER(ctx);
   PI_REQUIRE(ctx, pool && q_dev && out_dev && table_lens_host && pos_host && start_host, "null pointer");
+  PI_REQUIRE(ctx, pool->regions.empty(), "this call is for pools of one uniform layout");
   PI_REQUIRE(ctx, block_tables_host || max_blocks == 0, "null block tables");
   if (B == 0) return PI_OK;
   PI_REQUIRE(ctx, B > 0, "negative batch");
@@ -612,6 +638,7 @@ pi_status pi_paged_attention_host(pi_ctx* ctx, const pi_kv_pool* pool, int layer
                                   int B) {
   PI_ENTER(ctx);
   PI_REQUIRE(ctx, pool && q_host && out_host, "null pointer");
+  PI_REQUIRE(ctx, pool->regions.empty(), "this call is for pools of one uniform layout");
   if (B == 0) return PI_OK;
   PI_REQUIRE(ctx, B > 0 && num_heads > 0, "bad batch / head count");
   const size_t row = (size_t)num_heads * pool->L.head_dim, bytes = (size_t)B * row * sizeof(float);

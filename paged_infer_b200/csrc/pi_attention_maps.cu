@@ -1,0 +1,188 @@
+// Windowed attention with one or two softmax maps per head over the same values (differential attention), reading the
+// paged KV pool.
+//
+//   score_j = scale (q_j . k_j)           j = map, over the keys t - window < s <= t
+//   a_j     = softmax(score_j) V
+//   out     = a_1                                             (one map)
+//   o = a_1 - lambda a_2;  out = out_scale o / rms(o)          (two maps)
+//
+// Kernels: maps_rope_kv_kernel rotates q and k and writes k and v into the pool; maps_attn_plain_kernel is the f32
+// path (any sizes, one warp per row and head).
+#include <math.h>
+
+#include <algorithm>
+
+#include "pi_layered.cuh"
+
+namespace {
+
+struct RopeKvParams {
+  float* qkv;
+  size_t stride;
+  int heads, kv_heads, maps, dim, vdim, rot_dims;
+  const float *rope_cos, *rope_sin;
+  void* base;
+  int dp, vp, block_size;
+  const int32_t *row_seq, *row_pos, *lens, *tables;
+  int max_blocks;
+};
+
+// CTA per row.  Work item: two adjacent channels of a q or k vector of one map (a rotation pair, rot_dims is even), or
+// one channel of v.  Pool rows are padded with zeros up to dp / vp.
+template <typename T>
+__global__ void __launch_bounds__(256) maps_rope_kv_kernel(const RopeKvParams p) {
+  const int row = blockIdx.x;
+  const int seq = p.row_seq[row], pos = p.row_pos[row];
+  const int lb = pos / p.block_size, off = pos % p.block_size;
+  const bool mapped = lb < p.lens[seq];
+  const int pb = mapped ? p.tables[(size_t)seq * p.max_blocks + lb] : 0;
+  pi_grid_dependency_wait();
+  float* x = p.qkv + (size_t)row * p.stride;
+  const int nq = p.heads * p.maps, nk = p.kv_heads * p.maps, half = p.rot_dims >> 1;
+  const int pairs = (p.dp + 1) >> 1;     // dp >= dim, the pad is written too
+  const float* cs = p.rope_cos + (size_t)pos * half;
+  const float* sn = p.rope_sin + (size_t)pos * half;
+  const size_t tile = (size_t)p.block_size * (p.maps * p.dp + p.vp);
+  for (int i = threadIdx.x; i < (nq + nk) * pairs; i += blockDim.x) {
+    const int vec = i / pairs, j = i - vec * pairs, d = 2 * j;
+    const bool is_q = vec < nq;
+    if (is_q && j >= half) continue;     // q stays where it is
+    if (!is_q && !mapped) continue;
+    float* v = x + (size_t)vec * p.dim;  // k vectors follow the q vectors
+    float a = d < p.dim ? v[d] : 0.f, c = d + 1 < p.dim ? v[d + 1] : 0.f;
+    if (j < half) {
+      const float na = a * cs[j] - c * sn[j], nc = c * cs[j] + a * sn[j];
+      a = na;
+      c = nc;
+    }
+    if (is_q) {
+      v[d] = a;
+      v[d + 1] = c;
+    } else {
+      const int kv = vec - nq, g = kv / p.maps, m = kv - g * p.maps;
+      T* dst = static_cast<T*>(p.base) + ((size_t)pb * p.kv_heads + g) * tile + (size_t)off * p.maps * p.dp + (size_t)m * p.dp;
+      dst[d] = pi_from_f32<T>(a);
+      dst[d + 1] = pi_from_f32<T>(c);
+    }
+  }
+  if (!mapped) return;
+  const float* vsrc = x + (size_t)(nq + nk) * p.dim;
+  for (int i = threadIdx.x; i < p.kv_heads * p.vp; i += blockDim.x) {
+    const int g = i / p.vp, e = i - g * p.vp;
+    T* dst = static_cast<T*>(p.base) + ((size_t)pb * p.kv_heads + g) * tile + (size_t)p.block_size * p.maps * p.dp + (size_t)off * p.vp;
+    dst[e] = pi_from_f32<T>(e < p.vdim ? vsrc[(size_t)g * p.vdim + e] : 0.f);
+  }
+}
+
+struct MapsParams {
+  const float* q;
+  size_t stride;
+  void* out;
+  size_t out_stride;
+  const void* base;
+  int heads, kv_heads, maps, dim, vdim, dp, vp, block_size, window;
+  float scale, eps, lambda, out_scale;
+  const int32_t *row_seq, *row_pos, *lens, *tables;
+  int max_blocks;
+};
+
+// One CTA of 4 warps per (row, head): the warps take every fourth key and merge; lanes hold the channels.  f32
+// throughout, any sizes (smem: q, per-warp accumulators of both maps).
+constexpr int kPlainWarps = 4;
+template <typename T, typename O>
+__global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const MapsParams p) {
+  extern __shared__ float sm[];
+  const int row = blockIdx.y, head = blockIdx.x, g = head / (p.heads / p.kv_heads);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int seq = p.row_seq[row], pos = p.row_pos[row], len = p.lens[seq];
+  const int32_t* table = p.tables + (size_t)seq * p.max_blocks;
+  const int nm = p.maps, DP = p.dp;
+  float* sq = sm;                                   // [maps][dim]
+  float* acc = sm + nm * p.dim;                     // [warps][maps][vdim]
+  __shared__ float s_m[kPlainWarps][2], s_l[kPlainWarps][2], s_red[kPlainWarps];
+  pi_grid_dependency_wait();
+  for (int i = tid; i < nm * p.dim; i += blockDim.x) sq[i] = p.q[(size_t)row * p.stride + (size_t)head * nm * p.dim + i];
+  float* my = acc + (size_t)warp * nm * p.vdim;
+  for (int i = lane; i < nm * p.vdim; i += 32) my[i] = 0.f;
+  __syncthreads();
+  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const size_t tile = (size_t)p.block_size * (nm * DP + p.vp);
+  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  for (int t = lo + warp; t <= pos; t += kPlainWarps) {
+    const int lb = t / p.block_size, off = t - lb * p.block_size;
+    if (lb >= len) break;
+    const T* kt = static_cast<const T*>(p.base) + ((size_t)table[lb] * p.kv_heads + g) * tile;
+    const T* vt = kt + (size_t)p.block_size * nm * DP + (size_t)off * p.vp;
+    kt += (size_t)off * nm * DP;
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      if (m >= nm) break;
+      float d = 0.f;
+      for (int i = lane; i < p.dim; i += 32) d = fmaf(sq[m * p.dim + i], pi_to_f32(kt[m * DP + i]), d);
+      const float s = pi_warp_sum(d) * p.scale;
+      const float mn = fmaxf(mx[m], s), keep = expf(mx[m] - mn), w = expf(s - mn);
+      mx[m] = mn;
+      l[m] = l[m] * keep + w;
+      for (int i = lane; i < p.vdim; i += 32) my[m * p.vdim + i] = my[m * p.vdim + i] * keep + w * pi_to_f32(vt[i]);
+    }
+  }
+  if (lane == 0)
+    for (int m = 0; m < nm; ++m) {
+      s_m[warp][m] = mx[m];
+      s_l[warp][m] = l[m];
+    }
+  __syncthreads();
+  float f[2][kPlainWarps];
+  for (int m = 0; m < nm; ++m) {
+    float M = -INFINITY, L = 0.f;
+    for (int w = 0; w < kPlainWarps; ++w) M = fmaxf(M, s_m[w][m]);
+    for (int w = 0; w < kPlainWarps; ++w) L += s_m[w][m] == -INFINITY ? 0.f : s_l[w][m] * expf(s_m[w][m] - M);
+    for (int w = 0; w < kPlainWarps; ++w) f[m][w] = s_m[w][m] == -INFINITY ? 0.f : expf(s_m[w][m] - M) / L;
+  }
+  float sq_sum = 0.f;
+  for (int e = tid; e < p.vdim; e += blockDim.x) {
+    float a[2] = {0.f, 0.f};
+    for (int m = 0; m < nm; ++m)
+      for (int w = 0; w < kPlainWarps; ++w) a[m] += acc[((size_t)w * nm + m) * p.vdim + e] * f[m][w];
+    const float o = nm == 2 ? a[0] - p.lambda * a[1] : a[0];
+    sq_sum = fmaf(o, o, sq_sum);
+    acc[e] = o;   // warp 0, map 0: this thread is the only one that reads column e
+  }
+  float r = 1.0f;
+  if (nm == 2) {
+    sq_sum = pi_warp_sum(sq_sum);
+    if (lane == 0) s_red[warp] = sq_sum;
+    __syncthreads();
+    float t = 0.f;
+    for (int w = 0; w < kPlainWarps; ++w) t += s_red[w];
+    r = p.out_scale / sqrtf(t / (float)p.vdim + p.eps);
+  }
+  O* o = static_cast<O*>(p.out) + (size_t)row * p.out_stride + (size_t)head * p.vdim;
+  for (int e = tid; e < p.vdim; e += blockDim.x) o[e] = pi_from_f32<O>(acc[e] * r);
+}
+
+}  // namespace
+
+pi_status pi_launch_maps_rope_kv(pi_ctx* ctx, const pi_maps_attention& a, const pi_kv_view& kv, float* qkv, size_t stride,
+                                 const pi_seq_batch& b) {
+  pi_prof_scope prof(ctx, PI_PROF_ROPE_KV);
+  RopeKvParams p = {qkv, stride, a.heads, a.kv_heads, a.maps, a.dim, a.vdim, a.rot_dims, a.rope_cos, a.rope_sin, kv.base, kv.dp, kv.vp,
+                    kv.block_size, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks};
+  PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, kv.kind == PI_BF16 ? maps_rope_kv_kernel<__nv_bfloat16> : maps_rope_kv_kernel<float>,
+                                  dim3(b.rows), dim3(256), 0, 1, p));
+  return PI_OK;
+}
+
+pi_status pi_launch_maps_attention(pi_ctx* ctx, const pi_maps_attention& a, const pi_kv_view& kv, const float* qkv, size_t stride,
+                                   void* out, size_t out_stride, int out_kind, const pi_seq_batch& b) {
+  pi_prof_scope prof(ctx, PI_PROF_ATTENTION);
+  MapsParams p = {qkv, stride, out, out_stride, kv.base, a.heads, a.kv_heads, a.maps, a.dim, a.vdim, kv.dp, kv.vp, kv.block_size,
+                  a.window, a.scale, a.eps, a.lambda, a.out_scale, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks};
+  const size_t smem = sizeof(float) * ((size_t)a.maps * a.dim + (size_t)kPlainWarps * a.maps * a.vdim);
+  PI_REQUIRE(ctx, smem <= 48 * 1024, "attention heads of %d / %d channels are too wide", a.dim, a.vdim);
+  auto k = kv.kind == PI_BF16 ? (out_kind == PI_BF16 ? maps_attn_plain_kernel<__nv_bfloat16, __nv_bfloat16> : maps_attn_plain_kernel<__nv_bfloat16, float>)
+                              : (out_kind == PI_BF16 ? maps_attn_plain_kernel<float, __nv_bfloat16> : maps_attn_plain_kernel<float, float>);
+  // grid.y is limited to 65535 rows, far above any step
+  PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(a.heads, b.rows), dim3(kPlainWarps * 32), smem, 1, p));
+  return PI_OK;
+}

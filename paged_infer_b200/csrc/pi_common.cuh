@@ -149,7 +149,28 @@ struct pi_linear {
 enum pi_epilogue {
   PI_EPI_STORE = 0,     // out[m][r] = v
   PI_EPI_ADD = 1,       // out[m][r] += v           (residual add)
-  PI_EPI_SWIGLU = 2     // rows interleaved gate/up: out[m][r/2] = silu(v[2i]) * v[2i+1]
+  PI_EPI_SWIGLU = 2,    // rows interleaved gate/up: out[m][r/2] = silu(v[2i]) * v[2i+1]
+  PI_EPI_GEGLU = 3,     // the same with the tanh form of gelu
+  PI_EPI_DYT_RESIDUAL = 4   // x[m][r] += dyt(post, v); h[m][r] = dyt(next, x[m][r])   (pi_dyt_residual)
+};
+
+// Dynamic Tanh, a normalisation without statistics: tanh(alpha v) w + b, element by element.  Because it needs no row
+// sum, it folds into whatever kernel produces its input.
+struct pi_dyt {
+  float alpha = 0.f;
+  const float* w = nullptr;   // null: identity
+  const float* b = nullptr;
+};
+
+// The residual update of a layer that is normalised before and after each sublayer, as the epilogue of the
+// projection v that ends the sublayer: the sum stays in f32, and the input of the next sublayer comes out of the same
+// pass.  h is f32 on the CUDA-core path and bf16 on the tensor-core path; null: not wanted.
+struct pi_dyt_residual {
+  float* x = nullptr;
+  size_t x_stride = 0;
+  pi_dyt post, next;
+  void* h = nullptr;
+  size_t h_stride = 0;
 };
 
 // An activation matrix in the form the tensor-core GEMM consumes: three bf16 planes whose sum is the f32 value
@@ -205,8 +226,15 @@ struct pi_linear_args {
   // (peer memory of the other tensor-parallel ranks).
   float* out_also[8] = {};
   int n_out_also = 0;
+  // bf16 weights on the tensor cores (pi_gemm_bf16.cu): x as bf16 with row stride x_stride.  GEGLU then stores bf16 to
+  // `out_bf16`; a plain store is f32 as elsewhere.
+  const __nv_bfloat16* x_bf16 = nullptr;
+  __nv_bfloat16* out_bf16 = nullptr;
+  const pi_dyt_residual* residual = nullptr;   // PI_EPI_DYT_RESIDUAL
 };
 
+// tcgen05 GEMM for bf16 weights and bf16 activations with f32 accumulation (a.x_bf16; any shape).
+pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args& a);
 // CUDA-core dequant GEMV/GEMM (any shape, any M).
 pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args& a);
 // tcgen05 tensor-core GEMM for int8 weights (returns PI_ERR_UNSUPPORTED when the shape does not fit).
@@ -236,10 +264,19 @@ pi_status pi_launch_quantize(pi_ctx* ctx, const float* w_dev, size_t w_ld, size_
 // Device layout: [layer][block][kv_head][k|v][token][head_dim] f32, so one
 // (block, kv_head) K tile is block_size*head_dim contiguous floats with its V
 // tile right behind it, and one block of one layer is still one contiguous span.
+// A pool whose attention layers differ in geometry (layered designs) keeps one region per layer instead:
+// [block][kv_head]{ K: [token][maps * dp] | V: [token][vp] }, f32 or bf16, rows padded with zeros to dp / vp.
+struct pi_kv_region {
+  size_t offset = 0;       // bytes from the pool's base
+  int kv_heads = 0, maps = 0, dp = 0, vp = 0;
+  size_t block_bytes = 0;
+};
 struct pi_kv_pool {
   pi_kv_layout L;
   float* data = nullptr;
   size_t floats = 0;
+  std::vector<pi_kv_region> regions;   // empty: the uniform f32 layout above
+  int kind = PI_F32;                   // element type of the regions
   __host__ __device__ size_t block_stride() const { return (size_t)L.block_size * L.num_kv_heads * 2 * L.head_dim; }
 };
 
@@ -293,6 +330,10 @@ pi_status pi_launch_attention_flat(pi_ctx* ctx, const pi_kv_pool* pool, int laye
 pi_status pi_launch_attention(pi_ctx* ctx, const pi_kv_pool* pool, int layer, int num_heads, const float* q,
                               size_t q_stride, float* out, size_t out_stride, const pi_attn_batch& batch,
                               pi_act_planes* emit = nullptr, bool* emitted = nullptr);
+
+// ---- layered designs (pi_layered.cu) ---------------------------------------------------
+struct pi_layered;
+struct pi_state_pool;
 
 // ---- glue ----------------------------------------------------------------------------
 pi_status pi_launch_embed(pi_ctx* ctx, const uint16_t* table_bf16, int vocab, int hidden, const uint32_t* tokens_dev,
@@ -368,6 +409,18 @@ __device__ __forceinline__ float pi_warp_max(float v) {
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
   return v;
 }
+__device__ __forceinline__ float pi_dyt_apply(const pi_dyt& n, float v, int i) {
+  return n.w ? fmaf(tanhf(n.alpha * v), __ldg(n.w + i), __ldg(n.b + i)) : v;
+}
+// z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
+__device__ __forceinline__ float pi_gelu_tanh(float z) {
+  return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * fmaf(0.044715f * z * z, z, z)));
+}
+__device__ __forceinline__ float pi_sigmoid(float z) {   // no overflow on either side
+  const float e = expf(-fabsf(z));
+  return (z >= 0.f ? 1.0f : e) / (1.0f + e);
+}
+__device__ __forceinline__ float pi_log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float pi_bf16_bits_to_f32(uint16_t b) { return __uint_as_float(((uint32_t)b) << 16); }
 // Programmatic dependent launch: wait for the producer grid's memory, and allow
 // the consumer grid to start its prologue.

@@ -417,11 +417,9 @@ __global__ void __launch_bounds__(256) act_split_kernel(const float* __restrict_
   }
 }
 
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+}  // namespace
 
-EncodeTiledFn encode_tiled() {
+pi_tc::EncodeTiledFn pi_tc::encode_tiled_fn() {
   static EncodeTiledFn fn = nullptr;
   static bool tried = false;
   if (!tried) {
@@ -434,6 +432,10 @@ EncodeTiledFn encode_tiled() {
   }
   return fn;
 }
+
+namespace {
+
+inline EncodeTiledFn encode_tiled() { return encode_tiled_fn(); }
 
 
 // Dynamic shared memory of an instantiation: the pipeline stages, the receive area of the cluster reduction (PUSH: up

@@ -339,6 +339,11 @@ __device__ __forceinline__ float act_row_factor(const GemmParams& p, int m) {
 
 
 // ---- host side (pi_gemm_tc.cu) ----------------------------------------------------------------------------------
+typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+// cuTensorMapEncodeTiled, looked up once; null when the driver does not offer it.
+EncodeTiledFn encode_tiled_fn();
 // Activation rows per CTA tile: 16, 32 or 64.
 int pick_bn(int M);
 // Everything a launch of one projection needs: the parameter block and the tensor map over the activation planes

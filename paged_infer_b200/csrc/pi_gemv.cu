@@ -19,6 +19,7 @@
 // f32 twins (reference src/math.rs:93-275, :473-512) and math::quantize_rows_i8
 // (:456-469).
 #include <algorithm>
+#include <type_traits>
 
 #include "pi_common.cuh"
 
@@ -81,6 +82,7 @@ struct Widen<float> {
 };
 
 struct GemvParams {
+  pi_dyt_residual res;   // PI_EPI_DYT_RESIDUAL
   const void* W;
   const float* scales;
   const float* x;
@@ -315,10 +317,11 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
     if (npair < npairs) load_group(wnxt, npair, nkg);
     // residual add: the value this lane will add to is requested before the arithmetic of the pair's last group
     float old_out = 0.f;
-    if (EPI == PI_EPI_ADD && !ROPE && ks == 0 && kg + KS >= ngroups) {
+    if ((EPI == PI_EPI_ADD || EPI == PI_EPI_DYT_RESIDUAL) && !ROPE && ks == 0 && kg + KS >= ngroups) {
       const int r = lane / MB, m = lane - r * MB;
       if (r < kRows && m < mcount && pair * kRows + r < p.N)
-        old_out = p.out[(size_t)(m0 + m) * p.out_stride + pair * kRows + r];
+        old_out = EPI == PI_EPI_ADD ? p.out[(size_t)(m0 + m) * p.out_stride + pair * kRows + r]
+                                    : p.res.x[(size_t)(m0 + m) * p.res.x_stride + pair * kRows + r];
     }
     float sc[kRows] = {1.0f, 1.0f};   // the rows' scales, requested likewise
     if (kg + KS >= ngroups && ks == 0) {
@@ -430,15 +433,29 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
             }
           }
         }
-      } else if (EPI == PI_EPI_SWIGLU) {
+      } else if (EPI == PI_EPI_SWIGLU || EPI == PI_EPI_GEGLU) {
 #pragma unroll
         for (int m = 0; m < MB; ++m) {
           if (lane == m && m < mcount && row0 + 1 < p.N) {
             const float rf = row_factor(m);
             const float g = tot[0][m] * sc[0] * rf, u = tot[1][m] * sc[1] * rf;
-            p.out[(size_t)(m0 + m) * p.out_stride + (row0 >> 1)] = (g / (1.0f + expf(-g))) * u;
+            p.out[(size_t)(m0 + m) * p.out_stride + (row0 >> 1)] =
+                EPI == PI_EPI_GEGLU ? pi_gelu_tanh(g) * u : (g / (1.0f + expf(-g))) * u;
           }
         }
+      } else if (EPI == PI_EPI_DYT_RESIDUAL) {
+#pragma unroll
+        for (int r = 0; r < kRows; ++r)
+#pragma unroll
+          for (int m = 0; m < MB; ++m) {
+            if (lane == r * MB + m && m < mcount && row0 + r < p.N) {
+              const float v = tot[r][m] * sc[r] * row_factor(m);
+              const float xn = old_out + pi_dyt_apply(p.res.post, v, row0 + r);
+              p.res.x[(size_t)(m0 + m) * p.res.x_stride + row0 + r] = xn;
+              if (p.res.h)
+                static_cast<float*>(p.res.h)[(size_t)(m0 + m) * p.res.h_stride + row0 + r] = pi_dyt_apply(p.res.next, xn, row0 + r);
+            }
+          }
       } else {
 #pragma unroll
         for (int r = 0; r < kRows; ++r)
@@ -466,20 +483,28 @@ template <typename WT, int MB>
 cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, dim3 grid, int threads, size_t smem,
                           bool pdl, int ksplit) {
   void (*k)(const GemvParams) = nullptr;
+  constexpr bool kFloatW = !std::is_same<WT, int8_t>::value;   // layered designs keep bf16 weights
 #define PI_PICK(E, Nrm) k = gemv_kernel<WT, MB, E, Nrm, false>
   if (ksplit == kSplitWarps) {   // few long rows (pi_launch_gemv asks for it only without norm, rotary embedding, SwiGLU)
     if (epi == PI_EPI_ADD) k = gemv_kernel<WT, MB, PI_EPI_ADD, false, false, kSplitWarps>;
-    else k = gemv_kernel<WT, MB, PI_EPI_STORE, false, false, kSplitWarps>;
+    else if (epi == PI_EPI_DYT_RESIDUAL) {
+      if constexpr (kFloatW) k = gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false, kSplitWarps>;
+    } else k = gemv_kernel<WT, MB, PI_EPI_STORE, false, false, kSplitWarps>;
   } else if (epi == PI_EPI_STORE && p.rope_hd) {   // fused [q;k;v] projection: own instantiation, the others stay as they are
     if (norm) k = gemv_kernel<WT, MB, PI_EPI_STORE, true, true>; else k = gemv_kernel<WT, MB, PI_EPI_STORE, false, true>;
   } else if (epi == PI_EPI_STORE) {
     if (norm) PI_PICK(PI_EPI_STORE, true); else PI_PICK(PI_EPI_STORE, false);
   } else if (epi == PI_EPI_ADD) {
     if (norm) PI_PICK(PI_EPI_ADD, true); else PI_PICK(PI_EPI_ADD, false);
+  } else if (epi == PI_EPI_GEGLU) {
+    if constexpr (kFloatW) PI_PICK(PI_EPI_GEGLU, false);
+  } else if (epi == PI_EPI_DYT_RESIDUAL) {
+    if constexpr (kFloatW) PI_PICK(PI_EPI_DYT_RESIDUAL, false);
   } else {
     if (norm) PI_PICK(PI_EPI_SWIGLU, true); else PI_PICK(PI_EPI_SWIGLU, false);
   }
 #undef PI_PICK
+  if (!k) return cudaErrorInvalidDeviceFunction;
   static pi_smem_grant granted;  // per instantiation of this launcher; attribute calls are slow
   if (smem > std::max(granted.of(ctx), (size_t)48 * 1024)) {
     // the launcher covers several kernel variants: raise the limit on all of them at once
@@ -491,6 +516,13 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
                     gemv_kernel<WT, MB, PI_EPI_STORE, false, false, kSplitWarps>}) {
       cudaError_t e = cudaFuncSetAttribute(kk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return e;
+    }
+    if constexpr (kFloatW) {
+      for (auto kk : {gemv_kernel<WT, MB, PI_EPI_GEGLU, false, false>, gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false>,
+                      gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false, kSplitWarps>}) {
+        cudaError_t e = cudaFuncSetAttribute(kk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return e;
+      }
     }
     granted.of(ctx) = smem;
   }
@@ -572,7 +604,10 @@ bool pi_gemv_can_rope(const pi_ctx* ctx, const pi_linear* lin, const pi_linear_a
 
 pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args& a) {
   PI_REQUIRE(ctx, a.M >= 1, "projection batch must be at least 1");
-  PI_REQUIRE(ctx, a.epi != PI_EPI_SWIGLU || lin->rows % 2 == 0, "SwiGLU epilogue needs interleaved gate/up rows");
+  const bool glu = a.epi == PI_EPI_SWIGLU || a.epi == PI_EPI_GEGLU;
+  PI_REQUIRE(ctx, !glu || lin->rows % 2 == 0, "a gated epilogue needs interleaved gate/up rows");
+  PI_REQUIRE(ctx, a.epi < PI_EPI_GEGLU || (lin->kind != PI_INT8 && !a.norm_weight), "this epilogue is built for bf16 and f32 weights");
+  PI_REQUIRE(ctx, a.epi != PI_EPI_DYT_RESIDUAL || (a.residual && a.residual->x), "the residual epilogue needs its operands");
   if (lin->rows == 0) return PI_OK;
   int mb = a.M >= 4 ? 4 : a.M >= 2 ? 2 : 1;
   while (mb > 1 && (size_t)mb * lin->ld * sizeof(float) > ctx->smem_optin - 2048) mb >>= 1;
@@ -592,7 +627,7 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
   // Sets of three warps share a row pair instead: three times the loads in flight.
   int ksplit = 1;
   const size_t row_bytes = lin->ld * (lin->kind == PI_INT8 ? 1 : lin->kind == PI_BF16 ? 2 : 4);
-  if (!a.norm_weight && !a.rope && a.epi != PI_EPI_SWIGLU && row_bytes > (size_t)(kSplitWarps - 1) * kSteps * 512 &&
+  if (!a.norm_weight && !a.rope && !glu && row_bytes > (size_t)(kSplitWarps - 1) * kSteps * 512 &&
       npairs * 2 <= max_ctas * 8) {
     ksplit = kSplitWarps;
     warps = 2 * kSplitWarps;
@@ -613,6 +648,7 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
   p.K = (int)lin->cols;
   p.M = a.M;
   p.eps = a.norm_eps;
+  if (a.residual) p.res = *a.residual;
   p.err_flag = ctx->dev_err;
   p.rope_hd = 0;
   if (a.rope) {

@@ -10,6 +10,8 @@
 // KvLayout::copy_block (src/memory/layout.rs:82-96).
 #include <math.h>
 
+#include <algorithm>
+
 #include "pi_common.cuh"
 
 namespace {
@@ -350,6 +352,15 @@ pi_status pi_launch_argmax(pi_ctx* ctx, const float* logits, size_t stride, int 
 }
 
 pi_status pi_launch_copy_block(pi_ctx* ctx, pi_kv_pool* pool, int src, int dst) {
+  if (!pool->regions.empty()) {   // one region per attention layer, blocks of whole 16-byte groups
+    for (const pi_kv_region& g : pool->regions) {
+      const size_t floats = g.block_bytes / sizeof(float);
+      const unsigned n = (unsigned)std::min<size_t>(64, (floats / 4 + 255) / 256);
+      copy_block_kernel<<<dim3(n, 1), 256, 0, ctx->stream>>>(pool->data + g.offset / sizeof(float), 0, floats, src, dst);
+      PI_CHECK_LAUNCH(ctx);
+    }
+    return PI_OK;
+  }
   const size_t bs = pool->block_stride();
   const size_t layer_stride = bs * pool->L.num_blocks;
   unsigned chunks = (unsigned)((bs / 4 + 255) / 256);

@@ -20,10 +20,16 @@
 #include <algorithm>
 #include <new>
 
-#include "pi_common.cuh"
+#include "pi_layered.cuh"
+#include "pi_load.cuh"
+
+using pi_load::build_linear;
+using pi_load::Piece;
+using pi_load::Source;
 
 struct pi_model {
-  pi_model_config cfg;
+  pi_layered* layered = nullptr;   // a layered design: everything below is unused
+  pi_model_config cfg = {};
   int hd = 0, heads_local = 0, kv_heads_local = 0, inter_local = 0, vocab_local = 0;
   uint16_t* embed = nullptr;
   float* final_norm = nullptr;
@@ -53,15 +59,6 @@ struct pi_model {
 namespace {
 
 size_t esize(int kind) { return kind == PI_INT8 ? 1 : kind == PI_BF16 ? 2 : 4; }
-
-struct Source {
-  const pi_tensor* host = nullptr;  // host tensor, or
-  bool synthetic = false;           // device-generated N(0, std)
-  uint64_t seed = 0, stream_id = 0;
-  float std = 0.02f;
-  int kind = PI_F32;                // synthetic: kind AFTER load (PI_INT8 or PI_BF16)
-  size_t rows = 0, cols = 0;
-};
 
 // Load rows [src_r0, src_r0 + nrows) x cols [c0, c0 + dst->cols) of a source into
 // dst rows dst_r0, dst_r0 + step, ...  Whole rows are quantised before the
@@ -146,14 +143,9 @@ int loaded_kind(const Source& s) {
   return s.host->kind;
 }
 
-// A local (per-rank) matrix whose rows are slices of one or more sources.
-struct Piece {
-  Source src;
-  size_t src_r0, nrows;  // rows taken from the source
-  size_t dst_r0, step;   // where they land
-};
+}  // namespace
 
-pi_status build_linear(pi_ctx* ctx, const std::vector<Piece>& pieces, size_t local_rows, size_t local_cols, size_t c0,
+pi_status pi_load::build_linear(pi_ctx* ctx, const std::vector<Piece>& pieces, size_t local_rows, size_t local_cols, size_t c0,
                        pi_linear** out) {
   const int kind = loaded_kind(pieces[0].src);
   for (const Piece& p : pieces) PI_REQUIRE(ctx, loaded_kind(p.src) == kind, "projections fused into one matrix must share a kind");
@@ -168,6 +160,8 @@ pi_status build_linear(pi_ctx* ctx, const std::vector<Piece>& pieces, size_t loc
   for (const Piece& p : pieces) PI_TRY(load_rows(ctx, lin, p.dst_r0, p.step, p.src, p.src_r0, p.nrows, c0));
   return PI_OK;
 }
+
+namespace {
 
 pi_status alloc_f(pi_ctx* ctx, float** p, size_t n) {
   PI_CUDA(ctx, cudaMalloc(p, std::max<size_t>(n, 1) * sizeof(float)));
@@ -521,6 +515,7 @@ pi_status fetch_results(pi_ctx* ctx, pi_model* m, int rows, float* logits_host, 
 }
 
 pi_status check_pool(pi_ctx* ctx, const pi_model* m, const pi_kv_pool* pool) {
+  PI_REQUIRE(ctx, !m->layered, "a layered model is stepped with pi_model_step / pi_model_step_multi");
   PI_REQUIRE(ctx, pool != nullptr, "null KV pool");
   PI_REQUIRE(ctx, pool->L.num_layers == m->cfg.num_hidden_layers && pool->L.num_kv_heads == m->kv_heads_local &&
                       pool->L.head_dim == m->hd,
@@ -627,8 +622,55 @@ pi_status pi_model_create_synthetic(pi_ctx* ctx, const pi_model_config* cfg, uin
   return PI_OK;
 }
 
+static pi_status make_layered(pi_ctx* ctx, const pi_layered_config* cfg, const pi_named_tensor* tensors, int n, int gla_rank, uint64_t seed,
+                              float std, pi_model** out) {
+  pi_model* m = new (std::nothrow) pi_model();
+  if (!m) return pi_fail(ctx, PI_ERR_OOM, "host allocation failed");
+  const pi_status s = pi_layered_create(ctx, cfg, tensors, n, gla_rank, seed, std, &m->layered);
+  if (s != PI_OK) {
+    delete m;
+    return s;
+  }
+  m->capacity = pi_layered_max_rows(m->layered);
+  *out = m;
+  return PI_OK;
+}
+
+pi_status pi_model_create_layered(pi_ctx* ctx, const pi_layered_config* cfg, const pi_named_tensor* tensors, int n_tensors, pi_model** out) {
+  PI_ENTER(ctx);
+  PI_REQUIRE(ctx, cfg && tensors && n_tensors > 0 && out, "null pointer");
+  *out = nullptr;
+  for (int i = 0; i < n_tensors; ++i)
+    PI_REQUIRE(ctx, tensors[i].name && tensors[i].data && (tensors[i].kind == PI_BF16 || tensors[i].kind == PI_F32) && tensors[i].rows > 0 && tensors[i].cols > 0,
+               "tensor %d is incomplete", i);
+  return make_layered(ctx, cfg, tensors, n_tensors, 0, 0, 0.f, out);
+}
+
+pi_status pi_model_create_layered_synthetic(pi_ctx* ctx, const pi_layered_config* cfg, int gla_rank, uint64_t seed, float std, pi_model** out) {
+  PI_ENTER(ctx);
+  PI_REQUIRE(ctx, cfg && out, "null pointer");
+  *out = nullptr;
+  return make_layered(ctx, cfg, nullptr, 0, gla_rank, seed, std, out);
+}
+
+int pi_model_vocab_size(const pi_model* m) { return !m ? 0 : m->layered ? pi_layered_vocab(m->layered) : m->cfg.vocab_size; }
+size_t pi_model_state_bytes(const pi_model* m) { return m && m->layered ? pi_layered_state_floats(m->layered) * sizeof(float) : 0; }
+
+pi_status pi_model_trace_layers(pi_ctx* ctx, pi_model* m, int on) {
+  PI_ENTER(ctx);
+  PI_REQUIRE(ctx, m && m->layered, "only layered models trace their layers");
+  return pi_layered_trace(ctx, m->layered, on);
+}
+
+pi_status pi_model_read_layer(pi_ctx* ctx, const pi_model* m, int layer, int rows, float* x_host_out) {
+  PI_ENTER(ctx);
+  PI_REQUIRE(ctx, m && m->layered, "only layered models trace their layers");
+  return pi_layered_read_layer(ctx, m->layered, layer, rows, x_host_out);
+}
+
 void pi_model_destroy(pi_model* m) {
   if (!m) return;
+  pi_layered_destroy(m->layered);
   if (m->step_exec) cudaGraphExecDestroy(m->step_exec);
   for (auto* v : {&m->qkv, &m->wo, &m->gate_up, &m->down})
     for (pi_linear* l : *v) pi_linear_destroy(l);
@@ -643,7 +685,7 @@ void pi_model_destroy(pi_model* m) {
   delete m;
 }
 
-size_t pi_model_weight_bytes(const pi_model* m) { return m ? m->weight_bytes : 0; }
+size_t pi_model_weight_bytes(const pi_model* m) { return !m ? 0 : m->layered ? pi_layered_weight_bytes(m->layered) : m->weight_bytes; }
 int pi_model_max_batch(const pi_model* m) { return m ? m->capacity : 0; }
 
 pi_status pi_model_decode_batch_rows(pi_ctx* ctx, pi_model* m, pi_kv_pool* pool, const uint32_t* tokens_host,
@@ -843,4 +885,68 @@ pi_status pi_model_prefill(pi_ctx* ctx, pi_model* m, pi_kv_pool* pool, const uin
   return pi_ctx_synchronize(ctx);
 }
 
+// The ragged step of a uniform model: every token is an entry of its own in one batched forward, the portions of a
+// sequence sharing its table (all K/V writes of a layer precede its attention, so a portion is causal).
+static pi_status uniform_step(pi_ctx* ctx, pi_model* m, pi_kv_pool* pool, const pi_step_batch* in, float* logits_host, uint32_t* argmax_host) {
+  PI_REQUIRE(ctx, in->n_seqs > 0 && in->tokens && in->n_tokens && in->start_pos && in->table_lens, "a step needs at least one sequence");
+  PI_REQUIRE(ctx, in->block_tables || in->max_blocks == 0, "null block tables");
+  PI_REQUIRE(ctx, in->n_out >= 0 && (in->n_out == 0 || in->out_rows), "null output rows");
+  PI_TRY(check_pool(ctx, m, pool));
+  std::vector<int32_t> pos, lens, tables;
+  for (int i = 0; i < in->n_seqs; ++i) {
+    PI_REQUIRE(ctx, in->n_tokens[i] >= 1 && in->start_pos[i] >= 0 && in->table_lens[i] <= in->max_blocks, "sequence %d: bad portion", i);
+    for (int j = 0; j < in->n_tokens[i]; ++j) {
+      pos.push_back(in->start_pos[i] + j);
+      lens.push_back(in->table_lens[i]);
+      tables.insert(tables.end(), in->block_tables + (size_t)i * in->max_blocks, in->block_tables + (size_t)(i + 1) * in->max_blocks);
+    }
+  }
+  const int rows = (int)pos.size();
+  PI_REQUIRE(ctx, rows <= m->capacity, "the step's %d tokens exceed scratch capacity %d", rows, m->capacity);
+  bool all = in->n_out == rows;
+  for (int i = 0; i < in->n_out; ++i) {
+    PI_REQUIRE(ctx, in->out_rows[i] >= 0 && in->out_rows[i] < rows && (i == 0 || in->out_rows[i] > in->out_rows[i - 1]), "output row %d of %d",
+               in->out_rows[i], rows);
+    all = all && in->out_rows[i] == i;
+  }
+  pi_attn_batch batch;
+  PI_TRY(stage_batch(ctx, m, pool, in->tokens, pos.data(), tables.data(), in->max_blocks, lens.data(), rows, &batch));
+  x_planes_state xs;
+  PI_TRY(run_layers(ctx, m, pool, batch, rows, all ? &xs : nullptr));
+  if (in->n_out) {
+    if (!all) {   // wanted rows move to the front (increasing order: a row is never overwritten before it is read)
+      const size_t w = m->cfg.hidden_size;
+      for (int i = 0; i < in->n_out; ++i)
+        if (in->out_rows[i] != i)
+          PI_CUDA(ctx, cudaMemcpyAsync(m->x + i * w, m->x + in->out_rows[i] * w, w * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
+    }
+    PI_TRY(project_logits(ctx, m, 0, in->n_out, all ? &xs : nullptr));
+    PI_TRY(fetch_results(ctx, m, in->n_out, logits_host, argmax_host));
+  }
+  return pi_ctx_synchronize(ctx);
+}
+
+pi_status pi_model_step(pi_ctx* ctx, pi_model* m, pi_kv_pool* pool, pi_state_pool* state, const pi_step_batch* batch, float* logits_host,
+                        uint32_t* argmax_host) {
+  PI_ENTER(ctx);
+  PI_REQUIRE(ctx, m && pool && batch, "null pointer");
+  if (m->layered) return pi_layered_step(ctx, m->layered, pool, state, batch, logits_host, argmax_host);
+  return uniform_step(ctx, m, pool, batch, logits_host, argmax_host);
+}
+
+pi_status pi_model_step_multi(pi_ctx* ctx, pi_model* m, pi_kv_pool* pool, pi_state_pool* state, const pi_step_batch* batch, int n_steps,
+                              uint32_t* out_tokens_host) {
+  PI_ENTER(ctx);
+  PI_REQUIRE(ctx, m && pool && batch, "null pointer");
+  if (m->layered) return pi_layered_step_multi(ctx, m->layered, pool, state, batch, n_steps, out_tokens_host);
+  for (int i = 0; i < batch->n_seqs; ++i) PI_REQUIRE(ctx, batch->n_tokens && batch->n_tokens[i] == 1, "sequence %d brings more than one token", i);
+  return pi_model_decode_multi(ctx, m, pool, batch->tokens, batch->start_pos, batch->block_tables, batch->max_blocks, batch->table_lens, batch->n_seqs,
+                               n_steps, out_tokens_host);
+}
+
 }  // extern "C"
+
+const pi_layered* pi_model_layered(const pi_model* m, pi_kv_layout* L) {
+  *L = pi_kv_layout{m->cfg.num_hidden_layers, 0, 0, m->kv_heads_local, m->hd};
+  return m->layered;
+}

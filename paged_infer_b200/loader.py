@@ -74,8 +74,72 @@ class LlamaConfig:
             "intermediate_size", "vocab_size", "rms_norm_eps", "rope_theta", "attention_window", "rope_style")}
 
 
+MIXER_ATTENTION, MIXER_GLA, MIXER_MLSTM = 0, 1, 2
+
+
+@dataclass
+class LayerConfig:
+    """One layer of a layered design: a token mixer with its own sizes and, if ``ff``, a gated feed-forward.
+
+    ``window`` None: everything before.  ``maps`` 2: differential attention (``diff`` its constant).  ``tau`` belongs to the
+    gated linear recurrence, ``gate_cap`` to the matrix memory."""
+
+    mixer: int
+    heads: int
+    dim: int
+    vdim: int
+    kv_heads: int = 0
+    maps: int = 1
+    window: int | None = None
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+    scale: float = 1.0
+    diff: float = 0.0
+    tau: float = 1.0
+    gate_cap: float = 1.0
+    ff: int = 0
+
+
+@dataclass
+class LayeredConfig:
+    """A design whose layers each name a mixer (``pi_layered_config``)."""
+
+    width: int
+    vocab_size: int
+    norm_eps: float
+    layers: list
+
+    @property
+    def has_state(self) -> bool:
+        return any(l.mixer != MIXER_ATTENTION for l in self.layers)
+
+    @classmethod
+    def from_sumosun(cls, j: dict) -> "LayeredConfig":
+        """The Sumosun design's ``config.json``: differential attention, GLA and mLSTM layers in any order."""
+        layers = []
+        for i, e in enumerate(j["layers"]):
+            m, mlp = e["mixer"], e.get("mlp")
+            if mlp is not None and mlp["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            ff = int(mlp["ff"]) if mlp is not None else 0
+            common = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), ff=ff)
+            if e["type"] == "attention":
+                mask, rot = m.get("mask"), m.get("rot")
+                layers.append(LayerConfig(MIXER_ATTENTION, kv_heads=int(m["kv_heads"]), maps=2, window=int(mask["size"]) if mask else None,
+                                          rot_dims=int(rot["dims"]) if rot else 0, rot_base=float(rot["base"]) if rot else 1.0,
+                                          scale=float(m["scale"]), diff=float(m["diff"]), **common))
+            elif e["type"] == "gla":
+                layers.append(LayerConfig(MIXER_GLA, tau=float(m["tau"]), **common))
+            elif e["type"] == "mlstm":
+                layers.append(LayerConfig(MIXER_MLSTM, gate_cap=float(m["gate_cap"]), **common))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+        return cls(width=int(j["width"]), vocab_size=int(j["vocab"]), norm_eps=float(j["norm"]["eps"]), layers=layers)
+
+
 def read_safetensors(path: str) -> dict:
-    """name -> uint16 array of bf16 bits with the stored shape."""
+    """name -> array with the stored shape: bf16 tensors as uint16 bits, f32 and integer tables as they are."""
+    dtypes = {"BF16": "<u2", "F32": "<f4", "I32": "<i4"}
     with open(path, "rb") as f:
         raw = f.read()
     (hlen,) = struct.unpack("<Q", raw[:8])
@@ -85,10 +149,14 @@ def read_safetensors(path: str) -> dict:
     for name, info in header.items():
         if name == "__metadata__":
             continue
-        if info["dtype"] != "BF16":
+        if info["dtype"] not in dtypes:
             raise ValueError(f"{name}: only BF16 checkpoints are supported, got {info['dtype']}")
+        dt = np.dtype(dtypes[info["dtype"]])
         a, b = info["data_offsets"]
-        out[name] = np.frombuffer(raw, dtype="<u2", count=(b - a) // 2, offset=base + a).reshape(info["shape"])
+        if (base + a) % dt.itemsize:
+            out[name] = np.frombuffer(raw[base + a:base + b], dtype=dt).reshape(info["shape"])
+        else:
+            out[name] = np.frombuffer(raw, dtype=dt, count=(b - a) // dt.itemsize, offset=base + a).reshape(info["shape"])
     return out
 
 

@@ -20,11 +20,14 @@
 #include "../../include/paged_infer_engine.hpp"
 
 struct pi_ctx { std::string err; };
-struct pi_model { int capacity; };
-struct pi_kv_pool { pi_kv_layout L; std::vector<int> copies; };
+struct pi_model { int capacity; size_t state_bytes = 0; };
+struct pi_kv_pool { int num_blocks, block_size; };
+struct FakeState { int next_pos = -1; uint32_t sum = 0; };   // what a recurrent model would carry
+struct pi_state_pool { std::vector<FakeState> slots; };
 
-static std::vector<int> g_batches;        // rows of every batched forward
-static int g_prefills = 0, g_cow = 0;
+static std::vector<int> g_batches;        // rows of every batched forward whose sequences bring one token each
+static int g_mixed = 0;                   // forwards with portions of several tokens beside single ones
+static int g_cow = 0, g_state_copies = 0;
 static bool g_violation = false;
 
 static uint32_t next_token(uint32_t tok, int pos) { return (tok * 31u + (uint32_t)pos * 7u + 3u) % 997u; }
@@ -32,39 +35,73 @@ static uint32_t next_token(uint32_t tok, int pos) { return (tok * 31u + (uint32_
 extern "C" {
 const char* pi_last_error(const pi_ctx* c) { return c ? c->err.c_str() : ""; }
 int pi_model_max_batch(const pi_model* m) { return m->capacity; }
-pi_status pi_kv_pool_create(pi_ctx*, const pi_kv_layout* L, pi_kv_pool** out) {
-  *out = new pi_kv_pool{*L, {}};
+size_t pi_model_state_bytes(const pi_model* m) { return m->state_bytes; }
+pi_status pi_kv_pool_create_for_model(pi_ctx*, const pi_model*, int num_blocks, int block_size, pi_kv_pool** out) {
+  *out = new pi_kv_pool{num_blocks, block_size};
   return PI_OK;
 }
 void pi_kv_pool_destroy(pi_kv_pool* p) { delete p; }
+pi_status pi_state_pool_create(pi_ctx*, const pi_model*, int n, pi_state_pool** out) {
+  *out = new pi_state_pool{std::vector<FakeState>((size_t)n)};
+  return PI_OK;
+}
+void pi_state_pool_destroy(pi_state_pool* p) { delete p; }
+pi_status pi_state_copy_slot(pi_ctx*, pi_state_pool* p, int32_t src, int32_t dst) {
+  if (src == dst) g_violation = true;
+  p->slots.at(dst) = p->slots.at(src);
+  ++g_state_copies;
+  return PI_OK;
+}
 pi_status pi_kv_copy_block(pi_ctx* c, pi_kv_pool* p, int32_t src, int32_t dst) {
-  if (src == dst || src < 0 || dst < 0 || src >= p->L.num_blocks || dst >= p->L.num_blocks) {
+  if (src == dst || src < 0 || dst < 0 || src >= p->num_blocks || dst >= p->num_blocks) {
     c->err = "bad copy";
     return PI_ERR_INVALID_ARG;
   }
   ++g_cow;
   return PI_OK;
 }
-pi_status pi_model_prefill(pi_ctx*, pi_model*, pi_kv_pool* pool, const uint32_t* tokens, int n, int start_pos, const int32_t*,
-                           int table_len, int, float*, uint32_t* argmax) {
-  if (n < 1 || (start_pos + n + pool->L.block_size - 1) / pool->L.block_size > table_len) g_violation = true;
-  ++g_prefills;
-  if (argmax) *argmax = next_token(tokens[n - 1], start_pos + n - 1);
-  return PI_OK;
-}
-pi_status pi_model_decode_batch(pi_ctx* c, pi_model* m, pi_kv_pool* pool, const uint32_t* tokens, const int32_t* positions,
-                                const int32_t* tables, int max_blocks, const int32_t* lens, int B, float*, uint32_t* argmax) {
-  if (B > m->capacity) {
+pi_status pi_model_step(pi_ctx* c, pi_model* m, pi_kv_pool* pool, pi_state_pool* state, const pi_step_batch* b, float* logits, uint32_t* argmax) {
+  int rows = 0, singles = 0;
+  for (int i = 0; i < b->n_seqs; ++i) {
+    rows += b->n_tokens[i];
+    singles += b->n_tokens[i] == 1;
+  }
+  if (rows > m->capacity) {
     c->err = "batch exceeds scratch capacity";
     return PI_ERR_INVALID_ARG;
   }
-  g_batches.push_back(B);
-  std::set<int32_t> written;
-  for (int b = 0; b < B; ++b) {
-    const int lb = positions[b] / pool->L.block_size;
-    if (lb >= lens[b] || lens[b] > max_blocks) g_violation = true;
-    else if (!written.insert(tables[(size_t)b * max_blocks + lb]).second) g_violation = true;   // two rows write one block
-    argmax[b] = next_token(tokens[b], positions[b]);
+  if (singles == b->n_seqs) g_batches.push_back(b->n_seqs);
+  else if (singles > 0) ++g_mixed;
+  std::set<int32_t> written, slots;
+  std::vector<uint32_t> out;
+  const uint32_t* t = b->tokens;
+  for (int i = 0; i < b->n_seqs; ++i) {
+    const int first = b->start_pos[i] / pool->block_size, last = (b->start_pos[i] + b->n_tokens[i] - 1) / pool->block_size;
+    if (last >= b->table_lens[i] || b->table_lens[i] > b->max_blocks) g_violation = true;
+    else
+      for (int lb = first; lb <= last; ++lb)
+        if (!written.insert(b->block_tables[(size_t)i * b->max_blocks + lb]).second) g_violation = true;   // two sequences write one block
+    if ((m->state_bytes > 0) != (b->state_slots != nullptr)) g_violation = true;
+    FakeState* s = nullptr;
+    if (m->state_bytes) {
+      if (!slots.insert(b->state_slots[i]).second) g_violation = true;
+      s = &state->slots.at(b->state_slots[i]);
+      if (b->start_pos[i] == 0) *s = FakeState{0, 0};
+      if (s->next_pos != b->start_pos[i]) g_violation = true;   // a slot was lost, shared or not carried on
+    }
+    for (int j = 0; j < b->n_tokens[i]; ++j, ++t) {
+      uint32_t r = next_token(*t, b->start_pos[i] + j);
+      if (s) {
+        s->sum = s->sum * 13u + *t;
+        s->next_pos = b->start_pos[i] + j + 1;
+        r = (r + s->sum) % 997u;
+      }
+      out.push_back(r);
+    }
+  }
+  for (int i = 0; i < b->n_out; ++i) {
+    if (argmax) argmax[i] = out.at(b->out_rows[i]);
+    if (logits) logits[i] = (float)out.at(b->out_rows[i]);
   }
   return PI_OK;
 }
@@ -175,6 +212,82 @@ int main() {
     CHECK(run_all(e, 2, &done) == 0);
     CHECK(done[1][0].generated == expected(prompt(50, 60), 3) && done[2][0].generated == expected(prompt(51, 60), 3));
     std::printf("ok queue\n");
+  }
+  // the same with recurrent state: tokens depend on everything before them
+  auto expected_state = [](const std::vector<uint32_t>& p, size_t max_tokens) {
+    std::vector<uint32_t> out, all = p;
+    uint32_t sum = 0;
+    size_t done = 0;
+    while (out.size() < max_tokens) {
+      for (; done < all.size(); ++done) sum = sum * 13u + all[done];
+      out.push_back((next_token(all.back(), (int)all.size() - 1) + sum) % 997u);
+      all.push_back(out.back());
+    }
+    return out;
+  };
+  for (int mixed = 0; mixed < 2; ++mixed) {   // slots: fewer than requests, given back and used again; samples copy the state
+    g_mixed = g_state_copies = 0;
+    pi_model model{24, 128};
+    pi::EngineConfig cfg;
+    cfg.num_blocks = 64;
+    cfg.max_batch_size = 24;
+    cfg.prefill_chunk_size = 7;
+    cfg.mixed_batches = mixed != 0;
+    cfg.state_slots = 4;
+    pi::Engine e(&ctx, &model, cfg);
+    for (uint64_t r = 0; r < 9; ++r) e.add_request({r, prompt(70 + (uint32_t)r % 4, 3 + 11 * r), 5 + r % 3, r == 4 ? 3u : 1u});
+    std::map<uint64_t, std::vector<pi::Completion>> done;
+    CHECK(run_all(e, 11, &done) == 0);
+    for (uint64_t r = 0; r < 9; ++r)
+      for (auto& c : done[r]) CHECK(c.generated == expected_state(prompt(70 + (uint32_t)r % 4, 3 + 11 * r), 5 + r % 3) && c.cached_prompt_tokens == 0);
+    CHECK(g_state_copies == 2 && done[4].size() == 3 && (g_mixed > 0) == (mixed != 0));
+    CHECK(e.memory().free_state_slots() == 4 && e.memory().available_blocks() == 64);
+    std::printf("ok state slots (%s)\n", mixed ? "mixed batches" : "prefill at admission");
+  }
+  {  // mixed batches of a model without state: same tokens, the prefix cache still works
+    pi_model model{16};
+    pi::EngineConfig cfg;
+    cfg.num_blocks = 64;
+    cfg.max_batch_size = 16;
+    cfg.prefill_chunk_size = 5;
+    cfg.mixed_batches = true;
+    pi::Engine e(&ctx, &model, cfg);
+    for (uint64_t r = 0; r < 6; ++r) e.add_request({r, prompt(90, 40 + r), 6, 1});
+    std::map<uint64_t, std::vector<pi::Completion>> done;
+    CHECK(run_all(e, 6, &done) == 0);
+    e.add_request({99, prompt(90, 40), 4, 1});
+    CHECK(run_all(e, 1, &done) == 0);
+    for (uint64_t r = 0; r < 6; ++r) CHECK(done[r][0].generated == expected(prompt(90, 40 + r), 6));
+    CHECK(done[99][0].generated == expected(prompt(90, 40), 4) && done[99][0].cached_prompt_tokens == 32);
+    std::printf("ok mixed batches\n");
+  }
+  {  // feed: given tokens in portions, results of the wanted places, slots and blocks used again after end()
+    pi_model model{64, 64};
+    pi::EngineConfig cfg;
+    cfg.num_blocks = 6;
+    cfg.state_slots = 2;
+    cfg.prefix_cache = false;
+    pi::Engine e(&ctx, &model, cfg);
+    for (int round = 0; round < 3; ++round) {
+      const auto a = prompt(5 + round, 40), b = prompt(15 + round, 30);
+      auto sub = [](const std::vector<uint32_t>& v, size_t from, size_t to) { return std::vector<uint32_t>(v.begin() + from, v.begin() + to); };
+      float out[4];
+      e.feed({{1, sub(a, 0, 17), {}}}, out);
+      e.feed({{1, sub(a, 17, 18), {}}, {2, sub(b, 0, 29), {3, 28}}}, out);
+      CHECK(out[0] == (float)expected_state(sub(b, 0, 4), 1)[0] && out[1] == (float)expected_state(sub(b, 0, 29), 1)[0]);
+      e.feed({{2, sub(b, 29, 30), {0}}, {1, sub(a, 18, 40), {21}}}, out);
+      CHECK(out[0] == (float)expected_state(b, 1)[0] && out[1] == (float)expected_state(a, 1)[0]);
+      bool full = false;
+      try {
+        e.feed({{3, prompt(1, 2), {0}}}, out);
+      } catch (const pi::EngineError&) {
+        full = true;
+      }
+      CHECK(full);
+      e.end(1);
+      e.end(2);
+    }
+    std::printf("ok feed\n");
   }
   bool threw = false;
   try {

@@ -52,6 +52,7 @@ def test_engine_loop_over_a_fake_device_library(tmp_path):
     r = subprocess.run([exe], capture_output=True, text=True)
     assert r.returncode == 0, r.stdout + r.stderr
     lines = r.stdout.split("\n")
-    for name in ("oversize", "capacity", "passes", "queue"):
+    for name in ("oversize", "capacity", "passes", "queue", "state slots (mixed batches)", "state slots (prefill at admission)",
+                 "mixed batches", "feed"):
         assert f"ok {name}" in lines, name
     assert "all ok" in lines
