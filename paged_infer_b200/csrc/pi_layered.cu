@@ -407,7 +407,8 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
   int max_portion = 0;
   for (int i = 0; i < n; ++i) {
     const int k = in->n_tokens[i], p0 = in->start_pos[i];
-    PI_REQUIRE(ctx, k >= 1 && p0 >= 0 && p0 < (1 << 30) && k <= m->c.max_rows, "sequence %d: %d tokens from position %d", i, k, p0);
+    PI_REQUIRE(ctx, k >= 1 && p0 >= 0 && p0 < (1 << 30), "sequence %d: %d tokens from position %d", i, k, p0);
+    PI_REQUIRE(ctx, k <= m->c.max_rows - rows, "the step's tokens exceed the model's %d rows", m->c.max_rows);
     row0[i] = rows;
     for (int j = 0; j < k; ++j) {
       row_seq.push_back(i);
@@ -431,7 +432,6 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
     }
     rows += k;
     max_pos = std::max(max_pos, p0 + k - 1);
-    PI_REQUIRE(ctx, rows <= m->c.max_rows, "the step's tokens exceed the model's %d rows", m->c.max_rows);
     PI_REQUIRE(ctx, in->table_lens[i] >= 0 && in->table_lens[i] <= in->max_blocks, "sequence %d: %d mapped blocks, tables of %d", i,
                in->table_lens[i], in->max_blocks);
     for (int j = 0; j < in->table_lens[i]; ++j) {

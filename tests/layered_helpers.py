@@ -1,0 +1,162 @@
+"""Small random checkpoints of the Sumosun design for the tests: configurations, tensors under the checkpoint's names
+(values that bf16 represents exactly), the plain reference over them, and a writer for checkpoint folders."""
+from __future__ import annotations
+
+import json
+import struct
+
+import numpy as np
+
+from paged_infer_b200.loader import LayeredConfig, bf16_bits_to_f32, f32_to_bf16_bits
+
+
+def attention(heads=4, kv_heads=2, dim=16, vdim=32, window=24, rot=None, base=10000.0, diff=0.3, scale=None, ff=48):
+    return {"type": "attention", "mlp": {"kind": "dense", "ff": ff} if ff else None,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "diff": diff, "scale": dim ** -0.5 if scale is None else scale,
+                      "mask": {"size": window}, "rot": {"dims": dim if rot is None else rot, "base": base}}}
+
+
+def gla(heads=3, dim=16, vdim=24, tau=8.0, ff=0):
+    return {"type": "gla", "mlp": {"kind": "dense", "ff": ff} if ff else None, "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}}
+
+
+def mlstm(heads=2, dim=24, vdim=40, cap=10.0, ff=0):
+    return {"type": "mlstm", "mlp": {"kind": "dense", "ff": ff} if ff else None,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": cap}}
+
+
+def config(layers, width=64, vocab=96, eps=1e-5):
+    return {"architecture": "Sumosun", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def tensors(cfg, seed, rank=5):
+    """Random tensors (f32 values on the bf16 grid), scaled so that every part of the model moves the logits."""
+    rng = np.random.default_rng(seed)
+    W, V = cfg["width"], cfg["vocab"]
+    t = {}
+
+    def put(name, shape, std=None, mean=0.0):
+        x = rng.standard_normal(shape) * (1.0 / np.sqrt(shape[-1]) if std is None else std) + mean
+        t[name] = bf16_bits_to_f32(f32_to_bf16_bits(np.asarray(x, np.float32))).reshape(shape)
+
+    def norm(name, alpha):
+        put(name, (W,), 0.2, 1.0)
+        put(name + ".b", (W,), 0.1)
+        put(name + ".alpha", (), 0.0, alpha)
+
+    put("embed", (V, W), 1.0)
+    for i, e in enumerate(cfg["layers"]):
+        m, l = e["mixer"], f"l{i}"
+        H, D, E = m["heads"], m["dim"], m["vdim"]
+        norm(l + ".norm1", 0.7)
+        norm(l + ".norm1b", 0.9)
+        p = l + ".mix."
+        if e["type"] == "attention":
+            put(p + "q", (H * 2 * D, W), 1.5 / np.sqrt(W))
+            put(p + "k", (m["kv_heads"] * 2 * D, W), 1.5 / np.sqrt(W))
+            put(p + "v", (m["kv_heads"] * E, W))
+            for n in ("lq1", "lk1", "lq2", "lk2"):
+                put(p + n, (D,), 0.2)
+        else:
+            put(p + "q", (H * D, W))
+            put(p + "k", (H * D, W))
+            put(p + "v", (H * E, W))
+            put(p + "g", (H * E, W))
+            if e["type"] == "gla":
+                put(p + "a1", (rank, W))
+                put(p + "a2", (H * D, rank), 1.0)
+                put(p + "a2.b", (H * D,), 1.5, 1.0)
+                put(p + "norm", (E,), 0.2, 1.0)
+            else:
+                put(p + "i", (H, W))
+                put(p + "i.b", (H,), 1.0)
+                put(p + "f", (H, W))
+                put(p + "f.b", (H,), 1.0, 3.0)
+                put(p + "norm", (H * E,), 0.2, 1.0)
+        put(p + "o", (W, H * E))
+        if e["mlp"]:
+            F = e["mlp"]["ff"]
+            norm(l + ".norm2", 0.8)
+            norm(l + ".norm2b", 1.1)
+            put(l + ".mlp.gate", (F, W))
+            put(l + ".mlp.up", (F, W))
+            put(l + ".mlp.down", (W, F))
+    norm("final.norm", 0.6)
+    return t
+
+
+def bits(t):
+    return {k: f32_to_bf16_bits(np.asarray(v, np.float32)).reshape(np.shape(v)) for k, v in t.items()}
+
+
+def write_checkpoint(folder, cfg, t):
+    """config.json and model.safetensors as a user has them."""
+    (folder / "config.json").write_text(json.dumps(cfg))
+    header, blob = {}, b""
+    for name, a in bits(t).items():
+        raw = np.ascontiguousarray(a, "<u2").tobytes()
+        header[name] = {"dtype": "BF16", "shape": list(np.shape(t[name])), "data_offsets": [len(blob), len(blob) + len(raw)]}
+        blob += raw
+    h = json.dumps(header).encode()
+    (folder / "model.safetensors").write_bytes(struct.pack("<Q", len(h)) + h + blob)
+    return str(folder)
+
+
+def reference(cfg, t):
+    from oracle.layers import Sumosun
+    return Sumosun(cfg, t)
+
+
+def device_model(ctx, cfg, t, compute, max_rows=1024):
+    from paged_infer_b200 import api
+    return api.LayeredModel(ctx, LayeredConfig.from_sumosun(cfg), bits(t), compute, max_rows)
+
+
+def distance(got, want):
+    """Root mean square of the difference over the spread of the reference, per row (a common shift taken off)."""
+    got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
+    d = got - want
+    d = d - d.mean(-1, keepdims=True)
+    return np.sqrt((d * d).mean(-1)) / want.std()
+
+
+LIMIT = {"float32": 2e-5, "bfloat16": 4e-2}
+
+
+class Session:
+    """Sequences over one pool and state pool, with block tables and slots the test chooses (scattered on purpose)."""
+
+    def __init__(self, model, blocks=256, block_size=16, slots=6, seed=0):
+        self.m, self.bs = model, block_size
+        self.kv = model.kv_pool(blocks, block_size)
+        self.state = model.state_pool(slots) if model.state_bytes() else None
+        self.free = list(np.random.default_rng(seed).permutation(blocks))
+        self.slots = list(range(slots))[::-1]
+        self.seq = {}
+
+    def open(self, name):
+        self.seq[name] = [0, [], self.slots.pop()]
+
+    def close(self, name):
+        _, table, slot = self.seq.pop(name)
+        self.free = table[::-1] + self.free      # used again at once
+        self.slots.append(slot)
+
+    def run(self, portions, every_row=True):
+        """portions: [(name, tokens)] -> list of logits arrays, one per portion (every row, or the last)."""
+        starts, tables, slots = [], [], []
+        for name, toks in portions:
+            if name not in self.seq:
+                self.open(name)
+            s = self.seq[name]
+            starts.append(s[0])
+            s[0] += len(toks)
+            while len(s[1]) * self.bs < s[0]:
+                s[1].append(int(self.free.pop(0)))
+            tables.append(list(s[1]))
+            slots.append(s[2])
+        counts = [len(t) for _, t in portions]
+        ends = np.cumsum(counts)
+        rows = np.arange(ends[-1]) if every_row else ends - 1
+        out = self.m.step([t for _, t in portions], starts, tables, self.kv, self.state, slots if self.state else None, rows)
+        return np.split(out, ends[:-1]) if every_row else list(out[:, None])
