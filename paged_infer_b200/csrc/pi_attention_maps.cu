@@ -7,12 +7,12 @@
 //   o = a_1 - lambda a_2;  out = out_scale o / rms(o)          (two maps)
 //
 // Kernels: maps_rope_kv_kernel rotates q and k and writes k and v into the pool; maps_attn_plain_kernel is the f32
-// path (any sizes, one warp per row and head).
+// path and the one for sizes the tensor-core kernels of pi_attention_maps_tc.cu do not hold.
 #include <math.h>
 
 #include <algorithm>
 
-#include "pi_layered.cuh"
+#include "pi_attention_maps.cuh"
 
 namespace {
 
@@ -73,18 +73,6 @@ __global__ void __launch_bounds__(256) maps_rope_kv_kernel(const RopeKvParams p)
     dst[e] = pi_from_f32<T>(e < p.vdim ? vsrc[(size_t)g * p.vdim + e] : 0.f);
   }
 }
-
-struct MapsParams {
-  const float* q;
-  size_t stride;
-  void* out;
-  size_t out_stride;
-  const void* base;
-  int heads, kv_heads, maps, dim, vdim, dp, vp, block_size, window;
-  float scale, eps, lambda, out_scale;
-  const int32_t *row_seq, *row_pos, *lens, *tables;
-  int max_blocks;
-};
 
 // One CTA of 4 warps per (row, head): the warps take every fourth key and merge; lanes hold the channels.  f32
 // throughout, any sizes (smem: q, per-warp accumulators of both maps).
@@ -178,6 +166,7 @@ pi_status pi_launch_maps_attention(pi_ctx* ctx, const pi_maps_attention& a, cons
   pi_prof_scope prof(ctx, PI_PROF_ATTENTION);
   MapsParams p = {qkv, stride, out, out_stride, kv.base, a.heads, a.kv_heads, a.maps, a.dim, a.vdim, kv.dp, kv.vp, kv.block_size,
                   a.window, a.scale, a.eps, a.lambda, a.out_scale, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks};
+  if (pi_maps_attention_tc_usable(ctx, a, kv)) return pi_launch_maps_attention_tc(ctx, p, out_kind, b);
   const size_t smem = sizeof(float) * ((size_t)a.maps * a.dim + (size_t)kPlainWarps * a.maps * a.vdim);
   PI_REQUIRE(ctx, smem <= 48 * 1024, "attention heads of %d / %d channels are too wide", a.dim, a.vdim);
   auto k = kv.kind == PI_BF16 ? (out_kind == PI_BF16 ? maps_attn_plain_kernel<__nv_bfloat16, __nv_bfloat16> : maps_attn_plain_kernel<__nv_bfloat16, float>)

@@ -1,0 +1,650 @@
+// Multi-map windowed attention over a bf16 KV pool on the tensor cores (mma.sync; see pi_attention_maps.cu for the
+// mathematics).  Scores and weights are f32; the weights enter the product with V as two bf16 planes (16 bits).
+//
+// maps_decode_kernel: one row alone.  CTA = (row, kv head, group of heads, KV split).  The MMA's 16 rows are 16 heads, or
+//   8 heads x 2 maps: with two maps the query operand is block diagonal - rows 0-7 hold map 1 in the first half of the
+//   key channels and zero in the second, rows 8-15 the other way round - so one product over the concatenated channels
+//   scores both maps, and one product with V serves both.  Each warp streams 16-key tiles through a private ring of
+//   asynchronous copies; warps (and splits) merge by log-sum-exp.
+// maps_tile_kernel: portions.  CTA = (sequence, kv head, tile of (token, head) rows); a warp owns 16 rows of one map, the
+//   pair of warps with the two maps of the same rows meets in shared memory at the end.  64-key tiles, double buffered.
+#include <math.h>
+
+#include <algorithm>
+
+#include "pi_attention_maps.cuh"
+#include "pi_mma.cuh"
+
+namespace {
+using namespace pi_mma;
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+struct TcParams {
+  MapsParams m;
+  const int32_t* rows;              // decode: the rows that stand alone
+  const int32_t *portions, *seq_row0, *seq_n, *seq_start;
+  int group, ngroups, nsplit;       // heads per kv head; decode: groups of them per MMA, KV splits
+  float* part_acc;                  // [row][kv head][group][split][16][vp]
+  float* part_ml;                   // [...][16][2]
+  int out_bf16;
+};
+
+__device__ __forceinline__ void store_out(const TcParams& p, size_t i, float v) {
+  if (p.out_bf16) static_cast<__nv_bfloat16*>(p.m.out)[i] = __float2bfloat16_rn(v);
+  else static_cast<float*>(p.m.out)[i] = v;
+}
+
+// Address of key t's row in the pool (K part; V follows the block's keys).
+struct Paged {
+  const __nv_bfloat16* base;
+  const int32_t* table;
+  int block_size, kv_heads, head, kw, vp;
+  __device__ __forceinline__ const __nv_bfloat16* tile(int lb) const {
+    return base + ((size_t)table[lb] * kv_heads + head) * ((size_t)block_size * (kw + vp));
+  }
+};
+
+// Online softmax step of one accumulator row: running maximum, factor for what is already summed.
+__device__ __forceinline__ float new_max(float m, float s_max, float& keep) {
+  const float n = fmaxf(m, s_max);
+  keep = n == -INFINITY ? 1.f : exp2f(m - n);
+  return n;
+}
+
+constexpr int kDecWarps = 4, kDecStages = 3;
+
+template <int MAPS, int KMAX, int VMAX>
+__global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcParams p) {
+  constexpr int QR = MAPS == 2 ? 2 : 4;     // query registers per 16 channels
+  constexpr int HR = 16 / MAPS;             // heads per MMA
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const MapsParams& a = p.m;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int ri = blockIdx.x, g = blockIdx.y / p.ngroups, grp = blockIdx.y % p.ngroups, split_i = blockIdx.z;
+  const int row = p.rows[ri], seq = a.row_seq[row], pos = a.row_pos[row];
+  const int kw = MAPS * a.dp, ks_map = a.dp / 16, nks = MAPS * ks_map, nv = a.vp / 8;
+  const int kpitch = kw + 8, vpitch = a.vp + 8;
+  const int stage_elems = 16 * (kpitch + vpitch);
+  __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(smem_raw) + (size_t)warp * kDecStages * stage_elems;
+  const Paged pg = {static_cast<const __nv_bfloat16*>(a.base), a.tables + (size_t)seq * a.max_blocks, a.block_size, a.kv_heads, g, kw, a.vp};
+
+  // keys of this CTA: [k_lo, k_hi), tiles start on multiples of 16
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0, hi = min(pos + 1, a.lens[seq] * a.block_size);
+  const int t_first = lo / 16, n_tiles = (hi + 15) / 16 - t_first, per = (n_tiles + p.nsplit - 1) / p.nsplit;
+  const int tile_end = min(t_first + n_tiles, t_first + (split_i + 1) * per);
+  const int tile0 = t_first + split_i * per + warp;
+  const bool one_block = a.block_size % 16 == 0;
+
+  auto fetch = [&](int tile, int stage) {
+    __nv_bfloat16* ks = ring + (size_t)stage * stage_elems;
+    __nv_bfloat16* vs = ks + 16 * kpitch;
+    const int t0 = tile * 16;
+    const __nv_bfloat16* base = nullptr;
+    int off0 = 0;
+    if (one_block) {
+      base = pg.tile(t0 / a.block_size);
+      off0 = t0 % a.block_size;
+    }
+    auto copy = [&](__nv_bfloat16* dst, int pitch, int width, bool is_v) {
+      const int per_row = width / 8;
+      for (int c = lane; c < 16 * per_row; c += 32) {
+        const int r = c / per_row, x = (c - r * per_row) * 8, t = t0 + r;
+        const bool ok = t < hi;
+        const __nv_bfloat16* b = base;
+        int off = off0 + r;
+        if (!one_block && ok) {
+          b = pg.tile(t / a.block_size);
+          off = t % a.block_size;
+        }
+        const __nv_bfloat16* src = is_v ? b + (size_t)a.block_size * kw + (size_t)off * a.vp + x : b + (size_t)off * kw + x;
+        cp_async16(smem_addr(dst + r * pitch + x), ok ? (const void*)src : a.base, ok ? 16 : 0);
+      }
+    };
+    copy(ks, kpitch, kw, false);
+    copy(vs, vpitch, a.vp, true);
+  };
+
+  pi_grid_dependency_wait();
+#pragma unroll
+  for (int s = 0; s < kDecStages - 1; ++s) {
+    if (tile0 + s * kDecWarps < tile_end) fetch(tile0 + s * kDecWarps, s);
+    cp_async_commit();
+  }
+
+  // query operand: row r of the MMA = (map r / HR, head r % HR)
+  uint32_t qa[KMAX][QR];
+  {
+    const int r0 = lane >> 2, c0 = (lane & 3) * 2;
+    auto q2 = [&](int r, int ks, int c) -> uint32_t {   // channels c, c + 1 of k step ks of MMA row r
+      const int map = MAPS == 2 ? ks / ks_map : 0, head = grp * HR + r % HR;
+      const int d = (ks - map * ks_map) * 16 + c;
+      if (head >= p.group) return 0u;
+      const float* q = a.q + (size_t)row * a.stride + ((size_t)(g * p.group + head) * MAPS + map) * a.dim;
+      return pack(d < a.dim ? q[d] : 0.f, d + 1 < a.dim ? q[d + 1] : 0.f);
+    };
+#pragma unroll
+    for (int ks = 0; ks < KMAX; ++ks) {
+#pragma unroll
+      for (int j = 0; j < QR; ++j) qa[ks][j] = 0u;
+      if (ks < nks) {
+        if (MAPS == 2) {
+          qa[ks][0] = q2(r0, ks, c0);
+          qa[ks][1] = q2(r0, ks, c0 + 8);
+        } else {
+          qa[ks][0] = q2(r0, ks, c0);
+          qa[ks][1] = q2(r0 + 8, ks, c0);
+          qa[ks][QR - 2] = q2(r0, ks, c0 + 8);
+          qa[ks][QR - 1] = q2(r0 + 8, ks, c0 + 8);
+        }
+      }
+    }
+  }
+  float acc[VMAX / 8][4];
+#pragma unroll
+  for (int j = 0; j < VMAX / 8; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
+  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  const float sc = a.scale * kLog2e;
+
+  int stage = 0;
+  for (int tile = tile0; tile < tile_end; tile += kDecWarps) {
+    cp_async_wait<kDecStages - 2>();
+    __syncwarp();
+    const __nv_bfloat16* ks = ring + (size_t)stage * stage_elems;
+    const __nv_bfloat16* vs = ks + 16 * kpitch;
+    float s[2][4];
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s[j][i] = 0.f;
+#pragma unroll
+    for (int k = 0; k < KMAX; ++k) {
+      if (k < nks) {
+        uint32_t b[4];   // keys 0-7: channels 0-7, 8-15; keys 8-15 likewise
+        ldsm4(b, smem_addr(ks + (size_t)((lane & 7) + ((lane >> 4) << 3)) * kpitch + k * 16 + ((lane >> 3) & 1) * 8));
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          if (MAPS == 2) {
+            if (k < ks_map) mma(s[j], qa[k][0], 0u, qa[k][1], 0u, b[2 * j], b[2 * j + 1]);
+            else mma(s[j], 0u, qa[k][0], 0u, qa[k][1], b[2 * j], b[2 * j + 1]);
+          } else {
+            mma(s[j], qa[k][0], qa[k][1], qa[k][QR - 2], qa[k][QR - 1], b[2 * j], b[2 * j + 1]);
+          }
+        }
+      }
+    }
+    const int key = tile * 16 + (lane & 3) * 2;
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int t = key + 8 * j + (i & 1);
+        s[j][i] = (t >= lo && t < hi) ? s[j][i] * sc : -INFINITY;
+      }
+    uint32_t ph[4], pl[4];
+    float keep[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {   // MMA rows lane / 4 and lane / 4 + 8
+      const float tm = quad_max(fmaxf(fmaxf(s[0][2 * h], s[0][2 * h + 1]), fmaxf(s[1][2 * h], s[1][2 * h + 1])));
+      mx[h] = new_max(mx[h], tm, keep[h]);
+      const float ref = mx[h] == -INFINITY ? 0.f : mx[h];
+      float w[4];
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) w[2 * j + i] = exp2f(s[j][2 * h + i] - ref);
+      l[h] = l[h] * keep[h] + ((w[0] + w[1]) + (w[2] + w[3]));
+      split(w[0], w[1], ph[h], pl[h]);
+      split(w[2], w[3], ph[2 + h], pl[2 + h]);
+    }
+#pragma unroll
+    for (int j = 0; j < VMAX / 8; j += 2) {
+      if (j < nv) {
+        uint32_t b[4];   // value columns j*8.., keys 0-7 and 8-15; then the next eight columns
+        ldsm4_t(b, smem_addr(vs + (size_t)((lane & 7) + ((lane >> 3) & 1) * 8) * vpitch + j * 8 + (lane >> 4) * 8));
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          float* d = acc[j + h];
+          d[0] *= keep[0];
+          d[1] *= keep[0];
+          d[2] *= keep[1];
+          d[3] *= keep[1];
+          mma(d, ph[0], ph[1], ph[2], ph[3], b[2 * h], b[2 * h + 1]);
+          mma(d, pl[0], pl[1], pl[2], pl[3], b[2 * h], b[2 * h + 1]);
+        }
+      }
+    }
+    const int next = tile + (kDecStages - 1) * kDecWarps;
+    if (next < tile_end) fetch(next, (stage + kDecStages - 1) % kDecStages);
+    cp_async_commit();
+    stage = (stage + 1) % kDecStages;
+  }
+  cp_async_wait<0>();
+  l[0] = quad_sum(l[0]);
+  l[1] = quad_sum(l[1]);
+
+  // ---- merge the warps -----------------------------------------------------------------------------------------------
+  __syncthreads();
+  float* wacc = reinterpret_cast<float*>(smem_raw);      // [warps][16][vp + 4]
+  const int apitch = a.vp + 4;
+  __shared__ float s_m[kDecWarps][16], s_l[kDecWarps][16];
+  {
+    const int r0 = lane >> 2;
+    float* w = wacc + (size_t)warp * 16 * apitch;
+#pragma unroll
+    for (int j = 0; j < VMAX / 8; ++j)
+      if (j < nv) {
+        const int c = j * 8 + (lane & 3) * 2;
+        *reinterpret_cast<float2*>(w + (size_t)r0 * apitch + c) = make_float2(acc[j][0], acc[j][1]);
+        *reinterpret_cast<float2*>(w + (size_t)(r0 + 8) * apitch + c) = make_float2(acc[j][2], acc[j][3]);
+      }
+    if ((lane & 3) == 0) {
+      s_m[warp][r0] = mx[0];
+      s_m[warp][r0 + 8] = mx[1];
+      s_l[warp][r0] = l[0];
+      s_l[warp][r0 + 8] = l[1];
+    }
+  }
+  __syncthreads();
+  const size_t part = (((size_t)ri * a.kv_heads + g) * p.ngroups + grp) * p.nsplit + split_i;
+  for (int h = warp; h < HR; h += kDecWarps) {
+    const int head = grp * HR + h;
+    if (head >= p.group) continue;
+    float f[MAPS][kDecWarps];
+#pragma unroll
+    for (int m = 0; m < MAPS; ++m) {
+      const int r = h + m * HR;
+      float M = -INFINITY, L = 0.f;
+#pragma unroll
+      for (int w = 0; w < kDecWarps; ++w) M = fmaxf(M, s_m[w][r]);
+#pragma unroll
+      for (int w = 0; w < kDecWarps; ++w) {
+        f[m][w] = s_m[w][r] == -INFINITY ? 0.f : exp2f(s_m[w][r] - M);
+        L += s_l[w][r] * f[m][w];
+      }
+      if (p.nsplit == 1) {
+#pragma unroll
+        for (int w = 0; w < kDecWarps; ++w) f[m][w] = L > 0.f ? f[m][w] / L : 0.f;
+      } else if (lane == 0) {
+        p.part_ml[(part * 16 + r) * 2] = M;
+        p.part_ml[(part * 16 + r) * 2 + 1] = L;
+      }
+    }
+    float ss = 0.f;
+    for (int e = lane; e < a.vp; e += 32) {
+      float o[MAPS];
+#pragma unroll
+      for (int m = 0; m < MAPS; ++m) {
+        o[m] = 0.f;
+#pragma unroll
+        for (int w = 0; w < kDecWarps; ++w) o[m] += wacc[((size_t)w * 16 + h + m * HR) * apitch + e] * f[m][w];
+        if (p.nsplit > 1) p.part_acc[(part * 16 + h + m * HR) * a.vp + e] = o[m];
+      }
+      if (p.nsplit == 1) {
+        const float d = MAPS == 2 ? o[0] - a.lambda * o[MAPS - 1] : o[0];
+        ss = fmaf(d, d, ss);
+        wacc[(size_t)h * apitch + e] = d;   // this lane alone reads column e of row h (warp 0's area)
+      }
+    }
+    if (p.nsplit == 1) {
+      const float r = MAPS == 2 ? a.out_scale / sqrtf(pi_warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
+      const size_t o0 = (size_t)row * a.out_stride + (size_t)(g * p.group + head) * a.vdim;
+      for (int e = lane; e < a.vdim; e += 32) store_out(p, o0 + e, wacc[(size_t)h * apitch + e] * r);
+    }
+  }
+}
+
+// Merge the KV splits of a row: one warp per head.
+template <int MAPS>
+__global__ void __launch_bounds__(128) maps_merge_kernel(const TcParams p) {
+  constexpr int HR = 16 / MAPS;
+  const MapsParams& a = p.m;
+  const int ri = blockIdx.x, lane = threadIdx.x & 31, head = blockIdx.y * 4 + (threadIdx.x >> 5);
+  pi_grid_dependency_wait();
+  if (head >= a.heads) return;
+  const int row = p.rows[ri], g = head / p.group, hg = head % p.group, grp = hg / HR, h = hg % HR;
+  const size_t part0 = (((size_t)ri * a.kv_heads + g) * p.ngroups + grp) * p.nsplit;
+  float M[MAPS], L[MAPS];
+#pragma unroll
+  for (int m = 0; m < MAPS; ++m) {
+    const int r = h + m * HR;
+    M[m] = -INFINITY;
+    L[m] = 0.f;
+    for (int s = 0; s < p.nsplit; ++s) M[m] = fmaxf(M[m], p.part_ml[((part0 + s) * 16 + r) * 2]);
+    for (int s = 0; s < p.nsplit; ++s) {
+      const float ms = p.part_ml[((part0 + s) * 16 + r) * 2];
+      if (ms != -INFINITY) L[m] += p.part_ml[((part0 + s) * 16 + r) * 2 + 1] * exp2f(ms - M[m]);
+    }
+  }
+  constexpr int kMaxCols = 8;   // 256 value channels over 32 lanes
+  float d[kMaxCols], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kMaxCols; ++i) {
+    const int e = lane + 32 * i;
+    d[i] = 0.f;
+    if (e >= a.vdim) continue;
+    float o[MAPS];
+#pragma unroll
+    for (int m = 0; m < MAPS; ++m) {
+      const int r = h + m * HR;
+      o[m] = 0.f;
+      for (int s = 0; s < p.nsplit; ++s) {
+        const float ms = p.part_ml[((part0 + s) * 16 + r) * 2];
+        if (ms != -INFINITY) o[m] += p.part_acc[((part0 + s) * 16 + r) * a.vp + e] * exp2f(ms - M[m]);
+      }
+      o[m] = L[m] > 0.f ? o[m] / L[m] : 0.f;
+    }
+    d[i] = MAPS == 2 ? o[0] - a.lambda * o[MAPS - 1] : o[0];
+    ss = fmaf(d[i], d[i], ss);
+  }
+  const float r = MAPS == 2 ? a.out_scale / sqrtf(pi_warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
+  const size_t o0 = (size_t)row * a.out_stride + (size_t)head * a.vdim;
+#pragma unroll
+  for (int i = 0; i < kMaxCols; ++i)
+    if (lane + 32 * i < a.vdim) store_out(p, o0 + lane + 32 * i, d[i] * r);
+}
+
+constexpr int kTileWarps = 8, kTileKeys = 64;
+
+template <int MAPS, int KMAP, int VMAX>
+__global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcParams p) {
+  constexpr int RG = kTileWarps / MAPS, R = RG * 16;     // row groups of 16 rows
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const MapsParams& a = p.m;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int seq = p.portions[blockIdx.z], g = blockIdx.y, n = p.seq_n[seq];
+  const int per_tile = R / p.group;                      // tokens of a tile
+  // the last tiles see the most keys: they start first
+  const int tile = (int)gridDim.x - 1 - (int)blockIdx.x, tok0 = tile * per_tile;
+  if (tok0 >= n) {
+    pi_grid_dependency_wait();
+    return;
+  }
+  const int row0 = p.seq_row0[seq], start = p.seq_start[seq], n_tok = min(per_tile, n - tok0);
+  const int map = warp / RG, rg = warp % RG;
+  const int kw = MAPS * a.dp, nks = a.dp / 16, nv = a.vp / 8, kpitch = kw + 8, vpitch = a.vp + 8;
+  const int stage_elems = kTileKeys * (kpitch + vpitch);
+  __nv_bfloat16* sm = reinterpret_cast<__nv_bfloat16*>(smem_raw);
+  const Paged pg = {static_cast<const __nv_bfloat16*>(a.base), a.tables + (size_t)seq * a.max_blocks, a.block_size, a.kv_heads, g, kw, a.vp};
+  const int p_first = start + tok0, p_last = p_first + n_tok - 1;
+  const int lo = (a.window > 0 ? max(0, p_first - a.window + 1) : 0) & ~15, hi = min(p_last + 1, a.lens[seq] * a.block_size);
+  const int n_blocks = hi > lo ? (hi - lo + kTileKeys - 1) / kTileKeys : 0;
+
+  auto fetch = [&](int kb, int stage) {
+    __nv_bfloat16* ks = sm + (size_t)stage * stage_elems;
+    __nv_bfloat16* vs = ks + kTileKeys * kpitch;
+    const int t0 = lo + kb * kTileKeys;
+    // four threads per key: one table lookup serves all chunks of the row
+    const int r = tid >> 2, t = t0 + r;
+    const bool ok = t < hi;
+    const __nv_bfloat16* b = pg.base;
+    int off = 0;
+    if (ok) {
+      const int lb = t / a.block_size;
+      b = pg.tile(lb);
+      off = t - lb * a.block_size;
+    }
+    for (int x = (tid & 3) * 8; x < kw; x += 32)
+      cp_async16(smem_addr(ks + r * kpitch + x), ok ? (const void*)(b + (size_t)off * kw + x) : a.base, ok ? 16 : 0);
+    for (int x = (tid & 3) * 8; x < a.vp; x += 32)
+      cp_async16(smem_addr(vs + r * vpitch + x), ok ? (const void*)(b + (size_t)a.block_size * kw + (size_t)off * a.vp + x) : a.base, ok ? 16 : 0);
+  };
+
+  pi_grid_dependency_wait();
+  if (n_blocks > 0) fetch(0, 0);
+  cp_async_commit();
+
+  // this thread's two rows: lane / 4 and lane / 4 + 8 of the row group
+  int tpos[2];
+  uint32_t qa[KMAP][4];
+  {
+    const float* q[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = rg * 16 + (lane >> 2) + 8 * h, tok = r / p.group, head = r - tok * p.group;
+      const bool ok = tok < n_tok;
+      tpos[h] = ok ? p_first + tok : -1;      // -1: sees nothing
+      q[h] = ok ? a.q + (size_t)(row0 + tok0 + tok) * a.stride + ((size_t)(g * p.group + head) * MAPS + map) * a.dim : nullptr;
+    }
+#pragma unroll
+    for (int ks = 0; ks < KMAP; ++ks)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {           // a0: row, a1: row + 8, a2 / a3: channels + 8
+        const float* src = q[j & 1];
+        const int d = ks * 16 + (lane & 3) * 2 + (j >> 1) * 8;
+        qa[ks][j] = (ks < nks && src) ? pack(d < a.dim ? src[d] : 0.f, d + 1 < a.dim ? src[d + 1] : 0.f) : 0u;
+      }
+  }
+  float acc[VMAX / 8][4];
+#pragma unroll
+  for (int j = 0; j < VMAX / 8; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
+  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  const float sc = a.scale * kLog2e;
+  const int win = a.window > 0 ? a.window : 0x3fffffff;
+
+  for (int kb = 0; kb < n_blocks; ++kb) {
+    cp_async_wait<0>();
+    __syncthreads();                          // this block has landed, the other stage is free
+    if (kb + 1 < n_blocks) fetch(kb + 1, (kb + 1) & 1);
+    cp_async_commit();
+    const __nv_bfloat16* ks = sm + (size_t)(kb & 1) * stage_elems;
+    const __nv_bfloat16* vs = ks + kTileKeys * kpitch;
+    float s[kTileKeys / 8][4];
+#pragma unroll
+    for (int j = 0; j < kTileKeys / 8; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s[j][i] = 0.f;
+#pragma unroll
+    for (int k = 0; k < KMAP; ++k)
+      if (k < nks) {
+#pragma unroll
+        for (int j = 0; j < kTileKeys / 8; j += 2) {
+          uint32_t b[4];
+          ldsm4(b, smem_addr(ks + (size_t)(j * 8 + (lane & 7) + ((lane >> 4) << 3)) * kpitch + map * a.dp + k * 16 + ((lane >> 3) & 1) * 8));
+          mma(s[j], qa[k][0], qa[k][1], qa[k][2], qa[k][3], b[0], b[1]);
+          mma(s[j + 1], qa[k][0], qa[k][1], qa[k][2], qa[k][3], b[2], b[3]);
+        }
+      }
+    const int t0 = lo + kb * kTileKeys;
+    const bool inside = n_tok == per_tile && t0 + kTileKeys - 1 <= p_first && t0 > p_last - win && R == per_tile * p.group;
+    float keep[2], ref[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      float tm = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < kTileKeys / 8; ++j)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int t = t0 + j * 8 + (lane & 3) * 2 + i;
+          float& v = s[j][2 * h + i];
+          v = (inside || (t <= tpos[h] && t > tpos[h] - win && t < hi)) ? v * sc : -INFINITY;
+          tm = fmaxf(tm, v);
+        }
+      mx[h] = new_max(mx[h], quad_max(tm), keep[h]);
+      ref[h] = mx[h] == -INFINITY ? 0.f : mx[h];
+      l[h] *= keep[h];
+    }
+    if (__any_sync(0xffffffffu, keep[0] != 1.f || keep[1] != 1.f)) {
+#pragma unroll
+      for (int j = 0; j < VMAX / 8; ++j) {
+        acc[j][0] *= keep[0];
+        acc[j][1] *= keep[0];
+        acc[j][2] *= keep[1];
+        acc[j][3] *= keep[1];
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < kTileKeys / 16; ++c) {
+      uint32_t ph[4], pl[4];
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const float w0 = exp2f(s[2 * c + j][2 * h] - ref[h]), w1 = exp2f(s[2 * c + j][2 * h + 1] - ref[h]);
+          l[h] += w0 + w1;
+          split(w0, w1, ph[2 * j + h], pl[2 * j + h]);
+        }
+#pragma unroll
+      for (int j = 0; j < VMAX / 8; j += 2)
+        if (j < nv) {
+          uint32_t b[4];
+          ldsm4_t(b, smem_addr(vs + (size_t)(c * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * vpitch + j * 8 + (lane >> 4) * 8));
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            mma(acc[j + h], ph[0], ph[1], ph[2], ph[3], b[2 * h], b[2 * h + 1]);
+            mma(acc[j + h], pl[0], pl[1], pl[2], pl[3], b[2 * h], b[2 * h + 1]);
+          }
+        }
+    }
+  }
+  cp_async_wait<0>();
+  float inv[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const float t = quad_sum(l[h]);
+    inv[h] = t > 0.f ? 1.f / t : 0.f;
+  }
+  float ss[2] = {0.f, 0.f};
+  const int apitch = a.vp + 8, r0 = rg * 16 + (lane >> 2);
+  float* other = reinterpret_cast<float*>(smem_raw);     // [R][vp + 8]: the second map's rows
+  if (MAPS == 2) {
+    __syncthreads();
+    if (map == 1) {
+#pragma unroll
+      for (int j = 0; j < VMAX / 8; ++j)
+        if (j < nv) {
+          const int c = j * 8 + (lane & 3) * 2;
+          *reinterpret_cast<float2*>(other + (size_t)r0 * apitch + c) = make_float2(acc[j][0] * inv[0], acc[j][1] * inv[0]);
+          *reinterpret_cast<float2*>(other + (size_t)(r0 + 8) * apitch + c) = make_float2(acc[j][2] * inv[1], acc[j][3] * inv[1]);
+        }
+    }
+    __syncthreads();
+    if (map == 1) return;
+  }
+#pragma unroll
+  for (int j = 0; j < VMAX / 8; ++j)
+    if (j < nv) {
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          float& v = acc[j][2 * h + i];
+          v *= inv[h];
+          if (MAPS == 2) v -= a.lambda * other[(size_t)(r0 + 8 * h) * apitch + j * 8 + (lane & 3) * 2 + i];
+          ss[h] = fmaf(v, v, ss[h]);
+        }
+    }
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const float r = MAPS == 2 ? a.out_scale / sqrtf(quad_sum(ss[h]) / (float)a.vdim + a.eps) : 1.f;
+    const int rr = r0 + 8 * h, tok = rr / p.group, head = rr - tok * p.group;
+    if (tpos[h] < 0) continue;
+    const size_t o0 = (size_t)(row0 + tok0 + tok) * a.out_stride + (size_t)(g * p.group + head) * a.vdim;
+#pragma unroll
+    for (int j = 0; j < VMAX / 8; ++j)
+      if (j < nv) {
+        const int c = j * 8 + (lane & 3) * 2;
+        const float v0 = acc[j][2 * h] * r, v1 = acc[j][2 * h + 1] * r;
+        if (p.out_bf16 && c + 1 < a.vdim && ((o0 + c) & 1) == 0) {
+          *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(a.out) + o0 + c) = pack(v0, v1);
+        } else {
+          if (c < a.vdim) store_out(p, o0 + c, v0);
+          if (c + 1 < a.vdim) store_out(p, o0 + c + 1, v1);
+        }
+      }
+  }
+}
+
+size_t decode_smem(const MapsParams& a) {
+  const size_t ring = (size_t)kDecWarps * kDecStages * 16 * (a.maps * a.dp + 8 + a.vp + 8) * 2;
+  return std::max(ring, (size_t)kDecWarps * 16 * (a.vp + 4) * sizeof(float));
+}
+size_t tile_smem(const MapsParams& a) {
+  const size_t stages = (size_t)2 * kTileKeys * (a.maps * a.dp + 8 + a.vp + 8) * 2;
+  return std::max(stages, a.maps == 2 ? (size_t)(kTileWarps / 2) * 16 * (a.vp + 8) * sizeof(float) : (size_t)0);
+}
+
+typedef void (*TcKernel)(const TcParams);
+
+template <int MAPS, int VMAX>
+TcKernel pick_decode(int k) {
+  return k <= 8 ? maps_decode_kernel<MAPS, 8, VMAX> : maps_decode_kernel<MAPS, 16, VMAX>;
+}
+template <int MAPS>
+TcKernel pick_decode(int k, int vp) {
+  return vp <= 64 ? pick_decode<MAPS, 64>(k) : vp <= 128 ? pick_decode<MAPS, 128>(k) : pick_decode<MAPS, 256>(k);
+}
+template <int MAPS, int VMAX>
+TcKernel pick_tile(int k) {
+  return k <= 4 ? maps_tile_kernel<MAPS, 4, VMAX> : maps_tile_kernel<MAPS, 8, VMAX>;
+}
+template <int MAPS>
+TcKernel pick_tile(int k, int vp) {
+  return vp <= 64 ? pick_tile<MAPS, 64>(k) : vp <= 128 ? pick_tile<MAPS, 128>(k) : pick_tile<MAPS, 256>(k);
+}
+
+// The shared-memory limit of a kernel is raised once per device.
+cudaError_t grant(pi_ctx* ctx, TcKernel k, size_t smem) {
+  static std::vector<std::pair<TcKernel, pi_smem_grant>> granted;
+  for (auto& g : granted)
+    if (g.first == k) {
+      if (g.second.of(ctx) >= smem) return cudaSuccess;
+      g.second.of(ctx) = smem;
+      return cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    }
+  granted.push_back({k, pi_smem_grant()});
+  granted.back().second.of(ctx) = smem;
+  return smem > 48 * 1024 ? cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : cudaSuccess;
+}
+
+}  // namespace
+
+bool pi_maps_attention_tc_usable(const pi_ctx* ctx, const pi_maps_attention& a, const pi_kv_view& kv) {
+  return ctx->opt_tensor_gemm && kv.kind == PI_BF16 && kv.dp <= 128 && kv.vp <= 256 && a.heads / a.kv_heads <= 16 * kTileWarps / a.maps;
+}
+
+pi_status pi_launch_maps_attention_tc(pi_ctx* ctx, const MapsParams& a, int out_kind, const pi_seq_batch& b) {
+  TcParams p = {};
+  p.m = a;
+  p.out_bf16 = out_kind == PI_BF16;
+  p.group = a.heads / a.kv_heads;
+  p.rows = b.single_rows;
+  p.portions = b.portions;
+  p.seq_row0 = b.seq_row0;
+  p.seq_n = b.seq_n;
+  p.seq_start = b.seq_start;
+  if (b.n_portions > 0) {
+    const int per_tile = 16 * kTileWarps / a.maps / p.group, tiles = (b.max_portion + per_tile - 1) / per_tile;
+    const TcKernel k = a.maps == 2 ? pick_tile<2>(a.dp / 16, a.vp) : pick_tile<1>(a.dp / 16, a.vp);
+    const size_t smem = tile_smem(a);
+    PI_CUDA(ctx, grant(ctx, k, smem));
+    PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(tiles, a.kv_heads, b.n_portions), dim3(kTileWarps * 32), smem, 1, p));
+  }
+  if (b.n_single > 0) {
+    const int hr = 16 / a.maps;
+    p.ngroups = (p.group + hr - 1) / hr;
+    // KV splits: enough CTAs for the GPU, at least four 16-key tiles per warp
+    const int keys = a.window > 0 ? std::min(a.window, b.max_pos + 1) : b.max_pos + 1;
+    const long ctas = (long)b.n_single * a.kv_heads * p.ngroups;
+    const long want = (2L * ctx->sm_count + ctas - 1) / ctas, most = std::max(1, keys / (16 * kDecWarps * 2));
+    p.nsplit = (int)std::max(1L, std::min({want, most, 64L}));
+    if (p.nsplit > 1) {
+      const size_t parts = (size_t)ctas * p.nsplit * 16;
+      PI_TRY(pi_reserve(ctx, &ctx->attn_partial, parts * (a.vp + 2) * sizeof(float)));
+      p.part_acc = static_cast<float*>(ctx->attn_partial.ptr);
+      p.part_ml = p.part_acc + parts * a.vp;
+    }
+    const TcKernel k = a.maps == 2 ? pick_decode<2>(2 * a.dp / 16, a.vp) : pick_decode<1>(a.dp / 16, a.vp);
+    const size_t smem = decode_smem(a);
+    PI_CUDA(ctx, grant(ctx, k, smem));
+    PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(b.n_single, a.kv_heads * p.ngroups, p.nsplit), dim3(kDecWarps * 32), smem, 1, p));
+    if (p.nsplit > 1)
+      PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, a.maps == 2 ? maps_merge_kernel<2> : maps_merge_kernel<1>, dim3(b.n_single, (a.heads + 3) / 4),
+                                      dim3(128), 0, 1, p));
+  }
+  return PI_OK;
+}
