@@ -392,6 +392,11 @@ struct Staged {
   bool all_rows = false;               // every row, in order
 };
 
+// True when a projection over M rows takes bf16 activations (the tensor-core path).
+bool act_bf16(const pi_ctx* ctx, const pi_layered* m, int M) {
+  return m->c.compute == PI_BF16 && ctx->opt_tensor_gemm && M > ctx->opt_gemv_max_m;
+}
+
 pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_state_pool* state, const pi_step_batch* in, int extra_positions,
                 Staged* st) {
   PI_REQUIRE(ctx, in->n_seqs > 0 && in->tokens && in->n_tokens && in->start_pos && in->table_lens, "a step needs at least one sequence");
@@ -420,7 +425,7 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
       portions.push_back(i);
       max_portion = std::max(max_portion, k);
     }
-    if (m->chunked && k >= kRecurrenceChunk) {
+    if (m->chunked && k >= kRecurrenceChunk && act_bf16(ctx, m, k)) {
       for (int t = 0; t < k; t += kRecurrenceChunk) {
         chunks.push_back((int)chunk_seqs.size());
         chunks.push_back(t);
@@ -516,11 +521,6 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
   }
   if (m->trace_on) PI_TRY(pi_reserve(ctx, &m->trace, m->layers.size() * m->c.max_rows * m->c.width * sizeof(float)));
   return PI_OK;
-}
-
-// True when a projection over M rows takes bf16 activations (the tensor-core path).
-bool act_bf16(const pi_ctx* ctx, const pi_layered* m, int M) {
-  return m->c.compute == PI_BF16 && ctx->opt_tensor_gemm && M > ctx->opt_gemv_max_m;
 }
 
 pi_status project(pi_ctx* ctx, const pi_linear* lin, const void* in, size_t in_ld, int M, bool bf16, pi_linear_args a) {

@@ -93,9 +93,12 @@ inline size_t pi_recurrence_floats(int kind, int heads, int dim, int vdim) {
 pi_status pi_launch_recurrence(pi_ctx* ctx, const pi_recurrence& r, const float* proj, size_t stride, void* out, size_t out_stride,
                                int out_kind, const pi_seq_batch& b, float* scratch);
 size_t pi_recurrence_scratch_floats(const pi_recurrence& r, int n_chunks);
+// The chunked kernels (pi_recurrent_chunk.cu) for the sequences of b.chunk_seqs.
+pi_status pi_launch_recurrence_chunks(pi_ctx* ctx, const pi_recurrence& r, const float* proj, size_t stride, __nv_bfloat16* out, size_t out_stride,
+                                      const pi_seq_batch& b, float* scratch);
 // A portion of at least this many tokens takes the chunked kernels (when they hold the layer's sizes).
 constexpr int kRecurrenceChunk = 64;
-bool pi_recurrence_chunked(const pi_ctx* ctx, const pi_recurrence& r, int out_kind);
+bool pi_recurrence_chunked(const pi_ctx* ctx, const pi_recurrence& r, int compute);
 
 // ---- row-wise glue (pi_layered.cu) -----------------------------------------------------------------------------------
 template <typename K, typename... Args>

@@ -10,8 +10,8 @@
 // recur_scan_kernel walks the tokens of a sequence one by one with the state in registers: the decode kernel, and the
 // one that takes short portions.  A head's value channels are cut into slices of 128 columns; the CTAs of a head form
 // a thread-block cluster, which adds up the head's sum of squares through distributed shared memory and keeps the
-// shared n and m consistent (everybody reads them before anybody writes).  recur_scan_any_kernel is the same for key
-// sizes whose state does not fit the registers: the state stays in global memory.
+// shared n and m consistent (everybody reads them before anybody writes).  For key sizes whose state does not fit the
+// registers it stays in global memory (R = 0).  Long portions take the kernels of pi_recurrent_chunk.cu.
 #include <cooperative_groups.h>
 #include <math.h>
 
@@ -244,12 +244,8 @@ void (*pick_scan(int dim))(const RecParams) {
 
 }  // namespace
 
-bool pi_recurrence_chunked(const pi_ctx*, const pi_recurrence&, int) { return false; }
-size_t pi_recurrence_scratch_floats(const pi_recurrence&, int) { return 0; }
-
 pi_status pi_launch_recurrence(pi_ctx* ctx, const pi_recurrence& r, const float* proj, size_t stride, void* out, size_t out_stride,
                                int out_kind, const pi_seq_batch& b, float* scratch) {
-  (void)scratch;
   pi_prof_scope prof(ctx, PI_PROF_RECURRENCE);
   const int slices = (r.vdim + kSlice - 1) / kSlice;
   PI_REQUIRE(ctx, slices <= kMaxSlices && r.dim <= 1024, "recurrent heads of %d x %d channels are not supported (at most 1024 x %d)", r.dim,
@@ -262,6 +258,10 @@ pi_status pi_launch_recurrence(pi_ctx* ctx, const pi_recurrence& r, const float*
     else k = out_kind == PI_BF16 ? pick_scan<PI_REC_MLSTM, __nv_bfloat16>(r.dim) : pick_scan<PI_REC_MLSTM, float>(r.dim);
     const size_t smem = sizeof(float) * ((size_t)3 * r.dim + r.rank + 4 + kWarps * kSlice);
     PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(slices, r.heads, b.n_scan), dim3(kThreads), smem, slices, p));
+  }
+  if (b.n_chunks > 0) {
+    PI_REQUIRE(ctx, out_kind == PI_BF16 && scratch, "long portions run on the tensor-core path");
+    return pi_launch_recurrence_chunks(ctx, r, proj, stride, static_cast<__nv_bfloat16*>(out), out_stride, b, scratch);
   }
   return PI_OK;
 }
