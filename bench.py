@@ -907,6 +907,171 @@ def run_kernel_case(args):
                       "frac_of_hbm_peak": round(algo / us / 1e3 / hbm_peak, 3), "peak_kind": f"of {peak_kind}"}), flush=True)
 
 
+# ---- the layered design beside the closest uniform model ---------------------------------------------------------
+# Sizes that resemble a real model's layers, cut in depth so that both models fit comfortably.  Every layer of the layered
+# model has a feed-forward, so that a layer holds about as many weights as a Llama layer of the same width.
+LAYERED_SIZES = {
+    "w2048": dict(width=2048, ff=5632, vocab=32000, layers=21, window=1024,
+                  attention=dict(heads=16, kv_heads=4, dim=64, vdim=128), gla=dict(heads=16, dim=64, vdim=128), mlstm=dict(heads=8, dim=128, vdim=256),
+                  llama=dict(hidden_size=2048, num_attention_heads=32, num_key_value_heads=4, intermediate_size=5632)),
+    "w4096": dict(width=4096, ff=14336, vocab=32000, layers=6, window=1024,
+                  attention=dict(heads=32, kv_heads=8, dim=64, vdim=128), gla=dict(heads=32, dim=64, vdim=128), mlstm=dict(heads=16, dim=128, vdim=256),
+                  llama=dict(hidden_size=4096, num_attention_heads=32, num_key_value_heads=8, intermediate_size=14336)),
+}
+
+
+def layered_config(size):
+    from paged_infer_b200 import loader as ld
+    s = LAYERED_SIZES[size]
+    kinds = [ld.LayerConfig(ld.MIXER_ATTENTION, maps=2, window=s["window"], rot_dims=64, rot_base=500000.0, scale=0.125, diff=0.5, ff=s["ff"], **s["attention"]),
+             ld.LayerConfig(ld.MIXER_GLA, tau=16.0, ff=s["ff"], **s["gla"]),
+             ld.LayerConfig(ld.MIXER_MLSTM, gate_cap=15.0, ff=s["ff"], **s["mlstm"])]
+    return ld.LayeredConfig(s["width"], s["vocab"], 1e-6, [kinds[i % 3] for i in range(s["layers"])])
+
+
+def layered_work(cfg, model, B, ctx_len, M):
+    """Algorithmic bytes of a decode step (B sequences at ctx_len) and flops / bytes of a prefill of M tokens, by kernel class."""
+    from paged_infer_b200 import loader as ld
+    attn = [l for l in cfg.layers if l.mixer == ld.MIXER_ATTENTION]
+    rec = [l for l in cfg.layers if l.mixer != ld.MIXER_ATTENTION]
+    seen = sum(min(t + 1, attn[0].window) for t in range(M))
+    wb = model.weight_bytes()
+    body = (wb // 2 - cfg.vocab_size * cfg.width)
+    return {"decode_bytes": {"projections": wb, "attention": sum(B * min(ctx_len, l.window) * l.kv_heads * (l.maps * l.dim + l.vdim) * 2 for l in attn),
+                             "recurrence": 2 * B * model.state_bytes()},
+            "prefill_flops": {"gemm_tc": 2.0 * M * body, "attention": sum(l.heads * l.maps * 2 * (l.dim + l.vdim) * seen for l in attn)},
+            # f32 q, k, v, g in, bf16 result out, and the states between chunks of 64 tokens written and read once
+            "prefill_bytes": {"recurrence": sum(M * l.heads * (8 * l.dim + 10 * l.vdim) + 8 * (M // 64) * l.heads * l.dim * l.vdim for l in rec)}}
+
+
+def uniform_work(cfg, model, B, ctx_len, M):
+    wb = model.weight_bytes()
+    NL, H, KH, hd = cfg.num_hidden_layers, cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim
+    return {"decode_bytes": {"projections": wb, "attention": NL * B * ctx_len * KH * hd * 8},
+            "prefill_flops": {"gemm_tc": 2.0 * M * (wb - cfg.vocab_size * cfg.hidden_size), "attention": 4.0 * NL * H * hd * M * (M + 1) / 2},
+            "prefill_bytes": {}}
+
+
+def measure_steps(api, ctx, torch, model, work, ctx_len, batches, M, K, W, peaks):
+    """Decode (K device-resident greedy steps) at several batch sizes and prefill of one M-token portion, through the ragged step
+    call that the engine uses; per class its share of the device time and its roofline fraction."""
+    hbm, tflops = peaks
+    rng = np.random.default_rng(3)
+    out = {"weight_GB": round(model.weight_bytes() / 1e9, 3)}
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+
+    def timed(fn, reps):
+        fn()
+        total = 0.0
+        for _ in range(reps):
+            flush.fill_(0)            # nothing of the previous repetition is left in L2
+            torch.cuda.synchronize()
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            total += e0.elapsed_time(e1)
+        return total / reps
+
+    def classes(prof, ms_step, n_steps, achieved):
+        total = sum(ms for ms, _ in prof.values()) or 1e-9
+        r = {}
+        for c, (ms, n) in prof.items():
+            if n == 0:
+                continue
+            us = ms / total * ms_step * 1e3
+            r[c] = {"share": round(ms / total, 3), "us_per_step": round(us, 1), "launches_per_step": n / n_steps}
+            r[c].update(achieved(c, us))
+        return r
+
+    vocab = model.vocab_size()
+    per_seq = (ctx_len + K + W + 8) // BLOCK + 2
+    for B in batches:
+        kv = model.kv_pool(B * per_seq, BLOCK)
+        st = model.state_pool(B) if model.state_bytes() else None
+        tabs = [list(range(b * per_seq, (b + 1) * per_seq)) for b in range(B)]
+        for b in range(B):
+            model.step([rng.integers(0, vocab, ctx_len)], [0], [tabs[b]], kv, st, [b] if st else None, want_logits=False, want_argmax=True)
+        toks, pos, slots = rng.integers(0, vocab, B).tolist(), [ctx_len] * B, list(range(B)) if st else None
+        model.step_multi(toks, pos, tabs, kv, W, st, slots)
+        e0.record()
+        model.step_multi(toks, pos, tabs, kv, K, st, slots)
+        e1.record()
+        torch.cuda.synchronize()
+        ms = e0.elapsed_time(e1) / K
+        ctx.profile_begin()
+        model.step_multi(toks, pos, tabs, kv, 8, st, slots)
+        prof = ctx.profile_end()
+        w = work(B, ctx_len, M)["decode_bytes"]
+
+        def achieved(c, us):
+            key = "projections" if c in ("gemv", "gemm_tc") else c
+            if key not in w or (c == "gemv" and B > 4):
+                return {}
+            return {"GB/s": round(w[key] / us / 1e3, 1), "frac_hbm": round(w[key] / us / 1e3 / hbm, 3)}
+        out[f"decode_b{B}"] = {"ctx": ctx_len, "ms_per_step": round(ms, 3), "tok/s": round(B / ms * 1e3, 1), "classes": classes(prof, ms, 8, achieved)}
+        kv.close()
+        if st:
+            st.close()
+    kv = model.kv_pool(M // BLOCK + 1, BLOCK)
+    st = model.state_pool(1) if model.state_bytes() else None
+    prompt, tab = rng.integers(0, vocab, M), [list(range(M // BLOCK + 1))]
+    run = lambda: model.step([prompt], [0], tab, kv, st, [0] if st else None, want_logits=False, want_argmax=True)
+    run()
+    ms = timed(run, 5)
+    ctx.profile_begin()
+    run()
+    prof = ctx.profile_end()
+    w = work(1, ctx_len, M)
+
+    def achieved(c, us):
+        if c in w["prefill_flops"]:
+            return {"TFLOP/s": round(w["prefill_flops"][c] / us / 1e6, 1), "frac_bf16": round(w["prefill_flops"][c] / us / 1e6 / tflops, 3)}
+        if c in w["prefill_bytes"]:
+            return {"GB/s": round(w["prefill_bytes"][c] / us / 1e3, 1), "frac_hbm": round(w["prefill_bytes"][c] / us / 1e3 / hbm, 3)}
+        return {}
+    out[f"prefill_{M}"] = {"ms": round(ms, 3), "tok/s": round(M / ms * 1e3, 1), "classes": classes(prof, ms, 1, achieved)}
+    kv.close()
+    if st:
+        st.close()
+    return out
+
+
+def run_layered_workload(args):
+    """`--workload sumosun`: prefill and decode of the layered design at a few sizes, beside a Llama of the same width, depth,
+    feed-forward and vocabulary (random weights; bf16 there, int8 weights with f32 activations and KV here)."""
+    import torch
+    from paged_infer_b200 import api
+    from paged_infer_b200.loader import LlamaConfig
+    torch.cuda.set_device(0)
+    ctx = api.Context(0, torch.cuda.current_stream().cuda_stream)
+    hbm, tflops, kind = measured_peaks()
+    K, W = min(args.steps, 64), max(args.warmup, 3)
+    ctx_len, M, batches = 1024, 2048, (1, 8, 64)
+    clocks = ClockSampler(0)
+    clocks.start()
+    t0 = time.time()
+    res, launches = {}, ctx.kernel_launches()
+    for size, s in LAYERED_SIZES.items():
+        cfg = layered_config(size)
+        m = api.LayeredModel.synthetic(ctx, cfg, seed=1, max_rows=M)
+        res[size] = {"sumosun": measure_steps(api, ctx, torch, m, lambda B, c, n: layered_work(cfg, m, B, c, n), ctx_len, batches, M, K, W, (hbm, tflops))}
+        m.close()
+        lc = LlamaConfig(num_hidden_layers=s["layers"], vocab_size=s["vocab"], rms_norm_eps=1e-5, rope_theta=10000.0, quantization="int8", **s["llama"])
+        u = api.LlamaWeights.synthetic(ctx, lc, seed=1, std=0.02, max_batch=M, max_positions=M + 16)
+        res[size]["llama_int8"] = measure_steps(api, ctx, torch, u, lambda B, c, n: uniform_work(lc, u, B, c, n), ctx_len, batches, M, K, W, (hbm, tflops))
+        u.close()
+    t1 = time.time()
+    best = res["w2048"]["sumosun"]["decode_b64"]
+    print(json.dumps({"metric": "layered design: decode tokens/s at batch 64 (w2048)", "value": best["tok/s"], "unit": "tok/s", "n_gpus": 1, "steps": K,
+                      "warmup": W, "ms_per_step": best["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+                      "data": "synthetic", "config": {"model": "sumosun", "sizes": LAYERED_SIZES, "context": ctx_len, "prefill": M,
+                                                      "l2": "decode inputs exceed L2; flushed between prefill repetitions"},
+                      "gpu_launches": int(ctx.kernel_launches() - launches), "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind},
+                      "clocks": clocks.stop(t0, t1), "results": res}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--kernel-case", default=None,
@@ -916,7 +1081,7 @@ def main():
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="tinyllama_b64_paged", choices=["tinyllama_b64_paged", "llama3_8b_tp", "llama2_70b_tp"])
+    ap.add_argument("--workload", default="tinyllama_b64_paged", choices=["tinyllama_b64_paged", "llama3_8b_tp", "llama2_70b_tp", "sumosun"])
     ap.add_argument("--no-cpu", action="store_true", help="skip the cpu_baseline leg")
     ap.add_argument("--resident-only", action="store_true",
                     help="for a profiler's launch list: only the resident decode leg (warm-up + timed steps) over a pool filled with "
@@ -936,6 +1101,9 @@ def main():
         return
     if args.kernel_case:
         run_kernel_case(args)
+        return
+    if args.workload == "sumosun":
+        run_layered_workload(args)
         return
     if args.workload in TP_WORKLOADS:
         run_tp_workload(args, rank, world, local_rank)
