@@ -5,15 +5,19 @@
 //   8 heads x 2 maps: with two maps the query operand is block diagonal - rows 0-7 hold map 1 in the first half of the
 //   key channels and zero in the second, rows 8-15 the other way round - so one product over the concatenated channels
 //   scores both maps, and one product with V serves both.  Each warp streams 16-key tiles through a private ring of
-//   asynchronous copies; warps (and splits) merge by log-sum-exp.
+//   asynchronous copies; warps merge by log-sum-exp in shared memory, splits through the distributed shared memory of their
+//   cluster.
 // maps_tile_kernel: portions.  CTA = (sequence, kv head, tile of (token, head) rows); a warp owns 16 rows of one map, the
 //   pair of warps with the two maps of the same rows meets in shared memory at the end.  64-key tiles, double buffered.
+#include <cooperative_groups.h>
 #include <math.h>
 
 #include <algorithm>
 
 #include "pi_attention_maps.cuh"
 #include "pi_mma.cuh"
+
+namespace cg = cooperative_groups;
 
 namespace {
 using namespace pi_mma;
@@ -25,8 +29,6 @@ struct TcParams {
   const int32_t* rows;              // decode: the rows that stand alone
   const int32_t *portions, *seq_row0, *seq_n, *seq_start;
   int group, ngroups, nsplit;       // heads per kv head; decode: groups of them per MMA, KV splits
-  float* part_acc;                  // [row][kv head][group][split][16][vp]
-  float* part_ml;                   // [...][16][2]
   int out_bf16;
 };
 
@@ -52,7 +54,7 @@ __device__ __forceinline__ float new_max(float m, float s_max, float& keep) {
   return n;
 }
 
-constexpr int kDecWarps = 4, kDecStages = 3;
+constexpr int kDecWarps = 4, kDecStages = 3, kMaxSplits = 8;   // splits: a portable cluster
 
 template <int MAPS, int KMAX, int VMAX>
 __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcParams p) {
@@ -61,8 +63,8 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const MapsParams& a = p.m;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int ri = blockIdx.x, g = blockIdx.y / p.ngroups, grp = blockIdx.y % p.ngroups, split_i = blockIdx.z;
-  const int row = p.rows[ri], seq = a.row_seq[row], pos = a.row_pos[row];
+  const int g = blockIdx.z / p.ngroups, grp = blockIdx.z % p.ngroups, split_i = blockIdx.x;
+  const int row = p.rows[blockIdx.y], seq = a.row_seq[row], pos = a.row_pos[row];
   const int kw = MAPS * a.dp, ks_map = a.dp / 16, nks = MAPS * ks_map, nv = a.vp / 8;
   const int kpitch = kw + 8, vpitch = a.vp + 8;
   const int stage_elems = 16 * (kpitch + vpitch);
@@ -76,41 +78,62 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
   const int tile0 = t_first + split_i * per + warp;
   const bool one_block = a.block_size % 16 == 0;
 
-  auto fetch = [&](int tile, int stage) {
+  const int kpr = kw / 8, vpr = a.vp / 8;               // 16-byte pieces per row
+  // physical block of a tile that lies in one block; loaded one tile ahead of its use
+  auto block_of = [&](int tile) { return one_block && tile < tile_end ? pg.table[tile * 16 / a.block_size] : 0; };
+  auto fetch = [&](int tile, int stage, int pb) {
     __nv_bfloat16* ks = ring + (size_t)stage * stage_elems;
     __nv_bfloat16* vs = ks + 16 * kpitch;
     const int t0 = tile * 16;
-    const __nv_bfloat16* base = nullptr;
-    int off0 = 0;
-    if (one_block) {
-      base = pg.tile(t0 / a.block_size);
-      off0 = t0 % a.block_size;
-    }
-    auto copy = [&](__nv_bfloat16* dst, int pitch, int width, bool is_v) {
-      const int per_row = width / 8;
-      for (int c = lane; c < 16 * per_row; c += 32) {
-        const int r = c / per_row, x = (c - r * per_row) * 8, t = t0 + r;
-        const bool ok = t < hi;
-        const __nv_bfloat16* b = base;
-        int off = off0 + r;
-        if (!one_block && ok) {
-          b = pg.tile(t / a.block_size);
-          off = t % a.block_size;
+    if (one_block) {                                    // 16 rows of K in a piece, 16 rows of V in a piece
+      const int off = t0 % a.block_size;
+      const __nv_bfloat16* kb = pg.base + ((size_t)pb * a.kv_heads + g) * ((size_t)a.block_size * (kw + a.vp));
+      const __nv_bfloat16* vb = kb + (size_t)a.block_size * kw + (size_t)off * a.vp;
+      kb += (size_t)off * kw;
+      auto copy = [&](__nv_bfloat16* dst, int pitch, int pr, const __nv_bfloat16* src) {
+        int r = lane / pr, x = lane - r * pr;
+        const int dr = 32 / pr, dx = 32 - dr * pr;
+#pragma unroll 4
+        for (int c = lane; c < 16 * pr; c += 32) {
+          cp_async16(smem_addr(dst + r * pitch + x * 8), src + (size_t)c * 8, t0 + r < hi ? 16 : 0);
+          r += dr;
+          x += dx;
+          if (x >= pr) {
+            x -= pr;
+            ++r;
+          }
         }
-        const __nv_bfloat16* src = is_v ? b + (size_t)a.block_size * kw + (size_t)off * a.vp + x : b + (size_t)off * kw + x;
-        cp_async16(smem_addr(dst + r * pitch + x), ok ? (const void*)src : a.base, ok ? 16 : 0);
+      };
+      copy(ks, kpitch, kpr, kb);
+      copy(vs, vpitch, vpr, vb);
+      return;
+    }
+    auto copy = [&](__nv_bfloat16* dst, int pitch, int pr, bool is_v) {
+      for (int c = lane; c < 16 * pr; c += 32) {
+        const int r = c / pr, x = (c - r * pr) * 8, t = t0 + r;
+        const bool ok = t < hi;
+        const __nv_bfloat16* src = pg.base;
+        if (ok) {
+          const int off = t % a.block_size;
+          src = pg.tile(t / a.block_size) + (is_v ? (size_t)a.block_size * kw + (size_t)off * a.vp + x : (size_t)off * kw + x);
+        }
+        cp_async16(smem_addr(dst + r * pitch + x), src, ok ? 16 : 0);
       }
     };
-    copy(ks, kpitch, kw, false);
-    copy(vs, vpitch, a.vp, true);
+    copy(ks, kpitch, kpr, false);
+    copy(vs, vpitch, vpr, true);
   };
 
+  int pb[kDecStages];
+#pragma unroll
+  for (int s = 0; s < kDecStages; ++s) pb[s] = block_of(tile0 + s * kDecWarps);
   pi_grid_dependency_wait();
 #pragma unroll
   for (int s = 0; s < kDecStages - 1; ++s) {
-    if (tile0 + s * kDecWarps < tile_end) fetch(tile0 + s * kDecWarps, s);
+    if (tile0 + s * kDecWarps < tile_end) fetch(tile0 + s * kDecWarps, s, pb[s]);
     cp_async_commit();
   }
+  int pb_next = pb[kDecStages - 1];
 
   // query operand: row r of the MMA = (map r / HR, head r % HR)
   uint32_t qa[KMAX][QR];
@@ -217,7 +240,9 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
       }
     }
     const int next = tile + (kDecStages - 1) * kDecWarps;
-    if (next < tile_end) fetch(next, (stage + kDecStages - 1) % kDecStages);
+    const int pb_now = pb_next;
+    pb_next = block_of(next + kDecWarps);
+    if (next < tile_end) fetch(next, (stage + kDecStages - 1) % kDecStages, pb_now);
     cp_async_commit();
     stage = (stage + 1) % kDecStages;
   }
@@ -248,102 +273,77 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
     }
   }
   __syncthreads();
-  const size_t part = (((size_t)ri * a.kv_heads + g) * p.ngroups + grp) * p.nsplit + split_i;
-  for (int h = warp; h < HR; h += kDecWarps) {
+  // the CTA's own result, not yet divided by the sum of weights, replaces warp 0's part
+  __shared__ float c_m[16], c_l[16];
+  for (int r = warp; r < 16; r += kDecWarps) {
+    float f[kDecWarps], M = -INFINITY, L = 0.f;
+#pragma unroll
+    for (int w = 0; w < kDecWarps; ++w) M = fmaxf(M, s_m[w][r]);
+#pragma unroll
+    for (int w = 0; w < kDecWarps; ++w) {
+      f[w] = s_m[w][r] == -INFINITY ? 0.f : exp2f(s_m[w][r] - M);
+      L += s_l[w][r] * f[w];
+    }
+    for (int e = lane; e < a.vp; e += 32) {
+      float o = 0.f;
+#pragma unroll
+      for (int w = 0; w < kDecWarps; ++w) o = fmaf(wacc[((size_t)w * 16 + r) * apitch + e], f[w], o);
+      wacc[(size_t)r * apitch + e] = o;
+    }
+    if (lane == 0) {
+      c_m[r] = M;
+      c_l[r] = L;
+    }
+  }
+  // the splits of a row form a cluster: each of them finishes its share of the heads, adding the splits in rank order
+  cg::cluster_group cluster = cg::this_cluster();
+  if (p.nsplit > 1) cluster.sync();
+  else __syncthreads();
+  const int rank = p.nsplit > 1 ? (int)cluster.block_rank() : 0;
+  for (int h = warp * p.nsplit + rank; h < HR; h += kDecWarps * p.nsplit) {
     const int head = grp * HR + h;
     if (head >= p.group) continue;
-    float f[MAPS][kDecWarps];
+    float f[MAPS][kMaxSplits];
 #pragma unroll
     for (int m = 0; m < MAPS; ++m) {
       const int r = h + m * HR;
       float M = -INFINITY, L = 0.f;
 #pragma unroll
-      for (int w = 0; w < kDecWarps; ++w) M = fmaxf(M, s_m[w][r]);
-#pragma unroll
-      for (int w = 0; w < kDecWarps; ++w) {
-        f[m][w] = s_m[w][r] == -INFINITY ? 0.f : exp2f(s_m[w][r] - M);
-        L += s_l[w][r] * f[m][w];
+      for (int c = 0; c < kMaxSplits; ++c) {
+        f[m][c] = c < p.nsplit ? (p.nsplit > 1 ? cluster.map_shared_rank(c_m, c)[r] : c_m[r]) : -INFINITY;
+        M = fmaxf(M, f[m][c]);
       }
-      if (p.nsplit == 1) {
 #pragma unroll
-        for (int w = 0; w < kDecWarps; ++w) f[m][w] = L > 0.f ? f[m][w] / L : 0.f;
-      } else if (lane == 0) {
-        p.part_ml[(part * 16 + r) * 2] = M;
-        p.part_ml[(part * 16 + r) * 2 + 1] = L;
+      for (int c = 0; c < kMaxSplits; ++c) {
+        f[m][c] = f[m][c] == -INFINITY ? 0.f : exp2f(f[m][c] - M);
+        if (c < p.nsplit) L = fmaf(p.nsplit > 1 ? cluster.map_shared_rank(c_l, c)[r] : c_l[r], f[m][c], L);
       }
+#pragma unroll
+      for (int c = 0; c < kMaxSplits; ++c) f[m][c] = L > 0.f ? f[m][c] / L : 0.f;
     }
-    float ss = 0.f;
-    for (int e = lane; e < a.vp; e += 32) {
-      float o[MAPS];
+    float d[VMAX / 32], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VMAX / 32; ++i) {
+      const int e = lane + 32 * i;
+      d[i] = 0.f;
+      if (e >= a.vdim) continue;
 #pragma unroll
       for (int m = 0; m < MAPS; ++m) {
-        o[m] = 0.f;
+        float o = 0.f;
 #pragma unroll
-        for (int w = 0; w < kDecWarps; ++w) o[m] += wacc[((size_t)w * 16 + h + m * HR) * apitch + e] * f[m][w];
-        if (p.nsplit > 1) p.part_acc[(part * 16 + h + m * HR) * a.vp + e] = o[m];
+        for (int c = 0; c < kMaxSplits; ++c)
+          if (c < p.nsplit) o = fmaf((p.nsplit > 1 ? cluster.map_shared_rank(wacc, c) : wacc)[(size_t)(h + m * HR) * apitch + e], f[m][c], o);
+        d[i] = m == 0 ? o : d[i] - a.lambda * o;
       }
-      if (p.nsplit == 1) {
-        const float d = MAPS == 2 ? o[0] - a.lambda * o[MAPS - 1] : o[0];
-        ss = fmaf(d, d, ss);
-        wacc[(size_t)h * apitch + e] = d;   // this lane alone reads column e of row h (warp 0's area)
-      }
+      ss = fmaf(d[i], d[i], ss);
     }
-    if (p.nsplit == 1) {
-      const float r = MAPS == 2 ? a.out_scale / sqrtf(pi_warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
-      const size_t o0 = (size_t)row * a.out_stride + (size_t)(g * p.group + head) * a.vdim;
-      for (int e = lane; e < a.vdim; e += 32) store_out(p, o0 + e, wacc[(size_t)h * apitch + e] * r);
-    }
+    const float r = MAPS == 2 ? a.out_scale / sqrtf(pi_warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
+    const size_t o0 = (size_t)row * a.out_stride + (size_t)(g * p.group + head) * a.vdim;
+#pragma unroll
+    for (int i = 0; i < VMAX / 32; ++i)
+      if (lane + 32 * i < a.vdim) store_out(p, o0 + lane + 32 * i, d[i] * r);
   }
-}
-
-// Merge the KV splits of a row: one warp per head.
-template <int MAPS>
-__global__ void __launch_bounds__(128) maps_merge_kernel(const TcParams p) {
-  constexpr int HR = 16 / MAPS;
-  const MapsParams& a = p.m;
-  const int ri = blockIdx.x, lane = threadIdx.x & 31, head = blockIdx.y * 4 + (threadIdx.x >> 5);
-  pi_grid_dependency_wait();
-  if (head >= a.heads) return;
-  const int row = p.rows[ri], g = head / p.group, hg = head % p.group, grp = hg / HR, h = hg % HR;
-  const size_t part0 = (((size_t)ri * a.kv_heads + g) * p.ngroups + grp) * p.nsplit;
-  float M[MAPS], L[MAPS];
-#pragma unroll
-  for (int m = 0; m < MAPS; ++m) {
-    const int r = h + m * HR;
-    M[m] = -INFINITY;
-    L[m] = 0.f;
-    for (int s = 0; s < p.nsplit; ++s) M[m] = fmaxf(M[m], p.part_ml[((part0 + s) * 16 + r) * 2]);
-    for (int s = 0; s < p.nsplit; ++s) {
-      const float ms = p.part_ml[((part0 + s) * 16 + r) * 2];
-      if (ms != -INFINITY) L[m] += p.part_ml[((part0 + s) * 16 + r) * 2 + 1] * exp2f(ms - M[m]);
-    }
-  }
-  constexpr int kMaxCols = 8;   // 256 value channels over 32 lanes
-  float d[kMaxCols], ss = 0.f;
-#pragma unroll
-  for (int i = 0; i < kMaxCols; ++i) {
-    const int e = lane + 32 * i;
-    d[i] = 0.f;
-    if (e >= a.vdim) continue;
-    float o[MAPS];
-#pragma unroll
-    for (int m = 0; m < MAPS; ++m) {
-      const int r = h + m * HR;
-      o[m] = 0.f;
-      for (int s = 0; s < p.nsplit; ++s) {
-        const float ms = p.part_ml[((part0 + s) * 16 + r) * 2];
-        if (ms != -INFINITY) o[m] += p.part_acc[((part0 + s) * 16 + r) * a.vp + e] * exp2f(ms - M[m]);
-      }
-      o[m] = L[m] > 0.f ? o[m] / L[m] : 0.f;
-    }
-    d[i] = MAPS == 2 ? o[0] - a.lambda * o[MAPS - 1] : o[0];
-    ss = fmaf(d[i], d[i], ss);
-  }
-  const float r = MAPS == 2 ? a.out_scale / sqrtf(pi_warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
-  const size_t o0 = (size_t)row * a.out_stride + (size_t)head * a.vdim;
-#pragma unroll
-  for (int i = 0; i < kMaxCols; ++i)
-    if (lane + 32 * i < a.vdim) store_out(p, o0 + lane + 32 * i, d[i] * r);
+  if (p.nsplit > 1) cluster.sync();   // a peer may still be reading this CTA's part
 }
 
 constexpr int kTileWarps = 8, kTileKeys = 64;
@@ -627,24 +627,14 @@ pi_status pi_launch_maps_attention_tc(pi_ctx* ctx, const MapsParams& a, int out_
   if (b.n_single > 0) {
     const int hr = 16 / a.maps;
     p.ngroups = (p.group + hr - 1) / hr;
-    // KV splits: enough CTAs for the GPU, at least four 16-key tiles per warp
-    const int keys = a.window > 0 ? std::min(a.window, b.max_pos + 1) : b.max_pos + 1;
-    const long ctas = (long)b.n_single * a.kv_heads * p.ngroups;
-    const long want = (2L * ctx->sm_count + ctas - 1) / ctas, most = std::max(1, keys / (16 * kDecWarps * 2));
-    p.nsplit = (int)std::max(1L, std::min({want, most, 64L}));
-    if (p.nsplit > 1) {
-      const size_t parts = (size_t)ctas * p.nsplit * 16;
-      PI_TRY(pi_reserve(ctx, &ctx->attn_partial, parts * (a.vp + 2) * sizeof(float)));
-      p.part_acc = static_cast<float*>(ctx->attn_partial.ptr);
-      p.part_ml = p.part_acc + parts * a.vp;
-    }
+    // KV splits: one round of CTAs over the GPU, at least one 16-key tile per warp
     const TcKernel k = a.maps == 2 ? pick_decode<2>(2 * a.dp / 16, a.vp) : pick_decode<1>(a.dp / 16, a.vp);
     const size_t smem = decode_smem(a);
     PI_CUDA(ctx, grant(ctx, k, smem));
-    PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(b.n_single, a.kv_heads * p.ngroups, p.nsplit), dim3(kDecWarps * 32), smem, 1, p));
-    if (p.nsplit > 1)
-      PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, a.maps == 2 ? maps_merge_kernel<2> : maps_merge_kernel<1>, dim3(b.n_single, (a.heads + 3) / 4),
-                                      dim3(128), 0, 1, p));
+    const int keys = a.window > 0 ? std::min(a.window, b.max_pos + 1) : b.max_pos + 1;
+    const long ctas = (long)b.n_single * a.kv_heads * p.ngroups, resident = ctx->sm_count * std::max(1L, (long)(ctx->smem_optin / (smem + 2048)));
+    p.nsplit = (int)std::max(1L, std::min({resident / ctas, (long)keys / (16 * kDecWarps), (long)kMaxSplits}));
+    PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(p.nsplit, b.n_single, a.kv_heads * p.ngroups), dim3(kDecWarps * 32), smem, p.nsplit, p));
   }
   return PI_OK;
 }

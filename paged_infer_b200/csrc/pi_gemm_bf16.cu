@@ -376,7 +376,10 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
   if (a.residual) p.res = *a.residual;
   p.err_flag = ctx->dev_err;
   int bn = a.M <= 16 ? 16 : a.M <= 32 ? 32 : a.M <= 64 ? 64 : 128;
-  if (a.M > 128 && p.rtiles * ((a.M + 255) / 256) >= ctx->sm_count) bn = 256;
+  if (a.M > 128) {   // the wider tile where it does not cost more rounds of tiles over the SMs
+    const long t128 = (long)p.rtiles * ((a.M + 127) / 128), t256 = (long)p.rtiles * ((a.M + 255) / 256), sms = ctx->sm_count;
+    if ((t256 + sms - 1) / sms * 2 <= (t128 + sms - 1) / sms) bn = 256;
+  }
   p.tiles = p.rtiles * ((a.M + bn - 1) / bn);
   CUtensorMap w, x;
   PI_TRY(encode_2d(ctx, &w, lin->w, lin->cols, lin->rows, lin->ld, kTM));

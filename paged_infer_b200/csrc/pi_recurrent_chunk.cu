@@ -45,6 +45,7 @@ struct ChunkParams {
   float* FG;       // [chunk][head][2]              mLSTM: F and G at the chunk's end
   float* m_in;     // [chunk][head]                 mLSTM
   int dimp, vdimp;   // rounded up to 16
+  bool vec_k, vec_v;   // 16-byte loads of keys and queries / of values, output gates and state rows
 };
 
 struct ChunkAt {
@@ -65,22 +66,30 @@ __device__ __forceinline__ void gla_decays(const ChunkParams& p, const ChunkAt& 
   const pi_recurrence& r = p.r;
   for (int i = threadIdx.x; i < C * r.rank; i += kChunkThreads) {
     const int t = i / r.rank, j = i - t * r.rank;
-    low[i] = t < at.n ? p.proj[(size_t)(at.row0 + t) * p.stride + r.col_low + j] : 0.f;
+    low[i] = t < at.n ? __ldg(p.proj + (size_t)(at.row0 + t) * p.stride + r.col_low + j) : 0.f;
   }
   __syncthreads();
   for (int i = threadIdx.x; i < NSUB * p.dimp; i += kChunkThreads) {
-    const int J = i / p.dimp, d = i - J * p.dimp;
-    float b = 0.f;
-    const int c = head * r.dim + d;
-    const float* w = r.a2 + (size_t)c * r.rank;
-    const float bias = d < r.dim ? r.a2_b[c] : 0.f;
-    for (int t = J * SUB; t < (J + 1) * SUB; ++t) {
-      if (d < r.dim && t < at.n) {
-        float z = 0.f;
-        for (int j = 0; j < r.rank; ++j) z = fmaf(__ldg(w + j), low[t * r.rank + j], z);
-        b += pi_log_sigmoid(z + bias) / r.tau;
+    const int J = i / p.dimp, d = i - J * p.dimp, c = head * r.dim + d;
+    float z[SUB];
+#pragma unroll
+    for (int t = 0; t < SUB; ++t) z[t] = 0.f;
+    if (d < r.dim) {
+      const float* w = r.a2 + (size_t)c * r.rank;
+      for (int j = 0; j < r.rank; ++j) {
+        const float wj = __ldg(w + j);
+#pragma unroll
+        for (int t = 0; t < SUB; ++t) z[t] = fmaf(wj, low[(J * SUB + t) * r.rank + j], z[t]);
       }
-      bl[t * p.dimp + d] = b;
+      const float bias = __ldg(r.a2_b + c);
+#pragma unroll
+      for (int t = 0; t < SUB; ++t) z[t] = J * SUB + t < at.n ? pi_log_sigmoid(z[t] + bias) / r.tau : 0.f;
+    }
+    float b = 0.f;
+#pragma unroll
+    for (int t = 0; t < SUB; ++t) {
+      b += z[t];
+      bl[(J * SUB + t) * p.dimp + d] = b;
     }
     tot[J * p.dimp + d] = b;
   }
@@ -134,15 +143,51 @@ __device__ __forceinline__ void store_split(__nv_bfloat16* hi, __nv_bfloat16* lo
   hi[i] = h;
   lo[i] = __float2bfloat16_rn(v - __bfloat162float(h));
 }
+__device__ __forceinline__ void store_split4(__nv_bfloat16* hi, __nv_bfloat16* lo, int i, float4 v) {   // i: a multiple of 4
+  uint2 h, l;
+  split(v.x, v.y, h.x, l.x);
+  split(v.z, v.w, h.y, l.y);
+  *reinterpret_cast<uint2*>(hi + i) = h;
+  *reinterpret_cast<uint2*>(lo + i) = l;
+}
+
+// Four adjacent values, of which the first `n` exist (vec: 16-byte loads are possible where all four do).
+__device__ __forceinline__ float4 load4(const float* src, int n, bool vec) {
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (n >= 4 && vec) return __ldg(reinterpret_cast<const float4*>(src));
+  if (n > 0) v.x = __ldg(src);
+  if (n > 1) v.y = __ldg(src + 1);
+  if (n > 2) v.z = __ldg(src + 2);
+  if (n > 3) v.w = __ldg(src + 3);
+  return v;
+}
+// rows x cols (cols a multiple of 4) walked by the CTA four columns at a time, several loads in flight per thread before the
+// first of them is used: load(row, col) -> float4, use(row, col, float4).
+template <typename L, typename F>
+__device__ __forceinline__ void staged(int rows, int cols, L&& load, F&& use) {
+  constexpr int U = 4;
+  const int c4 = cols >> 2, count = rows * c4;
+  for (int i0 = threadIdx.x; i0 < count; i0 += U * kChunkThreads) {
+    float4 v[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * kChunkThreads;
+      if (i < count) v[u] = load(i / c4, (i % c4) * 4);
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * kChunkThreads;
+      if (i < count) use(i / c4, (i % c4) * 4, v[u]);
+    }
+  }
+}
 
 // value columns [c0, c0 + cols) of the chunk as two planes [C][pitch]
 __device__ __forceinline__ void load_v(const ChunkParams& p, const ChunkAt& at, int head, int c0, int cols, __nv_bfloat16* hi, __nv_bfloat16* lo,
                                        int pitch) {
-  for (int i = threadIdx.x; i < C * cols; i += kChunkThreads) {
-    const int t = i / cols, e = i - t * cols;
-    const float v = (t < at.n && c0 + e < p.r.vdim) ? p.proj[(size_t)(at.row0 + t) * p.stride + p.r.col_v + (size_t)head * p.r.vdim + c0 + e] : 0.f;
-    store_split(hi, lo, t * pitch + e, v);
-  }
+  const float* src = p.proj + (size_t)at.row0 * p.stride + p.r.col_v + (size_t)head * p.r.vdim + c0;
+  staged(C, cols, [&](int t, int e) { return load4(src + (size_t)t * p.stride + e, t < at.n ? p.r.vdim - c0 - e : 0, p.vec_v); },
+         [&](int t, int e, float4 v) { store_split4(hi, lo, t * pitch + e, v); });
 }
 
 template <int KIND>
@@ -176,21 +221,23 @@ __global__ void __launch_bounds__(kChunkThreads) recur_local_kernel(const ChunkP
       p.FG[2 * ch + 1] = G[C - 1];
     }
   }
-  for (int i = tid; i < C * p.dimp; i += kChunkThreads) {
-    const int t = i / p.dimp, d = i - t * p.dimp;
-    float v = 0.f;
-    if (t < at.n && d < r.dim) {
-      v = p.proj[(size_t)(at.row0 + t) * p.stride + r.col_k + (size_t)head * r.dim + d];
-      if (KIND == PI_REC_GLA) {
-        float e = tot[(t / SUB) * p.dimp + d] - bl[t * p.dimp + d];
-        for (int J = t / SUB + 1; J < NSUB; ++J) e += tot[J * p.dimp + d];
-        v *= expf(e);
-      } else {
-        v *= expf(F[C - 1] - F[t] + li[t] - G[C - 1]);   // the chunk's state is kept times e^-G
-      }
-    }
-    store_split(khi, klo, t * kp + d, v);
-  }
+  const float* ksrc = p.proj + (size_t)at.row0 * p.stride + r.col_k + (size_t)head * r.dim;
+  staged(C, p.dimp, [&](int t, int d) { return load4(ksrc + (size_t)t * p.stride + d, t < at.n ? r.dim - d : 0, p.vec_k); },
+         [&](int t, int d, float4 v) {
+           if (KIND == PI_REC_GLA) {
+             float4 e = make_float4(0.f, 0.f, 0.f, 0.f);
+             for (int J = t / SUB; J < NSUB; ++J) {
+               const float4 x = *reinterpret_cast<const float4*>(tot + J * p.dimp + d);
+               e = make_float4(e.x + x.x, e.y + x.y, e.z + x.z, e.w + x.w);
+             }
+             const float4 b = *reinterpret_cast<const float4*>(bl + t * p.dimp + d);
+             v = make_float4(v.x * expf(e.x - b.x), v.y * expf(e.y - b.y), v.z * expf(e.z - b.z), v.w * expf(e.w - b.w));
+           } else {
+             const float f = t < at.n ? expf(F[C - 1] - F[t] + li[t] - G[C - 1]) : 0.f;   // the chunk's state is kept times e^-G
+             v = make_float4(v.x * f, v.y * f, v.z * f, v.w * f);
+           }
+           store_split4(khi, klo, t * kp + d, v);
+         });
   load_v(p, at, head, 0, p.vdimp, vhi, vlo, vp);
   __syncthreads();
   if (KIND == PI_REC_MLSTM) {
@@ -366,22 +413,24 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
       st[(size_t)r.heads * r.dim * r.vdim + (size_t)r.heads * r.dim + head] = fmaxf(F[C - 1] + m_in, G[C - 1]);
     }
   }
-  for (int i = tid; i < C * p.dimp; i += kChunkThreads) {
-    const int t = i / p.dimp, d = i - t * p.dimp;
-    float q = 0.f, k = 0.f;
-    if (t < at.n && d < r.dim) {
-      const float* x = p.proj + (size_t)(at.row0 + t) * p.stride + (size_t)head * r.dim + d;
-      q = x[r.col_q] * r.q_scale;
-      k = x[r.col_k];
-      if (KIND == PI_REC_GLA) {
-        const float b = bl[t * p.dimp + d];
-        q *= expf(b);
-        k *= expf(tot[(t / SUB) * p.dimp + d] - b);
-      }
-    }
-    qf[t * qp + d] = q;
-    store_split(khi, klo, t * kp + d, k);
-  }
+  const float* src = p.proj + (size_t)at.row0 * p.stride + (size_t)head * r.dim;
+  staged(C, p.dimp, [&](int t, int d) { return load4(src + r.col_q + (size_t)t * p.stride + d, t < at.n ? r.dim - d : 0, p.vec_k); },
+         [&](int t, int d, float4 v) {
+           float4 e = make_float4(r.q_scale, r.q_scale, r.q_scale, r.q_scale);
+           if (KIND == PI_REC_GLA) {
+             const float4 b = *reinterpret_cast<const float4*>(bl + t * p.dimp + d);
+             e = make_float4(e.x * expf(b.x), e.y * expf(b.y), e.z * expf(b.z), e.w * expf(b.w));
+           }
+           *reinterpret_cast<float4*>(qf + t * qp + d) = make_float4(v.x * e.x, v.y * e.y, v.z * e.z, v.w * e.w);
+         });
+  staged(C, p.dimp, [&](int t, int d) { return load4(src + r.col_k + (size_t)t * p.stride + d, t < at.n ? r.dim - d : 0, p.vec_k); },
+         [&](int t, int d, float4 v) {
+           if (KIND == PI_REC_GLA) {
+             const float4 b = *reinterpret_cast<const float4*>(bl + t * p.dimp + d), e = *reinterpret_cast<const float4*>(tot + (t / SUB) * p.dimp + d);
+             v = make_float4(v.x * expf(e.x - b.x), v.y * expf(e.y - b.y), v.z * expf(e.z - b.z), v.w * expf(e.w - b.w));
+           }
+           store_split4(khi, klo, t * kp + d, v);
+         });
   __syncthreads();
 
   // A fragments of 16 query rows at k step ks, times a factor per channel
@@ -464,10 +513,8 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
     __syncthreads();            // the last slice (or the decays in its place) has been read
     load_v(p, at, head, c0, kVS, vhi, vlo, vp);
     const float* S = p.U + ch * r.dim * r.vdim;
-    for (int i = tid; i < p.dimp * kVS; i += kChunkThreads) {
-      const int d = i / kVS, e = i - d * kVS;
-      store_split(shi, slo, d * vp + e, (d < r.dim && c0 + e < r.vdim) ? S[(size_t)d * r.vdim + c0 + e] : 0.f);
-    }
+    staged(p.dimp, kVS, [&](int d, int e) { return load4(S + (size_t)d * r.vdim + c0 + e, d < r.dim ? r.vdim - c0 - e : 0, p.vec_v); },
+           [&](int d, int e, float4 v) { store_split4(shi, slo, d * vp + e, v); });
     __syncthreads();
     float (&acc)[4][4] = o[sl];
 #pragma unroll
@@ -549,14 +596,23 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
 #pragma unroll
     for (int sl = 0; sl < kMaxVdim / kVS; ++sl) {
       if (sl * kVS >= p.vdimp) break;
+      float gv[4][2], wv[4][2];
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int e = min(sl * kVS + half * 32 + j * 8 + (lane & 3) * 2 + i, r.vdim - 1);
+          gv[j][i] = __ldg(g + e);
+          wv[j][i] = __ldg(nw + e);
+        }
 #pragma unroll
       for (int j = 0; j < 4; ++j)
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
           const int e = sl * kVS + half * 32 + j * 8 + (lane & 3) * 2 + i;
           if (e >= r.vdim) continue;
-          const float gv = g[e], gate = r.gate_sigmoid ? pi_sigmoid(gv) : gv * pi_sigmoid(gv);
-          out[e] = __float2bfloat16_rn(o[sl][j][2 * h + i] * inv * nw[e] * gate);
+          const float gate = r.gate_sigmoid ? pi_sigmoid(gv[j][i]) : gv[j][i] * pi_sigmoid(gv[j][i]);
+          out[e] = __float2bfloat16_rn(o[sl][j][2 * h + i] * inv * wv[j][i] * gate);
         }
     }
   }
@@ -630,6 +686,8 @@ pi_status pi_launch_recurrence_chunks(pi_ctx* ctx, const pi_recurrence& r, const
   p.seq_start = b.seq_start;
   p.slot = b.slot;
   sizes(p);
+  p.vec_k = r.dim % 4 == 0 && r.col_q % 4 == 0 && r.col_k % 4 == 0 && stride % 4 == 0;
+  p.vec_v = r.vdim % 4 == 0 && r.col_v % 4 == 0 && stride % 4 == 0;
   const size_t ch = (size_t)b.n_chunks * r.heads;
   p.U = scratch;
   p.nU = p.U + (ch * r.dim * r.vdim + 3) / 4 * 4;
