@@ -139,27 +139,35 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
   uint32_t qa[KMAX][QR];
   {
     const int r0 = lane >> 2, c0 = (lane & 3) * 2;
-    auto q2 = [&](int r, int ks, int c) -> uint32_t {   // channels c, c + 1 of k step ks of MMA row r
-      const int map = MAPS == 2 ? ks / ks_map : 0, head = grp * HR + r % HR;
-      const int d = (ks - map * ks_map) * 16 + c;
-      if (head >= p.group) return 0u;
-      const float* q = a.q + (size_t)row * a.stride + ((size_t)(g * p.group + head) * MAPS + map) * a.dim;
-      return pack(d < a.dim ? q[d] : 0.f, d + 1 < a.dim ? q[d + 1] : 0.f);
-    };
+    // all loads first (addresses clamped instead of branches, so that they are in flight together), then the packing
+    float v[KMAX][QR][2];
+    bool ok[2];
+    const float* q[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int head = grp * HR + (r0 + 8 * h) % HR;
+      ok[h] = head < p.group;
+      q[h] = a.q + (size_t)row * a.stride + (size_t)(g * p.group + min(head, p.group - 1)) * MAPS * a.dim;
+    }
 #pragma unroll
     for (int ks = 0; ks < KMAX; ++ks) {
+      const int map = MAPS == 2 && ks >= ks_map ? 1 : 0, d0 = (ks - map * ks_map) * 16 + c0;
 #pragma unroll
-      for (int j = 0; j < QR; ++j) qa[ks][j] = 0u;
-      if (ks < nks) {
-        if (MAPS == 2) {
-          qa[ks][0] = q2(r0, ks, c0);
-          qa[ks][1] = q2(r0, ks, c0 + 8);
-        } else {
-          qa[ks][0] = q2(r0, ks, c0);
-          qa[ks][1] = q2(r0 + 8, ks, c0);
-          qa[ks][QR - 2] = q2(r0, ks, c0 + 8);
-          qa[ks][QR - 1] = q2(r0 + 8, ks, c0 + 8);
-        }
+      for (int j = 0; j < QR; ++j) {
+        const int d = d0 + (QR == 2 ? j : j >> 1) * 8;
+        const float* src = q[QR == 2 ? 0 : j & 1] + map * a.dim;
+        v[ks][j][0] = src[min(d, a.dim - 1)];
+        v[ks][j][1] = src[min(d + 1, a.dim - 1)];
+      }
+    }
+#pragma unroll
+    for (int ks = 0; ks < KMAX; ++ks) {
+      const int map = MAPS == 2 && ks >= ks_map ? 1 : 0, d0 = (ks - map * ks_map) * 16 + c0;
+#pragma unroll
+      for (int j = 0; j < QR; ++j) {
+        const int d = d0 + (QR == 2 ? j : j >> 1) * 8;
+        const bool is = ks < nks && ok[QR == 2 ? 0 : j & 1];
+        qa[ks][j] = pack(is && d < a.dim ? v[ks][j][0] : 0.f, is && d + 1 < a.dim ? v[ks][j][1] : 0.f);
       }
     }
   }
@@ -406,15 +414,24 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
       const int r = rg * 16 + (lane >> 2) + 8 * h, tok = r / p.group, head = r - tok * p.group;
       const bool ok = tok < n_tok;
       tpos[h] = ok ? p_first + tok : -1;      // -1: sees nothing
-      q[h] = ok ? a.q + (size_t)(row0 + tok0 + tok) * a.stride + ((size_t)(g * p.group + head) * MAPS + map) * a.dim : nullptr;
+      q[h] = a.q + (size_t)(row0 + tok0 + (ok ? tok : 0)) * a.stride + ((size_t)(g * p.group + head) * MAPS + map) * a.dim;
     }
+    float v[KMAP][4][2];                      // all loads first, addresses clamped instead of branches
 #pragma unroll
     for (int ks = 0; ks < KMAP; ++ks)
 #pragma unroll
       for (int j = 0; j < 4; ++j) {           // a0: row, a1: row + 8, a2 / a3: channels + 8
-        const float* src = q[j & 1];
         const int d = ks * 16 + (lane & 3) * 2 + (j >> 1) * 8;
-        qa[ks][j] = (ks < nks && src) ? pack(d < a.dim ? src[d] : 0.f, d + 1 < a.dim ? src[d + 1] : 0.f) : 0u;
+        v[ks][j][0] = q[j & 1][min(d, a.dim - 1)];
+        v[ks][j][1] = q[j & 1][min(d + 1, a.dim - 1)];
+      }
+#pragma unroll
+    for (int ks = 0; ks < KMAP; ++ks)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int d = ks * 16 + (lane & 3) * 2 + (j >> 1) * 8;
+        const bool is = ks < nks && tpos[j & 1] >= 0;
+        qa[ks][j] = pack(is && d < a.dim ? v[ks][j][0] : 0.f, is && d + 1 < a.dim ? v[ks][j][1] : 0.f);
       }
   }
   float acc[VMAX / 8][4];

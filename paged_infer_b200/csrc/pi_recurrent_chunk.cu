@@ -151,33 +151,37 @@ __device__ __forceinline__ void store_split4(__nv_bfloat16* hi, __nv_bfloat16* l
   *reinterpret_cast<uint2*>(lo + i) = l;
 }
 
-// Four adjacent values, of which the first `n` exist (vec: 16-byte loads are possible where all four do).
-__device__ __forceinline__ float4 load4(const float* src, int n, bool vec) {
-  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-  if (n >= 4 && vec) return __ldg(reinterpret_cast<const float4*>(src));
-  if (n > 0) v.x = __ldg(src);
-  if (n > 1) v.y = __ldg(src + 1);
-  if (n > 2) v.z = __ldg(src + 2);
-  if (n > 3) v.w = __ldg(src + 3);
-  return v;
-}
-// rows x cols (cols a multiple of 4) walked by the CTA four columns at a time, several loads in flight per thread before the
-// first of them is used: load(row, col) -> float4, use(row, col, float4).
-template <typename L, typename F>
-__device__ __forceinline__ void staged(int rows, int cols, L&& load, F&& use) {
+// A [rows][cols] piece of a matrix (cols a multiple of 4, zero outside the first `have_rows` rows and `have_cols` columns),
+// walked by the CTA four columns at a time: use(row, col, float4).  With `vec` (16-byte loads possible, have_cols a multiple
+// of 4) several loads are in flight per thread before the first of them is used; they clamp their address instead of
+// branching.
+template <typename F>
+__device__ __forceinline__ void staged(const float* src, size_t ld, int rows, int cols, int have_rows, int have_cols, bool vec, F&& use) {
   constexpr int U = 4;
   const int c4 = cols >> 2, count = rows * c4;
-  for (int i0 = threadIdx.x; i0 < count; i0 += U * kChunkThreads) {
-    float4 v[U];
+  if (vec) {
+    for (int i0 = threadIdx.x; i0 < count; i0 += U * kChunkThreads) {
+      float4 v[U];
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int i = i0 + u * kChunkThreads;
-      if (i < count) v[u] = load(i / c4, (i % c4) * 4);
+      for (int u = 0; u < U; ++u) {
+        const int i = min(i0 + u * kChunkThreads, count - 1), r = i / c4, c = (i - r * c4) * 4;
+        const bool ok = r < have_rows && c < have_cols;
+        v[u] = __ldg(reinterpret_cast<const float4*>(ok ? src + (size_t)r * ld + c : src));
+        if (!ok) v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int i = i0 + u * kChunkThreads, r = i / c4;
+        if (i < count) use(r, (i - r * c4) * 4, v[u]);
+      }
     }
+  } else {
+    for (int i = threadIdx.x; i < count; i += kChunkThreads) {
+      const int r = i / c4, c = (i - r * c4) * 4;
+      float x[4];
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int i = i0 + u * kChunkThreads;
-      if (i < count) use(i / c4, (i % c4) * 4, v[u]);
+      for (int j = 0; j < 4; ++j) x[j] = (r < have_rows && c + j < have_cols) ? __ldg(src + (size_t)r * ld + c + j) : 0.f;
+      use(r, c, make_float4(x[0], x[1], x[2], x[3]));
     }
   }
 }
@@ -186,8 +190,7 @@ __device__ __forceinline__ void staged(int rows, int cols, L&& load, F&& use) {
 __device__ __forceinline__ void load_v(const ChunkParams& p, const ChunkAt& at, int head, int c0, int cols, __nv_bfloat16* hi, __nv_bfloat16* lo,
                                        int pitch) {
   const float* src = p.proj + (size_t)at.row0 * p.stride + p.r.col_v + (size_t)head * p.r.vdim + c0;
-  staged(C, cols, [&](int t, int e) { return load4(src + (size_t)t * p.stride + e, t < at.n ? p.r.vdim - c0 - e : 0, p.vec_v); },
-         [&](int t, int e, float4 v) { store_split4(hi, lo, t * pitch + e, v); });
+  staged(src, p.stride, C, cols, at.n, p.r.vdim - c0, p.vec_v, [&](int t, int e, float4 v) { store_split4(hi, lo, t * pitch + e, v); });
 }
 
 template <int KIND>
@@ -222,7 +225,7 @@ __global__ void __launch_bounds__(kChunkThreads) recur_local_kernel(const ChunkP
     }
   }
   const float* ksrc = p.proj + (size_t)at.row0 * p.stride + r.col_k + (size_t)head * r.dim;
-  staged(C, p.dimp, [&](int t, int d) { return load4(ksrc + (size_t)t * p.stride + d, t < at.n ? r.dim - d : 0, p.vec_k); },
+  staged(ksrc, p.stride, C, p.dimp, at.n, r.dim, p.vec_k,
          [&](int t, int d, float4 v) {
            if (KIND == PI_REC_GLA) {
              float4 e = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -414,7 +417,7 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
     }
   }
   const float* src = p.proj + (size_t)at.row0 * p.stride + (size_t)head * r.dim;
-  staged(C, p.dimp, [&](int t, int d) { return load4(src + r.col_q + (size_t)t * p.stride + d, t < at.n ? r.dim - d : 0, p.vec_k); },
+  staged(src + r.col_q, p.stride, C, p.dimp, at.n, r.dim, p.vec_k,
          [&](int t, int d, float4 v) {
            float4 e = make_float4(r.q_scale, r.q_scale, r.q_scale, r.q_scale);
            if (KIND == PI_REC_GLA) {
@@ -423,7 +426,7 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
            }
            *reinterpret_cast<float4*>(qf + t * qp + d) = make_float4(v.x * e.x, v.y * e.y, v.z * e.z, v.w * e.w);
          });
-  staged(C, p.dimp, [&](int t, int d) { return load4(src + r.col_k + (size_t)t * p.stride + d, t < at.n ? r.dim - d : 0, p.vec_k); },
+  staged(src + r.col_k, p.stride, C, p.dimp, at.n, r.dim, p.vec_k,
          [&](int t, int d, float4 v) {
            if (KIND == PI_REC_GLA) {
              const float4 b = *reinterpret_cast<const float4*>(bl + t * p.dimp + d), e = *reinterpret_cast<const float4*>(tot + (t / SUB) * p.dimp + d);
@@ -513,8 +516,7 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
     __syncthreads();            // the last slice (or the decays in its place) has been read
     load_v(p, at, head, c0, kVS, vhi, vlo, vp);
     const float* S = p.U + ch * r.dim * r.vdim;
-    staged(p.dimp, kVS, [&](int d, int e) { return load4(S + (size_t)d * r.vdim + c0 + e, d < r.dim ? r.vdim - c0 - e : 0, p.vec_v); },
-           [&](int d, int e, float4 v) { store_split4(shi, slo, d * vp + e, v); });
+    staged(S + c0, r.vdim, p.dimp, kVS, r.dim, r.vdim - c0, p.vec_v, [&](int d, int e, float4 v) { store_split4(shi, slo, d * vp + e, v); });
     __syncthreads();
     float (&acc)[4][4] = o[sl];
 #pragma unroll
