@@ -13,6 +13,7 @@
 #include <math.h>
 
 #include <algorithm>
+#include <type_traits>
 
 #include "pi_attention_maps.cuh"
 #include "pi_mma.cuh"
@@ -308,49 +309,67 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
   if (p.nsplit > 1) cluster.sync();
   else __syncthreads();
   const int rank = p.nsplit > 1 ? (int)cluster.block_rank() : 0;
-  for (int h = warp * p.nsplit + rank; h < HR; h += kDecWarps * p.nsplit) {
-    const int head = grp * HR + h;
-    if (head >= p.group) continue;
-    float f[MAPS][kMaxSplits];
+  // NS parts are read whether they exist or not (ranks clamped, weights zero), so that the loads are in flight together
+  auto finish = [&](auto ns_c) {
+    constexpr int NS = decltype(ns_c)::value;
+    const float *pm[NS], *pl[NS], *pa[NS];
 #pragma unroll
-    for (int m = 0; m < MAPS; ++m) {
-      const int r = h + m * HR;
-      float M = -INFINITY, L = 0.f;
-#pragma unroll
-      for (int c = 0; c < kMaxSplits; ++c) {
-        f[m][c] = c < p.nsplit ? (p.nsplit > 1 ? cluster.map_shared_rank(c_m, c)[r] : c_m[r]) : -INFINITY;
-        M = fmaxf(M, f[m][c]);
-      }
-#pragma unroll
-      for (int c = 0; c < kMaxSplits; ++c) {
-        f[m][c] = f[m][c] == -INFINITY ? 0.f : exp2f(f[m][c] - M);
-        if (c < p.nsplit) L = fmaf(p.nsplit > 1 ? cluster.map_shared_rank(c_l, c)[r] : c_l[r], f[m][c], L);
-      }
-#pragma unroll
-      for (int c = 0; c < kMaxSplits; ++c) f[m][c] = L > 0.f ? f[m][c] / L : 0.f;
+    for (int c = 0; c < NS; ++c) {
+      const int cr = min(c, p.nsplit - 1);
+      pm[c] = NS > 1 ? cluster.map_shared_rank(c_m, cr) : c_m;
+      pl[c] = NS > 1 ? cluster.map_shared_rank(c_l, cr) : c_l;
+      pa[c] = NS > 1 ? cluster.map_shared_rank(wacc, cr) : wacc;
     }
-    float d[VMAX / 32], ss = 0.f;
+    for (int h = warp * p.nsplit + rank; h < HR; h += kDecWarps * p.nsplit) {
+      const int head = grp * HR + h;
+      if (head >= p.group) continue;
+      float f[MAPS][NS], l[MAPS][NS];
 #pragma unroll
-    for (int i = 0; i < VMAX / 32; ++i) {
-      const int e = lane + 32 * i;
-      d[i] = 0.f;
-      if (e >= a.vdim) continue;
+      for (int m = 0; m < MAPS; ++m)
+#pragma unroll
+        for (int c = 0; c < NS; ++c) {
+          f[m][c] = pm[c][h + m * HR];
+          l[m][c] = pl[c][h + m * HR];
+        }
 #pragma unroll
       for (int m = 0; m < MAPS; ++m) {
-        float o = 0.f;
+        float M = -INFINITY, L = 0.f;
 #pragma unroll
-        for (int c = 0; c < kMaxSplits; ++c)
-          if (c < p.nsplit) o = fmaf((p.nsplit > 1 ? cluster.map_shared_rank(wacc, c) : wacc)[(size_t)(h + m * HR) * apitch + e], f[m][c], o);
-        d[i] = m == 0 ? o : d[i] - a.lambda * o;
+        for (int c = 0; c < NS; ++c) M = fmaxf(M, f[m][c]);
+#pragma unroll
+        for (int c = 0; c < NS; ++c) {
+          f[m][c] = c >= p.nsplit || f[m][c] == -INFINITY ? 0.f : exp2f(f[m][c] - M);
+          L = fmaf(l[m][c], f[m][c], L);
+        }
+        const float inv = L > 0.f ? (m == 0 ? 1.f : -a.lambda) / L : 0.f;
+#pragma unroll
+        for (int c = 0; c < NS; ++c) f[m][c] *= inv;
       }
-      ss = fmaf(d[i], d[i], ss);
-    }
-    const float r = MAPS == 2 ? a.out_scale / sqrtf(pi_warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
-    const size_t o0 = (size_t)row * a.out_stride + (size_t)(g * p.group + head) * a.vdim;
+      float d[VMAX / 32], ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < VMAX / 32; ++i)
-      if (lane + 32 * i < a.vdim) store_out(p, o0 + lane + 32 * i, d[i] * r);
-  }
+      for (int i = 0; i < VMAX / 32; ++i) {
+        const int e = min(lane + 32 * i, a.vdim - 1);
+        float x[MAPS][NS];
+#pragma unroll
+        for (int m = 0; m < MAPS; ++m)
+#pragma unroll
+          for (int c = 0; c < NS; ++c) x[m][c] = pa[c][(size_t)(h + m * HR) * apitch + e];
+        d[i] = 0.f;
+#pragma unroll
+        for (int m = 0; m < MAPS; ++m)
+#pragma unroll
+          for (int c = 0; c < NS; ++c) d[i] = fmaf(x[m][c], f[m][c], d[i]);
+        if (lane + 32 * i < a.vdim) ss = fmaf(d[i], d[i], ss);
+      }
+      const float r = MAPS == 2 ? a.out_scale / sqrtf(pi_warp_sum(ss) / (float)a.vdim + a.eps) : 1.f;
+      const size_t o0 = (size_t)row * a.out_stride + (size_t)(g * p.group + head) * a.vdim;
+#pragma unroll
+      for (int i = 0; i < VMAX / 32; ++i)
+        if (lane + 32 * i < a.vdim) store_out(p, o0 + lane + 32 * i, d[i] * r);
+    }
+  };
+  if (p.nsplit > 1) finish(std::integral_constant<int, kMaxSplits>());
+  else finish(std::integral_constant<int, 1>());
   if (p.nsplit > 1) cluster.sync();   // a peer may still be reading this CTA's part
 }
 

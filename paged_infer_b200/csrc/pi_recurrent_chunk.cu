@@ -29,6 +29,7 @@ constexpr int kChunkThreads = 256, kChunkWarps = 8;
 constexpr int kVS = 64;               // value columns per pass of the output kernel
 constexpr int kMaxDim = 128, kMaxVdim = 256;
 constexpr float kSafeDecay = -60.f;
+constexpr int kFactors = NSUB * (NSUB + 1) / 2 + NSUB;
 static_assert(C == 64, "the kernels are laid out for 64 tokens");
 
 struct ChunkParams {
@@ -153,10 +154,10 @@ __device__ __forceinline__ void store_split4(__nv_bfloat16* hi, __nv_bfloat16* l
 
 // A [rows][cols] piece of a matrix (cols a multiple of 4, zero outside the first `have_rows` rows and `have_cols` columns),
 // walked by the CTA four columns at a time: use(row, col, float4).  With `vec` (16-byte loads possible, have_cols a multiple
-// of 4) several loads are in flight per thread before the first of them is used; they clamp their address instead of
-// branching.
+// of 4) several loads are in flight per thread before the first of them is used; instead of branching, what is outside reads
+// `safe`, any valid 16-byte aligned address.
 template <typename F>
-__device__ __forceinline__ void staged(const float* src, size_t ld, int rows, int cols, int have_rows, int have_cols, bool vec, F&& use) {
+__device__ __forceinline__ void staged(const float* safe, const float* src, size_t ld, int rows, int cols, int have_rows, int have_cols, bool vec, F&& use) {
   constexpr int U = 4;
   const int c4 = cols >> 2, count = rows * c4;
   if (vec) {
@@ -166,7 +167,7 @@ __device__ __forceinline__ void staged(const float* src, size_t ld, int rows, in
       for (int u = 0; u < U; ++u) {
         const int i = min(i0 + u * kChunkThreads, count - 1), r = i / c4, c = (i - r * c4) * 4;
         const bool ok = r < have_rows && c < have_cols;
-        v[u] = __ldg(reinterpret_cast<const float4*>(ok ? src + (size_t)r * ld + c : src));
+        v[u] = __ldg(reinterpret_cast<const float4*>(ok ? src + (size_t)r * ld + c : safe));
         if (!ok) v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
       }
 #pragma unroll
@@ -190,7 +191,7 @@ __device__ __forceinline__ void staged(const float* src, size_t ld, int rows, in
 __device__ __forceinline__ void load_v(const ChunkParams& p, const ChunkAt& at, int head, int c0, int cols, __nv_bfloat16* hi, __nv_bfloat16* lo,
                                        int pitch) {
   const float* src = p.proj + (size_t)at.row0 * p.stride + p.r.col_v + (size_t)head * p.r.vdim + c0;
-  staged(src, p.stride, C, cols, at.n, p.r.vdim - c0, p.vec_v, [&](int t, int e, float4 v) { store_split4(hi, lo, t * pitch + e, v); });
+  staged(p.proj, src, p.stride, C, cols, at.n, p.r.vdim - c0, p.vec_v, [&](int t, int e, float4 v) { store_split4(hi, lo, t * pitch + e, v); });
 }
 
 template <int KIND>
@@ -225,7 +226,7 @@ __global__ void __launch_bounds__(kChunkThreads) recur_local_kernel(const ChunkP
     }
   }
   const float* ksrc = p.proj + (size_t)at.row0 * p.stride + r.col_k + (size_t)head * r.dim;
-  staged(ksrc, p.stride, C, p.dimp, at.n, r.dim, p.vec_k,
+  staged(p.proj, ksrc, p.stride, C, p.dimp, at.n, r.dim, p.vec_k,
          [&](int t, int d, float4 v) {
            if (KIND == PI_REC_GLA) {
              float4 e = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -374,7 +375,9 @@ __global__ void __launch_bounds__(256) recur_pass_kernel(const ChunkParams p, in
   }
 }
 
-template <int KIND>
+// NS: passes of 64 value columns.  (Loops are kept rolled where they can be: the kernel is otherwise bound by instruction
+// fetch.)
+template <int KIND, int NS>
 __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const ChunkParams p) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const pi_recurrence& r = p.r;
@@ -383,16 +386,17 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
   const size_t ch = (size_t)chunk * r.heads + head;
   const int qp = p.dimp + 4, kp = p.dimp + 8, ap = C + 8, vp = kVS + 8, nks = p.dimp / 16;
   float* qf = reinterpret_cast<float*>(smem_raw);                   // [C][qp] queries (GLA: decayed from their subchunk's start)
-  float* tot = qf + C * qp;                                         // [NSUB][dimp]
-  __nv_bfloat16* khi = reinterpret_cast<__nv_bfloat16*>(tot + NSUB * p.dimp);   // [C][kp]
-  __nv_bfloat16* klo = khi + C * kp;
-  __nv_bfloat16* ahi = klo + C * kp;                                // [C][ap] weights inside the chunk
-  __nv_bfloat16* alo = ahi + C * ap;
-  __nv_bfloat16* vhi = alo + C * ap;                                // [C][vp], then the state [dimp][vp]
-  __nv_bfloat16* vlo = vhi + C * vp;
-  __nv_bfloat16* shi = vlo + C * vp;
+  float* tot = qf + C * qp;                                         // GLA: [NSUB][dimp], then the factors [kFactors][dimp]
+  float* fac = tot + NSUB * p.dimp;
+  __nv_bfloat16* khi = reinterpret_cast<__nv_bfloat16*>(fac + (KIND == PI_REC_GLA ? kFactors * p.dimp : 0));   // [C][kp] x 2, later
+  __nv_bfloat16* klo = khi + C * kp;                                //   in its place: the state [dimp][vp] x 2
+  __nv_bfloat16* shi = khi;
   __nv_bfloat16* slo = shi + p.dimp * vp;
-  float* bl = reinterpret_cast<float*>(vhi);                        // until the values arrive: [C][dimp], [C][rank]
+  __nv_bfloat16* ahi = khi + 2 * max(C * kp, p.dimp * vp);          // [C][ap] x 2: weights inside the chunk
+  __nv_bfloat16* alo = ahi + C * ap;
+  __nv_bfloat16* vhi = alo + C * ap;                                // [C][vp] x 2
+  __nv_bfloat16* vlo = vhi + C * vp;
+  float* bl = reinterpret_cast<float*>(vhi);                        // GLA, until the values arrive: [C][dimp], [C][rank]
   float* low = bl + C * p.dimp;
   __shared__ float li[C], F[C], G[C], den[C], inter[C], ssum[C][2];
   __shared__ int unsafe[NSUB];
@@ -403,6 +407,20 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
     gla_decays(p, at, head, low, bl, tot);
     for (int i = tid; i < NSUB * p.dimp; i += kChunkThreads)
       if (tot[i] < kSafeDecay) unsafe[i / p.dimp] = 1;
+    // factors between subchunks J <= I (row I (I + 1) / 2 + J), then from the chunk's start to subchunk I
+    for (int i = tid; i < kFactors * p.dimp; i += kChunkThreads) {
+      const int row = i / p.dimp, d = i - row * p.dimp;
+      int I = 0, J = row;
+      if (row < kFactors - NSUB) {
+        while (J > I) J -= ++I;
+      } else {
+        I = row - (kFactors - NSUB);
+        J = -1;
+      }
+      float e = I == J ? -tot[I * p.dimp + d] : 0.f;
+      for (int x = J + 1; x < I; ++x) e += tot[x * p.dimp + d];
+      fac[i] = expf(I == J ? fminf(e, -kSafeDecay) : e);            // beyond: summed pair by pair
+    }
   } else {
     mlstm_gates(p, at, head, li, F, G);
     m_in = p.m_in[ch];
@@ -417,7 +435,7 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
     }
   }
   const float* src = p.proj + (size_t)at.row0 * p.stride + (size_t)head * r.dim;
-  staged(src + r.col_q, p.stride, C, p.dimp, at.n, r.dim, p.vec_k,
+  staged(p.proj, src + r.col_q, p.stride, C, p.dimp, at.n, r.dim, p.vec_k,
          [&](int t, int d, float4 v) {
            float4 e = make_float4(r.q_scale, r.q_scale, r.q_scale, r.q_scale);
            if (KIND == PI_REC_GLA) {
@@ -426,7 +444,7 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
            }
            *reinterpret_cast<float4*>(qf + t * qp + d) = make_float4(v.x * e.x, v.y * e.y, v.z * e.z, v.w * e.w);
          });
-  staged(src + r.col_k, p.stride, C, p.dimp, at.n, r.dim, p.vec_k,
+  staged(p.proj, src + r.col_k, p.stride, C, p.dimp, at.n, r.dim, p.vec_k,
          [&](int t, int d, float4 v) {
            if (KIND == PI_REC_GLA) {
              const float4 b = *reinterpret_cast<const float4*>(bl + t * p.dimp + d), e = *reinterpret_cast<const float4*>(tot + (t / SUB) * p.dimp + d);
@@ -436,14 +454,18 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
          });
   __syncthreads();
 
-  // A fragments of 16 query rows at k step ks, times a factor per channel
-  auto q_frag = [&](int row0, int ks, auto&& factor, uint32_t* hi, uint32_t* lo) {
+  // A fragments of 16 query rows at k step ks, GLA: times a factor per channel
+  auto q_frag = [&](int row0, int ks, const float* factor, uint32_t* hi, uint32_t* lo) {
     const int rr = row0 + (lane >> 2), c = ks * 16 + (lane & 3) * 2;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int cc = c + (j >> 1) * 8;
-      const float2 v = *reinterpret_cast<const float2*>(qf + (rr + (j & 1) * 8) * qp + cc);
-      split(v.x * factor(cc), v.y * factor(cc + 1), hi[j], lo[j]);
+      float2 v = *reinterpret_cast<const float2*>(qf + (rr + (j & 1) * 8) * qp + cc);
+      if (KIND == PI_REC_GLA) {
+        const float2 f = *reinterpret_cast<const float2*>(factor + cc);
+        v = make_float2(v.x * f.x, v.y * f.y);
+      }
+      split(v.x, v.y, hi[j], lo[j]);
     }
   };
 
@@ -454,15 +476,10 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
     float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
     const bool by_pair = KIND == PI_REC_GLA && I == J && unsafe[I];
     if (!by_pair) {
-      auto factor = [&](int d) {
-        if (KIND == PI_REC_MLSTM) return 1.f;
-        float e = I == J ? -tot[I * p.dimp + d] : 0.f;
-        for (int x = J + 1; x < I; ++x) e += tot[x * p.dimp + d];
-        return expf(e);
-      };
+#pragma unroll 1
       for (int ks = 0; ks < nks; ++ks) {
         uint32_t qh[4], ql[4], bh[4], bo[4];
-        q_frag(I * SUB, ks, factor, qh, ql);
+        q_frag(I * SUB, ks, fac + item * p.dimp, qh, ql);
         const int br = J * SUB + (lane & 7) + ((lane >> 4) << 3), bc = ks * 16 + ((lane >> 3) & 1) * 8;
         ldsm4(bh, smem_addr(khi + br * kp + bc));
         ldsm4(bo, smem_addr(klo + br * kp + bc));
@@ -507,16 +524,15 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
 
   // ---- O = Q~ S + A V, 64 value columns at a time; warp = (16 rows, half of the columns) ------------------------------------
   const int I = warp >> 1, half = warp & 1;
-  float o[kMaxVdim / kVS][4][4];
+  float o[NS][4][4];
   float ss[2] = {0.f, 0.f};
 #pragma unroll
-  for (int sl = 0; sl < kMaxVdim / kVS; ++sl) {
+  for (int sl = 0; sl < NS; ++sl) {
     const int c0 = sl * kVS;
-    if (c0 >= p.vdimp) break;
     __syncthreads();            // the last slice (or the decays in its place) has been read
     load_v(p, at, head, c0, kVS, vhi, vlo, vp);
     const float* S = p.U + ch * r.dim * r.vdim;
-    staged(S + c0, r.vdim, p.dimp, kVS, r.dim, r.vdim - c0, p.vec_v, [&](int d, int e, float4 v) { store_split4(shi, slo, d * vp + e, v); });
+    staged(p.proj, S + c0, r.vdim, p.dimp, kVS, r.dim, r.vdim - c0, p.vec_v, [&](int d, int e, float4 v) { store_split4(shi, slo, d * vp + e, v); });
     __syncthreads();
     float (&acc)[4][4] = o[sl];
 #pragma unroll
@@ -538,14 +554,10 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
         }
       }
     };
+#pragma unroll 1
     for (int ks = 0; ks < nks; ++ks) {
       uint32_t qh[4], ql[4];
-      q_frag(I * SUB, ks, [&](int d) {
-        if (KIND == PI_REC_MLSTM) return 1.f;
-        float e = 0.f;
-        for (int x = 0; x < I; ++x) e += tot[x * p.dimp + d];
-        return expf(e);
-      }, qh, ql);
+      q_frag(I * SUB, ks, fac + (kFactors - NSUB + I) * p.dimp, qh, ql);
       products(qh, ql, shi, slo, ks * 16);
     }
     if (KIND == PI_REC_MLSTM) {
@@ -558,6 +570,7 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
         acc[j][3] *= f1;
       }
     }
+#pragma unroll 1
     for (int J = 0; J <= I; ++J) {
       uint32_t ah[4], al[4];
       const int ar = I * SUB + (lane & 7) + ((lane >> 3) & 1) * 8, ac = J * SUB + (lane >> 4) * 8;
@@ -596,8 +609,7 @@ __global__ void __launch_bounds__(kChunkThreads) recur_output_kernel(const Chunk
     __nv_bfloat16* out = p.out + (size_t)(at.row0 + t) * p.out_stride + (size_t)head * r.vdim;
     const float* nw = r.norm + (r.norm_per_head ? (size_t)head * r.vdim : 0);
 #pragma unroll
-    for (int sl = 0; sl < kMaxVdim / kVS; ++sl) {
-      if (sl * kVS >= p.vdimp) break;
+    for (int sl = 0; sl < NS; ++sl) {
       float gv[4][2], wv[4][2];
 #pragma unroll
       for (int j = 0; j < 4; ++j)
@@ -625,9 +637,10 @@ size_t local_smem(const ChunkParams& p) {
   return planes + (p.r.kind == PI_REC_GLA ? ((size_t)(C + NSUB) * p.dimp + (size_t)C * p.r.rank) * 4 : 0);
 }
 size_t output_smem(const ChunkParams& p) {
-  const size_t fixed = ((size_t)C * (p.dimp + 4) + (size_t)NSUB * p.dimp) * 4 + (size_t)2 * C * (p.dimp + 8) * 2 + (size_t)2 * C * (C + 8) * 2;
-  const size_t values = (size_t)2 * (C + p.dimp) * (kVS + 8) * 2;
-  return fixed + std::max(values, p.r.kind == PI_REC_GLA ? (size_t)C * (p.dimp + p.r.rank) * 4 : (size_t)0);
+  const bool gla = p.r.kind == PI_REC_GLA;
+  const size_t f32 = ((size_t)C * (p.dimp + 4) + (size_t)(NSUB + (gla ? kFactors : 0)) * p.dimp) * 4;
+  const size_t keys = (size_t)4 * std::max(C * (p.dimp + 8), p.dimp * (kVS + 8)), weights = (size_t)4 * C * (C + 8), values = (size_t)4 * C * (kVS + 8);
+  return f32 + keys + weights + std::max(values, gla ? (size_t)C * (p.dimp + p.r.rank) * 4 : (size_t)0);
 }
 
 cudaError_t grant(pi_ctx* ctx, void (*k)(const ChunkParams), size_t smem, pi_smem_grant& g) {
@@ -643,18 +656,20 @@ void sizes(ChunkParams& p) {
 
 template <int KIND>
 pi_status launch_chunks(pi_ctx* ctx, ChunkParams& p, int n_chunks, int n_seqs) {
-  static pi_smem_grant g1, g2;
+  static pi_smem_grant g1, g2[3];
   const pi_recurrence& r = p.r;
   const size_t s1 = local_smem(p), s2 = output_smem(p);
   PI_CUDA(ctx, grant(ctx, recur_local_kernel<KIND>, s1, g1));
-  PI_CUDA(ctx, grant(ctx, recur_output_kernel<KIND>, s2, g2));
+  const int passes = (p.vdimp + kVS - 1) / kVS, pick = passes <= 1 ? 0 : passes <= 2 ? 1 : 2;
+  void (*const output[3])(const ChunkParams) = {recur_output_kernel<KIND, 1>, recur_output_kernel<KIND, 2>, recur_output_kernel<KIND, 4>};
+  PI_CUDA(ctx, grant(ctx, output[pick], s2, g2[pick]));
   PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, recur_local_kernel<KIND>, dim3(n_chunks, r.heads), dim3(kChunkThreads), s1, 1, p));
   const int per_head = r.dim * r.vdim;
   const bool vec = r.vdim % 4 == 0 && r.state_off % 4 == 0 && r.state_stride % 4 == 0;
   const int elem_blocks = (per_head / (vec ? 4 : 1) + 255) / 256, n_blocks = KIND == PI_REC_MLSTM ? (r.dim + 255) / 256 : 0;
   PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, vec ? recur_pass_kernel<KIND, 4> : recur_pass_kernel<KIND, 1>, dim3(elem_blocks + n_blocks, r.heads, n_seqs),
                                   dim3(256), 0, 1, p, elem_blocks));
-  PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, recur_output_kernel<KIND>, dim3(n_chunks, r.heads), dim3(kChunkThreads), s2, 1, p));
+  PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, output[pick], dim3(n_chunks, r.heads), dim3(kChunkThreads), s2, 1, p));
   return PI_OK;
 }
 
