@@ -201,6 +201,10 @@ pi_status pi_linear_apply_host(pi_ctx* ctx, const pi_linear* lin, const float* x
  *    overlap on the GPU (other streams or contexts) race on it: order them. */
 pi_status pi_linear_apply_noalloc(pi_ctx* ctx, const pi_linear* lin, const float* x_dev, float* out_dev, int M);
 
+/* The projection of the layered designs' bf16 mode: bf16 weights, bf16 activations x_dev [M][x_stride] (bf16 bits, rows on
+ * 16-byte boundaries), f32 accumulation on the tensor cores, out_dev [M][rows] f32.  No counterpart in the reference. */
+pi_status pi_linear_apply_bf16(pi_ctx* ctx, const pi_linear* lin, const uint16_t* x_dev, size_t x_stride, float* out_dev, int M);
+
 /* ---- KV pool ------------------------------------------------------------------ */
 
 /* Replaces: KvLayout (src/memory/layout.rs:18-41). */
@@ -411,7 +415,8 @@ size_t pi_state_pool_bytes(const pi_state_pool* pool);
 pi_status pi_state_copy_slot(pi_ctx* ctx, pi_state_pool* pool, int32_t src, int32_t dst);
 
 /* A ragged batch: sequence i brings n_tokens[i] >= 1 consecutive tokens from position start_pos[i] on, portions of
- * prompts beside single decoded tokens.  Rows are numbered through in this order. */
+ * prompts beside single decoded tokens.  Rows are numbered through in this order.  The sequences are distinct: none of
+ * them reads keys that another one writes in the same step. */
 typedef struct {
   int32_t n_seqs;
   const uint32_t* tokens;        /* all portions, one after the other */

@@ -280,6 +280,10 @@ class Projection:
         check(_lib.lib().pi_linear_apply(self.ctx.handle, self.handle, _dev_ptr(x_dev), _dev_ptr(out_dev), batch), self.ctx.handle)
 
 
+    def apply_device_bf16(self, x_dev, x_stride: int, out_dev, batch: int) -> None:
+        """bf16 activations ([batch, x_stride], rows on 16-byte boundaries) through a bf16 projection on the tensor cores, f32 out."""
+        check(_lib.lib().pi_linear_apply_bf16(self.ctx.handle, self.handle, _dev_ptr(x_dev), x_stride, _dev_ptr(out_dev), batch), self.ctx.handle)
+
     def apply_device_noalloc(self, x_dev, out_dev, batch: int) -> None:
         """``apply_device`` through the entry point that allocates nothing (``pi_linear_apply_noalloc``).
 

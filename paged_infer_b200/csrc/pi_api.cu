@@ -463,6 +463,19 @@ pi_status pi_linear_apply(pi_ctx* ctx, const pi_linear* lin, const float* x_dev,
   return pi_linear_forward(ctx, lin, a);
 }
 
+pi_status pi_linear_apply_bf16(pi_ctx* ctx, const pi_linear* lin, const uint16_t* x_dev, size_t x_stride, float* out_dev, int M) {
+  PI_ENTER(ctx);
+  PI_REQUIRE(ctx, lin && x_dev && out_dev, "null pointer");
+  PI_REQUIRE(ctx, M >= 1, "batch must be at least 1, got %d", M);
+  pi_linear_args a;
+  a.x_bf16 = reinterpret_cast<const __nv_bfloat16*>(x_dev);
+  a.x_stride = x_stride;
+  a.out = out_dev;
+  a.out_stride = lin->rows;
+  a.M = M;
+  return pi_launch_gemm_bf16(ctx, lin, a);
+}
+
 pi_status pi_linear_apply_host(pi_ctx* ctx, const pi_linear* lin, const float* x_host, float* out_host, int M) {
   PI_ENTER(ctx);
   PI_REQUIRE(ctx, lin && x_host && out_host, "null pointer");

@@ -128,11 +128,19 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
   int pb[kDecStages];
 #pragma unroll
   for (int s = 0; s < kDecStages; ++s) pb[s] = block_of(tile0 + s * kDecWarps);
+  // Keys in front of this row's own position were written in earlier steps: their tiles are requested ahead of the dependency
+  // wait.  The tile with the row's own key is this step's work.
+#pragma unroll
+  for (int s = 0; s < kDecStages - 1; ++s) {
+    const int tile = tile0 + s * kDecWarps;
+    if (tile < tile_end && (tile + 1) * 16 <= pos) fetch(tile, s, pb[s]);
+  }
   pi_grid_dependency_wait();
 #pragma unroll
   for (int s = 0; s < kDecStages - 1; ++s) {
-    if (tile0 + s * kDecWarps < tile_end) fetch(tile0 + s * kDecWarps, s, pb[s]);
-    cp_async_commit();
+    const int tile = tile0 + s * kDecWarps;
+    if (tile < tile_end && (tile + 1) * 16 > pos) fetch(tile, s, pb[s]);
+    cp_async_commit();   // the first group also holds what was requested early
   }
   int pb_next = pb[kDecStages - 1];
 

@@ -376,3 +376,104 @@ def test_ragged_step_of_a_llama(ctx):
     assert np.abs(got - golden[[4, 19, 9]]).max() < 5e-4
     got, ids = m.step([toks[10:11].tolist(), toks[20:21].tolist()], [10, 20], [ta, tb], kv, want_argmax=True)
     assert np.abs(got - golden[[10, 20]]).max() < 5e-4 and ids.tolist() == golden[[10, 20]].argmax(-1).tolist()
+
+
+@pytest.mark.parametrize("n,k", [(33, 100), (128, 64), (576, 1000), (2048, 512), (20, 8), (4100, 2056), (130, 4096)])
+def test_bf16_projection(ctx, n, k):
+    """Every tile width, K split over clusters and not, sizes that are no multiple of anything, against f32 on the host."""
+    import torch
+    from paged_infer_b200 import api
+    from paged_infer_b200.loader import bf16_bits_to_f32, f32_to_bf16_bits
+    rng = np.random.default_rng(n)
+    w = f32_to_bf16_bits(rng.standard_normal((n, k)).astype(np.float32))
+    lin = api.Projection.f32(ctx, w)
+    ld = (k + 7) // 8 * 8
+    for m in (1, 5, 16, 17, 32, 40, 64, 100, 128, 129, 300, 700):
+        x = f32_to_bf16_bits(rng.standard_normal((m, ld)).astype(np.float32))   # what lies behind k is garbage
+        xd = torch.from_numpy(x.view(np.int16)).cuda()
+        out = torch.full((m, n), 7.0, device="cuda")
+        lin.apply_device_bf16(xd, ld, out, m)
+        ctx.synchronize()
+        want = bf16_bits_to_f32(x)[:, :k].astype(np.float64) @ bf16_bits_to_f32(w).T.astype(np.float64)
+        assert np.abs(out.cpu().numpy() - want).max() < 3e-5 * np.sqrt(k), (m, n, k)
+
+
+def extreme(t, kind):
+    """Gates far out: GLA decays that empty the state within a few tokens next to channels that never forget; mLSTM input
+    gates that jump over tens of units."""
+    if kind == "gla":
+        b = t["l0.mix.a2.b"]
+        b[::3], b[1::3], b[2::3] = -40.0, 12.0, 0.0
+    elif kind == "mlstm":
+        t["l0.mix.i"] *= 16
+        t["l0.mix.f"] *= 16
+    return t
+
+
+@pytest.mark.parametrize("layer", [gla(heads=2, dim=64, vdim=128, tau=0.5), gla(heads=3, dim=40, vdim=72, tau=16.0), gla(heads=1, dim=128, vdim=256, tau=2.0),
+                                   gla(heads=2, dim=13, vdim=19, tau=1.0), mlstm(heads=2, dim=128, vdim=256, cap=30.0), mlstm(heads=3, dim=24, vdim=40, cap=15.0),
+                                   mlstm(heads=1, dim=17, vdim=150, cap=60.0)], ids=lambda l: f"{l['type']}-{l['mixer']['dim']}-{l['mixer']['vdim']}")
+@pytest.mark.parametrize("gates", ["plain", "extreme"])
+def test_chunks_equal_token_by_token(ctx, layer, gates):
+    """The chunked kernels against the scan on the same projections (both in the bf16 mode): far tighter than bf16 itself."""
+    cfg = config([layer], width=48)
+    t = tensors(cfg, 41)
+    if gates == "extreme":
+        t = extreme(t, layer["type"])
+    m = device_model(ctx, cfg, t, "bfloat16")
+    toks = tokens(64 * 3 + 21, 42)
+    outs = []
+    for size in (len(toks), 63, 64 + 37):    # all chunks; scan only; both, with the state handed over
+        s = Session(m)
+        outs.append(np.concatenate([s.run([("a", toks[i:i + size])])[0] for i in range(0, len(toks), size)]))
+    assert np.isfinite(outs[0]).all()
+    assert distance(outs[0], outs[1]).max() < 6e-3 and distance(outs[2], outs[1]).max() < 6e-3
+    # steep gates turn the rounding of the bf16 input into a wider error; the f32 mode has none of it
+    want = reference(cfg, t).forward(toks)
+    assert distance(outs[0], want).max() < (LIMIT["bfloat16"] if gates == "plain" else 0.2)
+    exact = Session(device_model(ctx, cfg, t, "float32")).run([("a", toks)])[0]
+    assert distance(exact, want).max() < 5 * LIMIT["float32"]
+
+
+@pytest.mark.parametrize("compute", ["float32", "bfloat16"])
+def test_one_softmax_map(ctx, compute):
+    """Plain grouped attention (one map) is the same mechanism with its constants: against the reference's window softmax."""
+    from oracle import layers as L
+    from layered_helpers import bits
+    from paged_infer_b200 import api, loader
+    H, G, D, E, W, T = 20, 1, 24, 40, 48, 130
+    two = config([attention(H, G, D, E, 50, ff=0)], width=W)
+    t = tensors(two, 51)
+    t["l0.mix.q"] = t["l0.mix.q"].reshape(H, 2, D, W)[:, 0].reshape(H * D, W).copy()
+    t["l0.mix.k"] = t["l0.mix.k"].reshape(G, 2, D, W)[:, 0].reshape(G * D, W).copy()
+    cfg = loader.LayeredConfig(W, 96, 1e-5, [loader.LayerConfig(loader.MIXER_ATTENTION, heads=H, kv_heads=G, dim=D, vdim=E, maps=1, window=None,
+                                                               rot_dims=10, rot_base=300.0, scale=0.3)])
+    m = api.LayeredModel(ctx, cfg, bits(t), compute, 256)
+    toks = tokens(T, 52)
+    f = {k: np.asarray(v, np.float64) for k, v in t.items()}
+    x = f["embed"][toks]
+    h = L.dyt_norm(x, f["l0.norm1.alpha"], f["l0.norm1"], f["l0.norm1.b"])
+    q = L.rotate_interleaved((h @ f["l0.mix.q"].T).reshape(T, H, D), np.arange(T), 10, 300.0)
+    k = L.rotate_interleaved((h @ f["l0.mix.k"].T).reshape(T, G, D), np.arange(T), 10, 300.0)
+    v = (h @ f["l0.mix.v"].T).reshape(T, G, E)
+    a = np.stack([L.window_softmax(q[:, n], k[:, 0], v[:, 0], 0.3, None) for n in range(H)], 1)
+    x = x + L.dyt_norm(a.reshape(T, H * E) @ f["l0.mix.o"].T, f["l0.norm1b.alpha"], f["l0.norm1b"], f["l0.norm1b.b"])
+    want = L.dyt_norm(x, f["final.norm.alpha"], f["final.norm"], f["final.norm.b"]) @ f["embed"].T
+    s = Session(m)
+    got = np.concatenate([s.run([("a", toks[:100])])[0]] + [s.run([("a", [c])])[0] for c in toks[100:]])
+    assert distance(got, want).max() < LIMIT[compute]
+
+
+@pytest.mark.parametrize("window", [300, 2000])
+def test_long_context_decoding_splits_keys(ctx, window):
+    """One sequence far along: its keys are cut over a cluster of CTAs; a block size that tiles straddle, and one they do not."""
+    cfg = config([attention(heads=4, kv_heads=1, dim=32, vdim=64, window=window, ff=0)], width=64)
+    t = tensors(cfg, 61)
+    toks = tokens(901, 62)
+    want = reference(cfg, t).forward(toks)
+    m = device_model(ctx, cfg, t, "bfloat16")
+    for bs in (16, 12, 64):
+        s = Session(m, block_size=bs)
+        s.run([("a", toks[:895])], False)
+        for i in range(895, 901):
+            assert distance(s.run([("a", [toks[i]])])[0], want[i:i + 1]).max() < LIMIT["bfloat16"]
