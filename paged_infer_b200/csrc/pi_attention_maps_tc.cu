@@ -48,6 +48,22 @@ struct Paged {
   }
 };
 
+// 16 rows of K or V that may lie in several blocks (block sizes that are no multiple of 16): every piece finds its own block.
+// Kept out of line: the kernels are short enough for instruction fetch to count.
+__device__ __noinline__ void fetch_rows(Paged pg, __nv_bfloat16* dst, int pitch, int t0, int hi, int lane, bool is_v) {
+  const int width = is_v ? pg.vp : pg.kw, pr = width / 8;
+  for (int c = lane; c < 16 * pr; c += 32) {
+    const int r = c / pr, x = (c - r * pr) * 8, t = t0 + r;
+    const bool ok = t < hi;
+    const __nv_bfloat16* src = pg.base;
+    if (ok) {
+      const int off = t % pg.block_size;
+      src = pg.tile(t / pg.block_size) + (is_v ? (size_t)pg.block_size * pg.kw : (size_t)0) + (size_t)off * width + x;
+    }
+    cp_async16(smem_addr(dst + r * pitch + x), src, ok ? 16 : 0);
+  }
+}
+
 // Online softmax step of one accumulator row: running maximum, factor for what is already summed.
 __device__ __forceinline__ float new_max(float m, float s_max, float& keep) {
   const float n = fmaxf(m, s_max);
@@ -109,20 +125,8 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
       copy(vs, vpitch, vpr, vb);
       return;
     }
-    auto copy = [&](__nv_bfloat16* dst, int pitch, int pr, bool is_v) {
-      for (int c = lane; c < 16 * pr; c += 32) {
-        const int r = c / pr, x = (c - r * pr) * 8, t = t0 + r;
-        const bool ok = t < hi;
-        const __nv_bfloat16* src = pg.base;
-        if (ok) {
-          const int off = t % a.block_size;
-          src = pg.tile(t / a.block_size) + (is_v ? (size_t)a.block_size * kw + (size_t)off * a.vp + x : (size_t)off * kw + x);
-        }
-        cp_async16(smem_addr(dst + r * pitch + x), src, ok ? 16 : 0);
-      }
-    };
-    copy(ks, kpitch, kpr, false);
-    copy(vs, vpitch, vpr, true);
+    fetch_rows(pg, ks, kpitch, t0, hi, lane, false);
+    fetch_rows(pg, vs, vpitch, t0, hi, lane, true);
   };
 
   int pb[kDecStages];
@@ -130,17 +134,15 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
   for (int s = 0; s < kDecStages; ++s) pb[s] = block_of(tile0 + s * kDecWarps);
   // Keys in front of this row's own position were written in earlier steps: their tiles are requested ahead of the dependency
   // wait.  The tile with the row's own key is this step's work.
-#pragma unroll
-  for (int s = 0; s < kDecStages - 1; ++s) {
-    const int tile = tile0 + s * kDecWarps;
-    if (tile < tile_end && (tile + 1) * 16 <= pos) fetch(tile, s, pb[s]);
-  }
-  pi_grid_dependency_wait();
-#pragma unroll
-  for (int s = 0; s < kDecStages - 1; ++s) {
-    const int tile = tile0 + s * kDecWarps;
-    if (tile < tile_end && (tile + 1) * 16 > pos) fetch(tile, s, pb[s]);
-    cp_async_commit();   // the first group also holds what was requested early
+#pragma unroll 1
+  for (int late = 0; late < 2; ++late) {
+    if (late) pi_grid_dependency_wait();
+#pragma unroll 1
+    for (int s = 0; s < kDecStages - 1; ++s) {
+      const int tile = tile0 + s * kDecWarps;
+      if (tile < tile_end && ((tile + 1) * 16 > pos) == (late != 0)) fetch(tile, s, s == 0 ? pb[0] : pb[1]);
+      if (late) cp_async_commit();   // the first group also holds what was requested early
+    }
   }
   int pb_next = pb[kDecStages - 1];
 
