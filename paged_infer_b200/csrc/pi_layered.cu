@@ -406,7 +406,7 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
   PI_REQUIRE(ctx, pool && pool->regions.size() == (size_t)std::count_if(m->layers.begin(), m->layers.end(), [](const Layer& l) { return l.attn >= 0; }) &&
                       pool->kind == m->c.compute,
              "the KV pool was made for another model");
-  const int n = in->n_seqs, mb = std::max(in->max_blocks, 1);
+  const int n = in->n_seqs;
   int rows = 0, max_pos = 0;
   std::vector<int32_t> row_seq, row_pos, row0(n), single, portions, scan, chunk_seqs, chunks, chunk0(1, 0);
   int max_portion = 0;
@@ -508,7 +508,6 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
   b.max_pos = max_pos + extra_positions;
   st->out_rows = d + o_out;
   st->n_out = in->n_out;
-  (void)mb;
   // scratch is sized here, so that nothing allocates while a step is being captured
   size_t floats = 0;
   for (const Layer& L : m->layers)
