@@ -151,6 +151,7 @@ enum pi_epilogue {
   PI_EPI_ADD = 1,       // out[m][r] += v           (residual add)
   PI_EPI_SWIGLU = 2,    // rows interleaved gate/up: out[m][r/2] = silu(v[2i]) * v[2i+1]
   PI_EPI_GEGLU = 3,     // the same with the tanh form of gelu
+  PI_EPI_MAPS_QKV = 5,  // fused [q;k;v] of multi-map attention: rotary q to `out`, rotary k and v into the paged pool (pi_maps_kv)
   PI_EPI_DYT_RESIDUAL = 4   // x[m][r] += dyt(post, v); h[m][r] = dyt(next, x[m][r])   (pi_dyt_residual)
 };
 
@@ -204,6 +205,18 @@ struct pi_rope_kv {
   const pi_attn_batch* batch = nullptr;
 };
 
+// Where the epilogue of the fused [q;k;v] projection of a layered design puts its result: q rotated into `out`, k rotated
+// and v into the row's place in the pool (skipped when its block is not mapped).  Rotation pairs are adjacent channels, so
+// dim must be even (odd ones take pi_launch_maps_rope_kv).
+struct pi_maps_kv {
+  int q_rows = 0, k_rows = 0, maps = 1, dim = 0, vdim = 0, rot_dims = 0;
+  const float *rope_cos = nullptr, *rope_sin = nullptr;   // [positions][rot_dims / 2]
+  void* base = nullptr;
+  int kind = PI_F32, kv_heads = 0, dp = 0, vp = 0, block_size = 1;
+  const int32_t *row_seq = nullptr, *row_pos = nullptr, *lens = nullptr, *tables = nullptr;
+  int max_blocks = 0;
+};
+
 struct pi_linear_args {
   const float* x = nullptr;   // [M][x_stride]
   size_t x_stride = 0;
@@ -231,6 +244,7 @@ struct pi_linear_args {
   const __nv_bfloat16* x_bf16 = nullptr;
   __nv_bfloat16* out_bf16 = nullptr;
   const pi_dyt_residual* residual = nullptr;   // PI_EPI_DYT_RESIDUAL
+  const pi_maps_kv* maps_kv = nullptr;         // PI_EPI_MAPS_QKV
 };
 
 // tcgen05 GEMM for bf16 weights and bf16 activations with f32 accumulation (a.x_bf16; any shape).
@@ -411,6 +425,57 @@ __device__ __forceinline__ float pi_warp_max(float v) {
 }
 __device__ __forceinline__ float pi_dyt_apply(const pi_dyt& n, float v, int i) {
   return n.w ? fmaf(tanhf(n.alpha * v), __ldg(n.w + i), __ldg(n.b + i)) : v;
+}
+// Row m's place: position, physical block (-1: not mapped) and offset in it.
+struct pi_kv_place {
+  int pos, block, off;
+};
+__device__ __forceinline__ pi_kv_place pi_maps_kv_place(const pi_maps_kv& k, int m) {
+  pi_kv_place r;
+  const int seq = k.row_seq[m];
+  r.pos = k.row_pos[m];
+  const int lb = r.pos / k.block_size;
+  r.off = r.pos - lb * k.block_size;
+  r.block = lb < k.lens[seq] ? k.tables[(size_t)seq * k.max_blocks + lb] : -1;
+  return r;
+}
+// Column n of [q;k;v]: channel of its vector, whether it is rotated, and, behind q, its element in a block and the step
+// from one token of the block to the next.
+struct pi_maps_col {
+  int d;
+  bool rotated, is_q;
+  size_t elem;
+  int step;
+};
+__device__ __forceinline__ pi_maps_col pi_maps_column(const pi_maps_kv& k, int n) {
+  pi_maps_col c;
+  const size_t tile = (size_t)k.block_size * (k.maps * k.dp + k.vp);
+  c.is_q = n < k.q_rows;
+  c.elem = 0;
+  c.step = 0;
+  if (n < k.q_rows + k.k_rows) {
+    const int x = c.is_q ? n : n - k.q_rows, vec = x / k.dim;
+    c.d = x - vec * k.dim;
+    c.rotated = c.d < k.rot_dims;
+    if (!c.is_q) {
+      const int g = vec / k.maps, map = vec - g * k.maps;
+      c.step = k.maps * k.dp;
+      c.elem = g * tile + (size_t)map * k.dp + c.d;
+    }
+  } else {
+    const int x = n - k.q_rows - k.k_rows, g = x / k.vdim;
+    c.d = x - g * k.vdim;
+    c.rotated = false;
+    c.step = k.vp;
+    c.elem = g * tile + (size_t)k.block_size * k.maps * k.dp + c.d;
+  }
+  return c;
+}
+__device__ __forceinline__ void pi_maps_kv_store(const pi_maps_kv& k, const pi_maps_col& c, int block, int off, float v) {
+  if (block < 0) return;
+  const size_t i = (size_t)block * k.kv_heads * ((size_t)k.block_size * (k.maps * k.dp + k.vp)) + c.elem + (size_t)off * c.step;
+  if (k.kind == PI_BF16) static_cast<__nv_bfloat16*>(k.base)[i] = __float2bfloat16_rn(v);
+  else static_cast<float*>(k.base)[i] = v;
 }
 // z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 __device__ __forceinline__ float pi_gelu_tanh(float z) {

@@ -44,6 +44,7 @@ struct Bf16GemmParams {
   size_t out_stride;
   int N, K, M, nkb, rtiles, tiles, ksplit, epi;
   pi_dyt_residual res;
+  pi_maps_kv mkv;
   int* err_flag;
 };
 
@@ -61,9 +62,10 @@ __device__ __forceinline__ void tma_2d(uint32_t dst, const CUtensorMap* map, uin
       : "memory");
 }
 
-// C columns (activation rows m, m + dm, ...) of output column n, all lanes of the warp on adjacent n.
+// C columns (activation rows m, m + dm, ...) of output column n, all lanes of the warp on adjacent n.  `place`: of row m, if
+// it has been looked up already.
 template <int C>
-__device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int n, int m, int dm, const float* v) {
+__device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int n, int m, int dm, const float* v, const pi_kv_place* place = nullptr) {
   const bool ok = n < p.N;
   if (p.epi == PI_EPI_DYT_RESIDUAL) {
     float old[C];
@@ -78,6 +80,35 @@ __device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int n, int m, 
       p.res.x[(size_t)(m + j * dm) * p.res.x_stride + n] = x;
       static_cast<__nv_bfloat16*>(p.res.h)[(size_t)(m + j * dm) * p.res.h_stride + n] =
           __float2bfloat16_rn(fmaf(tanhf(p.res.next.alpha * x), wn, bn));
+    }
+  } else if (p.epi == PI_EPI_MAPS_QKV) {
+    // a rotation pair is two adjacent columns, so the partner is the neighbouring lane; lane j looks row j's place up
+    const pi_maps_kv& k = p.mkv;
+    const pi_maps_col col = pi_maps_column(k, min(n, p.N - 1));
+    const int lane = threadIdx.x & 31;
+    pi_kv_place mine = {0, -1, 0};
+    const int my_row = m + (C == 1 ? 0 : (lane % C) * dm);
+    if (place) mine = *place;
+    else if (my_row < p.M) mine = pi_maps_kv_place(k, my_row);
+    const int half = k.rot_dims >> 1, pair = col.rotated ? col.d >> 1 : 0;
+    float cs[C], sn[C];
+    if (half > 0) {
+#pragma unroll
+      for (int j = 0; j < C; ++j) {
+        const size_t at = (size_t)__shfl_sync(0xffffffffu, mine.pos, j) * half + pair;
+        cs[j] = __ldg(k.rope_cos + at);
+        sn[j] = __ldg(k.rope_sin + at);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < C; ++j) {
+      const float other = __shfl_xor_sync(0xffffffffu, v[j], 1);
+      const int block = __shfl_sync(0xffffffffu, mine.block, j), off = __shfl_sync(0xffffffffu, mine.off, j);
+      float r = v[j];
+      if (col.rotated) r = (n & 1) ? v[j] * cs[j] + other * sn[j] : v[j] * cs[j] - other * sn[j];
+      if (!ok || m + j * dm >= p.M) continue;
+      if (col.is_q) p.out[(size_t)(m + j * dm) * p.out_stride + n] = r;
+      else pi_maps_kv_store(k, col, block, off, r);
     }
   } else if (p.epi == PI_EPI_GEGLU) {
     // even n: gate rows, odd n: up rows; of two columns m the even lane finishes the first, the odd lane the second
@@ -112,6 +143,7 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
   __shared__ __align__(8) unsigned long long bars[2 * STAGES + 4];
   __shared__ uint32_t s_tmem;
   __shared__ volatile int s_abort, s_dep_ok;
+  __shared__ pi_kv_place s_place[SPLIT ? BN : 1];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const uint32_t full0 = smem_u32(&bars[0]), empty0 = smem_u32(&bars[STAGES]), acc_full0 = smem_u32(&bars[2 * STAGES]),
                  acc_empty0 = smem_u32(&bars[2 * STAGES + 2]);
@@ -216,6 +248,9 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
     // ---- epilogue: warp w reads TMEM lanes 32 (w % 4).., warps 0-3 the first half of the columns, 4-7 the second ----
     const int quad = warp & 3, half = warp >> 2;
     constexpr int kHalfCols = BN >= 32 ? BN / 2 : 16;
+    if (SPLIT && p.epi == PI_EPI_MAPS_QKV)   // the rows' places do not depend on the preceding kernel
+      for (int c = tid; c < BN && (tile0 / p.rtiles) * BN + c < p.M; c += kEpiWarps * 32)
+        s_place[c] = pi_maps_kv_place(p.mkv, (tile0 / p.rtiles) * BN + c);
     pi_grid_dependency_wait();   // the epilogue reads and writes what the preceding kernels use
     for (int t = 0; t < my_tiles; ++t) {
       const int a = t % kAcc, tile = tile0 + t * tile_step;
@@ -267,7 +302,7 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
         float v = 0.f;
 #pragma unroll
         for (int r = 0; r < 8; ++r) v += s[r];
-        epilogue<1>(p, n, m0 + c, 1, &v);
+        epilogue<1>(p, n, m0 + c, 1, &v, &s_place[c]);
       }
     }
     __syncwarp();
@@ -360,7 +395,7 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
   PI_REQUIRE(ctx, lin->kind == PI_BF16 && a.x_bf16 && a.M >= 1, "the bf16 GEMM takes bf16 weights and activations");
   PI_REQUIRE(ctx, (uintptr_t)a.x_bf16 % 16 == 0 && a.x_stride % 8 == 0 && (uintptr_t)lin->w % 16 == 0 && lin->ld % 8 == 0,
              "bf16 operands must start and step on 16-byte boundaries");
-  PI_REQUIRE(ctx, a.epi == PI_EPI_STORE || (a.epi == PI_EPI_GEGLU && a.out_bf16 && lin->rows % 2 == 0) ||
+  PI_REQUIRE(ctx, a.epi == PI_EPI_STORE || (a.epi == PI_EPI_MAPS_QKV && a.maps_kv && a.maps_kv->dim % 2 == 0) || (a.epi == PI_EPI_GEGLU && a.out_bf16 && lin->rows % 2 == 0) ||
                       (a.epi == PI_EPI_DYT_RESIDUAL && a.residual && a.residual->x && a.residual->h && a.residual->post.w && a.residual->next.w),
              "this epilogue is not built for the bf16 GEMM");
   Bf16GemmParams p = {};
@@ -374,6 +409,7 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
   p.rtiles = (p.N + kTM - 1) / kTM;
   p.epi = a.epi;
   if (a.residual) p.res = *a.residual;
+  if (a.maps_kv) p.mkv = *a.maps_kv;
   p.err_flag = ctx->dev_err;
   int bn = a.M <= 16 ? 16 : a.M <= 32 ? 32 : a.M <= 64 ? 64 : 128;
   if (a.M > 128) {   // the wider tile where it does not cost more rounds of tiles over the SMs

@@ -83,6 +83,7 @@ struct Widen<float> {
 
 struct GemvParams {
   pi_dyt_residual res;   // PI_EPI_DYT_RESIDUAL
+  pi_maps_kv mkv;        // PI_EPI_MAPS_QKV
   const void* W;
   const float* scales;
   const float* x;
@@ -191,6 +192,9 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
     const int lb = my_pos / p.L.block_size;
     if (lb < p.lens[gm]) my_pb = p.tables[(size_t)gm * p.max_blocks + lb];
   }
+
+  pi_kv_place place = {0, -1, 0};   // the same for the fused [q;k;v] of a layered design
+  if (EPI == PI_EPI_MAPS_QKV && lane < mcount) place = pi_maps_kv_place(p.mkv, m0 + lane);
 
   // ---- stage x[m0 .. m0+mcount) into shared memory, once per CTA ---------------------------------
   bool landed = false;
@@ -443,6 +447,29 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
                 EPI == PI_EPI_GEGLU ? pi_gelu_tanh(g) * u : (g / (1.0f + expf(-g))) * u;
           }
         }
+      } else if (EPI == PI_EPI_MAPS_QKV) {
+        // lane m finishes activation row m0+m; the pair of rows is a rotation pair (q and k)
+#pragma unroll
+        for (int m = 0; m < MB; ++m) {
+          if (lane == m && m < mcount) {
+            float a[kRows] = {tot[0][m] * sc[0] * row_factor(m), tot[1][m] * sc[1] * row_factor(m)};
+            const pi_maps_col c0 = pi_maps_column(p.mkv, row0);
+            if (c0.rotated) {
+              const size_t at = (size_t)place.pos * (p.mkv.rot_dims >> 1) + (c0.d >> 1);
+              const float cs = p.mkv.rope_cos[at], sn = p.mkv.rope_sin[at];
+              const float u = a[0] * cs - a[1] * sn;
+              a[1] = a[1] * cs + a[0] * sn;
+              a[0] = u;
+            }
+#pragma unroll
+            for (int r = 0; r < kRows; ++r) {
+              if (row0 + r >= p.N) continue;
+              const pi_maps_col c = r == 0 ? c0 : pi_maps_column(p.mkv, row0 + r);
+              if (c.is_q) p.out[(size_t)(m0 + m) * p.out_stride + row0 + r] = a[r];
+              else pi_maps_kv_store(p.mkv, c, place.block, place.off, a[r]);
+            }
+          }
+        }
       } else if (EPI == PI_EPI_DYT_RESIDUAL) {
 #pragma unroll
         for (int r = 0; r < kRows; ++r)
@@ -498,6 +525,8 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
     if (norm) PI_PICK(PI_EPI_ADD, true); else PI_PICK(PI_EPI_ADD, false);
   } else if (epi == PI_EPI_GEGLU) {
     if constexpr (kFloatW) PI_PICK(PI_EPI_GEGLU, false);
+  } else if (epi == PI_EPI_MAPS_QKV) {
+    if constexpr (kFloatW) PI_PICK(PI_EPI_MAPS_QKV, false);
   } else if (epi == PI_EPI_DYT_RESIDUAL) {
     if constexpr (kFloatW) PI_PICK(PI_EPI_DYT_RESIDUAL, false);
   } else {
@@ -519,6 +548,7 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
     }
     if constexpr (kFloatW) {
       for (auto kk : {gemv_kernel<WT, MB, PI_EPI_GEGLU, false, false>, gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false>,
+                      gemv_kernel<WT, MB, PI_EPI_MAPS_QKV, false, false>,
                       gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false, kSplitWarps>}) {
         cudaError_t e = cudaFuncSetAttribute(kk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
@@ -607,6 +637,7 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
   const bool glu = a.epi == PI_EPI_SWIGLU || a.epi == PI_EPI_GEGLU;
   PI_REQUIRE(ctx, !glu || lin->rows % 2 == 0, "a gated epilogue needs interleaved gate/up rows");
   PI_REQUIRE(ctx, a.epi < PI_EPI_GEGLU || (lin->kind != PI_INT8 && !a.norm_weight), "this epilogue is built for bf16 and f32 weights");
+  PI_REQUIRE(ctx, a.epi != PI_EPI_MAPS_QKV || (a.maps_kv && a.maps_kv->dim % 2 == 0), "the fused [q;k;v] epilogue needs its operands and an even dim");
   PI_REQUIRE(ctx, a.epi != PI_EPI_DYT_RESIDUAL || (a.residual && a.residual->x), "the residual epilogue needs its operands");
   if (lin->rows == 0) return PI_OK;
   int mb = a.M >= 4 ? 4 : a.M >= 2 ? 2 : 1;
@@ -627,7 +658,7 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
   // Sets of three warps share a row pair instead: three times the loads in flight.
   int ksplit = 1;
   const size_t row_bytes = lin->ld * (lin->kind == PI_INT8 ? 1 : lin->kind == PI_BF16 ? 2 : 4);
-  if (!a.norm_weight && !a.rope && !glu && row_bytes > (size_t)(kSplitWarps - 1) * kSteps * 512 &&
+  if (!a.norm_weight && !a.rope && !glu && a.epi != PI_EPI_MAPS_QKV && row_bytes > (size_t)(kSplitWarps - 1) * kSteps * 512 &&
       npairs * 2 <= max_ctas * 8) {
     ksplit = kSplitWarps;
     warps = 2 * kSplitWarps;
@@ -649,6 +680,7 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
   p.M = a.M;
   p.eps = a.norm_eps;
   if (a.residual) p.res = *a.residual;
+  if (a.maps_kv) p.mkv = *a.maps_kv;
   p.err_flag = ctx->dev_err;
   p.rope_hd = 0;
   if (a.rope) {

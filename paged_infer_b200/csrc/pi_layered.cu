@@ -6,9 +6,9 @@
 //
 // Dynamic Tanh needs no statistics, so all of it folds into the projection that ends a sublayer: its epilogue adds
 // the normalised result to the f32 residual stream and hands on the normalised input of the next sublayer.  Per layer:
-//   1. [q;k;v(;gates)] projection
-//   2. attention: rotary + KV write, attention (its own normalisation in the same kernel); or the recurrence with head
-//      norm and output gate in the same kernel
+//   1. [q;k;v(;gates)] projection; attention: rotary positions and the KV write in its epilogue
+//   2. attention (with its own normalisation in the same kernel); or the recurrence with head norm and output gate in the
+//      same kernel
 //   3. output projection, epilogue = residual update + next norm
 //   4. interleaved [gate;up] projection, epilogue = gelu(gate) * up      (layers with a feed-forward)
 //   5. down projection, epilogue = residual update + next norm
@@ -548,12 +548,9 @@ pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool
     const Layer& L = m->layers[i];
     const pi_layer_config& c = L.c;
     const pi_dyt after = i + 1 < NL ? m->layers[i + 1].norm1 : m->final_norm;
-    {
-      pi_linear_args a;
-      a.out = m->proj;
-      a.out_stride = m->ld_proj;
-      PI_TRY(project(ctx, L.in, m->h, m->ld_h, M, bf16, a));
-    }
+    pi_linear_args in;
+    in.out = m->proj;
+    in.out_stride = m->ld_proj;
     if (c.mixer == PI_MIXER_ATTENTION) {
       const pi_kv_region& g = pool->regions[L.attn];
       pi_kv_view kv;
@@ -578,9 +575,35 @@ pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool
       a.rot_dims = c.rot_dims;
       a.rope_cos = m->ropes[L.rope].cos;
       a.rope_sin = m->ropes[L.rope].sin;
-      PI_TRY(pi_launch_maps_rope_kv(ctx, a, kv, m->proj, m->ld_proj, b));
+      pi_maps_kv mk;
+      if (c.dim % 2 == 0) {   // rotary positions and the KV write fold into the projection
+        mk.q_rows = c.heads * c.maps * c.dim;
+        mk.k_rows = c.kv_heads * c.maps * c.dim;
+        mk.maps = c.maps;
+        mk.dim = c.dim;
+        mk.vdim = c.vdim;
+        mk.rot_dims = c.rot_dims;
+        mk.rope_cos = a.rope_cos;
+        mk.rope_sin = a.rope_sin;
+        mk.base = kv.base;
+        mk.kind = kv.kind;
+        mk.kv_heads = kv.kv_heads;
+        mk.dp = kv.dp;
+        mk.vp = kv.vp;
+        mk.block_size = kv.block_size;
+        mk.row_seq = b.row_seq;
+        mk.row_pos = b.row_pos;
+        mk.lens = b.lens;
+        mk.tables = b.tables;
+        mk.max_blocks = b.max_blocks;
+        in.epi = PI_EPI_MAPS_QKV;
+        in.maps_kv = &mk;
+      }
+      PI_TRY(project(ctx, L.in, m->h, m->ld_h, M, bf16, in));
+      if (in.epi != PI_EPI_MAPS_QKV) PI_TRY(pi_launch_maps_rope_kv(ctx, a, kv, m->proj, m->ld_proj, b));
       PI_TRY(pi_launch_maps_attention(ctx, a, kv, m->proj, m->ld_proj, m->core, m->ld_core, kind, b));
     } else {
+      PI_TRY(project(ctx, L.in, m->h, m->ld_h, M, bf16, in));
       pi_recurrence r = L.rec;
       r.state = state->data;
       r.state_stride = state->stride;
@@ -620,17 +643,17 @@ pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool
   if (st.n_out == 0) return PI_OK;
   // the last epilogue left the final norm of every row in h; anything but all rows in order is gathered from x
   const bool head_bf16 = act_bf16(ctx, m, st.n_out);
-  const void* in = m->h;
+  const void* last = m->h;
   if (!(st.all_rows && head_bf16 == bf16)) {
     pi_prof_scope prof(ctx, PI_PROF_OTHER);
     auto k = head_bf16 ? gather_dyt_kernel<__nv_bfloat16> : gather_dyt_kernel<float>;
     PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(st.n_out), dim3(256), 0, 1, (const float*)m->x, W, st.out_rows, m->final_norm, m->head_in.ptr, m->ld_h));
-    in = m->head_in.ptr;
+    last = m->head_in.ptr;
   }
   pi_linear_args a;
   a.out = static_cast<float*>(m->logits.ptr);
   a.out_stride = m->c.vocab_size;
-  return project(ctx, m->embed, in, m->ld_h, st.n_out, head_bf16, a);
+  return project(ctx, m->embed, last, m->ld_h, st.n_out, head_bf16, a);
 }
 
 pi_status multi_step(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool* state, const Staged& st, uint32_t* history, int* counter) {

@@ -28,6 +28,7 @@ ALONE = {
     "attention_mha": attention(heads=3, kv_heads=3, dim=64, vdim=128, window=100, rot=32, base=500.0, ff=0),
     "attention_wide": attention(heads=2, kv_heads=1, dim=128, vdim=256, window=1000, scale=0.2, ff=0),
     "attention_window1": attention(heads=2, kv_heads=1, dim=6, vdim=10, window=1, ff=0),
+    "attention_odd_dim": attention(heads=4, kv_heads=2, dim=11, vdim=9, window=19, rot=4, ff=0),
     "attention_no_rotation": attention(heads=5, kv_heads=1, dim=18, vdim=34, window=17, rot=0, ff=31),
     "attention_group12": attention(heads=12, kv_heads=1, dim=16, vdim=16, window=50, ff=0),
     "gla": gla(),
@@ -253,7 +254,7 @@ def test_wide_model_many_rows(ctx):
 @BOTH
 def test_sizes_that_are_multiples_of_nothing(ctx, compute):
     cfg = config([attention(heads=3, kv_heads=1, dim=10, vdim=7, window=21, rot=6, ff=13), gla(heads=1, dim=5, vdim=3, ff=1),
-                  mlstm(heads=1, dim=1, vdim=1), mlstm(heads=3, dim=9, vdim=131), gla(heads=2, dim=31, vdim=65, tau=1.5)], width=37, vocab=41)
+                  mlstm(heads=1, dim=3, vdim=6), mlstm(heads=3, dim=9, vdim=131), gla(heads=2, dim=31, vdim=65, tau=1.5)], width=37, vocab=41)
     t = tensors(cfg, 71, rank=3)
     toks = tokens(160, 72, 41)
     want = reference(cfg, t).forward(toks)
