@@ -184,3 +184,187 @@ class Sumosun:
             if layer_outputs is not None:
                 layer_outputs.append(x.copy())
         return linear(self.t["embed"], self.norm("final.norm", x))
+
+
+# ---- mechanisms of Lilosun ------------------------------------------------------------------------------------------
+# Notation: c = latent channel, n = state channel, e = value channel.
+
+def softplus(z):
+    return np.maximum(z, 0) + np.log1p(np.exp(-np.abs(z)))
+
+
+def layer_norm(x, w, eps):
+    """Zero mean and unit variance over the last axis, times w; no bias."""
+    d = x - np.mean(x, axis=-1, keepdims=True)
+    return d / np.sqrt(np.mean(d * d, axis=-1, keepdims=True) + eps) * w
+
+
+def yarn_frequencies(dims, base, scaling):
+    """(angle per position of every pair, factor of cos and sin).  ``scaling`` None: base^(-2i/dims) and 1."""
+    i = np.arange(dims // 2)
+    f = float(base) ** (-2.0 * i / dims)
+    if scaling is None:
+        return f, 1.0
+
+    def pair_that_turns(times):   # (fractional) pair index that makes this many turns within the original length
+        return dims * np.log(scaling["original"] / (2 * np.pi * times)) / (2 * np.log(base))
+
+    lo = max(np.floor(pair_that_turns(scaling["fast"])), 0)
+    hi = min(np.ceil(pair_that_turns(scaling["slow"])), dims - 1)
+    ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0, 1)
+    return f / scaling["factor"] * ramp + f * (1 - ramp), 0.1 * np.log(scaling["factor"]) + 1
+
+
+def rotate_pairs(x, positions, frequencies, gain):
+    """x [tokens, heads, dim]: the pairs (2i, 2i+1) turn by position * frequencies[i] and grow by ``gain``; the rest passes."""
+    out = x.copy()
+    for i, f in enumerate(frequencies):
+        a = np.asarray(positions, np.float64) * f
+        c, s = (gain * np.cos(a)).astype(x.dtype)[:, None], (gain * np.sin(a)).astype(x.dtype)[:, None]
+        u, v = x[:, :, 2 * i], x[:, :, 2 * i + 1]
+        out[:, :, 2 * i] = u * c - v * s
+        out[:, :, 2 * i + 1] = v * c + u * s
+    return out
+
+
+def latent_attention(h, w, heads, dim, rot_dim, vdim, rank, rot_base, scaling, scale, window, eps):
+    """w: dict q, dkv, dkv.norm, uk, uv, g, o.  Every head's keys and values are spelled out from the latent vector; the last
+    rot_dim key channels, rotated, are common to the heads."""
+    T = h.shape[0]
+    pos = np.arange(T)
+    f, gain = yarn_frequencies(rot_dim, rot_base, scaling)
+    q = linear(w["q"], h).reshape(T, heads, dim + rot_dim)
+    q_rot = rotate_pairs(q[:, :, dim:], pos, f, gain)
+    down = linear(w["dkv"], h)
+    c = unit_rms(down[:, :rank], eps) * w["dkv.norm"]
+    k_rot = rotate_pairs(down[:, None, rank:], pos, f, gain)[:, 0]
+    k = linear(w["uk"], c).reshape(T, heads, dim)
+    v = linear(w["uv"], c).reshape(T, heads, vdim)
+    o = np.zeros((T, heads, vdim), h.dtype)
+    for n in range(heads):
+        o[:, n] = window_softmax(np.concatenate([q[:, n, :dim], q_rot[:, n]], -1), np.concatenate([k[:, n], k_rot], -1), v[:, n], scale, window)
+    return linear(w["o"], o.reshape(T, heads * vdim) * sigmoid(linear(w["g"], h)))
+
+
+def causal_conv(x, w, b):
+    """Per channel: y_t = b + sum_j w[:, j] x_(t - taps + 1 + j), zeros before the start."""
+    T, taps = x.shape[0], w.shape[1]
+    past = np.concatenate([np.zeros((taps - 1, x.shape[1]), x.dtype), x])
+    y = np.zeros_like(x) + b
+    for j in range(taps):
+        y = y + w[:, j] * past[j:j + T]
+    return y
+
+
+def ssd_scan(x, B, C, dt, a_log, state):
+    """One head.  S_t = exp(-exp(a_log) dt_t) S_(t-1) + dt_t B_t x_t^T, y_t = S_t^T C_t.  -> (y [T, vdim], S)."""
+    S = state.copy()
+    y = np.zeros_like(x)
+    for t in range(x.shape[0]):
+        S = np.exp(-np.exp(a_log) * dt[t]) * S + dt[t] * np.outer(B[t], x[t])
+        y[t] = S.T @ C[t]
+    return y, S
+
+
+def grouped_unit_rms(x, groups, eps):
+    T, n = x.shape
+    return unit_rms(x.reshape(T, groups, n // groups), eps).reshape(T, n)
+
+
+def mamba2(h, w, heads, vdim, state, groups, norm_groups, eps):
+    """w: dict in, conv, conv.b, dt_bias, A_log, D, norm, o."""
+    T, inner, gn = h.shape[0], heads * vdim, groups * state
+    p = linear(w["in"], h)
+    z, xbc, dt = p[:, :inner], p[:, inner:2 * inner + 2 * gn], p[:, 2 * inner + 2 * gn:]
+    xbc = silu(causal_conv(xbc, w["conv"], w["conv.b"]))
+    x = xbc[:, :inner].reshape(T, heads, vdim)
+    B = xbc[:, inner:inner + gn].reshape(T, groups, state)
+    C = xbc[:, inner + gn:].reshape(T, groups, state)
+    dt = softplus(dt + w["dt_bias"])
+    y = np.zeros((T, heads, vdim), h.dtype)
+    for n in range(heads):
+        g = n // (heads // groups)
+        y[:, n] = ssd_scan(x[:, n], B[:, g], C[:, g], dt[:, n], w["A_log"][n], np.zeros((state, vdim), h.dtype))[0] + w["D"][n] * x[:, n]
+    return linear(w["o"], grouped_unit_rms(y.reshape(T, inner) * silu(z), norm_groups, eps) * w["norm"])
+
+
+def silu_mlp(x, gate, up, down):
+    return linear(down, silu(linear(gate, x)) * linear(up, x))
+
+
+def clamped_mlp(x, gate, up, down, limit):
+    """g sigmoid(1.702 g) (u + 1) with g cut from above and u on both sides."""
+    g, u = np.minimum(linear(gate, x), limit), np.clip(linear(up, x), -limit, limit)
+    return linear(down, g * sigmoid(1.702 * g) * (u + 1))
+
+
+def route(z, correction, top, groups, keep):
+    """Router logits [tokens, experts] -> (chosen experts [tokens, top], their weights).  Groups of neighbouring experts compete
+    by the sum of their two best corrected scores; the weights are the plain scores of the chosen, brought to sum 1."""
+    s = sigmoid(z)
+    choice = s + correction
+    T, E = z.shape
+    n = E // groups
+    ids = np.zeros((T, top), np.int64)
+    for t in range(T):
+        best = [np.sort(choice[t, g * n:(g + 1) * n])[-2:].sum() for g in range(groups)]
+        kept = set(np.argsort(best)[::-1][:keep].tolist())
+        allowed = [(choice[t, e], -e) for e in range(E) if e // n in kept]
+        ids[t] = [-e for _, e in sorted(allowed, reverse=True)[:top]]
+    w = np.take_along_axis(s, ids, 1)
+    return ids, w / (w.sum(-1, keepdims=True) + 1e-20)
+
+
+def moe(h, w, top, groups, keep, limit, shared_limit):
+    """w: dict router, correction, e<i>.gate/up/down and, with a shared expert, shared.gate/up/down/sg."""
+    ids, weights = route(linear(w["router"], h), w["correction"], top, groups, keep)
+    out = np.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, p in zip(ids[t], weights[t]):
+            n = f"e{e}."
+            out[t] += p * clamped_mlp(h[t], w[n + "gate"], w[n + "up"], w[n + "down"], limit)
+    if shared_limit is not None:
+        out = out + sigmoid(linear(w["shared.sg"], h)) * clamped_mlp(h, w["shared.gate"], w["shared.up"], w["shared.down"], shared_limit)
+    return out
+
+
+class Lilosun:
+    """The whole design from a config dict and a dict of float arrays under the checkpoint's tensor names."""
+
+    def __init__(self, config: dict, tensors: dict, dtype=np.float64):
+        self.c = config
+        self.t = {k: np.asarray(v, dtype) for k, v in tensors.items()}
+
+    def part(self, prefix):
+        return {k[len(prefix):]: v for k, v in self.t.items() if k.startswith(prefix)}
+
+    def mixer(self, i, layer, h):
+        w, m, eps = self.part(f"l{i}.mix."), layer["mixer"], self.c["norm"]["eps"]
+        if layer["type"] == "latent_attention":
+            rot, mask = m["rot"], m.get("mask")
+            return latent_attention(h, w, m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], rot["base"], rot.get("scaling"), m["scale"],
+                                    mask["size"] if mask else None, eps)
+        if layer["type"] == "mamba2":
+            return mamba2(h, w, m["heads"], m["vdim"], m["state"], m["groups"], m["norm_groups"], eps)
+        raise ValueError(f"unknown mixer {layer['type']}")
+
+    def feed_forward(self, i, mlp, h):
+        w = self.part(f"l{i}.mlp.")
+        if mlp["kind"] == "dense":
+            return silu_mlp(h, w["gate"], w["up"], w["down"])
+        r, g = mlp["router"], mlp["router"].get("groups") or {"count": 1, "keep": 1}
+        shared = mlp.get("shared")
+        return moe(h, w, r["top"], g["count"], g["keep"], mlp["expert"]["limit"], shared["limit"] if shared else None)
+
+    def forward(self, tokens, layer_outputs: list | None = None):
+        """Logits [tokens, vocab] of one sequence from its first token."""
+        eps = self.c["norm"]["eps"]
+        x = self.t["embed"][np.asarray(tokens)]
+        for i, layer in enumerate(self.c["layers"]):
+            l = f"l{i}."
+            x = x + self.t[l + "ls1"] * self.mixer(i, layer, layer_norm(x, self.t[l + "norm1"], eps))
+            if layer.get("mlp"):
+                x = x + self.t[l + "ls2"] * self.feed_forward(i, layer["mlp"], layer_norm(x, self.t[l + "norm2"], eps))
+            if layer_outputs is not None:
+                layer_outputs.append(x.copy())
+        return linear(self.t["head"], layer_norm(x, self.t["final.norm"], eps)) * self.c["logit_scale"]
