@@ -365,7 +365,11 @@ pi_status pi_kv_fill_normal(pi_ctx* ctx, pi_kv_pool* pool, uint64_t seed, float 
  * pi_model_step like every other model; what its mixers carry from token to token lives in a KV pool (attention) and
  * in a state pool (recurrences).  No counterpart in the reference. */
 
-enum { PI_MIXER_ATTENTION = 0, PI_MIXER_GLA = 1, PI_MIXER_MLSTM = 2 };
+enum { PI_MIXER_ATTENTION = 0, PI_MIXER_GLA = 1, PI_MIXER_MLSTM = 2, PI_MIXER_LATENT = 3 /* latent attention */, PI_MIXER_SSD = 4 /* state-space, scalar decay */ };
+enum { PI_FF_GELU = 0, PI_FF_SILU = 1, PI_FF_EXPERTS = 2 /* clamped gated units, routed */ };
+/* Normalisation: Dynamic Tanh before and after every sublayer, or layer norm (a weight, no bias) before it and a scale per
+ * channel behind it. */
+enum { PI_NORM_DYT = 0, PI_NORM_LAYER = 1 };
 
 typedef struct {
   int32_t mixer;
@@ -377,7 +381,20 @@ typedef struct {
   float rot_base, scale, diff;
   float tau;               /* GLA: log decay = log_sigmoid(z) / tau */
   float gate_cap;          /* mLSTM: soft cap of both gates */
-  int32_t ff;              /* feed-forward size, 0: the layer has none */
+  int32_t ff;              /* feed-forward size (of one expert), 0: the layer has none */
+  int32_t ff_kind;
+  /* latent attention: dim unrotated and rot_dims rotated channels per head, rank = latent channels.  Rotation frequencies may be
+   * stretched: pairs that turn less than rot_slow times within rot_original positions are slowed by rot_factor, those that turn
+   * more than rot_fast times are not; cos and sin grow by 0.1 ln(rot_factor) + 1.  rot_factor 1: plain. */
+  int32_t rank;
+  double rot_factor, rot_original, rot_fast, rot_slow;
+  /* state-space recurrence: dim = state channels, common to the heads of a group; conv = taps of the convolution ahead of it;
+   * the result is normalised in norm_groups parts */
+  int32_t groups, norm_groups, conv;
+  /* experts: of `experts`, `top` per token, out of the best keep_groups of expert_groups groups; shared_ff: an expert that
+   * every token meets (0: none); limits: where the units are clamped */
+  int32_t experts, top, expert_groups, keep_groups, shared_ff;
+  float limit, shared_limit;
 } pi_layer_config;
 
 typedef struct {
@@ -385,6 +402,9 @@ typedef struct {
   float norm_eps;
   int32_t compute;         /* PI_BF16: bf16 projections and KV, f32 accumulation; PI_F32: f32 throughout */
   int32_t max_rows;        /* tokens one step can take */
+  int32_t norm;            /* PI_NORM_* */
+  int32_t tied;            /* 1: the embedding is the output matrix, 0: "head" is */
+  float logit_scale;
   const pi_layer_config* layers;
 } pi_layered_config;
 
@@ -395,8 +415,7 @@ typedef struct {
   const void* data;        /* host */
 } pi_named_tensor;
 
-/* Layers pre- and post-normalised by Dynamic Tanh, gelu-gated feed-forward, tied embedding.  Tensors are looked up by
- * their checkpoint names; matrices are bf16. */
+/* Tensors are looked up by their checkpoint names; matrices are bf16. */
 pi_status pi_model_create_layered(pi_ctx* ctx, const pi_layered_config* cfg, const pi_named_tensor* tensors, int n_tensors, pi_model** out);
 /* Random matrices N(0, std) generated on the device; gla_rank = rank of the GLA decay's low-rank input. */
 pi_status pi_model_create_layered_synthetic(pi_ctx* ctx, const pi_layered_config* cfg, int gla_rank, uint64_t seed, float std, pi_model** out);

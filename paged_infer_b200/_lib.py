@@ -62,12 +62,16 @@ class ModelWeightsC(C.Structure):
 
 class LayerConfigC(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "maps", "window", "rot_dims")] + \
-               [(n, C.c_float) for n in ("rot_base", "scale", "diff", "tau", "gate_cap")] + [("ff", C.c_int32)]
+               [(n, C.c_float) for n in ("rot_base", "scale", "diff", "tau", "gate_cap")] + \
+               [(n, C.c_int32) for n in ("ff", "ff_kind", "rank")] + \
+               [(n, C.c_double) for n in ("rot_factor", "rot_original", "rot_fast", "rot_slow")] + \
+               [(n, C.c_int32) for n in ("groups", "norm_groups", "conv", "experts", "top", "expert_groups", "keep_groups", "shared_ff")] + \
+               [(n, C.c_float) for n in ("limit", "shared_limit")]
 
 
 class LayeredConfigC(C.Structure):
     _fields_ = [("width", C.c_int32), ("vocab_size", C.c_int32), ("num_layers", C.c_int32), ("norm_eps", C.c_float), ("compute", C.c_int32),
-                ("max_rows", C.c_int32), ("layers", C.POINTER(LayerConfigC))]
+                ("max_rows", C.c_int32), ("norm", C.c_int32), ("tied", C.c_int32), ("logit_scale", C.c_float), ("layers", C.POINTER(LayerConfigC))]
 
 
 class NamedTensorC(C.Structure):

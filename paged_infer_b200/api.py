@@ -613,8 +613,11 @@ class LayeredModel(_Steps):
     def _config(cls, config: LayeredConfig, compute: str, max_rows: int) -> _lib.LayeredConfigC:
         layers = (_lib.LayerConfigC * len(config.layers))(*[
             _lib.LayerConfigC(l.mixer, l.heads, l.kv_heads, l.dim, l.vdim, l.maps, 0 if l.window is None else l.window, l.rot_dims, l.rot_base,
-                              l.scale, l.diff, l.tau, l.gate_cap, l.ff) for l in config.layers])
-        cfg = _lib.LayeredConfigC(config.width, config.vocab_size, len(config.layers), config.norm_eps, cls.COMPUTE[compute], max_rows, layers)
+                              l.scale, l.diff, l.tau, l.gate_cap, l.ff, l.ff_kind, l.rank, l.rot_factor, l.rot_original, l.rot_fast, l.rot_slow,
+                              l.groups, l.norm_groups, l.conv, l.experts, l.top, l.expert_groups, l.keep_groups, l.shared_ff, l.limit, l.shared_limit)
+            for l in config.layers])
+        cfg = _lib.LayeredConfigC(config.width, config.vocab_size, len(config.layers), config.norm_eps, cls.COMPUTE[compute], max_rows, config.norm,
+                                  int(config.tied), config.logit_scale, layers)
         cfg._layers = layers
         return cfg
 

@@ -5,6 +5,7 @@
 //   a_j     = softmax(score_j) V
 //   out     = a_1                                             (one map)
 //   o = a_1 - lambda a_2;  out = out_scale o / rms(o)          (two maps)
+//   out *= sigmoid(gate)                                       (with an output gate)
 //
 // Kernels: maps_rope_kv_kernel rotates q and k and writes k and v into the pool; maps_attn_plain_kernel is the f32
 // path and the one for sizes the tensor-core kernels of pi_attention_maps_tc.cu do not hold.
@@ -102,6 +103,7 @@ __global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const
     const T* kt = static_cast<const T*>(p.base) + ((size_t)table[lb] * p.kv_heads + g) * tile;
     const T* vt = kt + (size_t)p.block_size * nm * DP + (size_t)off * p.vp;
     kt += (size_t)off * nm * DP;
+    if (p.v_in_k) vt = kt;
 #pragma unroll
     for (int m = 0; m < 2; ++m) {
       if (m >= nm) break;
@@ -146,7 +148,8 @@ __global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const
     r = p.out_scale / sqrtf(t / (float)p.vdim + p.eps);
   }
   O* o = static_cast<O*>(p.out) + (size_t)row * p.out_stride + (size_t)head * p.vdim;
-  for (int e = tid; e < p.vdim; e += blockDim.x) o[e] = pi_from_f32<O>(acc[e] * r);
+  const float* gate = p.gate ? p.gate + (size_t)row * p.gate_stride + (size_t)head * p.vdim : nullptr;
+  for (int e = tid; e < p.vdim; e += blockDim.x) o[e] = pi_from_f32<O>(acc[e] * (gate ? r * pi_sigmoid(gate[e]) : r));
 }
 
 }  // namespace
@@ -165,7 +168,7 @@ pi_status pi_launch_maps_attention(pi_ctx* ctx, const pi_maps_attention& a, cons
                                    void* out, size_t out_stride, int out_kind, const pi_seq_batch& b) {
   pi_prof_scope prof(ctx, PI_PROF_ATTENTION);
   MapsParams p = {qkv, stride, out, out_stride, kv.base, a.heads, a.kv_heads, a.maps, a.dim, a.vdim, kv.dp, kv.vp, kv.block_size,
-                  a.window, a.scale, a.eps, a.lambda, a.out_scale, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks};
+                  a.window, a.scale, a.eps, a.lambda, a.out_scale, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks, a.gate, a.gate_stride, a.v_in_k};
   if (pi_maps_attention_tc_usable(ctx, a, kv)) return pi_launch_maps_attention_tc(ctx, p, out_kind, b);
   const size_t smem = sizeof(float) * ((size_t)a.maps * a.dim + (size_t)kPlainWarps * a.maps * a.vdim);
   PI_REQUIRE(ctx, smem <= 48 * 1024, "attention heads of %d / %d channels are too wide", a.dim, a.vdim);

@@ -13,6 +13,9 @@ struct MapsParams {
   float scale, eps, lambda, out_scale;
   const int32_t *row_seq, *row_pos, *lens, *tables;
   int max_blocks;
+  const float* gate;
+  size_t gate_stride;
+  int v_in_k;
 };
 
 // bf16 pools: true when the tensor-core kernels hold these sizes.

@@ -375,7 +375,10 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
       const size_t o0 = (size_t)row * a.out_stride + (size_t)(g * p.group + head) * a.vdim;
 #pragma unroll
       for (int i = 0; i < VMAX / 32; ++i)
-        if (lane + 32 * i < a.vdim) store_out(p, o0 + lane + 32 * i, d[i] * r);
+        if (lane + 32 * i < a.vdim) {
+          const float gate = a.gate ? pi_sigmoid(a.gate[(size_t)row * a.gate_stride + (size_t)(g * p.group + head) * a.vdim + lane + 32 * i]) : 1.f;
+          store_out(p, o0 + lane + 32 * i, d[i] * r * gate);
+        }
     }
   };
   if (p.nsplit > 1) finish(std::integral_constant<int, kMaxSplits>());
@@ -445,23 +448,27 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
       tpos[h] = ok ? p_first + tok : -1;      // -1: sees nothing
       q[h] = a.q + (size_t)(row0 + tok0 + (ok ? tok : 0)) * a.stride + ((size_t)(g * p.group + head) * MAPS + map) * a.dim;
     }
-    float v[KMAP][4][2];                      // all loads first, addresses clamped instead of branches
+    constexpr int B = KMAP <= 8 ? KMAP : 4;   // of a batch of k steps all loads first, addresses clamped instead of branches
 #pragma unroll
-    for (int ks = 0; ks < KMAP; ++ks)
+    for (int k0 = 0; k0 < KMAP; k0 += B) {
+      float v[B][4][2];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {           // a0: row, a1: row + 8, a2 / a3: channels + 8
-        const int d = ks * 16 + (lane & 3) * 2 + (j >> 1) * 8;
-        v[ks][j][0] = q[j & 1][min(d, a.dim - 1)];
-        v[ks][j][1] = q[j & 1][min(d + 1, a.dim - 1)];
-      }
+      for (int ks = 0; ks < B; ++ks)
 #pragma unroll
-    for (int ks = 0; ks < KMAP; ++ks)
+        for (int j = 0; j < 4; ++j) {         // a0: row, a1: row + 8, a2 / a3: channels + 8
+          const int d = (k0 + ks) * 16 + (lane & 3) * 2 + (j >> 1) * 8;
+          v[ks][j][0] = q[j & 1][min(d, a.dim - 1)];
+          v[ks][j][1] = q[j & 1][min(d + 1, a.dim - 1)];
+        }
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int d = ks * 16 + (lane & 3) * 2 + (j >> 1) * 8;
-        const bool is = ks < nks && tpos[j & 1] >= 0;
-        qa[ks][j] = pack(is && d < a.dim ? v[ks][j][0] : 0.f, is && d + 1 < a.dim ? v[ks][j][1] : 0.f);
-      }
+      for (int ks = 0; ks < B; ++ks)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int d = (k0 + ks) * 16 + (lane & 3) * 2 + (j >> 1) * 8;
+          const bool is = k0 + ks < nks && tpos[j & 1] >= 0;
+          qa[k0 + ks][j] = pack(is && d < a.dim ? v[ks][j][0] : 0.f, is && d + 1 < a.dim ? v[ks][j][1] : 0.f);
+        }
+    }
   }
   float acc[VMAX / 8][4];
 #pragma unroll
@@ -594,7 +601,12 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
     for (int j = 0; j < VMAX / 8; ++j)
       if (j < nv) {
         const int c = j * 8 + (lane & 3) * 2;
-        const float v0 = acc[j][2 * h] * r, v1 = acc[j][2 * h + 1] * r;
+        float v0 = acc[j][2 * h] * r, v1 = acc[j][2 * h + 1] * r;
+        if (a.gate) {
+          const float* gate = a.gate + (size_t)(row0 + tok0 + tok) * a.gate_stride + (size_t)(g * p.group + head) * a.vdim;
+          v0 *= pi_sigmoid(gate[min(c, a.vdim - 1)]);
+          v1 *= pi_sigmoid(gate[min(c + 1, a.vdim - 1)]);
+        }
         if (p.out_bf16 && c + 1 < a.vdim && ((o0 + c) & 1) == 0) {
           *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(a.out) + o0 + c) = pack(v0, v1);
         } else {
@@ -626,6 +638,8 @@ TcKernel pick_decode(int k, int vp) {
 }
 template <int MAPS, int VMAX>
 TcKernel pick_tile(int k) {
+  if constexpr (MAPS == 1)   // one map may have wider keys
+    if (k > 8) return k <= 12 ? maps_tile_kernel<1, 12, VMAX> : maps_tile_kernel<1, 16, VMAX>;
   return k <= 4 ? maps_tile_kernel<MAPS, 4, VMAX> : maps_tile_kernel<MAPS, 8, VMAX>;
 }
 template <int MAPS>
@@ -650,7 +664,7 @@ cudaError_t grant(pi_ctx* ctx, TcKernel k, size_t smem) {
 }  // namespace
 
 bool pi_maps_attention_tc_usable(const pi_ctx* ctx, const pi_maps_attention& a, const pi_kv_view& kv) {
-  return ctx->opt_tensor_gemm && kv.kind == PI_BF16 && kv.dp <= 128 && kv.vp <= 256 && a.heads / a.kv_heads <= 16 * kTileWarps / a.maps;
+  return ctx->opt_tensor_gemm && kv.kind == PI_BF16 && kv.dp <= (a.maps == 1 ? 256 : 128) && kv.vp <= 256 && a.heads / a.kv_heads <= 16 * kTileWarps / a.maps;
 }
 
 pi_status pi_launch_maps_attention_tc(pi_ctx* ctx, const MapsParams& a, int out_kind, const pi_seq_batch& b) {

@@ -152,8 +152,11 @@ enum pi_epilogue {
   PI_EPI_SWIGLU = 2,    // rows interleaved gate/up: out[m][r/2] = silu(v[2i]) * v[2i+1]
   PI_EPI_GEGLU = 3,     // the same with the tanh form of gelu
   PI_EPI_MAPS_QKV = 5,  // fused [q;k;v] of multi-map attention: rotary q to `out`, rotary k and v into the paged pool (pi_maps_kv)
-  PI_EPI_DYT_RESIDUAL = 4   // x[m][r] += dyt(post, v); h[m][r] = dyt(next, x[m][r])   (pi_dyt_residual)
+  PI_EPI_DYT_RESIDUAL = 4,  // x[m][r] += dyt(post, v); h[m][r] = dyt(next, x[m][r])   (pi_dyt_residual)
+  PI_EPI_CLAMP_GLU = 6,     // rows interleaved gate/up: g = min(gate, limit), u = clamp(up, +-limit): g sigmoid(1.702 g) (u + 1)
+  PI_EPI_SCALE_ADD = 7      // out[m][r] += out_scale[r] v        (residual add with a layer scale)
 };
+inline bool pi_epi_glu(pi_epilogue e) { return e == PI_EPI_SWIGLU || e == PI_EPI_GEGLU || e == PI_EPI_CLAMP_GLU; }
 
 // Dynamic Tanh, a normalisation without statistics: tanh(alpha v) w + b, element by element.  Because it needs no row
 // sum, it folds into whatever kernel produces its input.
@@ -217,6 +220,19 @@ struct pi_maps_kv {
   int max_blocks = 0;
 };
 
+// A stack of equal matrices (the experts of a layer, one below the other), of which every row of the batch uses one.
+// CUDA-core path: row m of the output is expert[m]'s, its input is row m / x_div of x.  Tensor-core path: the rows lie grouped by
+// expert, tile i covers rows tiles[i].y .. + tiles[i].z of expert tiles[i].x; the table and its length are on the device.
+struct pi_expert_rows {
+  int experts = 0;
+  const int32_t* expert = nullptr;
+  int x_div = 1;
+  const int4* tiles = nullptr;
+  const int32_t* n_tiles = nullptr;
+  int max_tiles = 0;          // host-side bound
+  int tile_rows = 0;          // rows of a full tile: 16, 32, 64 or 128
+};
+
 struct pi_linear_args {
   const float* x = nullptr;   // [M][x_stride]
   size_t x_stride = 0;
@@ -245,6 +261,13 @@ struct pi_linear_args {
   __nv_bfloat16* out_bf16 = nullptr;
   const pi_dyt_residual* residual = nullptr;   // PI_EPI_DYT_RESIDUAL
   const pi_maps_kv* maps_kv = nullptr;         // PI_EPI_MAPS_QKV
+  float glu_limit = 0.f;                       // PI_EPI_CLAMP_GLU
+  // gated epilogues: only the first glu_rows rows are gate/up pairs (0: all), the rows behind them are stored to `rest` as f32
+  int glu_rows = 0;
+  float* rest = nullptr;
+  size_t rest_stride = 0;
+  const float* out_scale = nullptr;            // PI_EPI_SCALE_ADD
+  const pi_expert_rows* experts = nullptr;     // lin is a stack of experts
 };
 
 // tcgen05 GEMM for bf16 weights and bf16 activations with f32 accumulation (a.x_bf16; any shape).
@@ -485,6 +508,14 @@ __device__ __forceinline__ float pi_sigmoid(float z) {   // no overflow on eithe
   const float e = expf(-fabsf(z));
   return (z >= 0.f ? 1.0f : e) / (1.0f + e);
 }
+// gate and up value of one channel -> its activation
+__device__ __forceinline__ float pi_glu(int epi, float g, float u, float limit) {
+  if (epi == PI_EPI_GEGLU) return pi_gelu_tanh(g) * u;
+  if (epi == PI_EPI_SWIGLU) return g * pi_sigmoid(g) * u;
+  g = fminf(g, limit);
+  return g * pi_sigmoid(1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+}
+__device__ __forceinline__ float pi_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float pi_log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float pi_bf16_bits_to_f32(uint16_t b) { return __uint_as_float(((uint32_t)b) << 16); }
 // Programmatic dependent launch: wait for the producer grid's memory, and allow

@@ -12,6 +12,10 @@
 // K over a thread-block cluster: every CTA parks its partial tile in shared memory and finishes every ksplit-th column,
 // adding the slices in rank order.  Weight tiles of the first stages are requested before the dependency wait.  All
 // waits are bounded; one that runs out sets the context's error word.
+//
+// GROUPED: the weights are a stack of experts and the activation rows lie grouped by expert; a device-built table names the
+// column tiles (expert, first row, rows), so that the launch needs no routing result on the host.  Every tile is
+// multiplied in full; what belongs to the next expert is dropped in the epilogue.
 #include <cooperative_groups.h>
 
 #include <algorithm>
@@ -42,10 +46,22 @@ struct Bf16GemmParams {
   float* out;
   __nv_bfloat16* out_bf16;
   size_t out_stride;
-  int N, K, M, nkb, rtiles, tiles, ksplit, epi;
+  int N, K, M, nkb, rtiles, tiles, ksplit, epi;   // N: of one expert
   pi_dyt_residual res;
   pi_maps_kv mkv;
+  const float* out_scale;
+  float glu_limit;
+  int glu_rows;
+  float* rest;
+  size_t rest_stride;
+  const int4* table;              // GROUPED
+  const int32_t* n_table;
   int* err_flag;
+};
+
+// A column tile: which expert, its activation rows [m0, m_end).
+struct TileAt {
+  int expert, m0, m_end;
 };
 
 __device__ __forceinline__ void umma_f16_ss(uint32_t tmem_d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
@@ -62,20 +78,20 @@ __device__ __forceinline__ void tma_2d(uint32_t dst, const CUtensorMap* map, uin
       : "memory");
 }
 
-// C columns (activation rows m, m + dm, ...) of output column n, all lanes of the warp on adjacent n.  `place`: of row m, if
+// C columns (activation rows m, m + dm, ... < M) of output column n, all lanes of the warp on adjacent n.  `place`: of row m, if
 // it has been looked up already.
 template <int C>
-__device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int n, int m, int dm, const float* v, const pi_kv_place* place = nullptr) {
+__device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int M, int n, int m, int dm, const float* v, const pi_kv_place* place = nullptr) {
   const bool ok = n < p.N;
   if (p.epi == PI_EPI_DYT_RESIDUAL) {
     float old[C];
 #pragma unroll
-    for (int j = 0; j < C; ++j) old[j] = (ok && m + j * dm < p.M) ? p.res.x[(size_t)(m + j * dm) * p.res.x_stride + n] : 0.f;
+    for (int j = 0; j < C; ++j) old[j] = (ok && m + j * dm < M) ? p.res.x[(size_t)(m + j * dm) * p.res.x_stride + n] : 0.f;
     const float wp = ok ? __ldg(p.res.post.w + n) : 0.f, bp = ok ? __ldg(p.res.post.b + n) : 0.f;
     const float wn = ok ? __ldg(p.res.next.w + n) : 0.f, bn = ok ? __ldg(p.res.next.b + n) : 0.f;
 #pragma unroll
     for (int j = 0; j < C; ++j) {
-      if (!ok || m + j * dm >= p.M) continue;
+      if (!ok || m + j * dm >= M) continue;
       const float x = old[j] + fmaf(tanhf(p.res.post.alpha * v[j]), wp, bp);
       p.res.x[(size_t)(m + j * dm) * p.res.x_stride + n] = x;
       static_cast<__nv_bfloat16*>(p.res.h)[(size_t)(m + j * dm) * p.res.h_stride + n] =
@@ -89,7 +105,7 @@ __device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int n, int m, 
     pi_kv_place mine = {0, -1, 0};
     const int my_row = m + (C == 1 ? 0 : (lane % C) * dm);
     if (place) mine = *place;
-    else if (my_row < p.M) mine = pi_maps_kv_place(k, my_row);
+    else if (my_row < M) mine = pi_maps_kv_place(k, my_row);
     const int half = k.rot_dims >> 1, pair = col.rotated ? col.d >> 1 : 0;
     float cs[C], sn[C];
     if (half > 0) {
@@ -106,33 +122,51 @@ __device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int n, int m, 
       const int block = __shfl_sync(0xffffffffu, mine.block, j), off = __shfl_sync(0xffffffffu, mine.off, j);
       float r = v[j];
       if (col.rotated) r = (n & 1) ? v[j] * cs[j] + other * sn[j] : v[j] * cs[j] - other * sn[j];
-      if (!ok || m + j * dm >= p.M) continue;
+      if (!ok || m + j * dm >= M) continue;
       if (col.is_q) p.out[(size_t)(m + j * dm) * p.out_stride + n] = r;
       else pi_maps_kv_store(k, col, block, off, r);
     }
-  } else if (p.epi == PI_EPI_GEGLU) {
+  } else if (p.epi == PI_EPI_GEGLU || p.epi == PI_EPI_SWIGLU || p.epi == PI_EPI_CLAMP_GLU) {
     // even n: gate rows, odd n: up rows; of two columns m the even lane finishes the first, the odd lane the second
     const int odd = n & 1;
+    const bool pair = n < p.glu_rows;
     if (C == 1) {
       const float other = __shfl_xor_sync(0xffffffffu, v[0], 1);
-      if (!odd && n + 1 < p.N && m < p.M) p.out_bf16[(size_t)m * p.out_stride + (n >> 1)] = __float2bfloat16_rn(pi_gelu_tanh(v[0]) * other);
+      if (pair && !odd && m < M) p.out_bf16[(size_t)m * p.out_stride + (n >> 1)] = __float2bfloat16_rn(pi_glu(p.epi, v[0], other, p.glu_limit));
     } else {
 #pragma unroll
       for (int j = 0; j + 1 < C; j += 2) {
         const float other = __shfl_xor_sync(0xffffffffu, odd ? v[j] : v[j + 1], 1);
         const float g = odd ? other : v[j], u = odd ? v[j + 1] : other;
         const int mm = m + (j + odd) * dm;
-        if ((n | 1) < p.N && mm < p.M) p.out_bf16[(size_t)mm * p.out_stride + (n >> 1)] = __float2bfloat16_rn(pi_gelu_tanh(g) * u);
+        if (pair && mm < M) p.out_bf16[(size_t)mm * p.out_stride + (n >> 1)] = __float2bfloat16_rn(pi_glu(p.epi, g, u, p.glu_limit));
       }
     }
+    if (ok && !pair) {
+#pragma unroll
+      for (int j = 0; j < C; ++j)
+        if (m + j * dm < M) p.rest[(size_t)(m + j * dm) * p.rest_stride + (n - p.glu_rows)] = v[j];
+    }
+  } else if (p.epi == PI_EPI_SCALE_ADD) {
+    float old[C];
+#pragma unroll
+    for (int j = 0; j < C; ++j) old[j] = (ok && m + j * dm < M) ? p.out[(size_t)(m + j * dm) * p.out_stride + n] : 0.f;
+    const float w = ok ? __ldg(p.out_scale + n) : 0.f;
+#pragma unroll
+    for (int j = 0; j < C; ++j)
+      if (ok && m + j * dm < M) p.out[(size_t)(m + j * dm) * p.out_stride + n] = fmaf(w, v[j], old[j]);
+  } else if (p.out_bf16) {
+#pragma unroll
+    for (int j = 0; j < C; ++j)
+      if (ok && m + j * dm < M) p.out_bf16[(size_t)(m + j * dm) * p.out_stride + n] = __float2bfloat16_rn(v[j]);
   } else {
 #pragma unroll
     for (int j = 0; j < C; ++j)
-      if (ok && m + j * dm < p.M) p.out[(size_t)(m + j * dm) * p.out_stride + n] = v[j];
+      if (ok && m + j * dm < M) p.out[(size_t)(m + j * dm) * p.out_stride + n] = v[j];
   }
 }
 
-template <int BN, int STAGES, bool SPLIT>
+template <int BN, int STAGES, bool SPLIT, bool GROUPED = false>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x) {
   constexpr int kABytes = kTM * kTK * 2, kBBytes = BN * kTK * 2, kStageBytes = kABytes + kBBytes;
@@ -153,7 +187,19 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
   const int tile0 = SPLIT ? (int)blockIdx.x / p.ksplit : (int)blockIdx.x, tile_step = SPLIT ? p.tiles : (int)gridDim.x;
   const int kb0 = SPLIT ? (int)((long)rank * p.nkb / p.ksplit) : 0, kb1 = SPLIT ? (int)((long)(rank + 1) * p.nkb / p.ksplit) : p.nkb;
   const int nk = kb1 - kb0;
-  const int my_tiles = tile0 < p.tiles ? (p.tiles - tile0 + tile_step - 1) / tile_step : 0;
+  static_assert(!(SPLIT && GROUPED), "the table's length is not known when the launch is cut");
+  auto count = [&](int tiles) { return tile0 < tiles ? (tiles - tile0 + tile_step - 1) / tile_step : 0; };
+  int my_tiles = GROUPED ? 0 : count(p.tiles);   // GROUPED: every role reads it behind its own wait
+  auto tile_at = [&](int tile) {
+    TileAt t = {0, (tile / p.rtiles) * BN, p.M};
+    if (GROUPED) {
+      const int4 e = p.table[tile / p.rtiles];
+      t.expert = e.x;
+      t.m0 = e.y;
+      t.m_end = e.y + e.z;
+    }
+    return t;
+  };
 
   if (tid == 0) {
     for (int s = 0; s < STAGES; ++s) {
@@ -187,19 +233,24 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
   if (warp == kEpiWarps) {
     // ---- TMA ------------------------------------------------------------------------------------------------------
     if (lane == 0) {
+      if (GROUPED) {
+        pi_grid_dependency_wait();
+        s_dep_ok = 1;
+        my_tiles = count(*p.n_table * p.rtiles);
+      }
       const int total = my_tiles * nk;
       auto load_w = [&](int it) {
         const int tile = tile0 + (it / nk) * tile_step, kb = kb0 + it % nk, s = it % STAGES;
         mbar_arrive_expect_tx(full0 + 8 * s, kStageBytes);
-        tma_2d(base + s * kStageBytes, &map_w, full0 + 8 * s, kb * kTK, (tile % p.rtiles) * kTM);
+        tma_2d(base + s * kStageBytes, &map_w, full0 + 8 * s, kb * kTK, (GROUPED ? tile_at(tile).expert * p.N : 0) + (tile % p.rtiles) * kTM);
       };
       auto load_x = [&](int it) {
         const int tile = tile0 + (it / nk) * tile_step, kb = kb0 + it % nk, s = it % STAGES;
-        tma_2d(base + s * kStageBytes + kABytes, &map_x, full0 + 8 * s, kb * kTK, (tile / p.rtiles) * BN);
+        tma_2d(base + s * kStageBytes + kABytes, &map_x, full0 + 8 * s, kb * kTK, tile_at(tile).m0);
       };
       const int ahead = min(total, STAGES);
       for (int it = 0; it < ahead; ++it) load_w(it);   // weights never depend on the preceding kernel
-      pi_grid_dependency_wait();
+      if (!GROUPED) pi_grid_dependency_wait();
       s_dep_ok = 1;
       for (int it = 0; it < ahead; ++it) load_x(it);
       int issued = ahead;
@@ -217,6 +268,10 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
   } else if (warp == kEpiWarps + 1) {
     // ---- MMA ------------------------------------------------------------------------------------------------------
     if (lane == 0) {
+      if (GROUPED) {
+        pi_grid_dependency_wait();
+        my_tiles = count(*p.n_table * p.rtiles);
+      }
       const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(kTM >> 4) << 24);
       int it = 0;
       bool ok = true;
@@ -252,6 +307,7 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
       for (int c = tid; c < BN && (tile0 / p.rtiles) * BN + c < p.M; c += kEpiWarps * 32)
         s_place[c] = pi_maps_kv_place(p.mkv, (tile0 / p.rtiles) * BN + c);
     pi_grid_dependency_wait();   // the epilogue reads and writes what the preceding kernels use
+    if (GROUPED) my_tiles = count(*p.n_table * p.rtiles);
     for (int t = 0; t < my_tiles; ++t) {
       const int a = t % kAcc, tile = tile0 + t * tile_step;
       int got = 0;
@@ -262,11 +318,12 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
       got = __shfl_sync(0xffffffffu, got, 0);
       if (!got) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const int n = (tile % p.rtiles) * kTM + quad * 32 + lane, m0 = (tile / p.rtiles) * BN;
+      const TileAt at = tile_at(tile);
+      const int n = (tile % p.rtiles) * kTM + quad * 32 + lane, m0 = at.m0;
       if (BN >= 32 || half == 0) {
 #pragma unroll 1
         for (int c = half * kHalfCols; c < half * kHalfCols + kHalfCols; c += 16) {
-          if (!SPLIT && m0 + c >= p.M) break;
+          if (!SPLIT && m0 + c >= at.m_end) break;
           uint32_t r[16];
           tmem_ld16_issue(tmem + ((uint32_t)(quad * 32) << 16) + (uint32_t)(a * BN + c), r);
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -278,7 +335,7 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
 #pragma unroll
             for (int j = 0; j < 16; ++j) part[(c + j) * kTM + quad * 32 + lane] = v[j];
           } else {
-            epilogue<16>(p, n, m0 + c, 1, v);
+            epilogue<16>(p, at.m_end, n, m0 + c, 1, v);
           }
         }
       }
@@ -302,7 +359,7 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
         float v = 0.f;
 #pragma unroll
         for (int r = 0; r < 8; ++r) v += s[r];
-        epilogue<1>(p, n, m0 + c, 1, &v, &s_place[c]);
+        epilogue<1>(p, p.M, n, m0 + c, 1, &v, &s_place[c]);
       }
     }
     __syncwarp();
@@ -321,9 +378,9 @@ constexpr size_t gemm_smem() {
   return std::max((size_t)STAGES * (kTM + BN) * kTK * 2 + (SPLIT ? (size_t)BN * kTM * 4 : 0) + 1024, kMinSmemBytes);
 }
 
-template <int BN, int STAGES, bool SPLIT>
+template <int BN, int STAGES, bool SPLIT, bool GROUPED = false>
 cudaError_t launch(pi_ctx* ctx, const Bf16GemmParams& p, const CUtensorMap& w, const CUtensorMap& x, int ctas) {
-  auto k = gemm_bf16_kernel<BN, STAGES, SPLIT>;
+  auto k = gemm_bf16_kernel<BN, STAGES, SPLIT, GROUPED>;
   constexpr size_t smem = gemm_smem<BN, STAGES, SPLIT>();
   static pi_smem_grant granted;
   if (smem > granted.of(ctx)) {
@@ -375,6 +432,11 @@ cudaError_t run(pi_ctx* ctx, Bf16GemmParams& p, const CUtensorMap& w, const CUte
   p.ksplit = 1;
   return launch<BN, STAGES, false>(ctx, p, w, x, std::min(p.tiles, ctx->sm_count));
 }
+template <int BN, int STAGES>
+cudaError_t run_grouped(pi_ctx* ctx, Bf16GemmParams& p, const CUtensorMap& w, const CUtensorMap& x) {
+  p.ksplit = 1;
+  return launch<BN, STAGES, false, true>(ctx, p, w, x, std::min(p.tiles, ctx->sm_count));
+}
 
 pi_status encode_2d(pi_ctx* ctx, CUtensorMap* map, const void* base, size_t cols, size_t rows, size_t ld, int box_rows) {
   const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
@@ -395,14 +457,24 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
   PI_REQUIRE(ctx, lin->kind == PI_BF16 && a.x_bf16 && a.M >= 1, "the bf16 GEMM takes bf16 weights and activations");
   PI_REQUIRE(ctx, (uintptr_t)a.x_bf16 % 16 == 0 && a.x_stride % 8 == 0 && (uintptr_t)lin->w % 16 == 0 && lin->ld % 8 == 0,
              "bf16 operands must start and step on 16-byte boundaries");
-  PI_REQUIRE(ctx, a.epi == PI_EPI_STORE || (a.epi == PI_EPI_MAPS_QKV && a.maps_kv && a.maps_kv->dim % 2 == 0) || (a.epi == PI_EPI_GEGLU && a.out_bf16 && lin->rows % 2 == 0) ||
+  const pi_expert_rows* ex = a.experts;
+  PI_REQUIRE(ctx, !ex || (ex->experts > 0 && lin->rows % ex->experts == 0 && ex->tiles && ex->n_tiles && ex->max_tiles > 0), "a stack of experts needs its tile table");
+  const int N = (int)(ex ? lin->rows / ex->experts : lin->rows);
+  const bool glu = pi_epi_glu(a.epi) && a.out_bf16 && (a.glu_rows ? a.glu_rows % 2 == 0 && a.glu_rows <= N && a.rest : N % 2 == 0);
+  PI_REQUIRE(ctx, a.epi == PI_EPI_STORE || glu || (a.epi == PI_EPI_MAPS_QKV && a.maps_kv && a.maps_kv->dim % 2 == 0) ||
+                      (a.epi == PI_EPI_SCALE_ADD && a.out && a.out_scale) ||
                       (a.epi == PI_EPI_DYT_RESIDUAL && a.residual && a.residual->x && a.residual->h && a.residual->post.w && a.residual->next.w),
              "this epilogue is not built for the bf16 GEMM");
   Bf16GemmParams p = {};
   p.out = a.out;
   p.out_bf16 = a.out_bf16;
   p.out_stride = a.out_stride;
-  p.N = (int)lin->rows;
+  p.out_scale = a.out_scale;
+  p.glu_limit = a.glu_limit;
+  p.glu_rows = a.glu_rows ? a.glu_rows : N;
+  p.rest = a.rest;
+  p.rest_stride = a.rest_stride;
+  p.N = N;
   p.K = (int)lin->cols;
   p.M = a.M;
   p.nkb = (p.K + kTK - 1) / kTK;
@@ -416,13 +488,26 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
     const long t128 = (long)p.rtiles * ((a.M + 127) / 128), t256 = (long)p.rtiles * ((a.M + 255) / 256), sms = ctx->sm_count;
     if ((t256 + sms - 1) / sms * 2 <= (t128 + sms - 1) / sms) bn = 256;
   }
-  p.tiles = p.rtiles * ((a.M + bn - 1) / bn);
+  if (ex) {
+    bn = ex->tile_rows;
+    p.table = ex->tiles;
+    p.n_table = ex->n_tiles;
+  }
+  p.tiles = p.rtiles * (ex ? ex->max_tiles : (a.M + bn - 1) / bn);
   CUtensorMap w, x;
   PI_TRY(encode_2d(ctx, &w, lin->w, lin->cols, lin->rows, lin->ld, kTM));
   PI_TRY(encode_2d(ctx, &x, a.x_bf16, lin->cols, a.M, a.x_stride, bn));
   pi_prof_scope prof(ctx, PI_PROF_GEMM_TC);
   cudaError_t e;
-  switch (bn) {
+  if (ex) {
+    switch (bn) {
+      case 16: e = run_grouped<16, 8>(ctx, p, w, x); break;
+      case 32: e = run_grouped<32, 8>(ctx, p, w, x); break;
+      case 64: e = run_grouped<64, 6>(ctx, p, w, x); break;
+      case 128: e = run_grouped<128, 4>(ctx, p, w, x); break;
+      default: return pi_fail(ctx, PI_ERR_INVALID_ARG, "expert tiles of %d rows are not built", bn);
+    }
+  } else switch (bn) {
     case 16: e = run<16, 8>(ctx, p, w, x); break;
     case 32: e = run<32, 8>(ctx, p, w, x); break;
     case 64: e = run<64, 6>(ctx, p, w, x); break;

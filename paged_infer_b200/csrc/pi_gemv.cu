@@ -84,6 +84,13 @@ struct Widen<float> {
 struct GemvParams {
   pi_dyt_residual res;   // PI_EPI_DYT_RESIDUAL
   pi_maps_kv mkv;        // PI_EPI_MAPS_QKV
+  const float* out_scale;   // PI_EPI_SCALE_ADD
+  float glu_limit;          // PI_EPI_CLAMP_GLU
+  int glu_rows;             // gated epilogues: rows behind go to `rest`
+  float* rest;
+  size_t rest_stride;
+  const int32_t* expert;    // GROUPED
+  int x_div;
   const void* W;
   const float* scales;
   const float* x;
@@ -129,7 +136,8 @@ __device__ __forceinline__ int unit_swizzle(int group) {
 
 // KS > 1 (matrices with few, long rows): KS consecutive warps share a row pair, warp ks of them takes the K groups
 // ks, ks + KS, ...; the partial sums meet in shared memory and are added in warp order by the first warp of the set.
-template <typename WT, int MB, int EPI, bool NORM, bool ROPE, int KS = 1>
+// GROUPED (MB == 1): the weights are a stack of experts, the row's own one is known only behind the dependency wait.
+template <typename WT, int MB, int EPI, bool NORM, bool ROPE, int KS = 1, bool GROUPED = false>
 __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
   constexpr int EPL = Widen<WT>::EPL;
   constexpr int U = EPL / 4;
@@ -148,6 +156,12 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
   const int ngroups = (ld + kGroupElems - 1) / kGroupElems;
   const int total_warps = gridDim.x * nwarps;
   const int k_lane = lane * EPL;
+  const unsigned char* W = reinterpret_cast<const unsigned char*>(p.W);
+  if (GROUPED) {
+    pi_grid_dependency_wait();
+    W += (size_t)p.expert[m0] * p.N * ld * sizeof(WT);
+  }
+  const float* xrow = p.x + (size_t)(GROUPED ? m0 / p.x_div : m0) * p.x_stride;
 
   // Work items of this warp: (row pair, K group), row pairs strided by the number of warps in the grid.
   int4 wcur[kSteps][kRows], wnxt[kSteps][kRows];
@@ -155,7 +169,7 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
     const unsigned char* rowp[kRows];
 #pragma unroll
     for (int r = 0; r < kRows; ++r)
-      rowp[r] = reinterpret_cast<const unsigned char*>(p.W) + (size_t)min(gemv_row<ROPE>(p, pair, r), p.N - 1) * ld * sizeof(WT);
+      rowp[r] = W + (size_t)min(gemv_row<ROPE>(p, pair, r), p.N - 1) * ld * sizeof(WT);
 #pragma unroll
     for (int t = 0; t < kSteps; ++t) {
       const int k = kg * kGroupElems + t * kStepElems + k_lane;
@@ -181,7 +195,7 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
                                                               : make_float4(0.f, 0.f, 0.f, 0.f);
   }
 
-  pi_grid_dependency_wait();
+  if (!GROUPED) pi_grid_dependency_wait();
 
   // fused [q;k;v] projection: lane m finishes activation row m0+m; its position and the physical block that takes its
   // K and V are looked up now, off the path between the dot products and the stores
@@ -210,7 +224,7 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
         asm volatile(
             "cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
                 smem_u32(xs + (size_t)m * ld)),
-            "l"(p.x + (size_t)(m0 + m) * p.x_stride), "r"((uint32_t)(K * sizeof(float))), "r"(bar)
+            "l"(xrow + (size_t)m * p.x_stride), "r"((uint32_t)(K * sizeof(float))), "r"(bar)
             : "memory");
       }
     }
@@ -234,7 +248,7 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
   }
   if (!landed) {
     for (int m = 0; m < MB; ++m) {
-      const float* src = p.x + (size_t)(m0 + m) * p.x_stride;
+      const float* src = xrow + (size_t)m * p.x_stride;
       for (int k = tid; k < ld; k += blockDim.x) xs[(size_t)m * ld + k] = (m < mcount && k < K) ? src[k] : 0.f;
     }
     __syncthreads();
@@ -321,10 +335,11 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
     if (npair < npairs) load_group(wnxt, npair, nkg);
     // residual add: the value this lane will add to is requested before the arithmetic of the pair's last group
     float old_out = 0.f;
-    if ((EPI == PI_EPI_ADD || EPI == PI_EPI_DYT_RESIDUAL) && !ROPE && ks == 0 && kg + KS >= ngroups) {
+    constexpr bool kAdds = EPI == PI_EPI_ADD || EPI == PI_EPI_SCALE_ADD;
+    if ((kAdds || EPI == PI_EPI_DYT_RESIDUAL) && !ROPE && ks == 0 && kg + KS >= ngroups) {
       const int r = lane / MB, m = lane - r * MB;
       if (r < kRows && m < mcount && pair * kRows + r < p.N)
-        old_out = EPI == PI_EPI_ADD ? p.out[(size_t)(m0 + m) * p.out_stride + pair * kRows + r]
+        old_out = kAdds ? p.out[(size_t)(m0 + m) * p.out_stride + pair * kRows + r]
                                     : p.res.x[(size_t)(m0 + m) * p.res.x_stride + pair * kRows + r];
     }
     float sc[kRows] = {1.0f, 1.0f};   // the rows' scales, requested likewise
@@ -437,14 +452,20 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
             }
           }
         }
-      } else if (EPI == PI_EPI_SWIGLU || EPI == PI_EPI_GEGLU) {
+      } else if (EPI == PI_EPI_SWIGLU || EPI == PI_EPI_GEGLU || EPI == PI_EPI_CLAMP_GLU) {
 #pragma unroll
         for (int m = 0; m < MB; ++m) {
-          if (lane == m && m < mcount && row0 + 1 < p.N) {
+          if (lane == m && m < mcount) {
             const float rf = row_factor(m);
             const float g = tot[0][m] * sc[0] * rf, u = tot[1][m] * sc[1] * rf;
-            p.out[(size_t)(m0 + m) * p.out_stride + (row0 >> 1)] =
-                EPI == PI_EPI_GEGLU ? pi_gelu_tanh(g) * u : (g / (1.0f + expf(-g))) * u;
+            if (row0 < p.glu_rows) {
+              p.out[(size_t)(m0 + m) * p.out_stride + (row0 >> 1)] =
+                  EPI == PI_EPI_SWIGLU ? (g / (1.0f + expf(-g))) * u : pi_glu(EPI, g, u, p.glu_limit);
+            } else {
+              float* o = p.rest + (size_t)(m0 + m) * p.rest_stride + (row0 - p.glu_rows);
+              o[0] = g;
+              if (row0 + 1 < p.N) o[1] = u;
+            }
           }
         }
       } else if (EPI == PI_EPI_MAPS_QKV) {
@@ -491,7 +512,7 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
             if (lane == r * MB + m && m < mcount && row0 + r < p.N) {
               float* o = p.out + (size_t)(m0 + m) * p.out_stride + row0 + r;
               const float v = tot[r][m] * sc[r] * row_factor(m);
-              *o = (EPI == PI_EPI_ADD) ? (old_out + v) : v;
+              *o = EPI == PI_EPI_ADD ? old_out + v : EPI == PI_EPI_SCALE_ADD ? fmaf(__ldg(p.out_scale + row0 + r), v, old_out) : v;
             }
           }
       }
@@ -512,10 +533,18 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
   void (*k)(const GemvParams) = nullptr;
   constexpr bool kFloatW = !std::is_same<WT, int8_t>::value;   // layered designs keep bf16 weights
 #define PI_PICK(E, Nrm) k = gemv_kernel<WT, MB, E, Nrm, false>
-  if (ksplit == kSplitWarps) {   // few long rows (pi_launch_gemv asks for it only without norm, rotary embedding, SwiGLU)
+  if (p.expert) {
+    if constexpr (kFloatW && MB == 1) {
+      if (epi == PI_EPI_CLAMP_GLU) k = gemv_kernel<WT, 1, PI_EPI_CLAMP_GLU, false, false, 1, true>;
+      else if (epi == PI_EPI_SWIGLU) k = gemv_kernel<WT, 1, PI_EPI_SWIGLU, false, false, 1, true>;
+      else if (epi == PI_EPI_STORE) k = gemv_kernel<WT, 1, PI_EPI_STORE, false, false, 1, true>;
+    }
+  } else if (ksplit == kSplitWarps) {   // few long rows (pi_launch_gemv asks for it only without norm, rotary embedding, SwiGLU)
     if (epi == PI_EPI_ADD) k = gemv_kernel<WT, MB, PI_EPI_ADD, false, false, kSplitWarps>;
     else if (epi == PI_EPI_DYT_RESIDUAL) {
       if constexpr (kFloatW) k = gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false, kSplitWarps>;
+    } else if (epi == PI_EPI_SCALE_ADD) {
+      if constexpr (kFloatW) k = gemv_kernel<WT, MB, PI_EPI_SCALE_ADD, false, false, kSplitWarps>;
     } else k = gemv_kernel<WT, MB, PI_EPI_STORE, false, false, kSplitWarps>;
   } else if (epi == PI_EPI_STORE && p.rope_hd) {   // fused [q;k;v] projection: own instantiation, the others stay as they are
     if (norm) k = gemv_kernel<WT, MB, PI_EPI_STORE, true, true>; else k = gemv_kernel<WT, MB, PI_EPI_STORE, false, true>;
@@ -529,6 +558,10 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
     if constexpr (kFloatW) PI_PICK(PI_EPI_MAPS_QKV, false);
   } else if (epi == PI_EPI_DYT_RESIDUAL) {
     if constexpr (kFloatW) PI_PICK(PI_EPI_DYT_RESIDUAL, false);
+  } else if (epi == PI_EPI_SCALE_ADD) {
+    if constexpr (kFloatW) PI_PICK(PI_EPI_SCALE_ADD, false);
+  } else if (epi == PI_EPI_CLAMP_GLU) {
+    if constexpr (kFloatW) PI_PICK(PI_EPI_CLAMP_GLU, false);
   } else {
     if (norm) PI_PICK(PI_EPI_SWIGLU, true); else PI_PICK(PI_EPI_SWIGLU, false);
   }
@@ -548,10 +581,19 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
     }
     if constexpr (kFloatW) {
       for (auto kk : {gemv_kernel<WT, MB, PI_EPI_GEGLU, false, false>, gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false>,
-                      gemv_kernel<WT, MB, PI_EPI_MAPS_QKV, false, false>,
-                      gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false, kSplitWarps>}) {
+                      gemv_kernel<WT, MB, PI_EPI_MAPS_QKV, false, false>, gemv_kernel<WT, MB, PI_EPI_SCALE_ADD, false, false>,
+                      gemv_kernel<WT, MB, PI_EPI_CLAMP_GLU, false, false>,
+                      gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false, kSplitWarps>,
+                      gemv_kernel<WT, MB, PI_EPI_SCALE_ADD, false, false, kSplitWarps>}) {
         cudaError_t e = cudaFuncSetAttribute(kk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
+      }
+      if constexpr (MB == 1) {
+        for (auto kk : {gemv_kernel<WT, 1, PI_EPI_CLAMP_GLU, false, false, 1, true>, gemv_kernel<WT, 1, PI_EPI_SWIGLU, false, false, 1, true>,
+                        gemv_kernel<WT, 1, PI_EPI_STORE, false, false, 1, true>}) {
+          cudaError_t e = cudaFuncSetAttribute(kk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+          if (e != cudaSuccess) return e;
+        }
       }
     }
     granted.of(ctx) = smem;
@@ -634,20 +676,25 @@ bool pi_gemv_can_rope(const pi_ctx* ctx, const pi_linear* lin, const pi_linear_a
 
 pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args& a) {
   PI_REQUIRE(ctx, a.M >= 1, "projection batch must be at least 1");
-  const bool glu = a.epi == PI_EPI_SWIGLU || a.epi == PI_EPI_GEGLU;
-  PI_REQUIRE(ctx, !glu || lin->rows % 2 == 0, "a gated epilogue needs interleaved gate/up rows");
+  const bool glu = pi_epi_glu(a.epi);
+  const size_t n_rows = a.experts ? lin->rows / a.experts->experts : lin->rows;   // of the matrix one row of the batch meets
+  PI_REQUIRE(ctx, !glu || (a.glu_rows ? a.glu_rows % 2 == 0 && a.rest && (size_t)a.glu_rows <= n_rows : n_rows % 2 == 0),
+             "a gated epilogue needs interleaved gate/up rows");
+  PI_REQUIRE(ctx, !a.experts || (lin->kind != PI_INT8 && a.experts->expert && lin->rows % a.experts->experts == 0 && a.experts->x_div >= 1),
+             "a stack of experts needs float weights and the rows' experts");
+  PI_REQUIRE(ctx, a.epi != PI_EPI_SCALE_ADD || a.out_scale, "a scaled residual add needs its scale");
   PI_REQUIRE(ctx, a.epi < PI_EPI_GEGLU || (lin->kind != PI_INT8 && !a.norm_weight), "this epilogue is built for bf16 and f32 weights");
   PI_REQUIRE(ctx, a.epi != PI_EPI_MAPS_QKV || (a.maps_kv && a.maps_kv->dim % 2 == 0), "the fused [q;k;v] epilogue needs its operands and an even dim");
   PI_REQUIRE(ctx, a.epi != PI_EPI_DYT_RESIDUAL || (a.residual && a.residual->x), "the residual epilogue needs its operands");
   if (lin->rows == 0) return PI_OK;
-  int mb = a.M >= 4 ? 4 : a.M >= 2 ? 2 : 1;
+  int mb = a.experts ? 1 : a.M >= 4 ? 4 : a.M >= 2 ? 2 : 1;
   while (mb > 1 && (size_t)mb * lin->ld * sizeof(float) > ctx->smem_optin - 2048) mb >>= 1;
   const size_t smem = (size_t)mb * lin->ld * sizeof(float);
   PI_REQUIRE(ctx, smem <= ctx->smem_optin - 2048, "projection input of %zu columns does not fit shared memory", lin->cols);
 
   // Persistent grid: two CTAs of up to 8 warps per SM; narrower CTAs when there are few row pairs, so that
   // every SM still gets work.
-  const size_t npairs = (lin->rows + kRows - 1) / kRows;
+  const size_t npairs = (n_rows + kRows - 1) / kRows;
   const int mtiles = (a.M + mb - 1) / mb;
   const size_t max_ctas = std::max<size_t>(1, (size_t)ctx->sm_count * 2 / mtiles);
   int warps = 8;
@@ -658,7 +705,7 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
   // Sets of three warps share a row pair instead: three times the loads in flight.
   int ksplit = 1;
   const size_t row_bytes = lin->ld * (lin->kind == PI_INT8 ? 1 : lin->kind == PI_BF16 ? 2 : 4);
-  if (!a.norm_weight && !a.rope && !glu && a.epi != PI_EPI_MAPS_QKV && row_bytes > (size_t)(kSplitWarps - 1) * kSteps * 512 &&
+  if (!a.norm_weight && !a.rope && !glu && !a.experts && a.epi != PI_EPI_MAPS_QKV && row_bytes > (size_t)(kSplitWarps - 1) * kSteps * 512 &&
       npairs * 2 <= max_ctas * 8) {
     ksplit = kSplitWarps;
     warps = 2 * kSplitWarps;
@@ -675,7 +722,14 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
   p.ld = lin->ld;
   p.x_stride = a.x_stride;
   p.out_stride = a.out_stride;
-  p.N = (int)lin->rows;
+  p.out_scale = a.out_scale;
+  p.glu_limit = a.glu_limit;
+  p.glu_rows = a.glu_rows ? a.glu_rows : (int)n_rows;
+  p.rest = a.rest;
+  p.rest_stride = a.rest_stride;
+  p.expert = a.experts ? a.experts->expert : nullptr;
+  p.x_div = a.experts ? a.experts->x_div : 1;
+  p.N = (int)n_rows;
   p.K = (int)lin->cols;
   p.M = a.M;
   p.eps = a.norm_eps;

@@ -1,10 +1,12 @@
-// Layered designs: a decoder whose layers each name a token mixer - windowed attention with one or two softmax maps, a
-// gated linear recurrence (GLA), a matrix memory (mLSTM) - and, if they have one, a gelu-gated feed-forward; every
-// sublayer normalised before and after by Dynamic Tanh, embedding tied to the output.
+// Layered designs: a decoder whose layers each name a token mixer - windowed attention with one or two softmax maps, latent
+// attention, a gated linear recurrence (GLA), a matrix memory (mLSTM), a state-space recurrence (SSD) - and, if they have one,
+// a feed-forward: dense and gated, or routed experts.  Two ways of normalising:
 //
-//   x += dyt(norm1b, mixer(dyt(norm1, x)));   x += dyt(norm2b, ff(dyt(norm2, x)))
+//   Dynamic Tanh   x += dyt(norm1b, mixer(dyt(norm1, x)));   x += dyt(norm2b, ff(dyt(norm2, x)))
+//   layer norm     x += ls1 mixer(ln(norm1, x));             x += ls2 ff(ln(norm2, x))
 //
-// Dynamic Tanh needs no statistics, so all of it folds into the projection that ends a sublayer: its epilogue adds
+// Layer norm needs the whole row: the projection that ends a sublayer adds its scaled result to the residual stream, and a
+// row kernel writes the next sublayer's input (behind experts it also adds up their outputs).  Dynamic Tanh needs no statistics, so all of it folds into the projection that ends a sublayer: its epilogue adds
 // the normalised result to the f32 residual stream and hands on the normalised input of the next sublayer.  Per layer:
 //   1. [q;k;v(;gates)] projection; attention: rotary positions and the KV write in its epilogue
 //   2. attention (with its own normalisation in the same kernel); or the recurrence with head norm and output gate in the
@@ -41,18 +43,42 @@ namespace {
 struct Layer {
   pi_layer_config c;
   pi_dyt norm1, norm1b, norm2, norm2b;
+  pi_layer_norm ln1, ln2;
+  const float *ls1 = nullptr, *ls2 = nullptr;
+  // routed experts: gate_up holds [shared gate/up | router | shared gate of the token], down the shared expert's
   pi_linear *in = nullptr, *out = nullptr, *gate_up = nullptr, *down = nullptr;
+  pi_linear *expert_in = nullptr, *expert_out = nullptr;   // stacks of all experts
+  pi_linear *ukv = nullptr, *uk_t = nullptr;               // latent attention
   int attn = -1;                 // index of the layer's KV region
   int rope = -1;                 // index of its rotary table
   float lambda = 0.f;
   pi_recurrence rec;
+  pi_latent_attention lat;
+  pi_ssd ssd;
+  pi_moe moe;
 };
 
 struct RopeTable {
   int dims = 0, cap = 0;
-  float base = 1.f;
+  double base = 1., factor = 1., original = 1., fast = 1., slow = 1.;
   float *cos = nullptr, *sin = nullptr;
 };
+
+// Angle per position of every pair, and the factor of cos and sin.  With a factor above 1, pairs that turn less than `slow`
+// times within `original` positions are slowed by it, pairs that turn more than `fast` times are left alone, with a linear
+// ramp over the pair index in between.
+double rope_frequencies(const RopeTable& t, std::vector<double>* f) {
+  f->resize(t.dims / 2);
+  const bool stretched = t.factor != 1.0;
+  auto turns = [&](double n) { return t.dims * log(t.original / (2.0 * M_PI * n)) / (2.0 * log(t.base)); };
+  const double lo = stretched ? std::max(floor(turns(t.fast)), 0.0) : 0.0, hi = stretched ? std::min(ceil(turns(t.slow)), t.dims - 1.0) : 0.0;
+  for (int i = 0; i < t.dims / 2; ++i) {
+    const double plain = pow(t.base, -2.0 * i / t.dims);
+    const double ramp = stretched ? std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0) : 0.0;
+    (*f)[i] = plain / t.factor * ramp + plain * (1.0 - ramp);
+  }
+  return stretched ? 0.1 * log(t.factor) + 1.0 : 1.0;
+}
 
 }  // namespace
 
@@ -61,14 +87,25 @@ struct pi_layered {
   std::vector<Layer> layers;
   std::vector<RopeTable> ropes;
   std::vector<void*> owned;      // device vectors
-  pi_linear* embed = nullptr;
+  pi_linear *embed = nullptr, *head = nullptr;   // head: null if tied
   pi_dyt final_norm;
+  pi_layer_norm final_ln;        // its weight carries the logits' scale
   size_t weight_bytes = 0, state_floats = 0;
   bool chunked = false;          // every recurrent layer has a chunked kernel
+  bool latent = false, expand = false;   // latent attention; its long portions are expanded
+  int latent_window = 0;         // the widest (<= 0: everything before)
   // scratch for c.max_rows rows; activations are sized for f32 and hold bf16 on the tensor path
   float *x = nullptr, *proj = nullptr;
   void *h = nullptr, *core = nullptr, *ffh = nullptr;
   size_t ld_h = 0, ld_core = 0, ld_ff = 0, ld_proj = 0;
+  // latent attention, state-space recurrence, experts
+  void *lat_q = nullptr, *lat_o = nullptr;
+  float* ssd_y = nullptr;
+  float *route = nullptr, *shared = nullptr;
+  void *moe_h = nullptr, *moe_act = nullptr, *moe_y = nullptr, *moe_ints = nullptr;
+  size_t ld_route = 0, ld_act = 0;
+  size_t max_pairs = 0;
+  pi_buffer exp_keys, exp_pool;
   pi_buffer meta, head_in, logits, ids, scratch, trace, history;
   bool trace_on = false;
   cudaGraphExec_t step_exec = nullptr;
@@ -160,10 +197,13 @@ struct Loader {
   pi_status dev_vec(const std::string& name, size_t n, const float** out, float fill = 0.f) {
     std::vector<float> v;
     PI_TRY(vec(name, n, &v, fill));
+    return upload(v, out);
+  }
+  pi_status upload(const std::vector<float>& v, const float** out) {
     float* d = nullptr;
-    PI_CUDA(ctx, cudaMalloc(&d, std::max<size_t>(n, 1) * sizeof(float)));
+    PI_CUDA(ctx, cudaMalloc(&d, std::max<size_t>(v.size(), 1) * sizeof(float)));
     m->owned.push_back(d);
-    PI_CUDA(ctx, cudaMemcpy(d, v.data(), n * sizeof(float), cudaMemcpyHostToDevice));
+    PI_CUDA(ctx, cudaMemcpy(d, v.data(), v.size() * sizeof(float), cudaMemcpyHostToDevice));
     *out = d;
     return PI_OK;
   }
@@ -174,6 +214,13 @@ struct Loader {
     out->alpha = alpha[0];
     PI_TRY(dev_vec(name, n, &out->w, 1.f));
     return dev_vec(name + ".b", n, &out->b);
+  }
+  pi_status layer_norm(const std::string& name, pi_layer_norm* out, float scale = 1.f) {
+    std::vector<float> v;
+    PI_TRY(vec(name, m->c.width, &v, 1.f));
+    for (float& x : v) x *= scale;
+    out->eps = m->c.norm_eps;
+    return upload(v, &out->w);
   }
   // A matrix of the checkpoint as rows dst_r0, dst_r0 + step, ... of a fused one.
   pi_status piece(const std::string& name, size_t rows, size_t cols, size_t dst_r0, size_t step, std::vector<Piece>* out) {
@@ -198,6 +245,29 @@ struct Loader {
     out->push_back(Piece{s, 0, rows, dst_r0, step});
     return PI_OK;
   }
+  // Every head's [dim][rank] block of a matrix turned round: [heads * rank][dim].
+  pi_status transposed_heads(const std::string& name, size_t heads, size_t dim, size_t rank, pi_linear** out) {
+    std::vector<Piece> p;
+    std::vector<uint16_t> turned;
+    pi_tensor t = {};
+    if (synthetic) {
+      PI_TRY(piece(name, heads * rank, dim, 0, 1, &p));
+    } else {
+      PI_TRY(piece(name, heads * dim, rank, 0, 1, &p));   // checks the shape
+      const uint16_t* src = static_cast<const uint16_t*>(p[0].src.host->data);
+      turned.resize(heads * dim * rank);
+      for (size_t h = 0; h < heads; ++h)
+        for (size_t d = 0; d < dim; ++d)
+          for (size_t r = 0; r < rank; ++r) turned[(h * rank + r) * dim + d] = src[(h * dim + d) * rank + r];
+      t = pi_tensor{PI_BF16, 0, (int64_t)(heads * rank), (int64_t)dim, turned.data(), nullptr};
+      p[0].src.host = &t;
+      p[0].src.rows = p[0].nrows = heads * rank;
+      p[0].src.cols = dim;
+    }
+    PI_TRY(matrix(p, heads * rank, dim, out));
+    PI_CUDA(ctx, cudaStreamSynchronize(ctx->stream));     // `turned` may go
+    return PI_OK;
+  }
   pi_status matrix(const std::vector<Piece>& pieces, size_t rows, size_t cols, pi_linear** out) {
     PI_TRY(build_linear(ctx, pieces, rows, cols, 0, out));
     m->weight_bytes += pi_linear_weight_bytes(*out);
@@ -206,18 +276,258 @@ struct Loader {
 };
 
 pi_status check_layer(pi_ctx* ctx, int i, const pi_layer_config& c) {
-  PI_REQUIRE(ctx, c.mixer >= PI_MIXER_ATTENTION && c.mixer <= PI_MIXER_MLSTM, "layer %d: unknown mixer %d", i, c.mixer);
+  PI_REQUIRE(ctx, c.mixer >= PI_MIXER_ATTENTION && c.mixer <= PI_MIXER_SSD, "layer %d: unknown mixer %d", i, c.mixer);
   PI_REQUIRE(ctx, c.heads > 0 && c.dim > 0 && c.vdim > 0 && c.ff >= 0, "layer %d: sizes must be positive", i);
   if (c.mixer == PI_MIXER_ATTENTION) {
     PI_REQUIRE(ctx, c.kv_heads > 0 && c.heads % c.kv_heads == 0, "layer %d: %d heads do not share %d key/value heads", i, c.heads, c.kv_heads);
     PI_REQUIRE(ctx, c.maps == 1 || c.maps == 2, "layer %d: %d softmax maps", i, c.maps);
-    PI_REQUIRE(ctx, c.rot_dims >= 0 && c.rot_dims % 2 == 0 && c.rot_dims <= c.dim, "layer %d: %d rotary channels of %d", i, c.rot_dims, c.dim);
-    PI_REQUIRE(ctx, c.rot_dims == 0 || c.rot_base > 0.f, "layer %d: rotary base must be positive", i);
+    PI_REQUIRE(ctx, c.rot_dims <= c.dim, "layer %d: %d rotary channels of %d", i, c.rot_dims, c.dim);
+  } else if (c.mixer == PI_MIXER_LATENT) {
+    PI_REQUIRE(ctx, c.rank > 0, "layer %d: the latent needs channels", i);
   } else if (c.mixer == PI_MIXER_GLA) {
     PI_REQUIRE(ctx, c.tau != 0.f, "layer %d: tau is zero", i);
-  } else {
+  } else if (c.mixer == PI_MIXER_MLSTM) {
     PI_REQUIRE(ctx, c.gate_cap > 0.f, "layer %d: gate_cap must be positive", i);
+  } else {
+    PI_REQUIRE(ctx, c.groups > 0 && c.heads % c.groups == 0, "layer %d: %d heads do not form %d groups", i, c.heads, c.groups);
+    PI_REQUIRE(ctx, c.norm_groups > 0 && (c.heads * c.vdim) % c.norm_groups == 0, "layer %d: %d channels do not form %d parts", i, c.heads * c.vdim, c.norm_groups);
+    PI_REQUIRE(ctx, c.conv >= 1, "layer %d: the convolution needs taps", i);
   }
+  if (c.mixer == PI_MIXER_ATTENTION || c.mixer == PI_MIXER_LATENT) {
+    PI_REQUIRE(ctx, c.rot_dims >= 0 && c.rot_dims % 2 == 0, "layer %d: %d rotary channels", i, c.rot_dims);
+    PI_REQUIRE(ctx, c.rot_dims == 0 || c.rot_base > 0.f, "layer %d: rotary base must be positive", i);
+    PI_REQUIRE(ctx, c.rot_dims == 0 || c.rot_factor == 0.0 || c.rot_factor == 1.0 ||
+                        (c.rot_factor > 0.0 && c.rot_original > 0.0 && c.rot_fast > 0.0 && c.rot_slow > 0.0 && c.rot_base != 1.f),
+               "layer %d: rotary scaling constants must be positive", i);
+  }
+  if (c.ff > 0) {
+    PI_REQUIRE(ctx, c.ff_kind >= PI_FF_GELU && c.ff_kind <= PI_FF_EXPERTS, "layer %d: unknown feed-forward %d", i, c.ff_kind);
+    if (c.ff_kind == PI_FF_EXPERTS) {
+      PI_REQUIRE(ctx, c.experts > 0 && c.expert_groups > 0 && c.experts % c.expert_groups == 0, "layer %d: %d experts do not form %d groups", i, c.experts,
+                 c.expert_groups);
+      PI_REQUIRE(ctx, c.keep_groups >= 1 && c.keep_groups <= c.expert_groups, "layer %d: %d groups of %d are kept", i, c.keep_groups, c.expert_groups);
+      PI_REQUIRE(ctx, c.top >= 1 && c.top <= c.experts / c.expert_groups * c.keep_groups, "layer %d: %d experts per token", i, c.top);
+      PI_REQUIRE(ctx, c.shared_ff >= 0, "layer %d: sizes must be positive", i);
+    }
+  }
+  return PI_OK;
+}
+
+// Largest sizes of what a step needs beside the projections' outputs.
+struct Extents {
+  size_t in = 0, core = 1, ff = 1, lat_q = 0, lat_o = 0, inner = 0, route = 0, act = 0, top = 0, experts = 0;
+  bool chunk = true;
+  int attn = 0;
+};
+
+int add_rope(pi_layered* m, const pi_layer_config& c) {
+  RopeTable t;
+  t.dims = c.rot_dims;
+  t.base = c.rot_base;
+  if (c.rot_factor != 0.0 && c.rot_factor != 1.0) {
+    t.factor = c.rot_factor;
+    t.original = c.rot_original;
+    t.fast = c.rot_fast;
+    t.slow = c.rot_slow;
+  }
+  for (size_t i = 0; i < m->ropes.size(); ++i) {
+    const RopeTable& o = m->ropes[i];
+    if (o.dims == t.dims && o.base == t.base && o.factor == t.factor && o.original == t.original && o.fast == t.fast && o.slow == t.slow) return (int)i;
+  }
+  m->ropes.push_back(t);
+  return (int)m->ropes.size() - 1;
+}
+
+pi_status build_mixer(pi_ctx* ctx, Loader& ld, int i, int gla_rank, Layer& L, Extents& x) {
+  pi_layered* m = ld.m;
+  const pi_layer_config& c = L.c;
+  const size_t W = m->c.width, core = (size_t)c.heads * c.vdim;
+  const std::string mix = "l" + std::to_string(i) + ".mix.";
+  std::vector<Piece> p;
+  size_t rows = 0;
+  auto add = [&](const char* name, size_t n) -> pi_status {
+    PI_TRY(ld.piece(mix + name, n, W, rows, 1, &p));
+    rows += n;
+    return PI_OK;
+  };
+  if (c.mixer == PI_MIXER_ATTENTION) {
+    PI_TRY(add("q", (size_t)c.heads * c.maps * c.dim));
+    PI_TRY(add("k", (size_t)c.kv_heads * c.maps * c.dim));
+    PI_TRY(add("v", (size_t)c.kv_heads * c.vdim));
+    L.attn = x.attn++;
+    if (c.maps == 2) {   // lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, one number for the layer
+      double e[2];
+      for (int j = 0; j < 2; ++j) {
+        std::vector<float> a, b;
+        PI_TRY(ld.vec(mix + "lq" + std::to_string(j + 1), c.dim, &a));
+        PI_TRY(ld.vec(mix + "lk" + std::to_string(j + 1), c.dim, &b));
+        double d = 0;
+        for (int k = 0; k < c.dim; ++k) d += (double)a[k] * b[k];
+        e[j] = exp(d);
+      }
+      L.lambda = (float)(e[0] - e[1] + (double)c.diff);
+    }
+    L.rope = add_rope(m, c);
+  } else if (c.mixer == PI_MIXER_LATENT) {
+    pi_latent_attention& a = L.lat;
+    a.heads = c.heads;
+    a.dim = c.dim;
+    a.rot_dims = c.rot_dims;
+    a.vdim = c.vdim;
+    a.rank = c.rank;
+    a.window = c.window;
+    a.scale = c.scale;
+    a.eps = m->c.norm_eps;
+    PI_TRY(add("q", (size_t)c.heads * (c.dim + c.rot_dims)));
+    a.col_kv = (int)rows;
+    PI_TRY(add("dkv", (size_t)c.rank + c.rot_dims));
+    a.col_g = (int)rows;
+    PI_TRY(add("g", core));
+    PI_TRY(ld.dev_vec(mix + "dkv.norm", c.rank, &a.norm, 1.f));
+    std::vector<Piece> u;
+    PI_TRY(ld.piece(mix + "uk", (size_t)c.heads * c.dim, c.rank, 0, 1, &u));
+    PI_TRY(ld.piece(mix + "uv", core, c.rank, (size_t)c.heads * c.dim, 1, &u));
+    PI_TRY(ld.matrix(u, (size_t)c.heads * c.dim + core, c.rank, &L.ukv));
+    PI_TRY(ld.transposed_heads(mix + "uk", c.heads, c.dim, c.rank, &L.uk_t));
+    a.ukv = L.ukv;
+    a.uk_t = L.uk_t;
+    PI_REQUIRE(ctx, pi_latent_supported(ctx, a, m->c.compute), "layer %d: a latent of %d + %d channels is not supported", i, c.rank, c.rot_dims);
+    L.attn = x.attn++;
+    L.rope = add_rope(m, c);
+    if (!m->latent) {
+      m->expand = true;
+      m->latent_window = c.window;
+    }
+    m->latent = true;
+    m->expand = m->expand && pi_latent_expandable(ctx, a, m->c.compute);
+    m->latent_window = c.window <= 0 || m->latent_window <= 0 ? 0 : std::max(m->latent_window, c.window);
+    x.lat_q = std::max(x.lat_q, (size_t)c.heads * pi_latent_dp(c.rank, c.rot_dims));
+    x.lat_o = std::max(x.lat_o, (size_t)c.heads * c.rank);
+  } else if (c.mixer == PI_MIXER_SSD) {
+    pi_ssd& r = L.ssd;
+    r.heads = c.heads;
+    r.vdim = c.vdim;
+    r.dim = c.dim;
+    r.groups = c.groups;
+    r.norm_groups = c.norm_groups;
+    r.taps = c.conv;
+    r.eps = m->c.norm_eps;
+    r.col_x = (int)core;
+    r.col_dt = (int)(core + r.channels());
+    PI_TRY(add("in", core + r.channels() + c.heads));
+    PI_TRY(ld.dev_vec(mix + "conv", (size_t)r.channels() * c.conv, &r.conv, 0.25f));
+    PI_TRY(ld.dev_vec(mix + "conv.b", r.channels(), &r.conv_b));
+    PI_TRY(ld.dev_vec(mix + "dt_bias", c.heads, &r.dt_bias, -2.f));
+    PI_TRY(ld.dev_vec(mix + "A_log", c.heads, &r.a_log));
+    PI_TRY(ld.dev_vec(mix + "D", c.heads, &r.d, 1.f));
+    PI_TRY(ld.dev_vec(mix + "norm", core, &r.norm, 1.f));
+    r.state_off = m->state_floats;
+    m->state_floats += r.state_floats();
+    x.inner = std::max(x.inner, core);
+    x.chunk = x.chunk && pi_ssd_chunked(ctx, r, m->c.compute);
+  } else {
+    pi_recurrence& r = L.rec;
+    const size_t hd = (size_t)c.heads * c.dim;
+    r.kind = c.mixer == PI_MIXER_GLA ? PI_REC_GLA : PI_REC_MLSTM;
+    r.heads = c.heads;
+    r.dim = c.dim;
+    r.vdim = c.vdim;
+    r.eps = m->c.norm_eps;
+    r.q_scale = (float)(1.0 / sqrt((double)c.dim));
+    r.col_q = 0;
+    r.col_k = (int)hd;
+    r.col_v = (int)(2 * hd);
+    r.col_g = (int)(2 * hd + core);
+    PI_TRY(add("q", hd));
+    PI_TRY(add("k", hd));
+    PI_TRY(add("v", core));
+    PI_TRY(add("g", core));
+    if (r.kind == PI_REC_GLA) {
+      r.tau = c.tau;
+      r.rank = gla_rank;
+      if (!ld.synthetic) {   // the rank is what the checkpoint's matrix has
+        const pi_named_tensor* t;
+        PI_TRY(ld.find(mix + "a1", &t));
+        r.rank = (int)t->rows;
+      }
+      r.col_low = (int)rows;
+      PI_TRY(add("a1", r.rank));
+      PI_TRY(ld.dev_vec(mix + "a2", hd * r.rank, &r.a2, 0.01f));
+      PI_TRY(ld.dev_vec(mix + "a2.b", hd, &r.a2_b, 2.f));
+      PI_TRY(ld.dev_vec(mix + "norm", c.vdim, &r.norm, 1.f));
+    } else {
+      r.gate_cap = c.gate_cap;
+      r.gate_sigmoid = 1;
+      r.norm_per_head = true;
+      r.col_i = (int)rows;
+      PI_TRY(add("i", c.heads));
+      r.col_f = (int)rows;
+      PI_TRY(add("f", c.heads));
+      PI_TRY(ld.dev_vec(mix + "i.b", c.heads, &r.i_b, 0.f));
+      PI_TRY(ld.dev_vec(mix + "f.b", c.heads, &r.f_b, 3.f));
+      PI_TRY(ld.dev_vec(mix + "norm", core, &r.norm, 1.f));
+    }
+    r.state_off = m->state_floats;
+    m->state_floats += pi_recurrence_floats(r.kind, c.heads, c.dim, c.vdim);
+    x.chunk = x.chunk && pi_recurrence_chunked(ctx, r, m->c.compute);
+  }
+  PI_TRY(ld.matrix(p, rows, W, &L.in));
+  x.in = std::max(x.in, rows);
+  x.core = std::max(x.core, core);
+  p.clear();
+  PI_TRY(ld.piece(mix + "o", W, core, 0, 1, &p));
+  return ld.matrix(p, W, core, &L.out);
+}
+
+pi_status build_feed_forward(Loader& ld, int i, Layer& L, Extents& x) {
+  const pi_layer_config& c = L.c;
+  const size_t W = ld.m->c.width;
+  const std::string mlp = "l" + std::to_string(i) + ".mlp.";
+  std::vector<Piece> p;
+  auto gated = [&](const std::string& name, size_t ff, size_t at) -> pi_status {   // interleaved gate and up rows
+    PI_TRY(ld.piece(name + "gate", ff, W, at, 2, &p));
+    return ld.piece(name + "up", ff, W, at + 1, 2, &p);
+  };
+  if (c.ff_kind != PI_FF_EXPERTS) {
+    PI_TRY(gated(mlp, c.ff, 0));
+    PI_TRY(ld.matrix(p, 2 * (size_t)c.ff, W, &L.gate_up));
+    p.clear();
+    PI_TRY(ld.piece(mlp + "down", W, c.ff, 0, 1, &p));
+    x.ff = std::max(x.ff, (size_t)c.ff);
+    return ld.matrix(p, W, c.ff, &L.down);
+  }
+  pi_moe& e = L.moe;
+  e.experts = c.experts;
+  e.top = c.top;
+  e.groups = c.expert_groups;
+  e.keep = c.keep_groups;
+  PI_TRY(ld.dev_vec(mlp + "correction", c.experts, &e.correction));
+  size_t rows = 2 * (size_t)c.shared_ff;
+  if (c.shared_ff) PI_TRY(gated(mlp + "shared.", c.shared_ff, 0));
+  PI_TRY(ld.piece(mlp + "router", c.experts, W, rows, 1, &p));
+  rows += c.experts;
+  if (c.shared_ff) {
+    PI_TRY(ld.piece(mlp + "shared.sg", 1, W, rows, 1, &p));
+    ++rows;
+  }
+  PI_TRY(ld.matrix(p, rows, W, &L.gate_up));
+  if (c.shared_ff) {
+    p.clear();
+    PI_TRY(ld.piece(mlp + "shared.down", W, c.shared_ff, 0, 1, &p));
+    PI_TRY(ld.matrix(p, W, c.shared_ff, &L.down));
+  }
+  const size_t E = c.experts, ff = c.ff;
+  p.clear();
+  for (size_t k = 0; k < E; ++k) PI_TRY(gated(mlp + "e" + std::to_string(k) + ".", ff, k * 2 * ff));
+  PI_TRY(ld.matrix(p, E * 2 * ff, W, &L.expert_in));
+  p.clear();
+  for (size_t k = 0; k < E; ++k) PI_TRY(ld.piece(mlp + "e" + std::to_string(k) + ".down", W, ff, k * W, 1, &p));
+  PI_TRY(ld.matrix(p, E * W, ff, &L.expert_out));
+  x.ff = std::max(x.ff, (size_t)c.shared_ff);
+  x.route = std::max(x.route, E + 1);
+  x.act = std::max(x.act, ff);
+  x.top = std::max(x.top, (size_t)c.top);
+  x.experts = std::max(x.experts, E);
   return PI_OK;
 }
 
@@ -225,138 +535,89 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
   m->c = *cfg;
   m->c.layers = nullptr;
   const size_t W = cfg->width;
-  ld.keep.reserve((size_t)cfg->num_layers * 16 + 4);   // Source::host points into it
-  size_t max_in = 0, max_core = 1, max_ff = 1;
-  int n_attn = 0;
-  bool chunk = true;
+  const bool dyt = cfg->norm == PI_NORM_DYT;
+  size_t tensors = 8;
+  for (int i = 0; i < cfg->num_layers; ++i) tensors += 32 + 3 * (size_t)std::max(0, cfg->layers[i].experts);
+  ld.keep.reserve(tensors);   // Source::host points into it
+  Extents x;
   {
     std::vector<Piece> p;
     PI_TRY(ld.piece("embed", cfg->vocab_size, W, 0, 1, &p));
     PI_TRY(ld.matrix(p, cfg->vocab_size, W, &m->embed));
+    if (!cfg->tied) {
+      p.clear();
+      PI_TRY(ld.piece("head", cfg->vocab_size, W, 0, 1, &p));
+      PI_TRY(ld.matrix(p, cfg->vocab_size, W, &m->head));
+    }
   }
-  PI_TRY(ld.dyt("final.norm", &m->final_norm));
+  if (dyt) PI_TRY(ld.dyt("final.norm", &m->final_norm));
+  else PI_TRY(ld.layer_norm("final.norm", &m->final_ln, cfg->logit_scale));
   m->layers.resize(cfg->num_layers);
   for (int i = 0; i < cfg->num_layers; ++i) {
     Layer& L = m->layers[i];
     L.c = cfg->layers[i];
-    const pi_layer_config& c = L.c;
-    PI_TRY(check_layer(ctx, i, c));
-    const std::string l = "l" + std::to_string(i), mix = l + ".mix.";
-    const size_t core = (size_t)c.heads * c.vdim;
-    PI_TRY(ld.dyt(l + ".norm1", &L.norm1));
-    PI_TRY(ld.dyt(l + ".norm1b", &L.norm1b));
-    std::vector<Piece> p;
-    size_t rows = 0;
-    auto add = [&](const char* name, size_t n) -> pi_status {
-      PI_TRY(ld.piece(mix + name, n, W, rows, 1, &p));
-      rows += n;
-      return PI_OK;
+    PI_TRY(check_layer(ctx, i, L.c));
+    PI_REQUIRE(ctx, !dyt || L.c.ff == 0 || L.c.ff_kind == PI_FF_GELU, "layer %d: this feed-forward is not built behind Dynamic Tanh", i);
+    const std::string l = "l" + std::to_string(i);
+    auto norm = [&](const char* name, pi_dyt* before, pi_dyt* after, pi_layer_norm* ln, const char* scale_name, const float** scale) -> pi_status {
+      if (dyt) {
+        PI_TRY(ld.dyt(l + name, before));
+        return ld.dyt(l + name + "b", after);
+      }
+      PI_TRY(ld.layer_norm(l + name, ln));
+      return ld.dev_vec(l + scale_name, W, scale, 0.5f);
     };
-    if (c.mixer == PI_MIXER_ATTENTION) {
-      PI_TRY(add("q", (size_t)c.heads * c.maps * c.dim));
-      PI_TRY(add("k", (size_t)c.kv_heads * c.maps * c.dim));
-      PI_TRY(add("v", (size_t)c.kv_heads * c.vdim));
-      L.attn = n_attn++;
-      if (c.maps == 2) {   // lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, one number for the layer
-        double e[2];
-        for (int j = 0; j < 2; ++j) {
-          std::vector<float> a, b;
-          PI_TRY(ld.vec(mix + "lq" + std::to_string(j + 1), c.dim, &a));
-          PI_TRY(ld.vec(mix + "lk" + std::to_string(j + 1), c.dim, &b));
-          double d = 0;
-          for (int k = 0; k < c.dim; ++k) d += (double)a[k] * b[k];
-          e[j] = exp(d);
-        }
-        L.lambda = (float)(e[0] - e[1] + (double)c.diff);
-      }
-      for (size_t t = 0; t < m->ropes.size() && L.rope < 0; ++t)
-        if (m->ropes[t].dims == c.rot_dims && m->ropes[t].base == c.rot_base) L.rope = (int)t;
-      if (L.rope < 0) {
-        RopeTable t;
-        t.dims = c.rot_dims;
-        t.base = c.rot_base;
-        L.rope = (int)m->ropes.size();
-        m->ropes.push_back(t);
-      }
-    } else {
-      pi_recurrence& r = L.rec;
-      const size_t hd = (size_t)c.heads * c.dim;
-      r.kind = c.mixer == PI_MIXER_GLA ? PI_REC_GLA : PI_REC_MLSTM;
-      r.heads = c.heads;
-      r.dim = c.dim;
-      r.vdim = c.vdim;
-      r.eps = cfg->norm_eps;
-      r.q_scale = (float)(1.0 / sqrt((double)c.dim));
-      r.col_q = 0;
-      r.col_k = (int)hd;
-      r.col_v = (int)(2 * hd);
-      r.col_g = (int)(2 * hd + core);
-      PI_TRY(add("q", hd));
-      PI_TRY(add("k", hd));
-      PI_TRY(add("v", core));
-      PI_TRY(add("g", core));
-      if (r.kind == PI_REC_GLA) {
-        r.tau = c.tau;
-        r.rank = gla_rank;
-        if (!ld.synthetic) {   // the rank is what the checkpoint's matrix has
-          const pi_named_tensor* t;
-          PI_TRY(ld.find(mix + "a1", &t));
-          r.rank = (int)t->rows;
-        }
-        r.col_low = (int)rows;
-        PI_TRY(add("a1", r.rank));
-        std::vector<float> a2;
-        PI_TRY(ld.dev_vec(mix + "a2", hd * r.rank, &r.a2, 0.01f));
-        PI_TRY(ld.dev_vec(mix + "a2.b", hd, &r.a2_b, 2.f));
-        PI_TRY(ld.dev_vec(mix + "norm", c.vdim, &r.norm, 1.f));
-      } else {
-        r.gate_cap = c.gate_cap;
-        r.gate_sigmoid = 1;
-        r.norm_per_head = true;
-        r.col_i = (int)rows;
-        PI_TRY(add("i", c.heads));
-        r.col_f = (int)rows;
-        PI_TRY(add("f", c.heads));
-        PI_TRY(ld.dev_vec(mix + "i.b", c.heads, &r.i_b, 0.f));
-        PI_TRY(ld.dev_vec(mix + "f.b", c.heads, &r.f_b, 3.f));
-        PI_TRY(ld.dev_vec(mix + "norm", core, &r.norm, 1.f));
-      }
-      r.state_off = m->state_floats;
-      m->state_floats += pi_recurrence_floats(r.kind, c.heads, c.dim, c.vdim);
-      chunk = chunk && pi_recurrence_chunked(ctx, r, cfg->compute);
-    }
-    PI_TRY(ld.matrix(p, rows, W, &L.in));
-    max_in = std::max(max_in, rows);
-    max_core = std::max(max_core, core);
-    p.clear();
-    PI_TRY(ld.piece(mix + "o", W, core, 0, 1, &p));
-    PI_TRY(ld.matrix(p, W, core, &L.out));
-    if (c.ff > 0) {
-      PI_TRY(ld.dyt(l + ".norm2", &L.norm2));
-      PI_TRY(ld.dyt(l + ".norm2b", &L.norm2b));
-      p.clear();
-      PI_TRY(ld.piece(l + ".mlp.gate", c.ff, W, 0, 2, &p));
-      PI_TRY(ld.piece(l + ".mlp.up", c.ff, W, 1, 2, &p));
-      PI_TRY(ld.matrix(p, 2 * (size_t)c.ff, W, &L.gate_up));
-      p.clear();
-      PI_TRY(ld.piece(l + ".mlp.down", W, c.ff, 0, 1, &p));
-      PI_TRY(ld.matrix(p, W, c.ff, &L.down));
-      max_ff = std::max(max_ff, (size_t)c.ff);
+    PI_TRY(norm(".norm1", &L.norm1, &L.norm1b, &L.ln1, ".ls1", &L.ls1));
+    PI_TRY(build_mixer(ctx, ld, i, gla_rank, L, x));
+    if (L.c.ff > 0) {
+      PI_TRY(norm(".norm2", &L.norm2, &L.norm2b, &L.ln2, ".ls2", &L.ls2));
+      PI_TRY(build_feed_forward(ld, i, L, x));
     }
   }
-  m->chunked = chunk && m->state_floats > 0;
+  m->chunked = x.chunk && m->state_floats > 0;
   const size_t cap = cfg->max_rows;
   m->ld_h = round8(W);
-  m->ld_core = round8(max_core);
-  m->ld_ff = round8(max_ff);
-  m->ld_proj = round8(max_in);
-  PI_CUDA(ctx, cudaMalloc(&m->x, cap * W * sizeof(float)));
-  PI_CUDA(ctx, cudaMalloc(&m->proj, cap * m->ld_proj * sizeof(float)));
-  PI_CUDA(ctx, cudaMalloc(&m->h, cap * m->ld_h * sizeof(float)));
-  PI_CUDA(ctx, cudaMalloc(&m->core, cap * m->ld_core * sizeof(float)));
-  PI_CUDA(ctx, cudaMalloc(&m->ffh, cap * m->ld_ff * sizeof(float)));
+  m->ld_core = round8(x.core);
+  m->ld_ff = round8(x.ff);
+  m->ld_proj = round8(x.in);
+  m->ld_route = round8(x.route);
+  m->ld_act = round8(x.act);
+  m->max_pairs = cap * x.top;
+  auto alloc = [&](auto** p, size_t floats) -> pi_status {
+    if (floats) PI_CUDA(ctx, cudaMalloc(p, floats * sizeof(float)));
+    return PI_OK;
+  };
+  PI_TRY(alloc(&m->x, cap * W));
+  PI_TRY(alloc(&m->proj, cap * m->ld_proj));
+  PI_TRY(alloc(&m->h, cap * m->ld_h));
+  PI_TRY(alloc(&m->core, cap * m->ld_core));
+  PI_TRY(alloc(&m->ffh, cap * m->ld_ff));
+  const bool f32 = cfg->compute == PI_F32;
+  PI_TRY(alloc(&m->lat_q, cap * x.lat_q / (f32 ? 1 : 2)));
+  PI_TRY(alloc(&m->lat_o, (cap * x.lat_o + 1) / (f32 ? 1 : 2)));
+  PI_TRY(alloc(&m->ssd_y, cap * x.inner));
+  if (x.top) {
+    PI_TRY(alloc(&m->route, cap * m->ld_route));
+    PI_TRY(alloc(&m->shared, cap * W));
+    PI_TRY(alloc(&m->moe_h, m->max_pairs * m->ld_h / 2));
+    PI_TRY(alloc(&m->moe_act, m->max_pairs * m->ld_act));
+    PI_TRY(alloc(&m->moe_y, m->max_pairs * W));
+    // ids, weights, place, pair_at; then a tile (16 bytes) per pair at most
+    PI_TRY(alloc(&m->moe_ints, 8 * m->max_pairs + 16));
+  }
   PI_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
   return PI_OK;
+}
+
+pi_moe_lists moe_lists(const pi_layered* m) {
+  pi_moe_lists l;
+  l.tiles = static_cast<int4*>(m->moe_ints);
+  l.ids = reinterpret_cast<int32_t*>(l.tiles + m->max_pairs);
+  l.weights = reinterpret_cast<float*>(l.ids + m->max_pairs);
+  l.place = l.ids + 2 * m->max_pairs;
+  l.pair_at = l.ids + 3 * m->max_pairs;
+  l.n_tiles = l.ids + 4 * m->max_pairs;
+  return l;
 }
 
 pi_status ensure_ropes(pi_ctx* ctx, pi_layered* m, int positions) {
@@ -364,13 +625,13 @@ pi_status ensure_ropes(pi_ctx* ctx, pi_layered* m, int positions) {
     if (t.dims == 0 || positions <= t.cap) continue;
     const int cap = std::max(positions, std::max(2 * t.cap, 2048)), half = t.dims / 2;
     std::vector<float> c((size_t)cap * half), s(c.size());
-    for (int j = 0; j < half; ++j) {
-      const double f = pow((double)t.base, -2.0 * j / t.dims);
+    std::vector<double> f;
+    const double gain = rope_frequencies(t, &f);
+    for (int j = 0; j < half; ++j)
       for (int p = 0; p < cap; ++p) {
-        c[(size_t)p * half + j] = (float)cos(p * f);
-        s[(size_t)p * half + j] = (float)sin(p * f);
+        c[(size_t)p * half + j] = (float)(gain * cos(p * f[j]));
+        s[(size_t)p * half + j] = (float)(gain * sin(p * f[j]));
       }
-    }
     PI_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
     cudaFree(t.cos);
     cudaFree(t.sin);
@@ -385,6 +646,8 @@ pi_status ensure_ropes(pi_ctx* ctx, pi_layered* m, int positions) {
 }
 
 // ---- one step -----------------------------------------------------------------------------------------------------------
+constexpr size_t kExpandBytes = (size_t)4 << 30;   // of the scratch pool for expanded keys and values
+
 struct Staged {
   pi_seq_batch b;
   const int32_t* out_rows = nullptr;   // device
@@ -410,6 +673,43 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
   int rows = 0, max_pos = 0;
   std::vector<int32_t> row_seq, row_pos, row0(n), single, portions, scan, chunk_seqs, chunks, chunk0(1, 0);
   int max_portion = 0;
+  std::vector<int32_t> latent_rows, expand, exp_lo, exp_start, exp_lens, exp_tables, key_seq, key_pos;
+  int max_expand = 0, exp_max_blocks = 1, exp_blocks = 0;
+  const int wide = m->latent_window;
+  if (m->latent) {
+    exp_lo.assign(n, 0);
+    exp_start.assign(n, 0);
+    exp_lens.assign(n, 0);
+    size_t per_block = 0;
+    for (const Layer& L : m->layers)
+      if (L.c.mixer == PI_MIXER_LATENT) per_block = std::max(per_block, pi_latent_pool_elems(L.lat, 1) * sizeof(__nv_bfloat16));
+    for (int i = 0; i < n && m->expand; ++i) {   // which portions are expanded, and what they see
+      const int k = in->n_tokens[i], p0 = in->start_pos[i];
+      if (k < kExpandPortion || k > m->c.max_rows || p0 < 0 || p0 >= (1 << 30)) continue;
+      const int lo = wide > 0 ? std::max(0, p0 - wide + 1) / kExpandBlock * kExpandBlock : 0, blocks = (p0 + k - lo + kExpandBlock - 1) / kExpandBlock;
+      if ((exp_blocks + blocks) * per_block > kExpandBytes) {   // all or none, so that a row's length tells its way
+        expand.clear();
+        exp_blocks = 0;
+        break;
+      }
+      expand.push_back(i);
+      exp_lo[i] = lo;
+      exp_start[i] = p0 - lo;
+      exp_lens[i] = blocks;
+      exp_blocks += blocks;
+      exp_max_blocks = std::max(exp_max_blocks, blocks);
+      max_expand = std::max(max_expand, k);
+    }
+    exp_tables.assign((size_t)n * exp_max_blocks, 0);
+    int next = 0;
+    for (int i : expand) {
+      for (int j = 0; j < exp_lens[i]; ++j) exp_tables[(size_t)i * exp_max_blocks + j] = next++;
+      for (int t = 0; t < exp_start[i] + in->n_tokens[i]; ++t) {
+        key_seq.push_back(i);
+        key_pos.push_back(t);
+      }
+    }
+  }
   for (int i = 0; i < n; ++i) {
     const int k = in->n_tokens[i], p0 = in->start_pos[i];
     PI_REQUIRE(ctx, k >= 1 && p0 >= 0 && p0 < (1 << 30), "sequence %d: %d tokens from position %d", i, k, p0);
@@ -419,6 +719,8 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
       row_seq.push_back(i);
       row_pos.push_back(p0 + j);
     }
+    if (m->latent && (expand.empty() || k < kExpandPortion))
+      for (int j = 0; j < k; ++j) latent_rows.push_back(rows + j);
     if (k == 1) {
       single.push_back(rows);
     } else {
@@ -469,7 +771,10 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
                o_n = put(in->n_tokens, n), o_st = put(in->start_pos, n), o_sl = put(in->state_slots, in->state_slots ? n : 0),
                o_ln = put(in->table_lens, n), o_tb = put(in->block_tables, (size_t)n * in->max_blocks), o_si = put(single.data(), single.size()),
                o_po = put(portions.data(), portions.size()), o_sc = put(scan.data(), scan.size()), o_cs = put(chunk_seqs.data(), chunk_seqs.size()),
-               o_ch = put(chunks.data(), chunks.size()), o_c0 = put(chunk0.data(), chunk0.size()), o_out = put(in->out_rows, in->n_out);
+               o_ch = put(chunks.data(), chunks.size()), o_c0 = put(chunk0.data(), chunk0.size()), o_out = put(in->out_rows, in->n_out),
+               o_lr = put(latent_rows.data(), latent_rows.size()), o_ex = put(expand.data(), expand.size()), o_el = put(exp_lo.data(), exp_lo.size()),
+               o_es = put(exp_start.data(), exp_start.size()), o_en = put(exp_lens.data(), exp_lens.size()),
+               o_et = put(exp_tables.data(), exp_tables.size()), o_ks = put(key_seq.data(), key_seq.size()), o_kp = put(key_pos.data(), key_pos.size());
   PI_TRY(pi_reserve_pinned(ctx, words * 4));
   PI_TRY(pi_reserve(ctx, &m->meta, words * 4));
   int32_t* host = static_cast<int32_t*>(ctx->pinned);
@@ -506,12 +811,36 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
   b.n_chunks = (int)chunks.size() / 2;
   b.chunk0 = d + o_c0;
   b.max_pos = max_pos + extra_positions;
+  b.latent_rows = d + o_lr;
+  b.n_latent = (int)latent_rows.size();
+  b.expand = d + o_ex;
+  b.n_expand = (int)expand.size();
+  b.max_expand = max_expand;
+  b.exp_lo = d + o_el;
+  b.exp_start = d + o_es;
+  b.exp_lens = d + o_en;
+  b.exp_tables = d + o_et;
+  b.exp_max_blocks = exp_max_blocks;
+  b.exp_blocks = exp_blocks;
+  b.key_seq = d + o_ks;
+  b.key_pos = d + o_kp;
+  b.n_keys = (int)key_seq.size();
   st->out_rows = d + o_out;
   st->n_out = in->n_out;
   // scratch is sized here, so that nothing allocates while a step is being captured
-  size_t floats = 0;
-  for (const Layer& L : m->layers)
-    if (L.attn < 0) floats = std::max(floats, pi_recurrence_scratch_floats(L.rec, b.n_chunks));
+  size_t floats = 0, keys = 0, elems = 0;
+  for (const Layer& L : m->layers) {
+    if (L.c.mixer == PI_MIXER_SSD) floats = std::max(floats, pi_ssd_scratch_floats(L.ssd, b.n_chunks));
+    else if (L.attn < 0) floats = std::max(floats, pi_recurrence_scratch_floats(L.rec, b.n_chunks));
+    else if (L.c.mixer == PI_MIXER_LATENT) {
+      keys = std::max(keys, (size_t)b.n_keys * pi_latent_rp(L.c.rank));
+      elems = std::max(elems, pi_latent_pool_elems(L.lat, b.exp_blocks));
+    }
+  }
+  if (b.n_expand) {
+    PI_TRY(pi_reserve(ctx, &m->exp_keys, keys * sizeof(__nv_bfloat16)));
+    PI_TRY(pi_reserve(ctx, &m->exp_pool, elems * sizeof(__nv_bfloat16)));
+  }
   if (floats) PI_TRY(pi_reserve(ctx, &m->scratch, floats * sizeof(float)));
   if (in->n_out) {
     PI_TRY(pi_reserve(ctx, &m->head_in, (size_t)in->n_out * m->ld_h * sizeof(float)));
@@ -533,127 +862,288 @@ pi_status project(pi_ctx* ctx, const pi_linear* lin, const void* in, size_t in_l
   return pi_launch_gemv(ctx, lin, a);
 }
 
+pi_kv_view kv_view(const pi_kv_pool* pool, int attn) {
+  const pi_kv_region& g = pool->regions[attn];
+  pi_kv_view kv;
+  kv.base = reinterpret_cast<char*>(pool->data) + g.offset;
+  kv.kind = pool->kind;
+  kv.kv_heads = g.kv_heads;
+  kv.maps = g.maps;
+  kv.dp = g.dp;
+  kv.vp = g.vp;
+  kv.block_size = pool->L.block_size;
+  return kv;
+}
+
+// The layer's mixer, from h to core.
+pi_status run_mixer(pi_ctx* ctx, pi_layered* m, const Layer& L, pi_kv_pool* pool, pi_state_pool* state, const Staged& st, bool bf16) {
+  const pi_seq_batch& b = st.b;
+  const pi_layer_config& c = L.c;
+  const int M = b.rows, kind = bf16 ? PI_BF16 : PI_F32;
+  pi_linear_args in;
+  in.out = m->proj;
+  in.out_stride = m->ld_proj;
+  if (c.mixer == PI_MIXER_ATTENTION) {
+    const pi_kv_view kv = kv_view(pool, L.attn);
+    pi_maps_attention a;
+    a.heads = c.heads;
+    a.kv_heads = c.kv_heads;
+    a.maps = c.maps;
+    a.dim = c.dim;
+    a.vdim = c.vdim;
+    a.window = c.window;
+    a.scale = c.scale;
+    a.eps = m->c.norm_eps;
+    a.lambda = L.lambda;
+    a.out_scale = 1.0f - c.diff;
+    a.rot_dims = c.rot_dims;
+    a.rope_cos = m->ropes[L.rope].cos;
+    a.rope_sin = m->ropes[L.rope].sin;
+    pi_maps_kv mk;
+    if (c.dim % 2 == 0) {   // rotary positions and the KV write fold into the projection
+      mk.q_rows = c.heads * c.maps * c.dim;
+      mk.k_rows = c.kv_heads * c.maps * c.dim;
+      mk.maps = c.maps;
+      mk.dim = c.dim;
+      mk.vdim = c.vdim;
+      mk.rot_dims = c.rot_dims;
+      mk.rope_cos = a.rope_cos;
+      mk.rope_sin = a.rope_sin;
+      mk.base = kv.base;
+      mk.kind = kv.kind;
+      mk.kv_heads = kv.kv_heads;
+      mk.dp = kv.dp;
+      mk.vp = kv.vp;
+      mk.block_size = kv.block_size;
+      mk.row_seq = b.row_seq;
+      mk.row_pos = b.row_pos;
+      mk.lens = b.lens;
+      mk.tables = b.tables;
+      mk.max_blocks = b.max_blocks;
+      in.epi = PI_EPI_MAPS_QKV;
+      in.maps_kv = &mk;
+    }
+    PI_TRY(project(ctx, L.in, m->h, m->ld_h, M, bf16, in));
+    if (in.epi != PI_EPI_MAPS_QKV) PI_TRY(pi_launch_maps_rope_kv(ctx, a, kv, m->proj, m->ld_proj, b));
+    return pi_launch_maps_attention(ctx, a, kv, m->proj, m->ld_proj, m->core, m->ld_core, kind, b);
+  }
+  PI_TRY(project(ctx, L.in, m->h, m->ld_h, M, bf16, in));
+  if (c.mixer == PI_MIXER_LATENT) {
+    pi_latent_attention a = L.lat;
+    a.rope_cos = m->ropes[L.rope].cos;
+    a.rope_sin = m->ropes[L.rope].sin;
+    pi_latent_scratch s;
+    s.q = m->lat_q;
+    s.o = m->lat_o;
+    s.keys = static_cast<__nv_bfloat16*>(m->exp_keys.ptr);
+    s.pool = static_cast<__nv_bfloat16*>(m->exp_pool.ptr);
+    return pi_launch_latent_attention(ctx, a, kv_view(pool, L.attn), m->proj, m->ld_proj, m->core, m->ld_core, kind, b, s);
+  }
+  if (c.mixer == PI_MIXER_SSD) {
+    pi_ssd r = L.ssd;
+    r.state = state->data;
+    r.state_stride = state->stride;
+    return pi_launch_ssd(ctx, r, m->proj, m->ld_proj, m->ssd_y, m->core, m->ld_core, kind, b, static_cast<float*>(m->scratch.ptr));
+  }
+  pi_recurrence r = L.rec;
+  r.state = state->data;
+  r.state_stride = state->stride;
+  return pi_launch_recurrence(ctx, r, m->proj, m->ld_proj, m->core, m->ld_core, kind, b, static_cast<float*>(m->scratch.ptr));
+}
+
+// The layer's experts, from h to *sum (which the row kernel that follows adds up).
+pi_status run_experts(pi_ctx* ctx, pi_layered* m, const Layer& L, int M, bool bf16, pi_expert_sum* sum) {
+  const pi_layer_config& c = L.c;
+  const pi_moe_lists lists = moe_lists(m);
+  const int pairs = M * c.top;
+  // the shared expert's first projection carries the router's rows
+  pi_linear_args a;
+  if (c.shared_ff) {
+    a.epi = PI_EPI_CLAMP_GLU;
+    a.glu_limit = c.shared_limit;
+    a.glu_rows = 2 * c.shared_ff;
+    a.out = static_cast<float*>(m->ffh);
+    a.out_bf16 = static_cast<__nv_bfloat16*>(m->ffh);
+    a.out_stride = m->ld_ff;
+    a.rest = m->route;
+    a.rest_stride = m->ld_route;
+  } else {
+    a.out = m->route;
+    a.out_stride = m->ld_route;
+  }
+  PI_TRY(project(ctx, L.gate_up, m->h, m->ld_h, M, bf16, a));
+  PI_TRY(pi_launch_moe_route(ctx, L.moe, m->route, m->ld_route, M, lists));
+  pi_expert_rows rows;
+  rows.experts = c.experts;
+  const void* x = m->h;
+  if (bf16) {
+    PI_TRY(pi_launch_moe_gather(ctx, L.moe, M, lists, static_cast<const __nv_bfloat16*>(m->h), m->ld_h, static_cast<__nv_bfloat16*>(m->moe_h)));
+    rows.tiles = lists.tiles;
+    rows.n_tiles = lists.n_tiles;
+    rows.max_tiles = pi_moe_max_tiles(M, L.moe);
+    rows.tile_rows = pi_moe_tile_rows(M, L.moe);
+    x = m->moe_h;
+  } else {
+    rows.expert = lists.ids;
+    rows.x_div = c.top;
+  }
+  pi_linear_args e;
+  e.experts = &rows;
+  e.epi = PI_EPI_CLAMP_GLU;
+  e.glu_limit = c.limit;
+  e.out = static_cast<float*>(m->moe_act);
+  e.out_bf16 = static_cast<__nv_bfloat16*>(m->moe_act);
+  e.out_stride = m->ld_act;
+  PI_TRY(project(ctx, L.expert_in, x, m->ld_h, pairs, bf16, e));
+  rows.x_div = 1;
+  pi_linear_args d;
+  d.experts = &rows;
+  d.out = static_cast<float*>(m->moe_y);
+  d.out_bf16 = bf16 ? static_cast<__nv_bfloat16*>(m->moe_y) : nullptr;
+  d.out_stride = m->c.width;
+  PI_TRY(project(ctx, L.expert_out, m->moe_act, m->ld_act, pairs, bf16, d));
+  sum->top = c.top;
+  sum->weights = lists.weights;
+  sum->place = bf16 ? lists.place : nullptr;
+  sum->y = m->moe_y;
+  sum->y_bf16 = bf16;
+  sum->y_stride = m->c.width;
+  sum->scale = L.ls2;
+  if (c.shared_ff) {
+    pi_linear_args s;
+    s.out = m->shared;
+    s.out_stride = m->c.width;
+    PI_TRY(project(ctx, L.down, m->ffh, m->ld_ff, M, bf16, s));
+    sum->shared = m->shared;
+    sum->shared_stride = m->c.width;
+    sum->shared_gate = m->route + c.experts;
+    sum->shared_gate_stride = m->ld_route;
+  }
+  return PI_OK;
+}
+
 pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool* state, const Staged& st) {
   const pi_seq_batch& b = st.b;
   const int M = b.rows, W = m->c.width, NL = (int)m->layers.size();
-  const bool bf16 = act_bf16(ctx, m, M);
+  const bool bf16 = act_bf16(ctx, m, M), dyt = m->c.norm == PI_NORM_DYT;
   const int kind = bf16 ? PI_BF16 : PI_F32;
-  {
+  const bool head_bf16 = st.n_out && act_bf16(ctx, m, st.n_out);
+  pi_row_norm row;               // layer norm: from x to h
+  row.rows = M;
+  row.width = W;
+  row.x = m->x;
+  row.h = m->h;
+  row.ld_h = m->ld_h;
+  row.h_kind = kind;
+  if (dyt) {
     pi_prof_scope prof(ctx, PI_PROF_OTHER);
     auto k = bf16 ? embed_dyt_kernel<__nv_bfloat16> : embed_dyt_kernel<float>;
     PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(M), dim3(256), 0, 1, static_cast<const uint16_t*>(m->embed->w), m->embed->ld,
                                     m->c.vocab_size, W, b.tokens, m->x, m->layers[0].norm1, m->h, m->ld_h));
+  } else {
+    pi_row_norm e = row;
+    e.table = static_cast<const uint16_t*>(m->embed->w);
+    e.table_ld = m->embed->ld;
+    e.vocab = m->c.vocab_size;
+    e.tokens = b.tokens;
+    e.norm = m->layers[0].ln1;
+    PI_TRY(pi_launch_row_norm(ctx, e));
   }
+  bool final_done = false;       // head_in holds the normalised rows
   for (int i = 0; i < NL; ++i) {
     const Layer& L = m->layers[i];
     const pi_layer_config& c = L.c;
-    const pi_dyt after = i + 1 < NL ? m->layers[i + 1].norm1 : m->final_norm;
-    pi_linear_args in;
-    in.out = m->proj;
-    in.out_stride = m->ld_proj;
-    if (c.mixer == PI_MIXER_ATTENTION) {
-      const pi_kv_region& g = pool->regions[L.attn];
-      pi_kv_view kv;
-      kv.base = reinterpret_cast<char*>(pool->data) + g.offset;
-      kv.kind = pool->kind;
-      kv.kv_heads = g.kv_heads;
-      kv.maps = g.maps;
-      kv.dp = g.dp;
-      kv.vp = g.vp;
-      kv.block_size = pool->L.block_size;
-      pi_maps_attention a;
-      a.heads = c.heads;
-      a.kv_heads = c.kv_heads;
-      a.maps = c.maps;
-      a.dim = c.dim;
-      a.vdim = c.vdim;
-      a.window = c.window;
-      a.scale = c.scale;
-      a.eps = m->c.norm_eps;
-      a.lambda = L.lambda;
-      a.out_scale = 1.0f - c.diff;
-      a.rot_dims = c.rot_dims;
-      a.rope_cos = m->ropes[L.rope].cos;
-      a.rope_sin = m->ropes[L.rope].sin;
-      pi_maps_kv mk;
-      if (c.dim % 2 == 0) {   // rotary positions and the KV write fold into the projection
-        mk.q_rows = c.heads * c.maps * c.dim;
-        mk.k_rows = c.kv_heads * c.maps * c.dim;
-        mk.maps = c.maps;
-        mk.dim = c.dim;
-        mk.vdim = c.vdim;
-        mk.rot_dims = c.rot_dims;
-        mk.rope_cos = a.rope_cos;
-        mk.rope_sin = a.rope_sin;
-        mk.base = kv.base;
-        mk.kind = kv.kind;
-        mk.kv_heads = kv.kv_heads;
-        mk.dp = kv.dp;
-        mk.vp = kv.vp;
-        mk.block_size = kv.block_size;
-        mk.row_seq = b.row_seq;
-        mk.row_pos = b.row_pos;
-        mk.lens = b.lens;
-        mk.tables = b.tables;
-        mk.max_blocks = b.max_blocks;
-        in.epi = PI_EPI_MAPS_QKV;
-        in.maps_kv = &mk;
-      }
-      PI_TRY(project(ctx, L.in, m->h, m->ld_h, M, bf16, in));
-      if (in.epi != PI_EPI_MAPS_QKV) PI_TRY(pi_launch_maps_rope_kv(ctx, a, kv, m->proj, m->ld_proj, b));
-      PI_TRY(pi_launch_maps_attention(ctx, a, kv, m->proj, m->ld_proj, m->core, m->ld_core, kind, b));
-    } else {
-      PI_TRY(project(ctx, L.in, m->h, m->ld_h, M, bf16, in));
-      pi_recurrence r = L.rec;
-      r.state = state->data;
-      r.state_stride = state->stride;
-      PI_TRY(pi_launch_recurrence(ctx, r, m->proj, m->ld_proj, m->core, m->ld_core, kind, b, static_cast<float*>(m->scratch.ptr)));
-    }
-    pi_dyt_residual res;
-    res.x = m->x;
-    res.x_stride = W;
-    res.post = L.norm1b;
-    res.next = c.ff > 0 ? L.norm2 : after;
-    res.h = m->h;
-    res.h_stride = m->ld_h;
-    {
+    const bool last = i + 1 == NL;
+    PI_TRY(run_mixer(ctx, m, L, pool, state, st, bf16));
+    if (dyt) {
+      const pi_dyt after = last ? m->final_norm : m->layers[i + 1].norm1;
+      pi_dyt_residual res;
+      res.x = m->x;
+      res.x_stride = W;
+      res.post = L.norm1b;
+      res.next = c.ff > 0 ? L.norm2 : after;
+      res.h = m->h;
+      res.h_stride = m->ld_h;
       pi_linear_args a;
       a.epi = PI_EPI_DYT_RESIDUAL;
       a.residual = &res;
       PI_TRY(project(ctx, L.out, m->core, m->ld_core, M, bf16, a));
-    }
-    if (c.ff > 0) {
+      if (c.ff > 0) {
+        pi_linear_args g;
+        g.epi = PI_EPI_GEGLU;
+        g.out = static_cast<float*>(m->ffh);
+        g.out_bf16 = static_cast<__nv_bfloat16*>(m->ffh);
+        g.out_stride = m->ld_ff;
+        PI_TRY(project(ctx, L.gate_up, m->h, m->ld_h, M, bf16, g));
+        res.post = L.norm2b;
+        res.next = after;
+        PI_TRY(project(ctx, L.down, m->ffh, m->ld_ff, M, bf16, a));
+      }
+    } else {
       pi_linear_args a;
-      a.epi = PI_EPI_GEGLU;
-      a.out = static_cast<float*>(m->ffh);
-      a.out_bf16 = static_cast<__nv_bfloat16*>(m->ffh);
-      a.out_stride = m->ld_ff;
-      PI_TRY(project(ctx, L.gate_up, m->h, m->ld_h, M, bf16, a));
-      res.post = L.norm2b;
-      res.next = after;
-      pi_linear_args d;
-      d.epi = PI_EPI_DYT_RESIDUAL;
-      d.residual = &res;
-      PI_TRY(project(ctx, L.down, m->ffh, m->ld_ff, M, bf16, d));
+      a.epi = PI_EPI_SCALE_ADD;
+      a.out = m->x;
+      a.out_stride = W;
+      a.out_scale = L.ls1;
+      PI_TRY(project(ctx, L.out, m->core, m->ld_core, M, bf16, a));
+      pi_row_norm next = row;    // what the layer's end hands on; behind the last layer only the wanted rows are normalised
+      if (!last) next.norm = m->layers[i + 1].ln1;
+      else next.h = nullptr;
+      if (c.ff > 0) {
+        pi_row_norm n = row;
+        n.norm = L.ln2;
+        PI_TRY(pi_launch_row_norm(ctx, n));
+      }
+      pi_expert_sum sum;
+      if (c.ff > 0 && c.ff_kind == PI_FF_EXPERTS) {
+        PI_TRY(run_experts(ctx, m, L, M, bf16, &sum));
+        next.experts = &sum;
+        if (last && st.all_rows) {
+          next.norm = m->final_ln;
+          next.h = m->head_in.ptr;
+          next.h_kind = head_bf16 ? PI_BF16 : PI_F32;
+          final_done = true;
+        }
+      } else if (c.ff > 0) {
+        pi_linear_args g;
+        g.epi = c.ff_kind == PI_FF_SILU ? PI_EPI_SWIGLU : PI_EPI_GEGLU;
+        g.out = static_cast<float*>(m->ffh);
+        g.out_bf16 = static_cast<__nv_bfloat16*>(m->ffh);
+        g.out_stride = m->ld_ff;
+        PI_TRY(project(ctx, L.gate_up, m->h, m->ld_h, M, bf16, g));
+        a.out_scale = L.ls2;
+        PI_TRY(project(ctx, L.down, m->ffh, m->ld_ff, M, bf16, a));
+      }
+      if (next.h || next.experts) PI_TRY(pi_launch_row_norm(ctx, next));
     }
     if (m->trace_on)
       PI_CUDA(ctx, cudaMemcpyAsync(static_cast<float*>(m->trace.ptr) + (size_t)i * m->c.max_rows * W, m->x, (size_t)M * W * sizeof(float),
                                    cudaMemcpyDeviceToDevice, ctx->stream));
   }
   if (st.n_out == 0) return PI_OK;
-  // the last epilogue left the final norm of every row in h; anything but all rows in order is gathered from x
-  const bool head_bf16 = act_bf16(ctx, m, st.n_out);
-  const void* last = m->h;
-  if (!(st.all_rows && head_bf16 == bf16)) {
+  const void* last = m->head_in.ptr;
+  if (!dyt) {
+    if (!final_done) {
+      pi_row_norm n = row;
+      n.rows = st.n_out;
+      n.pick = st.out_rows;
+      n.norm = m->final_ln;
+      n.h = m->head_in.ptr;
+      n.h_kind = head_bf16 ? PI_BF16 : PI_F32;
+      PI_TRY(pi_launch_row_norm(ctx, n));
+    }
+  } else if (!(st.all_rows && head_bf16 == bf16)) {
+    // the last epilogue left the final norm of every row in h; anything but all rows in order is gathered from x
     pi_prof_scope prof(ctx, PI_PROF_OTHER);
     auto k = head_bf16 ? gather_dyt_kernel<__nv_bfloat16> : gather_dyt_kernel<float>;
     PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(st.n_out), dim3(256), 0, 1, (const float*)m->x, W, st.out_rows, m->final_norm, m->head_in.ptr, m->ld_h));
-    last = m->head_in.ptr;
+  } else {
+    last = m->h;
   }
   pi_linear_args a;
   a.out = static_cast<float*>(m->logits.ptr);
   a.out_stride = m->c.vocab_size;
-  return project(ctx, m->embed, last, m->ld_h, st.n_out, head_bf16, a);
+  return project(ctx, m->head ? m->head : m->embed, last, m->ld_h, st.n_out, head_bf16, a);
 }
 
 pi_status multi_step(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool* state, const Staged& st, uint32_t* history, int* counter) {
@@ -674,6 +1164,8 @@ pi_status pi_layered_create(pi_ctx* ctx, const pi_layered_config* cfg, const pi_
   PI_REQUIRE(ctx, ctx->tp == 1, "layered designs run on one GPU");
   PI_REQUIRE(ctx, cfg->width > 0 && cfg->vocab_size > 0 && cfg->num_layers > 0 && cfg->layers && cfg->max_rows > 0, "model config fields must be positive");
   PI_REQUIRE(ctx, cfg->compute == PI_BF16 || cfg->compute == PI_F32, "layered designs compute in bf16 or f32");
+  PI_REQUIRE(ctx, cfg->norm == PI_NORM_DYT || cfg->norm == PI_NORM_LAYER, "unknown normalisation %d", cfg->norm);
+  PI_REQUIRE(ctx, cfg->norm == PI_NORM_LAYER || cfg->logit_scale == 1.f, "logits are scaled behind layer norm only");
   PI_REQUIRE(ctx, tensors || gla_rank > 0, "synthetic weights need a rank for the decay's low-rank input");
   pi_layered* m = new (std::nothrow) pi_layered();
   if (!m) return pi_fail(ctx, PI_ERR_OOM, "host allocation failed");
@@ -697,14 +1189,16 @@ void pi_layered_destroy(pi_layered* m) {
   if (!m) return;
   if (m->step_exec) cudaGraphExecDestroy(m->step_exec);
   for (Layer& L : m->layers)
-    for (pi_linear* l : {L.in, L.out, L.gate_up, L.down}) pi_linear_destroy(l);
+    for (pi_linear* l : {L.in, L.out, L.gate_up, L.down, L.expert_in, L.expert_out, L.ukv, L.uk_t}) pi_linear_destroy(l);
   pi_linear_destroy(m->embed);
+  pi_linear_destroy(m->head);
   for (RopeTable& t : m->ropes) {
     cudaFree(t.cos);
     cudaFree(t.sin);
   }
   for (void* p : m->owned) cudaFree(p);
-  for (void* p : {(void*)m->x, (void*)m->proj, m->h, m->core, m->ffh, m->meta.ptr, m->head_in.ptr, m->logits.ptr, m->ids.ptr, m->scratch.ptr,
+  for (void* p : {(void*)m->x, (void*)m->proj, m->h, m->core, m->ffh, m->lat_q, m->lat_o, (void*)m->ssd_y, (void*)m->route, (void*)m->shared, m->moe_h, m->moe_act,
+                  m->moe_y, m->moe_ints, m->exp_keys.ptr, m->exp_pool.ptr, m->meta.ptr, m->head_in.ptr, m->logits.ptr, m->ids.ptr, m->scratch.ptr,
                   m->trace.ptr, m->history.ptr})
     if (p) cudaFree(p);
   delete m;
@@ -722,10 +1216,15 @@ pi_status pi_layered_kv_regions(pi_ctx* ctx, const pi_layered* m, int num_blocks
   for (const Layer& L : m->layers) {
     if (L.attn < 0) continue;
     pi_kv_region g;
-    g.kv_heads = L.c.kv_heads;
-    g.maps = L.c.maps;
-    g.dp = (L.c.dim + 15) / 16 * 16;
-    g.vp = (L.c.vdim + 15) / 16 * 16;
+    if (L.c.mixer == PI_MIXER_LATENT) {   // [latent | rotated key part], common to the heads
+      g.kv_heads = g.maps = 1;
+      g.dp = pi_latent_dp(L.c.rank, L.c.rot_dims);
+    } else {
+      g.kv_heads = L.c.kv_heads;
+      g.maps = L.c.maps;
+      g.dp = (L.c.dim + 15) / 16 * 16;
+      g.vp = (L.c.vdim + 15) / 16 * 16;
+    }
     g.block_bytes = (size_t)block_size * g.kv_heads * (g.maps * g.dp + g.vp) * es;
     g.offset = at;
     at += (g.block_bytes * num_blocks + 255) / 256 * 256;

@@ -1,5 +1,6 @@
 // Internal declarations of layered designs: models whose layers each name a token mixer (windowed multi-map attention,
-// a gated linear recurrence, a matrix memory) with sizes of its own.
+// latent attention, a gated linear recurrence, a matrix memory, a state-space recurrence) and a feed-forward (dense or
+// experts) with sizes of their own.
 #pragma once
 
 #include "pi_common.cuh"
@@ -35,7 +36,24 @@ struct pi_seq_batch {
   int n_chunks = 0;
   const int32_t* chunk0 = nullptr;      // [n_chunk_seqs + 1] first chunk of a sequence
   int max_pos = 0;                      // host-side bound on every position of the step
+  // latent attention: rows that attend to the cached latents as they are, and the portions that are long enough to have their
+  // keys and values spelled out first.  Those portions see keys from exp_lo[seq] on (a multiple of kExpandBlock); their
+  // expanded rows lie in a scratch pool with tables of its own, positions counted from exp_lo.
+  const int32_t* latent_rows = nullptr;
+  int n_latent = 0;
+  const int32_t* expand = nullptr;      // sequences
+  int n_expand = 0, max_expand = 0;     // ... their longest portion
+  const int32_t* exp_lo = nullptr;      // [n_seqs]
+  const int32_t* exp_start = nullptr;   // [n_seqs] position of the portion's first token, from exp_lo
+  const int32_t* exp_lens = nullptr;    // [n_seqs]
+  const int32_t* exp_tables = nullptr;  // [n_seqs][exp_max_blocks]
+  int exp_max_blocks = 0, exp_blocks = 0;
+  const int32_t* key_seq = nullptr;     // [n_keys] of every expanded key: sequence, position from exp_lo
+  const int32_t* key_pos = nullptr;
+  int n_keys = 0;
 };
+constexpr int kExpandBlock = 64;        // tokens of a block of the expanded pool
+constexpr int kExpandPortion = 64;      // a portion of at least this many tokens is expanded
 
 // ---- multi-map attention (pi_attention_maps.cu) -----------------------------------------------------------------
 // Per query head `maps` softmax maps over the same values.  maps == 1: plain attention.  maps == 2: the difference
@@ -45,6 +63,9 @@ struct pi_maps_attention {
   int window = 0;                       // <= 0: everything before
   float scale = 1.f, eps = 0.f;
   float lambda = 0.f, out_scale = 1.f;  // maps == 2
+  const float* gate = nullptr;          // the result is multiplied by sigmoid(gate[row][heads * vdim])
+  size_t gate_stride = 0;
+  bool v_in_k = false;                  // the values are the first channels of the keys (f32 kernel)
   int rot_dims = 0;
   const float* rope_cos = nullptr;      // [positions][rot_dims / 2]
   const float* rope_sin = nullptr;
@@ -59,6 +80,105 @@ pi_status pi_launch_maps_rope_kv(pi_ctx* ctx, const pi_maps_attention& a, const 
 // out[row][heads * vdim] as f32 or bf16 (out_kind).
 pi_status pi_launch_maps_attention(pi_ctx* ctx, const pi_maps_attention& a, const pi_kv_view& kv, const float* qkv, size_t stride,
                                    void* out, size_t out_stride, int out_kind, const pi_seq_batch& b);
+
+// ---- latent attention (pi_latent.cu) ------------------------------------------------------------------------------
+// Keys and values of all heads are linear in one latent vector c per token; beside it a rotated key part common to the
+// heads.  Only these two are cached: pool rows [c, padded to 16 | rotated part, padded to 16], one kv head, no V part.
+struct pi_latent_attention {
+  int heads = 0, dim = 0, rot_dims = 0, vdim = 0, rank = 0, window = 0;
+  float scale = 1.f, eps = 0.f;
+  const float* norm = nullptr;          // [rank]
+  const pi_linear* uk_t = nullptr;      // [heads * rank][dim]: a head's unrotated query into latent space
+  const pi_linear* ukv = nullptr;       // [heads * dim + heads * vdim][rank]
+  const float* rope_cos = nullptr;      // [positions][rot_dims / 2]
+  const float* rope_sin = nullptr;
+  int col_q = 0, col_kv = 0, col_g = 0; // columns of the fused projection: queries [head][dim | rot], [c | rotated key], gate
+};
+struct pi_latent_scratch {
+  void* q = nullptr;                    // [rows][heads][dp] queries in the layout of a pool row, pool's type
+  void* o = nullptr;                    // [rows][heads][rank] weighted latents
+  __nv_bfloat16 *keys = nullptr, *pool = nullptr;   // expanded portions: latents of the keys [n_keys][rp], scratch pool
+};
+inline int pi_latent_rp(int rank) { return (rank + 15) / 16 * 16; }
+inline int pi_latent_dp(int rank, int rot) { return pi_latent_rp(rank) + (rot + 15) / 16 * 16; }
+bool pi_latent_expandable(const pi_ctx* ctx, const pi_latent_attention& a, int compute);
+bool pi_latent_supported(const pi_ctx* ctx, const pi_latent_attention& a, int compute);
+size_t pi_latent_pool_elems(const pi_latent_attention& a, int blocks);   // scratch pool of that many blocks
+// out[row][heads * vdim], gated, as f32 or bf16 (out_kind).
+pi_status pi_launch_latent_attention(pi_ctx* ctx, const pi_latent_attention& a, const pi_kv_view& kv, float* proj, size_t stride, void* out,
+                                     size_t out_stride, int out_kind, const pi_seq_batch& b, const pi_latent_scratch& s);
+
+// ---- state-space recurrence (pi_ssd.cu, pi_ssd_chunk.cu) ---------------------------------------------------------------
+struct pi_ssd {
+  int heads = 0, vdim = 0, dim = 0, groups = 1, norm_groups = 1, taps = 1;   // dim: state channels
+  float eps = 0.f;
+  const float *conv = nullptr, *conv_b = nullptr;   // [channels][taps], [channels]; channels: x, B, C
+  const float *dt_bias = nullptr, *a_log = nullptr, *d = nullptr;   // [heads]
+  const float* norm = nullptr;          // [heads * vdim]
+  int col_z = 0, col_x = 0, col_dt = 0; // columns of the fused projection: z | x, B, C | dt
+  // state: per slot S [heads][dim][vdim], then the convolution's last inputs [taps - 1][channels]
+  float* state = nullptr;
+  size_t state_stride = 0, state_off = 0;
+  __host__ __device__ int inner() const { return heads * vdim; }
+  __host__ __device__ int channels() const { return heads * vdim + 2 * groups * dim; }
+  size_t state_floats() const { return ((size_t)heads * dim * vdim + (size_t)(taps - 1) * channels() + 31) / 32 * 32; }
+};
+// y: f32 scratch [rows][heads * vdim]; out: the gated, normalised result.
+pi_status pi_launch_ssd(pi_ctx* ctx, const pi_ssd& r, const float* proj, size_t stride, float* y, void* out, size_t out_stride, int out_kind,
+                        const pi_seq_batch& b, float* scratch);
+size_t pi_ssd_scratch_floats(const pi_ssd& r, int n_chunks);
+bool pi_ssd_chunked(const pi_ctx* ctx, const pi_ssd& r, int compute);
+pi_status pi_launch_ssd_chunks(pi_ctx* ctx, const pi_ssd& r, const float* proj, size_t stride, float* y, const pi_seq_batch& b, float* scratch);
+
+// ---- experts (pi_moe.cu; the products are pi_linear with pi_expert_rows) ---------------------------------------------------
+struct pi_moe {
+  int experts = 0, top = 0, groups = 1, keep = 1;
+  const float* correction = nullptr;    // [experts], part of the choice and not of the weights
+};
+struct pi_moe_lists {
+  int32_t* ids = nullptr;               // [rows][top]
+  float* weights = nullptr;             // [rows][top]
+  int32_t *place = nullptr, *pair_at = nullptr;   // [rows * top] where a pair lies among the rows grouped by expert, and back
+  int4* tiles = nullptr;
+  int32_t* n_tiles = nullptr;
+};
+int pi_moe_tile_rows(int rows, const pi_moe& m);
+int pi_moe_max_tiles(int rows, const pi_moe& m);
+pi_status pi_launch_moe_route(pi_ctx* ctx, const pi_moe& m, const float* logits, size_t stride, int rows, const pi_moe_lists& l);
+pi_status pi_launch_moe_gather(pi_ctx* ctx, const pi_moe& m, int rows, const pi_moe_lists& l, const __nv_bfloat16* h, size_t ld_h, __nv_bfloat16* out);
+
+// ---- rows: residual stream and layer norm (pi_rows.cu) -------------------------------------------------------------------
+struct pi_layer_norm {
+  const float* w = nullptr;
+  float eps = 0.f;
+};
+// scale (sum over k of weights[row][k] y[place[row][k]] + sigmoid(shared_gate[row]) shared[row])
+struct pi_expert_sum {
+  int top = 0;
+  const float* weights = nullptr;
+  const int32_t* place = nullptr;       // null: row * top + k
+  const void* y = nullptr;
+  int y_bf16 = 0;
+  size_t y_stride = 0;
+  const float *shared = nullptr, *shared_gate = nullptr;
+  size_t shared_stride = 0, shared_gate_stride = 0;
+  const float* scale = nullptr;         // [width]
+};
+struct pi_row_norm {
+  int rows = 0, width = 0;
+  float* x = nullptr;                   // [.][width]
+  const int32_t* pick = nullptr;        // row i is x[pick[i]]
+  const uint16_t* table = nullptr;      // x = table[token] first (the first kernel of a step)
+  size_t table_ld = 0;
+  int vocab = 0;
+  const uint32_t* tokens = nullptr;
+  const pi_expert_sum* experts = nullptr;   // x += experts first
+  pi_layer_norm norm;
+  void* h = nullptr;                    // null: no normalised row is wanted
+  size_t ld_h = 0;
+  int h_kind = PI_F32;
+};
+pi_status pi_launch_row_norm(pi_ctx* ctx, const pi_row_norm& n);
 
 // ---- recurrences (pi_recurrent.cu) --------------------------------------------------------------------------------
 enum pi_recurrence_kind { PI_REC_GLA = 0, PI_REC_MLSTM = 1 };

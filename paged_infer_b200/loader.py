@@ -74,7 +74,9 @@ class LlamaConfig:
             "intermediate_size", "vocab_size", "rms_norm_eps", "rope_theta", "attention_window", "rope_style")}
 
 
-MIXER_ATTENTION, MIXER_GLA, MIXER_MLSTM = 0, 1, 2
+MIXER_ATTENTION, MIXER_GLA, MIXER_MLSTM, MIXER_LATENT, MIXER_SSD = 0, 1, 2, 3, 4
+FF_GELU, FF_SILU, FF_EXPERTS = 0, 1, 2
+NORM_DYT, NORM_LAYER = 0, 1
 
 
 @dataclass
@@ -82,7 +84,10 @@ class LayerConfig:
     """One layer of a layered design: a token mixer with its own sizes and, if ``ff``, a gated feed-forward.
 
     ``window`` None: everything before.  ``maps`` 2: differential attention (``diff`` its constant).  ``tau`` belongs to the
-    gated linear recurrence, ``gate_cap`` to the matrix memory."""
+    gated linear recurrence, ``gate_cap`` to the matrix memory.  Latent attention: ``rank`` latent channels, ``dim`` unrotated and
+    ``rot_dims`` rotated channels per head, rotation stretched by ``rot_factor`` and the three constants behind it.  State-space
+    recurrence: ``dim`` state channels, heads in ``groups``, ``conv`` taps, ``norm_groups`` parts.  Routed experts: ``ff`` is one
+    expert's size, ``shared_ff`` that of the expert every token meets."""
 
     mixer: int
     heads: int
@@ -98,6 +103,22 @@ class LayerConfig:
     tau: float = 1.0
     gate_cap: float = 1.0
     ff: int = 0
+    ff_kind: int = FF_GELU
+    rank: int = 0
+    rot_factor: float = 1.0
+    rot_original: float = 1.0
+    rot_fast: float = 32.0
+    rot_slow: float = 1.0
+    groups: int = 1
+    norm_groups: int = 1
+    conv: int = 1
+    experts: int = 0
+    top: int = 0
+    expert_groups: int = 1
+    keep_groups: int = 1
+    shared_ff: int = 0
+    limit: float = 0.0
+    shared_limit: float = 0.0
 
 
 @dataclass
@@ -108,10 +129,13 @@ class LayeredConfig:
     vocab_size: int
     norm_eps: float
     layers: list
+    norm: int = NORM_DYT
+    tied: bool = True
+    logit_scale: float = 1.0
 
     @property
     def has_state(self) -> bool:
-        return any(l.mixer != MIXER_ATTENTION for l in self.layers)
+        return any(l.mixer not in (MIXER_ATTENTION, MIXER_LATENT) for l in self.layers)
 
     @classmethod
     def from_sumosun(cls, j: dict) -> "LayeredConfig":
@@ -135,6 +159,47 @@ class LayeredConfig:
             else:
                 raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
         return cls(width=int(j["width"]), vocab_size=int(j["vocab"]), norm_eps=float(j["norm"]["eps"]), layers=layers)
+
+    @classmethod
+    def from_lilosun(cls, j: dict) -> "LayeredConfig":
+        """The Lilosun design's ``config.json``: latent attention and Mamba-2 layers in any order, each with a dense or a routed
+        feed-forward or none."""
+        layers = []
+        for i, e in enumerate(j["layers"]):
+            m = e["mixer"]
+            kw = dict(heads=int(m["heads"]), vdim=int(m["vdim"]), **cls._lilosun_feed_forward(i, e.get("mlp")))
+            if e["type"] == "latent_attention":
+                mask, rot = m.get("mask"), m["rot"]
+                if int(rot["dims"]) != int(m["rot_dim"]):
+                    raise ValueError(f"layer {i}: {rot['dims']} rotated channels, the rotated part has {m['rot_dim']}")
+                scaling = rot.get("scaling")
+                if scaling:
+                    kw.update(rot_factor=float(scaling["factor"]), rot_original=float(scaling["original"]), rot_fast=float(scaling["fast"]),
+                              rot_slow=float(scaling["slow"]))
+                layers.append(LayerConfig(MIXER_LATENT, dim=int(m["dim"]), rank=int(m["kv_rank"]), window=int(mask["size"]) if mask else None,
+                                          rot_dims=int(m["rot_dim"]), rot_base=float(rot["base"]), scale=float(m["scale"]), **kw))
+            elif e["type"] == "mamba2":
+                layers.append(LayerConfig(MIXER_SSD, dim=int(m["state"]), groups=int(m["groups"]), norm_groups=int(m["norm_groups"]), conv=int(m["conv"]), **kw))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+        return cls(width=int(j["width"]), vocab_size=int(j["vocab"]), norm_eps=float(j["norm"]["eps"]), layers=layers, norm=NORM_LAYER, tied=False,
+                   logit_scale=float(j["logit_scale"]))
+
+    @staticmethod
+    def _lilosun_feed_forward(i: int, mlp: dict | None) -> dict:
+        if mlp is None:
+            return {}
+        if mlp["kind"] == "dense":
+            return dict(ff=int(mlp["ff"]), ff_kind=FF_SILU)
+        if mlp["kind"] != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        r, groups, shared = mlp["router"], mlp["router"].get("groups"), mlp.get("shared")
+        kw = dict(ff=int(mlp["expert"]["ff"]), ff_kind=FF_EXPERTS, limit=float(mlp["expert"]["limit"]), experts=int(r["experts"]), top=int(r["top"]))
+        if groups:
+            kw.update(expert_groups=int(groups["count"]), keep_groups=int(groups["keep"]))
+        if shared:
+            kw.update(shared_ff=int(shared["ff"]), shared_limit=float(shared["limit"]))
+        return kw
 
 
 def read_safetensors(path: str) -> dict:

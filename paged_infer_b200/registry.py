@@ -32,16 +32,19 @@ def _load_llama(ctx, folder, config, dtype, max_rows, quantization):
     return api.LlamaWeights(ctx, cfg, load_weights(_weights_file(folder), cfg), max_batch=max_rows)
 
 
-def _load_sumosun(ctx, folder, config, dtype, max_rows, quantization):
-    if quantization != QUANT_F32:
-        raise ValueError("this design keeps its bf16 weights: quantization is not offered")
-    return api.LayeredModel(ctx, LayeredConfig.from_sumosun(config), read_safetensors(_weights_file(folder)), dtype, max_rows)
+def _layered(read_config):
+    def load(ctx, folder, config, dtype, max_rows, quantization):
+        if quantization != QUANT_F32:
+            raise ValueError("this design keeps its bf16 weights: quantization is not offered")
+        return api.LayeredModel(ctx, read_config(config), read_safetensors(_weights_file(folder)), dtype, max_rows)
+    return load
 
 
 FAMILIES = {
     # activations and KV are f32 throughout, the bf16 checkpoint widens exactly
     "Llama": Family(_load_llama, ("float32",)),
-    "Sumosun": Family(_load_sumosun, ("bfloat16", "float32")),
+    "Sumosun": Family(_layered(LayeredConfig.from_sumosun), ("bfloat16", "float32")),
+    "Lilosun": Family(_layered(LayeredConfig.from_lilosun), ("bfloat16", "float32")),
 }
 
 
