@@ -315,6 +315,23 @@ def route(z, correction, top, groups, keep):
     return ids, w / (w.sum(-1, keepdims=True) + 1e-20)
 
 
+def route_margin(z, correction, top, groups, keep):
+    """By how much the choice scores of every token would have to move to change what ``route`` chooses: the gap behind the
+    last group that is kept, or behind the last expert that is chosen."""
+    choice = sigmoid(z) + correction
+    n = z.shape[1] // groups
+    out = np.full(z.shape[0], np.inf)
+    for t in range(z.shape[0]):
+        best = np.array([np.sort(choice[t, g * n:(g + 1) * n])[-2:].sum() for g in range(groups)])
+        order = np.argsort(best)[::-1]
+        if keep < groups:
+            out[t] = (best[order[keep - 1]] - best[order[keep]]) / 2
+        c = np.sort(np.concatenate([choice[t, g * n:(g + 1) * n] for g in order[:keep]]))[::-1]
+        if top < len(c):
+            out[t] = min(out[t], c[top - 1] - c[top])
+    return out
+
+
 def moe(h, w, top, groups, keep, limit, shared_limit):
     """w: dict router, correction, e<i>.gate/up/down and, with a shared expert, shared.gate/up/down/sg."""
     ids, weights = route(linear(w["router"], h), w["correction"], top, groups, keep)
@@ -334,6 +351,7 @@ class Lilosun:
     def __init__(self, config: dict, tensors: dict, dtype=np.float64):
         self.c = config
         self.t = {k: np.asarray(v, dtype) for k, v in tensors.items()}
+        self.margin = None    # per token of the last forward: the closest call of any router
 
     def part(self, prefix):
         return {k[len(prefix):]: v for k, v in self.t.items() if k.startswith(prefix)}
@@ -354,12 +372,14 @@ class Lilosun:
             return silu_mlp(h, w["gate"], w["up"], w["down"])
         r, g = mlp["router"], mlp["router"].get("groups") or {"count": 1, "keep": 1}
         shared = mlp.get("shared")
+        self.margin = np.minimum(self.margin, route_margin(linear(w["router"], h), w["correction"], r["top"], g["count"], g["keep"]))
         return moe(h, w, r["top"], g["count"], g["keep"], mlp["expert"]["limit"], shared["limit"] if shared else None)
 
     def forward(self, tokens, layer_outputs: list | None = None):
         """Logits [tokens, vocab] of one sequence from its first token."""
         eps = self.c["norm"]["eps"]
         x = self.t["embed"][np.asarray(tokens)]
+        self.margin = np.full(len(tokens), np.inf)
         for i, layer in enumerate(self.c["layers"]):
             l = f"l{i}."
             x = x + self.t[l + "ls1"] * self.mixer(i, layer, layer_norm(x, self.t[l + "norm1"], eps))

@@ -1,4 +1,4 @@
-"""Small random checkpoints of the Sumosun design for the tests: configurations, tensors under the checkpoint's names
+"""Small random checkpoints of the layered designs for the tests: configurations, tensors under the checkpoint's names
 (values that bf16 represents exactly), the plain reference over them, and a writer for checkpoint folders."""
 from __future__ import annotations
 
@@ -29,8 +29,135 @@ def config(layers, width=64, vocab=96, eps=1e-5):
     return {"architecture": "Sumosun", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
 
 
+# ---- Lilosun ------------------------------------------------------------------------------------------------------------------
+YARN = {"factor": 8.0, "original": 96, "fast": 20.0, "slow": 2.0}
+
+
+def latent(heads=3, dim=20, rot_dim=16, vdim=24, rank=48, window=28, base=10000.0, scaling=YARN, scale=None, mlp=None):
+    rot = {"dims": rot_dim, "base": base}
+    if scaling:
+        rot["scaling"] = scaling
+    return {"type": "latent_attention", "mlp": mlp,
+            "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": rank, "rot": rot,
+                      "scale": (dim + rot_dim) ** -0.5 if scale is None else scale, "mask": {"size": window} if window else None}}
+
+
+def mamba2(heads=6, vdim=20, state=24, groups=2, norm_groups=3, conv=3, mlp=None):
+    return {"type": "mamba2", "mlp": mlp,
+            "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "norm_groups": norm_groups, "conv": conv}}
+
+
+def dense(ff=72):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts=12, top=3, ff=40, limit=1.2, groups=(3, 2), shared=56, shared_limit=0.8):
+    r = {"experts": experts, "top": top}
+    if groups:
+        r["groups"] = {"count": groups[0], "keep": groups[1]}
+    return {"kind": "moe", "router": r, "expert": {"ff": ff, "limit": limit}, "shared": {"ff": shared, "limit": shared_limit} if shared else None}
+
+
+def lilosun(layers, width=88, vocab=400, eps=1e-5, logit_scale=1.5):
+    return {"architecture": "Lilosun", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width, "logit_scale": logit_scale}
+
+
+CODE = 16   # leading channels of the embedding that only the routers and norms see change: no sublayer writes them
+
+
+def lilosun_tensors(cfg, seed):
+    """Random tensors on the bf16 grid.  Routers read the leading channels, which carry a code per token that no sublayer touches, so
+    that (for the tokens of ``clear_tokens``) no choice hangs on a rounding."""
+    rng = np.random.default_rng(seed)
+    W, V = cfg["width"], cfg["vocab"]
+    t = {}
+
+    def put(name, shape, std=None, mean=0.0):
+        x = rng.standard_normal(shape) * (1.0 / np.sqrt(shape[-1]) if std is None else std) + mean
+        t[name] = bf16_bits_to_f32(f32_to_bf16_bits(np.asarray(x, np.float32))).reshape(shape)
+
+    def gated(p, F):
+        put(p + "gate", (F, W), 2.0 / np.sqrt(W))
+        put(p + "up", (F, W), 1.5 / np.sqrt(W))
+        put(p + "down", (W, F), 1.2 / np.sqrt(F))
+        t[p + "down"][:CODE] = 0
+
+    put("embed", (V, W), 1.0, 0.1)
+    t["embed"][:, :CODE] *= 1.5
+    for i, e in enumerate(cfg["layers"]):
+        m, l = e["mixer"], f"l{i}."
+        p = l + "mix."
+        put(l + "norm1", (W,), 0.2, 1.0)
+        put(l + "ls1", (W,), 0.2, 0.5)
+        H, E = m["heads"], m["vdim"]
+        if e["type"] == "latent_attention":
+            D, R, K = m["dim"], m["rot_dim"], m["kv_rank"]
+            put(p + "q", (H * (D + R), W), 1.5 / np.sqrt(W))
+            put(p + "dkv", (K + R, W), 1.5 / np.sqrt(W))
+            put(p + "dkv.norm", (K,), 0.2, 1.0)
+            put(p + "uk", (H * D, K))
+            put(p + "uv", (H * E, K))
+            put(p + "g", (H * E, W))
+        else:
+            N, G = m["state"], m["groups"]
+            ch = H * E + 2 * G * N
+            put(p + "in", (H * E + ch + H, W))
+            put(p + "conv", (ch, m["conv"]), 0.6)
+            put(p + "conv.b", (ch,), 0.3)
+            put(p + "dt_bias", (H,), 1.0, -2.0)
+            put(p + "A_log", (H,), 1.0)
+            put(p + "D", (H,), 0.5, 0.5)
+            put(p + "norm", (H * E,), 0.2, 1.0)
+        put(p + "o", (W, H * E), 1.5 / np.sqrt(H * E))
+        t[p + "o"][:CODE] = 0
+        f = e["mlp"]
+        if f:
+            put(l + "norm2", (W,), 0.2, 1.0)
+            put(l + "ls2", (W,), 0.2, 0.5)
+            p = l + "mlp."
+            if f["kind"] == "dense":
+                gated(p, f["ff"])
+            else:
+                n = f["router"]["experts"]
+                put(p + "router", (n, W), 0.9)
+                t[p + "router"][:, CODE:] = 0
+                put(p + "correction", (n,), 0.3, -0.2)
+                for k in range(n):
+                    gated(f"{p}e{k}.", f["expert"]["ff"])
+                if f.get("shared"):
+                    gated(p + "shared.", f["shared"]["ff"])
+                    put(p + "shared.sg", (1, W), 1.0 / np.sqrt(W))
+    put("final.norm", (W,), 0.2, 1.0)
+    put("head", (V, W))
+    return t
+
+
+def clear_tokens(cfg, t, margin=0.05):
+    """Token ids whose experts are chosen by a clear margin in every layer."""
+    r = reference(cfg, t)
+    r.forward(np.arange(cfg["vocab"]))
+    ids = np.flatnonzero(r.margin > margin)
+    assert len(ids) >= 12, len(ids)
+    return ids
+
+
+def draw(cfg, t, n, seed):
+    """n random tokens, every choice of an expert clear where they stand."""
+    rng, ids, r = np.random.default_rng(seed), clear_tokens(cfg, t), reference(cfg, t)
+    toks = rng.choice(ids, n)
+    for _ in range(30):
+        r.forward(toks)
+        close = np.flatnonzero(r.margin < 0.02)
+        if not len(close):
+            return toks.tolist()
+        toks[close] = rng.choice(ids, len(close))
+    raise AssertionError(f"{len(close)} close calls are left")
+
+
 def tensors(cfg, seed, rank=5):
     """Random tensors (f32 values on the bf16 grid), scaled so that every part of the model moves the logits."""
+    if cfg["architecture"] == "Lilosun":
+        return lilosun_tensors(cfg, seed)
     rng = np.random.default_rng(seed)
     W, V = cfg["width"], cfg["vocab"]
     t = {}
@@ -103,13 +230,18 @@ def write_checkpoint(folder, cfg, t):
 
 
 def reference(cfg, t):
-    from oracle.layers import Sumosun
-    return Sumosun(cfg, t)
+    """The plain reference over the values the checkpoint holds."""
+    from oracle import layers
+    return getattr(layers, cfg["architecture"])(cfg, {k: bf16_bits_to_f32(v).reshape(np.shape(v)) for k, v in bits(t).items()})
 
 
 def device_model(ctx, cfg, t, compute, max_rows=1024):
     from paged_infer_b200 import api
-    return api.LayeredModel(ctx, LayeredConfig.from_sumosun(cfg), bits(t), compute, max_rows)
+    return api.LayeredModel(ctx, layered_config(cfg), bits(t), compute, max_rows)
+
+
+def layered_config(cfg):
+    return LayeredConfig.from_lilosun(cfg) if cfg["architecture"] == "Lilosun" else LayeredConfig.from_sumosun(cfg)
 
 
 def distance(got, want):
