@@ -920,13 +920,68 @@ LAYERED_SIZES = {
 }
 
 
-def layered_config(size):
+def layered_config(size, layers=None):
     from paged_infer_b200 import loader as ld
     s = LAYERED_SIZES[size]
     kinds = [ld.LayerConfig(ld.MIXER_ATTENTION, maps=2, window=s["window"], rot_dims=64, rot_base=500000.0, scale=0.125, diff=0.5, ff=s["ff"], **s["attention"]),
              ld.LayerConfig(ld.MIXER_GLA, tau=16.0, ff=s["ff"], **s["gla"]),
              ld.LayerConfig(ld.MIXER_MLSTM, gate_cap=15.0, ff=s["ff"], **s["mlstm"])]
-    return ld.LayeredConfig(s["width"], s["vocab"], 1e-6, [kinds[i % 3] for i in range(s["layers"])])
+    return ld.LayeredConfig(s["width"], s["vocab"], 1e-6, [kinds[i % 3] for i in range(layers or s["layers"])])
+
+
+# Lilosun beside Sumosun: the same width, depth, vocabulary and window; what a token meets of a layer's experts (top of them and
+# the shared one) adds up to the dense feed-forward's size.
+LILOSUN_SIZES = {
+    "w2048": dict(width=2048, vocab=32000, layers=12, window=1024, dense=5632,
+                  latent=dict(heads=16, dim=128, rot_dims=64, vdim=128, rank=512), ssd=dict(heads=64, vdim=64, dim=128, groups=1, norm_groups=1, conv=4),
+                  moe=dict(experts=64, top=6, ff=704, expert_groups=8, keep_groups=4, shared_ff=1408), like="w2048"),
+    "w4096": dict(width=4096, vocab=32000, layers=6, window=1024, dense=14336,
+                  latent=dict(heads=32, dim=128, rot_dims=64, vdim=128, rank=512), ssd=dict(heads=128, vdim=64, dim=128, groups=8, norm_groups=8, conv=4),
+                  moe=dict(experts=32, top=4, ff=2560, expert_groups=4, keep_groups=2, shared_ff=4096), like="w4096"),
+}
+
+
+def lilosun_config(size):
+    from paged_infer_b200 import loader as ld
+    s = LILOSUN_SIZES[size]
+    moe, dense = dict(ff_kind=ld.FF_EXPERTS, limit=7.0, shared_limit=7.0, **s["moe"]), dict(ff_kind=ld.FF_SILU, ff=s["dense"])
+    attn = dict(window=s["window"], rot_base=50000.0, rot_factor=4.0, rot_original=4096, scale=192 ** -0.5, **s["latent"])
+    kinds = [ld.LayerConfig(ld.MIXER_LATENT, **attn, **moe), ld.LayerConfig(ld.MIXER_SSD, **s["ssd"], **dense), ld.LayerConfig(ld.MIXER_SSD, **s["ssd"], **moe)]
+    return ld.LayeredConfig(s["width"], s["vocab"], 1e-6, [kinds[i % 3] for i in range(s["layers"])], norm=ld.NORM_LAYER, tied=False)
+
+
+def lilosun_work(cfg, model, B, ctx_len, M):
+    """As layered_work; experts count as far as tokens meet them (B tokens of a decode step: the expected number of different ones)."""
+    from paged_infer_b200 import loader as ld
+    W = cfg.width
+    attn = [l for l in cfg.layers if l.mixer == ld.MIXER_LATENT]
+    rec = [l for l in cfg.layers if l.mixer == ld.MIXER_SSD]
+    inner = lambda l: l.heads * l.vdim
+    per_expert = lambda l: 3 * W * l.ff
+    fixed = flops = absorbed = 0
+    met = 0.0
+    for l in cfg.layers:
+        if l.mixer == ld.MIXER_LATENT:
+            own = W * (l.heads * (l.dim + l.rot_dims) + l.rank + l.rot_dims + 2 * inner(l))
+            absorbed += l.rank * l.heads * (l.dim + l.vdim)
+        else:
+            own = W * (3 * inner(l) + 2 * l.groups * l.dim + l.heads)
+        active = 0
+        if l.ff_kind == ld.FF_EXPERTS:
+            own += W * (3 * l.shared_ff + l.experts + 1)
+            active = l.top * per_expert(l)
+            met += per_expert(l) * l.experts * (1 - (1 - l.top / l.experts) ** B)
+        else:
+            own += 3 * W * l.ff
+        fixed += own
+        flops += own + active
+    seen = sum(min(t + 1, attn[0].window) for t in range(M))
+    row = lambda l: l.rank + l.rot_dims
+    return {"decode_bytes": {"projections": 2 * (fixed + met + cfg.vocab_size * W), "attention": sum(B * min(ctx_len, l.window) * row(l) * 2 for l in attn),
+                             "recurrence": 2 * B * model.state_bytes()},
+            "prefill_flops": {"gemm_tc": 2.0 * M * (flops + absorbed), "attention": sum(l.heads * 2 * (l.dim + l.rot_dims + l.vdim) * seen for l in attn)},
+            # f32 projections in, the gated sums to and from the norm, bf16 result out, and the states between chunks of 64 tokens written and read once
+            "prefill_bytes": {"recurrence": sum(M * (4 * (2 * inner(l) + 2 * l.groups * l.dim + l.heads) + 10 * inner(l)) + 8 * (M // 64) * inner(l) * l.dim for l in rec)}}
 
 
 def layered_work(cfg, model, B, ctx_len, M):
@@ -1040,7 +1095,8 @@ def measure_steps(api, ctx, torch, model, work, ctx_len, batches, M, K, W, peaks
 
 def run_layered_workload(args):
     """`--workload sumosun`: prefill and decode of the layered design at a few sizes, beside a Llama of the same width, depth,
-    feed-forward and vocabulary (random weights; bf16 there, int8 weights with f32 activations and KV here)."""
+    feed-forward and vocabulary (random weights; bf16 there, int8 weights with f32 activations and KV here).
+    `--workload lilosun`: Lilosun beside Sumosun, its closest model, both in bf16."""
     import torch
     from paged_infer_b200 import api
     from paged_infer_b200.loader import LlamaConfig
@@ -1053,20 +1109,28 @@ def run_layered_workload(args):
     clocks.start()
     t0 = time.time()
     res, launches = {}, ctx.kernel_launches()
-    for size, s in LAYERED_SIZES.items():
-        cfg = layered_config(size)
+    measure = lambda m, work: measure_steps(api, ctx, torch, m, work, ctx_len, batches, M, K, W, (hbm, tflops))
+    name = args.workload
+    sizes = LILOSUN_SIZES if name == "lilosun" else LAYERED_SIZES
+    for size, s in sizes.items():
+        cfg, work = (lilosun_config(size), lilosun_work) if name == "lilosun" else (layered_config(size), layered_work)
         m = api.LayeredModel.synthetic(ctx, cfg, seed=1, max_rows=M)
-        res[size] = {"sumosun": measure_steps(api, ctx, torch, m, lambda B, c, n: layered_work(cfg, m, B, c, n), ctx_len, batches, M, K, W, (hbm, tflops))}
+        res[size] = {name: measure(m, lambda B, c, n: work(cfg, m, B, c, n))}
         m.close()
-        lc = LlamaConfig(num_hidden_layers=s["layers"], vocab_size=s["vocab"], rms_norm_eps=1e-5, rope_theta=10000.0, quantization="int8", **s["llama"])
-        u = api.LlamaWeights.synthetic(ctx, lc, seed=1, std=0.02, max_batch=M, max_positions=M + 16)
-        res[size]["llama_int8"] = measure_steps(api, ctx, torch, u, lambda B, c, n: uniform_work(lc, u, B, c, n), ctx_len, batches, M, K, W, (hbm, tflops))
+        if name == "lilosun":
+            lc = layered_config(s["like"], s["layers"])
+            u = api.LayeredModel.synthetic(ctx, lc, seed=1, max_rows=M)
+            res[size]["sumosun"] = measure(u, lambda B, c, n: layered_work(lc, u, B, c, n))
+        else:
+            lc = LlamaConfig(num_hidden_layers=s["layers"], vocab_size=s["vocab"], rms_norm_eps=1e-5, rope_theta=10000.0, quantization="int8", **s["llama"])
+            u = api.LlamaWeights.synthetic(ctx, lc, seed=1, std=0.02, max_batch=M, max_positions=M + 16)
+            res[size]["llama_int8"] = measure(u, lambda B, c, n: uniform_work(lc, u, B, c, n))
         u.close()
     t1 = time.time()
-    best = res["w2048"]["sumosun"]["decode_b64"]
+    best = res["w2048"][name]["decode_b64"]
     print(json.dumps({"metric": "layered design: decode tokens/s at batch 64 (w2048)", "value": best["tok/s"], "unit": "tok/s", "n_gpus": 1, "steps": K,
                       "warmup": W, "ms_per_step": best["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
-                      "data": "synthetic", "config": {"model": "sumosun", "sizes": LAYERED_SIZES, "context": ctx_len, "prefill": M,
+                      "data": "synthetic", "config": {"model": name, "sizes": sizes, "context": ctx_len, "prefill": M,
                                                       "l2": "decode inputs exceed L2; flushed between prefill repetitions"},
                       "gpu_launches": int(ctx.kernel_launches() - launches), "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind},
                       "clocks": clocks.stop(t0, t1), "results": res}), flush=True)
@@ -1081,7 +1145,7 @@ def main():
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="tinyllama_b64_paged", choices=["tinyllama_b64_paged", "llama3_8b_tp", "llama2_70b_tp", "sumosun"])
+    ap.add_argument("--workload", default="tinyllama_b64_paged", choices=["tinyllama_b64_paged", "llama3_8b_tp", "llama2_70b_tp", "sumosun", "lilosun"])
     ap.add_argument("--no-cpu", action="store_true", help="skip the cpu_baseline leg")
     ap.add_argument("--resident-only", action="store_true",
                     help="for a profiler's launch list: only the resident decode leg (warm-up + timed steps) over a pool filled with "
@@ -1102,7 +1166,7 @@ def main():
     if args.kernel_case:
         run_kernel_case(args)
         return
-    if args.workload == "sumosun":
+    if args.workload in ("sumosun", "lilosun"):
         run_layered_workload(args)
         return
     if args.workload in TP_WORKLOADS:
