@@ -230,7 +230,7 @@ struct pi_expert_rows {
   const int4* tiles = nullptr;
   const int32_t* n_tiles = nullptr;
   int max_tiles = 0;          // host-side bound
-  int tile_rows = 0;          // rows of a full tile: 16, 32, 64 or 128
+  int tile_rows = 0;          // rows of a full tile: 16, 32, 64, 128 or 256
 };
 
 struct pi_linear_args {

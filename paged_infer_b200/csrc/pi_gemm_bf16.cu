@@ -486,7 +486,7 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
   int bn = a.M <= 16 ? 16 : a.M <= 32 ? 32 : a.M <= 64 ? 64 : 128;
   if (a.M > 128) {   // the wider tile where it does not cost more rounds of tiles over the SMs
     const long t128 = (long)p.rtiles * ((a.M + 127) / 128), t256 = (long)p.rtiles * ((a.M + 255) / 256), sms = ctx->sm_count;
-    if ((t256 + sms - 1) / sms * 2 <= (t128 + sms - 1) / sms) bn = 256;
+    if ((t256 + sms - 1) / sms * 3 <= (t128 + sms - 1) / sms * 2) bn = 256;
   }
   if (ex) {
     bn = ex->tile_rows;
@@ -505,6 +505,7 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
       case 32: e = run_grouped<32, 8>(ctx, p, w, x); break;
       case 64: e = run_grouped<64, 6>(ctx, p, w, x); break;
       case 128: e = run_grouped<128, 4>(ctx, p, w, x); break;
+      case 256: e = run_grouped<256, 4>(ctx, p, w, x); break;
       default: return pi_fail(ctx, PI_ERR_INVALID_ARG, "expert tiles of %d rows are not built", bn);
     }
   } else switch (bn) {

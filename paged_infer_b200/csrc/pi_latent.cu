@@ -12,10 +12,11 @@
 //               spells out keys and values of all heads into a scratch pool, and the windowed tile kernel of multi-map
 //               attention runs on it: a third of the arithmetic per (query, key) pair at a latent of four head sizes.
 //
-// latent_decode_kernel (bf16 pool, mma.sync): CTA = (row, group of 16 heads = the MMA's rows, KV split).  Tiles of 64 keys, two
-// in flight; a warp scores 8 keys over all channels, the softmax meets in shared memory, then every warp sums its own value
-// channels over all 64 keys, so that accumulators never merge inside a CTA.  The weights enter as two bf16 planes (16
-// bits).  Splits of a row form a cluster and merge through distributed shared memory.
+// latent_decode_kernel (bf16 pool, mma.sync): CTA = (row, group of 16 heads = the MMA's rows, KV split).  Tiles of 32 keys, three
+// in flight.  A warp scores 8 keys over half of the channels, its queries in registers; the scores meet in shared memory,
+// every warp forms the weights of all 32 keys for itself and sums its own value channels, so that neither weights nor
+// accumulators are exchanged.  The weights enter as two bf16 planes (16 bits).  Splits of a row form a cluster and merge
+// through distributed shared memory.
 #include <cooperative_groups.h>
 #include <limits.h>
 #include <math.h>
@@ -60,15 +61,38 @@ __device__ __forceinline__ void head_weights(const HeadTile& t, const __nv_bfloa
   }
   cp_async_commit();
 }
-// 16 rows at a time: x(i, k) of row i < rows, use(i, n, value).
+__device__ __forceinline__ float as_f32(float v) { return v; }
+__device__ __forceinline__ float as_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+// 16 rows at a time: x(i) points to the K inputs of row i < rows (f32 or bf16; `vec`: on 16-byte boundaries, K a multiple of 8),
+// use(i, n, value).
 template <typename X, typename F>
-__device__ __forceinline__ void head_rows(const HeadTile& t, int K, int N, int n0, int rows, int z, int nz, X&& x, F&& use) {
+__device__ __forceinline__ void head_rows(const HeadTile& t, int K, int N, int n0, int rows, int z, int nz, bool vec, X&& x, F&& use) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  constexpr bool kF32 = std::is_same<typename std::decay<decltype(*x(0))>::type, float>::value;
   for (int m0 = z * kHeadRows; m0 < rows; m0 += nz * kHeadRows) {
     __syncthreads();     // the last rows have been read
-    for (int i = threadIdx.x; i < kHeadRows * t.kp; i += kHeadThreads) {
-      const int m = i / t.kp, k = i - m * t.kp;
-      t.x[m * t.pitch + k] = __float2bfloat16_rn(m0 + m < rows && k < K ? x(m0 + m, k) : 0.f);
+    if (vec) {
+      const int pieces = t.kp / 8;
+#pragma unroll 4
+      for (int i = threadIdx.x; i < kHeadRows * pieces; i += kHeadThreads) {
+        const int m = i / pieces, k = (i - m * pieces) * 8;
+        const bool ok = m0 + m < rows && k < K;
+        const auto* src = x(min(m0 + m, rows - 1)) + min(k, K - 8);
+        __nv_bfloat16* dst = t.x + m * t.pitch + k;
+        if constexpr (kF32) {
+          const float4 a = *reinterpret_cast<const float4*>(src), b = *reinterpret_cast<const float4*>(src + 4);
+          *reinterpret_cast<uint4*>(dst) = ok ? make_uint4(pack(a.x, a.y), pack(a.z, a.w), pack(b.x, b.y), pack(b.z, b.w)) : make_uint4(0, 0, 0, 0);
+        } else {
+          cp_async16(smem_addr(dst), src, ok ? 16 : 0);
+        }
+      }
+      cp_async_commit();
+    } else {
+      for (int i = threadIdx.x; i < kHeadRows * t.kp; i += kHeadThreads) {
+        const int m = i / t.kp, k = i - m * t.kp;
+        t.x[m * t.pitch + k] = __float2bfloat16_rn(m0 + m < rows && k < K ? as_f32(x(m0 + m)[k]) : 0.f);
+      }
     }
     cp_async_wait<0>();
     __syncthreads();
@@ -141,8 +165,9 @@ __global__ void __launch_bounds__(kHeadThreads) latent_prepare_kernel(const Late
       const HeadTile t = head_tile(smem, p.dim);
       head_weights(t, static_cast<const __nv_bfloat16*>(p.uk_t) + (size_t)head * p.rank * p.uk_ld, p.uk_ld, p.rank, n0);
       pi_grid_dependency_wait();
-      head_rows(t, p.dim, p.rank, n0, p.n_latent, z, p.row_splits,
-                [&](int m, int k) { return p.proj[(size_t)p.latent_rows[m] * p.stride + p.col_q + (size_t)head * qd + k]; },
+      const bool vec = p.dim % 8 == 0 && qd % 4 == 0 && p.stride % 4 == 0 && p.col_q % 4 == 0;
+      head_rows(t, p.dim, p.rank, n0, p.n_latent, z, p.row_splits, vec,
+                [&](int m) { return p.proj + (size_t)p.latent_rows[m] * p.stride + p.col_q + (size_t)head * qd; },
                 [&](int m, int n, float v) { q[((size_t)p.latent_rows[m] * p.heads + head) * p.dp + n] = pi_from_f32<T>(v); });
     }
     return;
@@ -205,8 +230,8 @@ __global__ void __launch_bounds__(kHeadThreads) latent_out_kernel(const LatentPa
   head_weights(t, static_cast<const __nv_bfloat16*>(p.uv) + (size_t)head * p.vdim * p.uv_ld, p.uv_ld, p.vdim, n0);
   pi_grid_dependency_wait();
   const __nv_bfloat16* o = static_cast<const __nv_bfloat16*>(p.o);
-  head_rows(t, p.rank, p.vdim, n0, p.n_latent, blockIdx.z, gridDim.z,
-            [&](int m, int k) { return __bfloat162float(o[((size_t)p.latent_rows[m] * p.heads + head) * p.rank + k]); },
+  head_rows(t, p.rank, p.vdim, n0, p.n_latent, blockIdx.z, gridDim.z, p.rank % 8 == 0,
+            [&](int m) { return o + ((size_t)p.latent_rows[m] * p.heads + head) * p.rank; },
             [&](int m, int n, float v) {
               const size_t row = p.latent_rows[m];
               static_cast<O*>(p.out)[row * p.out_stride + head * p.vdim + n] = pi_from_f32<O>(v * pi_sigmoid(p.proj[row * p.stride + p.col_g + head * p.vdim + n]));
@@ -227,76 +252,83 @@ __global__ void __launch_bounds__(kHeadThreads) latent_out_f32_kernel(const Late
 }
 
 // ---- decode attention over the latents ---------------------------------------------------------------------------------------
-constexpr int kDecWarps = 8, kDecThreads = kDecWarps * 32, kKeys = 64, kStages = 2, kMaxSplits = 8;
-constexpr int kPPitch = kKeys + 8;
+constexpr int kDecWarps = 8, kDecThreads = kDecWarps * 32, kKeys = 32, kStages = 4, kMaxSplits = 8;
+constexpr int kSPitch = kKeys + 4;
 
 struct DecodeSmem {
-  size_t q, ring, p, acc, total;   // byte offsets
+  size_t s, acc, total;            // byte offsets: scores behind the ring; the finished sums take the ring's place
 };
 __host__ __device__ inline DecodeSmem decode_smem(int dp, int rp) {
   DecodeSmem s;
-  const size_t row = (size_t)(dp + 8) * 2;
-  s.q = 0;
-  s.p = 16 * row;
-  s.ring = s.p + 2 * 16 * kPPitch * 2;
-  s.acc = s.ring;                  // the finished sums take the ring's place
-  const size_t ring = kStages * kKeys * row, acc = (size_t)16 * (rp + 4) * 4;
-  s.total = s.ring + (ring > acc ? ring : acc);
+  const size_t ring = (size_t)kStages * kKeys * (dp + 8) * 2, acc = (size_t)16 * (rp + 4) * 4;
+  s.acc = 0;
+  s.s = ring > acc ? ring : acc;
+  s.total = s.s + (size_t)2 * 2 * 16 * kSPitch * 4;
   return s;
 }
 
-// UMAX: units of 16 value channels per warp.
-template <int UMAX>
+// QMAX: steps of 16 channels per warp (half of a row), UMAX: units of 16 value channels per warp.
+template <int QMAX, int UMAX>
 __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const LatentParams p) {
+  static_assert(QMAX % 2 == 0, "two steps per load");
   extern __shared__ __align__(16) unsigned char smem[];
   const DecodeSmem lay = decode_smem(p.dp, p.rp);
-  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem + lay.q);
-  __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(smem + lay.ring);
-  __nv_bfloat16* phi = reinterpret_cast<__nv_bfloat16*>(smem + lay.p);
-  __nv_bfloat16* plo = phi + 16 * kPPitch;
-  __shared__ float s_max[kDecWarps][16], s_l[kDecWarps][16], c_m[16], c_l[16];
+  __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(smem);
+  float* scores = reinterpret_cast<float*>(smem + lay.s);     // [parity][half of the channels][16][kSPitch]
+  __shared__ float c_m[16], c_l[16];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, split_i = blockIdx.x, h0 = blockIdx.z * 16;
   const int row = p.latent_rows[blockIdx.y], seq = p.row_seq[row], pos = p.row_pos[row], settled = p.seq_start[seq];
   const int32_t* table = p.tables + (size_t)seq * p.max_blocks;
   const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(p.base);
-  const int pitch = p.dp + 8, nks = p.dp / 16, units = p.rp / 16;
+  const int pitch = p.dp + 8, units = p.rp / 16;
+  // this warp scores keys 8 (warp % 4).. over its half of the channels
+  const int half = warp >> 2, nks = p.dp / 16, k0 = half ? (nks + 1) / 2 : 0, k1 = half ? nks : (nks + 1) / 2;
 
   const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, hi = min(pos + 1, p.lens[seq] * p.block_size);
   const int t_first = lo / kKeys, n_tiles = max(0, (hi + kKeys - 1) / kKeys - t_first), per = (n_tiles + p.nsplit - 1) / p.nsplit;
   const int tile0 = t_first + split_i * per, tile_end = min(t_first + n_tiles, tile0 + per);
 
-  auto fetch = [&](int tile, int stage) {   // four threads per key
-    const int r = tid >> 2, t = tile * kKeys + r;
-    const bool ok = t < hi;
-    const __nv_bfloat16* src = base;
-    if (ok) {
-      const int lb = t / p.block_size;
-      src = base + ((size_t)table[lb] * p.block_size + (t - lb * p.block_size)) * p.dp;
-    }
-    const uint32_t dst = smem_addr(ring + ((size_t)stage * kKeys + r) * pitch);
-#pragma unroll 4
-    for (int x = (tid & 3) * 8; x < p.dp; x += 32) cp_async16(dst + x * 2, ok ? src + x : base, ok ? 16 : 0);
+  // eight threads per key; its physical block is looked up a tile ahead of the request
+  const int fr = tid >> 3, fx = (tid & 7) * 8;
+  auto block_of = [&](int tile) {
+    const int t = tile * kKeys + fr;
+    return tile < tile_end && t < hi ? table[t / p.block_size] : -1;
   };
+  auto fetch = [&](int tile, int stage, int pb) {
+    const __nv_bfloat16* src = pb >= 0 ? base + ((size_t)pb * p.block_size + (tile * kKeys + fr) % p.block_size) * p.dp : base;
+    const uint32_t dst = smem_addr(ring + ((size_t)stage * kKeys + fr) * pitch);
+#pragma unroll 4
+    for (int x = fx; x < p.dp; x += 64) cp_async16(dst + x * 2, pb >= 0 ? src + x : base, pb >= 0 ? 16 : 0);
+  };
+  int pb[kStages];
+#pragma unroll
+  for (int s = 0; s < kStages; ++s) pb[s] = block_of(tile0 + s);
   // tiles of keys that earlier steps wrote are requested ahead of the dependency wait
-#pragma unroll 1
-  for (int late = 0; late < 2; ++late) {
-    if (late) {
-      pi_grid_dependency_wait();
-      const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + ((size_t)row * p.heads + h0) * p.dp;
-      const int pieces = p.dp / 8, live = min(16, p.heads - h0) * pieces;
-      for (int i = tid; i < 16 * pieces; i += kDecThreads) {
-        const int r = i / pieces;
-        cp_async16(smem_addr(qs + (size_t)r * pitch + (i - r * pieces) * 8), i < live ? q + (size_t)i * 8 : q, i < live ? 16 : 0);
-      }
-    }
-#pragma unroll 1
-    for (int s = 0; s < kStages; ++s) {
-      const int tile = tile0 + s;
-      if (tile < tile_end && ((tile + 1) * kKeys > settled) == (late != 0)) fetch(tile, s);
-      if (late) cp_async_commit();
-    }
+#pragma unroll
+  for (int s = 0; s < kStages - 1; ++s)
+    if (tile0 + s < tile_end && (tile0 + s + 1) * kKeys <= settled) fetch(tile0 + s, s, pb[s]);
+  pi_grid_dependency_wait();
+#pragma unroll
+  for (int s = 0; s < kStages - 1; ++s) {
+    if (tile0 + s < tile_end && (tile0 + s + 1) * kKeys > settled) fetch(tile0 + s, s, pb[s]);
+    cp_async_commit();             // the first group also holds what was requested early
   }
+  int pb_next = pb[kStages - 1];
 
+  uint32_t qa[QMAX][4];
+  {
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + ((size_t)row * p.heads + h0) * p.dp + (lane & 3) * 2;
+    const int r0 = lane >> 2, live = p.heads - h0;
+#pragma unroll
+    for (int k = 0; k < QMAX; ++k)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {   // a0: head, a1: head + 8, a2 / a3: channels + 8; outside: a valid address and zero
+        const int r = r0 + (j & 1) * 8, ks = k0 + k;
+        const bool ok = r < live && ks < k1;
+        const uint32_t v = *reinterpret_cast<const uint32_t*>(q + (ok ? (size_t)r * p.dp + ks * 16 + (j >> 1) * 8 : (size_t)0));
+        qa[k][j] = ok ? v : 0u;
+      }
+  }
   float acc[UMAX][2][4];
 #pragma unroll
   for (int u = 0; u < UMAX; ++u)
@@ -304,82 +336,94 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[u][j][i] = 0.f;
-  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};   // the same in every warp
   const float sc = p.scale * kLog2e;
   const int r0 = lane >> 2;
 
   for (int tile = tile0; tile < tile_end; ++tile) {
-    const int stage = (tile - tile0) % kStages;
+    const int i = tile - tile0, stage = i % kStages;
     const __nv_bfloat16* ks = ring + (size_t)stage * kKeys * pitch;
-    cp_async_wait<kStages - 1>();
-    __syncthreads();
-    // scores of 16 heads x this warp's 8 keys, two chains
-    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+    cp_async_wait<kStages - 2>();
+    __syncthreads();                 // the tile has landed; everybody is done with the tile before it
     {
-      const uint32_t qa = smem_addr(qs + (size_t)((lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (lane >> 4) * 8);
-      const uint32_t kb = smem_addr(ks + (size_t)(warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 8);
-      int k = 0;
-#pragma unroll 4
-      for (; k + 1 < nks; k += 2) {
-        uint32_t a0[4], a1[4], b[4];
-        ldsm4(a0, qa + k * 32);
-        ldsm4(a1, qa + k * 32 + 32);
-        ldsm4(b, kb + k * 32);         // channels 0-7, 8-15 of step k, then of step k + 1
-        mma(s[0], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
-        mma(s[1], a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
-      }
-      if (k < nks) {                   // an odd number of steps
-        uint32_t a0[4], b[4];
-        ldsm4(a0, qa + k * 32);
-        ldsm4(b, smem_addr(ks + (size_t)(warp * 8 + (lane & 7)) * pitch + k * 16 + ((lane >> 3) & 1) * 8));
-        mma(s[0], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
-      }
+      const int next = tile + kStages - 1, now = pb_next;
+      pb_next = block_of(next + 1);
+      if (next < tile_end) fetch(next, (i + kStages - 1) % kStages, now);
+      cp_async_commit();
     }
-    float v[2][2], tm[2];
+    {
+      float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+      const uint32_t kb = smem_addr(ks + (size_t)((warp & 3) * 8 + (lane & 7)) * pitch + k0 * 16 + (lane >> 3) * 8);
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = tile * kKeys + warp * 8 + (lane & 3) * 2 + i;
-        v[h][i] = (t >= lo && t < hi) ? (s[0][2 * h + i] + s[1][2 * h + i]) * sc : -INFINITY;
+      for (int k = 0; k < QMAX; k += 2) {
+        if (k0 + k < k1) {
+          uint32_t b[4];             // channels 0-7, 8-15 of step k, then of step k + 1
+          if (k0 + k + 1 < nks) ldsm4(b, kb + k * 32);
+          else ldsm4(b, kb + k * 32 - (lane >> 4) * 32);
+          mma(s[0], qa[k][0], qa[k][1], qa[k][2], qa[k][3], b[0], b[1]);
+          if (k0 + k + 1 < k1) mma(s[1], qa[k + 1][0], qa[k + 1][1], qa[k + 1][2], qa[k + 1][3], b[2], b[3]);
+        }
       }
-      tm[h] = quad_max(fmaxf(v[h][0], v[h][1]));
-      if ((lane & 3) == 0) s_max[warp][r0 + 8 * h] = tm[h];
+      float* out = scores + (size_t)(((i & 1) * 2 + half) * 16) * kSPitch + (warp & 3) * 8 + (lane & 3) * 2;
+      *reinterpret_cast<float2*>(out + r0 * kSPitch) = make_float2(s[0][0] + s[1][0], s[0][1] + s[1][1]);
+      *reinterpret_cast<float2*>(out + (r0 + 8) * kSPitch) = make_float2(s[0][2] + s[1][2], s[0][3] + s[1][3]);
     }
     __syncthreads();
+    // every warp forms the weights of all 32 keys for itself, in the layout of the product's left operand
+    float w[2][2][4];                // [16 keys][head r0, r0 + 8][keys 0, 1, 8, 9 behind the lane's first]
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const float* a = scores + (size_t)((i & 1) * 32 + r0 + 8 * h) * kSPitch + c * 16 + (lane & 3) * 2 + j * 8;
+          const float2 x = *reinterpret_cast<const float2*>(a), y = *reinterpret_cast<const float2*>(a + 16 * kSPitch);
+          const int t = tile * kKeys + c * 16 + (lane & 3) * 2 + j * 8;
+          w[c][h][2 * j] = t >= lo && t < hi ? (x.x + y.x) * sc : -INFINITY;
+          w[c][h][2 * j + 1] = t + 1 >= lo && t + 1 < hi ? (x.y + y.y) * sc : -INFINITY;
+        }
     float keep[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      float n = mx[h];
+      float n = -INFINITY;
 #pragma unroll
-      for (int w = 0; w < kDecWarps; ++w) n = fmaxf(n, s_max[w][r0 + 8 * h]);
+      for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) n = fmaxf(n, w[c][h][j]);
+      n = fmaxf(mx[h], quad_max(n));
       keep[h] = n == -INFINITY ? 1.f : exp2f(mx[h] - n);
       mx[h] = n;
-      const float ref = n == -INFINITY ? 0.f : n, w0 = exp2f(v[h][0] - ref), w1 = exp2f(v[h][1] - ref);
-      l[h] = l[h] * keep[h] + (w0 + w1);
-      uint32_t hi2, lo2;
-      split(w0, w1, hi2, lo2);
-      const int at = (r0 + 8 * h) * kPPitch + warp * 8 + (lane & 3) * 2;
-      *reinterpret_cast<uint32_t*>(phi + at) = hi2;
-      *reinterpret_cast<uint32_t*>(plo + at) = lo2;
+      const float ref = n == -INFINITY ? 0.f : n;
+      float sum = 0.f;
+#pragma unroll
+      for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          w[c][h][j] = exp2f(w[c][h][j] - ref);
+          sum += w[c][h][j];
+        }
+      l[h] = l[h] * keep[h] + sum;
     }
-    __syncthreads();
+    if (__any_sync(0xffffffffu, keep[0] != 1.f || keep[1] != 1.f)) {
 #pragma unroll
-    for (int u = 0; u < UMAX; ++u)
+      for (int u = 0; u < UMAX; ++u)
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        acc[u][j][0] *= keep[0];
-        acc[u][j][1] *= keep[0];
-        acc[u][j][2] *= keep[1];
-        acc[u][j][3] *= keep[1];
-      }
+        for (int j = 0; j < 2; ++j) {
+          acc[u][j][0] *= keep[0];
+          acc[u][j][1] *= keep[0];
+          acc[u][j][2] *= keep[1];
+          acc[u][j][3] *= keep[1];
+        }
+    }
 #pragma unroll
-    for (int k = 0; k < kKeys / 16; ++k) {
+    for (int c = 0; c < 2; ++c) {
       uint32_t ph[4], pl[4];
-      const int pr = ((lane & 7) + ((lane >> 3) & 1) * 8) * kPPitch + k * 16 + (lane >> 4) * 8;
-      ldsm4(ph, smem_addr(phi + pr));
-      ldsm4(pl, smem_addr(plo + pr));
-      const uint32_t vb = smem_addr(ks + (size_t)(k * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (lane >> 4) * 8);
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) split(w[c][h][2 * j], w[c][h][2 * j + 1], ph[2 * j + h], pl[2 * j + h]);
+      const uint32_t vb = smem_addr(ks + (size_t)(c * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (lane >> 4) * 8);
 #pragma unroll
       for (int u = 0; u < UMAX; ++u) {
         const int unit = warp + u * kDecWarps;
@@ -394,9 +438,6 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
         }
       }
     }
-    __syncthreads();                   // the stage and the weights have been read
-    if (tile + kStages < tile_end) fetch(tile + kStages, stage);
-    cp_async_commit();
   }
   cp_async_wait<0>();
   __syncthreads();
@@ -418,17 +459,10 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     l[h] = quad_sum(l[h]);
-    if ((lane & 3) == 0) {
-      s_l[warp][r0 + 8 * h] = l[h];
-      if (warp == 0) c_m[r0 + 8 * h] = mx[h];
+    if (warp == 0 && (lane & 3) == 0) {
+      c_m[r0 + 8 * h] = mx[h];
+      c_l[r0 + 8 * h] = l[h];
     }
-  }
-  __syncthreads();
-  if (tid < 16) {
-    float t = 0.f;
-#pragma unroll
-    for (int w = 0; w < kDecWarps; ++w) t += s_l[w][tid];
-    c_l[tid] = t;
   }
   cg::cluster_group cluster = cg::this_cluster();
   if (p.nsplit > 1) cluster.sync();
@@ -523,9 +557,12 @@ cudaError_t grant(pi_ctx* ctx, LatentKernel k, size_t smem) {   // a kernel's sh
   return cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
 }
 
-LatentKernel pick_decode(int rp) {
-  const int units = (rp / 16 + kDecWarps - 1) / kDecWarps;
-  return units <= 1 ? latent_decode_kernel<1> : units <= 2 ? latent_decode_kernel<2> : units <= 4 ? latent_decode_kernel<4> : latent_decode_kernel<8>;
+constexpr int kMaxDecodeDp = 768;
+LatentKernel pick_decode(int dp, int rp) {
+  if (rp <= 128 && dp <= 192) return latent_decode_kernel<6, 1>;
+  if (rp <= 256 && dp <= 384) return latent_decode_kernel<12, 2>;
+  if (rp <= 512 && dp <= 576) return latent_decode_kernel<18, 4>;
+  return rp <= 512 ? latent_decode_kernel<24, 4> : latent_decode_kernel<24, 8>;
 }
 
 }  // namespace
@@ -539,7 +576,7 @@ bool pi_latent_expandable(const pi_ctx* ctx, const pi_latent_attention& a, int c
 bool pi_latent_supported(const pi_ctx* ctx, const pi_latent_attention& a, int compute) {
   const int rp = pi_latent_rp(a.rank), dp = pi_latent_dp(a.rank, a.rot_dims);
   if (compute == PI_F32) return ((size_t)dp + 4 * a.rank) * sizeof(float) <= 48 * 1024 && (size_t)a.dim * sizeof(float) <= 48 * 1024;
-  return rp <= 16 * 8 * kDecWarps && decode_smem(dp, rp).total + 4096 <= ctx->smem_optin && std::max(head_smem(a.dim), head_smem(a.rank)) + 1024 <= ctx->smem_optin;
+  return dp <= kMaxDecodeDp && decode_smem(dp, rp).total + 4096 <= ctx->smem_optin && std::max(head_smem(a.dim), head_smem(a.rank)) + 1024 <= ctx->smem_optin;
 }
 
 pi_status pi_launch_latent_attention(pi_ctx* ctx, const pi_latent_attention& a, const pi_kv_view& kv, float* proj, size_t stride, void* out,
@@ -611,7 +648,7 @@ pi_status pi_launch_latent_attention(pi_ctx* ctx, const pi_latent_attention& a, 
     PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(a.heads, b.n_latent), dim3(kHeadThreads), (size_t)a.rank * sizeof(float), 1, p));
   } else if (b.n_latent > 0) {
     p.groups = (a.heads + 15) / 16;
-    const LatentKernel k = pick_decode(p.rp);
+    const LatentKernel k = pick_decode(p.dp, p.rp);
     const size_t smem = decode_smem(p.dp, p.rp).total;
     PI_CUDA(ctx, grant(ctx, k, smem));
     // KV splits: one round of CTAs over the GPU, at least a tile each

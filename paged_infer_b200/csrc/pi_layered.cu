@@ -415,7 +415,17 @@ pi_status build_mixer(pi_ctx* ctx, Loader& ld, int i, int gla_rank, Layer& L, Ex
     r.col_x = (int)core;
     r.col_dt = (int)(core + r.channels());
     PI_TRY(add("in", core + r.channels() + c.heads));
-    PI_TRY(ld.dev_vec(mix + "conv", (size_t)r.channels() * c.conv, &r.conv, 0.25f));
+    std::vector<float> taps;
+    PI_TRY(ld.vec(mix + "conv", (size_t)r.channels() * c.conv, &taps, 0.25f));
+    PI_TRY(ld.upload(taps, &r.conv));
+    if (c.conv <= 4) {
+      std::vector<float> four((size_t)r.channels() * 4, 0.f);
+      for (int ch = 0; ch < r.channels(); ++ch)
+        for (int j = 0; j < c.conv; ++j) four[(size_t)ch * 4 + 4 - c.conv + j] = taps[(size_t)ch * c.conv + j];
+      const float* d;
+      PI_TRY(ld.upload(four, &d));
+      r.conv4 = reinterpret_cast<const float4*>(d);
+    }
     PI_TRY(ld.dev_vec(mix + "conv.b", r.channels(), &r.conv_b));
     PI_TRY(ld.dev_vec(mix + "dt_bias", c.heads, &r.dt_bias, -2.f));
     PI_TRY(ld.dev_vec(mix + "A_log", c.heads, &r.a_log));

@@ -113,6 +113,7 @@ struct pi_ssd {
   int heads = 0, vdim = 0, dim = 0, groups = 1, norm_groups = 1, taps = 1;   // dim: state channels
   float eps = 0.f;
   const float *conv = nullptr, *conv_b = nullptr;   // [channels][taps], [channels]; channels: x, B, C
+  const float4* conv4 = nullptr;        // up to four taps: the same, with zeros in front
   const float *dt_bias = nullptr, *a_log = nullptr, *d = nullptr;   // [heads]
   const float* norm = nullptr;          // [heads * vdim]
   int col_z = 0, col_x = 0, col_dt = 0; // columns of the fused projection: z | x, B, C | dt

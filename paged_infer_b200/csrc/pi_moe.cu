@@ -157,7 +157,7 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* h, size_t 
 
 int pi_moe_tile_rows(int rows, const pi_moe& m) {
   const int mean = (rows * m.top + m.experts - 1) / m.experts;
-  return mean <= 16 ? 16 : mean <= 32 ? 32 : mean <= 64 ? 64 : 128;
+  return mean <= 16 ? 16 : mean <= 32 ? 32 : mean <= 64 ? 64 : mean <= 112 ? 128 : 256;
 }
 int pi_moe_max_tiles(int rows, const pi_moe& m) {
   const int pairs = rows * m.top;

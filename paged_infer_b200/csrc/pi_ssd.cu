@@ -34,8 +34,9 @@ struct ScanParams {
 
 __device__ __forceinline__ float silu(float v) { return v * pi_sigmoid(v); }
 
-template <int R>
-__global__ void __launch_bounds__(kThreads) ssd_scan_kernel(const ScanParams p) {
+// ITEMS: channels of the convolution per thread.
+template <int R, int ITEMS>
+__global__ void __launch_bounds__(kThreads, R == 0 || R > 16 ? 1 : R > 8 || ITEMS > 2 ? 2 : 4) ssd_scan_kernel(const ScanParams p) {
   extern __shared__ __align__(16) float sm[];
   const pi_ssd& r = p.r;
   const int e_first = blockIdx.x * kSlice, head = blockIdx.y, seq = p.seqs[blockIdx.z];
@@ -43,7 +44,6 @@ __global__ void __launch_bounds__(kThreads) ssd_scan_kernel(const ScanParams p) 
   float* sx = sm;                          // [kSlice] x, [N] B, [N] C behind the convolution
   float* sB = sx + kSlice;
   float* sC = sB + N;
-  float* pre = sC + N;                     // [kSlice + 2 N] what the first token's convolution takes from earlier steps
   __shared__ __align__(16) float part[kWarps][kSlice];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int row0 = p.seq_row0[seq], n_tok = p.seq_n[seq];
@@ -77,13 +77,14 @@ __global__ void __launch_bounds__(kThreads) ssd_scan_kernel(const ScanParams p) 
       if (nv > 3) dst[3] = v.w;
     }
   };
-  // item i of this CTA's channels: its channel among x, B, C (-1: a column past the head)
-  const int items = kSlice + 2 * N;
+  // item i of this CTA's channels: its channel among x, B, C, and its place in shared memory
+  const int items = cols + 2 * N;
   auto channel = [&](int i) {
-    if (i < kSlice) return i < cols ? head * r.vdim + e_first + i : -1;
-    i -= kSlice;
+    if (i < cols) return head * r.vdim + e_first + i;
+    i -= cols;
     return i < N ? inner + group * N + i : inner + r.groups * N + group * N + (i - N);
   };
+  for (int i = cols + tid; i < kSlice; i += kThreads) sx[i] = 0.f;
 
   // what earlier steps left may be read ahead of the dependency wait
   float4 s[R > 0 ? R : 1];
@@ -95,39 +96,52 @@ __global__ void __launch_bounds__(kThreads) ssd_scan_kernel(const ScanParams p) 
       if (!fresh && n < N) s[i] = load4(S + (size_t)n * r.vdim);
     }
   }
-  for (int i = tid; i < items; i += kThreads) {
-    const int c = channel(i);
-    float v = 0.f;
-    if (c >= 0) {
-      v = __ldg(r.conv_b + c);
-      if (!fresh)
-        for (int j = 0; j < r.taps - 1; ++j) v = fmaf(__ldg(r.conv + (size_t)c * r.taps + j), past[(size_t)j * channels + c], v);
+  float hist[ITEMS][3];                    // up to four taps: the channel's last three inputs
+  if (r.conv4) {
+#pragma unroll
+    for (int q = 0; q < ITEMS; ++q) {
+      const int i = tid + q * kThreads, c = i < items ? channel(i) : 0;
+#pragma unroll
+      for (int j = 0; j < 3; ++j) {
+        const int back = r.taps - 4 + j;   // place among the inputs kept; below 0: a tap there is not
+        hist[q][j] = !fresh && i < items && back >= 0 ? past[(size_t)back * channels + c] : 0.f;
+      }
     }
-    pre[i] = v;
   }
   pi_grid_dependency_wait();
 
   for (int t = 0; t < n_tok; ++t) {
     const float* x = p.proj + (size_t)(row0 + t) * p.stride;
     __syncthreads();                       // the last token's channels and partial sums have been read
-    for (int i = tid; i < items; i += kThreads) {
-      const int c = channel(i);
-      float v = 0.f;
-      if (c >= 0) {
-        const float* w = r.conv + (size_t)c * r.taps;
-        if (t == 0) {
-          v = pre[i];
-        } else {
-          v = __ldg(r.conv_b + c);
-          for (int j = 0; j < r.taps - 1; ++j) {
-            const int tt = t - r.taps + 1 + j;
-            const float u = tt >= 0 ? p.proj[(size_t)(row0 + tt) * p.stride + r.col_x + c] : fresh ? 0.f : past[(size_t)(r.taps - 1 + tt) * channels + c];
-            v = fmaf(__ldg(w + j), u, v);
-          }
-        }
-        v = silu(fmaf(__ldg(w + r.taps - 1), x[r.col_x + c], v));
+    if (r.conv4) {
+      float u[ITEMS];
+      float4 w[ITEMS];
+#pragma unroll
+      for (int q = 0; q < ITEMS; ++q) {
+        const int i = tid + q * kThreads, c = channel(min(i, items - 1));
+        u[q] = x[r.col_x + c];
+        w[q] = __ldg(r.conv4 + c);
       }
-      sm[i] = v;
+#pragma unroll
+      for (int q = 0; q < ITEMS; ++q) {
+        const int i = tid + q * kThreads;
+        const float v = fmaf(w[q].w, u[q], fmaf(w[q].z, hist[q][2], fmaf(w[q].y, hist[q][1], fmaf(w[q].x, hist[q][0], __ldg(r.conv_b + channel(min(i, items - 1)))))));
+        hist[q][0] = hist[q][1];
+        hist[q][1] = hist[q][2];
+        hist[q][2] = u[q];
+        if (i < items) sm[i < cols ? i : i - cols + kSlice] = silu(v);
+      }
+    } else {
+      for (int i = tid; i < items; i += kThreads) {
+        const int c = channel(i);
+        float v = __ldg(r.conv_b + c);
+        for (int j = 0; j < r.taps; ++j) {
+          const int tt = t - r.taps + 1 + j;
+          const float u = tt >= 0 ? p.proj[(size_t)(row0 + tt) * p.stride + r.col_x + c] : fresh ? 0.f : past[(size_t)(r.taps - 1 + tt) * channels + c];
+          v = fmaf(__ldg(r.conv + (size_t)c * r.taps + j), u, v);
+        }
+        sm[i < cols ? i : i - cols + kSlice] = silu(v);
+      }
     }
     const float dt = pi_softplus(x[r.col_dt + head] + dt_bias), keep = expf(a_neg * dt);
     __syncthreads();
@@ -195,7 +209,8 @@ struct NormParams {
   const int32_t *seq_row0, *seq_n, *seq_start, *slot;
 };
 
-// blockIdx.x < rows: (row, part of the channels); behind them: (sequence, share of the convolution's channels).
+// blockIdx.x < rows: (row, part of the channels); behind them: 256 of the convolution's channels of a sequence.
+constexpr int kHeld = 4;                   // groups of four channels a thread keeps between the two passes
 template <typename O>
 __global__ void __launch_bounds__(kThreads) ssd_norm_kernel(const NormParams p) {
   const pi_ssd& r = p.r;
@@ -203,21 +218,43 @@ __global__ void __launch_bounds__(kThreads) ssd_norm_kernel(const NormParams p) 
   __shared__ float red[kWarps];
   pi_grid_dependency_wait();
   if ((int)blockIdx.x >= p.rows) {
-    const int seq = (int)blockIdx.x - p.rows, channels = r.channels(), n = p.seq_n[seq], keep = r.taps - 1;
+    const int channels = r.channels(), blocks = (channels + kThreads - 1) / kThreads, i = (int)blockIdx.x - p.rows, seq = i / blocks;
+    const int n = p.seq_n[seq], keep = r.taps - 1, c = (i - seq * blocks) * kThreads + tid;
+    if (blockIdx.y > 0 || c >= channels) return;
     const bool fresh = p.seq_start[seq] == 0;
-    float* past = r.state + (size_t)p.slot[seq] * r.state_stride + r.state_off + (size_t)r.heads * r.dim * r.vdim;
-    const float* x = p.proj + (size_t)p.seq_row0[seq] * p.stride + r.col_x;
-    for (int c = blockIdx.y * kThreads + tid; c < channels; c += gridDim.y * kThreads)
-      for (int j = 0; j < keep; ++j) {       // ascending: an input moves towards the front
-        const int t = n - keep + j;
-        past[(size_t)j * channels + c] = t >= 0 ? x[(size_t)t * p.stride + c] : fresh ? 0.f : past[(size_t)(j + n) * channels + c];
-      }
+    float* past = r.state + (size_t)p.slot[seq] * r.state_stride + r.state_off + (size_t)r.heads * r.dim * r.vdim + c;
+    const float* x = p.proj + (size_t)p.seq_row0[seq] * p.stride + r.col_x + c;
+    auto input = [&](int j) {                // what stands at place j from now on
+      const int t = n - keep + j;
+      return t >= 0 ? x[(size_t)t * p.stride] : fresh ? 0.f : past[(size_t)(j + n) * channels];
+    };
+    if (keep <= 3) {
+      float v[3];
+#pragma unroll
+      for (int j = 0; j < 3; ++j) v[j] = j < keep ? input(j) : 0.f;
+#pragma unroll
+      for (int j = 0; j < 3; ++j)
+        if (j < keep) past[(size_t)j * channels] = v[j];
+    } else {
+      for (int j = 0; j < keep; ++j) past[(size_t)j * channels] = input(j);   // ascending: an input moves towards the front
+    }
     return;
   }
   const int n = inner / r.norm_groups, c0 = blockIdx.y * n;
   const float* y = p.y + (size_t)blockIdx.x * inner + c0;
+  const bool held = n % 4 == 0 && n <= kHeld * 4 * kThreads;
+  float4 v[kHeld];
   float ss = 0.f;
-  for (int i = tid; i < n; i += kThreads) ss = fmaf(y[i], y[i], ss);
+  if (held) {
+#pragma unroll
+    for (int j = 0; j < kHeld; ++j) {
+      const int i = (tid + j * kThreads) * 4;
+      v[j] = *reinterpret_cast<const float4*>(y + min(i, n - 4));
+      if (i < n) ss = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, fmaf(v[j].w, v[j].w, ss))));
+    }
+  } else {
+    for (int i = tid; i < n; i += kThreads) ss = fmaf(y[i], y[i], ss);
+  }
   ss = pi_warp_sum(ss);
   if ((tid & 31) == 0) red[tid >> 5] = ss;
   __syncthreads();
@@ -226,7 +263,24 @@ __global__ void __launch_bounds__(kThreads) ssd_norm_kernel(const NormParams p) 
   for (int w = 0; w < kWarps; ++w) ss += red[w];
   const float inv = 1.0f / sqrtf(ss / (float)n + r.eps);
   O* out = static_cast<O*>(p.out) + (size_t)blockIdx.x * p.out_stride + c0;
-  for (int i = tid; i < n; i += kThreads) out[i] = pi_from_f32<O>(y[i] * inv * __ldg(r.norm + c0 + i));
+  if (held) {
+#pragma unroll
+    for (int j = 0; j < kHeld; ++j) {
+      const int i = (tid + j * kThreads) * 4;
+      if (i >= n) break;
+      const float e[4] = {v[j].x, v[j].y, v[j].z, v[j].w};
+#pragma unroll
+      for (int k = 0; k < 4; ++k) out[i + k] = pi_from_f32<O>(e[k] * inv * __ldg(r.norm + c0 + i + k));
+    }
+  } else {
+    for (int i = tid; i < n; i += kThreads) out[i] = pi_from_f32<O>(y[i] * inv * __ldg(r.norm + c0 + i));
+  }
+}
+
+template <int ITEMS>
+void (*pick_scan(int rows))(const ScanParams) {
+  return rows <= 2 ? ssd_scan_kernel<2, ITEMS> : rows <= 4 ? ssd_scan_kernel<4, ITEMS> : rows <= 8 ? ssd_scan_kernel<8, ITEMS>
+         : rows <= 16 ? ssd_scan_kernel<16, ITEMS> : rows <= 32 ? ssd_scan_kernel<32, ITEMS> : ssd_scan_kernel<0, ITEMS>;
 }
 
 }  // namespace
@@ -239,15 +293,15 @@ pi_status pi_launch_ssd(pi_ctx* ctx, const pi_ssd& r, const float* proj, size_t 
     while ((4 << p.lanes_log2) < std::min(r.vdim, kSlice)) ++p.lanes_log2;
     p.vec = r.vdim % 4 == 0 && r.state_off % 4 == 0 && r.state_stride % 4 == 0;
     const int rpp = kThreads >> p.lanes_log2, need = (r.dim + rpp - 1) / rpp;
-    void (*k)(const ScanParams) = need <= 2 ? ssd_scan_kernel<2> : need <= 4 ? ssd_scan_kernel<4> : need <= 8 ? ssd_scan_kernel<8>
-                                  : need <= 16 ? ssd_scan_kernel<16> : need <= 32 ? ssd_scan_kernel<32> : ssd_scan_kernel<0>;
-    const size_t smem = (size_t)2 * (kSlice + 2 * r.dim) * sizeof(float);
-    PI_REQUIRE(ctx, smem <= 40 * 1024, "%d state channels are too many", r.dim);
+    const int items = (std::min(r.vdim, kSlice) + 2 * r.dim + kThreads - 1) / kThreads;   // per thread
+    PI_REQUIRE(ctx, items <= 8, "%d state channels are too many", r.dim);
+    void (*k)(const ScanParams) = items <= 2 ? pick_scan<2>(need) : items <= 4 ? pick_scan<4>(need) : pick_scan<8>(need);
+    const size_t smem = (size_t)(kSlice + 2 * r.dim) * sizeof(float);
     PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3((r.vdim + kSlice - 1) / kSlice, r.heads, b.n_scan), dim3(kThreads), smem, 1, p));
   }
   if (b.n_chunks > 0) PI_TRY(pi_launch_ssd_chunks(ctx, r, proj, stride, y, b, scratch));
   const NormParams n = {r, proj, stride, y, out, out_stride, b.rows, b.seq_row0, b.seq_n, b.seq_start, b.slot};
   PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, out_kind == PI_BF16 ? ssd_norm_kernel<__nv_bfloat16> : ssd_norm_kernel<float>,
-                                  dim3(b.rows + (r.taps > 1 ? b.n_seqs : 0), r.norm_groups), dim3(kThreads), 0, 1, n));
+                                  dim3(b.rows + (r.taps > 1 ? b.n_seqs * ((r.channels() + kThreads - 1) / kThreads) : 0), r.norm_groups), dim3(kThreads), 0, 1, n));
   return PI_OK;
 }
