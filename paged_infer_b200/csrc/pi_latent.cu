@@ -12,11 +12,10 @@
 //               spells out keys and values of all heads into a scratch pool, and the windowed tile kernel of multi-map
 //               attention runs on it: a third of the arithmetic per (query, key) pair at a latent of four head sizes.
 //
-// latent_decode_kernel (bf16 pool, mma.sync): CTA = (row, group of 16 heads = the MMA's rows, KV split).  Tiles of 32 keys, three
-// in flight.  A warp scores 8 keys over half of the channels, its queries in registers; the scores meet in shared memory,
-// every warp forms the weights of all 32 keys for itself and sums its own value channels, so that neither weights nor
-// accumulators are exchanged.  The weights enter as two bf16 planes (16 bits).  Splits of a row form a cluster and merge
-// through distributed shared memory.
+// latent_decode_kernel (bf16 pool, mma.sync): CTA = (row, group of 16 heads = the MMA's rows, KV split).  Tiles of 64 keys, two
+// in flight.  A warp scores 16 keys over half of the channels, its queries in registers; the softmax meets in shared
+// memory, every warp sums its own value channels over all 64 keys, so that accumulators never merge inside a CTA.  The
+// weights enter as two bf16 planes (16 bits).  Splits of a row form a cluster and merge through distributed shared memory.
 #include <cooperative_groups.h>
 #include <limits.h>
 #include <math.h>
@@ -140,6 +139,7 @@ struct LatentParams {
   int max_blocks, rows, n_latent, expand_min;
   int slices, row_splits;      // absorb: 64-channel slices of the latent, CTAs that share the rows of one
   int groups, nsplit;          // decode: groups of 16 heads, KV splits
+  int block_shift;             // block_size is 1 << block_shift; -1: it is no power of two
 };
 
 // CTA i < rows: row i into the pool, its queries rotated.  The CTAs behind: queries of the latent rows into latent space.
@@ -252,68 +252,70 @@ __global__ void __launch_bounds__(kHeadThreads) latent_out_f32_kernel(const Late
 }
 
 // ---- decode attention over the latents ---------------------------------------------------------------------------------------
-constexpr int kDecWarps = 8, kDecThreads = kDecWarps * 32, kKeys = 32, kStages = 4, kMaxSplits = 8;
-constexpr int kSPitch = kKeys + 4;
+constexpr int kDecWarps = 8, kDecThreads = kDecWarps * 32, kKeys = 64, kStages = 2, kMaxSplits = 16;
+constexpr int kSPitch = kKeys + 8, kPPitch = kKeys + 8;
 
 struct DecodeSmem {
-  size_t s, acc, total;            // byte offsets: scores behind the ring; the finished sums take the ring's place
+  size_t s, p, acc, total;         // byte offsets: scores and weights behind the ring; the finished sums take the ring's place
 };
 __host__ __device__ inline DecodeSmem decode_smem(int dp, int rp) {
   DecodeSmem s;
   const size_t ring = (size_t)kStages * kKeys * (dp + 8) * 2, acc = (size_t)16 * (rp + 4) * 4;
   s.acc = 0;
   s.s = ring > acc ? ring : acc;
-  s.total = s.s + (size_t)2 * 2 * 16 * kSPitch * 4;
+  s.p = s.s + (size_t)2 * 16 * kSPitch * 4;
+  s.total = s.p + (size_t)2 * 16 * kPPitch * 2;
   return s;
 }
 
 // QMAX: steps of 16 channels per warp (half of a row), UMAX: units of 16 value channels per warp.
 template <int QMAX, int UMAX>
 __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const LatentParams p) {
-  static_assert(QMAX % 2 == 0, "two steps per load");
+  static_assert(kStages == 2, "the tile behind the current one is in flight");
   extern __shared__ __align__(16) unsigned char smem[];
   const DecodeSmem lay = decode_smem(p.dp, p.rp);
   __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(smem);
-  float* scores = reinterpret_cast<float*>(smem + lay.s);     // [parity][half of the channels][16][kSPitch]
-  __shared__ float c_m[16], c_l[16];
+  float* scores = reinterpret_cast<float*>(smem + lay.s);     // [half of the channels][16][kSPitch]
+  __nv_bfloat16* phi = reinterpret_cast<__nv_bfloat16*>(smem + lay.p);   // weights, two planes [16][kPPitch]
+  __nv_bfloat16* plo = phi + 16 * kPPitch;
+  __shared__ float s_keep[16], c_m[16], c_l[16];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, split_i = blockIdx.x, h0 = blockIdx.z * 16;
   const int row = p.latent_rows[blockIdx.y], seq = p.row_seq[row], pos = p.row_pos[row], settled = p.seq_start[seq];
   const int32_t* table = p.tables + (size_t)seq * p.max_blocks;
   const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(p.base);
   const int pitch = p.dp + 8, units = p.rp / 16;
-  // this warp scores keys 8 (warp % 4).. over its half of the channels
-  const int half = warp >> 2, nks = p.dp / 16, k0 = half ? (nks + 1) / 2 : 0, k1 = half ? nks : (nks + 1) / 2;
+  // this warp scores keys 16 (warp % 4).. over its half of the channels
+  const int half = warp >> 2, nks = p.dp / 16, k0 = half ? (nks + 1) / 2 : 0, n_k = half ? nks / 2 : (nks + 1) / 2;
 
   const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, hi = min(pos + 1, p.lens[seq] * p.block_size);
   const int t_first = lo / kKeys, n_tiles = max(0, (hi + kKeys - 1) / kKeys - t_first), per = (n_tiles + p.nsplit - 1) / p.nsplit;
   const int tile0 = t_first + split_i * per, tile_end = min(t_first + n_tiles, tile0 + per);
 
-  // eight threads per key; its physical block is looked up a tile ahead of the request
-  const int fr = tid >> 3, fx = (tid & 7) * 8;
+  // four threads per key; its physical block is looked up a tile ahead of the request
+  const int fr = tid >> 2, fx = (tid & 3) * 8;
+  auto logical = [&](int t) { return p.block_shift >= 0 ? t >> p.block_shift : t / p.block_size; };
   auto block_of = [&](int tile) {
     const int t = tile * kKeys + fr;
-    return tile < tile_end && t < hi ? table[t / p.block_size] : -1;
+    return tile < tile_end && t < hi ? table[logical(t)] : -1;
   };
   auto fetch = [&](int tile, int stage, int pb) {
-    const __nv_bfloat16* src = pb >= 0 ? base + ((size_t)pb * p.block_size + (tile * kKeys + fr) % p.block_size) * p.dp : base;
-    const uint32_t dst = smem_addr(ring + ((size_t)stage * kKeys + fr) * pitch);
-#pragma unroll 4
-    for (int x = fx; x < p.dp; x += 64) cp_async16(dst + x * 2, pb >= 0 ? src + x : base, pb >= 0 ? 16 : 0);
+    const int t = tile * kKeys + fr;
+    const __nv_bfloat16* src = (pb >= 0 ? base + ((size_t)pb * p.block_size + (t - logical(t) * p.block_size)) * p.dp : base) + fx;
+    const uint32_t dst = smem_addr(ring + ((size_t)stage * kKeys + fr) * pitch + fx), bytes = pb >= 0 ? 16 : 0;
+#pragma unroll 6
+    for (int x = 0; x < p.dp - fx; x += 32) cp_async16(dst + x * 2, src + x, bytes);
   };
-  int pb[kStages];
-#pragma unroll
-  for (int s = 0; s < kStages; ++s) pb[s] = block_of(tile0 + s);
+  const int pb0 = block_of(tile0), pb1 = block_of(tile0 + 1);
   // tiles of keys that earlier steps wrote are requested ahead of the dependency wait
-#pragma unroll
-  for (int s = 0; s < kStages - 1; ++s)
-    if (tile0 + s < tile_end && (tile0 + s + 1) * kKeys <= settled) fetch(tile0 + s, s, pb[s]);
+  const bool early0 = (tile0 + 1) * kKeys <= settled, early1 = (tile0 + 2) * kKeys <= settled;
+  if (early0 && tile0 < tile_end) fetch(tile0, 0, pb0);
+  if (early0 && early1 && tile0 + 1 < tile_end) fetch(tile0 + 1, 1, pb1);
   pi_grid_dependency_wait();
-#pragma unroll
-  for (int s = 0; s < kStages - 1; ++s) {
-    if (tile0 + s < tile_end && (tile0 + s + 1) * kKeys > settled) fetch(tile0 + s, s, pb[s]);
-    cp_async_commit();             // the first group also holds what was requested early
-  }
-  int pb_next = pb[kStages - 1];
+  if (!early0 && tile0 < tile_end) fetch(tile0, 0, pb0);
+  cp_async_commit();                 // the first group also holds what was requested early
+  if (!(early0 && early1) && tile0 + 1 < tile_end) fetch(tile0 + 1, 1, pb1);
+  cp_async_commit();
+  int pb_next = block_of(tile0 + 2);
 
   uint32_t qa[QMAX][4];
   {
@@ -323,9 +325,9 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
     for (int k = 0; k < QMAX; ++k)
 #pragma unroll
       for (int j = 0; j < 4; ++j) {   // a0: head, a1: head + 8, a2 / a3: channels + 8; outside: a valid address and zero
-        const int r = r0 + (j & 1) * 8, ks = k0 + k;
-        const bool ok = r < live && ks < k1;
-        const uint32_t v = *reinterpret_cast<const uint32_t*>(q + (ok ? (size_t)r * p.dp + ks * 16 + (j >> 1) * 8 : (size_t)0));
+        const int r = r0 + (j & 1) * 8;
+        const bool ok = r < live && k < n_k;
+        const uint32_t v = *reinterpret_cast<const uint32_t*>(q + (ok ? (size_t)r * p.dp + (k0 + k) * 16 + (j >> 1) * 8 : (size_t)0));
         qa[k][j] = ok ? v : 0u;
       }
   }
@@ -336,94 +338,80 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[u][j][i] = 0.f;
-  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};   // the same in every warp
+  // softmax: thread = (head tid / 16, keys 4 (tid % 16)..)
+  const int sh = tid >> 4, sk = (tid & 15) * 4;
+  float mx = -INFINITY, l = 0.f;
   const float sc = p.scale * kLog2e;
   const int r0 = lane >> 2;
 
   for (int tile = tile0; tile < tile_end; ++tile) {
-    const int i = tile - tile0, stage = i % kStages;
+    const int stage = (tile - tile0) & 1;
     const __nv_bfloat16* ks = ring + (size_t)stage * kKeys * pitch;
-    cp_async_wait<kStages - 2>();
-    __syncthreads();                 // the tile has landed; everybody is done with the tile before it
-    {
-      const int next = tile + kStages - 1, now = pb_next;
-      pb_next = block_of(next + 1);
-      if (next < tile_end) fetch(next, (i + kStages - 1) % kStages, now);
-      cp_async_commit();
-    }
+    cp_async_wait<1>();
+    __syncthreads();                 // the tile has landed
     {
       float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-      const uint32_t kb = smem_addr(ks + (size_t)((warp & 3) * 8 + (lane & 7)) * pitch + k0 * 16 + (lane >> 3) * 8);
+      const uint32_t kb = smem_addr(ks + (size_t)((warp & 3) * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch + k0 * 16 + ((lane >> 3) & 1) * 8);
 #pragma unroll
-      for (int k = 0; k < QMAX; k += 2) {
-        if (k0 + k < k1) {
-          uint32_t b[4];             // channels 0-7, 8-15 of step k, then of step k + 1
-          if (k0 + k + 1 < nks) ldsm4(b, kb + k * 32);
-          else ldsm4(b, kb + k * 32 - (lane >> 4) * 32);
+      for (int k = 0; k < QMAX; ++k) {
+        if (k < n_k) {
+          uint32_t b[4];             // keys 0-7: channels 0-7, 8-15; keys 8-15 likewise
+          ldsm4(b, kb + k * 32);
           mma(s[0], qa[k][0], qa[k][1], qa[k][2], qa[k][3], b[0], b[1]);
-          if (k0 + k + 1 < k1) mma(s[1], qa[k + 1][0], qa[k + 1][1], qa[k + 1][2], qa[k + 1][3], b[2], b[3]);
+          mma(s[1], qa[k][0], qa[k][1], qa[k][2], qa[k][3], b[2], b[3]);
         }
       }
-      float* out = scores + (size_t)(((i & 1) * 2 + half) * 16) * kSPitch + (warp & 3) * 8 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(out + r0 * kSPitch) = make_float2(s[0][0] + s[1][0], s[0][1] + s[1][1]);
-      *reinterpret_cast<float2*>(out + (r0 + 8) * kSPitch) = make_float2(s[0][2] + s[1][2], s[0][3] + s[1][3]);
+      float* out = scores + (size_t)(half * 16 + r0) * kSPitch + (warp & 3) * 16 + (lane & 3) * 2;
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        *reinterpret_cast<float2*>(out + j * 8) = make_float2(s[j][0], s[j][1]);
+        *reinterpret_cast<float2*>(out + 8 * kSPitch + j * 8) = make_float2(s[j][2], s[j][3]);
+      }
     }
     __syncthreads();
-    // every warp forms the weights of all 32 keys for itself, in the layout of the product's left operand
-    float w[2][2][4];                // [16 keys][head r0, r0 + 8][keys 0, 1, 8, 9 behind the lane's first]
+    {
+      const float4 x = *reinterpret_cast<const float4*>(scores + (size_t)sh * kSPitch + sk), y = *reinterpret_cast<const float4*>(scores + (size_t)(16 + sh) * kSPitch + sk);
+      const int t = tile * kKeys + sk;
+      float v[4] = {(x.x + y.x) * sc, (x.y + y.y) * sc, (x.z + y.z) * sc, (x.w + y.w) * sc};
 #pragma unroll
-    for (int c = 0; c < 2; ++c)
+      for (int j = 0; j < 4; ++j)
+        if (t + j < lo || t + j >= hi) v[j] = -INFINITY;
+      float n = fmaxf(fmaxf(v[0], v[1]), fmaxf(v[2], v[3]));
 #pragma unroll
-      for (int h = 0; h < 2; ++h)
+      for (int o = 8; o > 0; o >>= 1) n = fmaxf(n, __shfl_xor_sync(0xffffffffu, n, o));
+      n = fmaxf(mx, n);
+      const float keep = n == -INFINITY ? 1.f : exp2f(mx - n), ref = n == -INFINITY ? 0.f : n;
+      mx = n;
 #pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          const float* a = scores + (size_t)((i & 1) * 32 + r0 + 8 * h) * kSPitch + c * 16 + (lane & 3) * 2 + j * 8;
-          const float2 x = *reinterpret_cast<const float2*>(a), y = *reinterpret_cast<const float2*>(a + 16 * kSPitch);
-          const int t = tile * kKeys + c * 16 + (lane & 3) * 2 + j * 8;
-          w[c][h][2 * j] = t >= lo && t < hi ? (x.x + y.x) * sc : -INFINITY;
-          w[c][h][2 * j + 1] = t + 1 >= lo && t + 1 < hi ? (x.y + y.y) * sc : -INFINITY;
-        }
-    float keep[2];
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      float n = -INFINITY;
-#pragma unroll
-      for (int c = 0; c < 2; ++c)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) n = fmaxf(n, w[c][h][j]);
-      n = fmaxf(mx[h], quad_max(n));
-      keep[h] = n == -INFINITY ? 1.f : exp2f(mx[h] - n);
-      mx[h] = n;
-      const float ref = n == -INFINITY ? 0.f : n;
-      float sum = 0.f;
-#pragma unroll
-      for (int c = 0; c < 2; ++c)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          w[c][h][j] = exp2f(w[c][h][j] - ref);
-          sum += w[c][h][j];
-        }
-      l[h] = l[h] * keep[h] + sum;
+      for (int j = 0; j < 4; ++j) v[j] = exp2f(v[j] - ref);
+      l = l * keep + ((v[0] + v[1]) + (v[2] + v[3]));
+      uint2 hi2, lo2;
+      split(v[0], v[1], hi2.x, lo2.x);
+      split(v[2], v[3], hi2.y, lo2.y);
+      *reinterpret_cast<uint2*>(phi + sh * kPPitch + sk) = hi2;
+      *reinterpret_cast<uint2*>(plo + sh * kPPitch + sk) = lo2;
+      if ((tid & 15) == 0) s_keep[sh] = keep;
     }
-    if (__any_sync(0xffffffffu, keep[0] != 1.f || keep[1] != 1.f)) {
+    __syncthreads();
+    const float keep0 = s_keep[r0], keep1 = s_keep[r0 + 8];
+    if (__any_sync(0xffffffffu, keep0 != 1.f || keep1 != 1.f)) {
 #pragma unroll
       for (int u = 0; u < UMAX; ++u)
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
-          acc[u][j][0] *= keep[0];
-          acc[u][j][1] *= keep[0];
-          acc[u][j][2] *= keep[1];
-          acc[u][j][3] *= keep[1];
+          acc[u][j][0] *= keep0;
+          acc[u][j][1] *= keep0;
+          acc[u][j][2] *= keep1;
+          acc[u][j][3] *= keep1;
         }
     }
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
+    for (int k = 0; k < kKeys / 16; ++k) {
       uint32_t ph[4], pl[4];
-#pragma unroll
-      for (int h = 0; h < 2; ++h)
-#pragma unroll
-        for (int j = 0; j < 2; ++j) split(w[c][h][2 * j], w[c][h][2 * j + 1], ph[2 * j + h], pl[2 * j + h]);
-      const uint32_t vb = smem_addr(ks + (size_t)(c * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (lane >> 4) * 8);
+      const int pr = ((lane & 7) + ((lane >> 3) & 1) * 8) * kPPitch + k * 16 + (lane >> 4) * 8;
+      ldsm4(ph, smem_addr(phi + pr));
+      ldsm4(pl, smem_addr(plo + pr));
+      const uint32_t vb = smem_addr(ks + (size_t)(k * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (lane >> 4) * 8);
 #pragma unroll
       for (int u = 0; u < UMAX; ++u) {
         const int unit = warp + u * kDecWarps;
@@ -438,6 +426,10 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
         }
       }
     }
+    __syncthreads();                 // the stage has been read
+    if (tile + 2 < tile_end) fetch(tile + 2, stage, pb_next);
+    cp_async_commit();
+    pb_next = block_of(tile + 3);
   }
   cp_async_wait<0>();
   __syncthreads();
@@ -457,12 +449,10 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
       }
   }
 #pragma unroll
-  for (int h = 0; h < 2; ++h) {
-    l[h] = quad_sum(l[h]);
-    if (warp == 0 && (lane & 3) == 0) {
-      c_m[r0 + 8 * h] = mx[h];
-      c_l[r0 + 8 * h] = l[h];
-    }
+  for (int o = 8; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+  if ((tid & 15) == 0) {
+    c_m[sh] = mx;
+    c_l[sh] = l;
   }
   cg::cluster_group cluster = cg::this_cluster();
   if (p.nsplit > 1) cluster.sync();
@@ -506,7 +496,8 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
       }
     }
   };
-  if (p.nsplit > 1) finish(std::integral_constant<int, kMaxSplits>());
+  if (p.nsplit > 8) finish(std::integral_constant<int, kMaxSplits>());
+  else if (p.nsplit > 1) finish(std::integral_constant<int, 8>());
   else finish(std::integral_constant<int, 1>());
   if (p.nsplit > 1) cluster.sync();   // a peer may still be reading this CTA's part
 }
@@ -557,7 +548,17 @@ cudaError_t grant(pi_ctx* ctx, LatentKernel k, size_t smem) {   // a kernel's sh
   return cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
 }
 
-constexpr int kMaxDecodeDp = 768;
+// Clusters of 16 CTAs have to be asked for, once per kernel and device.
+pi_status allow_wide_clusters(pi_ctx* ctx, LatentKernel k) {
+  static std::vector<std::pair<LatentKernel, int>> done;
+  for (auto& d : done)
+    if (d.first == k && d.second == ctx->device) return PI_OK;
+  PI_CUDA(ctx, cudaFuncSetAttribute(k, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+  done.push_back({k, ctx->device});
+  return PI_OK;
+}
+
+constexpr int kMaxDecodeDp = 704;
 LatentKernel pick_decode(int dp, int rp) {
   if (rp <= 128 && dp <= 192) return latent_decode_kernel<6, 1>;
   if (rp <= 256 && dp <= 384) return latent_decode_kernel<12, 2>;
@@ -594,6 +595,9 @@ pi_status pi_launch_latent_attention(pi_ctx* ctx, const pi_latent_attention& a, 
   p.dp = kv.dp;
   p.window = a.window;
   p.block_size = kv.block_size;
+  p.block_shift = -1;
+  for (int i = 0; i < 31; ++i)
+    if (1 << i == kv.block_size) p.block_shift = i;
   p.col_q = a.col_q;
   p.col_kv = a.col_kv;
   p.col_g = a.col_g;
@@ -651,6 +655,7 @@ pi_status pi_launch_latent_attention(pi_ctx* ctx, const pi_latent_attention& a, 
     const LatentKernel k = pick_decode(p.dp, p.rp);
     const size_t smem = decode_smem(p.dp, p.rp).total;
     PI_CUDA(ctx, grant(ctx, k, smem));
+    PI_TRY(allow_wide_clusters(ctx, k));
     // KV splits: one round of CTAs over the GPU, at least a tile each
     const int keys = a.window > 0 ? std::min(a.window, b.max_pos + 1) : b.max_pos + 1;
     const long ctas = (long)b.n_latent * p.groups, resident = ctx->sm_count * std::max(1L, (long)(ctx->smem_optin / (smem + 2048)));
