@@ -13,7 +13,7 @@
 //               attention runs on it: a third of the arithmetic per (query, key) pair at a latent of four head sizes.
 //
 // latent_decode_kernel (bf16 pool, mma.sync): CTA = (row, group of 16 heads = the MMA's rows, KV split).  Tiles of 64 keys, two
-// in flight.  A warp scores 16 keys over half of the channels, its queries in registers; the softmax meets in shared
+// in flight.  A warp scores 16 keys over a quarter of the channels, its queries in registers; the softmax meets in shared
 // memory, every warp sums its own value channels over all 64 keys, so that accumulators never merge inside a CTA.  The
 // weights enter as two bf16 planes (16 bits).  Splits of a row form a cluster and merge through distributed shared memory.
 #include <cooperative_groups.h>
@@ -252,7 +252,7 @@ __global__ void __launch_bounds__(kHeadThreads) latent_out_f32_kernel(const Late
 }
 
 // ---- decode attention over the latents ---------------------------------------------------------------------------------------
-constexpr int kDecWarps = 8, kDecThreads = kDecWarps * 32, kKeys = 64, kStages = 2, kMaxSplits = 16;
+constexpr int kDecWarps = 16, kDecThreads = kDecWarps * 32, kKeys = 64, kStages = 2, kMaxSplits = 16;
 constexpr int kSPitch = kKeys + 8, kPPitch = kKeys + 8;
 
 struct DecodeSmem {
@@ -263,19 +263,19 @@ __host__ __device__ inline DecodeSmem decode_smem(int dp, int rp) {
   const size_t ring = (size_t)kStages * kKeys * (dp + 8) * 2, acc = (size_t)16 * (rp + 4) * 4;
   s.acc = 0;
   s.s = ring > acc ? ring : acc;
-  s.p = s.s + (size_t)2 * 16 * kSPitch * 4;
+  s.p = s.s + (size_t)4 * 16 * kSPitch * 4;
   s.total = s.p + (size_t)2 * 16 * kPPitch * 2;
   return s;
 }
 
-// QMAX: steps of 16 channels per warp (half of a row), UMAX: units of 16 value channels per warp.
+// QMAX: steps of 16 channels per warp (a quarter of a row), UMAX: units of 16 value channels per warp.
 template <int QMAX, int UMAX>
 __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const LatentParams p) {
   static_assert(kStages == 2, "the tile behind the current one is in flight");
   extern __shared__ __align__(16) unsigned char smem[];
   const DecodeSmem lay = decode_smem(p.dp, p.rp);
   __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(smem);
-  float* scores = reinterpret_cast<float*>(smem + lay.s);     // [half of the channels][16][kSPitch]
+  float* scores = reinterpret_cast<float*>(smem + lay.s);     // [quarter of the channels][16][kSPitch]
   __nv_bfloat16* phi = reinterpret_cast<__nv_bfloat16*>(smem + lay.p);   // weights, two planes [16][kPPitch]
   __nv_bfloat16* plo = phi + 16 * kPPitch;
   __shared__ float s_keep[16], c_m[16], c_l[16];
@@ -284,15 +284,15 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
   const int32_t* table = p.tables + (size_t)seq * p.max_blocks;
   const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(p.base);
   const int pitch = p.dp + 8, units = p.rp / 16;
-  // this warp scores keys 16 (warp % 4).. over its half of the channels
-  const int half = warp >> 2, nks = p.dp / 16, k0 = half ? (nks + 1) / 2 : 0, n_k = half ? nks / 2 : (nks + 1) / 2;
+  // this warp scores keys 16 (warp % 4).. over its quarter of the channels
+  const int quarter = warp >> 2, nks = p.dp / 16, k0 = nks * quarter / 4, n_k = nks * (quarter + 1) / 4 - k0;
 
   const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, hi = min(pos + 1, p.lens[seq] * p.block_size);
   const int t_first = lo / kKeys, n_tiles = max(0, (hi + kKeys - 1) / kKeys - t_first), per = (n_tiles + p.nsplit - 1) / p.nsplit;
   const int tile0 = t_first + split_i * per, tile_end = min(t_first + n_tiles, tile0 + per);
 
-  // four threads per key; its physical block is looked up a tile ahead of the request
-  const int fr = tid >> 2, fx = (tid & 3) * 8;
+  // eight threads per key; its physical block is looked up a tile ahead of the request
+  const int fr = tid >> 3, fx = (tid & 7) * 8;
   auto logical = [&](int t) { return p.block_shift >= 0 ? t >> p.block_shift : t / p.block_size; };
   auto block_of = [&](int tile) {
     const int t = tile * kKeys + fr;
@@ -302,8 +302,8 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
     const int t = tile * kKeys + fr;
     const __nv_bfloat16* src = (pb >= 0 ? base + ((size_t)pb * p.block_size + (t - logical(t) * p.block_size)) * p.dp : base) + fx;
     const uint32_t dst = smem_addr(ring + ((size_t)stage * kKeys + fr) * pitch + fx), bytes = pb >= 0 ? 16 : 0;
-#pragma unroll 6
-    for (int x = 0; x < p.dp - fx; x += 32) cp_async16(dst + x * 2, src + x, bytes);
+#pragma unroll 3
+    for (int x = 0; x < p.dp - fx; x += 64) cp_async16(dst + x * 2, src + x, bytes);
   };
   const int pb0 = block_of(tile0), pb1 = block_of(tile0 + 1);
   // tiles of keys that earlier steps wrote are requested ahead of the dependency wait
@@ -338,8 +338,8 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[u][j][i] = 0.f;
-  // softmax: thread = (head tid / 16, keys 4 (tid % 16)..)
-  const int sh = tid >> 4, sk = (tid & 15) * 4;
+  // softmax: warp = head, lane = two keys
+  const int sk = lane * 2;
   float mx = -INFINITY, l = 0.f;
   const float sc = p.scale * kLog2e;
   const int r0 = lane >> 2;
@@ -361,7 +361,7 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
           mma(s[1], qa[k][0], qa[k][1], qa[k][2], qa[k][3], b[2], b[3]);
         }
       }
-      float* out = scores + (size_t)(half * 16 + r0) * kSPitch + (warp & 3) * 16 + (lane & 3) * 2;
+      float* out = scores + (size_t)(quarter * 16 + r0) * kSPitch + (warp & 3) * 16 + (lane & 3) * 2;
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         *reinterpret_cast<float2*>(out + j * 8) = make_float2(s[j][0], s[j][1]);
@@ -370,27 +370,24 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
     }
     __syncthreads();
     {
-      const float4 x = *reinterpret_cast<const float4*>(scores + (size_t)sh * kSPitch + sk), y = *reinterpret_cast<const float4*>(scores + (size_t)(16 + sh) * kSPitch + sk);
+      float v[2] = {0.f, 0.f};
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float2 x = *reinterpret_cast<const float2*>(scores + (size_t)(q * 16 + warp) * kSPitch + sk);
+        v[0] += x.x;
+        v[1] += x.y;
+      }
       const int t = tile * kKeys + sk;
-      float v[4] = {(x.x + y.x) * sc, (x.y + y.y) * sc, (x.z + y.z) * sc, (x.w + y.w) * sc};
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (t + j < lo || t + j >= hi) v[j] = -INFINITY;
-      float n = fmaxf(fmaxf(v[0], v[1]), fmaxf(v[2], v[3]));
-#pragma unroll
-      for (int o = 8; o > 0; o >>= 1) n = fmaxf(n, __shfl_xor_sync(0xffffffffu, n, o));
-      n = fmaxf(mx, n);
+      for (int j = 0; j < 2; ++j) v[j] = t + j >= lo && t + j < hi ? v[j] * sc : -INFINITY;
+      const float n = fmaxf(mx, pi_warp_max(fmaxf(v[0], v[1])));
       const float keep = n == -INFINITY ? 1.f : exp2f(mx - n), ref = n == -INFINITY ? 0.f : n;
       mx = n;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) v[j] = exp2f(v[j] - ref);
-      l = l * keep + ((v[0] + v[1]) + (v[2] + v[3]));
-      uint2 hi2, lo2;
-      split(v[0], v[1], hi2.x, lo2.x);
-      split(v[2], v[3], hi2.y, lo2.y);
-      *reinterpret_cast<uint2*>(phi + sh * kPPitch + sk) = hi2;
-      *reinterpret_cast<uint2*>(plo + sh * kPPitch + sk) = lo2;
-      if ((tid & 15) == 0) s_keep[sh] = keep;
+      for (int j = 0; j < 2; ++j) v[j] = exp2f(v[j] - ref);
+      l = l * keep + (v[0] + v[1]);
+      split(v[0], v[1], *reinterpret_cast<uint32_t*>(phi + warp * kPPitch + sk), *reinterpret_cast<uint32_t*>(plo + warp * kPPitch + sk));
+      if (lane == 0) s_keep[warp] = keep;
     }
     __syncthreads();
     const float keep0 = s_keep[r0], keep1 = s_keep[r0 + 8];
@@ -448,17 +445,16 @@ __global__ void __launch_bounds__(kDecThreads, 1) latent_decode_kernel(const Lat
         *reinterpret_cast<float2*>(wacc + (size_t)(r0 + 8) * apitch + c) = make_float2(acc[u][j][2], acc[u][j][3]);
       }
   }
-#pragma unroll
-  for (int o = 8; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-  if ((tid & 15) == 0) {
-    c_m[sh] = mx;
-    c_l[sh] = l;
+  l = pi_warp_sum(l);
+  if (lane == 0) {
+    c_m[warp] = mx;
+    c_l[warp] = l;
   }
   cg::cluster_group cluster = cg::this_cluster();
   if (p.nsplit > 1) cluster.sync();
   else __syncthreads();
   const int rank = p.nsplit > 1 ? (int)cluster.block_rank() : 0;
-  // warp = heads warp, warp + 8; channels are dealt to the splits.  NS parts are read whether they exist or not (ranks
+  // warp = head; channels are dealt to the splits.  NS parts are read whether they exist or not (ranks
   // clamped, weights zero), so that the loads are in flight together.
   auto finish = [&](auto ns_c) {
     constexpr int NS = decltype(ns_c)::value;
@@ -558,12 +554,42 @@ pi_status allow_wide_clusters(pi_ctx* ctx, LatentKernel k) {
   return PI_OK;
 }
 
+// Clusters of `splits` CTAs the device holds at once.
+int max_clusters(pi_ctx* ctx, LatentKernel k, size_t smem, int splits) {
+  struct Known {
+    LatentKernel k;
+    size_t smem;
+    int splits, device, n;
+  };
+  static std::vector<Known> known;
+  for (const Known& c : known)
+    if (c.k == k && c.smem == smem && c.splits == splits && c.device == ctx->device) return c.n;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(splits);
+  cfg.blockDim = dim3(kDecThreads);
+  cfg.dynamicSmemBytes = smem;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = splits;
+  attr[0].val.clusterDim.y = 1;
+  attr[0].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  int n = 0;
+  if (cudaOccupancyMaxActiveClusters(&n, k, &cfg) != cudaSuccess) {
+    cudaGetLastError();
+    n = 0;
+  }
+  known.push_back({k, smem, splits, ctx->device, n});
+  return n;
+}
+
 constexpr int kMaxDecodeDp = 704;
 LatentKernel pick_decode(int dp, int rp) {
-  if (rp <= 128 && dp <= 192) return latent_decode_kernel<6, 1>;
-  if (rp <= 256 && dp <= 384) return latent_decode_kernel<12, 2>;
-  if (rp <= 512 && dp <= 576) return latent_decode_kernel<18, 4>;
-  return rp <= 512 ? latent_decode_kernel<24, 4> : latent_decode_kernel<24, 8>;
+  if (rp <= 256 && dp <= 192) return latent_decode_kernel<3, 1>;
+  if (rp <= 256 && dp <= 384) return latent_decode_kernel<6, 1>;
+  if (rp <= 512 && dp <= 576) return latent_decode_kernel<9, 2>;
+  return rp <= 512 ? latent_decode_kernel<12, 2> : latent_decode_kernel<12, 4>;
 }
 
 }  // namespace
@@ -658,8 +684,9 @@ pi_status pi_launch_latent_attention(pi_ctx* ctx, const pi_latent_attention& a, 
     PI_TRY(allow_wide_clusters(ctx, k));
     // KV splits: one round of CTAs over the GPU, at least a tile each
     const int keys = a.window > 0 ? std::min(a.window, b.max_pos + 1) : b.max_pos + 1;
-    const long ctas = (long)b.n_latent * p.groups, resident = ctx->sm_count * std::max(1L, (long)(ctx->smem_optin / (smem + 2048)));
-    p.nsplit = (int)std::max(1L, std::min({resident / ctas, (long)(keys + kKeys - 1) / kKeys, (long)kMaxSplits}));
+    const long ctas = (long)b.n_latent * p.groups, tiles = (keys + kKeys - 1) / kKeys;
+    p.nsplit = (int)std::max(1L, std::min({(long)ctx->sm_count / ctas, tiles, (long)kMaxSplits}));
+    while (p.nsplit > 1 && ctas > max_clusters(ctx, k, smem, p.nsplit)) --p.nsplit;
     {
       pi_prof_scope prof(ctx, PI_PROF_ATTENTION);
       PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(p.nsplit, b.n_latent, p.groups), dim3(kDecThreads), smem, p.nsplit, p));
