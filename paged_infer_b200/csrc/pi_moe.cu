@@ -29,14 +29,10 @@ struct Best {
   float v;
   int i;
 };
-__device__ __forceinline__ Best warp_best(Best b) {   // the largest value, ties to the lower index
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float v = __shfl_xor_sync(0xffffffffu, b.v, o);
-    const int i = __shfl_xor_sync(0xffffffffu, b.i, o);
-    if (v > b.v || (v == b.v && i < b.i)) b = {v, i};
-  }
-  return b;
+// The largest value of the warp, ties to the lower index.  Bits of a float, turned so that their order as an integer is its own.
+__device__ __forceinline__ Best warp_best(Best b) {
+  const uint32_t bits = __float_as_uint(b.v), key = bits & 0x80000000u ? ~bits : bits | 0x80000000u, top = __reduce_max_sync(0xffffffffu, key);
+  return {b.v, (int)__reduce_min_sync(0xffffffffu, key == top ? (uint32_t)b.i : 0x7fffffffu)};
 }
 
 __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const RouteParams p) {
@@ -83,20 +79,24 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const Route
     __syncwarp();
   }
   float sum = 0.f;
+  int mine[2] = {0, 0};                                // choices lane and lane + 32
   for (int k = 0; k < p.top; ++k) {
     Best b = {-INFINITY, 0x7fffffff};
     for (int e = lane; e < p.experts; e += 32)
       if (choice[e] > b.v || (choice[e] == b.v && choice[e] > -INFINITY && e < b.i)) b = {choice[e], e};
     b = warp_best(b);
     const int e = min(b.i, p.experts - 1);             // (a row of NaN chooses something valid)
-    if (lane == 0) {
-      p.ids[(size_t)row * p.top + k] = e;
-      choice[e] = -INFINITY;
-    }
+    if (lane == (k & 31)) mine[k >> 5] = e;
     sum += score[e];
+    if (lane == 0) choice[e] = -INFINITY;
     __syncwarp();
   }
-  for (int k = lane; k < p.top; k += 32) p.weights[(size_t)row * p.top + k] = score[p.ids[(size_t)row * p.top + k]] / (sum + 1e-20f);
+#pragma unroll
+  for (int j = 0; j < 2; ++j)
+    if (lane + 32 * j < p.top) {
+      p.ids[(size_t)row * p.top + lane + 32 * j] = mine[j];
+      p.weights[(size_t)row * p.top + lane + 32 * j] = score[mine[j]] / (sum + 1e-20f);
+    }
 }
 
 __global__ void __launch_bounds__(kListThreads) moe_lists_kernel(const int32_t* ids, int pairs, int experts, int tile_rows, int32_t* place, int32_t* pair_at,
@@ -168,7 +168,7 @@ pi_status pi_launch_moe_route(pi_ctx* ctx, const pi_moe& m, const float* logits,
   pi_prof_scope prof(ctx, PI_PROF_OTHER);
   const RouteParams p = {logits, stride, m.correction, rows, m.experts, m.groups, m.keep, m.top, l.ids, l.weights};
   const size_t smem = (size_t)kRouteWarps * (2 * m.experts + m.groups) * sizeof(float);
-  PI_REQUIRE(ctx, smem <= 48 * 1024, "%d experts are too many", m.experts);
+  PI_REQUIRE(ctx, smem <= 48 * 1024 && m.top <= 64, "%d of %d experts are too many", m.top, m.experts);
   PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, moe_route_kernel, dim3((rows + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32), smem, 1, p));
   return PI_OK;
 }
