@@ -945,7 +945,7 @@ def lilosun_config(size):
     from paged_infer_b200 import loader as ld
     s = LILOSUN_SIZES[size]
     moe, dense = dict(ff_kind=ld.FF_EXPERTS, limit=7.0, shared_limit=7.0, **s["moe"]), dict(ff_kind=ld.FF_SILU, ff=s["dense"])
-    attn = dict(window=s["window"], rot_base=50000.0, rot_factor=4.0, rot_original=4096, scale=192 ** -0.5, **s["latent"])
+    attn = dict(window=s["window"], rot_base=10000.0, rot_factor=8.0, rot_original=4096, scale=192 ** -0.5, **s["latent"])
     kinds = [ld.LayerConfig(ld.MIXER_LATENT, **attn, **moe), ld.LayerConfig(ld.MIXER_SSD, **s["ssd"], **dense), ld.LayerConfig(ld.MIXER_SSD, **s["ssd"], **moe)]
     return ld.LayeredConfig(s["width"], s["vocab"], 1e-6, [kinds[i % 3] for i in range(s["layers"])], norm=ld.NORM_LAYER, tied=False)
 

@@ -6,8 +6,9 @@
 //   layer norm     x += ls1 mixer(ln(norm1, x));             x += ls2 ff(ln(norm2, x))
 //
 // Layer norm needs the whole row: the projection that ends a sublayer adds its scaled result to the residual stream, and a
-// row kernel writes the next sublayer's input (behind experts it also adds up their outputs).  Dynamic Tanh needs no statistics, so all of it folds into the projection that ends a sublayer: its epilogue adds
-// the normalised result to the f32 residual stream and hands on the normalised input of the next sublayer.  Per layer:
+// row kernel writes the next sublayer's input (behind experts it also adds up their outputs).
+// Dynamic Tanh needs no statistics, so all of it folds into the projection that ends a sublayer: its epilogue adds the
+// normalised result to the f32 residual stream and hands on the normalised input of the next sublayer.  Per layer:
 //   1. [q;k;v(;gates)] projection; attention: rotary positions and the KV write in its epilogue
 //   2. attention (with its own normalisation in the same kernel); or the recurrence with head norm and output gate in the
 //      same kernel
