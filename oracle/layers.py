@@ -388,3 +388,195 @@ class Lilosun:
             if layer_outputs is not None:
                 layer_outputs.append(x.copy())
         return linear(self.t["head"], layer_norm(x, self.t["final.norm"], eps)) * self.c["logit_scale"]
+
+
+# ---- mechanisms of Rubuvik ------------------------------------------------------------------------------------------
+
+def rms_around_one(x, w, eps):
+    """Unit root mean square, times 1 + w: the stored weight says by how much a channel differs from 1."""
+    return unit_rms(x, eps) * (1 + w)
+
+
+def distance_slopes(heads):
+    """How much a head takes off a score per token of distance: 2^(-8 (n + 1) / heads), n = 0, 1, ..."""
+    return 2.0 ** (-8.0 * (np.arange(heads) + 1) / heads)
+
+
+def query_temperature(positions, coef, every):
+    """1 + coef ln(1 + number of whole stretches of ``every`` tokens up to and with the position)."""
+    return 1 + coef * np.log(np.floor((np.asarray(positions, np.float64) + 1) / every) + 1)
+
+
+def biased_window_softmax(q, k, v, scale, slope, window, sink=None):
+    """One head: scores scale (q_t . k_s) - slope (t - s) over 0 <= t - s < window; ``sink`` adds exp(sink) to the sum of weights."""
+    out = np.zeros((q.shape[0], v.shape[1]), q.dtype)
+    for t in range(q.shape[0]):
+        lo = 0 if window is None else max(0, t - window + 1)
+        s = (k[lo:t + 1] @ q[t]) * scale - slope * (t - np.arange(lo, t + 1))
+        top = s.max() if sink is None else max(s.max(), sink)
+        p = np.exp(s - top)
+        out[t] = (p @ v[lo:t + 1]) / (p.sum() + (0 if sink is None else np.exp(sink - top)))
+    return out
+
+
+def mixed_values(v, first, lam):
+    """Values drawn towards those that the first layer of the kind gave the same token."""
+    return (1 - lam) * v + lam * first
+
+
+def biased_attention(h, w, heads, kv_heads, dim, vdim, scale, window, eps, temperature=None, biases=False, unit_qk=False, sink=False, gate=False,
+                     first=None):
+    """w: dict q, k, v, o and what the options need (q.b, k.b, v.b; sink; g; vmix).  ``temperature``: (coef, every).  ``first``: the first
+    layer's values [T, kv_heads, vdim] to mix in.  -> (output, this layer's values before mixing)."""
+    T = h.shape[0]
+
+    def part(name, n, d):
+        return (linear(w[name], h) + (w[name + ".b"] if biases else 0)).reshape(T, n, d)
+
+    q, k, v = part("q", heads, dim), part("k", kv_heads, dim), part("v", kv_heads, vdim)
+    own = v
+    if unit_qk:
+        q, k = unit_rms(q, eps), unit_rms(k, eps)
+    if temperature is not None:
+        q = q * query_temperature(np.arange(T), *temperature)[:, None, None].astype(q.dtype)
+    if first is not None:
+        v = mixed_values(v, first, w["vmix"])
+    slopes = distance_slopes(heads)
+    o = np.zeros((T, heads, vdim), h.dtype)
+    for n in range(heads):
+        g = n // (heads // kv_heads)
+        o[:, n] = biased_window_softmax(q[:, n], k[:, g], v[:, g], scale, slopes[n], window, w["sink"][n] if sink else None)
+    if gate:
+        o = o * sigmoid(linear(w["g"], h))[:, :, None]
+    return linear(w["o"], o.reshape(T, heads * vdim)), own
+
+
+def decayed_scan(q, k, v, decay, state):
+    """One head.  S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t.  -> (o [T, vdim], S)."""
+    S = state.copy()
+    o = np.zeros((q.shape[0], v.shape[1]), q.dtype)
+    for t in range(q.shape[0]):
+        S = decay * S + np.outer(k[t], v[t])
+        o[t] = S.T @ q[t]
+    return o, S
+
+
+def lightning(h, w, heads, dim, vdim, decay, eps):
+    """w: dict q, k, v, g, o, norm.  The heads are normalised together, the gate follows the norm."""
+    T = h.shape[0]
+    q, k = silu(linear(w["q"], h)).reshape(T, heads, dim), silu(linear(w["k"], h)).reshape(T, heads, dim)
+    v = silu(linear(w["v"], h)).reshape(T, heads, vdim)
+    o = np.zeros((T, heads, vdim), h.dtype)
+    for n in range(heads):
+        o[:, n] = decayed_scan(q[:, n], k[:, n], v[:, n], decay[n], np.zeros((dim, vdim), h.dtype))[0]
+    return linear(w["o"], unit_rms(o.reshape(T, heads * vdim), eps) * w["norm"] * sigmoid(linear(w["g"], h)))
+
+
+def softmax_scores(z):
+    p = np.exp(z - z.max(-1, keepdims=True))
+    return p / p.sum(-1, keepdims=True)
+
+
+def route_softmax(z, correction, top, groups, keep, scale):
+    """Router logits [tokens, experts] -> (chosen experts [tokens, top], their weights).  Groups of neighbouring experts compete
+    by their best corrected score; the weights are the plain scores of the chosen times ``scale``."""
+    s = softmax_scores(z)
+    choice = s + correction
+    T, E = z.shape
+    n = E // groups
+    ids = np.zeros((T, top), np.int64)
+    for t in range(T):
+        best = choice[t].reshape(groups, n).max(-1)
+        kept = np.argsort(-best, kind="stable")[:keep]
+        masked = np.full(E, -np.inf)
+        for g in kept:
+            masked[g * n:(g + 1) * n] = choice[t, g * n:(g + 1) * n]
+        ids[t] = np.argsort(-masked, kind="stable")[:top]
+    return ids, np.take_along_axis(s, ids, 1) * scale
+
+
+def route_softmax_margin(z, correction, top, groups, keep):
+    """As route_margin, for ``route_softmax``."""
+    choice = softmax_scores(z) + correction
+    out = np.full(z.shape[0], np.inf)
+    for t in range(z.shape[0]):
+        by_group = choice[t].reshape(groups, -1)
+        order = np.argsort(-by_group.max(-1))
+        if keep < groups:
+            best = by_group.max(-1)
+            out[t] = best[order[keep - 1]] - best[order[keep]]
+        c = np.sort(by_group[order[:keep]].ravel())[::-1]
+        if top < len(c):
+            out[t] = min(out[t], c[top - 1] - c[top])
+    return out
+
+
+def softmax_moe(h, w, top, groups, keep, scale, shared):
+    """w: dict router, correction, e<i>.gate/up/down and, with a shared expert, shared.gate/up/down."""
+    ids, weights = route_softmax(linear(w["router"], h), w["correction"], top, groups, keep, scale)
+    out = np.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, p in zip(ids[t], weights[t]):
+            n = f"e{e}."
+            out[t] += p * silu_mlp(h[t], w[n + "gate"], w[n + "up"], w[n + "down"])
+    if shared:
+        out = out + silu_mlp(h, w["shared.gate"], w["shared.up"], w["shared.down"])
+    return out
+
+
+def token_side(x, e, w, eps):
+    """What a layer's own row of the token table adds: w: dict gate, proj, norm; e [tokens, dim]."""
+    return unit_rms(linear(w["proj"], gelu_tanh(linear(w["gate"], x)) * e), eps) * w["norm"]
+
+
+class Rubuvik:
+    """The whole design from a config dict and a dict of float arrays under the checkpoint's tensor names."""
+
+    def __init__(self, config: dict, tensors: dict, dtype=np.float64):
+        self.c = config
+        self.t = {k: np.asarray(v, dtype) for k, v in tensors.items()}
+        self.margin = None    # per token of the last forward: the closest call of any router
+
+    def part(self, prefix):
+        return {k[len(prefix):]: v for k, v in self.t.items() if k.startswith(prefix)}
+
+    def norm(self, name, x):
+        return rms_around_one(x, self.t[name], self.c["norm"]["eps"])
+
+    def mixer(self, i, layer, h):
+        w, m, eps = self.part(f"l{i}.mix."), layer["mixer"], self.c["norm"]["eps"]
+        if layer["type"] == "lightning":
+            return lightning(h, w, m["heads"], m["dim"], m["vdim"], m["decay"], eps)
+        more = {"attention": {}, "attention_2": dict(biases=True, unit_qk=True, sink=True, gate=True)}[layer["type"]]
+        mask, temp, mix = m.get("mask"), m.get("q_temp"), m.get("v_mix", False)
+        y, v = biased_attention(h, w, m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["scale"], mask["size"] if mask else None, eps,
+                                temperature=(temp["coef"], temp["every"]) if temp else None, first=self.first_values if mix else None, **more)
+        if mix and self.first_values is None:
+            self.first_values = v
+        return y
+
+    def feed_forward(self, i, mlp, h):
+        w = self.part(f"l{i}.mlp.")
+        if mlp["kind"] == "dense":
+            return silu_mlp(h, w["gate"], w["up"], w["down"])
+        r, g = mlp["router"], mlp["router"].get("groups") or {"count": 1, "keep": 1}
+        self.margin = np.minimum(self.margin, route_softmax_margin(linear(w["router"], h), w["correction"], r["top"], g["count"], g["keep"]))
+        return softmax_moe(h, w, r["top"], g["count"], g["keep"], r["scale"], bool(mlp.get("shared")))
+
+    def forward(self, tokens, layer_outputs: list | None = None):
+        """Logits [tokens, vocab] of one sequence from its first token."""
+        tokens, eps, m, side = np.asarray(tokens), self.c["norm"]["eps"], self.c["residual_mult"], self.c["token_side"]
+        x = self.t["embed"][tokens] * self.c["embedding"]["scale"]
+        self.margin = np.full(len(tokens), np.inf)
+        self.first_values = None
+        for i, layer in enumerate(self.c["layers"]):
+            l = f"l{i}."
+            x = x + m * self.norm(l + "norm1b", self.mixer(i, layer, self.norm(l + "norm1", x)))
+            if layer.get("mlp"):
+                x = x + m * self.norm(l + "norm2b", self.feed_forward(i, layer["mlp"], self.norm(l + "norm2", x)))
+            if side:
+                d = side["dim"]
+                x = x + m * token_side(x, self.t["side.embed"][tokens, i * d:(i + 1) * d], self.part(l + "side."), eps)
+            if layer_outputs is not None:
+                layer_outputs.append(x.copy())
+        return linear(self.t["embed"], self.norm("final.norm", x))
