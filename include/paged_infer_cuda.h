@@ -365,11 +365,15 @@ pi_status pi_kv_fill_normal(pi_ctx* ctx, pi_kv_pool* pool, uint64_t seed, float 
  * pi_model_step like every other model; what its mixers carry from token to token lives in a KV pool (attention) and
  * in a state pool (recurrences).  No counterpart in the reference. */
 
-enum { PI_MIXER_ATTENTION = 0, PI_MIXER_GLA = 1, PI_MIXER_MLSTM = 2, PI_MIXER_LATENT = 3 /* latent attention */, PI_MIXER_SSD = 4 /* state-space, scalar decay */ };
-enum { PI_FF_GELU = 0, PI_FF_SILU = 1, PI_FF_EXPERTS = 2 /* clamped gated units, routed */ };
-/* Normalisation: Dynamic Tanh before and after every sublayer, or layer norm (a weight, no bias) before it and a scale per
- * channel behind it. */
-enum { PI_NORM_DYT = 0, PI_NORM_LAYER = 1 };
+enum { PI_MIXER_ATTENTION = 0, PI_MIXER_GLA = 1, PI_MIXER_MLSTM = 2, PI_MIXER_LATENT = 3 /* latent attention */, PI_MIXER_SSD = 4 /* state-space, scalar decay */,
+       PI_MIXER_LIGHTNING = 5 /* a constant decay per head */ };
+enum { PI_FF_GELU = 0, PI_FF_SILU = 1, PI_FF_EXPERTS = 2 /* routed */ };
+/* Experts: their units, and the scores the router makes of its logits. */
+enum { PI_UNIT_CLAMPED = 0 /* clamped gated units */, PI_UNIT_SILU = 1 };
+enum { PI_SCORE_SIGMOID = 0, PI_SCORE_SOFTMAX = 1 };
+/* Normalisation: Dynamic Tanh before and after every sublayer; or layer norm (a weight, no bias) before it and a scale per
+ * channel behind it; or RMS norm (times 1 + weight) before and after it, the result times residual_mult. */
+enum { PI_NORM_DYT = 0, PI_NORM_LAYER = 1, PI_NORM_RMS = 2 };
 
 typedef struct {
   int32_t mixer;
@@ -395,6 +399,17 @@ typedef struct {
    * every token meets (0: none); limits: where the units are clamped */
   int32_t experts, top, expert_groups, keep_groups, shared_ff;
   float limit, shared_limit;
+  /* attention with one map: biases of q, k and v; q and k brought to unit root mean square per head; a distance bias (head n takes
+   * 2^(-8 (n + 1) / heads) off a score per token of distance); a learned sink per head in the sum of weights; a gate per head;
+   * values mixed with those of the first layer that has v_mix; q times 1 + coef ln(floor((p + 1) / every) + 1) at position p
+   * (q_temp_every 0: not) */
+  int32_t biases, unit_qk, distance_bias, sink, head_gate, v_mix;
+  double q_temp_coef, q_temp_every;
+  const double* decay;     /* lightning: [heads], in [0, 1] */
+  /* experts: a group is as good as the sum of its group_best (1 or 2) best scores; renorm: the chosen weights are brought to sum 1;
+   * they are multiplied by route_scale; shared_gate: the shared expert has a gate per token */
+  int32_t unit, score, group_best, renorm, shared_gate;
+  float route_scale;
 } pi_layer_config;
 
 typedef struct {
@@ -405,6 +420,9 @@ typedef struct {
   int32_t norm;            /* PI_NORM_* */
   int32_t tied;            /* 1: the embedding is the output matrix, 0: "head" is */
   float logit_scale;
+  float embed_scale;       /* of the embedding, not of the output matrix */
+  float residual_mult;     /* PI_NORM_RMS: of everything that is added to the residual stream */
+  int32_t side_dim;        /* PI_NORM_RMS: channels of a layer's own row of a table of tokens, added behind its sublayers; 0: none */
   const pi_layer_config* layers;
 } pi_layered_config;
 

@@ -66,12 +66,16 @@ class LayerConfigC(C.Structure):
                [(n, C.c_int32) for n in ("ff", "ff_kind", "rank")] + \
                [(n, C.c_double) for n in ("rot_factor", "rot_original", "rot_fast", "rot_slow")] + \
                [(n, C.c_int32) for n in ("groups", "norm_groups", "conv", "experts", "top", "expert_groups", "keep_groups", "shared_ff")] + \
-               [(n, C.c_float) for n in ("limit", "shared_limit")]
+               [(n, C.c_float) for n in ("limit", "shared_limit")] + \
+               [(n, C.c_int32) for n in ("biases", "unit_qk", "distance_bias", "sink", "head_gate", "v_mix")] + \
+               [(n, C.c_double) for n in ("q_temp_coef", "q_temp_every")] + [("decay", C.POINTER(C.c_double))] + \
+               [(n, C.c_int32) for n in ("unit", "score", "group_best", "renorm", "shared_gate")] + [("route_scale", C.c_float)]
 
 
 class LayeredConfigC(C.Structure):
     _fields_ = [("width", C.c_int32), ("vocab_size", C.c_int32), ("num_layers", C.c_int32), ("norm_eps", C.c_float), ("compute", C.c_int32),
-                ("max_rows", C.c_int32), ("norm", C.c_int32), ("tied", C.c_int32), ("logit_scale", C.c_float), ("layers", C.POINTER(LayerConfigC))]
+                ("max_rows", C.c_int32), ("norm", C.c_int32), ("tied", C.c_int32), ("logit_scale", C.c_float), ("embed_scale", C.c_float), ("residual_mult", C.c_float),
+                ("side_dim", C.c_int32), ("layers", C.POINTER(LayerConfigC))]
 
 
 class NamedTensorC(C.Structure):

@@ -611,13 +611,19 @@ class LayeredModel(_Steps):
 
     @classmethod
     def _config(cls, config: LayeredConfig, compute: str, max_rows: int) -> _lib.LayeredConfigC:
-        layers = (_lib.LayerConfigC * len(config.layers))(*[
-            _lib.LayerConfigC(l.mixer, l.heads, l.kv_heads, l.dim, l.vdim, l.maps, 0 if l.window is None else l.window, l.rot_dims, l.rot_base,
-                              l.scale, l.diff, l.tau, l.gate_cap, l.ff, l.ff_kind, l.rank, l.rot_factor, l.rot_original, l.rot_fast, l.rot_slow,
-                              l.groups, l.norm_groups, l.conv, l.experts, l.top, l.expert_groups, l.keep_groups, l.shared_ff, l.limit, l.shared_limit)
-            for l in config.layers])
+        layers = (_lib.LayerConfigC * len(config.layers))()
+        for c, l in zip(layers, config.layers):
+            for name, _ in _lib.LayerConfigC._fields_:
+                v = getattr(l, name)
+                if name == "decay":
+                    if v is not None and len(v) != l.heads:
+                        raise ValueError(f"{len(v)} decays for {l.heads} heads")
+                    v = None if v is None else (C.c_double * len(v))(*v)     # the structure keeps the array alive
+                elif name == "window":
+                    v = 0 if v is None else v
+                setattr(c, name, v)
         cfg = _lib.LayeredConfigC(config.width, config.vocab_size, len(config.layers), config.norm_eps, cls.COMPUTE[compute], max_rows, config.norm,
-                                  int(config.tied), config.logit_scale, layers)
+                                  int(config.tied), config.logit_scale, config.embed_scale, config.residual_mult, config.side_dim, layers)
         cfg._layers = layers
         return cfg
 

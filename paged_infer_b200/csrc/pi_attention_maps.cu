@@ -1,13 +1,14 @@
 // Windowed attention with one or two softmax maps per head over the same values (differential attention), reading the
 // paged KV pool.
 //
-//   score_j = scale (q_j . k_j)           j = map, over the keys t - window < s <= t
-//   a_j     = softmax(score_j) V
+//   score_j = scale (q_j . k_j) - slope (t - s)     j = map, over the keys t - window < s <= t; slope: of the head, if there is one
+//   a_j     = softmax(score_j) V          (with a sink, exp(sink) is one more term of the denominator)
 //   out     = a_1                                             (one map)
 //   o = a_1 - lambda a_2;  out = out_scale o / rms(o)          (two maps)
-//   out *= sigmoid(gate)                                       (with an output gate)
+//   out *= sigmoid(gate)                                       (with an output gate, per channel or per head)
 //
-// Kernels: maps_rope_kv_kernel rotates q and k and writes k and v into the pool; maps_attn_plain_kernel is the f32
+// Kernels: maps_prepare_kernel brings q, k and v into their final form (bias, unit root mean square, rotation, temperature of the
+// queries, mixing of the values) and writes k and v into the pool; maps_attn_plain_kernel is the f32
 // path and the one for sizes the tensor-core kernels of pi_attention_maps_tc.cu do not hold.
 #include <math.h>
 
@@ -17,7 +18,7 @@
 
 namespace {
 
-struct RopeKvParams {
+struct PrepareParams {
   float* qkv;
   size_t stride;
   int heads, kv_heads, maps, dim, vdim, rot_dims;
@@ -26,53 +27,84 @@ struct RopeKvParams {
   int dp, vp, block_size;
   const int32_t *row_seq, *row_pos, *lens, *tables;
   int max_blocks;
+  float eps;
+  pi_maps_prepare x;
 };
 
-// CTA per row.  Work item: two adjacent channels of a q or k vector of one map (a rotation pair, rot_dims is even), or
-// one channel of v.  Pool rows are padded with zeros up to dp / vp.
+// Warp per vector of a row: a q or k vector of one map, or a head's values.  Lanes hold pairs of adjacent channels (rot_dims is
+// even, so a rotation pair stays together), up to kHeld of them in registers; longer vectors are read twice.  Pool rows are
+// padded with zeros up to dp / vp.
+constexpr int kPrepareWarps = 4, kHeld = 4;
 template <typename T>
-__global__ void __launch_bounds__(256) maps_rope_kv_kernel(const RopeKvParams p) {
-  const int row = blockIdx.x;
+__global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const PrepareParams p) {
+  const int row = blockIdx.x, lane = threadIdx.x & 31, vec = blockIdx.y * kPrepareWarps + (threadIdx.x >> 5);
+  const int nq = p.heads * p.maps, nk = p.kv_heads * p.maps, half = p.rot_dims >> 1;
   const int seq = p.row_seq[row], pos = p.row_pos[row];
   const int lb = pos / p.block_size, off = pos % p.block_size;
   const bool mapped = lb < p.lens[seq];
   const int pb = mapped ? p.tables[(size_t)seq * p.max_blocks + lb] : 0;
   pi_grid_dependency_wait();
-  float* x = p.qkv + (size_t)row * p.stride;
-  const int nq = p.heads * p.maps, nk = p.kv_heads * p.maps, half = p.rot_dims >> 1;
+  if (vec >= nq + nk + p.kv_heads) return;
+  const size_t tile = (size_t)p.block_size * (p.maps * p.dp + p.vp);
+  if (vec >= nq + nk) {
+    const int g = vec - nq - nk, at = (nq + nk) * p.dim + g * p.vdim;
+    const float* v = p.qkv + (size_t)row * p.stride + at;
+    T* dst = static_cast<T*>(p.base) + ((size_t)pb * p.kv_heads + g) * tile + (size_t)p.block_size * p.maps * p.dp + (size_t)off * p.vp;
+    for (int e = lane; e < p.vp; e += 32) {
+      float r = 0.f;
+      if (e < p.vdim) r = pi_mix_value(p.x.mix, row, g * p.vdim + e, v[e] + (p.x.bias ? __ldg(p.x.bias + at + e) : 0.f));
+      if (mapped) dst[e] = pi_from_f32<T>(r);
+    }
+    return;
+  }
+  const bool is_q = vec < nq;
   const int pairs = (p.dp + 1) >> 1;     // dp >= dim, the pad is written too
+  float* v = p.qkv + (size_t)row * p.stride + (size_t)vec * p.dim;   // k vectors follow the q vectors
+  const float* bias = p.x.bias ? p.x.bias + (size_t)vec * p.dim : nullptr;
+  auto load = [&](int j) {
+    const int d = 2 * j;
+    float2 c = make_float2(d < p.dim ? v[d] : 0.f, d + 1 < p.dim ? v[d + 1] : 0.f);
+    if (bias) {
+      if (d < p.dim) c.x += __ldg(bias + d);
+      if (d + 1 < p.dim) c.y += __ldg(bias + d + 1);
+    }
+    return c;
+  };
+  float2 held[kHeld];
+#pragma unroll
+  for (int i = 0; i < kHeld; ++i) held[i] = lane + 32 * i < pairs ? load(lane + 32 * i) : make_float2(0.f, 0.f);
+  float factor = is_q && p.x.q_temp ? __ldg(p.x.q_temp + pos) : 1.f;
+  if (p.x.unit_qk) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kHeld; ++i) ss = fmaf(held[i].x, held[i].x, fmaf(held[i].y, held[i].y, ss));
+    for (int j = lane + 32 * kHeld; j < pairs; j += 32) {
+      const float2 c = load(j);
+      ss = fmaf(c.x, c.x, fmaf(c.y, c.y, ss));
+    }
+    factor /= sqrtf(pi_warp_sum(ss) / (float)p.dim + p.eps);
+  }
+  const int kv = vec - nq, g = is_q ? 0 : kv / p.maps, m = kv - g * p.maps;
+  T* dst = static_cast<T*>(p.base) + ((size_t)pb * p.kv_heads + g) * tile + (size_t)off * p.maps * p.dp + (size_t)m * p.dp;
   const float* cs = p.rope_cos + (size_t)pos * half;
   const float* sn = p.rope_sin + (size_t)pos * half;
-  const size_t tile = (size_t)p.block_size * (p.maps * p.dp + p.vp);
-  for (int i = threadIdx.x; i < (nq + nk) * pairs; i += blockDim.x) {
-    const int vec = i / pairs, j = i - vec * pairs, d = 2 * j;
-    const bool is_q = vec < nq;
-    if (is_q && j >= half) continue;     // q stays where it is
-    if (!is_q && !mapped) continue;
-    float* v = x + (size_t)vec * p.dim;  // k vectors follow the q vectors
-    float a = d < p.dim ? v[d] : 0.f, c = d + 1 < p.dim ? v[d + 1] : 0.f;
-    if (j < half) {
-      const float na = a * cs[j] - c * sn[j], nc = c * cs[j] + a * sn[j];
-      a = na;
-      c = nc;
-    }
+  auto finish = [&](int j, float2 c) {
+    const int d = 2 * j;
+    if (j < half) c = make_float2(c.x * cs[j] - c.y * sn[j], c.y * cs[j] + c.x * sn[j]);
+    c.x *= factor;
+    c.y *= factor;
     if (is_q) {
-      v[d] = a;
-      v[d + 1] = c;
-    } else {
-      const int kv = vec - nq, g = kv / p.maps, m = kv - g * p.maps;
-      T* dst = static_cast<T*>(p.base) + ((size_t)pb * p.kv_heads + g) * tile + (size_t)off * p.maps * p.dp + (size_t)m * p.dp;
-      dst[d] = pi_from_f32<T>(a);
-      dst[d + 1] = pi_from_f32<T>(c);
+      if (d < p.dim) v[d] = c.x;
+      if (d + 1 < p.dim) v[d + 1] = c.y;
+    } else if (mapped) {
+      dst[d] = pi_from_f32<T>(c.x);
+      dst[d + 1] = pi_from_f32<T>(c.y);
     }
-  }
-  if (!mapped) return;
-  const float* vsrc = x + (size_t)(nq + nk) * p.dim;
-  for (int i = threadIdx.x; i < p.kv_heads * p.vp; i += blockDim.x) {
-    const int g = i / p.vp, e = i - g * p.vp;
-    T* dst = static_cast<T*>(p.base) + ((size_t)pb * p.kv_heads + g) * tile + (size_t)p.block_size * p.maps * p.dp + (size_t)off * p.vp;
-    dst[e] = pi_from_f32<T>(e < p.vdim ? vsrc[(size_t)g * p.vdim + e] : 0.f);
-  }
+  };
+#pragma unroll
+  for (int i = 0; i < kHeld; ++i)
+    if (lane + 32 * i < pairs) finish(lane + 32 * i, held[i]);
+  for (int j = lane + 32 * kHeld; j < pairs; j += 32) finish(j, load(j));
 }
 
 // One CTA of 4 warps per (row, head): the warps take every fourth key and merge; lanes hold the channels.  f32
@@ -97,6 +129,7 @@ __global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const
   const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
   const size_t tile = (size_t)p.block_size * (nm * DP + p.vp);
   float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  const float slope = p.slopes ? __ldg(p.slopes + head) : 0.f, sink = p.sinks ? __ldg(p.sinks + head) : -INFINITY;
   for (int t = lo + warp; t <= pos; t += kPlainWarps) {
     const int lb = t / p.block_size, off = t - lb * p.block_size;
     if (lb >= len) break;
@@ -109,7 +142,7 @@ __global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const
       if (m >= nm) break;
       float d = 0.f;
       for (int i = lane; i < p.dim; i += 32) d = fmaf(sq[m * p.dim + i], pi_to_f32(kt[m * DP + i]), d);
-      const float s = pi_warp_sum(d) * p.scale;
+      const float s = pi_warp_sum(d) * p.scale - slope * (float)(pos - t);
       const float mn = fmaxf(mx[m], s), keep = expf(mx[m] - mn), w = expf(s - mn);
       mx[m] = mn;
       l[m] = l[m] * keep + w;
@@ -124,8 +157,9 @@ __global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const
   __syncthreads();
   float f[2][kPlainWarps];
   for (int m = 0; m < nm; ++m) {
-    float M = -INFINITY, L = 0.f;
+    float M = sink, L = 0.f;
     for (int w = 0; w < kPlainWarps; ++w) M = fmaxf(M, s_m[w][m]);
+    if (p.sinks) L = expf(sink - M);
     for (int w = 0; w < kPlainWarps; ++w) L += s_m[w][m] == -INFINITY ? 0.f : s_l[w][m] * expf(s_m[w][m] - M);
     for (int w = 0; w < kPlainWarps; ++w) f[m][w] = s_m[w][m] == -INFINITY ? 0.f : expf(s_m[w][m] - M) / L;
   }
@@ -148,19 +182,20 @@ __global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const
     r = p.out_scale / sqrtf(t / (float)p.vdim + p.eps);
   }
   O* o = static_cast<O*>(p.out) + (size_t)row * p.out_stride + (size_t)head * p.vdim;
-  const float* gate = p.gate ? p.gate + (size_t)row * p.gate_stride + (size_t)head * p.vdim : nullptr;
-  for (int e = tid; e < p.vdim; e += blockDim.x) o[e] = pi_from_f32<O>(acc[e] * (gate ? r * pi_sigmoid(gate[e]) : r));
+  const float* gate = p.gate ? p.gate + (size_t)row * p.gate_stride + (p.gate_per_head ? head : (size_t)head * p.vdim) : nullptr;
+  for (int e = tid; e < p.vdim; e += blockDim.x) o[e] = pi_from_f32<O>(acc[e] * (gate ? r * pi_sigmoid(gate[p.gate_per_head ? 0 : e]) : r));
 }
 
 }  // namespace
 
-pi_status pi_launch_maps_rope_kv(pi_ctx* ctx, const pi_maps_attention& a, const pi_kv_view& kv, float* qkv, size_t stride,
+pi_status pi_launch_maps_prepare(pi_ctx* ctx, const pi_maps_attention& a, const pi_maps_prepare& x, const pi_kv_view& kv, float* qkv, size_t stride,
                                  const pi_seq_batch& b) {
   pi_prof_scope prof(ctx, PI_PROF_ROPE_KV);
-  RopeKvParams p = {qkv, stride, a.heads, a.kv_heads, a.maps, a.dim, a.vdim, a.rot_dims, a.rope_cos, a.rope_sin, kv.base, kv.dp, kv.vp,
-                    kv.block_size, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks};
-  PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, kv.kind == PI_BF16 ? maps_rope_kv_kernel<__nv_bfloat16> : maps_rope_kv_kernel<float>,
-                                  dim3(b.rows), dim3(256), 0, 1, p));
+  PrepareParams p = {qkv, stride, a.heads, a.kv_heads, a.maps, a.dim, a.vdim, a.rot_dims, a.rope_cos, a.rope_sin, kv.base, kv.dp, kv.vp,
+                     kv.block_size, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks, a.eps, x};
+  const int vectors = (a.heads + a.kv_heads) * a.maps + a.kv_heads;
+  PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, kv.kind == PI_BF16 ? maps_prepare_kernel<__nv_bfloat16> : maps_prepare_kernel<float>,
+                                  dim3(b.rows, (vectors + kPrepareWarps - 1) / kPrepareWarps), dim3(kPrepareWarps * 32), 0, 1, p));
   return PI_OK;
 }
 
@@ -168,10 +203,11 @@ pi_status pi_launch_maps_attention(pi_ctx* ctx, const pi_maps_attention& a, cons
                                    void* out, size_t out_stride, int out_kind, const pi_seq_batch& b) {
   pi_prof_scope prof(ctx, PI_PROF_ATTENTION);
   MapsParams p = {qkv, stride, out, out_stride, kv.base, a.heads, a.kv_heads, a.maps, a.dim, a.vdim, kv.dp, kv.vp, kv.block_size,
-                  a.window, a.scale, a.eps, a.lambda, a.out_scale, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks, a.gate, a.gate_stride, a.v_in_k};
+                  a.window, a.scale, a.eps, a.lambda, a.out_scale, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks, a.gate, a.gate_stride, a.gate_per_head,
+                  a.slopes, a.sinks, a.v_in_k};
   if (pi_maps_attention_tc_usable(ctx, a, kv)) return pi_launch_maps_attention_tc(ctx, p, out_kind, b);
   const size_t smem = sizeof(float) * ((size_t)a.maps * a.dim + (size_t)kPlainWarps * a.maps * a.vdim);
-  PI_REQUIRE(ctx, smem <= 48 * 1024, "attention heads of %d / %d channels are too wide", a.dim, a.vdim);
+  PI_REQUIRE(ctx, smem <= kSmemFit, "attention heads of %d / %d channels are too wide", a.dim, a.vdim);
   auto k = kv.kind == PI_BF16 ? (out_kind == PI_BF16 ? maps_attn_plain_kernel<__nv_bfloat16, __nv_bfloat16> : maps_attn_plain_kernel<__nv_bfloat16, float>)
                               : (out_kind == PI_BF16 ? maps_attn_plain_kernel<float, __nv_bfloat16> : maps_attn_plain_kernel<float, float>);
   // grid.y is limited to 65535 rows, far above any step

@@ -15,6 +15,8 @@ struct MapsParams {
   int max_blocks;
   const float* gate;
   size_t gate_stride;
+  int gate_per_head;
+  const float *slopes, *sinks;
   int v_in_k;
 };
 

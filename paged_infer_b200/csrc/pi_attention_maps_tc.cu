@@ -1,5 +1,5 @@
 // Multi-map windowed attention over a bf16 KV pool on the tensor cores (mma.sync; see pi_attention_maps.cu for the
-// mathematics).  Scores and weights are f32; the weights enter the product with V as two bf16 planes (16 bits).
+// mathematics).  Scores (in the log2 domain, the distance bias with them) and weights are f32; the weights enter the product with V as two bf16 planes (16 bits).
 //
 // maps_decode_kernel: one row alone.  CTA = (row, kv head, group of heads, KV split).  The MMA's 16 rows are 16 heads, or
 //   8 heads x 2 maps: with two maps the query operand is block diagonal - rows 0-7 hold map 1 in the first half of the
@@ -189,6 +189,11 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
     for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
   float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const float sc = a.scale * kLog2e;
+  float slope[2] = {0.f, 0.f};
+  if (a.slopes) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) slope[h] = __ldg(a.slopes + g * p.group + min(grp * HR + ((lane >> 2) + 8 * h) % HR, p.group - 1)) * kLog2e;
+  }
 
   int stage = 0;
   for (int tile = tile0; tile < tile_end; tile += kDecWarps) {
@@ -223,7 +228,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int t = key + 8 * j + (i & 1);
-        s[j][i] = (t >= lo && t < hi) ? s[j][i] * sc : -INFINITY;
+        s[j][i] = (t >= lo && t < hi) ? fmaf(slope[i >> 1], (float)(t - pos), s[j][i] * sc) : -INFINITY;
       }
     uint32_t ph[4], pl[4];
     float keep[2];
@@ -341,11 +346,13 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
           f[m][c] = pm[c][h + m * HR];
           l[m][c] = pl[c][h + m * HR];
         }
+      const float sink = a.sinks ? __ldg(a.sinks + g * p.group + head) * kLog2e : -INFINITY;
 #pragma unroll
       for (int m = 0; m < MAPS; ++m) {
-        float M = -INFINITY, L = 0.f;
+        float M = sink, L = 0.f;
 #pragma unroll
         for (int c = 0; c < NS; ++c) M = fmaxf(M, f[m][c]);
+        if (a.sinks) L = exp2f(sink - M);
 #pragma unroll
         for (int c = 0; c < NS; ++c) {
           f[m][c] = c >= p.nsplit || f[m][c] == -INFINITY ? 0.f : exp2f(f[m][c] - M);
@@ -376,7 +383,8 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
 #pragma unroll
       for (int i = 0; i < VMAX / 32; ++i)
         if (lane + 32 * i < a.vdim) {
-          const float gate = a.gate ? pi_sigmoid(a.gate[(size_t)row * a.gate_stride + (size_t)(g * p.group + head) * a.vdim + lane + 32 * i]) : 1.f;
+          const size_t at = a.gate_per_head ? (size_t)(g * p.group + head) : (size_t)(g * p.group + head) * a.vdim + lane + 32 * i;
+          const float gate = a.gate ? pi_sigmoid(a.gate[(size_t)row * a.gate_stride + at]) : 1.f;
           store_out(p, o0 + lane + 32 * i, d[i] * r * gate);
         }
     }
@@ -477,6 +485,13 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
     for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
   float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const float sc = a.scale * kLog2e;
+  float slope[2], sink[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int head = g * p.group + (rg * 16 + (lane >> 2) + 8 * h) % p.group;
+    slope[h] = a.slopes ? __ldg(a.slopes + head) * kLog2e : 0.f;
+    sink[h] = a.sinks ? __ldg(a.sinks + head) * kLog2e : -INFINITY;
+  }
   const int win = a.window > 0 ? a.window : 0x3fffffff;
 
   for (int kb = 0; kb < n_blocks; ++kb) {
@@ -514,7 +529,7 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
         for (int i = 0; i < 2; ++i) {
           const int t = t0 + j * 8 + (lane & 3) * 2 + i;
           float& v = s[j][2 * h + i];
-          v = (inside || (t <= tpos[h] && t > tpos[h] - win && t < hi)) ? v * sc : -INFINITY;
+          v = (inside || (t <= tpos[h] && t > tpos[h] - win && t < hi)) ? fmaf(slope[h], (float)(t - tpos[h]), v * sc) : -INFINITY;
           tm = fmaxf(tm, v);
         }
       mx[h] = new_max(mx[h], quad_max(tm), keep[h]);
@@ -558,8 +573,9 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
   float inv[2];
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
-    const float t = quad_sum(l[h]);
-    inv[h] = t > 0.f ? 1.f / t : 0.f;
+    const float M = fmaxf(mx[h], sink[h]), f = mx[h] == -INFINITY ? 0.f : exp2f(mx[h] - M);   // the sink joins in
+    const float t = quad_sum(l[h]) * f + (a.sinks ? exp2f(sink[h] - M) : 0.f);
+    inv[h] = t > 0.f ? f / t : 0.f;
   }
   float ss[2] = {0.f, 0.f};
   const int apitch = a.vp + 8, r0 = rg * 16 + (lane >> 2);
@@ -591,11 +607,13 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
           ss[h] = fmaf(v, v, ss[h]);
         }
     }
+  float hg[2] = {1.f, 1.f};
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const float r = MAPS == 2 ? a.out_scale / sqrtf(quad_sum(ss[h]) / (float)a.vdim + a.eps) : 1.f;
     const int rr = r0 + 8 * h, tok = rr / p.group, head = rr - tok * p.group;
     if (tpos[h] < 0) continue;
+    if (a.gate && a.gate_per_head) hg[h] = pi_sigmoid(a.gate[(size_t)(row0 + tok0 + tok) * a.gate_stride + g * p.group + head]);
     const size_t o0 = (size_t)(row0 + tok0 + tok) * a.out_stride + (size_t)(g * p.group + head) * a.vdim;
 #pragma unroll
     for (int j = 0; j < VMAX / 8; ++j)
@@ -603,9 +621,15 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
         const int c = j * 8 + (lane & 3) * 2;
         float v0 = acc[j][2 * h] * r, v1 = acc[j][2 * h + 1] * r;
         if (a.gate) {
-          const float* gate = a.gate + (size_t)(row0 + tok0 + tok) * a.gate_stride + (size_t)(g * p.group + head) * a.vdim;
-          v0 *= pi_sigmoid(gate[min(c, a.vdim - 1)]);
-          v1 *= pi_sigmoid(gate[min(c + 1, a.vdim - 1)]);
+          const float* gate = a.gate + (size_t)(row0 + tok0 + tok) * a.gate_stride;
+          if (a.gate_per_head) {
+            v0 *= hg[h];
+            v1 *= hg[h];
+          } else {
+            gate += (size_t)(g * p.group + head) * a.vdim;
+            v0 *= pi_sigmoid(gate[min(c, a.vdim - 1)]);
+            v1 *= pi_sigmoid(gate[min(c + 1, a.vdim - 1)]);
+          }
         }
         if (p.out_bf16 && c + 1 < a.vdim && ((o0 + c) & 1) == 0) {
           *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(a.out) + o0 + c) = pack(v0, v1);
@@ -658,7 +682,7 @@ cudaError_t grant(pi_ctx* ctx, TcKernel k, size_t smem) {
     }
   granted.push_back({k, pi_smem_grant()});
   granted.back().second.of(ctx) = smem;
-  return smem > 48 * 1024 ? cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : cudaSuccess;
+  return smem > kSmemFree ? cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : cudaSuccess;
 }
 
 }  // namespace

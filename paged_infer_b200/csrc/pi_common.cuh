@@ -154,7 +154,8 @@ enum pi_epilogue {
   PI_EPI_MAPS_QKV = 5,  // fused [q;k;v] of multi-map attention: rotary q to `out`, rotary k and v into the paged pool (pi_maps_kv)
   PI_EPI_DYT_RESIDUAL = 4,  // x[m][r] += dyt(post, v); h[m][r] = dyt(next, x[m][r])   (pi_dyt_residual)
   PI_EPI_CLAMP_GLU = 6,     // rows interleaved gate/up: g = min(gate, limit), u = clamp(up, +-limit): g sigmoid(1.702 g) (u + 1)
-  PI_EPI_SCALE_ADD = 7      // out[m][r] += out_scale[r] v        (residual add with a layer scale)
+  PI_EPI_SCALE_ADD = 7,     // out[m][r] += out_scale[r] v        (residual add with a layer scale)
+  PI_EPI_GELU_TABLE = 8     // out[m][r] = gelu_tanh(v) table[token of m][r]   (pi_token_table)
 };
 inline bool pi_epi_glu(pi_epilogue e) { return e == PI_EPI_SWIGLU || e == PI_EPI_GEGLU || e == PI_EPI_CLAMP_GLU; }
 
@@ -208,6 +209,15 @@ struct pi_rope_kv {
   const pi_attn_batch* batch = nullptr;
 };
 
+// Values of the attention layers of a model drawn towards those of the first of them: that one keeps its values, the others
+// take (1 - lambda) v + lambda first, row by row of the step.
+struct pi_value_mix {
+  float* first = nullptr;            // [rows][stride]; null: values stay as they are
+  size_t stride = 0;
+  float lambda = 0.f;
+  int keeps = 0;                     // 1: this layer is the first
+};
+
 // Where the epilogue of the fused [q;k;v] projection of a layered design puts its result: q rotated into `out`, k rotated
 // and v into the row's place in the pool (skipped when its block is not mapped).  Rotation pairs are adjacent channels, so
 // dim must be even (odd ones take pi_launch_maps_rope_kv).
@@ -218,6 +228,17 @@ struct pi_maps_kv {
   int kind = PI_F32, kv_heads = 0, dp = 0, vp = 0, block_size = 1;
   const int32_t *row_seq = nullptr, *row_pos = nullptr, *lens = nullptr, *tables = nullptr;
   int max_blocks = 0;
+  const float* bias = nullptr;       // [q_rows + k_rows + v rows]
+  const float* q_temp = nullptr;     // [positions] factor of q
+  pi_value_mix mix;
+};
+
+// Rows of a table of bf16 numbers, chosen by token.
+struct pi_token_table {
+  const uint16_t* base = nullptr;
+  size_t ld = 0;
+  int vocab = 1;
+  const uint32_t* tokens = nullptr;  // [M]
 };
 
 // A stack of equal matrices (the experts of a layer, one below the other), of which every row of the batch uses one.
@@ -267,6 +288,7 @@ struct pi_linear_args {
   float* rest = nullptr;
   size_t rest_stride = 0;
   const float* out_scale = nullptr;            // PI_EPI_SCALE_ADD
+  pi_token_table table;                        // PI_EPI_GELU_TABLE
   const pi_expert_rows* experts = nullptr;     // lin is a stack of experts
 };
 
@@ -418,6 +440,9 @@ pi_status pi_tp_peer_reduce_add(pi_ctx* ctx, float* x, int rows, int cols, pi_ac
 // ---- device helpers ----------------------------------------------------------------------
 // cudaFuncSetAttribute(MaxDynamicSharedMemorySize) is per device and slow: what each launcher has already been granted,
 // per device of the calling context.
+// A kernel may use 48 KB of shared memory without asking, its static part counted: up to kSmemFree of dynamic memory nobody
+// has to ask; kSmemFit is what kernels with less than 1 KB of static memory can have at most without it.
+constexpr size_t kSmemFree = 40 * 1024, kSmemFit = 47 * 1024;
 struct pi_smem_grant {
   size_t bytes[64] = {};
   size_t& of(const pi_ctx* ctx) { return bytes[(unsigned)ctx->device & 63u]; }
@@ -499,6 +524,22 @@ __device__ __forceinline__ void pi_maps_kv_store(const pi_maps_kv& k, const pi_m
   const size_t i = (size_t)block * k.kv_heads * ((size_t)k.block_size * (k.maps * k.dp + k.vp)) + c.elem + (size_t)off * c.step;
   if (k.kind == PI_BF16) static_cast<__nv_bfloat16*>(k.base)[i] = __float2bfloat16_rn(v);
   else static_cast<float*>(k.base)[i] = v;
+}
+__device__ __forceinline__ float pi_mix_value(const pi_value_mix& x, int row, int channel, float v) {
+  if (!x.first) return v;
+  float* f = x.first + (size_t)row * x.stride + channel;
+  if (x.keeps) *f = v;
+  else v = fmaf(x.lambda, *f, (1.f - x.lambda) * v);
+  return v;
+}
+// Column n of [q;k;v] of row m on its way out (behind bias and rotation): queries grow with the position, values are mixed.
+__device__ __forceinline__ float pi_maps_finish(const pi_maps_kv& k, const pi_maps_col& c, int m, int n, int pos, float v) {
+  if (c.is_q) return k.q_temp ? v * __ldg(k.q_temp + pos) : v;
+  if (n >= k.q_rows + k.k_rows) return pi_mix_value(k.mix, m, n - k.q_rows - k.k_rows, v);
+  return v;
+}
+__device__ __forceinline__ float pi_table_value(const pi_token_table& t, int m, int n) {
+  return __uint_as_float((uint32_t)__ldg(t.base + (size_t)(t.tokens[m] % (uint32_t)t.vocab) * t.ld + n) << 16);
 }
 // z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 __device__ __forceinline__ float pi_gelu_tanh(float z) {

@@ -50,12 +50,13 @@ struct Bf16GemmParams {
   pi_dyt_residual res;
   pi_maps_kv mkv;
   const float* out_scale;
+  pi_token_table table;
   float glu_limit;
   int glu_rows;
   float* rest;
   size_t rest_stride;
-  const int4* table;              // GROUPED
-  const int32_t* n_table;
+  const int4* tile_table;         // GROUPED
+  const int32_t* n_tiles;
   int* err_flag;
 };
 
@@ -116,13 +117,15 @@ __device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int M, int n, 
         sn[j] = __ldg(k.rope_sin + at);
       }
     }
+    const float bias = k.bias ? __ldg(k.bias + min(n, p.N - 1)) : 0.f;
 #pragma unroll
     for (int j = 0; j < C; ++j) {
-      const float other = __shfl_xor_sync(0xffffffffu, v[j], 1);
-      const int block = __shfl_sync(0xffffffffu, mine.block, j), off = __shfl_sync(0xffffffffu, mine.off, j);
-      float r = v[j];
-      if (col.rotated) r = (n & 1) ? v[j] * cs[j] + other * sn[j] : v[j] * cs[j] - other * sn[j];
+      float r = v[j] + bias;
+      const float other = __shfl_xor_sync(0xffffffffu, r, 1);
+      const int pos = __shfl_sync(0xffffffffu, mine.pos, j), block = __shfl_sync(0xffffffffu, mine.block, j), off = __shfl_sync(0xffffffffu, mine.off, j);
+      if (col.rotated) r = (n & 1) ? r * cs[j] + other * sn[j] : r * cs[j] - other * sn[j];
       if (!ok || m + j * dm >= M) continue;
+      r = pi_maps_finish(k, col, m + j * dm, n, pos, r);
       if (col.is_q) p.out[(size_t)(m + j * dm) * p.out_stride + n] = r;
       else pi_maps_kv_store(k, col, block, off, r);
     }
@@ -155,6 +158,13 @@ __device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int M, int n, 
 #pragma unroll
     for (int j = 0; j < C; ++j)
       if (ok && m + j * dm < M) p.out[(size_t)(m + j * dm) * p.out_stride + n] = fmaf(w, v[j], old[j]);
+  } else if (p.epi == PI_EPI_GELU_TABLE) {
+    float e[C];
+#pragma unroll
+    for (int j = 0; j < C; ++j) e[j] = pi_table_value(p.table, min(m + j * dm, M - 1), min(n, p.N - 1));
+#pragma unroll
+    for (int j = 0; j < C; ++j)
+      if (ok && m + j * dm < M) p.out_bf16[(size_t)(m + j * dm) * p.out_stride + n] = __float2bfloat16_rn(pi_gelu_tanh(v[j]) * e[j]);
   } else if (p.out_bf16) {
 #pragma unroll
     for (int j = 0; j < C; ++j)
@@ -193,7 +203,7 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
   auto tile_at = [&](int tile) {
     TileAt t = {0, (tile / p.rtiles) * BN, p.M};
     if (GROUPED) {
-      const int4 e = p.table[tile / p.rtiles];
+      const int4 e = p.tile_table[tile / p.rtiles];
       t.expert = e.x;
       t.m0 = e.y;
       t.m_end = e.y + e.z;
@@ -236,7 +246,7 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
       if (GROUPED) {
         pi_grid_dependency_wait();
         s_dep_ok = 1;
-        my_tiles = count(*p.n_table * p.rtiles);
+        my_tiles = count(*p.n_tiles * p.rtiles);
       }
       const int total = my_tiles * nk;
       auto load_w = [&](int it) {
@@ -270,7 +280,7 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
     if (lane == 0) {
       if (GROUPED) {
         pi_grid_dependency_wait();
-        my_tiles = count(*p.n_table * p.rtiles);
+        my_tiles = count(*p.n_tiles * p.rtiles);
       }
       const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(kTM >> 4) << 24);
       int it = 0;
@@ -307,7 +317,7 @@ gemm_bf16_kernel(const Bf16GemmParams p, const __grid_constant__ CUtensorMap map
       for (int c = tid; c < BN && (tile0 / p.rtiles) * BN + c < p.M; c += kEpiWarps * 32)
         s_place[c] = pi_maps_kv_place(p.mkv, (tile0 / p.rtiles) * BN + c);
     pi_grid_dependency_wait();   // the epilogue reads and writes what the preceding kernels use
-    if (GROUPED) my_tiles = count(*p.n_table * p.rtiles);
+    if (GROUPED) my_tiles = count(*p.n_tiles * p.rtiles);
     for (int t = 0; t < my_tiles; ++t) {
       const int a = t % kAcc, tile = tile0 + t * tile_step;
       int got = 0;
@@ -462,7 +472,7 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
   const int N = (int)(ex ? lin->rows / ex->experts : lin->rows);
   const bool glu = pi_epi_glu(a.epi) && a.out_bf16 && (a.glu_rows ? a.glu_rows % 2 == 0 && a.glu_rows <= N && a.rest : N % 2 == 0);
   PI_REQUIRE(ctx, a.epi == PI_EPI_STORE || glu || (a.epi == PI_EPI_MAPS_QKV && a.maps_kv && a.maps_kv->dim % 2 == 0) ||
-                      (a.epi == PI_EPI_SCALE_ADD && a.out && a.out_scale) ||
+                      (a.epi == PI_EPI_SCALE_ADD && a.out && a.out_scale) || (a.epi == PI_EPI_GELU_TABLE && a.out_bf16 && a.table.base && a.table.tokens) ||
                       (a.epi == PI_EPI_DYT_RESIDUAL && a.residual && a.residual->x && a.residual->h && a.residual->post.w && a.residual->next.w),
              "this epilogue is not built for the bf16 GEMM");
   Bf16GemmParams p = {};
@@ -470,6 +480,7 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
   p.out_bf16 = a.out_bf16;
   p.out_stride = a.out_stride;
   p.out_scale = a.out_scale;
+  p.table = a.table;
   p.glu_limit = a.glu_limit;
   p.glu_rows = a.glu_rows ? a.glu_rows : N;
   p.rest = a.rest;
@@ -490,8 +501,8 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
   }
   if (ex) {
     bn = ex->tile_rows;
-    p.table = ex->tiles;
-    p.n_table = ex->n_tiles;
+    p.tile_table = ex->tiles;
+    p.n_tiles = ex->n_tiles;
   }
   p.tiles = p.rtiles * (ex ? ex->max_tiles : (a.M + bn - 1) / bn);
   CUtensorMap w, x;

@@ -85,6 +85,7 @@ struct GemvParams {
   pi_dyt_residual res;   // PI_EPI_DYT_RESIDUAL
   pi_maps_kv mkv;        // PI_EPI_MAPS_QKV
   const float* out_scale;   // PI_EPI_SCALE_ADD
+  pi_token_table table;     // PI_EPI_GELU_TABLE
   float glu_limit;          // PI_EPI_CLAMP_GLU
   int glu_rows;             // gated epilogues: rows behind go to `rest`
   float* rest;
@@ -475,6 +476,10 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
           if (lane == m && m < mcount) {
             float a[kRows] = {tot[0][m] * sc[0] * row_factor(m), tot[1][m] * sc[1] * row_factor(m)};
             const pi_maps_col c0 = pi_maps_column(p.mkv, row0);
+            if (p.mkv.bias) {
+              a[0] += __ldg(p.mkv.bias + row0);
+              if (row0 + 1 < p.N) a[1] += __ldg(p.mkv.bias + row0 + 1);
+            }
             if (c0.rotated) {
               const size_t at = (size_t)place.pos * (p.mkv.rot_dims >> 1) + (c0.d >> 1);
               const float cs = p.mkv.rope_cos[at], sn = p.mkv.rope_sin[at];
@@ -486,8 +491,9 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
             for (int r = 0; r < kRows; ++r) {
               if (row0 + r >= p.N) continue;
               const pi_maps_col c = r == 0 ? c0 : pi_maps_column(p.mkv, row0 + r);
-              if (c.is_q) p.out[(size_t)(m0 + m) * p.out_stride + row0 + r] = a[r];
-              else pi_maps_kv_store(p.mkv, c, place.block, place.off, a[r]);
+              const float v = pi_maps_finish(p.mkv, c, m0 + m, row0 + r, place.pos, a[r]);
+              if (c.is_q) p.out[(size_t)(m0 + m) * p.out_stride + row0 + r] = v;
+              else pi_maps_kv_store(p.mkv, c, place.block, place.off, v);
             }
           }
         }
@@ -512,7 +518,8 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
             if (lane == r * MB + m && m < mcount && row0 + r < p.N) {
               float* o = p.out + (size_t)(m0 + m) * p.out_stride + row0 + r;
               const float v = tot[r][m] * sc[r] * row_factor(m);
-              *o = EPI == PI_EPI_ADD ? old_out + v : EPI == PI_EPI_SCALE_ADD ? fmaf(__ldg(p.out_scale + row0 + r), v, old_out) : v;
+              if (EPI == PI_EPI_GELU_TABLE) *o = pi_gelu_tanh(v) * pi_table_value(p.table, m0 + m, row0 + r);
+              else *o = EPI == PI_EPI_ADD ? old_out + v : EPI == PI_EPI_SCALE_ADD ? fmaf(__ldg(p.out_scale + row0 + r), v, old_out) : v;
             }
           }
       }
@@ -545,6 +552,8 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
       if constexpr (kFloatW) k = gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false, kSplitWarps>;
     } else if (epi == PI_EPI_SCALE_ADD) {
       if constexpr (kFloatW) k = gemv_kernel<WT, MB, PI_EPI_SCALE_ADD, false, false, kSplitWarps>;
+    } else if (epi == PI_EPI_GELU_TABLE) {
+      if constexpr (kFloatW) k = gemv_kernel<WT, MB, PI_EPI_GELU_TABLE, false, false, kSplitWarps>;
     } else k = gemv_kernel<WT, MB, PI_EPI_STORE, false, false, kSplitWarps>;
   } else if (epi == PI_EPI_STORE && p.rope_hd) {   // fused [q;k;v] projection: own instantiation, the others stay as they are
     if (norm) k = gemv_kernel<WT, MB, PI_EPI_STORE, true, true>; else k = gemv_kernel<WT, MB, PI_EPI_STORE, false, true>;
@@ -560,6 +569,8 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
     if constexpr (kFloatW) PI_PICK(PI_EPI_DYT_RESIDUAL, false);
   } else if (epi == PI_EPI_SCALE_ADD) {
     if constexpr (kFloatW) PI_PICK(PI_EPI_SCALE_ADD, false);
+  } else if (epi == PI_EPI_GELU_TABLE) {
+    if constexpr (kFloatW) PI_PICK(PI_EPI_GELU_TABLE, false);
   } else if (epi == PI_EPI_CLAMP_GLU) {
     if constexpr (kFloatW) PI_PICK(PI_EPI_CLAMP_GLU, false);
   } else {
@@ -568,7 +579,7 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
 #undef PI_PICK
   if (!k) return cudaErrorInvalidDeviceFunction;
   static pi_smem_grant granted;  // per instantiation of this launcher; attribute calls are slow
-  if (smem > std::max(granted.of(ctx), (size_t)48 * 1024)) {
+  if (smem > std::max(granted.of(ctx), kSmemFree)) {
     // the launcher covers several kernel variants: raise the limit on all of them at once
     for (auto kk : {gemv_kernel<WT, MB, PI_EPI_STORE, true, false>, gemv_kernel<WT, MB, PI_EPI_STORE, false, false>,
                     gemv_kernel<WT, MB, PI_EPI_ADD, true, false>, gemv_kernel<WT, MB, PI_EPI_ADD, false, false>,
@@ -582,7 +593,8 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
     if constexpr (kFloatW) {
       for (auto kk : {gemv_kernel<WT, MB, PI_EPI_GEGLU, false, false>, gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false>,
                       gemv_kernel<WT, MB, PI_EPI_MAPS_QKV, false, false>, gemv_kernel<WT, MB, PI_EPI_SCALE_ADD, false, false>,
-                      gemv_kernel<WT, MB, PI_EPI_CLAMP_GLU, false, false>,
+                      gemv_kernel<WT, MB, PI_EPI_CLAMP_GLU, false, false>, gemv_kernel<WT, MB, PI_EPI_GELU_TABLE, false, false>,
+                      gemv_kernel<WT, MB, PI_EPI_GELU_TABLE, false, false, kSplitWarps>,
                       gemv_kernel<WT, MB, PI_EPI_DYT_RESIDUAL, false, false, kSplitWarps>,
                       gemv_kernel<WT, MB, PI_EPI_SCALE_ADD, false, false, kSplitWarps>}) {
         cudaError_t e = cudaFuncSetAttribute(kk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -683,6 +695,7 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
   PI_REQUIRE(ctx, !a.experts || (lin->kind != PI_INT8 && a.experts->expert && lin->rows % a.experts->experts == 0 && a.experts->x_div >= 1),
              "a stack of experts needs float weights and the rows' experts");
   PI_REQUIRE(ctx, a.epi != PI_EPI_SCALE_ADD || a.out_scale, "a scaled residual add needs its scale");
+  PI_REQUIRE(ctx, a.epi != PI_EPI_GELU_TABLE || (a.table.base && a.table.tokens), "this epilogue needs its table");
   PI_REQUIRE(ctx, a.epi < PI_EPI_GEGLU || (lin->kind != PI_INT8 && !a.norm_weight), "this epilogue is built for bf16 and f32 weights");
   PI_REQUIRE(ctx, a.epi != PI_EPI_MAPS_QKV || (a.maps_kv && a.maps_kv->dim % 2 == 0), "the fused [q;k;v] epilogue needs its operands and an even dim");
   PI_REQUIRE(ctx, a.epi != PI_EPI_DYT_RESIDUAL || (a.residual && a.residual->x), "the residual epilogue needs its operands");
@@ -723,6 +736,7 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
   p.x_stride = a.x_stride;
   p.out_stride = a.out_stride;
   p.out_scale = a.out_scale;
+  p.table = a.table;
   p.glu_limit = a.glu_limit;
   p.glu_rows = a.glu_rows ? a.glu_rows : (int)n_rows;
   p.rest = a.rest;

@@ -532,7 +532,7 @@ int expanded_vp(const pi_latent_attention& a) { return (a.vdim + 15) / 16 * 16; 
 typedef void (*LatentKernel)(const LatentParams);
 cudaError_t grant(pi_ctx* ctx, LatentKernel k, size_t smem) {   // a kernel's shared-memory limit is raised once per device
   static std::vector<std::pair<LatentKernel, pi_smem_grant>> granted;
-  if (smem <= 48 * 1024) return cudaSuccess;
+  if (smem <= kSmemFree) return cudaSuccess;
   for (auto& g : granted)
     if (g.first == k) {
       if (g.second.of(ctx) >= smem) return cudaSuccess;
@@ -602,7 +602,7 @@ bool pi_latent_expandable(const pi_ctx* ctx, const pi_latent_attention& a, int c
 }
 bool pi_latent_supported(const pi_ctx* ctx, const pi_latent_attention& a, int compute) {
   const int rp = pi_latent_rp(a.rank), dp = pi_latent_dp(a.rank, a.rot_dims);
-  if (compute == PI_F32) return ((size_t)dp + 4 * a.rank) * sizeof(float) <= 48 * 1024 && (size_t)a.dim * sizeof(float) <= 48 * 1024;
+  if (compute == PI_F32) return ((size_t)dp + 4 * a.rank) * sizeof(float) <= kSmemFit && (size_t)a.dim * sizeof(float) <= kSmemFit;
   return dp <= kMaxDecodeDp && decode_smem(dp, rp).total + 4096 <= ctx->smem_optin && std::max(head_smem(a.dim), head_smem(a.rank)) + 1024 <= ctx->smem_optin;
 }
 

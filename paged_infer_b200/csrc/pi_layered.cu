@@ -1,10 +1,14 @@
 // Layered designs: a decoder whose layers each name a token mixer - windowed attention with one or two softmax maps, latent
-// attention, a gated linear recurrence (GLA), a matrix memory (mLSTM), a state-space recurrence (SSD) - and, if they have one,
-// a feed-forward: dense and gated, or routed experts.  Two ways of normalising:
+// attention, a gated linear recurrence (GLA), a matrix memory (mLSTM), a state-space recurrence (SSD), lightning attention - and,
+// if they have one, a feed-forward: dense and gated, or routed experts.  Three ways of normalising:
 //
-//   Dynamic Tanh   x += dyt(norm1b, mixer(dyt(norm1, x)));   x += dyt(norm2b, ff(dyt(norm2, x)))
-//   layer norm     x += ls1 mixer(ln(norm1, x));             x += ls2 ff(ln(norm2, x))
+//   Dynamic Tanh   x += dyt(norm1b, mixer(dyt(norm1, x)));    x += dyt(norm2b, ff(dyt(norm2, x)))
+//   layer norm     x += ls1 mixer(ln(norm1, x));              x += ls2 ff(ln(norm2, x))
+//   RMS norm       x += mu rms(norm1b, mixer(rms(norm1, x))); x += mu rms(norm2b, ff(rms(norm2, x)));
+//                  x += mu rms(side, proj(gelu(gate x) * e)), e: the layer's part of the token's row of a table
 //
+// With RMS norms the projection that ends a sublayer stores its result, and the row kernel behind it normalises that, adds it to
+// the residual stream and writes the next sublayer's input, all with the row in registers.
 // Layer norm needs the whole row: the projection that ends a sublayer adds its scaled result to the residual stream, and a
 // row kernel writes the next sublayer's input (behind experts it also adds up their outputs).
 // Dynamic Tanh needs no statistics, so all of it folds into the projection that ends a sublayer: its epilogue adds the
@@ -44,7 +48,14 @@ namespace {
 struct Layer {
   pi_layer_config c;
   pi_dyt norm1, norm1b, norm2, norm2b;
-  pi_layer_norm ln1, ln2;
+  pi_layer_norm ln1, ln2;                                  // also the RMS norms before the sublayers
+  pi_layer_norm post1, post2, post_side;                   // ... and behind them, times residual_mult
+  pi_linear *side_gate = nullptr, *side_proj = nullptr;
+  const float *bias = nullptr, *slopes = nullptr, *sinks = nullptr;   // attention: see pi_maps_attention, pi_maps_prepare
+  int col_gate = -1;                                       // column of the gate per head
+  int temp = -1;                                           // index of its table of query factors
+  float v_lambda = 0.f;
+  bool v_first = false;
   const float *ls1 = nullptr, *ls2 = nullptr;
   // routed experts: gate_up holds [shared gate/up | router | shared gate of the token], down the shared expert's
   pi_linear *in = nullptr, *out = nullptr, *gate_up = nullptr, *down = nullptr;
@@ -63,6 +74,12 @@ struct RopeTable {
   int dims = 0, cap = 0;
   double base = 1., factor = 1., original = 1., fast = 1., slow = 1.;
   float *cos = nullptr, *sin = nullptr;
+};
+
+struct TempTable {               // what queries are multiplied by, per position
+  double coef = 0., every = 1.;
+  int cap = 0;
+  float* f = nullptr;
 };
 
 // Angle per position of every pair, and the factor of cos and sin.  With a factor above 1, pairs that turn less than `slow`
@@ -87,8 +104,11 @@ struct pi_layered {
   pi_layered_config c;
   std::vector<Layer> layers;
   std::vector<RopeTable> ropes;
+  std::vector<TempTable> temps;
   std::vector<void*> owned;      // device vectors
   pi_linear *embed = nullptr, *head = nullptr;   // head: null if tied
+  pi_linear* side_embed = nullptr;
+  size_t mix_stride = 0;         // values of a row that are mixed between layers
   pi_dyt final_norm;
   pi_layer_norm final_ln;        // its weight carries the logits' scale
   size_t weight_bytes = 0, state_floats = 0;
@@ -98,6 +118,9 @@ struct pi_layered {
   // scratch for c.max_rows rows; activations are sized for f32 and hold bf16 on the tensor path
   float *x = nullptr, *proj = nullptr;
   void *h = nullptr, *core = nullptr, *ffh = nullptr;
+  float *y = nullptr, *first_v = nullptr;   // RMS norm: a sublayer's result; values of the first layer that mixes them
+  void* side_h = nullptr;
+  size_t ld_side = 0;
   size_t ld_h = 0, ld_core = 0, ld_ff = 0, ld_proj = 0;
   // latent attention, state-space recurrence, experts
   void *lat_q = nullptr, *lat_o = nullptr;
@@ -223,6 +246,14 @@ struct Loader {
     out->eps = m->c.norm_eps;
     return upload(v, &out->w);
   }
+  // Times scale (one + stored weight).
+  pi_status rms_norm(const std::string& name, pi_layer_norm* out, float one, float scale) {
+    std::vector<float> v;
+    PI_TRY(vec(name, m->c.width, &v, 1.f - one));
+    for (float& x : v) x = scale * (one + x);
+    out->eps = m->c.norm_eps;
+    return upload(v, &out->w);
+  }
   // A matrix of the checkpoint as rows dst_r0, dst_r0 + step, ... of a fused one.
   pi_status piece(const std::string& name, size_t rows, size_t cols, size_t dst_r0, size_t step, std::vector<Piece>* out) {
     Source s;
@@ -277,18 +308,23 @@ struct Loader {
 };
 
 pi_status check_layer(pi_ctx* ctx, int i, const pi_layer_config& c) {
-  PI_REQUIRE(ctx, c.mixer >= PI_MIXER_ATTENTION && c.mixer <= PI_MIXER_SSD, "layer %d: unknown mixer %d", i, c.mixer);
+  PI_REQUIRE(ctx, c.mixer >= PI_MIXER_ATTENTION && c.mixer <= PI_MIXER_LIGHTNING, "layer %d: unknown mixer %d", i, c.mixer);
   PI_REQUIRE(ctx, c.heads > 0 && c.dim > 0 && c.vdim > 0 && c.ff >= 0, "layer %d: sizes must be positive", i);
   if (c.mixer == PI_MIXER_ATTENTION) {
     PI_REQUIRE(ctx, c.kv_heads > 0 && c.heads % c.kv_heads == 0, "layer %d: %d heads do not share %d key/value heads", i, c.heads, c.kv_heads);
     PI_REQUIRE(ctx, c.maps == 1 || c.maps == 2, "layer %d: %d softmax maps", i, c.maps);
     PI_REQUIRE(ctx, c.rot_dims <= c.dim, "layer %d: %d rotary channels of %d", i, c.rot_dims, c.dim);
+    PI_REQUIRE(ctx, c.maps == 1 || !(c.distance_bias || c.sink || c.head_gate), "layer %d: distance bias, sink and head gate belong to one softmax map", i);
+    PI_REQUIRE(ctx, c.q_temp_every >= 0., "layer %d: queries grow every %g tokens", i, c.q_temp_every);
   } else if (c.mixer == PI_MIXER_LATENT) {
     PI_REQUIRE(ctx, c.rank > 0, "layer %d: the latent needs channels", i);
   } else if (c.mixer == PI_MIXER_GLA) {
     PI_REQUIRE(ctx, c.tau != 0.f, "layer %d: tau is zero", i);
   } else if (c.mixer == PI_MIXER_MLSTM) {
     PI_REQUIRE(ctx, c.gate_cap > 0.f, "layer %d: gate_cap must be positive", i);
+  } else if (c.mixer == PI_MIXER_LIGHTNING) {
+    PI_REQUIRE(ctx, c.decay, "layer %d: no decays", i);
+    for (int h = 0; h < c.heads; ++h) PI_REQUIRE(ctx, c.decay[h] >= 0. && c.decay[h] <= 1., "layer %d: a decay of %g", i, c.decay[h]);
   } else {
     PI_REQUIRE(ctx, c.groups > 0 && c.heads % c.groups == 0, "layer %d: %d heads do not form %d groups", i, c.heads, c.groups);
     PI_REQUIRE(ctx, c.norm_groups > 0 && (c.heads * c.vdim) % c.norm_groups == 0, "layer %d: %d channels do not form %d parts", i, c.heads * c.vdim, c.norm_groups);
@@ -309,6 +345,8 @@ pi_status check_layer(pi_ctx* ctx, int i, const pi_layer_config& c) {
       PI_REQUIRE(ctx, c.keep_groups >= 1 && c.keep_groups <= c.expert_groups, "layer %d: %d groups of %d are kept", i, c.keep_groups, c.expert_groups);
       PI_REQUIRE(ctx, c.top >= 1 && c.top <= c.experts / c.expert_groups * c.keep_groups, "layer %d: %d experts per token", i, c.top);
       PI_REQUIRE(ctx, c.shared_ff >= 0, "layer %d: sizes must be positive", i);
+      PI_REQUIRE(ctx, (c.unit == PI_UNIT_CLAMPED || c.unit == PI_UNIT_SILU) && (c.score == PI_SCORE_SIGMOID || c.score == PI_SCORE_SOFTMAX) &&
+                          (c.group_best == 1 || c.group_best == 2), "layer %d: unknown kind of experts", i);
     }
   }
   return PI_OK;
@@ -339,6 +377,50 @@ int add_rope(pi_layered* m, const pi_layer_config& c) {
   return (int)m->ropes.size() - 1;
 }
 
+int add_temp(pi_layered* m, const pi_layer_config& c) {
+  for (size_t i = 0; i < m->temps.size(); ++i)
+    if (m->temps[i].coef == c.q_temp_coef && m->temps[i].every == c.q_temp_every) return (int)i;
+  TempTable t;
+  t.coef = c.q_temp_coef;
+  t.every = c.q_temp_every;
+  m->temps.push_back(t);
+  return (int)m->temps.size() - 1;
+}
+
+// Attention with one map: what else a layer has beside q, k, v.
+pi_status build_attention_options(pi_ctx* ctx, Loader& ld, int i, const std::string& mix, Layer& L) {
+  pi_layered* m = ld.m;
+  const pi_layer_config& c = L.c;
+  const size_t nq = (size_t)c.heads * c.maps * c.dim, nk = (size_t)c.kv_heads * c.maps * c.dim, nv = (size_t)c.kv_heads * c.vdim;
+  if (c.biases) {
+    std::vector<float> all, part;
+    const std::pair<const char*, size_t> parts[3] = {{"q.b", nq}, {"k.b", nk}, {"v.b", nv}};
+    for (const auto& p : parts) {
+      PI_TRY(ld.vec(mix + p.first, p.second, &part));
+      all.insert(all.end(), part.begin(), part.end());
+    }
+    PI_TRY(ld.upload(all, &L.bias));
+  }
+  if (c.sink) PI_TRY(ld.dev_vec(mix + "sink", c.heads, &L.sinks));
+  if (c.distance_bias) {
+    std::vector<float> s(c.heads);
+    for (int h = 0; h < c.heads; ++h) s[h] = (float)exp2(-8.0 * (h + 1) / c.heads);
+    PI_TRY(ld.upload(s, &L.slopes));
+  }
+  if (c.q_temp_every > 0.) L.temp = add_temp(m, c);
+  if (c.v_mix) {
+    L.v_first = m->mix_stride == 0;
+    if (L.v_first) m->mix_stride = nv;
+    PI_REQUIRE(ctx, m->mix_stride == nv, "layer %d: %zu value channels do not mix with the first layer's %zu", i, nv, m->mix_stride);
+    if (!L.v_first) {
+      std::vector<float> lambda;
+      PI_TRY(ld.vec(mix + "vmix", 1, &lambda, 0.5f));
+      L.v_lambda = lambda[0];
+    }
+  }
+  return PI_OK;
+}
+
 pi_status build_mixer(pi_ctx* ctx, Loader& ld, int i, int gla_rank, Layer& L, Extents& x) {
   pi_layered* m = ld.m;
   const pi_layer_config& c = L.c;
@@ -355,6 +437,11 @@ pi_status build_mixer(pi_ctx* ctx, Loader& ld, int i, int gla_rank, Layer& L, Ex
     PI_TRY(add("q", (size_t)c.heads * c.maps * c.dim));
     PI_TRY(add("k", (size_t)c.kv_heads * c.maps * c.dim));
     PI_TRY(add("v", (size_t)c.kv_heads * c.vdim));
+    PI_TRY(build_attention_options(ctx, ld, i, mix, L));
+    if (c.head_gate) {
+      L.col_gate = (int)rows;
+      PI_TRY(add("g", c.heads));
+    }
     L.attn = x.attn++;
     if (c.maps == 2) {   // lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, one number for the layer
       double e[2];
@@ -436,6 +523,30 @@ pi_status build_mixer(pi_ctx* ctx, Loader& ld, int i, int gla_rank, Layer& L, Ex
     m->state_floats += r.state_floats();
     x.inner = std::max(x.inner, core);
     x.chunk = x.chunk && pi_ssd_chunked(ctx, r, m->c.compute);
+  } else if (c.mixer == PI_MIXER_LIGHTNING) {
+    pi_ssd& r = L.ssd;               // keys are B, queries C, a group per head
+    r.heads = r.groups = c.heads;
+    r.vdim = c.vdim;
+    r.dim = c.dim;
+    r.eps = m->c.norm_eps;
+    r.gate_last = true;
+    r.col_x = (int)core;
+    PI_TRY(add("g", core));
+    PI_TRY(add("v", core));
+    PI_TRY(add("k", (size_t)c.heads * c.dim));
+    PI_TRY(add("q", (size_t)c.heads * c.dim));
+    std::vector<float> decay(c.heads), log_decay(c.heads);
+    for (int h = 0; h < c.heads; ++h) {
+      decay[h] = (float)c.decay[h];
+      log_decay[h] = (float)std::max(log(c.decay[h]), -1e4);   // a decay of 0 is one that leaves nothing
+    }
+    PI_TRY(ld.upload(decay, &r.decay));
+    PI_TRY(ld.upload(log_decay, &r.log_decay));
+    PI_TRY(ld.dev_vec(mix + "norm", core, &r.norm, 1.f));
+    r.state_off = m->state_floats;
+    m->state_floats += r.state_floats();
+    x.inner = std::max(x.inner, core);
+    x.chunk = x.chunk && pi_ssd_chunked(ctx, r, m->c.compute);
   } else {
     pi_recurrence& r = L.rec;
     const size_t hd = (size_t)c.heads * c.dim;
@@ -512,12 +623,16 @@ pi_status build_feed_forward(Loader& ld, int i, Layer& L, Extents& x) {
   e.top = c.top;
   e.groups = c.expert_groups;
   e.keep = c.keep_groups;
+  e.score = c.score;
+  e.group_best = c.group_best;
+  e.renorm = c.renorm;
+  e.scale = c.route_scale;
   PI_TRY(ld.dev_vec(mlp + "correction", c.experts, &e.correction));
   size_t rows = 2 * (size_t)c.shared_ff;
   if (c.shared_ff) PI_TRY(gated(mlp + "shared.", c.shared_ff, 0));
   PI_TRY(ld.piece(mlp + "router", c.experts, W, rows, 1, &p));
   rows += c.experts;
-  if (c.shared_ff) {
+  if (c.shared_ff && c.shared_gate) {
     PI_TRY(ld.piece(mlp + "shared.sg", 1, W, rows, 1, &p));
     ++rows;
   }
@@ -546,9 +661,9 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
   m->c = *cfg;
   m->c.layers = nullptr;
   const size_t W = cfg->width;
-  const bool dyt = cfg->norm == PI_NORM_DYT;
+  const bool dyt = cfg->norm == PI_NORM_DYT, rms = cfg->norm == PI_NORM_RMS;
   size_t tensors = 8;
-  for (int i = 0; i < cfg->num_layers; ++i) tensors += 32 + 3 * (size_t)std::max(0, cfg->layers[i].experts);
+  for (int i = 0; i < cfg->num_layers; ++i) tensors += 40 + 3 * (size_t)std::max(0, cfg->layers[i].experts);
   ld.keep.reserve(tensors);   // Source::host points into it
   Extents x;
   {
@@ -561,7 +676,14 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
       PI_TRY(ld.matrix(p, cfg->vocab_size, W, &m->head));
     }
   }
+  if (cfg->side_dim > 0) {
+    std::vector<Piece> p;
+    const size_t cols = (size_t)cfg->side_dim * cfg->num_layers;
+    PI_TRY(ld.piece("side.embed", cfg->vocab_size, cols, 0, 1, &p));
+    PI_TRY(ld.matrix(p, cfg->vocab_size, cols, &m->side_embed));
+  }
   if (dyt) PI_TRY(ld.dyt("final.norm", &m->final_norm));
+  else if (rms) PI_TRY(ld.rms_norm("final.norm", &m->final_ln, 1.f, cfg->logit_scale));
   else PI_TRY(ld.layer_norm("final.norm", &m->final_ln, cfg->logit_scale));
   m->layers.resize(cfg->num_layers);
   for (int i = 0; i < cfg->num_layers; ++i) {
@@ -570,7 +692,12 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
     PI_TRY(check_layer(ctx, i, L.c));
     PI_REQUIRE(ctx, !dyt || L.c.ff == 0 || L.c.ff_kind == PI_FF_GELU, "layer %d: this feed-forward is not built behind Dynamic Tanh", i);
     const std::string l = "l" + std::to_string(i);
-    auto norm = [&](const char* name, pi_dyt* before, pi_dyt* after, pi_layer_norm* ln, const char* scale_name, const float** scale) -> pi_status {
+    auto norm = [&](const char* name, pi_dyt* before, pi_dyt* after, pi_layer_norm* ln, pi_layer_norm* post, const char* scale_name,
+                    const float** scale) -> pi_status {
+      if (rms) {
+        PI_TRY(ld.rms_norm(l + name, ln, 1.f, 1.f));
+        return ld.rms_norm(l + name + "b", post, 1.f, cfg->residual_mult);
+      }
       if (dyt) {
         PI_TRY(ld.dyt(l + name, before));
         return ld.dyt(l + name + "b", after);
@@ -578,12 +705,22 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
       PI_TRY(ld.layer_norm(l + name, ln));
       return ld.dev_vec(l + scale_name, W, scale, 0.5f);
     };
-    PI_TRY(norm(".norm1", &L.norm1, &L.norm1b, &L.ln1, ".ls1", &L.ls1));
+    PI_TRY(norm(".norm1", &L.norm1, &L.norm1b, &L.ln1, &L.post1, ".ls1", &L.ls1));
     PI_TRY(build_mixer(ctx, ld, i, gla_rank, L, x));
     if (L.c.ff > 0) {
-      PI_TRY(norm(".norm2", &L.norm2, &L.norm2b, &L.ln2, ".ls2", &L.ls2));
+      PI_TRY(norm(".norm2", &L.norm2, &L.norm2b, &L.ln2, &L.post2, ".ls2", &L.ls2));
       PI_TRY(build_feed_forward(ld, i, L, x));
     }
+    if (m->side_embed) {
+      std::vector<Piece> p;
+      PI_TRY(ld.piece(l + ".side.gate", cfg->side_dim, W, 0, 1, &p));
+      PI_TRY(ld.matrix(p, cfg->side_dim, W, &L.side_gate));
+      p.clear();
+      PI_TRY(ld.piece(l + ".side.proj", W, cfg->side_dim, 0, 1, &p));
+      PI_TRY(ld.matrix(p, W, cfg->side_dim, &L.side_proj));
+      PI_TRY(ld.rms_norm(l + ".side.norm", &L.post_side, 0.f, cfg->residual_mult));
+    }
+    L.c.decay = nullptr;             // the caller's
   }
   m->chunked = x.chunk && m->state_floats > 0;
   const size_t cap = cfg->max_rows;
@@ -603,6 +740,10 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
   PI_TRY(alloc(&m->h, cap * m->ld_h));
   PI_TRY(alloc(&m->core, cap * m->ld_core));
   PI_TRY(alloc(&m->ffh, cap * m->ld_ff));
+  if (rms) PI_TRY(alloc(&m->y, cap * W));
+  PI_TRY(alloc(&m->first_v, cap * m->mix_stride));
+  m->ld_side = round8(cfg->side_dim);
+  PI_TRY(alloc(&m->side_h, cap * m->ld_side));
   const bool f32 = cfg->compute == PI_F32;
   PI_TRY(alloc(&m->lat_q, cap * x.lat_q / (f32 ? 1 : 2)));
   PI_TRY(alloc(&m->lat_o, (cap * x.lat_o + 1) / (f32 ? 1 : 2)));
@@ -631,7 +772,21 @@ pi_moe_lists moe_lists(const pi_layered* m) {
   return l;
 }
 
-pi_status ensure_ropes(pi_ctx* ctx, pi_layered* m, int positions) {
+// Tables per position, grown to cover `positions`.
+pi_status ensure_tables(pi_ctx* ctx, pi_layered* m, int positions) {
+  for (TempTable& t : m->temps) {
+    if (positions <= t.cap) continue;
+    const int cap = std::max(positions, std::max(2 * t.cap, 2048));
+    std::vector<float> f(cap);
+    for (int p = 0; p < cap; ++p) f[p] = (float)(1.0 + t.coef * log(floor((p + 1) / t.every) + 1.0));
+    PI_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    cudaFree(t.f);
+    t.f = nullptr;
+    t.cap = 0;
+    PI_CUDA(ctx, cudaMalloc(&t.f, f.size() * sizeof(float)));
+    PI_CUDA(ctx, cudaMemcpy(t.f, f.data(), f.size() * sizeof(float), cudaMemcpyHostToDevice));
+    t.cap = cap;
+  }
   for (RopeTable& t : m->ropes) {
     if (t.dims == 0 || positions <= t.cap) continue;
     const int cap = std::max(positions, std::max(2 * t.cap, 2048)), half = t.dims / 2;
@@ -768,7 +923,7 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
     PI_REQUIRE(ctx, in->out_rows[i] >= 0 && in->out_rows[i] < rows, "output row %d of %d", in->out_rows[i], rows);
     if (in->out_rows[i] != i) st->all_rows = false;
   }
-  PI_TRY(ensure_ropes(ctx, m, max_pos + 1 + extra_positions));
+  PI_TRY(ensure_tables(ctx, m, max_pos + 1 + extra_positions));
 
   size_t words = 0;
   std::vector<std::pair<const void*, size_t>> parts;
@@ -841,7 +996,7 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
   // scratch is sized here, so that nothing allocates while a step is being captured
   size_t floats = 0, keys = 0, elems = 0;
   for (const Layer& L : m->layers) {
-    if (L.c.mixer == PI_MIXER_SSD) floats = std::max(floats, pi_ssd_scratch_floats(L.ssd, b.n_chunks));
+    if (L.c.mixer == PI_MIXER_SSD || L.c.mixer == PI_MIXER_LIGHTNING) floats = std::max(floats, pi_ssd_scratch_floats(L.ssd, b.n_chunks));
     else if (L.attn < 0) floats = std::max(floats, pi_recurrence_scratch_floats(L.rec, b.n_chunks));
     else if (L.c.mixer == PI_MIXER_LATENT) {
       keys = std::max(keys, (size_t)b.n_keys * pi_latent_rp(L.c.rank));
@@ -910,8 +1065,24 @@ pi_status run_mixer(pi_ctx* ctx, pi_layered* m, const Layer& L, pi_kv_pool* pool
     a.rot_dims = c.rot_dims;
     a.rope_cos = m->ropes[L.rope].cos;
     a.rope_sin = m->ropes[L.rope].sin;
+    a.slopes = L.slopes;
+    a.sinks = L.sinks;
+    if (c.head_gate) {
+      a.gate = m->proj + L.col_gate;
+      a.gate_stride = m->ld_proj;
+      a.gate_per_head = true;
+    }
+    pi_maps_prepare prep;
+    prep.bias = L.bias;
+    prep.unit_qk = c.unit_qk != 0;
+    prep.q_temp = L.temp >= 0 ? m->temps[L.temp].f : nullptr;
+    if (c.v_mix) prep.mix = pi_value_mix{m->first_v, m->mix_stride, L.v_lambda, L.v_first};
     pi_maps_kv mk;
-    if (c.dim % 2 == 0) {   // rotary positions and the KV write fold into the projection
+    // biases, rotary positions, temperature, value mixing and the KV write fold into the projection; what needs a whole head does not
+    if (c.dim % 2 == 0 && !c.unit_qk && !c.head_gate) {
+      mk.bias = prep.bias;
+      mk.q_temp = prep.q_temp;
+      mk.mix = prep.mix;
       mk.q_rows = c.heads * c.maps * c.dim;
       mk.k_rows = c.kv_heads * c.maps * c.dim;
       mk.maps = c.maps;
@@ -935,7 +1106,7 @@ pi_status run_mixer(pi_ctx* ctx, pi_layered* m, const Layer& L, pi_kv_pool* pool
       in.maps_kv = &mk;
     }
     PI_TRY(project(ctx, L.in, m->h, m->ld_h, M, bf16, in));
-    if (in.epi != PI_EPI_MAPS_QKV) PI_TRY(pi_launch_maps_rope_kv(ctx, a, kv, m->proj, m->ld_proj, b));
+    if (in.epi != PI_EPI_MAPS_QKV) PI_TRY(pi_launch_maps_prepare(ctx, a, prep, kv, m->proj, m->ld_proj, b));
     return pi_launch_maps_attention(ctx, a, kv, m->proj, m->ld_proj, m->core, m->ld_core, kind, b);
   }
   PI_TRY(project(ctx, L.in, m->h, m->ld_h, M, bf16, in));
@@ -950,7 +1121,7 @@ pi_status run_mixer(pi_ctx* ctx, pi_layered* m, const Layer& L, pi_kv_pool* pool
     s.pool = static_cast<__nv_bfloat16*>(m->exp_pool.ptr);
     return pi_launch_latent_attention(ctx, a, kv_view(pool, L.attn), m->proj, m->ld_proj, m->core, m->ld_core, kind, b, s);
   }
-  if (c.mixer == PI_MIXER_SSD) {
+  if (c.mixer == PI_MIXER_SSD || c.mixer == PI_MIXER_LIGHTNING) {
     pi_ssd r = L.ssd;
     r.state = state->data;
     r.state_stride = state->stride;
@@ -967,10 +1138,11 @@ pi_status run_experts(pi_ctx* ctx, pi_layered* m, const Layer& L, int M, bool bf
   const pi_layer_config& c = L.c;
   const pi_moe_lists lists = moe_lists(m);
   const int pairs = M * c.top;
+  const pi_epilogue unit = c.unit == PI_UNIT_SILU ? PI_EPI_SWIGLU : PI_EPI_CLAMP_GLU;
   // the shared expert's first projection carries the router's rows
   pi_linear_args a;
   if (c.shared_ff) {
-    a.epi = PI_EPI_CLAMP_GLU;
+    a.epi = unit;
     a.glu_limit = c.shared_limit;
     a.glu_rows = 2 * c.shared_ff;
     a.out = static_cast<float*>(m->ffh);
@@ -1000,7 +1172,7 @@ pi_status run_experts(pi_ctx* ctx, pi_layered* m, const Layer& L, int M, bool bf
   }
   pi_linear_args e;
   e.experts = &rows;
-  e.epi = PI_EPI_CLAMP_GLU;
+  e.epi = unit;
   e.glu_limit = c.limit;
   e.out = static_cast<float*>(m->moe_act);
   e.out_bf16 = static_cast<__nv_bfloat16*>(m->moe_act);
@@ -1027,19 +1199,79 @@ pi_status run_experts(pi_ctx* ctx, pi_layered* m, const Layer& L, int M, bool bf
     PI_TRY(project(ctx, L.down, m->ffh, m->ld_ff, M, bf16, s));
     sum->shared = m->shared;
     sum->shared_stride = m->c.width;
-    sum->shared_gate = m->route + c.experts;
-    sum->shared_gate_stride = m->ld_route;
+    if (c.shared_gate) {
+      sum->shared_gate = m->route + c.experts;
+      sum->shared_gate_stride = m->ld_route;
+    }
   }
   return PI_OK;
+}
+
+// The layer's gated feed-forward, from h through the projection `down` describes.
+pi_status run_dense(pi_ctx* ctx, pi_layered* m, const Layer& L, int M, bool bf16, const pi_linear_args& down) {
+  pi_linear_args g;
+  g.epi = L.c.ff_kind == PI_FF_SILU ? PI_EPI_SWIGLU : PI_EPI_GEGLU;
+  g.out = static_cast<float*>(m->ffh);
+  g.out_bf16 = static_cast<__nv_bfloat16*>(m->ffh);
+  g.out_stride = m->ld_ff;
+  PI_TRY(project(ctx, L.gate_up, m->h, m->ld_h, M, bf16, g));
+  return project(ctx, L.down, m->ffh, m->ld_ff, M, bf16, down);
+}
+
+// Layer i with RMS norms, from h behind its mixer to `after`: the input of the next layer (or null for the last one's x alone).
+pi_status run_sandwich(pi_ctx* ctx, pi_layered* m, const Layer& L, int i, const Staged& st, bool bf16, const pi_row_norm& row, const pi_row_norm& after) {
+  const int M = st.b.rows;
+  const pi_layer_config& c = L.c;
+  const bool side = L.side_gate != nullptr;
+  pi_linear_args a;
+  a.out = m->y;
+  a.out_stride = m->c.width;
+  PI_TRY(project(ctx, L.out, m->core, m->ld_core, M, bf16, a));
+  pi_row_norm n = c.ff > 0 || side ? row : after;
+  n.y = m->y;
+  n.y_stride = m->c.width;
+  n.post = L.post1;
+  if (c.ff > 0) n.norm = L.ln2;           // without: the side reads x as it stands
+  PI_TRY(pi_launch_row_norm(ctx, n));
+  if (c.ff > 0) {
+    n = side ? row : after;
+    n.post = L.post2;
+    pi_expert_sum sum;
+    if (c.ff_kind == PI_FF_EXPERTS) {
+      PI_TRY(run_experts(ctx, m, L, M, bf16, &sum));
+      n.experts = &sum;
+    } else {
+      PI_TRY(run_dense(ctx, m, L, M, bf16, a));
+      n.y = m->y;
+      n.y_stride = m->c.width;
+    }
+    PI_TRY(pi_launch_row_norm(ctx, n));
+  }
+  if (!side) return PI_OK;
+  pi_linear_args g;
+  g.epi = PI_EPI_GELU_TABLE;
+  g.out = static_cast<float*>(m->side_h);
+  g.out_bf16 = static_cast<__nv_bfloat16*>(m->side_h);
+  g.out_stride = m->ld_side;
+  g.table = pi_token_table{static_cast<const uint16_t*>(m->side_embed->w) + (size_t)i * m->c.side_dim, m->side_embed->ld, m->c.vocab_size, st.b.tokens};
+  PI_TRY(project(ctx, L.side_gate, m->h, m->ld_h, M, bf16, g));
+  PI_TRY(project(ctx, L.side_proj, m->side_h, m->ld_side, M, bf16, a));
+  n = after;
+  n.y = m->y;
+  n.y_stride = m->c.width;
+  n.post = L.post_side;
+  return pi_launch_row_norm(ctx, n);
 }
 
 pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool* state, const Staged& st) {
   const pi_seq_batch& b = st.b;
   const int M = b.rows, W = m->c.width, NL = (int)m->layers.size();
-  const bool bf16 = act_bf16(ctx, m, M), dyt = m->c.norm == PI_NORM_DYT;
+  const bool bf16 = act_bf16(ctx, m, M), dyt = m->c.norm == PI_NORM_DYT, rms = m->c.norm == PI_NORM_RMS;
   const int kind = bf16 ? PI_BF16 : PI_F32;
   const bool head_bf16 = st.n_out && act_bf16(ctx, m, st.n_out);
-  pi_row_norm row;               // layer norm: from x to h
+  pi_row_norm row;               // layer or RMS norm: from x to h
+  row.rms = rms;
+  row.embed_scale = m->c.embed_scale;
   row.rows = M;
   row.width = W;
   row.x = m->x;
@@ -1080,16 +1312,23 @@ pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool
       a.residual = &res;
       PI_TRY(project(ctx, L.out, m->core, m->ld_core, M, bf16, a));
       if (c.ff > 0) {
-        pi_linear_args g;
-        g.epi = PI_EPI_GEGLU;
-        g.out = static_cast<float*>(m->ffh);
-        g.out_bf16 = static_cast<__nv_bfloat16*>(m->ffh);
-        g.out_stride = m->ld_ff;
-        PI_TRY(project(ctx, L.gate_up, m->h, m->ld_h, M, bf16, g));
         res.post = L.norm2b;
         res.next = after;
-        PI_TRY(project(ctx, L.down, m->ffh, m->ld_ff, M, bf16, a));
+        PI_TRY(run_dense(ctx, m, L, M, bf16, a));
       }
+    } else if (rms) {
+      pi_row_norm after = row;
+      if (!last) {
+        after.norm = m->layers[i + 1].ln1;
+      } else if (st.all_rows) {
+        after.norm = m->final_ln;
+        after.h = m->head_in.ptr;
+        after.h_kind = head_bf16 ? PI_BF16 : PI_F32;
+        final_done = true;
+      } else {
+        after.h = nullptr;
+      }
+      PI_TRY(run_sandwich(ctx, m, L, i, st, bf16, row, after));
     } else {
       pi_linear_args a;
       a.epi = PI_EPI_SCALE_ADD;
@@ -1116,14 +1355,8 @@ pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool
           final_done = true;
         }
       } else if (c.ff > 0) {
-        pi_linear_args g;
-        g.epi = c.ff_kind == PI_FF_SILU ? PI_EPI_SWIGLU : PI_EPI_GEGLU;
-        g.out = static_cast<float*>(m->ffh);
-        g.out_bf16 = static_cast<__nv_bfloat16*>(m->ffh);
-        g.out_stride = m->ld_ff;
-        PI_TRY(project(ctx, L.gate_up, m->h, m->ld_h, M, bf16, g));
         a.out_scale = L.ls2;
-        PI_TRY(project(ctx, L.down, m->ffh, m->ld_ff, M, bf16, a));
+        PI_TRY(run_dense(ctx, m, L, M, bf16, a));
       }
       if (next.h || next.experts) PI_TRY(pi_launch_row_norm(ctx, next));
     }
@@ -1175,8 +1408,11 @@ pi_status pi_layered_create(pi_ctx* ctx, const pi_layered_config* cfg, const pi_
   PI_REQUIRE(ctx, ctx->tp == 1, "layered designs run on one GPU");
   PI_REQUIRE(ctx, cfg->width > 0 && cfg->vocab_size > 0 && cfg->num_layers > 0 && cfg->layers && cfg->max_rows > 0, "model config fields must be positive");
   PI_REQUIRE(ctx, cfg->compute == PI_BF16 || cfg->compute == PI_F32, "layered designs compute in bf16 or f32");
-  PI_REQUIRE(ctx, cfg->norm == PI_NORM_DYT || cfg->norm == PI_NORM_LAYER, "unknown normalisation %d", cfg->norm);
-  PI_REQUIRE(ctx, cfg->norm == PI_NORM_LAYER || cfg->logit_scale == 1.f, "logits are scaled behind layer norm only");
+  PI_REQUIRE(ctx, cfg->norm >= PI_NORM_DYT && cfg->norm <= PI_NORM_RMS, "unknown normalisation %d", cfg->norm);
+  PI_REQUIRE(ctx, cfg->norm != PI_NORM_DYT || cfg->logit_scale == 1.f, "logits are not scaled behind Dynamic Tanh");
+  PI_REQUIRE(ctx, cfg->side_dim >= 0, "sizes must be positive");
+  PI_REQUIRE(ctx, cfg->norm == PI_NORM_RMS || (cfg->embed_scale == 1.f && cfg->residual_mult == 1.f && cfg->side_dim == 0),
+             "a scale of the embedding, a factor of the residual update and a table of tokens belong to RMS norms");
   PI_REQUIRE(ctx, tensors || gla_rank > 0, "synthetic weights need a rank for the decay's low-rank input");
   pi_layered* m = new (std::nothrow) pi_layered();
   if (!m) return pi_fail(ctx, PI_ERR_OOM, "host allocation failed");
@@ -1200,9 +1436,11 @@ void pi_layered_destroy(pi_layered* m) {
   if (!m) return;
   if (m->step_exec) cudaGraphExecDestroy(m->step_exec);
   for (Layer& L : m->layers)
-    for (pi_linear* l : {L.in, L.out, L.gate_up, L.down, L.expert_in, L.expert_out, L.ukv, L.uk_t}) pi_linear_destroy(l);
+    for (pi_linear* l : {L.in, L.out, L.gate_up, L.down, L.expert_in, L.expert_out, L.ukv, L.uk_t, L.side_gate, L.side_proj}) pi_linear_destroy(l);
   pi_linear_destroy(m->embed);
   pi_linear_destroy(m->head);
+  pi_linear_destroy(m->side_embed);
+  for (TempTable& t : m->temps) cudaFree(t.f);
   for (RopeTable& t : m->ropes) {
     cudaFree(t.cos);
     cudaFree(t.sin);
@@ -1210,7 +1448,7 @@ void pi_layered_destroy(pi_layered* m) {
   for (void* p : m->owned) cudaFree(p);
   for (void* p : {(void*)m->x, (void*)m->proj, m->h, m->core, m->ffh, m->lat_q, m->lat_o, (void*)m->ssd_y, (void*)m->route, (void*)m->shared, m->moe_h, m->moe_act,
                   m->moe_y, m->moe_ints, m->exp_keys.ptr, m->exp_pool.ptr, m->meta.ptr, m->head_in.ptr, m->logits.ptr, m->ids.ptr, m->scratch.ptr,
-                  m->trace.ptr, m->history.ptr})
+                  m->trace.ptr, (void*)m->y, (void*)m->first_v, m->side_h, m->history.ptr})
     if (p) cudaFree(p);
   delete m;
 }

@@ -1,6 +1,6 @@
 // Internal declarations of layered designs: models whose layers each name a token mixer (windowed multi-map attention,
-// latent attention, a gated linear recurrence, a matrix memory, a state-space recurrence) and a feed-forward (dense or
-// experts) with sizes of their own.
+// latent attention, a gated linear recurrence, a matrix memory, a state-space recurrence, lightning attention) and a
+// feed-forward (dense or experts) with sizes of their own.
 #pragma once
 
 #include "pi_common.cuh"
@@ -63,8 +63,11 @@ struct pi_maps_attention {
   int window = 0;                       // <= 0: everything before
   float scale = 1.f, eps = 0.f;
   float lambda = 0.f, out_scale = 1.f;  // maps == 2
-  const float* gate = nullptr;          // the result is multiplied by sigmoid(gate[row][heads * vdim])
+  const float* gate = nullptr;          // the result is multiplied by sigmoid(gate[row][heads * vdim]), or [row][heads]
   size_t gate_stride = 0;
+  bool gate_per_head = false;
+  const float* slopes = nullptr;        // [heads] taken off a score per token of distance
+  const float* sinks = nullptr;         // [heads] exp(sink) joins the sum of weights, once, without a value
   bool v_in_k = false;                  // the values are the first channels of the keys (f32 kernel)
   int rot_dims = 0;
   const float* rope_cos = nullptr;      // [positions][rot_dims / 2]
@@ -74,8 +77,16 @@ struct pi_kv_view {                     // one layer's region of the pool
   void* base = nullptr;
   int kind = PI_F32, kv_heads = 0, maps = 0, dp = 0, vp = 0, block_size = 0;
 };
-// Rotate q (in place) and k, and write k and v of every row into the pool.  qkv rows: [q: heads*maps*dim | k | v].
-pi_status pi_launch_maps_rope_kv(pi_ctx* ctx, const pi_maps_attention& a, const pi_kv_view& kv, float* qkv, size_t stride,
+// What happens to q, k and v between projection and attention beside the rotation (all optional).
+struct pi_maps_prepare {
+  const float* bias = nullptr;          // [q | k | v]
+  bool unit_qk = false;                 // q and k over their root mean square, per head and map (eps of the attention)
+  const float* q_temp = nullptr;        // [positions] factor of q
+  pi_value_mix mix;
+};
+// Bring q (in place), k and v of every row into their final form and write k and v into the pool.  qkv rows: [q: heads*maps*dim |
+// k | v].
+pi_status pi_launch_maps_prepare(pi_ctx* ctx, const pi_maps_attention& a, const pi_maps_prepare& x, const pi_kv_view& kv, float* qkv, size_t stride,
                                  const pi_seq_batch& b);
 // out[row][heads * vdim] as f32 or bf16 (out_kind).
 pi_status pi_launch_maps_attention(pi_ctx* ctx, const pi_maps_attention& a, const pi_kv_view& kv, const float* qkv, size_t stride,
@@ -112,9 +123,12 @@ pi_status pi_launch_latent_attention(pi_ctx* ctx, const pi_latent_attention& a, 
 struct pi_ssd {
   int heads = 0, vdim = 0, dim = 0, groups = 1, norm_groups = 1, taps = 1;   // dim: state channels
   float eps = 0.f;
-  const float *conv = nullptr, *conv_b = nullptr;   // [channels][taps], [channels]; channels: x, B, C
+  const float *conv = nullptr, *conv_b = nullptr;   // [channels][taps], [channels]; channels: x, B, C.  Null: no convolution (taps 1)
   const float4* conv4 = nullptr;        // up to four taps: the same, with zeros in front
   const float *dt_bias = nullptr, *a_log = nullptr, *d = nullptr;   // [heads]
+  // a constant decay per head instead: dt = 1, no dt column, dt_bias, a_log and d are null
+  const float *decay = nullptr, *log_decay = nullptr;   // [heads]
+  bool gate_last = false;               // out = norm(y) sigmoid(z) instead of norm(y silu(z))
   const float* norm = nullptr;          // [heads * vdim]
   int col_z = 0, col_x = 0, col_dt = 0; // columns of the fused projection: z | x, B, C | dt
   // state: per slot S [heads][dim][vdim], then the convolution's last inputs [taps - 1][channels]
@@ -134,6 +148,8 @@ pi_status pi_launch_ssd_chunks(pi_ctx* ctx, const pi_ssd& r, const float* proj, 
 // ---- experts (pi_moe.cu; the products are pi_linear with pi_expert_rows) ---------------------------------------------------
 struct pi_moe {
   int experts = 0, top = 0, groups = 1, keep = 1;
+  int score = PI_SCORE_SIGMOID, group_best = 2, renorm = 1;
+  float scale = 1.f;                    // of the weights
   const float* correction = nullptr;    // [experts], part of the choice and not of the weights
 };
 struct pi_moe_lists {
@@ -148,12 +164,12 @@ int pi_moe_max_tiles(int rows, const pi_moe& m);
 pi_status pi_launch_moe_route(pi_ctx* ctx, const pi_moe& m, const float* logits, size_t stride, int rows, const pi_moe_lists& l);
 pi_status pi_launch_moe_gather(pi_ctx* ctx, const pi_moe& m, int rows, const pi_moe_lists& l, const __nv_bfloat16* h, size_t ld_h, __nv_bfloat16* out);
 
-// ---- rows: residual stream and layer norm (pi_rows.cu) -------------------------------------------------------------------
+// ---- rows: residual stream and norms (pi_rows.cu) -------------------------------------------------------------------
 struct pi_layer_norm {
   const float* w = nullptr;
   float eps = 0.f;
 };
-// scale (sum over k of weights[row][k] y[place[row][k]] + sigmoid(shared_gate[row]) shared[row])
+// scale (sum over k of weights[row][k] y[place[row][k]] + sigmoid(shared_gate[row]) shared[row]); null: no gate, no scale
 struct pi_expert_sum {
   int top = 0;
   const float* weights = nullptr;
@@ -166,6 +182,12 @@ struct pi_expert_sum {
   const float* scale = nullptr;         // [width]
 };
 struct pi_row_norm {
+  bool rms = false;                     // RMS norms (weights as they multiply) instead of layer norm; then also:
+  const float* y = nullptr;             //   x += post(y) first; post applies to the experts' sum too
+  size_t y_stride = 0;
+  pi_layer_norm post;
+  float embed_scale = 1.f;              //   x = embed_scale table[token]
+                                        //   norm.w null: h is x as it stands
   int rows = 0, width = 0;
   float* x = nullptr;                   // [.][width]
   const int32_t* pick = nullptr;        // row i is x[pick[i]]

@@ -1,8 +1,9 @@
 // Routing of tokens to experts.
 //
-// moe_route_kernel: a warp per token.  Scores s = sigmoid(logit), choice scores s + correction; the experts form equal groups
-// of neighbours, a group's score is the sum of its two best choice scores, and only the experts of the best groups can be
-// chosen; among them the best choice scores win, ties to the lower index.  Weights: the chosen scores s over their sum.
+// moe_route_kernel: a warp per token.  Scores s = sigmoid(logit), or the softmax of all logits; choice scores s + correction; the
+// experts form equal groups of neighbours, a group's score is its best choice score or the sum of its two best, and only the
+// experts of the best groups can be chosen; among them the best choice scores win, ties to the lower index.  Weights: the
+// chosen scores s, over their sum if they are brought to sum 1, times a constant.
 // moe_lists_kernel: one CTA sorts the (token, choice) pairs by expert - a histogram, its prefix sum, a place for every pair -
 // and cuts the experts' rows into column tiles for the grouped GEMM.  (The order of the pairs inside an expert does not
 // matter: every row is computed alike wherever it lies.)
@@ -20,7 +21,8 @@ struct RouteParams {
   const float* logits;
   size_t stride;
   const float* correction;
-  int rows, experts, groups, keep, top;
+  int rows, experts, groups, keep, top, softmax, group_best, renorm;
+  float scale;
   int32_t* ids;
   float* weights;
 };
@@ -44,8 +46,15 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const Route
   pi_grid_dependency_wait();
   if (row >= p.rows) return;
   const float* z = p.logits + (size_t)row * p.stride;
+  float top_z = -INFINITY, z_sum = 0.f;
+  if (p.softmax) {
+    for (int e = lane; e < p.experts; e += 32) top_z = fmaxf(top_z, z[e]);
+    top_z = pi_warp_max(top_z);
+    for (int e = lane; e < p.experts; e += 32) z_sum += expf(z[e] - top_z);
+    z_sum = pi_warp_sum(z_sum);
+  }
   for (int e = lane; e < p.experts; e += 32) {
-    const float s = pi_sigmoid(z[e]);
+    const float s = p.softmax ? expf(z[e] - top_z) / z_sum : pi_sigmoid(z[e]);
     score[e] = s;
     choice[e] = s + (p.correction ? __ldg(p.correction + e) : 0.f);
   }
@@ -63,7 +72,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const Route
           b = c;
         }
       }
-      group[g] = n > 1 ? a + b : a;
+      group[g] = n > 1 && p.group_best > 1 ? a + b : a;
     }
     __syncwarp();
     for (int k = 0; k < p.keep; ++k) {                 // a kept group is marked by NaN
@@ -95,7 +104,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const Route
   for (int j = 0; j < 2; ++j)
     if (lane + 32 * j < p.top) {
       p.ids[(size_t)row * p.top + lane + 32 * j] = mine[j];
-      p.weights[(size_t)row * p.top + lane + 32 * j] = score[mine[j]] / (sum + 1e-20f);
+      p.weights[(size_t)row * p.top + lane + 32 * j] = p.scale * (p.renorm ? score[mine[j]] / (sum + 1e-20f) : score[mine[j]]);
     }
 }
 
@@ -166,9 +175,10 @@ int pi_moe_max_tiles(int rows, const pi_moe& m) {
 
 pi_status pi_launch_moe_route(pi_ctx* ctx, const pi_moe& m, const float* logits, size_t stride, int rows, const pi_moe_lists& l) {
   pi_prof_scope prof(ctx, PI_PROF_OTHER);
-  const RouteParams p = {logits, stride, m.correction, rows, m.experts, m.groups, m.keep, m.top, l.ids, l.weights};
+  const RouteParams p = {logits, stride, m.correction, rows, m.experts, m.groups, m.keep, m.top, m.score == PI_SCORE_SOFTMAX, m.group_best,
+                         m.renorm, m.scale, l.ids, l.weights};
   const size_t smem = (size_t)kRouteWarps * (2 * m.experts + m.groups) * sizeof(float);
-  PI_REQUIRE(ctx, smem <= 48 * 1024 && m.top <= 64, "%d of %d experts are too many", m.top, m.experts);
+  PI_REQUIRE(ctx, smem <= kSmemFit && m.top <= 64, "%d of %d experts are too many", m.top, m.experts);
   PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, moe_route_kernel, dim3((rows + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32), smem, 1, p));
   return PI_OK;
 }

@@ -644,7 +644,7 @@ size_t output_smem(const ChunkParams& p) {
 }
 
 cudaError_t grant(pi_ctx* ctx, void (*k)(const ChunkParams), size_t smem, pi_smem_grant& g) {
-  if (smem <= g.of(ctx) || smem <= 48 * 1024) return cudaSuccess;
+  if (smem <= g.of(ctx) || smem <= kSmemFree) return cudaSuccess;
   g.of(ctx) = smem;
   return cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
 }

@@ -1,11 +1,14 @@
-// State-space recurrence with a scalar decay per head (Mamba-2), f32 throughout:
+// Recurrences with a scalar decay per head, f32 throughout.  State space (Mamba-2):
 //
 //   u_t = silu(b + sum_j w_j (x, B, C)_(t - taps + 1 + j))       per channel, zeros before the start
 //   dt  = softplus(dt_t + bias),  a = exp(-exp(A_log) dt)         per head
 //   S_t = a S_(t-1) + dt B_t x_t^T,   y_t = (S_t^T C_t + D x_t) silu(z_t)
 //   out = y / rms(y) * norm                                       over each of norm_groups equal parts of all heads together
 //
-// B and C are common to the heads of a group.
+// B and C are common to the heads of a group.  Lightning attention is the same with a constant decay, dt = 1, no convolution and no
+// D, a group per head (B: keys, C: queries, x: values) and the gate behind the norm:
+//
+//   u_t = silu(x, B, C);  S_t = decay S_(t-1) + B_t x_t^T,   y_t = S_t^T C_t,   out = y / rms(y) * norm * sigmoid(z)
 //
 // ssd_scan_kernel walks the tokens of a sequence with the state in registers (decoding, short portions, f32): CTA = (128 value
 // columns of a head, sequence); a thread holds four columns of every (256 / lanes per row)-th state channel.  The
@@ -53,7 +56,8 @@ __global__ void __launch_bounds__(kThreads, R == 0 || R > 16 ? 1 : R > 8 || ITEM
   float* slot = r.state + (size_t)p.slot[seq] * r.state_stride + r.state_off;
   float* S = slot + ((size_t)head * N) * r.vdim + e_first + c4;
   const float* past = slot + (size_t)r.heads * N * r.vdim;   // [taps - 1][channels]
-  const float a_neg = -expf(__ldg(r.a_log + head)), dt_bias = __ldg(r.dt_bias + head), skip = __ldg(r.d + head);
+  const float a_neg = r.decay ? 0.f : -expf(__ldg(r.a_log + head)), dt_bias = r.decay ? 0.f : __ldg(r.dt_bias + head), skip = r.d ? __ldg(r.d + head) : 0.f;
+  const float fixed = r.decay ? __ldg(r.decay + head) : 0.f;
 
   auto load4 = [&](const float* src) {
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -131,6 +135,15 @@ __global__ void __launch_bounds__(kThreads, R == 0 || R > 16 ? 1 : R > 8 || ITEM
         hist[q][2] = u[q];
         if (i < items) sm[i < cols ? i : i - cols + kSlice] = silu(v);
       }
+    } else if (!r.conv) {
+      float u[ITEMS];
+#pragma unroll
+      for (int q = 0; q < ITEMS; ++q) u[q] = x[r.col_x + channel(min(tid + q * kThreads, items - 1))];
+#pragma unroll
+      for (int q = 0; q < ITEMS; ++q) {
+        const int i = tid + q * kThreads;
+        if (i < items) sm[i < cols ? i : i - cols + kSlice] = silu(u[q]);
+      }
     } else {
       for (int i = tid; i < items; i += kThreads) {
         const int c = channel(i);
@@ -143,7 +156,7 @@ __global__ void __launch_bounds__(kThreads, R == 0 || R > 16 ? 1 : R > 8 || ITEM
         sm[i < cols ? i : i - cols + kSlice] = silu(v);
       }
     }
-    const float dt = pi_softplus(x[r.col_dt + head] + dt_bias), keep = expf(a_neg * dt);
+    const float dt = r.decay ? 1.f : pi_softplus(x[r.col_dt + head] + dt_bias), keep = r.decay ? fixed : expf(a_neg * dt);
     __syncthreads();
     float4 xv = *reinterpret_cast<const float4*>(sx + c4);
     xv = make_float4(dt * xv.x, dt * xv.y, dt * xv.z, dt * xv.w);
@@ -186,7 +199,7 @@ __global__ void __launch_bounds__(kThreads, R == 0 || R > 16 ? 1 : R > 8 || ITEM
 #pragma unroll
       for (int w = 0; w < kWarps; ++w) v += part[w][tid];
       const int e = head * r.vdim + e_first + tid;
-      p.y[(size_t)(row0 + t) * inner + e] = v * silu(x[r.col_z + e]);
+      p.y[(size_t)(row0 + t) * inner + e] = r.gate_last ? v : v * silu(x[r.col_z + e]);
     }
   }
   if (R > 0) {
@@ -263,17 +276,23 @@ __global__ void __launch_bounds__(kThreads) ssd_norm_kernel(const NormParams p) 
   for (int w = 0; w < kWarps; ++w) ss += red[w];
   const float inv = 1.0f / sqrtf(ss / (float)n + r.eps);
   O* out = static_cast<O*>(p.out) + (size_t)blockIdx.x * p.out_stride + c0;
+  const float* z = p.proj + (size_t)blockIdx.x * p.stride + r.col_z + c0;
   if (held) {
 #pragma unroll
     for (int j = 0; j < kHeld; ++j) {
       const int i = (tid + j * kThreads) * 4;
       if (i >= n) break;
       const float e[4] = {v[j].x, v[j].y, v[j].z, v[j].w};
+      float gate[4] = {1.f, 1.f, 1.f, 1.f};
+      if (r.gate_last) {
 #pragma unroll
-      for (int k = 0; k < 4; ++k) out[i + k] = pi_from_f32<O>(e[k] * inv * __ldg(r.norm + c0 + i + k));
+        for (int k = 0; k < 4; ++k) gate[k] = pi_sigmoid(z[i + k]);
+      }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) out[i + k] = pi_from_f32<O>(e[k] * inv * __ldg(r.norm + c0 + i + k) * gate[k]);
     }
   } else {
-    for (int i = tid; i < n; i += kThreads) out[i] = pi_from_f32<O>(y[i] * inv * __ldg(r.norm + c0 + i));
+    for (int i = tid; i < n; i += kThreads) out[i] = pi_from_f32<O>(y[i] * inv * __ldg(r.norm + c0 + i) * (r.gate_last ? pi_sigmoid(z[i]) : 1.f));
   }
 }
 

@@ -9,7 +9,8 @@
 // The recurrence is f32: operands of the tensor-core products (mma.sync) are pairs of bf16 planes, hi + lo (16 bits), three
 // products each.  The convolution leaves x, B and C as planes, padded to 16 channels and to whole chunks, so that the later
 // kernels only copy; the pass leaves the state as packed pairs.  B and C are common to a group's heads: a CTA takes several
-// heads of one group and scores C . B once for all of them.
+// heads of one group and scores C . B once for all of them.  (Lightning attention: no convolution, dt = 1, F = t ln(decay), no D; the
+// gate follows with the norm.)
 #include <math.h>
 
 #include <algorithm>
@@ -61,6 +62,14 @@ __global__ void __launch_bounds__(128) ssd_conv_kernel(const ChunkParams p, int 
     const int head = ((int)blockIdx.x - channel_blocks) * 128 + threadIdx.x;
     pi_grid_dependency_wait();
     if (head >= r.heads) return;
+    if (r.decay) {
+      const float a = __ldg(r.log_decay + head);
+      for (int t = 0; t < C; ++t) {      // tokens past the end: no decay, no input
+        p.dt[((size_t)chunk * r.heads + head) * C + t] = t < at.n ? 1.f : 0.f;
+        p.F[((size_t)chunk * r.heads + head) * C + t] = a * (float)min(t + 1, at.n);
+      }
+      return;
+    }
     const float a = -expf(__ldg(r.a_log + head)), bias = __ldg(r.dt_bias + head);
     const float* src = p.proj + (size_t)at.row0 * p.stride + r.col_dt + head;
     float* dt = p.dt + ((size_t)chunk * r.heads + head) * C;
@@ -89,8 +98,8 @@ __global__ void __launch_bounds__(128) ssd_conv_kernel(const ChunkParams p, int 
     const int k = i - r.heads * p.vdimp, g = k / p.dimp, n = k - g * p.dimp;   // g: B's groups, then C's
     if (n < r.dim) c = inner + (g < r.groups ? g * r.dim + n : gn + (g - r.groups) * r.dim + n);
   }
-  const float* w = r.conv + (size_t)max(c, 0) * r.taps;
-  const float bias = c >= 0 ? __ldg(r.conv_b + c) : 0.f;
+  const float* w = r.conv + (size_t)max(c, 0) * r.taps;   // not read without a convolution
+  const float bias = c >= 0 && r.conv ? __ldg(r.conv_b + c) : 0.f;
   const int channels = r.channels();
   const bool fresh = p.seq_start[at.seq] == 0;
   const float* past = r.state + (size_t)p.slot[at.seq] * r.state_stride + r.state_off + (size_t)r.heads * r.dim * r.vdim;
@@ -113,7 +122,7 @@ __global__ void __launch_bounds__(128) ssd_conv_kernel(const ChunkParams p, int 
     float w4[4] = {0.f, 0.f, 0.f, 0.f}, u[3] = {0.f, 0.f, 0.f};
 #pragma unroll
     for (int j = 0; j < 4; ++j)          // aligned to the current token: w4[3] is its own
-      if (j >= 4 - r.taps) w4[j] = __ldg(w + j - (4 - r.taps));
+      if (j >= 4 - r.taps) w4[j] = r.conv ? __ldg(w + j - (4 - r.taps)) : 1.f;
 #pragma unroll
     for (int j = 0; j < 3; ++j)
       if (j >= 4 - r.taps) u[j] = input(at.t0 - 3 + j);
@@ -332,7 +341,7 @@ __global__ void __launch_bounds__(kThreads, 2) ssd_output_kernel(const ChunkPara
   const int I = warp >> 1, half = warp & 1, rt = I * 16 + (lane >> 2);
   for (int h = h0; h < h0 + nh; ++h) {
     const size_t ch = (size_t)chunk * r.heads + h;
-    const float skip = __ldg(r.d + h);
+    const float skip = r.d ? __ldg(r.d + h) : 0.f;
     for (int c0 = 0; c0 < r.vdim; c0 += kVS) {
       const int cols = min(kVS, p.vdimp - c0);
       __syncthreads();                   // the last pass (or the scores) has read what is overwritten now
@@ -438,8 +447,12 @@ __global__ void __launch_bounds__(kThreads, 2) ssd_output_kernel(const ChunkPara
 #pragma unroll
           for (int k = 0; k < 2; ++k) {
             if (c0 + e + k >= r.vdim) break;
-            const float g = z[c0 + e + k];
-            y[c0 + e + k] = fmaf(skip, k ? x.y : x.x, acc[j][2 * i + k]) * g * pi_sigmoid(g);
+            float v = fmaf(skip, k ? x.y : x.x, acc[j][2 * i + k]);
+            if (!r.gate_last) {
+              const float g = z[c0 + e + k];
+              v *= g * pi_sigmoid(g);
+            }
+            y[c0 + e + k] = v;
           }
         }
       }
@@ -460,7 +473,7 @@ void sizes(ChunkParams& p) {
   while (p.heads_cta > 1 && local_smem(p) > 110 * 1024) --p.heads_cta;
 }
 cudaError_t grant(pi_ctx* ctx, void (*k)(const ChunkParams), size_t smem, pi_smem_grant& g) {
-  if (smem <= g.of(ctx) || smem <= 48 * 1024) return cudaSuccess;
+  if (smem <= g.of(ctx) || smem <= kSmemFree) return cudaSuccess;
   g.of(ctx) = smem;
   return cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
 }

@@ -74,9 +74,11 @@ class LlamaConfig:
             "intermediate_size", "vocab_size", "rms_norm_eps", "rope_theta", "attention_window", "rope_style")}
 
 
-MIXER_ATTENTION, MIXER_GLA, MIXER_MLSTM, MIXER_LATENT, MIXER_SSD = 0, 1, 2, 3, 4
+MIXER_ATTENTION, MIXER_GLA, MIXER_MLSTM, MIXER_LATENT, MIXER_SSD, MIXER_LIGHTNING = 0, 1, 2, 3, 4, 5
 FF_GELU, FF_SILU, FF_EXPERTS = 0, 1, 2
-NORM_DYT, NORM_LAYER = 0, 1
+UNIT_CLAMPED, UNIT_SILU = 0, 1
+SCORE_SIGMOID, SCORE_SOFTMAX = 0, 1
+NORM_DYT, NORM_LAYER, NORM_RMS = 0, 1, 2
 
 
 @dataclass
@@ -87,7 +89,12 @@ class LayerConfig:
     gated linear recurrence, ``gate_cap`` to the matrix memory.  Latent attention: ``rank`` latent channels, ``dim`` unrotated and
     ``rot_dims`` rotated channels per head, rotation stretched by ``rot_factor`` and the three constants behind it.  State-space
     recurrence: ``dim`` state channels, heads in ``groups``, ``conv`` taps, ``norm_groups`` parts.  Routed experts: ``ff`` is one
-    expert's size, ``shared_ff`` that of the expert every token meets."""
+    expert's size, ``shared_ff`` that of the expert every token meets (``shared_gate``: with a gate per token), ``unit`` their
+    activation, ``score`` what the router makes of its logits; a group of experts is as good as its ``group_best`` best scores
+    together; the chosen weights are brought to sum 1 if ``renorm`` and multiplied by ``route_scale``.  Attention with one map may
+    have ``biases``, q and k of unit root mean square (``unit_qk``), a ``distance_bias``, a ``sink`` and a gate per head, queries
+    that grow with the position (``q_temp_coef``, ``q_temp_every``; 0: not) and values mixed with those of the first layer that has
+    ``v_mix``.  ``decay``: the constant decay of every head of lightning attention."""
 
     mixer: int
     heads: int
@@ -119,6 +126,21 @@ class LayerConfig:
     shared_ff: int = 0
     limit: float = 0.0
     shared_limit: float = 0.0
+    biases: bool = False
+    unit_qk: bool = False
+    distance_bias: bool = False
+    sink: bool = False
+    head_gate: bool = False
+    v_mix: bool = False
+    q_temp_coef: float = 0.0
+    q_temp_every: float = 0.0
+    decay: tuple | None = None
+    unit: int = UNIT_CLAMPED
+    score: int = SCORE_SIGMOID
+    group_best: int = 2
+    renorm: bool = True
+    shared_gate: bool = True
+    route_scale: float = 1.0
 
 
 @dataclass
@@ -132,6 +154,9 @@ class LayeredConfig:
     norm: int = NORM_DYT
     tied: bool = True
     logit_scale: float = 1.0
+    embed_scale: float = 1.0
+    residual_mult: float = 1.0
+    side_dim: int = 0
 
     @property
     def has_state(self) -> bool:
@@ -185,21 +210,63 @@ class LayeredConfig:
         return cls(width=int(j["width"]), vocab_size=int(j["vocab"]), norm_eps=float(j["norm"]["eps"]), layers=layers, norm=NORM_LAYER, tied=False,
                    logit_scale=float(j["logit_scale"]))
 
-    @staticmethod
-    def _lilosun_feed_forward(i: int, mlp: dict | None) -> dict:
+    @classmethod
+    def _lilosun_feed_forward(cls, i: int, mlp: dict | None) -> dict:
         if mlp is None:
             return {}
         if mlp["kind"] == "dense":
             return dict(ff=int(mlp["ff"]), ff_kind=FF_SILU)
         if mlp["kind"] != "moe":
             raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        kw = dict(limit=float(mlp["expert"]["limit"]), **cls._experts(mlp))
+        if mlp.get("shared"):
+            kw.update(shared_limit=float(mlp["shared"]["limit"]))
+        return kw
+
+    @staticmethod
+    def _experts(mlp: dict) -> dict:
         r, groups, shared = mlp["router"], mlp["router"].get("groups"), mlp.get("shared")
-        kw = dict(ff=int(mlp["expert"]["ff"]), ff_kind=FF_EXPERTS, limit=float(mlp["expert"]["limit"]), experts=int(r["experts"]), top=int(r["top"]))
+        kw = dict(ff=int(mlp["expert"]["ff"]), ff_kind=FF_EXPERTS, experts=int(r["experts"]), top=int(r["top"]))
         if groups:
             kw.update(expert_groups=int(groups["count"]), keep_groups=int(groups["keep"]))
         if shared:
-            kw.update(shared_ff=int(shared["ff"]), shared_limit=float(shared["limit"]))
+            kw.update(shared_ff=int(shared["ff"]))
         return kw
+
+    @classmethod
+    def from_rubuvik(cls, j: dict) -> "LayeredConfig":
+        """The Rubuvik design's ``config.json``: two kinds of attention with a distance bias and lightning attention in any order, each
+        with a dense or a routed feed-forward or none, and a table of tokens beside the layers."""
+        layers = []
+        for i, e in enumerate(j["layers"]):
+            m = e["mixer"]
+            kw = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), **cls._rubuvik_feed_forward(i, e.get("mlp")))
+            if e["type"] in ("attention", "attention_2"):
+                mask, temp = m.get("mask"), m.get("q_temp")
+                if e["type"] == "attention_2":
+                    kw.update(biases=True, unit_qk=True, sink=True, head_gate=True)
+                if temp:
+                    kw.update(q_temp_coef=float(temp["coef"]), q_temp_every=float(temp["every"]))
+                layers.append(LayerConfig(MIXER_ATTENTION, kv_heads=int(m["kv_heads"]), window=int(mask["size"]) if mask else None, scale=float(m["scale"]),
+                                          distance_bias=True, v_mix=bool(m.get("v_mix", False)), **kw))
+            elif e["type"] == "lightning":
+                layers.append(LayerConfig(MIXER_LIGHTNING, decay=tuple(float(d) for d in m["decay"]), **kw))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+        side = j.get("token_side")
+        return cls(width=int(j["width"]), vocab_size=int(j["vocab"]), norm_eps=float(j["norm"]["eps"]), layers=layers, norm=NORM_RMS,
+                   embed_scale=float(j["embedding"]["scale"]), residual_mult=float(j["residual_mult"]), side_dim=int(side["dim"]) if side else 0)
+
+    @classmethod
+    def _rubuvik_feed_forward(cls, i: int, mlp: dict | None) -> dict:
+        if mlp is None:
+            return {}
+        if mlp["kind"] == "dense":
+            return dict(ff=int(mlp["ff"]), ff_kind=FF_SILU)
+        if mlp["kind"] != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        return dict(unit=UNIT_SILU, score=SCORE_SOFTMAX, group_best=1, renorm=False, shared_gate=False, route_scale=float(mlp["router"]["scale"]),
+                    **cls._experts(mlp))
 
 
 def read_safetensors(path: str) -> dict:

@@ -45,6 +45,7 @@ FAMILIES = {
     "Llama": Family(_load_llama, ("float32",)),
     "Sumosun": Family(_layered(LayeredConfig.from_sumosun), ("bfloat16", "float32")),
     "Lilosun": Family(_layered(LayeredConfig.from_lilosun), ("bfloat16", "float32")),
+    "Rubuvik": Family(_layered(LayeredConfig.from_rubuvik), ("bfloat16", "float32")),
 }
 
 

@@ -62,6 +62,107 @@ def lilosun(layers, width=88, vocab=400, eps=1e-5, logit_scale=1.5):
     return {"architecture": "Lilosun", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width, "logit_scale": logit_scale}
 
 
+# ---- Rubuvik ------------------------------------------------------------------------------------------------------------------
+def biased(heads=6, kv_heads=2, dim=20, vdim=28, window=30, scale=None, v_mix=True, temp=(0.4, 9), mlp=None):
+    """'attention': distance bias and query temperature."""
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5 if scale is None else scale, "v_mix": v_mix,
+         "mask": {"size": window} if window else None}
+    if temp:
+        m["q_temp"] = {"coef": temp[0], "every": temp[1]}
+    return {"type": "attention", "mlp": mlp, "mixer": m}
+
+
+def sunk(heads=6, kv_heads=2, dim=20, vdim=28, window=30, scale=None, v_mix=True, mlp=None):
+    """'attention_2': distance bias, biases, unit queries and keys, sink and gate per head."""
+    return dict(biased(heads, kv_heads, dim, vdim, window, 3.0 * dim ** -0.5 if scale is None else scale, v_mix, None, mlp), type="attention_2")
+
+
+def lightning(heads=4, dim=24, vdim=20, decay=(0.5, 0.83, 0.97, 0.998), mlp=None):
+    return {"type": "lightning", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay)}}
+
+
+def softmax_moe(experts=12, top=3, ff=40, groups=(3, 2), shared=56, scale=1.7):
+    r = {"experts": experts, "top": top, "scale": scale}
+    if groups:
+        r["groups"] = {"count": groups[0], "keep": groups[1]}
+    return {"kind": "moe", "router": r, "expert": {"ff": ff}, "shared": {"ff": shared} if shared else None}
+
+
+def rubuvik(layers, width=84, vocab=400, eps=1e-5, embed_scale=3.0, mult=0.6, side=12):
+    return {"architecture": "Rubuvik", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width, "embedding": {"scale": embed_scale},
+            "residual_mult": mult, "token_side": {"dim": side} if side else None}
+
+
+def rubuvik_tensors(cfg, seed):
+    """As lilosun_tensors: no sublayer writes the channels the routers read."""
+    rng = np.random.default_rng(seed)
+    W, V = cfg["width"], cfg["vocab"]
+    t = {}
+
+    def put(name, shape, std=None, mean=0.0):
+        x = rng.standard_normal(shape) * (1.0 / np.sqrt(shape[-1]) if std is None else std) + mean
+        t[name] = bf16_bits_to_f32(f32_to_bf16_bits(np.asarray(x, np.float32))).reshape(shape)
+
+    def gated(p, F):
+        put(p + "gate", (F, W), 2.0 / np.sqrt(W))
+        put(p + "up", (F, W), 1.5 / np.sqrt(W))
+        put(p + "down", (W, F), 1.2 / np.sqrt(F))
+        t[p + "down"][:CODE] = 0
+
+    put("embed", (V, W), 0.5, 0.05)
+    side = (cfg["token_side"] or {}).get("dim", 0)
+    if side:
+        put("side.embed", (V, side * len(cfg["layers"])), 1.0)
+    for i, e in enumerate(cfg["layers"]):
+        m, l = e["mixer"], f"l{i}."
+        p = l + "mix."
+        H, D, E = m["heads"], m["dim"], m["vdim"]
+        for n in ("norm1", "norm1b"):
+            put(l + n, (W,), 0.2)
+        if e["type"] == "lightning":
+            put(p + "q", (H * D, W), 1.5 / np.sqrt(W))
+            put(p + "k", (H * D, W), 1.5 / np.sqrt(W))
+            put(p + "v", (H * E, W), 1.5 / np.sqrt(W))
+            put(p + "g", (H * E, W), 1.5 / np.sqrt(W))
+            put(p + "norm", (H * E,), 0.2, 1.0)
+        else:
+            G = m["kv_heads"]
+            for n, rows in (("q", H * D), ("k", G * D), ("v", G * E)):
+                put(p + n, (rows, W), 1.5 / np.sqrt(W))
+                if e["type"] == "attention_2":
+                    put(p + n + ".b", (rows,), 0.5)
+            if e["type"] == "attention_2":
+                put(p + "sink", (H,), 1.5, 0.5)
+                put(p + "g", (H, W), 2.0 / np.sqrt(W))
+            if m["v_mix"]:
+                put(p + "vmix", (), 0.05, 0.4)
+        put(p + "o", (W, H * E))
+        t[p + "o"][:CODE] = 0
+        f = e["mlp"]
+        if f:
+            for n in ("norm2", "norm2b"):
+                put(l + n, (W,), 0.2)
+            p = l + "mlp."
+            if f["kind"] == "dense":
+                gated(p, f["ff"])
+            else:
+                n = f["router"]["experts"]
+                put(p + "router", (n, W), 0.45)
+                t[p + "router"][:, CODE:] = 0
+                put(p + "correction", (n,), 0.15, -0.1)
+                for k in range(n):
+                    gated(f"{p}e{k}.", f["expert"]["ff"])
+                if f.get("shared"):
+                    gated(p + "shared.", f["shared"]["ff"])
+        if side:
+            put(l + "side.gate", (side, W), 1.5 / np.sqrt(W))
+            put(l + "side.proj", (W, side))
+            t[l + "side.proj"][:CODE] = 0
+            put(l + "side.norm", (W,), 0.2, 0.7)
+    put("final.norm", (W,), 0.2)
+    return t
+
+
 CODE = 16   # leading channels of the embedding that only the routers and norms see change: no sublayer writes them
 
 
@@ -158,6 +259,8 @@ def tensors(cfg, seed, rank=5):
     """Random tensors (f32 values on the bf16 grid), scaled so that every part of the model moves the logits."""
     if cfg["architecture"] == "Lilosun":
         return lilosun_tensors(cfg, seed)
+    if cfg["architecture"] == "Rubuvik":
+        return rubuvik_tensors(cfg, seed)
     rng = np.random.default_rng(seed)
     W, V = cfg["width"], cfg["vocab"]
     t = {}
@@ -241,7 +344,7 @@ def device_model(ctx, cfg, t, compute, max_rows=1024):
 
 
 def layered_config(cfg):
-    return LayeredConfig.from_lilosun(cfg) if cfg["architecture"] == "Lilosun" else LayeredConfig.from_sumosun(cfg)
+    return getattr(LayeredConfig, "from_" + cfg["architecture"].lower())(cfg)
 
 
 def distance(got, want):
