@@ -984,6 +984,62 @@ def lilosun_work(cfg, model, B, ctx_len, M):
             "prefill_bytes": {"recurrence": sum(M * (4 * (2 * inner(l) + 2 * l.groups * l.dim + l.heads) + 10 * inner(l)) + 8 * (M // 64) * inner(l) * l.dim for l in rec)}}
 
 
+# Rubuvik beside Lilosun (the same experts, scalar-decay recurrences) and Sumosun (windowed attention over paged keys and values): the
+# same width, depth, vocabulary and window.
+RUBUVIK_SIZES = {
+    "w2048": dict(attention=dict(heads=16, kv_heads=4, dim=128, vdim=128), lightning=dict(heads=16, dim=128, vdim=128), side=128, like="w2048"),
+    "w4096": dict(attention=dict(heads=32, kv_heads=8, dim=128, vdim=128), lightning=dict(heads=32, dim=128, vdim=128), side=256, like="w4096"),
+}
+
+
+def rubuvik_config(size):
+    from paged_infer_b200 import loader as ld
+    s = RUBUVIK_SIZES[size]
+    l = LILOSUN_SIZES[s["like"]]
+    moe = dict(ff_kind=ld.FF_EXPERTS, unit=ld.UNIT_SILU, score=ld.SCORE_SOFTMAX, group_best=1, renorm=False, shared_gate=False, route_scale=2.5, **l["moe"])
+    dense = dict(ff_kind=ld.FF_SILU, ff=l["dense"])
+    attn = dict(window=l["window"], scale=128 ** -0.5, distance_bias=True, v_mix=True, **s["attention"])
+    rec = dict(decay=tuple(1 - 2.0 ** -(3 + 7 * h / s["lightning"]["heads"]) for h in range(s["lightning"]["heads"])), **s["lightning"])
+    kinds = [ld.LayerConfig(ld.MIXER_ATTENTION, biases=True, unit_qk=True, sink=True, head_gate=True, **attn, **moe), ld.LayerConfig(ld.MIXER_LIGHTNING, **rec, **dense),
+             ld.LayerConfig(ld.MIXER_ATTENTION, q_temp_coef=0.1, q_temp_every=512.0, **attn, **moe)]
+    return ld.LayeredConfig(l["width"], l["vocab"], 1e-6, [kinds[i % 3] for i in range(l["layers"])], norm=ld.NORM_RMS, embed_scale=1.0, residual_mult=0.5,
+                            side_dim=s["side"])
+
+
+def rubuvik_work(cfg, model, B, ctx_len, M):
+    """As lilosun_work."""
+    from paged_infer_b200 import loader as ld
+    W = cfg.width
+    attn = [l for l in cfg.layers if l.mixer == ld.MIXER_ATTENTION]
+    rec = [l for l in cfg.layers if l.mixer == ld.MIXER_LIGHTNING]
+    inner = lambda l: l.heads * l.vdim
+    per_expert = lambda l: 3 * W * l.ff
+    fixed = flops = 0
+    met = 0.0
+    for l in cfg.layers:
+        if l.mixer == ld.MIXER_ATTENTION:
+            own = W * (l.heads * l.dim + l.kv_heads * (l.dim + l.vdim) + inner(l) + l.head_gate * l.heads)
+        else:
+            own = W * (2 * l.heads * l.dim + 3 * inner(l))
+        own += 2 * W * cfg.side_dim
+        active = 0
+        if l.ff_kind == ld.FF_EXPERTS:
+            own += W * (3 * l.shared_ff + l.experts)
+            active = l.top * per_expert(l)
+            met += per_expert(l) * l.experts * (1 - (1 - l.top / l.experts) ** B)
+        else:
+            own += 3 * W * l.ff
+        fixed += own
+        flops += own + active
+    seen = sum(min(t + 1, attn[0].window) for t in range(M))
+    return {"decode_bytes": {"projections": 2 * (fixed + met + cfg.vocab_size * W),
+                             "attention": sum(B * min(ctx_len, l.window) * l.kv_heads * (l.dim + l.vdim) * 2 for l in attn),
+                             "recurrence": 2 * B * model.state_bytes()},
+            "prefill_flops": {"gemm_tc": 2.0 * M * flops, "attention": sum(l.heads * 2 * (l.dim + l.vdim) * seen for l in attn)},
+            # f32 projections in, the sums to and from the norm, bf16 result out, and the states between chunks of 64 tokens written and read once
+            "prefill_bytes": {"recurrence": sum(M * (4 * (2 * inner(l) + 2 * l.heads * l.dim) + 10 * inner(l)) + 8 * (M // 64) * inner(l) * l.dim for l in rec)}}
+
+
 def layered_work(cfg, model, B, ctx_len, M):
     """Algorithmic bytes of a decode step (B sequences at ctx_len) and flops / bytes of a prefill of M tokens, by kernel class."""
     from paged_infer_b200 import loader as ld
@@ -1096,7 +1152,8 @@ def measure_steps(api, ctx, torch, model, work, ctx_len, batches, M, K, W, peaks
 def run_layered_workload(args):
     """`--workload sumosun`: prefill and decode of the layered design at a few sizes, beside a Llama of the same width, depth,
     feed-forward and vocabulary (random weights; bf16 there, int8 weights with f32 activations and KV here).
-    `--workload lilosun`: Lilosun beside Sumosun, its closest model, both in bf16."""
+    `--workload lilosun`: Lilosun beside Sumosun, its closest model, both in bf16.
+    `--workload rubuvik`: Rubuvik beside Lilosun and Sumosun, all in bf16."""
     import torch
     from paged_infer_b200 import api
     from paged_infer_b200.loader import LlamaConfig
@@ -1111,21 +1168,28 @@ def run_layered_workload(args):
     res, launches = {}, ctx.kernel_launches()
     measure = lambda m, work: measure_steps(api, ctx, torch, m, work, ctx_len, batches, M, K, W, (hbm, tflops))
     name = args.workload
-    sizes = LILOSUN_SIZES if name == "lilosun" else LAYERED_SIZES
-    for size, s in sizes.items():
-        cfg, work = (lilosun_config(size), lilosun_work) if name == "lilosun" else (layered_config(size), layered_work)
+    sizes = {"sumosun": LAYERED_SIZES, "lilosun": LILOSUN_SIZES, "rubuvik": RUBUVIK_SIZES}[name]
+
+    def layered(label, cfg, work):
         m = api.LayeredModel.synthetic(ctx, cfg, seed=1, max_rows=M)
-        res[size] = {name: measure(m, lambda B, c, n: work(cfg, m, B, c, n))}
+        res[size][label] = measure(m, lambda B, c, n: work(cfg, m, B, c, n))
         m.close()
-        if name == "lilosun":
-            lc = layered_config(s["like"], s["layers"])
-            u = api.LayeredModel.synthetic(ctx, lc, seed=1, max_rows=M)
-            res[size]["sumosun"] = measure(u, lambda B, c, n: layered_work(lc, u, B, c, n))
+
+    for size, s in sizes.items():
+        res[size] = {}
+        if name == "rubuvik":
+            layered(name, rubuvik_config(size), rubuvik_work)
+            layered("lilosun", lilosun_config(s["like"]), lilosun_work)
+            layered("sumosun", layered_config(s["like"], LILOSUN_SIZES[s["like"]]["layers"]), layered_work)
+        elif name == "lilosun":
+            layered(name, lilosun_config(size), lilosun_work)
+            layered("sumosun", layered_config(s["like"], s["layers"]), layered_work)
         else:
+            layered(name, layered_config(size), layered_work)
             lc = LlamaConfig(num_hidden_layers=s["layers"], vocab_size=s["vocab"], rms_norm_eps=1e-5, rope_theta=10000.0, quantization="int8", **s["llama"])
             u = api.LlamaWeights.synthetic(ctx, lc, seed=1, std=0.02, max_batch=M, max_positions=M + 16)
             res[size]["llama_int8"] = measure(u, lambda B, c, n: uniform_work(lc, u, B, c, n))
-        u.close()
+            u.close()
     t1 = time.time()
     best = res["w2048"][name]["decode_b64"]
     print(json.dumps({"metric": "layered design: decode tokens/s at batch 64 (w2048)", "value": best["tok/s"], "unit": "tok/s", "n_gpus": 1, "steps": K,
@@ -1145,7 +1209,7 @@ def main():
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="tinyllama_b64_paged", choices=["tinyllama_b64_paged", "llama3_8b_tp", "llama2_70b_tp", "sumosun", "lilosun"])
+    ap.add_argument("--workload", default="tinyllama_b64_paged", choices=["tinyllama_b64_paged", "llama3_8b_tp", "llama2_70b_tp", "sumosun", "lilosun", "rubuvik"])
     ap.add_argument("--no-cpu", action="store_true", help="skip the cpu_baseline leg")
     ap.add_argument("--resident-only", action="store_true",
                     help="for a profiler's launch list: only the resident decode leg (warm-up + timed steps) over a pool filled with "
@@ -1166,7 +1230,7 @@ def main():
     if args.kernel_case:
         run_kernel_case(args)
         return
-    if args.workload in ("sumosun", "lilosun"):
+    if args.workload in ("sumosun", "lilosun", "rubuvik"):
         run_layered_workload(args)
         return
     if args.workload in TP_WORKLOADS:
