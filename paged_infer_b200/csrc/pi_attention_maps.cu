@@ -39,10 +39,15 @@ template <typename T>
 __global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const PrepareParams p) {
   const int row = blockIdx.x, lane = threadIdx.x & 31, vec = blockIdx.y * kPrepareWarps + (threadIdx.x >> 5);
   const int nq = p.heads * p.maps, nk = p.kv_heads * p.maps, half = p.rot_dims >> 1;
-  const int seq = p.row_seq[row], pos = p.row_pos[row];
-  const int lb = pos / p.block_size, off = pos % p.block_size;
-  const bool mapped = lb < p.lens[seq];
-  const int pb = mapped ? p.tables[(size_t)seq * p.max_blocks + lb] : 0;
+  const bool is_q = vec < nq;
+  const int pos = p.row_pos[row], off = pos % p.block_size;
+  bool mapped = false;
+  int pb = 0;
+  if (!is_q) {
+    const int seq = p.row_seq[row], lb = pos / p.block_size;
+    mapped = lb < p.lens[seq];
+    if (mapped) pb = p.tables[(size_t)seq * p.max_blocks + lb];
+  }
   pi_grid_dependency_wait();
   if (vec >= nq + nk + p.kv_heads) return;
   const size_t tile = (size_t)p.block_size * (p.maps * p.dp + p.vp);
@@ -57,7 +62,6 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const 
     }
     return;
   }
-  const bool is_q = vec < nq;
   const int pairs = (p.dp + 1) >> 1;     // dp >= dim, the pad is written too
   float* v = p.qkv + (size_t)row * p.stride + (size_t)vec * p.dim;   // k vectors follow the q vectors
   const float* bias = p.x.bias ? p.x.bias + (size_t)vec * p.dim : nullptr;

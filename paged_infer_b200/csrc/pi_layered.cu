@@ -1223,44 +1223,54 @@ pi_status run_sandwich(pi_ctx* ctx, pi_layered* m, const Layer& L, int i, const 
   const int M = st.b.rows;
   const pi_layer_config& c = L.c;
   const bool side = L.side_gate != nullptr;
-  pi_linear_args a;
+  pi_linear_args a;                       // a sublayer's result
   a.out = m->y;
   a.out_stride = m->c.width;
+  auto result = [&](const pi_row_norm& to, const pi_layer_norm& post) {
+    pi_row_norm n = to;
+    n.y = m->y;
+    n.y_stride = m->c.width;
+    n.post = post;
+    return n;
+  };
   PI_TRY(project(ctx, L.out, m->core, m->ld_core, M, bf16, a));
-  pi_row_norm n = c.ff > 0 || side ? row : after;
-  n.y = m->y;
-  n.y_stride = m->c.width;
-  n.post = L.post1;
-  if (c.ff > 0) n.norm = L.ln2;           // without: the side reads x as it stands
-  PI_TRY(pi_launch_row_norm(ctx, n));
+  pi_row_norm n = result(side ? row : after, L.post1);   // the row step behind the last sublayer
+  pi_expert_sum sum;
   if (c.ff > 0) {
-    n = side ? row : after;
+    pi_row_norm between = result(row, L.post1);
+    between.norm = L.ln2;
+    PI_TRY(pi_launch_row_norm(ctx, between));
     n.post = L.post2;
-    pi_expert_sum sum;
     if (c.ff_kind == PI_FF_EXPERTS) {
       PI_TRY(run_experts(ctx, m, L, M, bf16, &sum));
+      n.y = nullptr;
       n.experts = &sum;
     } else {
       PI_TRY(run_dense(ctx, m, L, M, bf16, a));
-      n.y = m->y;
-      n.y_stride = m->c.width;
     }
-    PI_TRY(pi_launch_row_norm(ctx, n));
   }
-  if (!side) return PI_OK;
+  if (!side) return pi_launch_row_norm(ctx, n);
+  pi_token_side t;
+  t.gate = L.side_gate;
+  t.proj = L.side_proj;
+  t.post = L.post_side;
+  t.table = pi_token_table{static_cast<const uint16_t*>(m->side_embed->w) + (size_t)i * m->c.side_dim, m->side_embed->ld, m->c.vocab_size, st.b.tokens};
+  if (pi_token_side_usable(ctx, t, M, m->c.width)) {
+    n.norm = after.norm;
+    n.h = after.h;
+    n.h_kind = after.h_kind;
+    return pi_launch_token_side(ctx, t, n);
+  }
+  PI_TRY(pi_launch_row_norm(ctx, n));     // h: x as it stands
   pi_linear_args g;
   g.epi = PI_EPI_GELU_TABLE;
   g.out = static_cast<float*>(m->side_h);
   g.out_bf16 = static_cast<__nv_bfloat16*>(m->side_h);
   g.out_stride = m->ld_side;
-  g.table = pi_token_table{static_cast<const uint16_t*>(m->side_embed->w) + (size_t)i * m->c.side_dim, m->side_embed->ld, m->c.vocab_size, st.b.tokens};
+  g.table = t.table;
   PI_TRY(project(ctx, L.side_gate, m->h, m->ld_h, M, bf16, g));
   PI_TRY(project(ctx, L.side_proj, m->side_h, m->ld_side, M, bf16, a));
-  n = after;
-  n.y = m->y;
-  n.y_stride = m->c.width;
-  n.post = L.post_side;
-  return pi_launch_row_norm(ctx, n);
+  return pi_launch_row_norm(ctx, result(after, L.post_side));
 }
 
 pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool* state, const Staged& st) {

@@ -203,6 +203,17 @@ struct pi_row_norm {
 };
 pi_status pi_launch_row_norm(pi_ctx* ctx, const pi_row_norm& n);
 
+// ---- the token table beside the layers (pi_side.cu) ---------------------------------------------------------------------------
+struct pi_token_side {
+  const pi_linear *gate = nullptr, *proj = nullptr;   // [dim][width], [width][dim]
+  pi_token_table table;                 // the layer's columns
+  pi_layer_norm post;                   // RMS norm of what it adds
+};
+constexpr int kSideRows = 8;            // steps of up to this many rows
+bool pi_token_side_usable(const pi_ctx* ctx, const pi_token_side& s, int rows, int width);
+// What the sublayer before left (n.y or n.experts, with n.post), the token's contribution, and n.h.
+pi_status pi_launch_token_side(pi_ctx* ctx, const pi_token_side& s, const pi_row_norm& n);
+
 // ---- recurrences (pi_recurrent.cu) --------------------------------------------------------------------------------
 enum pi_recurrence_kind { PI_REC_GLA = 0, PI_REC_MLSTM = 1 };
 struct pi_recurrence {

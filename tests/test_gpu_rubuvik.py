@@ -108,6 +108,27 @@ def test_sizes_and_constants_around_the_layers(ctx, change, compute):
     check_alone(ctx, cfg, t, draw(cfg, t, 80, 6), compute)
 
 
+@BOTH
+@pytest.mark.parametrize("width,side", [(512, 8), (1024, 384), (2048, 100), (3000, 256)])
+def test_token_table_at_every_number_of_rows(ctx, width, side, compute):
+    """One launch for few rows, projections and row steps for more, and for matrices that are too large: the same numbers."""
+    cfg = rubuvik([sunk(mlp=softmax_moe(experts=6, top=3, groups=None, ff=24)), lightning(mlp=dense(40)), biased()], width=width, vocab=240, side=side)
+    t = tensors(cfg, 15)
+    toks = draw(cfg, t, 100, 8)
+    want = reference(cfg, t).forward(toks)
+    s = Session(device_model(ctx, cfg, t, compute))
+    at, got = 0, []
+    for n in (1, 2, 4, 5, 8, 9, 23, 48):
+        got.append(s.run([("a", toks[at:at + n])])[0])
+        at += n
+    assert at == len(toks) and distance(np.concatenate(got), want).max() < LIMIT[compute]
+    seqs = [draw(cfg, t, 9, 50 + i) for i in range(5)]       # five rows of five sequences
+    for i in range(9):
+        outs = s.run([(f"s{j}", [q[i]]) for j, q in enumerate(seqs)])
+    for q, out in zip(seqs, outs):
+        assert distance(out, reference(cfg, t).forward(q)[-1:]).max() < 1.5 * LIMIT[compute]
+
+
 def test_token_table_of_one_channel(ctx):
     """Its normalised contribution is a sign times a vector: in the f32 mode only, where no rounding turns the sign."""
     cfg = rubuvik([lightning(), biased(mlp=dense(20))], width=72, vocab=96, side=1)
