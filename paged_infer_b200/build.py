@@ -51,7 +51,8 @@ def _newer(target: str, deps) -> bool:
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(verbose: bool = False, force: bool = False, ptxas_info: bool = False) -> str:
+def build(verbose: bool = False, force: bool = False, ptxas_info: bool = False, bookkeeping: bool = True) -> str:
+    """The CUDA library and the engine; ``bookkeeping``: also the host block bookkeeping on its own, which neither of them uses."""
     os.makedirs(OBJ, exist_ok=True)
     sources = sorted(glob.glob(os.path.join(CSRC, "*.cu")))
     headers = sorted(glob.glob(os.path.join(CSRC, "*.cuh"))) + sorted(glob.glob(os.path.join(INCLUDE, "*.h")))
@@ -81,7 +82,8 @@ def build(verbose: bool = False, force: bool = False, ptxas_info: bool = False) 
         if r.returncode != 0:
             sys.stderr.write(r.stdout + r.stderr)
             raise RuntimeError("linking libpaged_infer_cuda.so failed")
-    build_host()
+    if bookkeeping:
+        build_host()
     build_engine()
     return LIB
 

@@ -31,11 +31,21 @@ struct PrepareParams {
   pi_maps_prepare x;
 };
 
-// Warp per vector of a row: a q or k vector of one map, or a head's values.  Lanes hold pairs of adjacent channels (rot_dims is
-// even, so a rotation pair stays together), up to kHeld of them in registers; longer vectors are read twice.  Pool rows are
-// padded with zeros up to dp / vp.
-constexpr int kPrepareWarps = 4, kHeld = 4;
 template <typename T>
+__device__ __forceinline__ void store4(T* p, float4 v);
+template <>
+__device__ __forceinline__ void store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <>
+__device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+// Warp per vector of a row: a q or k vector of one map, or a head's values.  Lanes hold groups of adjacent channels (rot_dims is
+// even, so a rotation pair stays together): four (VEC: sizes are multiples of 4, at most 256), or two, up to kHeld of them in
+// registers, longer vectors are read twice.  Pool rows are padded with zeros up to dp / vp.
+constexpr int kPrepareWarps = 4, kHeld = 4;
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const PrepareParams p) {
   const int row = blockIdx.x, lane = threadIdx.x & 31, vec = blockIdx.y * kPrepareWarps + (threadIdx.x >> 5);
   const int nq = p.heads * p.maps, nk = p.kv_heads * p.maps, half = p.rot_dims >> 1;
@@ -55,6 +65,31 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const 
     const int g = vec - nq - nk, at = (nq + nk) * p.dim + g * p.vdim;
     const float* v = p.qkv + (size_t)row * p.stride + at;
     T* dst = static_cast<T*>(p.base) + ((size_t)pb * p.kv_heads + g) * tile + (size_t)p.block_size * p.maps * p.dp + (size_t)off * p.vp;
+    if (VEC) {
+      for (int e = lane * 4; e < p.vp; e += 128) {
+        float4 r = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (e < p.vdim) {
+          r = *reinterpret_cast<const float4*>(v + e);
+          if (p.x.bias) {
+            const float4 b = __ldg(reinterpret_cast<const float4*>(p.x.bias + at + e));
+            r = make_float4(r.x + b.x, r.y + b.y, r.z + b.z, r.w + b.w);
+          }
+          const pi_value_mix& m = p.x.mix;
+          if (m.first) {
+            float4* f = reinterpret_cast<float4*>(m.first + (size_t)row * m.stride + g * p.vdim + e);
+            if (m.keeps) {
+              *f = r;
+            } else {
+              const float4 o = *f;
+              const float l = m.lambda, k = 1.f - l;
+              r = make_float4(fmaf(l, o.x, k * r.x), fmaf(l, o.y, k * r.y), fmaf(l, o.z, k * r.z), fmaf(l, o.w, k * r.w));
+            }
+          }
+        }
+        if (mapped) store4<T>(dst + e, r);
+      }
+      return;
+    }
     for (int e = lane; e < p.vp; e += 32) {
       float r = 0.f;
       if (e < p.vdim) r = pi_mix_value(p.x.mix, row, g * p.vdim + e, v[e] + (p.x.bias ? __ldg(p.x.bias + at + e) : 0.f));
@@ -65,6 +100,46 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const 
   const int pairs = (p.dp + 1) >> 1;     // dp >= dim, the pad is written too
   float* v = p.qkv + (size_t)row * p.stride + (size_t)vec * p.dim;   // k vectors follow the q vectors
   const float* bias = p.x.bias ? p.x.bias + (size_t)vec * p.dim : nullptr;
+  const int kv = vec - nq, kg = is_q ? 0 : kv / p.maps, km = kv - kg * p.maps;
+  T* dst = static_cast<T*>(p.base) + ((size_t)pb * p.kv_heads + kg) * tile + (size_t)off * p.maps * p.dp + (size_t)km * p.dp;
+  const float* cs = p.rope_cos + (size_t)pos * half;
+  const float* sn = p.rope_sin + (size_t)pos * half;
+  float factor = is_q && p.x.q_temp ? __ldg(p.x.q_temp + pos) : 1.f;
+  if (VEC) {
+    float4 c[2];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int d = lane * 4 + 128 * i;
+      c[i] = d < p.dim ? *reinterpret_cast<const float4*>(v + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+      if (bias && d < p.dim) {
+        const float4 b = __ldg(reinterpret_cast<const float4*>(bias + d));
+        c[i] = make_float4(c[i].x + b.x, c[i].y + b.y, c[i].z + b.z, c[i].w + b.w);
+      }
+      ss = fmaf(c[i].x, c[i].x, fmaf(c[i].y, c[i].y, fmaf(c[i].z, c[i].z, fmaf(c[i].w, c[i].w, ss))));
+    }
+    if (p.x.unit_qk) factor /= sqrtf(pi_warp_sum(ss) / (float)p.dim + p.eps);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int d = lane * 4 + 128 * i, j = d >> 1;
+      float4 r = c[i];
+      if (j < half) {
+        r.x = c[i].x * cs[j] - c[i].y * sn[j];
+        r.y = c[i].y * cs[j] + c[i].x * sn[j];
+      }
+      if (j + 1 < half) {
+        r.z = c[i].z * cs[j + 1] - c[i].w * sn[j + 1];
+        r.w = c[i].w * cs[j + 1] + c[i].z * sn[j + 1];
+      }
+      r = make_float4(r.x * factor, r.y * factor, r.z * factor, r.w * factor);
+      if (is_q) {
+        if (d < p.dim) *reinterpret_cast<float4*>(v + d) = r;
+      } else if (mapped && d < p.dp) {
+        store4<T>(dst + d, r);
+      }
+    }
+    return;
+  }
   auto load = [&](int j) {
     const int d = 2 * j;
     float2 c = make_float2(d < p.dim ? v[d] : 0.f, d + 1 < p.dim ? v[d + 1] : 0.f);
@@ -77,7 +152,6 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const 
   float2 held[kHeld];
 #pragma unroll
   for (int i = 0; i < kHeld; ++i) held[i] = lane + 32 * i < pairs ? load(lane + 32 * i) : make_float2(0.f, 0.f);
-  float factor = is_q && p.x.q_temp ? __ldg(p.x.q_temp + pos) : 1.f;
   if (p.x.unit_qk) {
     float ss = 0.f;
 #pragma unroll
@@ -88,10 +162,6 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const 
     }
     factor /= sqrtf(pi_warp_sum(ss) / (float)p.dim + p.eps);
   }
-  const int kv = vec - nq, g = is_q ? 0 : kv / p.maps, m = kv - g * p.maps;
-  T* dst = static_cast<T*>(p.base) + ((size_t)pb * p.kv_heads + g) * tile + (size_t)off * p.maps * p.dp + (size_t)m * p.dp;
-  const float* cs = p.rope_cos + (size_t)pos * half;
-  const float* sn = p.rope_sin + (size_t)pos * half;
   auto finish = [&](int j, float2 c) {
     const int d = 2 * j;
     if (j < half) c = make_float2(c.x * cs[j] - c.y * sn[j], c.y * cs[j] + c.x * sn[j]);
@@ -198,8 +268,11 @@ pi_status pi_launch_maps_prepare(pi_ctx* ctx, const pi_maps_attention& a, const 
   PrepareParams p = {qkv, stride, a.heads, a.kv_heads, a.maps, a.dim, a.vdim, a.rot_dims, a.rope_cos, a.rope_sin, kv.base, kv.dp, kv.vp,
                      kv.block_size, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks, a.eps, x};
   const int vectors = (a.heads + a.kv_heads) * a.maps + a.kv_heads;
-  PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, kv.kind == PI_BF16 ? maps_prepare_kernel<__nv_bfloat16> : maps_prepare_kernel<float>,
-                                  dim3(b.rows, (vectors + kPrepareWarps - 1) / kPrepareWarps), dim3(kPrepareWarps * 32), 0, 1, p));
+  const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.dim <= 256 && a.vdim <= 256 && stride % 4 == 0 && x.mix.stride % 4 == 0;
+  void (*k)(const PrepareParams);
+  if (kv.kind == PI_BF16) k = vec ? maps_prepare_kernel<__nv_bfloat16, true> : maps_prepare_kernel<__nv_bfloat16, false>;
+  else k = vec ? maps_prepare_kernel<float, true> : maps_prepare_kernel<float, false>;
+  PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(b.rows, (vectors + kPrepareWarps - 1) / kPrepareWarps), dim3(kPrepareWarps * 32), 0, 1, p));
   return PI_OK;
 }
 

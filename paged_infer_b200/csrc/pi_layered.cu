@@ -1041,6 +1041,8 @@ pi_kv_view kv_view(const pi_kv_pool* pool, int attn) {
   return kv;
 }
 
+constexpr int kFoldRows = 128;
+
 // The layer's mixer, from h to core.
 pi_status run_mixer(pi_ctx* ctx, pi_layered* m, const Layer& L, pi_kv_pool* pool, pi_state_pool* state, const Staged& st, bool bf16) {
   const pi_seq_batch& b = st.b;
@@ -1078,8 +1080,9 @@ pi_status run_mixer(pi_ctx* ctx, pi_layered* m, const Layer& L, pi_kv_pool* pool
     prep.q_temp = L.temp >= 0 ? m->temps[L.temp].f : nullptr;
     if (c.v_mix) prep.mix = pi_value_mix{m->first_v, m->mix_stride, L.v_lambda, L.v_first};
     pi_maps_kv mk;
-    // biases, rotary positions, temperature, value mixing and the KV write fold into the projection; what needs a whole head does not
-    if (c.dim % 2 == 0 && !c.unit_qk && !c.head_gate) {
+    // biases, rotary positions, temperature, value mixing and the KV write fold into the projection; what needs a whole head does not,
+    // and where nothing is rotated a kernel of its own is faster for many rows than the look-ups in the epilogue
+    if (c.dim % 2 == 0 && !c.unit_qk && !c.head_gate && (M <= kFoldRows || c.rot_dims > 0)) {
       mk.bias = prep.bias;
       mk.q_temp = prep.q_temp;
       mk.mix = prep.mix;

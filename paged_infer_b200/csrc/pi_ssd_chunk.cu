@@ -1,7 +1,7 @@
 // Portions of many tokens through the recurrence of pi_ssd.cu, in chunks of 64 tokens that run side by side.  With
 // F_t = running sum of -exp(A_log) dt inside the chunk (never positive):
 //
-//   1. ssd_conv_kernel      convolution and silu of x, B, C; dt and F
+//   1. ssd_conv_kernel      convolution and silu of x, B, C; dt and F     (silu_planes_kernel: without a convolution)
 //   2. ssd_local_kernel     what the chunk adds to the state: U = sum_s e^(F_end - F_s) dt_s B_s x_s^T
 //   3. ssd_pass_kernel      the state in front of every chunk, one pass over the chunks (S <- e^F_end S + U); it takes U's place
 //   4. ssd_output_kernel    y_t = e^(F_t) S^T C_t + sum_(s <= t) (C_t . B_s) e^(F_t - F_s) dt_s x_s + D x_t, times silu(z_t)
@@ -148,6 +148,54 @@ __global__ void __launch_bounds__(128) ssd_conv_kernel(const ChunkParams p, int 
   }
 }
 
+// The same without a convolution, four channels at a time: CTA = (512 padded channels, chunk, 16 of its tokens).  Behind the
+// channels: the heads' dt and F.
+constexpr int kPlaneTokens = 16;
+__global__ void __launch_bounds__(128) silu_planes_kernel(const ChunkParams p, int channel_blocks) {
+  const pi_ssd& r = p.r;
+  const int chunk = blockIdx.y, t0 = blockIdx.z * kPlaneTokens;
+  const ChunkAt at = chunk_at(p, chunk);
+  if ((int)blockIdx.x >= channel_blocks) {
+    const int i = ((int)blockIdx.x - channel_blocks) * 128 + threadIdx.x, head = i / kPlaneTokens, t = t0 + i % kPlaneTokens;
+    pi_grid_dependency_wait();
+    if (head >= r.heads) return;
+    p.dt[((size_t)chunk * r.heads + head) * C + t] = t < at.n ? 1.f : 0.f;   // tokens past the end: no decay, no input
+    p.F[((size_t)chunk * r.heads + head) * C + t] = __ldg(r.log_decay + head) * (float)min(t + 1, at.n);
+    return;
+  }
+  const int i = ((int)blockIdx.x * 128 + threadIdx.x) * 4, inner = r.inner(), gn = r.groups * r.dim;
+  int c = -1;                            // first channel among x, B, C
+  if (i < r.heads * p.vdimp) {
+    const int h = i / p.vdimp, e = i - h * p.vdimp;
+    if (e < r.vdim) c = h * r.vdim + e;
+  } else if (i < (int)p.row) {
+    const int k = i - r.heads * p.vdimp, g = k / p.dimp, n = k - g * p.dimp;   // g: B's groups, then C's
+    if (n < r.dim) c = inner + (g < r.groups ? g * r.dim + n : gn + (g - r.groups) * r.dim + n);
+  }
+  pi_grid_dependency_wait();
+  if (i >= (int)p.row) return;
+  const float* x = p.proj + (size_t)at.row0 * p.stride + r.col_x + max(c, 0);
+  const size_t to = (size_t)chunk * C * p.row + i;
+#pragma unroll
+  for (int half = 0; half < kPlaneTokens; half += 8) {
+    float4 v[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = *reinterpret_cast<const float4*>(x + (size_t)min(t0 + half + j, at.n - 1) * p.stride);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int t = t0 + half + j;
+      const bool ok = c >= 0 && t < at.n;
+      const float a[4] = {ok ? v[j].x * pi_sigmoid(v[j].x) : 0.f, ok ? v[j].y * pi_sigmoid(v[j].y) : 0.f, ok ? v[j].z * pi_sigmoid(v[j].z) : 0.f,
+                          ok ? v[j].w * pi_sigmoid(v[j].w) : 0.f};
+      uint2 hi, lo;
+      split(a[0], a[1], hi.x, lo.x);
+      split(a[2], a[3], hi.y, lo.y);
+      *reinterpret_cast<uint2*>(p.hi + to + (size_t)t * p.row) = hi;
+      *reinterpret_cast<uint2*>(p.lo + to + (size_t)t * p.row) = lo;
+    }
+  }
+}
+
 // rows x cols (a multiple of 8) of both planes into shared memory
 __device__ __forceinline__ void copy_planes(const ChunkParams& p, int chunk, size_t col, int cols, __nv_bfloat16* hi, __nv_bfloat16* lo, int pitch) {
   const int pieces = cols / 8;
@@ -252,7 +300,7 @@ __global__ void __launch_bounds__(256) ssd_pass_kernel(const ChunkParams p) {
   }
   pi_grid_dependency_wait();
   if (!live) return;
-  constexpr int A = 4;                   // chunks fetched ahead
+  constexpr int A = 8;                   // chunks fetched ahead
   for (int c = c0; c < c1; c += A) {
     float u[A][V], keep[A];
 #pragma unroll
@@ -518,7 +566,12 @@ pi_status pi_launch_ssd_chunks(pi_ctx* ctx, const pi_ssd& r, const float* proj, 
   p.F = p.dt + gates;
   p.U = p.F + gates;
   const int channel_blocks = (int)((p.row + 127) / 128), head_blocks = (r.heads + 127) / 128;
-  PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, ssd_conv_kernel, dim3(channel_blocks + head_blocks, b.n_chunks), dim3(128), 0, 1, p, channel_blocks));
+  if (!r.conv && r.decay && r.vdim % 4 == 0 && r.dim % 4 == 0 && r.col_x % 4 == 0 && stride % 4 == 0) {
+    const int four = (int)((p.row + 511) / 512), heads = (r.heads * kPlaneTokens + 127) / 128;
+    PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, silu_planes_kernel, dim3(four + heads, b.n_chunks, C / kPlaneTokens), dim3(128), 0, 1, p, four));
+  } else {
+    PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, ssd_conv_kernel, dim3(channel_blocks + head_blocks, b.n_chunks), dim3(128), 0, 1, p, channel_blocks));
+  }
   const int per_group = r.heads / r.groups, blocks = r.groups * ((per_group + p.heads_cta - 1) / p.heads_cta), per_head = r.dim * r.vdim;
   const size_t s1 = local_smem(p), s2 = output_smem(p);
   PI_CUDA(ctx, grant(ctx, ssd_local_kernel, s1, g1));
