@@ -32,7 +32,7 @@ ALONE = {
     "attention_no_temperature": biased(temp=None, v_mix=False),
     "attention_odd": biased(heads=3, kv_heads=3, dim=11, vdim=9, window=19),
     "attention_17_per_group": biased(heads=34, kv_heads=2, dim=16, vdim=16, window=90),
-    "attention_one_head": biased(heads=1, kv_heads=1, dim=64, vdim=48, window=65),
+    "attention_one_head": biased(heads=1, kv_heads=1, dim=80, vdim=32, window=65),
     "attention_big_heads": biased(heads=2, kv_heads=1, dim=200, vdim=150, window=50),
     "attention_wide_values": biased(heads=4, kv_heads=2, dim=128, vdim=256, window=77),
     "attention_huge_keys": biased(heads=2, kv_heads=2, dim=300, vdim=20, window=40, scale=0.03),
@@ -40,11 +40,11 @@ ALONE = {
     "attention_2_everything": sunk(window=None, heads=7, kv_heads=1),
     "attention_2_window1": sunk(window=1, heads=2, kv_heads=2),
     "attention_2_odd": sunk(heads=9, kv_heads=3, dim=13, vdim=7, window=33),
-    "attention_2_one_head": sunk(heads=1, kv_heads=1, dim=64, vdim=48, window=129),
+    "attention_2_one_head": sunk(heads=1, kv_heads=1, dim=80, vdim=32, window=129),
     "attention_2_wide": sunk(heads=8, kv_heads=2, dim=128, vdim=64, window=100),
     "attention_2_huge_keys": sunk(heads=2, kv_heads=1, dim=300, vdim=300, window=70),
     "lightning": lightning(),
-    "lightning_one_head": lightning(heads=1, dim=32, vdim=64, decay=(0.99,)),
+    "lightning_one_head": lightning(heads=1, dim=48, vdim=80, decay=(0.99,)),
     "lightning_extremes": lightning(heads=5, dim=16, vdim=16, decay=(0.0, 1e-30, 0.02, 0.99999, 1.0)),
     "lightning_odd": lightning(heads=3, dim=5, vdim=7, decay=(0.3, 0.9, 0.97)),
     "lightning_large": lightning(heads=4, dim=128, vdim=128, decay=(0.6, 0.9, 0.98, 0.999)),
