@@ -220,7 +220,7 @@ struct pi_value_mix {
 
 // Where the epilogue of the fused [q;k;v] projection of a layered design puts its result: q rotated into `out`, k rotated
 // and v into the row's place in the pool (skipped when its block is not mapped).  Rotation pairs are adjacent channels, so
-// dim must be even (odd ones take pi_launch_maps_rope_kv).
+// dim must be even (odd ones take pi_launch_maps_prepare).
 struct pi_maps_kv {
   int q_rows = 0, k_rows = 0, maps = 1, dim = 0, vdim = 0, rot_dims = 0;
   const float *rope_cos = nullptr, *rope_sin = nullptr;   // [positions][rot_dims / 2]
