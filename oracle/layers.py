@@ -580,3 +580,158 @@ class Rubuvik:
             if layer_outputs is not None:
                 layer_outputs.append(x.copy())
         return linear(self.t["embed"], self.norm("final.norm", x))
+
+
+# ---- mechanisms of Noresun ------------------------------------------------------------------------------------------
+
+def bigram_rows(tokens, buckets, mul_prev, mul_cur):
+    """Row of the table of token pairs for every token of a sequence; the last row, number ``buckets``, for the first token."""
+    t = [int(x) for x in tokens]
+    return np.array([buckets] + [(t[i - 1] * mul_prev + t[i] * mul_cur) % buckets for i in range(1, len(t))], np.int64)
+
+
+def banded_frequencies(dims, base, scaling):
+    """Angle per position of every pair.  ``scaling``: pairs with a wavelength under original / high keep theirs, those over
+    original / low are slowed by ``factor``, those in between are blended by where original / wavelength lies between the two."""
+    f = float(base) ** (-2.0 * np.arange(dims // 2) / dims)
+    if scaling is None:
+        return f
+    out = f.copy()
+    for i in range(len(f)):
+        turns = scaling["original"] * f[i] / (2 * np.pi)          # within the original length
+        if turns > scaling["high"]:
+            continue
+        if turns < scaling["low"]:
+            out[i] = f[i] / scaling["factor"]
+        else:
+            s = (turns - scaling["low"]) / (scaling["high"] - scaling["low"])
+            out[i] = (1 - s) * f[i] / scaling["factor"] + s * f[i]
+    return out
+
+
+def window_sigmoid(q, k, v, scale, bias, window):
+    """One head: every visible key weighs sigmoid(scale (q_t . k_s) + bias), whatever the others weigh; 0 <= t - s < window."""
+    out = np.zeros((q.shape[0], v.shape[1]), q.dtype)
+    for t in range(q.shape[0]):
+        lo = 0 if window is None else max(0, t - window + 1)
+        out[t] = sigmoid((k[lo:t + 1] @ q[t]) * scale + bias) @ v[lo:t + 1]
+    return out
+
+
+def keys_and_values(h, w, kv_heads, dim, vdim, frequencies, eps):
+    """k normalised over the whole projection, then rotated; v as it is."""
+    T = h.shape[0]
+    k = (unit_rms(linear(w["k"], h), eps) * w["k.norm"]).reshape(T, kv_heads, dim)
+    return rotate_pairs(k, np.arange(T), frequencies, 1.0), linear(w["v"], h).reshape(T, kv_heads, vdim)
+
+
+def sigmoid_attention(h, w, heads, dim, frequencies, scale, window, eps, k, v):
+    """w: dict q, q.norm, pb, o; k, v: of this layer or of the one it shares them with."""
+    T, kv_heads, vdim = v.shape
+    q = (unit_rms(linear(w["q"], h), eps) * w["q.norm"]).reshape(T, heads, dim)
+    q = rotate_pairs(q, np.arange(T), frequencies, 1.0)
+    o = np.zeros((T, heads, vdim), h.dtype)
+    for n in range(heads):
+        g = n // (heads // kv_heads)
+        o[:, n] = window_sigmoid(q[:, n], k[:, g], v[:, g], scale, w["pb"][n], window)
+    return linear(w["o"], o.reshape(T, heads * vdim))
+
+
+def positive_candidate(u):
+    """u + 1/2 from zero up, sigmoid(u) below: positive and continuous."""
+    return np.where(u >= 0, u + 0.5, sigmoid(u))
+
+
+def min_gru_scan(z, candidate, state):
+    """S_t = (1 - z_t) S_(t-1) + z_t candidate_t, element by element.  -> (S of every token, the last S)."""
+    S = state.copy()
+    out = np.zeros_like(z)
+    for t in range(z.shape[0]):
+        S = (1 - z[t]) * S + z[t] * candidate[t]
+        out[t] = S
+    return out, S
+
+
+def min_gru(h, w):
+    """w: dict z, z.b, x, x.b, g, o."""
+    z, u = sigmoid(linear(w["z"], h) + w["z.b"]), linear(w["x"], h) + w["x.b"]
+    s, _ = min_gru_scan(z, positive_candidate(u), np.zeros(z.shape[1], h.dtype))
+    return linear(w["o"], s * silu(linear(w["g"], h)))
+
+
+def route_chosen(z, top):
+    """Router logits [tokens, experts] -> (the ``top`` largest [tokens, top], softmax over these alone)."""
+    ids = np.argsort(-z, axis=-1, kind="stable")[:, :top]
+    return ids, softmax_scores(np.take_along_axis(z, ids, 1))
+
+
+def relu2_moe(h, w, top):
+    """w: dict router, router.b, e<i>.up/down."""
+    ids, weights = route_chosen(linear(w["router"], h) + w["router.b"], top)
+    out = np.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, p in zip(ids[t], weights[t]):
+            out[t] += p * linear(w[f"e{e}.down"], np.maximum(linear(w[f"e{e}.up"], h[t]), 0) ** 2)
+    return out
+
+
+class Noresun:
+    """The whole design from a config dict and a dict of float arrays under the checkpoint's tensor names."""
+
+    def __init__(self, config: dict, tensors: dict, dtype=np.float64):
+        self.c = config
+        self.t = {k: np.asarray(v, dtype) for k, v in tensors.items()}
+        self.margin = None    # per token of the last forward: the closest call of any router, in logits
+
+    def part(self, prefix):
+        return {k[len(prefix):]: v for k, v in self.t.items() if k.startswith(prefix)}
+
+    def embed(self, tokens):
+        e = self.c["embedding"]
+        x = self.t["embed"][tokens] * e["scale"]
+        if e.get("bigram"):
+            b = e["bigram"]
+            x = x + self.t["bigram"][bigram_rows(tokens, b["buckets"], b["mul_prev"], b["mul_cur"])]
+        return x
+
+    def mixer(self, i, layer, h):
+        w, m, eps = self.part(f"l{i}.mix."), layer["mixer"], self.c["norm"]["eps"]
+        if layer["type"] == "mingru":
+            return min_gru(h, w)
+        if layer["type"] != "attention":
+            raise ValueError(f"unknown mixer {layer['type']}")
+        rot, mask = m.get("rot"), m.get("mask")
+        f = banded_frequencies(rot["dims"], rot["base"], rot.get("scaling")) if rot else []
+        if m.get("kv_from") is None:
+            self.kv[i] = keys_and_values(h, w, m["kv_heads"], m["dim"], m["vdim"], f, eps)
+        k, v = self.kv[i if m.get("kv_from") is None else m["kv_from"]]
+        return sigmoid_attention(h, w, m["heads"], m["dim"], f, m["scale"], mask["size"] if mask else None, eps, k, v)
+
+    def feed_forward(self, i, mlp, h):
+        w, top = self.part(f"l{i}.mlp."), mlp["router"]["top"]
+        if mlp["kind"] != "moe":
+            raise ValueError(f"unknown feed-forward {mlp['kind']}")
+        z = np.sort(linear(w["router"], h) + w["router.b"], axis=-1)[:, ::-1]
+        if top < z.shape[1]:
+            self.margin = np.minimum(self.margin, z[:, top - 1] - z[:, top])
+        return relu2_moe(h, w, top)
+
+    def forward(self, tokens, layer_outputs: list | None = None):
+        """Logits [tokens, vocab] of one sequence from its first token."""
+        tokens, eps, alpha = np.asarray(tokens), self.c["norm"]["eps"], self.c["postln_alpha"]
+        x = self.embed(tokens)
+        self.margin = np.full(len(tokens), np.inf)
+        self.kv = {}
+
+        def after(name, x, gate, y):
+            y = y * sigmoid(linear(self.t[gate], x) + self.t[gate + ".b"])
+            return unit_rms(alpha * x + y, eps) * self.t[name]
+
+        for i, layer in enumerate(self.c["layers"]):
+            l = f"l{i}."
+            x = after(l + "norm1", x, l + "rg1", self.mixer(i, layer, x))
+            if layer.get("mlp"):
+                x = after(l + "norm2", x, l + "rg2", self.feed_forward(i, layer["mlp"], x))
+            if layer_outputs is not None:
+                layer_outputs.append(x.copy())
+        return linear(self.t["embed"], unit_rms(x, eps) * self.t["final.norm"])
