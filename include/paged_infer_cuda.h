@@ -366,14 +366,15 @@ pi_status pi_kv_fill_normal(pi_ctx* ctx, pi_kv_pool* pool, uint64_t seed, float 
  * in a state pool (recurrences).  No counterpart in the reference. */
 
 enum { PI_MIXER_ATTENTION = 0, PI_MIXER_GLA = 1, PI_MIXER_MLSTM = 2, PI_MIXER_LATENT = 3 /* latent attention */, PI_MIXER_SSD = 4 /* state-space, scalar decay */,
-       PI_MIXER_LIGHTNING = 5 /* a constant decay per head */ };
+       PI_MIXER_LIGHTNING = 5 /* a constant decay per head */, PI_MIXER_MINGRU = 6 /* gated recurrence, element by element */ };
 enum { PI_FF_GELU = 0, PI_FF_SILU = 1, PI_FF_EXPERTS = 2 /* routed */ };
 /* Experts: their units, and the scores the router makes of its logits. */
-enum { PI_UNIT_CLAMPED = 0 /* clamped gated units */, PI_UNIT_SILU = 1 };
-enum { PI_SCORE_SIGMOID = 0, PI_SCORE_SOFTMAX = 1 };
+enum { PI_UNIT_CLAMPED = 0 /* clamped gated units */, PI_UNIT_SILU = 1, PI_UNIT_RELU2 = 2 /* no gate: the square of relu */ };
+enum { PI_SCORE_SIGMOID = 0, PI_SCORE_SOFTMAX = 1, PI_SCORE_CHOSEN = 2 /* chosen by their logits, softmax over the chosen alone */ };
 /* Normalisation: Dynamic Tanh before and after every sublayer; or layer norm (a weight, no bias) before it and a scale per
- * channel behind it; or RMS norm (times 1 + weight) before and after it, the result times residual_mult. */
-enum { PI_NORM_DYT = 0, PI_NORM_LAYER = 1, PI_NORM_RMS = 2 };
+ * channel behind it; or RMS norm (times 1 + weight) before and after it, the result times residual_mult; or RMS norm (times
+ * weight) of the sum, residual_keep x + result, which sublayers then read as it is. */
+enum { PI_NORM_DYT = 0, PI_NORM_LAYER = 1, PI_NORM_RMS = 2, PI_NORM_SUM = 3 };
 
 typedef struct {
   int32_t mixer;
@@ -410,6 +411,14 @@ typedef struct {
    * they are multiplied by route_scale; shared_gate: the shared expert has a gate per token */
   int32_t unit, score, group_best, renorm, shared_gate;
   float route_scale;
+  int32_t router_bias;     /* experts: a bias of the logits ("router.b") instead of a correction of the choice */
+  /* rotation: rot_factor by wavelength instead, without a factor of cos and sin: between rot_slow and rot_fast turns within
+   * rot_original positions the slowed and the plain frequency are blended linearly in the number of turns */
+  int32_t rot_banded;
+  /* attention with one map: q and k normalised over the whole projection (RMS, weights "q.norm" and "k.norm") ahead of the rotation;
+   * a key weighs sigmoid(score + a bias of the head), not normalised over the keys; kv_from: 1 + the layer whose keys and values
+   * this one reads instead of having its own, 0: its own */
+  int32_t norm_qk, sigmoid_weights, kv_from;
 } pi_layer_config;
 
 typedef struct {
@@ -423,6 +432,11 @@ typedef struct {
   float embed_scale;       /* of the embedding, not of the output matrix */
   float residual_mult;     /* PI_NORM_RMS: of everything that is added to the residual stream */
   int32_t side_dim;        /* PI_NORM_RMS: channels of a layer's own row of a table of tokens, added behind its sublayers; 0: none */
+  float residual_keep;     /* PI_NORM_SUM: of the residual stream in the sum */
+  int32_t sublayer_gate;   /* PI_NORM_SUM: a sublayer's result times sigmoid(rg h + b), h the sublayer's input */
+  /* a table of token pairs added to the embedding: row (previous token pair_prev + token pair_cur) mod pair_buckets, for a sequence's
+   * first token row pair_buckets; the factors are in [0, pair_buckets).  0 buckets: none */
+  int32_t pair_buckets, pair_prev, pair_cur;
   const pi_layer_config* layers;
 } pi_layered_config;
 

@@ -69,13 +69,15 @@ class LayerConfigC(C.Structure):
                [(n, C.c_float) for n in ("limit", "shared_limit")] + \
                [(n, C.c_int32) for n in ("biases", "unit_qk", "distance_bias", "sink", "head_gate", "v_mix")] + \
                [(n, C.c_double) for n in ("q_temp_coef", "q_temp_every")] + [("decay", C.POINTER(C.c_double))] + \
-               [(n, C.c_int32) for n in ("unit", "score", "group_best", "renorm", "shared_gate")] + [("route_scale", C.c_float)]
+               [(n, C.c_int32) for n in ("unit", "score", "group_best", "renorm", "shared_gate")] + [("route_scale", C.c_float)] + \
+               [(n, C.c_int32) for n in ("router_bias", "rot_banded", "norm_qk", "sigmoid_weights", "kv_from")]
 
 
 class LayeredConfigC(C.Structure):
     _fields_ = [("width", C.c_int32), ("vocab_size", C.c_int32), ("num_layers", C.c_int32), ("norm_eps", C.c_float), ("compute", C.c_int32),
                 ("max_rows", C.c_int32), ("norm", C.c_int32), ("tied", C.c_int32), ("logit_scale", C.c_float), ("embed_scale", C.c_float), ("residual_mult", C.c_float),
-                ("side_dim", C.c_int32), ("layers", C.POINTER(LayerConfigC))]
+                ("side_dim", C.c_int32), ("residual_keep", C.c_float)] + \
+               [(n, C.c_int32) for n in ("sublayer_gate", "pair_buckets", "pair_prev", "pair_cur")] + [("layers", C.POINTER(LayerConfigC))]
 
 
 class NamedTensorC(C.Structure):

@@ -621,9 +621,12 @@ class LayeredModel(_Steps):
                     v = None if v is None else (C.c_double * len(v))(*v)     # the structure keeps the array alive
                 elif name == "window":
                     v = 0 if v is None else v
+                elif name == "kv_from":
+                    v = 0 if v is None else v + 1
                 setattr(c, name, v)
         cfg = _lib.LayeredConfigC(config.width, config.vocab_size, len(config.layers), config.norm_eps, cls.COMPUTE[compute], max_rows, config.norm,
-                                  int(config.tied), config.logit_scale, config.embed_scale, config.residual_mult, config.side_dim, layers)
+                                  int(config.tied), config.logit_scale, config.embed_scale, config.residual_mult, config.side_dim, config.residual_keep,
+                                  int(config.sublayer_gate), config.pair_buckets, config.pair_prev, config.pair_cur, layers)
         cfg._layers = layers
         return cfg
 

@@ -7,8 +7,11 @@
 //   o = a_1 - lambda a_2;  out = out_scale o / rms(o)          (two maps)
 //   out *= sigmoid(gate)                                       (with an output gate, per channel or per head)
 //
+// or, with one map, keys that weigh by themselves: a_1 = sum over the keys of sigmoid(score_1 + bias of the head) v.
+//
 // Kernels: maps_prepare_kernel brings q, k and v into their final form (bias, unit root mean square, rotation, temperature of the
-// queries, mixing of the values) and writes k and v into the pool; maps_attn_plain_kernel is the f32
+// queries, mixing of the values) and writes k and v into the pool; maps_prepare_whole_kernel is the one for q and k that are
+// normalised over the whole projection; maps_attn_plain_kernel is the f32
 // path and the one for sizes the tensor-core kernels of pi_attention_maps_tc.cu do not hold.
 #include <math.h>
 
@@ -181,6 +184,138 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const 
   for (int j = lane + 32 * kHeld; j < pairs; j += 32) finish(j, load(j));
 }
 
+// CTA per row: q and k (which follow one another) each over the root mean square of all their heads, times a weight per channel, then
+// rotated; v as it is.  Groups of four adjacent channels (VEC: sizes are multiples of 4) or pairs, up to kWholeHeld of them per thread
+// in registers, the others are read twice.  Pool rows are padded with zeros up to dp / vp.
+constexpr int kWholeThreads = 256, kWholeHeld = 5;
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kWholeThreads) maps_prepare_whole_kernel(const PrepareParams p) {
+  constexpr int G = VEC ? 4 : 2;
+  __shared__ float red[2][kWholeThreads / 32];
+  const int row = blockIdx.x, tid = threadIdx.x, half = p.rot_dims >> 1;
+  const int gd = (p.dim + G - 1) / G, nq = p.heads * gd, n = nq + (p.x.q_only ? 0 : p.kv_heads * gd);   // groups: of a head, of q, of all
+  const int pos = p.row_pos[row], off = pos % p.block_size;
+  bool mapped = false;
+  int pb = 0;
+  if (!p.x.q_only) {
+    const int seq = p.row_seq[row], lb = pos / p.block_size;
+    mapped = lb < p.lens[seq];
+    if (mapped) pb = p.tables[(size_t)seq * p.max_blocks + lb];
+  }
+  const float* cs = p.rope_cos + (size_t)pos * half;
+  const float* sn = p.rope_sin + (size_t)pos * half;
+  float* qkv = p.qkv + (size_t)row * p.stride;
+  struct Group {
+    float v[G];
+  };
+  auto load = [&](const float* src, int i) {
+    const int vec = i / gd, d = (i - vec * gd) * G;
+    src += (size_t)vec * p.dim + d;
+    Group g;
+    if (VEC) {
+      const float4 f = *reinterpret_cast<const float4*>(src);
+      g.v[0] = f.x;
+      g.v[1] = f.y;
+      g.v[G - 2] = f.z;
+      g.v[G - 1] = f.w;
+    } else {
+      g.v[0] = src[0];
+      g.v[1] = d + 1 < p.dim ? src[1] : 0.f;
+    }
+    return g;
+  };
+  auto square = [&](const Group& g) {
+    float s = 0.f;
+#pragma unroll
+    for (int k = 0; k < G; ++k) s = fmaf(g.v[k], g.v[k], s);
+    return s;
+  };
+  Group w[kWholeHeld];                    // constants: ahead of the dependency wait
+#pragma unroll
+  for (int j = 0; j < kWholeHeld; ++j) w[j] = load(p.x.norm_qk, min(tid + j * kWholeThreads, n - 1));
+  pi_grid_dependency_wait();
+  Group held[kWholeHeld];
+  float ss[2] = {0.f, 0.f};
+#pragma unroll
+  for (int j = 0; j < kWholeHeld; ++j) held[j] = load(qkv, min(tid + j * kWholeThreads, n - 1));
+#pragma unroll
+  for (int j = 0; j < kWholeHeld; ++j) {
+    const int i = tid + j * kWholeThreads;
+    if (i < nq) ss[0] += square(held[j]);
+    else if (i < n) ss[1] += square(held[j]);
+  }
+  for (int i = tid + kWholeHeld * kWholeThreads; i < n; i += kWholeThreads) ss[i < nq ? 0 : 1] += square(load(qkv, i));
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    ss[k] = pi_warp_sum(ss[k]);
+    if ((tid & 31) == 0) red[k][tid >> 5] = ss[k];
+  }
+  // the values do not wait for the sums
+  const size_t tile = (size_t)p.block_size * (p.dp + p.vp);
+  T* blk = static_cast<T*>(p.base) + (size_t)pb * p.kv_heads * tile;
+  if (mapped) {
+    const float* v = qkv + (size_t)(p.heads + p.kv_heads) * p.dim;
+    for (int i = tid; i < p.kv_heads * (p.vp / G); i += kWholeThreads) {
+      const int g = i / (p.vp / G), e = (i - g * (p.vp / G)) * G;
+      T* dst = blk + g * tile + (size_t)p.block_size * p.dp + (size_t)off * p.vp + e;
+      if (VEC) {
+        store4<T>(dst, e < p.vdim ? *reinterpret_cast<const float4*>(v + (size_t)g * p.vdim + e) : make_float4(0.f, 0.f, 0.f, 0.f));
+      } else {
+#pragma unroll
+        for (int k = 0; k < G; ++k) dst[k] = pi_from_f32<T>(e + k < p.vdim ? v[(size_t)g * p.vdim + e + k] : 0.f);
+      }
+    }
+    for (int i = tid; i < p.kv_heads * (p.dp - p.dim); i += kWholeThreads) {
+      const int g = i / (p.dp - p.dim), d = p.dim + i - g * (p.dp - p.dim);
+      blk[g * tile + (size_t)off * p.dp + d] = pi_from_f32<T>(0.f);
+    }
+  }
+  __syncthreads();
+  float inv[2] = {0.f, 0.f};
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+#pragma unroll
+    for (int j = 0; j < kWholeThreads / 32; ++j) inv[k] += red[k][j];
+    inv[k] = 1.0f / sqrtf(inv[k] / (float)((k ? p.kv_heads : p.heads) * p.dim) + p.eps);
+  }
+  auto finish = [&](int i, Group g, const Group& w) {
+    const int vec = i / gd, d = (i - vec * gd) * G;
+    const float f = inv[i < nq ? 0 : 1];
+#pragma unroll
+    for (int k = 0; k < G; ++k) g.v[k] = g.v[k] * f * w.v[k];
+#pragma unroll
+    for (int k = 0; k < G; k += 2) {
+      const int j = (d + k) >> 1;
+      if (j < half) {
+        const float a = g.v[k], b = g.v[k + 1];
+        g.v[k] = a * cs[j] - b * sn[j];
+        g.v[k + 1] = b * cs[j] + a * sn[j];
+      }
+    }
+    if (i < nq) {
+      float* dst = qkv + (size_t)vec * p.dim + d;
+      if (VEC) {
+        *reinterpret_cast<float4*>(dst) = make_float4(g.v[0], g.v[1], g.v[G - 2], g.v[G - 1]);
+      } else {
+        dst[0] = g.v[0];
+        if (d + 1 < p.dim) dst[1] = g.v[1];
+      }
+    } else if (mapped) {
+      T* dst = blk + (vec - p.heads) * tile + (size_t)off * p.dp + d;
+      if (VEC) {
+        store4<T>(dst, make_float4(g.v[0], g.v[1], g.v[G - 2], g.v[G - 1]));
+      } else {
+        dst[0] = pi_from_f32<T>(g.v[0]);
+        if (d + 1 < p.dim) dst[1] = pi_from_f32<T>(g.v[1]);
+      }
+    }
+  };
+#pragma unroll
+  for (int j = 0; j < kWholeHeld; ++j)
+    if (tid + j * kWholeThreads < n) finish(tid + j * kWholeThreads, held[j], w[j]);
+  for (int i = tid + kWholeHeld * kWholeThreads; i < n; i += kWholeThreads) finish(i, load(qkv, i), load(p.x.norm_qk, i));
+}
+
 // One CTA of 4 warps per (row, head): the warps take every fourth key and merge; lanes hold the channels.  f32
 // throughout, any sizes (smem: q, per-warp accumulators of both maps).
 constexpr int kPlainWarps = 4;
@@ -204,6 +339,8 @@ __global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const
   const size_t tile = (size_t)p.block_size * (nm * DP + p.vp);
   float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const float slope = p.slopes ? __ldg(p.slopes + head) : 0.f, sink = p.sinks ? __ldg(p.sinks + head) : -INFINITY;
+  const bool by_itself = p.sigmoid_bias != nullptr;
+  const float self_bias = by_itself ? __ldg(p.sigmoid_bias + head) : 0.f;
   for (int t = lo + warp; t <= pos; t += kPlainWarps) {
     const int lb = t / p.block_size, off = t - lb * p.block_size;
     if (lb >= len) break;
@@ -217,6 +354,11 @@ __global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const
       float d = 0.f;
       for (int i = lane; i < p.dim; i += 32) d = fmaf(sq[m * p.dim + i], pi_to_f32(kt[m * DP + i]), d);
       const float s = pi_warp_sum(d) * p.scale - slope * (float)(pos - t);
+      if (by_itself) {
+        const float w = pi_sigmoid(s + self_bias);
+        for (int i = lane; i < p.vdim; i += 32) my[i] = fmaf(w, pi_to_f32(vt[i]), my[i]);
+        continue;
+      }
       const float mn = fmaxf(mx[m], s), keep = expf(mx[m] - mn), w = expf(s - mn);
       mx[m] = mn;
       l[m] = l[m] * keep + w;
@@ -235,7 +377,7 @@ __global__ void __launch_bounds__(kPlainWarps * 32) maps_attn_plain_kernel(const
     for (int w = 0; w < kPlainWarps; ++w) M = fmaxf(M, s_m[w][m]);
     if (p.sinks) L = expf(sink - M);
     for (int w = 0; w < kPlainWarps; ++w) L += s_m[w][m] == -INFINITY ? 0.f : s_l[w][m] * expf(s_m[w][m] - M);
-    for (int w = 0; w < kPlainWarps; ++w) f[m][w] = s_m[w][m] == -INFINITY ? 0.f : expf(s_m[w][m] - M) / L;
+    for (int w = 0; w < kPlainWarps; ++w) f[m][w] = by_itself ? 1.f : s_m[w][m] == -INFINITY ? 0.f : expf(s_m[w][m] - M) / L;
   }
   float sq_sum = 0.f;
   for (int e = tid; e < p.vdim; e += blockDim.x) {
@@ -269,6 +411,14 @@ pi_status pi_launch_maps_prepare(pi_ctx* ctx, const pi_maps_attention& a, const 
                      kv.block_size, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks, a.eps, x};
   const int vectors = (a.heads + a.kv_heads) * a.maps + a.kv_heads;
   const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.dim <= 256 && a.vdim <= 256 && stride % 4 == 0 && x.mix.stride % 4 == 0;
+  if (x.norm_qk) {
+    PI_REQUIRE(ctx, a.maps == 1 && !x.bias && !x.unit_qk && !x.q_temp && !x.mix.first, "norms over whole projections stand alone");
+    auto k = kv.kind == PI_BF16 ? (vec ? maps_prepare_whole_kernel<__nv_bfloat16, true> : maps_prepare_whole_kernel<__nv_bfloat16, false>)
+                                : (vec ? maps_prepare_whole_kernel<float, true> : maps_prepare_whole_kernel<float, false>);
+    PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(b.rows), dim3(kWholeThreads), 0, 1, p));
+    return PI_OK;
+  }
+  PI_REQUIRE(ctx, !x.q_only, "keys of another layer go with norms over whole projections");
   void (*k)(const PrepareParams);
   if (kv.kind == PI_BF16) k = vec ? maps_prepare_kernel<__nv_bfloat16, true> : maps_prepare_kernel<__nv_bfloat16, false>;
   else k = vec ? maps_prepare_kernel<float, true> : maps_prepare_kernel<float, false>;
@@ -281,7 +431,8 @@ pi_status pi_launch_maps_attention(pi_ctx* ctx, const pi_maps_attention& a, cons
   pi_prof_scope prof(ctx, PI_PROF_ATTENTION);
   MapsParams p = {qkv, stride, out, out_stride, kv.base, a.heads, a.kv_heads, a.maps, a.dim, a.vdim, kv.dp, kv.vp, kv.block_size,
                   a.window, a.scale, a.eps, a.lambda, a.out_scale, b.row_seq, b.row_pos, b.lens, b.tables, b.max_blocks, a.gate, a.gate_stride, a.gate_per_head,
-                  a.slopes, a.sinks, a.v_in_k};
+                  a.slopes, a.sinks, a.sigmoid_bias, a.v_in_k};
+  PI_REQUIRE(ctx, !a.sigmoid_bias || (a.maps == 1 && !a.slopes && !a.sinks), "keys that weigh by themselves go with one map and plain scores");
   if (pi_maps_attention_tc_usable(ctx, a, kv)) return pi_launch_maps_attention_tc(ctx, p, out_kind, b);
   const size_t smem = sizeof(float) * ((size_t)a.maps * a.dim + (size_t)kPlainWarps * a.maps * a.vdim);
   PI_REQUIRE(ctx, smem <= kSmemFit, "attention heads of %d / %d channels are too wide", a.dim, a.vdim);

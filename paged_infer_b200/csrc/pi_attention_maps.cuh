@@ -16,7 +16,7 @@ struct MapsParams {
   const float* gate;
   size_t gate_stride;
   int gate_per_head;
-  const float *slopes, *sinks;
+  const float *slopes, *sinks, *sigmoid_bias;
   int v_in_k;
 };
 

@@ -71,9 +71,13 @@ __device__ __forceinline__ float new_max(float m, float s_max, float& keep) {
   return n;
 }
 
+// Weight of a key that weighs by itself: sigmoid of a score in the log2 domain (0 for one of minus infinity).
+__device__ __forceinline__ float self_weight(float s) { return __fdividef(1.f, 1.f + exp2f(-s)); }
+
 constexpr int kDecWarps = 4, kDecStages = 3, kMaxSplits = 8;   // splits: a portable cluster
 
-template <int MAPS, int KMAX, int VMAX>
+// SELF: sigmoid weights, which need neither maximum nor sum - the merges then just add.
+template <int MAPS, int KMAX, int VMAX, bool SELF = false>
 __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcParams p) {
   constexpr int QR = MAPS == 2 ? 2 : 4;     // query registers per 16 channels
   constexpr int HR = 16 / MAPS;             // heads per MMA
@@ -194,6 +198,15 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
 #pragma unroll
     for (int h = 0; h < 2; ++h) slope[h] = __ldg(a.slopes + g * p.group + min(grp * HR + ((lane >> 2) + 8 * h) % HR, p.group - 1)) * kLog2e;
   }
+  float self[2] = {0.f, 0.f};
+  if (SELF) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      self[h] = __ldg(a.sigmoid_bias + g * p.group + min(grp * HR + ((lane >> 2) + 8 * h) % HR, p.group - 1)) * kLog2e;
+      mx[h] = 0.f;                          // warps and splits merge with factors of 1
+      l[h] = 1.f;
+    }
+  }
 
   int stage = 0;
   for (int tile = tile0; tile < tile_end; tile += kDecWarps) {
@@ -228,21 +241,30 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int t = key + 8 * j + (i & 1);
-        s[j][i] = (t >= lo && t < hi) ? fmaf(slope[i >> 1], (float)(t - pos), s[j][i] * sc) : -INFINITY;
+        const float v = SELF ? fmaf(s[j][i], sc, self[i >> 1]) : fmaf(slope[i >> 1], (float)(t - pos), s[j][i] * sc);
+        s[j][i] = (t >= lo && t < hi) ? v : -INFINITY;
       }
     uint32_t ph[4], pl[4];
     float keep[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {   // MMA rows lane / 4 and lane / 4 + 8
-      const float tm = quad_max(fmaxf(fmaxf(s[0][2 * h], s[0][2 * h + 1]), fmaxf(s[1][2 * h], s[1][2 * h + 1])));
-      mx[h] = new_max(mx[h], tm, keep[h]);
-      const float ref = mx[h] == -INFINITY ? 0.f : mx[h];
       float w[4];
+      if (SELF) {
+        keep[h] = 1.f;
 #pragma unroll
-      for (int j = 0; j < 2; ++j)
+        for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int i = 0; i < 2; ++i) w[2 * j + i] = exp2f(s[j][2 * h + i] - ref);
-      l[h] = l[h] * keep[h] + ((w[0] + w[1]) + (w[2] + w[3]));
+          for (int i = 0; i < 2; ++i) w[2 * j + i] = self_weight(s[j][2 * h + i]);
+      } else {
+        const float tm = quad_max(fmaxf(fmaxf(s[0][2 * h], s[0][2 * h + 1]), fmaxf(s[1][2 * h], s[1][2 * h + 1])));
+        mx[h] = new_max(mx[h], tm, keep[h]);
+        const float ref = mx[h] == -INFINITY ? 0.f : mx[h];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int i = 0; i < 2; ++i) w[2 * j + i] = exp2f(s[j][2 * h + i] - ref);
+        l[h] = l[h] * keep[h] + ((w[0] + w[1]) + (w[2] + w[3]));
+      }
       split(w[0], w[1], ph[h], pl[h]);
       split(w[2], w[3], ph[2 + h], pl[2 + h]);
     }
@@ -254,10 +276,12 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
           float* d = acc[j + h];
-          d[0] *= keep[0];
-          d[1] *= keep[0];
-          d[2] *= keep[1];
-          d[3] *= keep[1];
+          if (!SELF) {
+            d[0] *= keep[0];
+            d[1] *= keep[0];
+            d[2] *= keep[1];
+            d[3] *= keep[1];
+          }
           mma(d, ph[0], ph[1], ph[2], ph[3], b[2 * h], b[2 * h + 1]);
           mma(d, pl[0], pl[1], pl[2], pl[3], b[2 * h], b[2 * h + 1]);
         }
@@ -358,7 +382,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
           f[m][c] = c >= p.nsplit || f[m][c] == -INFINITY ? 0.f : exp2f(f[m][c] - M);
           L = fmaf(l[m][c], f[m][c], L);
         }
-        const float inv = L > 0.f ? (m == 0 ? 1.f : -a.lambda) / L : 0.f;
+        const float inv = SELF ? 1.f : L > 0.f ? (m == 0 ? 1.f : -a.lambda) / L : 0.f;
 #pragma unroll
         for (int c = 0; c < NS; ++c) f[m][c] *= inv;
       }
@@ -396,7 +420,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) maps_decode_kernel(const TcPar
 
 constexpr int kTileWarps = 8, kTileKeys = 64;
 
-template <int MAPS, int KMAP, int VMAX>
+template <int MAPS, int KMAP, int VMAX, bool SELF = false>
 __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcParams p) {
   constexpr int RG = kTileWarps / MAPS, R = RG * 16;     // row groups of 16 rows
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -485,12 +509,13 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
     for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
   float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const float sc = a.scale * kLog2e;
-  float slope[2], sink[2];
+  float slope[2], sink[2], self[2] = {0.f, 0.f};
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const int head = g * p.group + (rg * 16 + (lane >> 2) + 8 * h) % p.group;
     slope[h] = a.slopes ? __ldg(a.slopes + head) * kLog2e : 0.f;
     sink[h] = a.sinks ? __ldg(a.sinks + head) * kLog2e : -INFINITY;
+    if (SELF) self[h] = __ldg(a.sigmoid_bias + head) * kLog2e;
   }
   const int win = a.window > 0 ? a.window : 0x3fffffff;
 
@@ -519,7 +544,16 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
       }
     const int t0 = lo + kb * kTileKeys;
     const bool inside = n_tok == per_tile && t0 + kTileKeys - 1 <= p_first && t0 > p_last - win && R == per_tile * p.group;
-    float keep[2], ref[2];
+    float keep[2] = {1.f, 1.f}, ref[2] = {0.f, 0.f};
+    if (SELF) {
+#pragma unroll
+      for (int j = 0; j < kTileKeys / 8; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int t = t0 + j * 8 + (lane & 3) * 2 + (i & 1), q = tpos[i >> 1];
+          s[j][i] = (inside || (t <= q && t > q - win && t < hi)) ? self_weight(fmaf(s[j][i], sc, self[i >> 1])) : 0.f;
+        }
+    } else {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       float tm = -INFINITY;
@@ -536,7 +570,8 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
       ref[h] = mx[h] == -INFINITY ? 0.f : mx[h];
       l[h] *= keep[h];
     }
-    if (__any_sync(0xffffffffu, keep[0] != 1.f || keep[1] != 1.f)) {
+    }
+    if (!SELF && __any_sync(0xffffffffu, keep[0] != 1.f || keep[1] != 1.f)) {
 #pragma unroll
       for (int j = 0; j < VMAX / 8; ++j) {
         acc[j][0] *= keep[0];
@@ -552,8 +587,9 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
       for (int h = 0; h < 2; ++h)
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
-          const float w0 = exp2f(s[2 * c + j][2 * h] - ref[h]), w1 = exp2f(s[2 * c + j][2 * h + 1] - ref[h]);
-          l[h] += w0 + w1;
+          const float s0 = s[2 * c + j][2 * h], s1 = s[2 * c + j][2 * h + 1];
+          const float w0 = SELF ? s0 : exp2f(s0 - ref[h]), w1 = SELF ? s1 : exp2f(s1 - ref[h]);
+          if (!SELF) l[h] += w0 + w1;
           split(w0, w1, ph[2 * j + h], pl[2 * j + h]);
         }
 #pragma unroll
@@ -575,7 +611,7 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
   for (int h = 0; h < 2; ++h) {
     const float M = fmaxf(mx[h], sink[h]), f = mx[h] == -INFINITY ? 0.f : exp2f(mx[h] - M);   // the sink joins in
     const float t = quad_sum(l[h]) * f + (a.sinks ? exp2f(sink[h] - M) : 0.f);
-    inv[h] = t > 0.f ? f / t : 0.f;
+    inv[h] = SELF ? 1.f : t > 0.f ? f / t : 0.f;
   }
   float ss[2] = {0.f, 0.f};
   const int apitch = a.vp + 8, r0 = rg * 16 + (lane >> 2);
@@ -652,23 +688,23 @@ size_t tile_smem(const MapsParams& a) {
 
 typedef void (*TcKernel)(const TcParams);
 
-template <int MAPS, int VMAX>
+template <int MAPS, int VMAX, bool SELF>
 TcKernel pick_decode(int k) {
-  return k <= 8 ? maps_decode_kernel<MAPS, 8, VMAX> : maps_decode_kernel<MAPS, 16, VMAX>;
+  return k <= 8 ? maps_decode_kernel<MAPS, 8, VMAX, SELF> : maps_decode_kernel<MAPS, 16, VMAX, SELF>;
 }
-template <int MAPS>
+template <int MAPS, bool SELF = false>
 TcKernel pick_decode(int k, int vp) {
-  return vp <= 64 ? pick_decode<MAPS, 64>(k) : vp <= 128 ? pick_decode<MAPS, 128>(k) : pick_decode<MAPS, 256>(k);
+  return vp <= 64 ? pick_decode<MAPS, 64, SELF>(k) : vp <= 128 ? pick_decode<MAPS, 128, SELF>(k) : pick_decode<MAPS, 256, SELF>(k);
 }
-template <int MAPS, int VMAX>
+template <int MAPS, int VMAX, bool SELF>
 TcKernel pick_tile(int k) {
   if constexpr (MAPS == 1)   // one map may have wider keys
-    if (k > 8) return k <= 12 ? maps_tile_kernel<1, 12, VMAX> : maps_tile_kernel<1, 16, VMAX>;
-  return k <= 4 ? maps_tile_kernel<MAPS, 4, VMAX> : maps_tile_kernel<MAPS, 8, VMAX>;
+    if (k > 8) return k <= 12 ? maps_tile_kernel<1, 12, VMAX, SELF> : maps_tile_kernel<1, 16, VMAX, SELF>;
+  return k <= 4 ? maps_tile_kernel<MAPS, 4, VMAX, SELF> : maps_tile_kernel<MAPS, 8, VMAX, SELF>;
 }
-template <int MAPS>
+template <int MAPS, bool SELF = false>
 TcKernel pick_tile(int k, int vp) {
-  return vp <= 64 ? pick_tile<MAPS, 64>(k) : vp <= 128 ? pick_tile<MAPS, 128>(k) : pick_tile<MAPS, 256>(k);
+  return vp <= 64 ? pick_tile<MAPS, 64, SELF>(k) : vp <= 128 ? pick_tile<MAPS, 128, SELF>(k) : pick_tile<MAPS, 256, SELF>(k);
 }
 
 // The shared-memory limit of a kernel is raised once per device.
@@ -703,7 +739,7 @@ pi_status pi_launch_maps_attention_tc(pi_ctx* ctx, const MapsParams& a, int out_
   p.seq_start = b.seq_start;
   if (b.n_portions > 0) {
     const int per_tile = 16 * kTileWarps / a.maps / p.group, tiles = (b.max_portion + per_tile - 1) / per_tile;
-    const TcKernel k = a.maps == 2 ? pick_tile<2>(a.dp / 16, a.vp) : pick_tile<1>(a.dp / 16, a.vp);
+    const TcKernel k = a.maps == 2 ? pick_tile<2>(a.dp / 16, a.vp) : a.sigmoid_bias ? pick_tile<1, true>(a.dp / 16, a.vp) : pick_tile<1>(a.dp / 16, a.vp);
     const size_t smem = tile_smem(a);
     PI_CUDA(ctx, grant(ctx, k, smem));
     PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(tiles, a.kv_heads, b.n_portions), dim3(kTileWarps * 32), smem, 1, p));
@@ -712,7 +748,7 @@ pi_status pi_launch_maps_attention_tc(pi_ctx* ctx, const MapsParams& a, int out_
     const int hr = 16 / a.maps;
     p.ngroups = (p.group + hr - 1) / hr;
     // KV splits: one round of CTAs over the GPU, at least one 16-key tile per warp
-    const TcKernel k = a.maps == 2 ? pick_decode<2>(2 * a.dp / 16, a.vp) : pick_decode<1>(a.dp / 16, a.vp);
+    const TcKernel k = a.maps == 2 ? pick_decode<2>(2 * a.dp / 16, a.vp) : a.sigmoid_bias ? pick_decode<1, true>(a.dp / 16, a.vp) : pick_decode<1>(a.dp / 16, a.vp);
     const size_t smem = decode_smem(a);
     PI_CUDA(ctx, grant(ctx, k, smem));
     const int keys = a.window > 0 ? std::min(a.window, b.max_pos + 1) : b.max_pos + 1;

@@ -155,7 +155,8 @@ enum pi_epilogue {
   PI_EPI_DYT_RESIDUAL = 4,  // x[m][r] += dyt(post, v); h[m][r] = dyt(next, x[m][r])   (pi_dyt_residual)
   PI_EPI_CLAMP_GLU = 6,     // rows interleaved gate/up: g = min(gate, limit), u = clamp(up, +-limit): g sigmoid(1.702 g) (u + 1)
   PI_EPI_SCALE_ADD = 7,     // out[m][r] += out_scale[r] v        (residual add with a layer scale)
-  PI_EPI_GELU_TABLE = 8     // out[m][r] = gelu_tanh(v) table[token of m][r]   (pi_token_table)
+  PI_EPI_GELU_TABLE = 8,    // out[m][r] = gelu_tanh(v) table[token of m][r]   (pi_token_table)
+  PI_EPI_RELU2 = 9          // out[m][r] = max(v, 0)^2
 };
 inline bool pi_epi_glu(pi_epilogue e) { return e == PI_EPI_SWIGLU || e == PI_EPI_GEGLU || e == PI_EPI_CLAMP_GLU; }
 

@@ -165,6 +165,12 @@ __device__ __forceinline__ void epilogue(const Bf16GemmParams& p, int M, int n, 
 #pragma unroll
     for (int j = 0; j < C; ++j)
       if (ok && m + j * dm < M) p.out_bf16[(size_t)(m + j * dm) * p.out_stride + n] = __float2bfloat16_rn(pi_gelu_tanh(v[j]) * e[j]);
+  } else if (p.epi == PI_EPI_RELU2) {
+#pragma unroll
+    for (int j = 0; j < C; ++j) {
+      const float r = fmaxf(v[j], 0.f);
+      if (ok && m + j * dm < M) p.out_bf16[(size_t)(m + j * dm) * p.out_stride + n] = __float2bfloat16_rn(r * r);
+    }
   } else if (p.out_bf16) {
 #pragma unroll
     for (int j = 0; j < C; ++j)
@@ -473,6 +479,7 @@ pi_status pi_launch_gemm_bf16(pi_ctx* ctx, const pi_linear* lin, const pi_linear
   const bool glu = pi_epi_glu(a.epi) && a.out_bf16 && (a.glu_rows ? a.glu_rows % 2 == 0 && a.glu_rows <= N && a.rest : N % 2 == 0);
   PI_REQUIRE(ctx, a.epi == PI_EPI_STORE || glu || (a.epi == PI_EPI_MAPS_QKV && a.maps_kv && a.maps_kv->dim % 2 == 0) ||
                       (a.epi == PI_EPI_SCALE_ADD && a.out && a.out_scale) || (a.epi == PI_EPI_GELU_TABLE && a.out_bf16 && a.table.base && a.table.tokens) ||
+                      (a.epi == PI_EPI_RELU2 && a.out_bf16) ||
                       (a.epi == PI_EPI_DYT_RESIDUAL && a.residual && a.residual->x && a.residual->h && a.residual->post.w && a.residual->next.w),
              "this epilogue is not built for the bf16 GEMM");
   Bf16GemmParams p = {};

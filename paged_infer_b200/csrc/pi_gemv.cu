@@ -518,7 +518,8 @@ __global__ void __launch_bounds__(256) gemv_kernel(const GemvParams p) {
             if (lane == r * MB + m && m < mcount && row0 + r < p.N) {
               float* o = p.out + (size_t)(m0 + m) * p.out_stride + row0 + r;
               const float v = tot[r][m] * sc[r] * row_factor(m);
-              if (EPI == PI_EPI_GELU_TABLE) *o = pi_gelu_tanh(v) * pi_table_value(p.table, m0 + m, row0 + r);
+              if (EPI == PI_EPI_RELU2) *o = fmaxf(v, 0.f) * fmaxf(v, 0.f);
+              else if (EPI == PI_EPI_GELU_TABLE) *o = pi_gelu_tanh(v) * pi_table_value(p.table, m0 + m, row0 + r);
               else *o = EPI == PI_EPI_ADD ? old_out + v : EPI == PI_EPI_SCALE_ADD ? fmaf(__ldg(p.out_scale + row0 + r), v, old_out) : v;
             }
           }
@@ -544,6 +545,7 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
     if constexpr (kFloatW && MB == 1) {
       if (epi == PI_EPI_CLAMP_GLU) k = gemv_kernel<WT, 1, PI_EPI_CLAMP_GLU, false, false, 1, true>;
       else if (epi == PI_EPI_SWIGLU) k = gemv_kernel<WT, 1, PI_EPI_SWIGLU, false, false, 1, true>;
+      else if (epi == PI_EPI_RELU2) k = gemv_kernel<WT, 1, PI_EPI_RELU2, false, false, 1, true>;
       else if (epi == PI_EPI_STORE) k = gemv_kernel<WT, 1, PI_EPI_STORE, false, false, 1, true>;
     }
   } else if (ksplit == kSplitWarps) {   // few long rows (pi_launch_gemv asks for it only without norm, rotary embedding, SwiGLU)
@@ -602,7 +604,7 @@ cudaError_t launch_gemv_t(pi_ctx* ctx, const GemvParams& p, int epi, bool norm, 
       }
       if constexpr (MB == 1) {
         for (auto kk : {gemv_kernel<WT, 1, PI_EPI_CLAMP_GLU, false, false, 1, true>, gemv_kernel<WT, 1, PI_EPI_SWIGLU, false, false, 1, true>,
-                        gemv_kernel<WT, 1, PI_EPI_STORE, false, false, 1, true>}) {
+                        gemv_kernel<WT, 1, PI_EPI_RELU2, false, false, 1, true>, gemv_kernel<WT, 1, PI_EPI_STORE, false, false, 1, true>}) {
           cudaError_t e = cudaFuncSetAttribute(kk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
           if (e != cudaSuccess) return e;
         }
@@ -694,6 +696,7 @@ pi_status pi_launch_gemv(pi_ctx* ctx, const pi_linear* lin, const pi_linear_args
              "a gated epilogue needs interleaved gate/up rows");
   PI_REQUIRE(ctx, !a.experts || (lin->kind != PI_INT8 && a.experts->expert && lin->rows % a.experts->experts == 0 && a.experts->x_div >= 1),
              "a stack of experts needs float weights and the rows' experts");
+  PI_REQUIRE(ctx, a.epi != PI_EPI_RELU2 || a.experts, "this epilogue is built for stacks of experts");
   PI_REQUIRE(ctx, a.epi != PI_EPI_SCALE_ADD || a.out_scale, "a scaled residual add needs its scale");
   PI_REQUIRE(ctx, a.epi != PI_EPI_GELU_TABLE || (a.table.base && a.table.tokens), "this epilogue needs its table");
   PI_REQUIRE(ctx, a.epi < PI_EPI_GEGLU || (lin->kind != PI_INT8 && !a.norm_weight), "this epilogue is built for bf16 and f32 weights");

@@ -1,12 +1,16 @@
 // Layered designs: a decoder whose layers each name a token mixer - windowed attention with one or two softmax maps, latent
-// attention, a gated linear recurrence (GLA), a matrix memory (mLSTM), a state-space recurrence (SSD), lightning attention - and,
-// if they have one, a feed-forward: dense and gated, or routed experts.  Three ways of normalising:
+// attention, a gated linear recurrence (GLA), a matrix memory (mLSTM), a state-space recurrence (SSD), lightning attention, a
+// gated recurrence of single channels (minGRU) - and, if they have one, a feed-forward: dense and gated, or routed experts.  Four
+// ways of normalising:
 //
 //   Dynamic Tanh   x += dyt(norm1b, mixer(dyt(norm1, x)));    x += dyt(norm2b, ff(dyt(norm2, x)))
 //   layer norm     x += ls1 mixer(ln(norm1, x));              x += ls2 ff(ln(norm2, x))
 //   RMS norm       x += mu rms(norm1b, mixer(rms(norm1, x))); x += mu rms(norm2b, ff(rms(norm2, x)));
 //                  x += mu rms(side, proj(gelu(gate x) * e)), e: the layer's part of the token's row of a table
+//   norm of the sum  x = rms(norm1, keep x + g1 mixer(x));   x = rms(norm2, keep x + g2 ff(x)),  g = sigmoid(rg x + b) per channel
 //
+// A norm of the sum leaves nothing between x and the next sublayer's input; the rows of a sublayer gate ride behind those of the
+// projection that reads the same input, and the row kernel applies it.
 // With RMS norms the projection that ends a sublayer stores its result, and the row kernel behind it normalises that, adds it to
 // the residual stream and writes the next sublayer's input, all with the row in registers.
 // Layer norm needs the whole row: the projection that ends a sublayer adds its scaled result to the residual stream, and a
@@ -54,6 +58,9 @@ struct Layer {
   const float *bias = nullptr, *slopes = nullptr, *sinks = nullptr;   // attention: see pi_maps_attention, pi_maps_prepare
   int col_gate = -1;                                       // column of the gate per head
   int temp = -1;                                           // index of its table of query factors
+  const float *qk_norm = nullptr, *sigmoid_bias = nullptr;
+  const float *gate1_b = nullptr, *gate2_b = nullptr;      // sublayer gates: biases and columns (of the mixer's projection, of `route`)
+  int col_gate1 = 0, col_router = 0;
   float v_lambda = 0.f;
   bool v_first = false;
   const float *ls1 = nullptr, *ls2 = nullptr;
@@ -61,17 +68,19 @@ struct Layer {
   pi_linear *in = nullptr, *out = nullptr, *gate_up = nullptr, *down = nullptr;
   pi_linear *expert_in = nullptr, *expert_out = nullptr;   // stacks of all experts
   pi_linear *ukv = nullptr, *uk_t = nullptr;               // latent attention
-  int attn = -1;                 // index of the layer's KV region
+  int attn = -1;                 // index of the KV region it reads, its own or another layer's
   int rope = -1;                 // index of its rotary table
   float lambda = 0.f;
   pi_recurrence rec;
   pi_latent_attention lat;
   pi_ssd ssd;
+  pi_mingru gru;
   pi_moe moe;
 };
 
 struct RopeTable {
   int dims = 0, cap = 0;
+  bool banded = false;
   double base = 1., factor = 1., original = 1., fast = 1., slow = 1.;
   float *cos = nullptr, *sin = nullptr;
 };
@@ -84,10 +93,18 @@ struct TempTable {               // what queries are multiplied by, per position
 
 // Angle per position of every pair, and the factor of cos and sin.  With a factor above 1, pairs that turn less than `slow`
 // times within `original` positions are slowed by it, pairs that turn more than `fast` times are left alone, with a linear
-// ramp over the pair index in between.
+// ramp over the pair index in between.  Banded: the ramp runs over the number of turns, and cos and sin do not grow.
 double rope_frequencies(const RopeTable& t, std::vector<double>* f) {
   f->resize(t.dims / 2);
   const bool stretched = t.factor != 1.0;
+  if (stretched && t.banded) {
+    for (int i = 0; i < t.dims / 2; ++i) {
+      const double plain = pow(t.base, -2.0 * i / t.dims), turns = t.original * plain / (2.0 * M_PI);
+      const double s = turns > t.fast ? 1.0 : turns < t.slow ? 0.0 : t.fast > t.slow ? (turns - t.slow) / (t.fast - t.slow) : 1.0;
+      (*f)[i] = (1.0 - s) * plain / t.factor + s * plain;
+    }
+    return 1.0;
+  }
   auto turns = [&](double n) { return t.dims * log(t.original / (2.0 * M_PI * n)) / (2.0 * log(t.base)); };
   const double lo = stretched ? std::max(floor(turns(t.fast)), 0.0) : 0.0, hi = stretched ? std::min(ceil(turns(t.slow)), t.dims - 1.0) : 0.0;
   for (int i = 0; i < t.dims / 2; ++i) {
@@ -108,6 +125,8 @@ struct pi_layered {
   std::vector<void*> owned;      // device vectors
   pi_linear *embed = nullptr, *head = nullptr;   // head: null if tied
   pi_linear* side_embed = nullptr;
+  pi_linear* pairs = nullptr;    // table of token pairs
+  int regions = 0;               // of the KV pool
   size_t mix_stride = 0;         // values of a row that are mixed between layers
   pi_dyt final_norm;
   pi_layer_norm final_ln;        // its weight carries the logits' scale
@@ -308,7 +327,7 @@ struct Loader {
 };
 
 pi_status check_layer(pi_ctx* ctx, int i, const pi_layer_config& c) {
-  PI_REQUIRE(ctx, c.mixer >= PI_MIXER_ATTENTION && c.mixer <= PI_MIXER_LIGHTNING, "layer %d: unknown mixer %d", i, c.mixer);
+  PI_REQUIRE(ctx, c.mixer >= PI_MIXER_ATTENTION && c.mixer <= PI_MIXER_MINGRU, "layer %d: unknown mixer %d", i, c.mixer);
   PI_REQUIRE(ctx, c.heads > 0 && c.dim > 0 && c.vdim > 0 && c.ff >= 0, "layer %d: sizes must be positive", i);
   if (c.mixer == PI_MIXER_ATTENTION) {
     PI_REQUIRE(ctx, c.kv_heads > 0 && c.heads % c.kv_heads == 0, "layer %d: %d heads do not share %d key/value heads", i, c.heads, c.kv_heads);
@@ -316,6 +335,12 @@ pi_status check_layer(pi_ctx* ctx, int i, const pi_layer_config& c) {
     PI_REQUIRE(ctx, c.rot_dims <= c.dim, "layer %d: %d rotary channels of %d", i, c.rot_dims, c.dim);
     PI_REQUIRE(ctx, c.maps == 1 || !(c.distance_bias || c.sink || c.head_gate), "layer %d: distance bias, sink and head gate belong to one softmax map", i);
     PI_REQUIRE(ctx, c.q_temp_every >= 0., "layer %d: queries grow every %g tokens", i, c.q_temp_every);
+    PI_REQUIRE(ctx, !c.norm_qk || (c.maps == 1 && !c.biases && !c.unit_qk && !c.v_mix && c.q_temp_every == 0.),
+               "layer %d: norms over whole projections go with nothing else between projection and rotation", i);
+    PI_REQUIRE(ctx, !c.sigmoid_weights || (c.maps == 1 && !c.distance_bias && !c.sink), "layer %d: sigmoid weights go with one map and plain scores", i);
+    PI_REQUIRE(ctx, c.kv_from == 0 || c.norm_qk, "layer %d: keys of another layer go with norms over whole projections", i);
+  } else if (c.mixer == PI_MIXER_MINGRU) {
+    PI_REQUIRE(ctx, c.heads == 1, "layer %d: this recurrence has one head", i);
   } else if (c.mixer == PI_MIXER_LATENT) {
     PI_REQUIRE(ctx, c.rank > 0, "layer %d: the latent needs channels", i);
   } else if (c.mixer == PI_MIXER_GLA) {
@@ -345,8 +370,9 @@ pi_status check_layer(pi_ctx* ctx, int i, const pi_layer_config& c) {
       PI_REQUIRE(ctx, c.keep_groups >= 1 && c.keep_groups <= c.expert_groups, "layer %d: %d groups of %d are kept", i, c.keep_groups, c.expert_groups);
       PI_REQUIRE(ctx, c.top >= 1 && c.top <= c.experts / c.expert_groups * c.keep_groups, "layer %d: %d experts per token", i, c.top);
       PI_REQUIRE(ctx, c.shared_ff >= 0, "layer %d: sizes must be positive", i);
-      PI_REQUIRE(ctx, (c.unit == PI_UNIT_CLAMPED || c.unit == PI_UNIT_SILU) && (c.score == PI_SCORE_SIGMOID || c.score == PI_SCORE_SOFTMAX) &&
+      PI_REQUIRE(ctx, c.unit >= PI_UNIT_CLAMPED && c.unit <= PI_UNIT_RELU2 && c.score >= PI_SCORE_SIGMOID && c.score <= PI_SCORE_CHOSEN &&
                           (c.group_best == 1 || c.group_best == 2), "layer %d: unknown kind of experts", i);
+      PI_REQUIRE(ctx, c.unit != PI_UNIT_RELU2 || c.shared_ff == 0, "layer %d: a shared expert has gated units", i);
     }
   }
   return PI_OK;
@@ -357,6 +383,7 @@ struct Extents {
   size_t in = 0, core = 1, ff = 1, lat_q = 0, lat_o = 0, inner = 0, route = 0, act = 0, top = 0, experts = 0;
   bool chunk = true;
   int attn = 0;
+  std::vector<int> own;            // per layer: its KV region, -1: it has none of its own
 };
 
 int add_rope(pi_layered* m, const pi_layer_config& c) {
@@ -368,10 +395,11 @@ int add_rope(pi_layered* m, const pi_layer_config& c) {
     t.original = c.rot_original;
     t.fast = c.rot_fast;
     t.slow = c.rot_slow;
+    t.banded = c.rot_banded != 0;
   }
   for (size_t i = 0; i < m->ropes.size(); ++i) {
     const RopeTable& o = m->ropes[i];
-    if (o.dims == t.dims && o.base == t.base && o.factor == t.factor && o.original == t.original && o.fast == t.fast && o.slow == t.slow) return (int)i;
+    if (o.dims == t.dims && o.banded == t.banded && o.base == t.base && o.factor == t.factor && o.original == t.original && o.fast == t.fast && o.slow == t.slow) return (int)i;
   }
   m->ropes.push_back(t);
   return (int)m->ropes.size() - 1;
@@ -402,6 +430,14 @@ pi_status build_attention_options(pi_ctx* ctx, Loader& ld, int i, const std::str
     PI_TRY(ld.upload(all, &L.bias));
   }
   if (c.sink) PI_TRY(ld.dev_vec(mix + "sink", c.heads, &L.sinks));
+  if (c.sigmoid_weights) PI_TRY(ld.dev_vec(mix + "pb", c.heads, &L.sigmoid_bias, -3.f));
+  if (c.norm_qk) {
+    std::vector<float> q, k;
+    PI_TRY(ld.vec(mix + "q.norm", nq, &q, 1.f));
+    if (c.kv_from == 0) PI_TRY(ld.vec(mix + "k.norm", nk, &k, 1.f));
+    q.insert(q.end(), k.begin(), k.end());
+    PI_TRY(ld.upload(q, &L.qk_norm));
+  }
   if (c.distance_bias) {
     std::vector<float> s(c.heads);
     for (int h = 0; h < c.heads; ++h) s[h] = (float)exp2(-8.0 * (h + 1) / c.heads);
@@ -435,14 +471,22 @@ pi_status build_mixer(pi_ctx* ctx, Loader& ld, int i, int gla_rank, Layer& L, Ex
   };
   if (c.mixer == PI_MIXER_ATTENTION) {
     PI_TRY(add("q", (size_t)c.heads * c.maps * c.dim));
-    PI_TRY(add("k", (size_t)c.kv_heads * c.maps * c.dim));
-    PI_TRY(add("v", (size_t)c.kv_heads * c.vdim));
+    if (c.kv_from > 0) {
+      const int j = c.kv_from - 1;
+      PI_REQUIRE(ctx, j < i && x.own[j] >= 0 && m->layers[j].c.mixer == PI_MIXER_ATTENTION, "layer %d: layer %d has no keys and values to share", i, j);
+      const pi_layer_config& o = m->layers[j].c;
+      PI_REQUIRE(ctx, o.kv_heads == c.kv_heads && o.maps == c.maps && o.dim == c.dim && o.vdim == c.vdim, "layer %d: its heads differ from those of layer %d", i, j);
+      L.attn = x.own[j];
+    } else {
+      PI_TRY(add("k", (size_t)c.kv_heads * c.maps * c.dim));
+      PI_TRY(add("v", (size_t)c.kv_heads * c.vdim));
+      L.attn = x.own[i] = x.attn++;
+    }
     PI_TRY(build_attention_options(ctx, ld, i, mix, L));
     if (c.head_gate) {
       L.col_gate = (int)rows;
       PI_TRY(add("g", c.heads));
     }
-    L.attn = x.attn++;
     if (c.maps == 2) {   // lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, one number for the layer
       double e[2];
       for (int j = 0; j < 2; ++j) {
@@ -480,7 +524,7 @@ pi_status build_mixer(pi_ctx* ctx, Loader& ld, int i, int gla_rank, Layer& L, Ex
     a.ukv = L.ukv;
     a.uk_t = L.uk_t;
     PI_REQUIRE(ctx, pi_latent_supported(ctx, a, m->c.compute), "layer %d: a latent of %d + %d channels is not supported", i, c.rank, c.rot_dims);
-    L.attn = x.attn++;
+    L.attn = x.own[i] = x.attn++;
     L.rope = add_rope(m, c);
     if (!m->latent) {
       m->expand = true;
@@ -547,6 +591,18 @@ pi_status build_mixer(pi_ctx* ctx, Loader& ld, int i, int gla_rank, Layer& L, Ex
     m->state_floats += r.state_floats();
     x.inner = std::max(x.inner, core);
     x.chunk = x.chunk && pi_ssd_chunked(ctx, r, m->c.compute);
+  } else if (c.mixer == PI_MIXER_MINGRU) {
+    pi_mingru& r = L.gru;
+    r.width = c.vdim;
+    r.col_x = c.vdim;
+    r.col_g = 2 * c.vdim;
+    PI_TRY(add("z", core));
+    PI_TRY(add("x", core));
+    PI_TRY(add("g", core));
+    PI_TRY(ld.dev_vec(mix + "z.b", core, &r.z_bias));
+    PI_TRY(ld.dev_vec(mix + "x.b", core, &r.x_bias));
+    r.state_off = m->state_floats;
+    m->state_floats += r.state_floats();
   } else {
     pi_recurrence& r = L.rec;
     const size_t hd = (size_t)c.heads * c.dim;
@@ -593,6 +649,13 @@ pi_status build_mixer(pi_ctx* ctx, Loader& ld, int i, int gla_rank, Layer& L, Ex
     m->state_floats += pi_recurrence_floats(r.kind, c.heads, c.dim, c.vdim);
     x.chunk = x.chunk && pi_recurrence_chunked(ctx, r, m->c.compute);
   }
+  if (m->c.sublayer_gate) {
+    const std::string gate = "l" + std::to_string(i) + ".rg1";
+    L.col_gate1 = (int)rows;
+    PI_TRY(ld.piece(gate, W, W, rows, 1, &p));
+    PI_TRY(ld.dev_vec(gate + ".b", W, &L.gate1_b));
+    rows += W;
+  }
   PI_TRY(ld.matrix(p, rows, W, &L.in));
   x.in = std::max(x.in, rows);
   x.core = std::max(x.core, core);
@@ -610,9 +673,18 @@ pi_status build_feed_forward(Loader& ld, int i, Layer& L, Extents& x) {
     PI_TRY(ld.piece(name + "gate", ff, W, at, 2, &p));
     return ld.piece(name + "up", ff, W, at + 1, 2, &p);
   };
+  const size_t gate_rows = ld.m->c.sublayer_gate ? W : 0;
+  auto sublayer_gate = [&](size_t at) -> pi_status {
+    if (!gate_rows) return PI_OK;
+    const std::string gate = "l" + std::to_string(i) + ".rg2";
+    PI_TRY(ld.piece(gate, W, W, at, 1, &p));
+    x.route = std::max(x.route, W);
+    return ld.dev_vec(gate + ".b", W, &L.gate2_b);
+  };
   if (c.ff_kind != PI_FF_EXPERTS) {
     PI_TRY(gated(mlp, c.ff, 0));
-    PI_TRY(ld.matrix(p, 2 * (size_t)c.ff, W, &L.gate_up));
+    PI_TRY(sublayer_gate(2 * (size_t)c.ff));
+    PI_TRY(ld.matrix(p, 2 * (size_t)c.ff + gate_rows, W, &L.gate_up));
     p.clear();
     PI_TRY(ld.piece(mlp + "down", W, c.ff, 0, 1, &p));
     x.ff = std::max(x.ff, (size_t)c.ff);
@@ -627,9 +699,13 @@ pi_status build_feed_forward(Loader& ld, int i, Layer& L, Extents& x) {
   e.group_best = c.group_best;
   e.renorm = c.renorm;
   e.scale = c.route_scale;
-  PI_TRY(ld.dev_vec(mlp + "correction", c.experts, &e.correction));
+  if (c.router_bias) PI_TRY(ld.dev_vec(mlp + "router.b", c.experts, &e.bias));
+  else PI_TRY(ld.dev_vec(mlp + "correction", c.experts, &e.correction));
   size_t rows = 2 * (size_t)c.shared_ff;
   if (c.shared_ff) PI_TRY(gated(mlp + "shared.", c.shared_ff, 0));
+  PI_TRY(sublayer_gate(rows));
+  rows += gate_rows;
+  L.col_router = (int)gate_rows;
   PI_TRY(ld.piece(mlp + "router", c.experts, W, rows, 1, &p));
   rows += c.experts;
   if (c.shared_ff && c.shared_gate) {
@@ -644,13 +720,18 @@ pi_status build_feed_forward(Loader& ld, int i, Layer& L, Extents& x) {
   }
   const size_t E = c.experts, ff = c.ff;
   p.clear();
-  for (size_t k = 0; k < E; ++k) PI_TRY(gated(mlp + "e" + std::to_string(k) + ".", ff, k * 2 * ff));
-  PI_TRY(ld.matrix(p, E * 2 * ff, W, &L.expert_in));
+  const bool unit_gated = c.unit != PI_UNIT_RELU2;
+  for (size_t k = 0; k < E; ++k) {
+    const std::string name = mlp + "e" + std::to_string(k) + ".";
+    if (unit_gated) PI_TRY(gated(name, ff, k * 2 * ff));
+    else PI_TRY(ld.piece(name + "up", ff, W, k * ff, 1, &p));
+  }
+  PI_TRY(ld.matrix(p, E * ff * (unit_gated ? 2 : 1), W, &L.expert_in));
   p.clear();
   for (size_t k = 0; k < E; ++k) PI_TRY(ld.piece(mlp + "e" + std::to_string(k) + ".down", W, ff, k * W, 1, &p));
   PI_TRY(ld.matrix(p, E * W, ff, &L.expert_out));
   x.ff = std::max(x.ff, (size_t)c.shared_ff);
-  x.route = std::max(x.route, E + 1);
+  x.route = std::max(x.route, gate_rows + E + 1);
   x.act = std::max(x.act, ff);
   x.top = std::max(x.top, (size_t)c.top);
   x.experts = std::max(x.experts, E);
@@ -661,11 +742,12 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
   m->c = *cfg;
   m->c.layers = nullptr;
   const size_t W = cfg->width;
-  const bool dyt = cfg->norm == PI_NORM_DYT, rms = cfg->norm == PI_NORM_RMS;
+  const bool dyt = cfg->norm == PI_NORM_DYT, rms = cfg->norm == PI_NORM_RMS, of_sum = cfg->norm == PI_NORM_SUM;
   size_t tensors = 8;
   for (int i = 0; i < cfg->num_layers; ++i) tensors += 40 + 3 * (size_t)std::max(0, cfg->layers[i].experts);
   ld.keep.reserve(tensors);   // Source::host points into it
   Extents x;
+  x.own.assign(cfg->num_layers, -1);
   {
     std::vector<Piece> p;
     PI_TRY(ld.piece("embed", cfg->vocab_size, W, 0, 1, &p));
@@ -682,7 +764,14 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
     PI_TRY(ld.piece("side.embed", cfg->vocab_size, cols, 0, 1, &p));
     PI_TRY(ld.matrix(p, cfg->vocab_size, cols, &m->side_embed));
   }
+  if (cfg->pair_buckets > 0) {
+    std::vector<Piece> p;
+    PI_TRY(ld.piece("bigram", (size_t)cfg->pair_buckets + 1, W, 0, 1, &p));
+    PI_TRY(ld.matrix(p, (size_t)cfg->pair_buckets + 1, W, &m->pairs));
+    m->state_floats = 32;            // the previous token, in front of what the layers keep
+  }
   if (dyt) PI_TRY(ld.dyt("final.norm", &m->final_norm));
+  else if (of_sum) PI_TRY(ld.rms_norm("final.norm", &m->final_ln, 0.f, cfg->logit_scale));
   else if (rms) PI_TRY(ld.rms_norm("final.norm", &m->final_ln, 1.f, cfg->logit_scale));
   else PI_TRY(ld.layer_norm("final.norm", &m->final_ln, cfg->logit_scale));
   m->layers.resize(cfg->num_layers);
@@ -694,6 +783,7 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
     const std::string l = "l" + std::to_string(i);
     auto norm = [&](const char* name, pi_dyt* before, pi_dyt* after, pi_layer_norm* ln, pi_layer_norm* post, const char* scale_name,
                     const float** scale) -> pi_status {
+      if (of_sum) return ld.rms_norm(l + name, post, 0.f, 1.f);
       if (rms) {
         PI_TRY(ld.rms_norm(l + name, ln, 1.f, 1.f));
         return ld.rms_norm(l + name + "b", post, 1.f, cfg->residual_mult);
@@ -723,6 +813,7 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
     L.c.decay = nullptr;             // the caller's
   }
   m->chunked = x.chunk && m->state_floats > 0;
+  m->regions = x.attn;
   const size_t cap = cfg->max_rows;
   m->ld_h = round8(W);
   m->ld_core = round8(x.core);
@@ -740,7 +831,7 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
   PI_TRY(alloc(&m->h, cap * m->ld_h));
   PI_TRY(alloc(&m->core, cap * m->ld_core));
   PI_TRY(alloc(&m->ffh, cap * m->ld_ff));
-  if (rms) PI_TRY(alloc(&m->y, cap * W));
+  if (rms || of_sum) PI_TRY(alloc(&m->y, cap * W));
   PI_TRY(alloc(&m->first_v, cap * m->mix_stride));
   m->ld_side = round8(cfg->side_dim);
   PI_TRY(alloc(&m->side_h, cap * m->ld_side));
@@ -748,8 +839,8 @@ pi_status build(pi_ctx* ctx, const pi_layered_config* cfg, Loader& ld, int gla_r
   PI_TRY(alloc(&m->lat_q, cap * x.lat_q / (f32 ? 1 : 2)));
   PI_TRY(alloc(&m->lat_o, (cap * x.lat_o + 1) / (f32 ? 1 : 2)));
   PI_TRY(alloc(&m->ssd_y, cap * x.inner));
+  PI_TRY(alloc(&m->route, cap * m->ld_route));
   if (x.top) {
-    PI_TRY(alloc(&m->route, cap * m->ld_route));
     PI_TRY(alloc(&m->shared, cap * W));
     PI_TRY(alloc(&m->moe_h, m->max_pairs * m->ld_h / 2));
     PI_TRY(alloc(&m->moe_act, m->max_pairs * m->ld_act));
@@ -832,8 +923,7 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
   PI_REQUIRE(ctx, in->block_tables || in->max_blocks == 0, "null block tables");
   PI_REQUIRE(ctx, m->state_floats == 0 || (state && in->state_slots), "this model carries recurrent state: the step needs a state pool and slots");
   PI_REQUIRE(ctx, m->state_floats == 0 || state->stride == m->state_floats, "the state pool was made for another model");
-  PI_REQUIRE(ctx, pool && pool->regions.size() == (size_t)std::count_if(m->layers.begin(), m->layers.end(), [](const Layer& l) { return l.attn >= 0; }) &&
-                      pool->kind == m->c.compute,
+  PI_REQUIRE(ctx, pool && pool->regions.size() == (size_t)m->regions && pool->kind == m->c.compute,
              "the KV pool was made for another model");
   const int n = in->n_seqs;
   int rows = 0, max_pos = 0;
@@ -997,7 +1087,7 @@ pi_status stage(pi_ctx* ctx, pi_layered* m, const pi_kv_pool* pool, const pi_sta
   size_t floats = 0, keys = 0, elems = 0;
   for (const Layer& L : m->layers) {
     if (L.c.mixer == PI_MIXER_SSD || L.c.mixer == PI_MIXER_LIGHTNING) floats = std::max(floats, pi_ssd_scratch_floats(L.ssd, b.n_chunks));
-    else if (L.attn < 0) floats = std::max(floats, pi_recurrence_scratch_floats(L.rec, b.n_chunks));
+    else if (L.c.mixer == PI_MIXER_GLA || L.c.mixer == PI_MIXER_MLSTM) floats = std::max(floats, pi_recurrence_scratch_floats(L.rec, b.n_chunks));
     else if (L.c.mixer == PI_MIXER_LATENT) {
       keys = std::max(keys, (size_t)b.n_keys * pi_latent_rp(L.c.rank));
       elems = std::max(elems, pi_latent_pool_elems(L.lat, b.exp_blocks));
@@ -1069,12 +1159,15 @@ pi_status run_mixer(pi_ctx* ctx, pi_layered* m, const Layer& L, pi_kv_pool* pool
     a.rope_sin = m->ropes[L.rope].sin;
     a.slopes = L.slopes;
     a.sinks = L.sinks;
+    a.sigmoid_bias = L.sigmoid_bias;
     if (c.head_gate) {
       a.gate = m->proj + L.col_gate;
       a.gate_stride = m->ld_proj;
       a.gate_per_head = true;
     }
     pi_maps_prepare prep;
+    prep.norm_qk = L.qk_norm;
+    prep.q_only = c.kv_from > 0;
     prep.bias = L.bias;
     prep.unit_qk = c.unit_qk != 0;
     prep.q_temp = L.temp >= 0 ? m->temps[L.temp].f : nullptr;
@@ -1082,7 +1175,7 @@ pi_status run_mixer(pi_ctx* ctx, pi_layered* m, const Layer& L, pi_kv_pool* pool
     pi_maps_kv mk;
     // biases, rotary positions, temperature, value mixing and the KV write fold into the projection; what needs a whole head does not,
     // and where nothing is rotated a kernel of its own is faster for many rows than the look-ups in the epilogue
-    if (c.dim % 2 == 0 && !c.unit_qk && !c.head_gate && (M <= kFoldRows || c.rot_dims > 0)) {
+    if (c.dim % 2 == 0 && !c.unit_qk && !c.norm_qk && !c.head_gate && L.gate1_b == nullptr && (M <= kFoldRows || c.rot_dims > 0)) {
       mk.bias = prep.bias;
       mk.q_temp = prep.q_temp;
       mk.mix = prep.mix;
@@ -1124,6 +1217,12 @@ pi_status run_mixer(pi_ctx* ctx, pi_layered* m, const Layer& L, pi_kv_pool* pool
     s.pool = static_cast<__nv_bfloat16*>(m->exp_pool.ptr);
     return pi_launch_latent_attention(ctx, a, kv_view(pool, L.attn), m->proj, m->ld_proj, m->core, m->ld_core, kind, b, s);
   }
+  if (c.mixer == PI_MIXER_MINGRU) {
+    pi_mingru r = L.gru;
+    r.state = state->data;
+    r.state_stride = state->stride;
+    return pi_launch_mingru(ctx, r, m->proj, m->ld_proj, m->core, m->ld_core, kind, b);
+  }
   if (c.mixer == PI_MIXER_SSD || c.mixer == PI_MIXER_LIGHTNING) {
     pi_ssd r = L.ssd;
     r.state = state->data;
@@ -1141,8 +1240,8 @@ pi_status run_experts(pi_ctx* ctx, pi_layered* m, const Layer& L, int M, bool bf
   const pi_layer_config& c = L.c;
   const pi_moe_lists lists = moe_lists(m);
   const int pairs = M * c.top;
-  const pi_epilogue unit = c.unit == PI_UNIT_SILU ? PI_EPI_SWIGLU : PI_EPI_CLAMP_GLU;
-  // the shared expert's first projection carries the router's rows
+  const pi_epilogue unit = c.unit == PI_UNIT_SILU ? PI_EPI_SWIGLU : c.unit == PI_UNIT_RELU2 ? PI_EPI_RELU2 : PI_EPI_CLAMP_GLU;
+  // the shared expert's first projection carries the rows of the sublayer gate and the router
   pi_linear_args a;
   if (c.shared_ff) {
     a.epi = unit;
@@ -1158,7 +1257,7 @@ pi_status run_experts(pi_ctx* ctx, pi_layered* m, const Layer& L, int M, bool bf
     a.out_stride = m->ld_route;
   }
   PI_TRY(project(ctx, L.gate_up, m->h, m->ld_h, M, bf16, a));
-  PI_TRY(pi_launch_moe_route(ctx, L.moe, m->route, m->ld_route, M, lists));
+  PI_TRY(pi_launch_moe_route(ctx, L.moe, m->route + L.col_router, m->ld_route, M, lists));
   pi_expert_rows rows;
   rows.experts = c.experts;
   const void* x = m->h;
@@ -1203,7 +1302,7 @@ pi_status run_experts(pi_ctx* ctx, pi_layered* m, const Layer& L, int M, bool bf
     sum->shared = m->shared;
     sum->shared_stride = m->c.width;
     if (c.shared_gate) {
-      sum->shared_gate = m->route + c.experts;
+      sum->shared_gate = m->route + L.col_router + c.experts;
       sum->shared_gate_stride = m->ld_route;
     }
   }
@@ -1217,11 +1316,16 @@ pi_status run_dense(pi_ctx* ctx, pi_layered* m, const Layer& L, int M, bool bf16
   g.out = static_cast<float*>(m->ffh);
   g.out_bf16 = static_cast<__nv_bfloat16*>(m->ffh);
   g.out_stride = m->ld_ff;
+  if (L.gate2_b) {
+    g.glu_rows = 2 * L.c.ff;
+    g.rest = m->route;
+    g.rest_stride = m->ld_route;
+  }
   PI_TRY(project(ctx, L.gate_up, m->h, m->ld_h, M, bf16, g));
   return project(ctx, L.down, m->ffh, m->ld_ff, M, bf16, down);
 }
 
-// Layer i with RMS norms, from h behind its mixer to `after`: the input of the next layer (or null for the last one's x alone).
+// Layer i with RMS norms of the results or of the sums, from core, the mixer's heads, to `after`: the input of the next layer (or null for the last one's x alone).
 pi_status run_sandwich(pi_ctx* ctx, pi_layered* m, const Layer& L, int i, const Staged& st, bool bf16, const pi_row_norm& row, const pi_row_norm& after) {
   const int M = st.b.rows;
   const pi_layer_config& c = L.c;
@@ -1229,8 +1333,17 @@ pi_status run_sandwich(pi_ctx* ctx, pi_layered* m, const Layer& L, int i, const 
   pi_linear_args a;                       // a sublayer's result
   a.out = m->y;
   a.out_stride = m->c.width;
+  const bool of_sum = m->c.norm == PI_NORM_SUM;
+  auto gate = [&](pi_row_norm* n, const float* z, size_t stride, const float* bias) {
+    if (!bias) return;
+    n->gate = z;
+    n->gate_stride = stride;
+    n->gate_bias = bias;
+  };
   auto result = [&](const pi_row_norm& to, const pi_layer_norm& post) {
     pi_row_norm n = to;
+    n.of_sum = of_sum;
+    n.keep = m->c.residual_keep;
     n.y = m->y;
     n.y_stride = m->c.width;
     n.post = post;
@@ -1241,9 +1354,11 @@ pi_status run_sandwich(pi_ctx* ctx, pi_layered* m, const Layer& L, int i, const 
   pi_expert_sum sum;
   if (c.ff > 0) {
     pi_row_norm between = result(row, L.post1);
-    between.norm = L.ln2;
+    between.norm = L.ln2;            // null behind a norm of the sum: h is x as it stands
+    gate(&between, m->proj + L.col_gate1, m->ld_proj, L.gate1_b);
     PI_TRY(pi_launch_row_norm(ctx, between));
     n.post = L.post2;
+    gate(&n, m->route, m->ld_route, L.gate2_b);
     if (c.ff_kind == PI_FF_EXPERTS) {
       PI_TRY(run_experts(ctx, m, L, M, bf16, &sum));
       n.y = nullptr;
@@ -1251,6 +1366,8 @@ pi_status run_sandwich(pi_ctx* ctx, pi_layered* m, const Layer& L, int i, const 
     } else {
       PI_TRY(run_dense(ctx, m, L, M, bf16, a));
     }
+  } else {
+    gate(&n, m->proj + L.col_gate1, m->ld_proj, L.gate1_b);
   }
   if (!side) return pi_launch_row_norm(ctx, n);
   pi_token_side t;
@@ -1279,7 +1396,7 @@ pi_status run_sandwich(pi_ctx* ctx, pi_layered* m, const Layer& L, int i, const 
 pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool* state, const Staged& st) {
   const pi_seq_batch& b = st.b;
   const int M = b.rows, W = m->c.width, NL = (int)m->layers.size();
-  const bool bf16 = act_bf16(ctx, m, M), dyt = m->c.norm == PI_NORM_DYT, rms = m->c.norm == PI_NORM_RMS;
+  const bool bf16 = act_bf16(ctx, m, M), dyt = m->c.norm == PI_NORM_DYT, rms = m->c.norm == PI_NORM_RMS || m->c.norm == PI_NORM_SUM;
   const int kind = bf16 ? PI_BF16 : PI_F32;
   const bool head_bf16 = st.n_out && act_bf16(ctx, m, st.n_out);
   pi_row_norm row;               // layer or RMS norm: from x to h
@@ -1303,6 +1420,9 @@ pi_status run_layers(pi_ctx* ctx, pi_layered* m, pi_kv_pool* pool, pi_state_pool
     e.vocab = m->c.vocab_size;
     e.tokens = b.tokens;
     e.norm = m->layers[0].ln1;
+    if (m->pairs)
+      e.pairs = pi_token_pairs{static_cast<const uint16_t*>(m->pairs->w), m->pairs->ld, m->c.pair_buckets, m->c.pair_prev, m->c.pair_cur,
+                               b.row_seq, b.seq_row0, b.seq_n, b.seq_start, b.slot, state->data, state->stride};
     PI_TRY(pi_launch_row_norm(ctx, e));
   }
   bool final_done = false;       // head_in holds the normalised rows
@@ -1421,11 +1541,15 @@ pi_status pi_layered_create(pi_ctx* ctx, const pi_layered_config* cfg, const pi_
   PI_REQUIRE(ctx, ctx->tp == 1, "layered designs run on one GPU");
   PI_REQUIRE(ctx, cfg->width > 0 && cfg->vocab_size > 0 && cfg->num_layers > 0 && cfg->layers && cfg->max_rows > 0, "model config fields must be positive");
   PI_REQUIRE(ctx, cfg->compute == PI_BF16 || cfg->compute == PI_F32, "layered designs compute in bf16 or f32");
-  PI_REQUIRE(ctx, cfg->norm >= PI_NORM_DYT && cfg->norm <= PI_NORM_RMS, "unknown normalisation %d", cfg->norm);
+  PI_REQUIRE(ctx, cfg->norm >= PI_NORM_DYT && cfg->norm <= PI_NORM_SUM, "unknown normalisation %d", cfg->norm);
   PI_REQUIRE(ctx, cfg->norm != PI_NORM_DYT || cfg->logit_scale == 1.f, "logits are not scaled behind Dynamic Tanh");
   PI_REQUIRE(ctx, cfg->side_dim >= 0, "sizes must be positive");
-  PI_REQUIRE(ctx, cfg->norm == PI_NORM_RMS || (cfg->embed_scale == 1.f && cfg->residual_mult == 1.f && cfg->side_dim == 0),
-             "a scale of the embedding, a factor of the residual update and a table of tokens belong to RMS norms");
+  PI_REQUIRE(ctx, cfg->norm == PI_NORM_RMS || (cfg->residual_mult == 1.f && cfg->side_dim == 0),
+             "a factor of the residual update and a table of tokens belong to RMS norms of the results");
+  PI_REQUIRE(ctx, cfg->norm == PI_NORM_SUM || (cfg->residual_keep == 1.f && !cfg->sublayer_gate), "sublayer gates and a factor of the residual stream belong to norms of the sum");
+  PI_REQUIRE(ctx, cfg->norm >= PI_NORM_RMS || (cfg->embed_scale == 1.f && cfg->pair_buckets == 0), "a scale of the embedding and a table of token pairs belong to RMS norms");
+  PI_REQUIRE(ctx, cfg->pair_buckets == 0 || (cfg->pair_buckets > 0 && cfg->pair_prev >= 0 && cfg->pair_prev < cfg->pair_buckets && cfg->pair_cur >= 0 &&
+                                             cfg->pair_cur < cfg->pair_buckets), "the factors of a token pair are taken modulo the table's length");
   PI_REQUIRE(ctx, tensors || gla_rank > 0, "synthetic weights need a rank for the decay's low-rank input");
   pi_layered* m = new (std::nothrow) pi_layered();
   if (!m) return pi_fail(ctx, PI_ERR_OOM, "host allocation failed");
@@ -1453,6 +1577,7 @@ void pi_layered_destroy(pi_layered* m) {
   pi_linear_destroy(m->embed);
   pi_linear_destroy(m->head);
   pi_linear_destroy(m->side_embed);
+  pi_linear_destroy(m->pairs);
   for (TempTable& t : m->temps) cudaFree(t.f);
   for (RopeTable& t : m->ropes) {
     cudaFree(t.cos);
@@ -1476,7 +1601,7 @@ pi_status pi_layered_kv_regions(pi_ctx* ctx, const pi_layered* m, int num_blocks
   size_t at = 0;
   pool->kind = m->c.compute;
   for (const Layer& L : m->layers) {
-    if (L.attn < 0) continue;
+    if (L.attn < (int)pool->regions.size()) continue;   // none, or another layer's
     pi_kv_region g;
     if (L.c.mixer == PI_MIXER_LATENT) {   // [latent | rotated key part], common to the heads
       g.kv_heads = g.maps = 1;

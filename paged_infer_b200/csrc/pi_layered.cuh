@@ -1,5 +1,5 @@
 // Internal declarations of layered designs: models whose layers each name a token mixer (windowed multi-map attention,
-// latent attention, a gated linear recurrence, a matrix memory, a state-space recurrence, lightning attention) and a
+// latent attention, a gated linear recurrence, a matrix memory, a state-space recurrence, lightning attention, minGRU) and a
 // feed-forward (dense or experts) with sizes of their own.
 #pragma once
 
@@ -68,6 +68,7 @@ struct pi_maps_attention {
   bool gate_per_head = false;
   const float* slopes = nullptr;        // [heads] taken off a score per token of distance
   const float* sinks = nullptr;         // [heads] exp(sink) joins the sum of weights, once, without a value
+  const float* sigmoid_bias = nullptr;  // [heads] a key weighs sigmoid(score + bias) instead, not normalised (maps == 1; no slopes, sinks)
   bool v_in_k = false;                  // the values are the first channels of the keys (f32 kernel)
   int rot_dims = 0;
   const float* rope_cos = nullptr;      // [positions][rot_dims / 2]
@@ -77,8 +78,10 @@ struct pi_kv_view {                     // one layer's region of the pool
   void* base = nullptr;
   int kind = PI_F32, kv_heads = 0, maps = 0, dp = 0, vp = 0, block_size = 0;
 };
-// What happens to q, k and v between projection and attention beside the rotation (all optional).
+// What happens to q, k and v between projection and attention beside the rotation (all optional; norm_qk stands alone).
 struct pi_maps_prepare {
+  const float* norm_qk = nullptr;       // [q | k] weights of an RMS norm over all of q, and one over all of k (eps of the attention)
+  bool q_only = false;                  // k and v are another layer's
   const float* bias = nullptr;          // [q | k | v]
   bool unit_qk = false;                 // q and k over their root mean square, per head and map (eps of the attention)
   const float* q_temp = nullptr;        // [positions] factor of q
@@ -150,6 +153,7 @@ struct pi_moe {
   int experts = 0, top = 0, groups = 1, keep = 1;
   int score = PI_SCORE_SIGMOID, group_best = 2, renorm = 1;
   float scale = 1.f;                    // of the weights
+  const float* bias = nullptr;          // [experts], of the logits
   const float* correction = nullptr;    // [experts], part of the choice and not of the weights
 };
 struct pi_moe_lists {
@@ -181,12 +185,27 @@ struct pi_expert_sum {
   size_t shared_stride = 0, shared_gate_stride = 0;
   const float* scale = nullptr;         // [width]
 };
+// A table of token pairs beside the embedding: row (previous token mul_prev + token mul_cur) mod buckets, for a sequence's first token
+// row `buckets`.  The previous token of a portion's first row is in the sequence's state slot; the step leaves its last token there.
+struct pi_token_pairs {
+  const uint16_t* table = nullptr;
+  size_t ld = 0;
+  int buckets = 0, mul_prev = 0, mul_cur = 0;
+  const int32_t *row_seq = nullptr, *seq_row0 = nullptr, *seq_n = nullptr, *seq_start = nullptr, *slot = nullptr;
+  float* state = nullptr;               // the token as an integer, in the first word of a slot
+  size_t state_stride = 0;
+};
 struct pi_row_norm {
   bool rms = false;                     // RMS norms (weights as they multiply) instead of layer norm; then also:
   const float* y = nullptr;             //   x += post(y) first; post applies to the experts' sum too
   size_t y_stride = 0;
   pi_layer_norm post;
-  float embed_scale = 1.f;              //   x = embed_scale table[token]
+  bool of_sum = false;                  //   x = post(keep x + y) instead
+  float keep = 1.f;
+  const float *gate = nullptr, *gate_bias = nullptr;   // the result times sigmoid(gate[row][.] + gate_bias[.]) (null: not)
+  size_t gate_stride = 0;
+  float embed_scale = 1.f;              //   x = embed_scale table[token] + pairs[its pair]
+  pi_token_pairs pairs;
                                         //   norm.w null: h is x as it stands
   int rows = 0, width = 0;
   float* x = nullptr;                   // [.][width]
@@ -253,6 +272,19 @@ pi_status pi_launch_recurrence_chunks(pi_ctx* ctx, const pi_recurrence& r, const
 // A portion of at least this many tokens takes the chunked kernels (when they hold the layer's sizes).
 constexpr int kRecurrenceChunk = 64;
 bool pi_recurrence_chunked(const pi_ctx* ctx, const pi_recurrence& r, int compute);
+
+// ---- minGRU (pi_mingru.cu) -------------------------------------------------------------------------------------------
+// S = (1 - z) S + z c per channel, z = sigmoid(zl), c = u + 1/2 (u >= 0) or sigmoid(u); out = S silu(g).
+struct pi_mingru {
+  int width = 0;
+  const float *z_bias = nullptr, *x_bias = nullptr;   // [width]
+  int col_z = 0, col_x = 0, col_g = 0;  // columns of the fused projection
+  float* state = nullptr;               // S [width] per slot
+  size_t state_stride = 0, state_off = 0;
+  size_t state_floats() const { return ((size_t)width + 31) / 32 * 32; }
+};
+pi_status pi_launch_mingru(pi_ctx* ctx, const pi_mingru& r, const float* proj, size_t stride, void* out, size_t out_stride, int out_kind,
+                           const pi_seq_batch& b);
 
 // ---- row-wise glue (pi_layered.cu) -----------------------------------------------------------------------------------
 template <typename K, typename... Args>

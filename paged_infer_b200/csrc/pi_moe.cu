@@ -1,6 +1,7 @@
 // Routing of tokens to experts.
 //
-// moe_route_kernel: a warp per token.  Scores s = sigmoid(logit), or the softmax of all logits; choice scores s + correction; the
+// moe_route_kernel: a warp per token.  Scores s = sigmoid(logit), or the softmax of all logits, or the logits themselves (the weights
+// are then the softmax over the chosen alone); choice scores s + correction; the
 // experts form equal groups of neighbours, a group's score is its best choice score or the sum of its two best, and only the
 // experts of the best groups can be chosen; among them the best choice scores win, ties to the lower index.  Weights: the
 // chosen scores s, over their sum if they are brought to sum 1, times a constant.
@@ -20,8 +21,8 @@ constexpr int kListThreads = 1024;
 struct RouteParams {
   const float* logits;
   size_t stride;
-  const float* correction;
-  int rows, experts, groups, keep, top, softmax, group_best, renorm;
+  const float *bias, *correction;
+  int rows, experts, groups, keep, top, score, group_best, renorm;
   float scale;
   int32_t* ids;
   float* weights;
@@ -47,14 +48,15 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const Route
   if (row >= p.rows) return;
   const float* z = p.logits + (size_t)row * p.stride;
   float top_z = -INFINITY, z_sum = 0.f;
-  if (p.softmax) {
-    for (int e = lane; e < p.experts; e += 32) top_z = fmaxf(top_z, z[e]);
+  auto logit = [&](int e) { return z[e] + (p.bias ? __ldg(p.bias + e) : 0.f); };
+  if (p.score == PI_SCORE_SOFTMAX) {
+    for (int e = lane; e < p.experts; e += 32) top_z = fmaxf(top_z, logit(e));
     top_z = pi_warp_max(top_z);
-    for (int e = lane; e < p.experts; e += 32) z_sum += expf(z[e] - top_z);
+    for (int e = lane; e < p.experts; e += 32) z_sum += expf(logit(e) - top_z);
     z_sum = pi_warp_sum(z_sum);
   }
   for (int e = lane; e < p.experts; e += 32) {
-    const float s = p.softmax ? expf(z[e] - top_z) / z_sum : pi_sigmoid(z[e]);
+    const float s = p.score == PI_SCORE_CHOSEN ? logit(e) : p.score == PI_SCORE_SOFTMAX ? expf(logit(e) - top_z) / z_sum : pi_sigmoid(logit(e));
     score[e] = s;
     choice[e] = s + (p.correction ? __ldg(p.correction + e) : 0.f);
   }
@@ -87,7 +89,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const Route
       if (!isnan(group[e / n])) choice[e] = -INFINITY;
     __syncwarp();
   }
-  float sum = 0.f;
+  float sum = 0.f, first = -INFINITY;
   int mine[2] = {0, 0};                                // choices lane and lane + 32
   for (int k = 0; k < p.top; ++k) {
     Best b = {-INFINITY, 0x7fffffff};
@@ -96,9 +98,24 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const Route
     b = warp_best(b);
     const int e = min(b.i, p.experts - 1);             // (a row of NaN chooses something valid)
     if (lane == (k & 31)) mine[k >> 5] = e;
+    first = fmaxf(first, score[e]);
     sum += score[e];
     if (lane == 0) choice[e] = -INFINITY;
     __syncwarp();
+  }
+  if (p.score == PI_SCORE_CHOSEN) {
+    sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+      if (lane + 32 * j < p.top) sum += expf(score[mine[j]] - first);
+    sum = pi_warp_sum(sum);
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+      if (lane + 32 * j < p.top) {
+        p.ids[(size_t)row * p.top + lane + 32 * j] = mine[j];
+        p.weights[(size_t)row * p.top + lane + 32 * j] = p.scale * expf(score[mine[j]] - first) / sum;
+      }
+    return;
   }
 #pragma unroll
   for (int j = 0; j < 2; ++j)
@@ -175,7 +192,7 @@ int pi_moe_max_tiles(int rows, const pi_moe& m) {
 
 pi_status pi_launch_moe_route(pi_ctx* ctx, const pi_moe& m, const float* logits, size_t stride, int rows, const pi_moe_lists& l) {
   pi_prof_scope prof(ctx, PI_PROF_OTHER);
-  const RouteParams p = {logits, stride, m.correction, rows, m.experts, m.groups, m.keep, m.top, m.score == PI_SCORE_SOFTMAX, m.group_best,
+  const RouteParams p = {logits, stride, m.bias, m.correction, rows, m.experts, m.groups, m.keep, m.top, m.score, m.group_best,
                          m.renorm, m.scale, l.ids, l.weights};
   const size_t smem = (size_t)kRouteWarps * (2 * m.experts + m.groups) * sizeof(float);
   PI_REQUIRE(ctx, smem <= kSmemFit && m.top <= 64, "%d of %d experts are too many", m.top, m.experts);

@@ -4,7 +4,8 @@
 // row_norm_kernel: sublayers that are normalised before (layer norm: zero mean, unit variance, a weight, no bias); mean and
 // variance are two passes over the row in shared memory.
 // row_rms_kernel: sublayers that are normalised before and after: x += rms norm of the result, then h = rms norm of x (or x as it
-// stands).  The row stays in registers between the two norms.
+// stands); or sublayers whose sum is normalised: x = rms norm of (keep x + result).  The result may be gated channel by channel
+// first.  The row stays in registers between the two norms.  The embedding may have a row of a table of token pairs beside it.
 #include <algorithm>
 
 #include "pi_layered.cuh"
@@ -33,6 +34,11 @@ struct RowParams {
   size_t y_stride;
   const float* post_w;
   float post_eps, embed_scale;
+  int of_sum;
+  float keep;
+  const float *gate, *gate_bias;
+  size_t gate_stride;
+  pi_token_pairs pairs;
 };
 
 __device__ __forceinline__ float row_sum(float v, float* red) {   // over the CTA; the same bits in every thread
@@ -153,6 +159,29 @@ __device__ __forceinline__ void store_row4<__nv_bfloat16>(__nv_bfloat16* p, floa
   *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
 }
 
+// The pair of row r's token: its row of the table.  Thread 0 of the CTA that owns a portion's first row reads the previous token and
+// leaves the portion's last one in its place.
+__device__ __forceinline__ const uint16_t* pair_row(const RowParams& p, int r, long long* s_row) {
+  const pi_token_pairs& k = p.pairs;
+  if (threadIdx.x == 0) {
+    const int seq = k.row_seq[r], row0 = k.seq_row0[seq];
+    long long at = k.buckets;
+    uint32_t* kept = reinterpret_cast<uint32_t*>(k.state + (size_t)k.slot[seq] * k.state_stride);
+    if (r > row0 || k.seq_start[seq] > 0) {
+      const uint32_t prev = r > row0 ? p.tokens[r - 1] : *kept;
+      at = ((long long)prev * k.mul_prev + (long long)p.tokens[r] * k.mul_cur) % k.buckets;
+    }
+    if (r == row0) *kept = p.tokens[row0 + k.seq_n[seq] - 1];
+    *s_row = at;
+  }
+  __syncthreads();
+  return k.table + (size_t)*s_row * k.ld;
+}
+__device__ __forceinline__ float4 widen4(const uint16_t* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+}
+
 // HOLD: groups of four channels per thread, 0: any width, through shared memory one channel at a time.
 template <typename T, RowSource SRC, int HOLD>
 __global__ void __launch_bounds__(kRowThreads) row_rms_kernel(const RowParams p) {
@@ -173,6 +202,9 @@ __global__ void __launch_bounds__(kRowThreads) row_rms_kernel(const RowParams p)
   else pi_grid_dependency_wait();
   float* x = p.x + (size_t)src * p.width;
   const uint16_t* t = SRC == kFromEmbedding ? p.table + (size_t)(p.tokens[r] % (uint32_t)p.vocab) * p.table_ld : nullptr;
+  __shared__ long long s_pair;
+  const uint16_t* pair = SRC == kFromEmbedding && p.pairs.table ? pair_row(p, r, &s_pair) : nullptr;
+  const float* gate = POST && p.gate ? p.gate + (size_t)r * p.gate_stride : nullptr;
   if (SRC == kFromExperts) {
     if (tid < e.top) {
       s_w[tid] = e.weights[(size_t)r * e.top + tid];
@@ -189,9 +221,7 @@ __global__ void __launch_bounds__(kRowThreads) row_rms_kernel(const RowParams p)
     for (int j = 0; j < HOLD; ++j) {         // past the end: the last channels again, not counted
       const int i = (tid + j * kRowThreads) * 4, at = min(i, p.width - 4);
       if (SRC == kFromEmbedding) {
-        const uint2 u = *reinterpret_cast<const uint2*>(t + at);
-        v[j] = make_float4(p.embed_scale * __uint_as_float(u.x << 16), p.embed_scale * __uint_as_float(u.x & 0xffff0000u),
-                           p.embed_scale * __uint_as_float(u.y << 16), p.embed_scale * __uint_as_float(u.y & 0xffff0000u));
+        v[j] = fma4(p.embed_scale, widen4(t + at), pair ? widen4(pair + at) : make_float4(0.f, 0.f, 0.f, 0.f));
       } else {
         v[j] = *reinterpret_cast<const float4*>(x + at);
       }
@@ -215,13 +245,20 @@ __global__ void __launch_bounds__(kRowThreads) row_rms_kernel(const RowParams p)
               if (k0 + k < e.top) y[j] = fma4(s_w[k0 + k], z[k], y[j]);
           }
         }
+        if (gate) {
+          const float4 z = *reinterpret_cast<const float4*>(gate + at), b = __ldg(reinterpret_cast<const float4*>(p.gate_bias + at));
+          y[j] = make_float4(y[j].x * pi_sigmoid(z.x + b.x), y[j].y * pi_sigmoid(z.y + b.y), y[j].z * pi_sigmoid(z.z + b.z), y[j].w * pi_sigmoid(z.w + b.w));
+        }
+        if (p.of_sum) y[j] = fma4(p.keep, v[j], y[j]);
         if (i < p.width) ss += dot4(y[j]);
       }
       const float inv = 1.0f / sqrtf(row_sum_once(ss, red[0]) / (float)p.width + p.post_eps);
 #pragma unroll
-      for (int j = 0; j < HOLD; ++j)
+      for (int j = 0; j < HOLD; ++j) {
+        if (p.of_sum) v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
         v[j] = make_float4(fmaf(y[j].x * inv, wp[j].x, v[j].x), fmaf(y[j].y * inv, wp[j].y, v[j].y), fmaf(y[j].z * inv, wp[j].z, v[j].z),
                            fmaf(y[j].w * inv, wp[j].w, v[j].w));
+      }
     }
     ss = 0.f;
 #pragma unroll
@@ -252,20 +289,22 @@ __global__ void __launch_bounds__(kRowThreads) row_rms_kernel(const RowParams p)
         if (e.shared) v = shared_gate * e.shared[(size_t)r * e.shared_stride + i];
         for (int k = 0; k < e.top; ++k) v = fmaf(s_w[k], expert_value(e, (size_t)s_at[k] * e.y_stride + i), v);
       }
+      if (gate) v *= pi_sigmoid(gate[i] + __ldg(p.gate_bias + i));
+      if (p.of_sum) v = fmaf(p.keep, x[i], v);
       row[i] = v;
       ss = fmaf(v, v, ss);
     }
     const float inv = 1.0f / sqrtf(row_sum_once(ss, red[0]) / (float)p.width + p.post_eps);
     ss = 0.f;
     for (int i = tid; i < p.width; i += kRowThreads) {   // every thread its own channels, as above
-      const float v = fmaf(row[i] * inv, __ldg(p.post_w + i), x[i]);
+      const float v = fmaf(row[i] * inv, __ldg(p.post_w + i), p.of_sum ? 0.f : x[i]);
       x[i] = v;
       row[i] = v;
       ss = fmaf(v, v, ss);
     }
   } else {
     for (int i = tid; i < p.width; i += kRowThreads) {
-      const float v = SRC == kFromEmbedding ? p.embed_scale * pi_bf16_bits_to_f32(t[i]) : x[i];
+      const float v = SRC == kFromEmbedding ? fmaf(p.embed_scale, pi_bf16_bits_to_f32(t[i]), pair ? pi_bf16_bits_to_f32(pair[i]) : 0.f) : x[i];
       if (SRC == kFromEmbedding) x[i] = v;
       row[i] = v;
       ss = fmaf(v, v, ss);
@@ -292,7 +331,7 @@ void (*pick_rms(RowSource s, const RowParams& p, bool in_registers))(const RowPa
 pi_status pi_launch_row_norm(pi_ctx* ctx, const pi_row_norm& n) {
   pi_prof_scope prof(ctx, PI_PROF_OTHER);
   RowParams p = {n.x, n.width, n.pick, n.table, n.table_ld, n.vocab, n.tokens, {}, n.norm.w, n.norm.eps, n.h, n.ld_h,
-                 n.y, n.y_stride, n.post.w, n.post.eps, n.embed_scale};
+                 n.y, n.y_stride, n.post.w, n.post.eps, n.embed_scale, n.of_sum, n.keep, n.gate, n.gate_bias, n.gate_stride, n.pairs};
   if (n.experts) p.e = *n.experts;
   PI_REQUIRE(ctx, p.e.top <= 64, "at most 64 experts per token, not %d", p.e.top);
   const bool bf16 = n.h_kind == PI_BF16;
@@ -302,10 +341,14 @@ pi_status pi_launch_row_norm(pi_ctx* ctx, const pi_row_norm& n) {
     PI_REQUIRE(ctx, !(n.y || n.experts) || n.post.w, "a sublayer's result needs its norm");
     const RowSource src = n.table ? kFromEmbedding : n.experts ? kFromExperts : n.y ? kFromResult : kFromX;
     const bool aligned = n.width % 4 == 0 && n.ld_h % 4 == 0 && (!n.table || n.table_ld % 4 == 0) && (!n.y || n.y_stride % 4 == 0) &&
-                         (!n.experts || (p.e.y_stride % 4 == 0 && p.e.shared_stride % 4 == 0 && !p.e.scale));
+                         (!n.experts || (p.e.y_stride % 4 == 0 && p.e.shared_stride % 4 == 0 && !p.e.scale)) &&
+                         (!n.gate || (n.gate_stride % 4 == 0 && (uintptr_t)n.gate % 16 == 0)) && (!n.pairs.table || n.pairs.ld % 4 == 0);
     PI_REQUIRE(ctx, !n.experts || !p.e.scale, "a scale per channel belongs to layer norm");
+    PI_REQUIRE(ctx, !n.gate || n.gate_bias, "a gate needs its bias");
     in_registers = aligned && n.width <= 16 * kRowThreads;
     k = bf16 ? pick_rms<__nv_bfloat16>(src, p, in_registers) : pick_rms<float>(src, p, in_registers);
+  } else if (n.of_sum || n.gate || n.pairs.table) {
+    return pi_fail(ctx, PI_ERR_INVALID_ARG, "norms of the sum, gates and token pairs belong to RMS norms");
   } else if (n.table) k = bf16 ? row_norm_kernel<__nv_bfloat16, kFromEmbedding> : row_norm_kernel<float, kFromEmbedding>;
   else if (n.experts) k = bf16 ? row_norm_kernel<__nv_bfloat16, kFromExperts> : row_norm_kernel<float, kFromExperts>;
   else k = bf16 ? row_norm_kernel<__nv_bfloat16, kFromX> : row_norm_kernel<float, kFromX>;

@@ -74,11 +74,11 @@ class LlamaConfig:
             "intermediate_size", "vocab_size", "rms_norm_eps", "rope_theta", "attention_window", "rope_style")}
 
 
-MIXER_ATTENTION, MIXER_GLA, MIXER_MLSTM, MIXER_LATENT, MIXER_SSD, MIXER_LIGHTNING = 0, 1, 2, 3, 4, 5
+MIXER_ATTENTION, MIXER_GLA, MIXER_MLSTM, MIXER_LATENT, MIXER_SSD, MIXER_LIGHTNING, MIXER_MINGRU = 0, 1, 2, 3, 4, 5, 6
 FF_GELU, FF_SILU, FF_EXPERTS = 0, 1, 2
-UNIT_CLAMPED, UNIT_SILU = 0, 1
-SCORE_SIGMOID, SCORE_SOFTMAX = 0, 1
-NORM_DYT, NORM_LAYER, NORM_RMS = 0, 1, 2
+UNIT_CLAMPED, UNIT_SILU, UNIT_RELU2 = 0, 1, 2
+SCORE_SIGMOID, SCORE_SOFTMAX, SCORE_CHOSEN = 0, 1, 2
+NORM_DYT, NORM_LAYER, NORM_RMS, NORM_SUM = 0, 1, 2, 3
 
 
 @dataclass
@@ -94,7 +94,10 @@ class LayerConfig:
     together; the chosen weights are brought to sum 1 if ``renorm`` and multiplied by ``route_scale``.  Attention with one map may
     have ``biases``, q and k of unit root mean square (``unit_qk``), a ``distance_bias``, a ``sink`` and a gate per head, queries
     that grow with the position (``q_temp_coef``, ``q_temp_every``; 0: not) and values mixed with those of the first layer that has
-    ``v_mix``.  ``decay``: the constant decay of every head of lightning attention."""
+    ``v_mix``; or q and k normalised over the whole projection (``norm_qk``), ``sigmoid_weights`` that are not normalised over the
+    keys, and the keys and values of the layer ``kv_from`` in place of its own.  ``rot_banded``: the rotation is stretched by
+    wavelength.  ``decay``: the constant decay of every head of lightning attention.  The element-wise recurrence (minGRU) has one head
+    of ``vdim`` channels.  ``router_bias``: of the router's logits, in place of a correction of the choice."""
 
     mixer: int
     heads: int
@@ -141,6 +144,11 @@ class LayerConfig:
     renorm: bool = True
     shared_gate: bool = True
     route_scale: float = 1.0
+    router_bias: bool = False
+    rot_banded: bool = False
+    norm_qk: bool = False
+    sigmoid_weights: bool = False
+    kv_from: int | None = None
 
 
 @dataclass
@@ -157,10 +165,16 @@ class LayeredConfig:
     embed_scale: float = 1.0
     residual_mult: float = 1.0
     side_dim: int = 0
+    residual_keep: float = 1.0
+    sublayer_gate: bool = False
+    pair_buckets: int = 0        # rows of the table of token pairs, but for the one of first tokens
+    pair_prev: int = 0
+    pair_cur: int = 0
 
     @property
     def has_state(self) -> bool:
-        return any(l.mixer not in (MIXER_ATTENTION, MIXER_LATENT) for l in self.layers)
+        """Whether a sequence carries more than its cache: a recurrence, or the previous token."""
+        return self.pair_buckets > 0 or any(l.mixer not in (MIXER_ATTENTION, MIXER_LATENT) for l in self.layers)
 
     @classmethod
     def from_sumosun(cls, j: dict) -> "LayeredConfig":
@@ -267,6 +281,41 @@ class LayeredConfig:
             raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
         return dict(unit=UNIT_SILU, score=SCORE_SOFTMAX, group_best=1, renorm=False, shared_gate=False, route_scale=float(mlp["router"]["scale"]),
                     **cls._experts(mlp))
+
+    @classmethod
+    def from_noresun(cls, j: dict) -> "LayeredConfig":
+        """The Noresun design's ``config.json``: attention with sigmoid weights, which may share the keys and values of an earlier layer,
+        and minGRU layers in any order, each with routed experts or no feed-forward; gated sublayers, norms of the sum; a table of token
+        pairs beside the embedding."""
+        layers = []
+        for i, e in enumerate(j["layers"]):
+            m, mlp = e["mixer"], e.get("mlp")
+            kw = {}
+            if mlp is not None:
+                if mlp["kind"] != "moe":
+                    raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+                kw = dict(unit=UNIT_RELU2, score=SCORE_CHOSEN, shared_gate=False, router_bias=True, **cls._experts(mlp))
+            if e["type"] == "attention":
+                mask, rot, kv_from = m.get("mask"), m.get("rot"), m.get("kv_from")
+                if rot:
+                    kw.update(rot_dims=int(rot["dims"]), rot_base=float(rot["base"]))
+                    if rot.get("scaling"):
+                        s = rot["scaling"]
+                        kw.update(rot_banded=True, rot_factor=float(s["factor"]), rot_original=float(s["original"]), rot_fast=float(s["high"]),
+                                  rot_slow=float(s["low"]))
+                layers.append(LayerConfig(MIXER_ATTENTION, heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                                          window=int(mask["size"]) if mask else None, scale=float(m["scale"]), norm_qk=True, sigmoid_weights=True,
+                                          kv_from=None if kv_from is None else int(kv_from), **kw))
+            elif e["type"] == "mingru":
+                layers.append(LayerConfig(MIXER_MINGRU, heads=1, dim=1, vdim=int(m["width"]), **kw))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+        pairs, kw = j["embedding"].get("bigram"), {}
+        if pairs:
+            n = int(pairs["buckets"])
+            kw = dict(pair_buckets=n, pair_prev=int(pairs["mul_prev"]) % n, pair_cur=int(pairs["mul_cur"]) % n)
+        return cls(width=int(j["width"]), vocab_size=int(j["vocab"]), norm_eps=float(j["norm"]["eps"]), layers=layers, norm=NORM_SUM,
+                   embed_scale=float(j["embedding"]["scale"]), residual_keep=float(j["postln_alpha"]), sublayer_gate=True, **kw)
 
 
 def read_safetensors(path: str) -> dict:

@@ -46,6 +46,7 @@ FAMILIES = {
     "Sumosun": Family(_layered(LayeredConfig.from_sumosun), ("bfloat16", "float32")),
     "Lilosun": Family(_layered(LayeredConfig.from_lilosun), ("bfloat16", "float32")),
     "Rubuvik": Family(_layered(LayeredConfig.from_rubuvik), ("bfloat16", "float32")),
+    "Noresun": Family(_layered(LayeredConfig.from_noresun), ("bfloat16", "float32")),
 }
 
 
