@@ -1040,6 +1040,54 @@ def rubuvik_work(cfg, model, B, ctx_len, M):
             "prefill_bytes": {"recurrence": sum(M * (4 * (2 * inner(l) + 2 * l.heads * l.dim) + 10 * inner(l)) + 8 * (M // 64) * inner(l) * l.dim for l in rec)}}
 
 
+# Noresun beside Rubuvik (paged windowed attention with one map, routed experts, norms of whole rows): the same width, depth, vocabulary,
+# window and attention heads.  Experts have two matrices instead of three and there is no shared one; what a token meets of a layer's
+# experts, and the weights behind them, are about the same.
+NORESUN_SIZES = {
+    "w2048": dict(attention=dict(heads=16, kv_heads=4, dim=128, vdim=128), gru=4096, moe=dict(experts=64, top=8, ff=1056), like="w2048"),
+    "w4096": dict(attention=dict(heads=32, kv_heads=8, dim=128, vdim=128), gru=8192, moe=dict(experts=32, top=6, ff=3584), like="w4096"),
+}
+
+
+def noresun_config(size):
+    from paged_infer_b200 import loader as ld
+    s = NORESUN_SIZES[size]
+    l = LILOSUN_SIZES[s["like"]]
+    moe = dict(ff_kind=ld.FF_EXPERTS, unit=ld.UNIT_RELU2, score=ld.SCORE_CHOSEN, shared_gate=False, router_bias=True, **s["moe"])
+    attn = dict(window=l["window"], scale=128 ** -0.5, rot_dims=64, rot_base=500000.0, rot_banded=True, rot_factor=8.0, rot_original=8192, rot_fast=4.0, rot_slow=1.0,
+                norm_qk=True, sigmoid_weights=True, **s["attention"])
+    kinds = [lambda i: ld.LayerConfig(ld.MIXER_ATTENTION, **attn, **moe), lambda i: ld.LayerConfig(ld.MIXER_MINGRU, heads=1, dim=1, vdim=s["gru"], **moe),
+             lambda i: ld.LayerConfig(ld.MIXER_ATTENTION, kv_from=i - 2, **attn, **moe)]
+    return ld.LayeredConfig(l["width"], l["vocab"], 1e-6, [kinds[i % 3](i) for i in range(l["layers"])], norm=ld.NORM_SUM, embed_scale=1.0, residual_keep=2.0,
+                            sublayer_gate=True, pair_buckets=65536, pair_prev=31, pair_cur=7)
+
+
+def noresun_work(cfg, model, B, ctx_len, M):
+    """As rubuvik_work; the recurrence's state is a vector, so its operands and results count in a decode step too."""
+    from paged_infer_b200 import loader as ld
+    W = cfg.width
+    attn = [l for l in cfg.layers if l.mixer == ld.MIXER_ATTENTION]
+    rec = [l for l in cfg.layers if l.mixer == ld.MIXER_MINGRU]
+    fixed = flops = 0
+    met = 0.0
+    for l in cfg.layers:
+        own = W * (2 * W + l.experts)                        # sublayer gates, router
+        if l.mixer == ld.MIXER_ATTENTION:
+            own += W * (l.heads * (l.dim + l.vdim) + (l.kv_heads * (l.dim + l.vdim) if l.kv_from is None else 0))
+        else:
+            own += W * 4 * l.vdim
+        per_expert = 2 * W * l.ff
+        met += per_expert * l.experts * (1 - (1 - l.top / l.experts) ** B)
+        fixed += own
+        flops += own + l.top * per_expert
+    seen = sum(min(t + 1, attn[0].window) for t in range(M))
+    return {"decode_bytes": {"projections": 2 * (fixed + met + cfg.vocab_size * W),
+                             "attention": sum(B * min(ctx_len, l.window) * l.kv_heads * (l.dim + l.vdim) * 2 for l in attn),
+                             "recurrence": sum(B * l.vdim * (2 * 4 + 3 * 4 + (2 if B > 4 else 4)) for l in rec)},
+            "prefill_flops": {"gemm_tc": 2.0 * M * flops, "attention": sum(l.heads * 2 * (l.dim + l.vdim) * seen for l in attn)},
+            "prefill_bytes": {"recurrence": sum(M * l.vdim * (3 * 4 + 2) for l in rec)}}     # f32 projections in, bf16 result out
+
+
 def layered_work(cfg, model, B, ctx_len, M):
     """Algorithmic bytes of a decode step (B sequences at ctx_len) and flops / bytes of a prefill of M tokens, by kernel class."""
     from paged_infer_b200 import loader as ld
@@ -1153,7 +1201,8 @@ def run_layered_workload(args):
     """`--workload sumosun`: prefill and decode of the layered design at a few sizes, beside a Llama of the same width, depth,
     feed-forward and vocabulary (random weights; bf16 there, int8 weights with f32 activations and KV here).
     `--workload lilosun`: Lilosun beside Sumosun, its closest model, both in bf16.
-    `--workload rubuvik`: Rubuvik beside Lilosun and Sumosun, all in bf16."""
+    `--workload rubuvik`: Rubuvik beside Lilosun and Sumosun, all in bf16.
+    `--workload noresun`: Noresun beside Rubuvik, both in bf16."""
     import torch
     from paged_infer_b200 import api
     from paged_infer_b200.loader import LlamaConfig
@@ -1168,7 +1217,7 @@ def run_layered_workload(args):
     res, launches = {}, ctx.kernel_launches()
     measure = lambda m, work: measure_steps(api, ctx, torch, m, work, ctx_len, batches, M, K, W, (hbm, tflops))
     name = args.workload
-    sizes = {"sumosun": LAYERED_SIZES, "lilosun": LILOSUN_SIZES, "rubuvik": RUBUVIK_SIZES}[name]
+    sizes = {"sumosun": LAYERED_SIZES, "lilosun": LILOSUN_SIZES, "rubuvik": RUBUVIK_SIZES, "noresun": NORESUN_SIZES}[name]
 
     def layered(label, cfg, work):
         m = api.LayeredModel.synthetic(ctx, cfg, seed=1, max_rows=M)
@@ -1177,7 +1226,10 @@ def run_layered_workload(args):
 
     for size, s in sizes.items():
         res[size] = {}
-        if name == "rubuvik":
+        if name == "noresun":
+            layered(name, noresun_config(size), noresun_work)
+            layered("rubuvik", rubuvik_config(s["like"]), rubuvik_work)
+        elif name == "rubuvik":
             layered(name, rubuvik_config(size), rubuvik_work)
             layered("lilosun", lilosun_config(s["like"]), lilosun_work)
             layered("sumosun", layered_config(s["like"], LILOSUN_SIZES[s["like"]]["layers"]), layered_work)
@@ -1209,7 +1261,7 @@ def main():
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="tinyllama_b64_paged", choices=["tinyllama_b64_paged", "llama3_8b_tp", "llama2_70b_tp", "sumosun", "lilosun", "rubuvik"])
+    ap.add_argument("--workload", default="tinyllama_b64_paged", choices=["tinyllama_b64_paged", "llama3_8b_tp", "llama2_70b_tp", "sumosun", "lilosun", "rubuvik", "noresun"])
     ap.add_argument("--no-cpu", action="store_true", help="skip the cpu_baseline leg")
     ap.add_argument("--resident-only", action="store_true",
                     help="for a profiler's launch list: only the resident decode leg (warm-up + timed steps) over a pool filled with "
@@ -1230,7 +1282,7 @@ def main():
     if args.kernel_case:
         run_kernel_case(args)
         return
-    if args.workload in ("sumosun", "lilosun", "rubuvik"):
+    if args.workload in ("sumosun", "lilosun", "rubuvik", "noresun"):
         run_layered_workload(args)
         return
     if args.workload in TP_WORKLOADS:

@@ -163,6 +163,96 @@ def rubuvik_tensors(cfg, seed):
     return t
 
 
+# ---- Noresun ------------------------------------------------------------------------------------------------------------------
+BANDS = {"factor": 6.0, "low": 1.5, "high": 5.0, "original": 160}
+
+
+def sigmoid_attention(heads=6, kv_heads=2, dim=20, vdim=28, window=30, rot=12, base=10000.0, scaling=BANDS, scale=None, kv_from=None, mlp=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5 if scale is None else scale,
+         "mask": {"size": window} if window else None}
+    if rot:
+        m["rot"] = {"dims": rot, "base": base}
+        if scaling:
+            m["rot"]["scaling"] = scaling
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mlp": mlp, "mixer": m}
+
+
+def mingru(width=44, mlp=None):
+    return {"type": "mingru", "mlp": mlp, "mixer": {"width": width}}
+
+
+def relu2_moe(experts=12, top=3, ff=40):
+    return {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff}}
+
+
+def noresun(layers, width=84, vocab=400, eps=1e-5, embed_scale=3.0, alpha=1.7, bigram=(211, 5, 3)):
+    e = {"scale": embed_scale}
+    if bigram:
+        e["bigram"] = dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))
+    return {"architecture": "Noresun", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width, "embedding": e, "postln_alpha": alpha}
+
+
+def noresun_tensors(cfg, seed):
+    """As lilosun_tensors: no sublayer and no token pair writes the channels the routers read."""
+    rng = np.random.default_rng(seed)
+    W, V = cfg["width"], cfg["vocab"]
+    t = {}
+
+    def put(name, shape, std=None, mean=0.0):
+        x = rng.standard_normal(shape) * (1.0 / np.sqrt(shape[-1]) if std is None else std) + mean
+        t[name] = bf16_bits_to_f32(f32_to_bf16_bits(np.asarray(x, np.float32))).reshape(shape)
+
+    def norm_and_gate(l, n):
+        put(f"{l}norm{n}", (W,), 0.2, 1.0)
+        t[f"{l}norm{n}"][:CODE] = 1.25
+        put(f"{l}rg{n}", (W, W), 1.5 / np.sqrt(W))
+        put(f"{l}rg{n}.b", (W,), 0.7, 0.3)
+
+    put("embed", (V, W), 0.5, 0.05)
+    t["embed"][:, :CODE] *= 1.5
+    if cfg["embedding"].get("bigram"):
+        put("bigram", (cfg["embedding"]["bigram"]["buckets"] + 1, W), 1.0)
+        t["bigram"][:, :CODE] = 0
+    for i, e in enumerate(cfg["layers"]):
+        m, l = e["mixer"], f"l{i}."
+        p = l + "mix."
+        norm_and_gate(l, 1)
+        if e["type"] == "mingru":
+            inner = m["width"]
+            for n in ("z", "x", "g"):
+                put(p + n, (inner, W), 1.5 / np.sqrt(W))
+            put(p + "z.b", (inner,), 1.5, -1.5)
+            put(p + "x.b", (inner,), 0.7)
+        else:
+            H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            inner = H * E
+            put(p + "q", (H * D, W), 1.5 / np.sqrt(W))
+            put(p + "q.norm", (H * D,), 0.3, 1.2)
+            put(p + "pb", (H,), 0.7, -1.5)
+            if m.get("kv_from") is None:
+                put(p + "k", (G * D, W), 1.5 / np.sqrt(W))
+                put(p + "k.norm", (G * D,), 0.3, 1.2)
+                put(p + "v", (G * E, W))
+        put(p + "o", (W, inner), 1.0 / np.sqrt(inner))
+        t[p + "o"][:CODE] = 0
+        f = e["mlp"]
+        if f:
+            norm_and_gate(l, 2)
+            p = l + "mlp."
+            n, F = f["router"]["experts"], f["expert"]["ff"]
+            put(p + "router", (n, W), 1.2)
+            t[p + "router"][:, CODE:] = 0
+            put(p + "router.b", (n,), 0.6)
+            for k in range(n):
+                put(f"{p}e{k}.up", (F, W), 1.3 / np.sqrt(W))
+                put(f"{p}e{k}.down", (W, F), 1.0 / np.sqrt(F))
+                t[f"{p}e{k}.down"][:CODE] = 0
+    put("final.norm", (W,), 0.2, 1.0)
+    return t
+
+
 CODE = 16   # leading channels of the embedding that only the routers and norms see change: no sublayer writes them
 
 
@@ -237,7 +327,7 @@ def clear_tokens(cfg, t, margin=0.05):
     """Token ids whose experts are chosen by a clear margin in every layer."""
     r = reference(cfg, t)
     r.forward(np.arange(cfg["vocab"]))
-    ids = np.flatnonzero(r.margin > margin)
+    ids = np.flatnonzero(r.margin > (2 * margin if cfg["architecture"] == "Noresun" else margin))
     assert len(ids) >= 12, len(ids)
     return ids
 
@@ -246,9 +336,9 @@ def draw(cfg, t, n, seed):
     """n random tokens, every choice of an expert clear where they stand."""
     rng, ids, r = np.random.default_rng(seed), clear_tokens(cfg, t), reference(cfg, t)
     toks = rng.choice(ids, n)
-    for _ in range(30):
+    for _ in range(60):
         r.forward(toks)
-        close = np.flatnonzero(r.margin < 0.02)
+        close = np.flatnonzero(r.margin < (0.08 if cfg["architecture"] == "Noresun" else 0.02))   # logits there, scores elsewhere
         if not len(close):
             return toks.tolist()
         toks[close] = rng.choice(ids, len(close))
@@ -261,6 +351,8 @@ def tensors(cfg, seed, rank=5):
         return lilosun_tensors(cfg, seed)
     if cfg["architecture"] == "Rubuvik":
         return rubuvik_tensors(cfg, seed)
+    if cfg["architecture"] == "Noresun":
+        return noresun_tensors(cfg, seed)
     rng = np.random.default_rng(seed)
     W, V = cfg["width"], cfg["vocab"]
     t = {}
