@@ -187,11 +187,11 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) maps_prepare_kernel(const 
 // CTA per row: q and k (which follow one another) each over the root mean square of all their heads, times a weight per channel, then
 // rotated; v as it is.  Groups of four adjacent channels (VEC: sizes are multiples of 4) or pairs, up to kWholeHeld of them per thread
 // in registers, the others are read twice.  Pool rows are padded with zeros up to dp / vp.
-constexpr int kWholeThreads = 256, kWholeHeld = 5;
-template <typename T, bool VEC>
-__global__ void __launch_bounds__(kWholeThreads) maps_prepare_whole_kernel(const PrepareParams p) {
+constexpr int kWholeHeld = 5;
+template <typename T, bool VEC, int THREADS>
+__global__ void __launch_bounds__(THREADS) maps_prepare_whole_kernel(const PrepareParams p) {
   constexpr int G = VEC ? 4 : 2;
-  __shared__ float red[2][kWholeThreads / 32];
+  __shared__ float red[2][THREADS / 32];
   const int row = blockIdx.x, tid = threadIdx.x, half = p.rot_dims >> 1;
   const int gd = (p.dim + G - 1) / G, nq = p.heads * gd, n = nq + (p.x.q_only ? 0 : p.kv_heads * gd);   // groups: of a head, of q, of all
   const int pos = p.row_pos[row], off = pos % p.block_size;
@@ -209,16 +209,16 @@ __global__ void __launch_bounds__(kWholeThreads) maps_prepare_whole_kernel(const
     float v[G];
   };
   auto load = [&](const float* src, int i) {
-    const int vec = i / gd, d = (i - vec * gd) * G;
-    src += (size_t)vec * p.dim + d;
     Group g;
-    if (VEC) {
-      const float4 f = *reinterpret_cast<const float4*>(src);
+    if (VEC) {                            // no group is ragged
+      const float4 f = reinterpret_cast<const float4*>(src)[i];
       g.v[0] = f.x;
       g.v[1] = f.y;
       g.v[G - 2] = f.z;
       g.v[G - 1] = f.w;
     } else {
+      const int vec = i / gd, d = (i - vec * gd) * G;
+      src += (size_t)vec * p.dim + d;
       g.v[0] = src[0];
       g.v[1] = d + 1 < p.dim ? src[1] : 0.f;
     }
@@ -232,19 +232,19 @@ __global__ void __launch_bounds__(kWholeThreads) maps_prepare_whole_kernel(const
   };
   Group w[kWholeHeld];                    // constants: ahead of the dependency wait
 #pragma unroll
-  for (int j = 0; j < kWholeHeld; ++j) w[j] = load(p.x.norm_qk, min(tid + j * kWholeThreads, n - 1));
+  for (int j = 0; j < kWholeHeld; ++j) w[j] = load(p.x.norm_qk, min(tid + j * THREADS, n - 1));
   pi_grid_dependency_wait();
   Group held[kWholeHeld];
   float ss[2] = {0.f, 0.f};
 #pragma unroll
-  for (int j = 0; j < kWholeHeld; ++j) held[j] = load(qkv, min(tid + j * kWholeThreads, n - 1));
+  for (int j = 0; j < kWholeHeld; ++j) held[j] = load(qkv, min(tid + j * THREADS, n - 1));
 #pragma unroll
   for (int j = 0; j < kWholeHeld; ++j) {
-    const int i = tid + j * kWholeThreads;
+    const int i = tid + j * THREADS;
     if (i < nq) ss[0] += square(held[j]);
     else if (i < n) ss[1] += square(held[j]);
   }
-  for (int i = tid + kWholeHeld * kWholeThreads; i < n; i += kWholeThreads) ss[i < nq ? 0 : 1] += square(load(qkv, i));
+  for (int i = tid + kWholeHeld * THREADS; i < n; i += THREADS) ss[i < nq ? 0 : 1] += square(load(qkv, i));
 #pragma unroll
   for (int k = 0; k < 2; ++k) {
     ss[k] = pi_warp_sum(ss[k]);
@@ -255,7 +255,7 @@ __global__ void __launch_bounds__(kWholeThreads) maps_prepare_whole_kernel(const
   T* blk = static_cast<T*>(p.base) + (size_t)pb * p.kv_heads * tile;
   if (mapped) {
     const float* v = qkv + (size_t)(p.heads + p.kv_heads) * p.dim;
-    for (int i = tid; i < p.kv_heads * (p.vp / G); i += kWholeThreads) {
+    for (int i = tid; i < p.kv_heads * (p.vp / G); i += THREADS) {
       const int g = i / (p.vp / G), e = (i - g * (p.vp / G)) * G;
       T* dst = blk + g * tile + (size_t)p.block_size * p.dp + (size_t)off * p.vp + e;
       if (VEC) {
@@ -265,7 +265,7 @@ __global__ void __launch_bounds__(kWholeThreads) maps_prepare_whole_kernel(const
         for (int k = 0; k < G; ++k) dst[k] = pi_from_f32<T>(e + k < p.vdim ? v[(size_t)g * p.vdim + e + k] : 0.f);
       }
     }
-    for (int i = tid; i < p.kv_heads * (p.dp - p.dim); i += kWholeThreads) {
+    for (int i = tid; i < p.kv_heads * (p.dp - p.dim); i += THREADS) {
       const int g = i / (p.dp - p.dim), d = p.dim + i - g * (p.dp - p.dim);
       blk[g * tile + (size_t)off * p.dp + d] = pi_from_f32<T>(0.f);
     }
@@ -275,7 +275,7 @@ __global__ void __launch_bounds__(kWholeThreads) maps_prepare_whole_kernel(const
 #pragma unroll
   for (int k = 0; k < 2; ++k) {
 #pragma unroll
-    for (int j = 0; j < kWholeThreads / 32; ++j) inv[k] += red[k][j];
+    for (int j = 0; j < THREADS / 32; ++j) inv[k] += red[k][j];
     inv[k] = 1.0f / sqrtf(inv[k] / (float)((k ? p.kv_heads : p.heads) * p.dim) + p.eps);
   }
   auto finish = [&](int i, Group g, const Group& w) {
@@ -312,8 +312,8 @@ __global__ void __launch_bounds__(kWholeThreads) maps_prepare_whole_kernel(const
   };
 #pragma unroll
   for (int j = 0; j < kWholeHeld; ++j)
-    if (tid + j * kWholeThreads < n) finish(tid + j * kWholeThreads, held[j], w[j]);
-  for (int i = tid + kWholeHeld * kWholeThreads; i < n; i += kWholeThreads) finish(i, load(qkv, i), load(p.x.norm_qk, i));
+    if (tid + j * THREADS < n) finish(tid + j * THREADS, held[j], w[j]);
+  for (int i = tid + kWholeHeld * THREADS; i < n; i += THREADS) finish(i, load(qkv, i), load(p.x.norm_qk, i));
 }
 
 // One CTA of 4 warps per (row, head): the warps take every fourth key and merge; lanes hold the channels.  f32
@@ -413,9 +413,14 @@ pi_status pi_launch_maps_prepare(pi_ctx* ctx, const pi_maps_attention& a, const 
   const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.dim <= 256 && a.vdim <= 256 && stride % 4 == 0 && x.mix.stride % 4 == 0;
   if (x.norm_qk) {
     PI_REQUIRE(ctx, a.maps == 1 && !x.bias && !x.unit_qk && !x.q_temp && !x.mix.first, "norms over whole projections stand alone");
-    auto k = kv.kind == PI_BF16 ? (vec ? maps_prepare_whole_kernel<__nv_bfloat16, true> : maps_prepare_whole_kernel<__nv_bfloat16, false>)
-                                : (vec ? maps_prepare_whole_kernel<float, true> : maps_prepare_whole_kernel<float, false>);
-    PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(b.rows), dim3(kWholeThreads), 0, 1, p));
+    const int groups = (a.heads + (x.q_only ? 0 : a.kv_heads)) * ((a.dim + (vec ? 3 : 1)) / (vec ? 4 : 2)), threads = groups <= 128 * kWholeHeld && b.rows > ctx->sm_count ? 128 : 256;
+    auto pick = [&](auto few, auto many) { return threads == 128 ? few : many; };
+    void (*k)(const PrepareParams);
+    if (kv.kind == PI_BF16) k = vec ? pick(maps_prepare_whole_kernel<__nv_bfloat16, true, 128>, maps_prepare_whole_kernel<__nv_bfloat16, true, 256>)
+                                    : pick(maps_prepare_whole_kernel<__nv_bfloat16, false, 128>, maps_prepare_whole_kernel<__nv_bfloat16, false, 256>);
+    else k = vec ? pick(maps_prepare_whole_kernel<float, true, 128>, maps_prepare_whole_kernel<float, true, 256>)
+                 : pick(maps_prepare_whole_kernel<float, false, 128>, maps_prepare_whole_kernel<float, false, 256>);
+    PI_LAUNCH_OK(ctx, pi_launch_dep(ctx, k, dim3(b.rows), dim3(threads), 0, 1, p));
     return PI_OK;
   }
   PI_REQUIRE(ctx, !x.q_only, "keys of another layer go with norms over whole projections");
