@@ -555,21 +555,21 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) maps_tile_kernel(const TcP
         }
     } else {
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      float tm = -INFINITY;
+      for (int h = 0; h < 2; ++h) {
+        float tm = -INFINITY;
 #pragma unroll
-      for (int j = 0; j < kTileKeys / 8; ++j)
+        for (int j = 0; j < kTileKeys / 8; ++j)
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const int t = t0 + j * 8 + (lane & 3) * 2 + i;
-          float& v = s[j][2 * h + i];
-          v = (inside || (t <= tpos[h] && t > tpos[h] - win && t < hi)) ? fmaf(slope[h], (float)(t - tpos[h]), v * sc) : -INFINITY;
-          tm = fmaxf(tm, v);
-        }
-      mx[h] = new_max(mx[h], quad_max(tm), keep[h]);
-      ref[h] = mx[h] == -INFINITY ? 0.f : mx[h];
-      l[h] *= keep[h];
-    }
+          for (int i = 0; i < 2; ++i) {
+            const int t = t0 + j * 8 + (lane & 3) * 2 + i;
+            float& v = s[j][2 * h + i];
+            v = (inside || (t <= tpos[h] && t > tpos[h] - win && t < hi)) ? fmaf(slope[h], (float)(t - tpos[h]), v * sc) : -INFINITY;
+            tm = fmaxf(tm, v);
+          }
+        mx[h] = new_max(mx[h], quad_max(tm), keep[h]);
+        ref[h] = mx[h] == -INFINITY ? 0.f : mx[h];
+        l[h] *= keep[h];
+      }
     }
     if (!SELF && __any_sync(0xffffffffu, keep[0] != 1.f || keep[1] != 1.f)) {
 #pragma unroll
